@@ -76,26 +76,14 @@ def build_serving(a):
     if world > 1:
         from .serving.split import build_split_serving
         return build_split_serving(a, world)
-    from .config import spec_from_snapshot, spec_by_name, NAMED_SPECS, QuantSpec
-    from .engine.engine import Engine
     from .engine.kv import PagePool
-    from .models.weights import DeviceWeights
-    from .ref.model import init_weights
+    from .engine.registry import build_engine, load_weights, model_spec
     from .serving.prefix import PrefixCache
     from .serving.runner import EngineRunner, attach_pool
     from .serving.scheduler import NgramDrafter, Scheduler
-    spec = spec_by_name(a.model) if a.model in NAMED_SPECS else spec_from_snapshot(a.model)
+    spec = model_spec(a.model, layers=getattr(a, "layers", 0), dtype=getattr(a, "dtype", "bfloat16"))
     dev = torch.device("cuda", a.device)
-    layers = getattr(a, "layers", 0)
-    if layers:
-        spec = spec.replace(n_layers=layers)
-    if os.path.isdir(a.model) and spec.attn.kind == "gqa":
-        from .loader.checkpoint import load_device_weights
-        weights = load_device_weights(a.model, spec, dev)      # tensors in their stored formats, no repacking
-    elif spec.name == "tiny":
-        weights = DeviceWeights.from_masters(spec, init_weights(spec, 0), dev)
-    else:
-        weights = DeviceWeights.random(spec, dev, seed=1)      # named shapes without a snapshot: synthetic weights
+    weights = load_weights(a.model, spec, dev)
     n_pages = a.pool_tokens // 64 if a.pool_tokens else 4096
     if getattr(a, "gpu_occupancy_percent", 0):
         # pool sized by the start-up capacity policy from the memory measured now (the weights are already resident); a pool that was
@@ -107,7 +95,7 @@ def build_serving(a):
                             model_max_context=spec.max_context, weights_loaded=True)
         print(f"[serve] capacity: {cap.describe()}", file=sys.stderr)
         n_pages = cap.pool_pages
-    eng = Engine(weights, n_pages=n_pages, max_seqs=a.max_sequences, max_pages_per_seq=min(n_pages, a.max_context // 64 + 1))
+    eng = build_engine(spec, weights, n_pages=n_pages, max_seqs=a.max_sequences, max_pages_per_seq=min(n_pages, min(a.max_context, spec.max_context) // 64 + 1))
     pool = PagePool(n_pages)
     runner = attach_pool(EngineRunner(eng, max_rows=a.prefill_batch_tokens), pool)
     host = None
@@ -398,6 +386,12 @@ def cmd_golden(a) -> int:
     return 0 if all(r["rel_l2"] < 0.25 for r in out) else 1
 
 
+def cmd_trace(a) -> int:
+    """Replay given token ids step by step and write the logits of chosen positions (no sampling)."""
+    from .serving.trace import run
+    return run(a)
+
+
 def cmd_expertd(a) -> int:
     """Host-path expert service: answers framed expert waves over TCP with the synthetic executor (protocol bring-up
     and multi-host tests); the in-node data path uses peer memory and needs no daemon."""
@@ -614,6 +608,7 @@ def main(argv=None) -> int:
     _gateway_args(p)
     p.add_argument("--draft-limit", type=int, default=3); p.add_argument("--api-key-file"); p.add_argument("--model-id")
     p.add_argument("--layers", type=int, default=0, help="debug: run only the first N layers of a named shape")
+    p.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="float32: weights, activations and cache in fp32 (latent-attention stacks only)")
     p.add_argument("--n-micro", type=int, default=0, help="multi-GPU: micro-batches the attention ranks keep in flight (0 = the layout's default)")
     p.add_argument("--vision", default="auto", help="auto (tower of the snapshot, if it has one) | off | random[:DEPTH]")
     p.add_argument("--gpu-occupancy-percent", type=int, default=0,
@@ -653,6 +648,9 @@ def main(argv=None) -> int:
     p.add_argument("--model", "--snapshot", dest="model", default="tiny"); p.add_argument("--windows", type=int, default=8)
     p.add_argument("--window-tokens", type=int, default=64); p.set_defaults(fn=cmd_golden)
     p = sub.add_parser("expertd"); p.add_argument("--listen", default="127.0.0.1:7000"); p.add_argument("--rank", type=int, default=0); p.set_defaults(fn=cmd_expertd)
+    p = sub.add_parser("trace", help="replay given token ids step by step (JSON lines on standard input) and write logits")
+    from .serving.trace import add_arguments
+    add_arguments(p); p.set_defaults(fn=cmd_trace)
     p = sub.add_parser("bench"); p.add_argument("rest", nargs=argparse.REMAINDER); p.set_defaults(fn=cmd_bench)
     a = ap.parse_args(argv)
     return a.fn(a)

@@ -17,7 +17,7 @@ from typing import Optional
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    kind: str = "gqa"              # "gqa" | "mla"
+    kind: str = "gqa"              # "gqa" | "mla" | "latent" (latent attention without positions; per layer, see BlockSpec)
     n_heads: int = 8
     n_kv_heads: int = 2
     head_dim: int = 32
@@ -52,6 +52,14 @@ class AttentionSpec:
     linear_k_heads: int = 2
     linear_v_heads: int = 4
     linear_per_channel: bool = False
+    # Latent attention without a rotated part (kind "latent"): head_dim, v_head_dim and kv_lora_rank as above, `scale` multiplies the scores
+    # (0 = head_dim ** -0.5), `out_gate` multiplies each head's output by a sigmoid of the layer's input.
+    scale: float = 0.0
+    out_gate: bool = False
+
+    @property
+    def softmax_scale(self) -> float:
+        return self.scale or self.head_dim ** -0.5
 
     @property
     def q_dim(self) -> int:
@@ -64,6 +72,8 @@ class AttentionSpec:
         """Cached elements per token per layer."""
         if self.kind == "mla":
             return self.kv_lora_rank + self.qk_rope_head_dim
+        if self.kind == "latent":
+            return self.kv_lora_rank
         return 2 * self.n_kv_heads * self.head_dim
 
 
@@ -83,6 +93,8 @@ class MoESpec:
     first_dense: int = 0            # leading dense layers
     dense_intermediate: int = 0
     swiglu_limit: float = 0.0       # clamp on gate/up (0 = off)
+    activation: str = "swiglu"      # "swiglu" (gate and up projections) | "relu2" (up projection only, squared ReLU)
+    group_score: str = "top2"       # what ranks a group of experts: the sum of its two best scores, or its best one ("max")
 
     @property
     def shared_inter(self) -> int:
@@ -96,6 +108,22 @@ class QuantSpec:
     dense: str = "bf16"             # bf16 | fp8_block128 | fp8_block32 | nvfp4
     kv: str = "bf16"                # bf16 | fp8
     exl3_bits: int = 4
+
+
+@dataclass(frozen=True)
+class BlockSpec:
+    """One layer of a stack whose layers differ: its attention and its feed-forward (None = the layer has none)."""
+    attn: AttentionSpec = field(default_factory=lambda: AttentionSpec(kind="latent"))
+    moe: Optional[MoESpec] = None
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers [start, stop) run `times` times in a row with the same weights and a cache of their own per pass; each pass opens with a
+    projection of [x; embedding output] and a learned vector of the pass."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass(frozen=True)
@@ -123,6 +151,19 @@ class ModelSpec:
     init_std: float = 0.02
     tie_embeddings: bool = False
     max_context: int = 1 << 20
+    # Stacks of unequal layers (`blocks` non-empty; `attn` / `moe` above then describe the first layer of their kind): parallel layers
+    # (one norm, attention and feed-forward read it, both scaled per channel and added to an fp32 residual), Dynamic Tanh for a norm.
+    blocks: tuple = ()
+    loop: Optional[LoopSpec] = None
+    learned_positions: int = 0      # rows of the learned position table (0 = none); also the longest context
+
+    def layer_runs(self) -> list:
+        """[(layer, pass index where a pass of the loop opens with this run, else None)] in the order the layers run."""
+        lp, n = self.loop, self.n_layers
+        if lp is None:
+            return [(i, None) for i in range(n)]
+        return ([(i, None) for i in range(lp.start)] + [(i, t if i == lp.start else None) for t in range(lp.times) for i in range(lp.start, lp.stop)] +
+                [(i, None) for i in range(lp.stop, n)])
 
     def replace(self, **kw) -> "ModelSpec":
         return dataclasses.replace(self, **kw)
@@ -169,8 +210,11 @@ class ModelSpec:
     def expert_params(self) -> int:
         return 3 * self.hidden * self.moe.intermediate
 
-    def attn_params(self) -> int:
-        a, h = self.attn, self.hidden
+    def attn_params(self, attn: Optional[AttentionSpec] = None) -> int:
+        a, h = attn or self.attn, self.hidden
+        if a.kind == "latent":
+            return (h * (a.n_heads * a.head_dim + a.kv_lora_rank + (a.n_heads if a.out_gate else 0)) +
+                    a.n_heads * (a.head_dim + a.v_head_dim) * a.kv_lora_rank + a.n_heads * a.v_head_dim * h)
         if a.kind == "mla":
             qk = a.qk_nope_head_dim + a.qk_rope_head_dim
             q = h * a.q_lora_rank + a.q_lora_rank * a.n_heads * qk if a.q_lora_rank else h * a.n_heads * qk
@@ -179,11 +223,18 @@ class ModelSpec:
         return h * (a.n_heads + 2 * a.n_kv_heads) * a.head_dim + a.n_heads * a.head_dim * h
 
     def bits(self, fmt: str) -> float:
-        return {"bf16": 16.0, "fp8_block128": 8.0 + 32.0 / (128 * 128), "fp8_block32": 8.0 + 8.0 / (32 * 32),
+        return {"f32": 32.0, "bf16": 16.0, "fp8_block128": 8.0 + 32.0 / (128 * 128), "fp8_block32": 8.0 + 8.0 / (32 * 32),
                 "mxfp4": 4.25, "nvfp4": 4.5, "exl3": float(self.quant.exl3_bits)}[fmt]
 
     def weight_bytes(self) -> dict:
         """Bytes per category for the whole model (planner input)."""
+        if self.blocks:
+            eb, db = self.bits(self.quant.experts) / 8, self.bits(self.quant.dense) / 8
+            ffs = [b.moe for b in self.blocks if b.moe is not None]
+            return {"routed_experts": sum((2 if m.activation == "relu2" else 3) * self.hidden * m.intermediate * m.n_experts for m in ffs) * eb,
+                    "shared_experts": 0.0, "dense_ffn": 0.0, "attention": sum(self.attn_params(b.attn) for b in self.blocks) * db,
+                    "router": sum(m.n_experts for m in ffs) * self.hidden * db,
+                    "embed_head": (2 * self.vocab + self.learned_positions) * self.hidden * 2 + (2 * self.hidden ** 2 * db if self.loop else 0)}
         moe_layers = self.n_layers - self.moe.first_dense
         eb = self.bits(self.quant.experts) / 8
         db = self.bits(self.quant.dense) / 8
@@ -197,7 +248,9 @@ class ModelSpec:
                 "attention": attn, "router": router, "embed_head": embed}
 
     def kv_bytes_per_token(self) -> float:
-        per = 1.0 if self.quant.kv == "fp8" else 2.0
+        per = {"fp8": 1.0, "f32": 4.0}.get(self.quant.kv, 2.0)
+        if self.blocks:             # one row width for every layer run (the widest latent, in whole 64-element chunks)
+            return len(self.layer_runs()) * max(-(-b.attn.kv_token_elems // 64) * 64 for b in self.blocks) * per
         return self.n_layers * self.attn.kv_token_elems * per
 
 
@@ -267,6 +320,19 @@ def hybrid_gdn_spec(n_layers: int = 48, per_channel: bool = False) -> ModelSpec:
         quant=QuantSpec(experts="nvfp4", dense="bf16", kv="bf16"))
 
 
+def bedovik_spec(n_layers: int = 8, heads: int = 32, hidden: int = 4096, rank: int = 512, experts: int = 64, ff: int = 1536, loop_times: int = 2) -> ModelSpec:
+    """Bedovik at the size of a real model's layers (synthetic weights): parallel latent-attention layers, gated and plain ones in turn,
+    squared-ReLU experts behind group-limited softmax routing, the middle half of the stack looped."""
+    moe = MoESpec(n_experts=experts, top_k=8, intermediate=ff, n_shared=0, scoring="softmax", normalize=True, route_scale=2.5, n_group=8, topk_group=4,
+                  activation="relu2", group_score="max")
+    attn = AttentionSpec(kind="latent", n_heads=heads, n_kv_heads=heads, head_dim=128, v_head_dim=128, kv_lora_rank=rank, scale=128 ** -0.5)
+    blocks = tuple(BlockSpec(dataclasses.replace(attn, out_gate=i % 2 == 0), moe) for i in range(n_layers))
+    lo, hi = n_layers // 4, n_layers - n_layers // 4
+    return ModelSpec(name="bedovik-shape", family="bedovik", vocab=65536, hidden=hidden, n_layers=n_layers, rms_eps=1e-6, attn=blocks[0].attn, moe=moe,
+                     quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=blocks,
+                     loop=LoopSpec(lo, hi, loop_times) if loop_times > 1 and hi > lo else None, learned_positions=65536, max_context=65536)
+
+
 NAMED_SPECS = {
     "tiny": tiny_spec,
     "hybrid-gdn": hybrid_gdn_spec,
@@ -274,6 +340,7 @@ NAMED_SPECS = {
     "deepseek-v3": deepseek_v3_spec,
     "deepseek-v32": deepseek_v32_spec,
     "qwen3-235b": qwen3_235b_spec,
+    "bedovik": bedovik_spec,
     "ep-microbench": ep_microbench_spec,
 }
 
@@ -299,6 +366,7 @@ FAMILY_BY_ARCH = {
     "MiMoV2FlashForCausalLM": "mimo_v2",
     "MixtralForCausalLM": "mixtral",
     "Qwen3NextForCausalLM": "hybrid_linear",
+    "Bedovik": "bedovik",
 }
 
 
@@ -320,16 +388,50 @@ def detect_quant(cfg: dict) -> QuantSpec:
     return QuantSpec()
 
 
+def _bedovik_config(cfg: dict) -> ModelSpec:
+    """`config.json` of the Bedovik design: every layer names its mixer and its feed-forward with their sizes."""
+    blocks = []
+    for i, layer in enumerate(cfg["layers"]):
+        if layer["type"] not in ("latent_attention", "latent_attention_2"):
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        m = layer["mixer"]
+        attn = AttentionSpec(kind="latent", n_heads=int(m["heads"]), n_kv_heads=int(m["heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]),
+                             kv_lora_rank=int(m["kv_rank"]), scale=float(m["scale"]), out_gate=layer["type"] == "latent_attention")
+        mlp, moe = layer.get("mlp"), None
+        if mlp is not None:
+            if mlp.get("kind", "moe") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            r = mlp["router"]
+            groups = r.get("groups") or {"count": 1, "keep": 1}
+            moe = MoESpec(n_experts=int(r["experts"]), top_k=int(r["top"]), intermediate=int(mlp["expert"]["ff"]), n_shared=0, scoring="softmax",
+                          normalize=True, route_scale=float(r.get("scale", 1.0)), n_group=int(groups["count"]), topk_group=int(groups["keep"]),
+                          activation="relu2", group_score="max")
+            if moe.n_experts % moe.n_group or not 1 <= moe.topk_group <= moe.n_group or moe.top_k > moe.n_experts // moe.n_group * moe.topk_group:
+                raise ValueError(f"layer {i}: {moe.n_experts} experts in {moe.n_group} groups, {moe.topk_group} kept, top {moe.top_k}: not a routing")
+        blocks.append(BlockSpec(attn, moe))
+    loop = None
+    if cfg.get("loop"):
+        loop = LoopSpec(int(cfg["loop"]["start"]), int(cfg["loop"]["stop"]), int(cfg["loop"]["times"]))
+        if not (0 <= loop.start < loop.stop <= len(blocks) and loop.times >= 1):
+            raise ValueError(f"loop {cfg['loop']} does not fit {len(blocks)} layers")
+    n_pos = int(cfg["max_positions"])
+    return ModelSpec(name="bedovik", family="bedovik", vocab=int(cfg["vocab"]), hidden=int(cfg["width"]), n_layers=len(blocks),
+                     rms_eps=float(cfg["norm"]["eps"]), attn=blocks[0].attn, moe=next((b.moe for b in blocks if b.moe is not None), MoESpec(n_experts=0, n_shared=0)),
+                     quant=QuantSpec(), blocks=tuple(blocks), loop=loop, learned_positions=n_pos, max_context=n_pos)
+
+
 def from_hf_config(cfg: dict | str | Path) -> ModelSpec:
     """Build a ModelSpec from a Hugging Face `config.json` (dict or path)."""
     if not isinstance(cfg, dict):
         p = Path(cfg)
         p = p / "config.json" if p.is_dir() else p
         cfg = json.loads(p.read_text())
-    archs = cfg.get("architectures") or ["?"]
+    archs = cfg.get("architectures") or [cfg.get("architecture", "?")]
     family = FAMILY_BY_ARCH.get(archs[0])
     if family is None:
         raise ValueError(f"unsupported architecture {archs[0]!r} (supported: {sorted(FAMILY_BY_ARCH)})")
+    if family == "bedovik":
+        return _bedovik_config(cfg)
     hidden = cfg["hidden_size"]
     heads = cfg["num_attention_heads"]
     if "kv_lora_rank" in cfg:
@@ -396,6 +498,11 @@ def spec_from_json(d: dict) -> ModelSpec:
     d = dict(d)
     if "engram_layers" in d:
         d["engram_layers"] = tuple(d["engram_layers"])
+    if d.get("blocks"):
+        d["blocks"] = tuple(BlockSpec(AttentionSpec(**b["attn"]), MoESpec(**b["moe"]) if b["moe"] else None) for b in d["blocks"])
+    d["blocks"] = tuple(d.get("blocks") or ())
+    if d.get("loop"):
+        d["loop"] = LoopSpec(**d["loop"])
     return ModelSpec(attn=AttentionSpec(**d.pop("attn")), moe=MoESpec(**d.pop("moe")), quant=QuantSpec(**d.pop("quant")), **d)
 
 

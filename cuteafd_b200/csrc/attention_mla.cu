@@ -38,10 +38,12 @@ struct MlaArgs {
   const CUtensorMap* kv_map;    // 2-D (as 3-D): {576, slots, 1}, box {64, 32, 1}, 128-byte swizzle
   const int* page_table; const int* kv_len; const int* q_start; const int* q_len;
   bf16* out;                // [Hl, T, 512] head-major
+  const float* gate;        // [T, Hl] factor of each head's output, or null
   float* part_o;            // [splits, T, Hl, 512]
   float* part_ml;           // [splits, T, Hl, 2]
   int* status;
   int Hl, max_pages, n_splits, max_q_tiles, T;
+  int ldt;                  // rows between two heads of the head-major buffers (>= T)
   float scale;
 };
 
@@ -63,26 +65,42 @@ __device__ __forceinline__ void mla_tmem_st_x16(uint32_t addr, const uint32_t* r
                  "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]) : "memory");
 }
 
-#define QT_CH 6                             // Q chunks 0..5 live in tensor memory (192 columns), chunks 6..8 in shared memory
-#define NST 2                               // latent tile stages
-#define SQ_BYTES ((NCH - QT_CH) * 16384)    // 3 chunks x [128 rows x 128 B]
 #define SK_CHUNK (MKEYS * 128)              // one 64-wide chunk of a tile: [64 keys x 128 B]
-#define SK_STAGE (NCH * SK_CHUNK)           // 9 chunks
 #define SP_BYTES (128 * MKEYS * 2)          // [128 rows x 64 keys] bf16, core-matrix layout
-#define MLA_SMEM (SQ_BYTES + NST * SK_STAGE + SP_BYTES + 128)
 
-__global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant__ MlaArgs a) {
+// Geometry of one instantiation: NC 64-wide chunks of the score dimension, the first NL of them the latent (= the value); NC = NL + 1
+// carries a rotated chunk behind the latent (DeepSeek-V3: 9 / 8), NC = NL is latent attention without positions (any rank up to 512,
+// padded to whole chunks).  Up to 256 value columns per CTA: ranks above that split the values over two CTAs.
+template <int NC, int NL>
+struct MlaGeo {
+  static constexpr int QT = NC < 6 ? NC : 6;                    // query chunks in tensor memory, the rest in shared memory
+  static constexpr int VCH = NL <= 4 ? NL : (NL + 1) / 2;       // value chunks of the first CTA
+  static constexpr int NVH = NL <= 4 ? 1 : 2;
+  static constexpr int STAGE = NC * SK_CHUNK;
+  static constexpr int NST_ = NC >= 8 ? 2 : (NC >= 6 ? 3 : 4);
+  static constexpr int SQ = (NC - QT) * 16384;
+  static constexpr int SMEM = SQ + NST_ * STAGE + SP_BYTES + 128;
+  static constexpr int O_COL = 64, Q_COL = 64 + VCH * 64, COLS = Q_COL + 32 * QT;
+  static constexpr int TMEM = COLS <= 256 ? 256 : 512;
+  static constexpr int OCC = TMEM == 256 && SMEM <= 110 * 1024 ? 2 : 1;
+  static_assert(COLS <= 512 && SMEM <= 227 * 1024, "latent attention tile does not fit");
+};
+
+template <int NC, int NL>
+__global__ void __launch_bounds__(192, MlaGeo<NC, NL>::OCC) mla_attn_kernel(const __grid_constant__ MlaArgs a) {
+  using G = MlaGeo<NC, NL>;
+  constexpr int NST_ = G::NST_, LAT = NL * 64;
   pdl_launch(); pdl_wait();
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t* sQ = smem;
-  uint8_t* sK = smem + SQ_BYTES;
-  uint8_t* sP = sK + NST * SK_STAGE;
+  uint8_t* sK = smem + G::SQ;
+  uint8_t* sP = sK + NST_ * G::STAGE;
   uint64_t* bars = (uint64_t*)(sP + SP_BYTES);
-  uint64_t* k_full = bars; uint64_t* k_empty = bars + NST;
-  uint64_t& s_full = bars[2 * NST]; uint64_t& s_free = bars[2 * NST + 1];
-  uint64_t& p_full = bars[2 * NST + 2]; uint64_t& o_done = bars[2 * NST + 3];
-  uint32_t& tmem_slot = *(uint32_t*)(bars + 2 * NST + 4);
-  int& abort_flag = *(int*)(bars + 2 * NST + 5);
+  uint64_t* k_full = bars; uint64_t* k_empty = bars + NST_;
+  uint64_t& s_full = bars[2 * NST_]; uint64_t& s_free = bars[2 * NST_ + 1];
+  uint64_t& p_full = bars[2 * NST_ + 2]; uint64_t& o_done = bars[2 * NST_ + 3];
+  uint32_t& tmem_slot = *(uint32_t*)(bars + 2 * NST_ + 4);
+  int& abort_flag = *(int*)(bars + 2 * NST_ + 5);
   if (smem_u32(smem) & 1023) { if (threadIdx.x == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0xA12); return; }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
 
@@ -101,25 +119,27 @@ __global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant_
   const int per = (last_tile + a.n_splits - 1) / a.n_splits;
   const int t0 = split * per, t1 = min(last_tile, t0 + per);
   const int n_tiles = max(0, t1 - t0);
+  const int nv = vh == 0 ? G::VCH : NL - G::VCH;                      // 64-wide value chunks of this CTA
 
   if (tid == 0) {
-    for (int s = 0; s < NST; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
+    for (int s = 0; s < NST_; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
     mbar_init(&s_full, 1); mbar_init(&s_free, 128);
     mbar_init(&p_full, 128); mbar_init(&o_done, 1);
     abort_flag = 0;
     fence_barrier_init();
   }
-  if (warp == 1) { tmem_alloc(&tmem_slot, 512); tmem_relinquish(); }
-  // Q rows: the 64-wide chunks 6, 7 (q_lat) and 8 (q_rope) become swizzled K-major tiles in shared memory ...
-  for (int i = tid; i < 128 * 24; i += 192) {
-    const int r = i / 24, c = 8 * QT_CH + i % 24;        // 16-byte chunk c (8 elements) of row r
+  if (warp == 1) { tmem_alloc(&tmem_slot, G::TMEM); tmem_relinquish(); }
+  // Q rows: the 64-wide chunks from 6 on (the rest of q_lat, then q_rope) become swizzled K-major tiles in shared memory ...
+  constexpr int QS16 = NC > G::QT ? (NC - G::QT) * 8 : 1;        // their 16-byte chunks per row
+  for (int i = tid; NC > G::QT && i < 128 * QS16; i += 192) {
+    const int r = i / QS16, c = 8 * G::QT + i % QS16;    // 16-byte chunk c (8 elements) of row r
     uint4 v = make_uint4(0, 0, 0, 0);
     if (r < R) {
       const int t = row_base + r / a.Hl, h = r % a.Hl;
-      v = (c < 64) ? *(const uint4*)(a.q_lat + ((size_t)h * a.T + t) * DV + c * 8)
-                   : *(const uint4*)(a.q_rope + ((size_t)t * a.Hl + h) * 64 + (c - 64) * 8);
+      v = (NC == NL || c < NL * 8) ? *(const uint4*)(a.q_lat + ((size_t)h * a.ldt + t) * LAT + c * 8)
+                                   : *(const uint4*)(a.q_rope + ((size_t)t * a.Hl + h) * 64 + (c - NL * 8) * 8);
     }
-    *(uint4*)(sQ + ((c >> 3) - QT_CH) * 16384 + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+    *(uint4*)(sQ + ((c >> 3) - G::QT) * 16384 + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
   }
   fence_proxy_async_smem();
   tc_fence_before();
@@ -127,16 +147,16 @@ __global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant_
   tc_fence_after();
   const uint32_t tmem = tmem_slot;
   volatile int* abortp = &abort_flag;
-  const uint32_t S_COL = 0, O_COL = 64, QT_COL = 320;
-  // ... and chunks 0..5 go to tensor memory (row = lane, two elements per 32-bit column), where the score MMAs
+  const uint32_t S_COL = 0, O_COL = G::O_COL, QT_COL = G::Q_COL;
+  // ... and chunks 0..5 (all of them up to rank 384) go to tensor memory (row = lane, two elements per 32-bit column), where the score MMAs
   // read them as the A operand without touching shared memory; that leaves room there for two 64-key stages, and Q is
   // the same for every tile.
   if (warp >= 2) {
     const int r = (warp & 3) * 32 + lane;
     const uint32_t dst = tmem + ((uint32_t)((warp & 3) * 32) << 16) + QT_COL;
-    const bf16* src = a.q_lat + ((size_t)((r < R ? r : 0) % a.Hl) * a.T + row_base + (r < R ? r : 0) / a.Hl) * DV;
+    const bf16* src = a.q_lat + ((size_t)((r < R ? r : 0) % a.Hl) * a.ldt + row_base + (r < R ? r : 0) / a.Hl) * LAT;
 #pragma unroll 1
-    for (int g = 0; g < QT_CH * 2; ++g) {                // 16 columns = 32 elements per store
+    for (int g = 0; g < G::QT * 2; ++g) {                // 16 columns = 32 elements per store
       uint32_t w[16];
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
@@ -154,21 +174,21 @@ __global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant_
   if (warp == 0) {
     // ------------------------------------------------------------------ latent tile producer
     for (int i = 0; i < n_tiles && !*abortp; ++i) {
-      const int s = i % NST;
-      if (!mbar_wait_bounded(&k_empty[s], ((i / NST) & 1) ^ 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); break; }
+      const int s = i % NST_;
+      if (!mbar_wait_bounded(&k_empty[s], ((i / NST_) & 1) ^ 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); break; }
       if (lane == 0) {
         const int key0 = (t0 + i) * MKEYS;
         const int page = a.page_table[(size_t)seq * a.max_pages + key0 / MPAGE];
         const int slot0 = page * MPAGE + key0 % MPAGE;
-        mbar_expect_tx(&k_full[s], SK_STAGE);
+        mbar_expect_tx(&k_full[s], G::STAGE);
 #pragma unroll
-        for (int c = 0; c < NCH; ++c) tma_load_3d(sK + s * SK_STAGE + c * SK_CHUNK, a.kv_map, &k_full[s], c * 64, slot0, 0);
+        for (int c = 0; c < NC; ++c) tma_load_3d(sK + s * G::STAGE + c * SK_CHUNK, a.kv_map, &k_full[s], c * 64, slot0, 0);
       }
       __syncwarp();
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
-    const uint32_t id_s = mla_idesc(MKEYS, 0), id_o = mla_idesc(256, 1);
+    const uint32_t id_s = mla_idesc(MKEYS, 0), id_o = mla_idesc(nv * 64, 1);
     // One thread issues everything.  It polls two conditions and serves whichever is ready: "the latent tile qk has
     // landed and the score buffer is free" (issue its scores) and "the probabilities of tile pv are in shared memory"
     // (issue its PV product, which also releases the tile's stage to the producer).  The 36 score MMAs of a tile
@@ -183,8 +203,8 @@ __global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant_
       auto try_pv = [&]() -> bool {
         if (pv >= qk || !mbar_test(&p_full, pv & 1)) return false;
         tc_fence_after();
-        const int s = pv % NST;
-        const uint32_t v0 = smem_u32(sK + s * SK_STAGE) + (4 * vh) * SK_CHUNK;
+        const int s = pv % NST_;
+        const uint32_t v0 = smem_u32(sK + s * G::STAGE) + (G::VCH * vh) * SK_CHUNK;
 #pragma unroll
         for (int k = 0; k < MKEYS / 16; ++k)       // 16 keys per MMA: two 8-key groups = 2048 B along K
           tc_mma_f16(tmem + O_COL, mla_desc_k_plain(smem_u32(sP) + k * 256, 128, MKEYS * 16), mla_desc_mn_sw128(v0 + k * 2048, SK_CHUNK, 1024), id_o,
@@ -196,21 +216,21 @@ __global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant_
       };
       while (pv < n_tiles) {
         bool did = try_pv();
-        if (qk < n_tiles && (qk == 0 || mbar_test(&s_free, (qk - 1) & 1)) && mbar_test(&k_full[qk % NST], (qk / NST) & 1)) {
+        if (qk < n_tiles && (qk == 0 || mbar_test(&s_free, (qk - 1) & 1)) && mbar_test(&k_full[qk % NST_], (qk / NST_) & 1)) {
           tc_fence_after();
-          const uint32_t k0 = smem_u32(sK + (qk % NST) * SK_STAGE), d = tmem + S_COL;
+          const uint32_t k0 = smem_u32(sK + (qk % NST_) * G::STAGE), d = tmem + S_COL;
 #pragma unroll 1
-          for (int c = 0; c < NCH; ++c) {
-            if (c < QT_CH) {
+          for (int c = 0; c < NC; ++c) {
+            if (c < G::QT) {
 #pragma unroll
               for (int k = 0; k < 4; ++k)
                 tc_mma_f16_ta(d, tmem + QT_COL + c * 32 + k * 8, mla_desc_k_sw128(k0 + c * SK_CHUNK) + 2 * k, id_s, (c | k) ? 1u : 0u);
             } else {
 #pragma unroll
               for (int k = 0; k < 4; ++k)
-                tc_mma_f16(d, mla_desc_k_sw128(smem_u32(sQ) + (c - QT_CH) * 16384) + 2 * k, mla_desc_k_sw128(k0 + c * SK_CHUNK) + 2 * k, id_s, 1u);
+                tc_mma_f16(d, mla_desc_k_sw128(smem_u32(sQ) + (c - G::QT) * 16384) + 2 * k, mla_desc_k_sw128(k0 + c * SK_CHUNK) + 2 * k, id_s, 1u);
             }
-            if (c + 1 < NCH) try_pv();
+            if (c + 1 < NC) try_pv();
           }
           tc_commit(&s_full);
           ++qk;
@@ -274,7 +294,7 @@ __global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant_
       tc_fence_after();
       if (i > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {       // warp-uniform: tcgen05.ld/st are warp collectives
 #pragma unroll 1
-        for (int c = 0; c < 16; ++c) {
+        for (int c = 0; c < nv * 4; ++c) {
           uint32_t o[16];
           tmem_ld_x16(tmem + lane_addr + O_COL + c * 16, o);
           tc_wait_ld();
@@ -298,11 +318,11 @@ __global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant_
       const int rr = live ? r : 0;
       const int t = row_base + rr / a.Hl, h = rr % a.Hl;
       const float m_nat = (m_ref == -INFINITY) ? -INFINITY : m_ref * 0.6931471805599453f;
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      bf16* dst = a.out + ((size_t)h * a.T + t) * DV + vh * 256;
-      float* po = a.n_splits > 1 ? a.part_o + (((size_t)split * a.T + t) * a.Hl + h) * DV + vh * 256 : nullptr;
+      const float inv = (l > 0.f ? 1.f / l : 0.f) * ((a.gate && live) ? a.gate[(size_t)t * a.Hl + h] : 1.f);      // output gate of the head
+      bf16* dst = a.out + ((size_t)h * a.ldt + t) * LAT + vh * (G::VCH * 64);
+      float* po = a.n_splits > 1 ? a.part_o + (((size_t)split * a.T + t) * a.Hl + h) * LAT + vh * (G::VCH * 64) : nullptr;
 #pragma unroll 1
-      for (int c = 0; c < 16; ++c) {
+      for (int c = 0; c < nv * 4; ++c) {
         uint32_t o[16];
         if (n_tiles > 0) { tmem_ld_x16(tmem + lane_addr + O_COL + c * 16, o); tc_wait_ld(); }
         else {
@@ -330,7 +350,7 @@ __global__ void __launch_bounds__(192, 1) mla_attn_kernel(const __grid_constant_
   if (*abortp && warp == 0) { const long long c0 = clock64(); while (clock64() - c0 < 400000) __nanosleep(1000); }
   tc_fence_before();
   __syncthreads();
-  if (warp == 1) tmem_dealloc(tmem, 512);
+  if (warp == 1) tmem_dealloc(tmem, G::TMEM);
 }
 
 // ------------------------------------------------------------------------------------------------------------
@@ -671,9 +691,9 @@ __global__ void __launch_bounds__(192, 1) mla_attn_pair_kernel(const __grid_cons
 }
 
 // out[h, t, :] = sum_s o_s * exp(m_s - M) / sum_s l_s * exp(m_s - M); partials are token-major, the output head-major.
-__global__ void __launch_bounds__(128) mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out, int T, int Hl,
-                                                        int n_splits) {
-  // One block of 128 threads per (token, head), four output columns per thread.  The (m, l) pairs of all splits are read at once by
+__global__ void __launch_bounds__(128) mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ gate,
+                                                        bf16* __restrict__ out, int T, int ldt, int Hl, int D, int n_splits) {
+  // One block per (token, head), four output columns per thread (D / 4 threads, at least a warp).  The (m, l) pairs of all splits are read at once by
   // one warp (weights exp(m - M) and the denominator land in shared memory); the partial rows then come eight splits at a time,
   // every load issued before the first use.  (Reading m, branching, then loading the row made the merge a chain of one L2 round
   // trip per split: 21 us at 32 splits on a batch-1 step.)
@@ -701,13 +721,14 @@ __global__ void __launch_bounds__(128) mla_merge_kernel(const float* __restrict_
   }
   __syncthreads();
   const int d0 = threadIdx.x * 4;
+  if (d0 >= D) return;
   float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int s0 = 0; s0 < n_splits; s0 += 8) {
     float4 pv[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const int sidx = min(s0 + j, n_splits - 1);
-      pv[j] = *(const float4*)(part_o + (((size_t)sidx * T + t) * Hl + h) * DV + d0);
+      pv[j] = *(const float4*)(part_o + (((size_t)sidx * T + t) * Hl + h) * D + d0);
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -715,15 +736,30 @@ __global__ void __launch_bounds__(128) mla_merge_kernel(const float* __restrict_
       if (w != 0.f) { acc.x += pv[j].x * w; acc.y += pv[j].y * w; acc.z += pv[j].z * w; acc.w += pv[j].w * w; }
     }
   }
-  const float L = Lsh, inv = L > 0.f ? 1.f / L : 0.f;
+  const float L = Lsh, inv = (L > 0.f ? 1.f / L : 0.f) * (gate ? gate[(size_t)t * Hl + h] : 1.f);
   bf16 ob[4] = {__float2bfloat16(acc.x * inv), __float2bfloat16(acc.y * inv), __float2bfloat16(acc.z * inv), __float2bfloat16(acc.w * inv)};
-  *(uint2*)(out + ((size_t)h * T + t) * DV + d0) = *(const uint2*)ob;
+  *(uint2*)(out + ((size_t)h * ldt + t) * D + d0) = *(const uint2*)ob;
 }
 
 __global__ void mla_fill_ml_kernel(float* ml, long long n) {
   pdl_launch(); pdl_wait();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i < n) ml[i] = (i & 1) ? 0.f : -INFINITY;
+}
+
+template <int NC, int NL>
+static int mla_launch(const MlaArgs& a, dim3 grid, cudaStream_t s) {
+  using G = MlaGeo<NC, NL>;
+  auto kern = mla_attn_kernel<NC, NL>;
+  static bool attr_set[64] = {false};
+  int dev = 0; cudaGetDevice(&dev);
+  if (!attr_set[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, G::SMEM);
+    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(mla_attn)");
+    attr_set[dev & 63] = true;
+  }
+  CA_LAUNCH_PDL(kern, grid, 192, G::SMEM, s, a);
+  return CA_OK;
 }
 
 extern "C" int cuteafd_mla_attention(const void* q_lat, const void* q_rope, const void* kv_map, const int* page_table, const int* kv_len,
@@ -735,16 +771,10 @@ extern "C" int cuteafd_mla_attention(const void* q_lat, const void* q_rope, cons
   MlaArgs a;
   a.q_lat = (const bf16*)q_lat; a.q_rope = (const bf16*)q_rope; a.kv_map = (const CUtensorMap*)kv_map; a.page_table = page_table;
   a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len; a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.status = status;
-  a.Hl = Hl; a.max_pages = max_pages; a.n_splits = n_splits; a.T = T; a.scale = scale;
+  a.Hl = Hl; a.max_pages = max_pages; a.n_splits = n_splits; a.T = T; a.ldt = T; a.gate = nullptr; a.scale = scale;
   const int tpt = 128 / Hl;
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
-  static bool attr_set[64] = {false};
   int dev = 0; cudaGetDevice(&dev);
-  if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(mla_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, MLA_SMEM);
-    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(mla_attn)");
-    attr_set[dev & 63] = true;
-  }
   if (n_splits > 1) {
     const long long n = (long long)n_splits * T * Hl * 2;
     CA_LAUNCH_PDL(mla_fill_ml_kernel, (int)((n + 255) / 256), 256, 0, s, part_ml, n);
@@ -773,13 +803,65 @@ extern "C" int cuteafd_mla_attention(const void* q_lat, const void* q_rope, cons
     cudaError_t le = cudaLaunchKernelEx(&cfg, mla_attn_pair_kernel, a);
     if (le != cudaSuccess) return ca_cuda(le, "mla_attn_pair launch");
   } else {
-    CA_LAUNCH_PDL(mla_attn_kernel, grid, 192, MLA_SMEM, s, a);
+    const int rc = mla_launch<9, 8>(a, grid, s);
+    if (rc) return rc;
   }
   CA_CHECK_LAUNCH("mla_attention");
   if (n_splits > 1) {
-    CA_LAUNCH_PDL(mla_merge_kernel, dim3(T, Hl), 128, 0, s, part_o, part_ml, (bf16*)out, T, Hl, n_splits);
+    CA_LAUNCH_PDL(mla_merge_kernel, dim3(T, Hl), 128, 0, s, part_o, part_ml, (const float*)nullptr, (bf16*)out, T, T, Hl, DV, n_splits);
     CA_CHECK_LAUNCH("mla_merge");
   }
+  return CA_OK;
+}
+
+// Latent attention without positions: the absorbed kernel over cache rows of `rank_pad` values (a multiple of 64, 64..512; the pad of a
+// narrower latent is zero in the cache and in the queries).  q_lat, out: head-major [Hl, ldt, rank_pad]; any Hl <= 128 (a query tile
+// takes 128 / Hl whole tokens).  `gate` [T, Hl] multiplies each head's output (null: none).
+extern "C" int cuteafd_latent_attention(const void* q_lat, const void* kv_map, const int* page_table, const int* kv_len, const int* q_start,
+                                        const int* q_len, const float* gate, void* out, float* part_o, float* part_ml, int T, int ldt, int n_seq,
+                                        int max_q_len, int Hl, int rank_pad, int max_pages, int n_splits, float scale, int* status, cudaStream_t s) {
+  CA_REQUIRE(q_lat && kv_map && page_table && kv_len && q_start && q_len && out, "latent_attention: null argument");
+  CA_REQUIRE(Hl >= 1 && Hl <= 128 && ldt >= T, "latent_attention: 1..128 heads (got %d), head stride >= rows", Hl);
+  CA_REQUIRE(rank_pad % 64 == 0 && rank_pad >= 64 && rank_pad <= 512, "latent_attention: padded rank %d (64..512, a multiple of 64)", rank_pad);
+  CA_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (part_o && part_ml)), "latent_attention: 1..64 KV splits, and split-KV needs scratch");
+  if (T <= 0 || n_seq <= 0) return CA_OK;
+  MlaArgs a;
+  a.q_lat = (const bf16*)q_lat; a.q_rope = nullptr; a.kv_map = (const CUtensorMap*)kv_map; a.page_table = page_table;
+  a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len; a.gate = n_splits > 1 ? nullptr : gate; a.out = (bf16*)out; a.part_o = part_o;
+  a.part_ml = part_ml; a.status = status; a.Hl = Hl; a.max_pages = max_pages; a.n_splits = n_splits; a.T = T; a.ldt = ldt; a.scale = scale;
+  const int tpt = 128 / Hl, nl = rank_pad / 64;
+  a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
+  const dim3 grid(n_splits, nl <= 4 ? 1 : 2, n_seq * a.max_q_tiles);
+  int rc;
+  switch (nl) {
+    case 1: rc = mla_launch<1, 1>(a, grid, s); break;
+    case 2: rc = mla_launch<2, 2>(a, grid, s); break;
+    case 3: rc = mla_launch<3, 3>(a, grid, s); break;
+    case 4: rc = mla_launch<4, 4>(a, grid, s); break;
+    case 5: rc = mla_launch<5, 5>(a, grid, s); break;
+    case 6: rc = mla_launch<6, 6>(a, grid, s); break;
+    case 7: rc = mla_launch<7, 7>(a, grid, s); break;
+    default: rc = mla_launch<8, 8>(a, grid, s); break;
+  }
+  if (rc) return rc;
+  CA_CHECK_LAUNCH("latent_attention");
+  if (n_splits > 1) {
+    const int threads = rank_pad / 4 < 32 ? 32 : rank_pad / 4;
+    CA_LAUNCH_PDL(mla_merge_kernel, dim3(T, Hl), threads, 0, s, part_o, part_ml, gate, (bf16*)out, T, ldt, Hl, rank_pad, n_splits);
+    CA_CHECK_LAUNCH("mla_merge");
+  }
+  return CA_OK;
+}
+
+// Descriptor of one layer's latent cache [slots, row_stride] bf16 of which the first `width` columns are the layer's: box {64 elements,
+// one page}.
+extern "C" int cuteafd_tmap_encode_latent_rows(void* out128, const void* base, uint64_t n_slots, uint64_t width, uint64_t row_stride) {
+  CA_REQUIRE(width % 64 == 0 && width <= row_stride && row_stride % 8 == 0, "tmap_encode_latent_rows: bad width / stride");
+  CUtensorMap m;
+  int rc = ca_encode_tmap_3d(&m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, width, n_slots, 1, row_stride * 2, row_stride * 2 * n_slots, 64, MKEYS, 1,
+                             CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return rc;
+  memcpy(out128, &m, sizeof(m));
   return CA_OK;
 }
 

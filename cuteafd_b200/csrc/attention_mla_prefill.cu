@@ -31,9 +31,7 @@
 #define PF_NSV 2                  // V stages
 #define PF_Q_BYTES 0              // the query tile lives in tensor memory (A operand of the score MMAs)
 #define PF_P_BYTES 32768          // 2 chunks (64 keys each) x [128 rows x 128 B]
-#define PF_K_STAGE 49152          // 3 chunks x [128 keys x 128 B]
 #define PF_V_STAGE 32768          // 2 chunks (64 dims each) x [128 keys x 128 B]
-#define PF_SMEM (PF_Q_BYTES + PF_P_BYTES + PF_NS * PF_K_STAGE + PF_NSV * PF_V_STAGE + 256)
 
 struct MlaPrefillArgs {
   const bf16* q_nope;           // [Hl, T, 128] head-major
@@ -44,9 +42,11 @@ struct MlaPrefillArgs {
   const int* kv_len;
   const int* q_start;
   const int* q_len;
-  bf16* out;                    // [T, Hl * 128] token-major
+  const float* gate;            // [T, Hl] factor of each head's output, or null
+  bf16* out;                    // [T, ldo] token-major, head h at column h * dv
   int* status;
   int T, Hl, max_q_tiles;
+  int ldt, ldo, dv;             // rows between two heads of q_nope, output row stride, value width
   float scale;
 };
 
@@ -68,13 +68,17 @@ __device__ __forceinline__ void pf_tmem_st_x16(uint32_t addr, const uint32_t* r)
                  "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]) : "memory");
 }
 
+// KN 64-wide chunks of per-head key columns, KR rotated chunks shared by the heads (0 = attention without positions), NV chunks of value
+// columns; the expanded buffer holds (KN + NV) * 64 columns per head.  DeepSeek-V3: 2, 1, 2.
+template <int KN, int KR, int NV>
 __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_constant__ MlaPrefillArgs a) {
   pdl_launch(); pdl_wait();
+  constexpr int NK = KN + KR, K_STAGE = NK * 16384, V_STAGE = NV * 16384, HEAD_W = (KN + NV) * 64;
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t* sP = smem;
   uint8_t* sK = sP + PF_P_BYTES;
-  uint8_t* sV = sK + PF_NS * PF_K_STAGE;
-  uint64_t* bars = (uint64_t*)(sV + PF_NSV * PF_V_STAGE);
+  uint8_t* sV = sK + PF_NS * K_STAGE;
+  uint64_t* bars = (uint64_t*)(sV + PF_NSV * V_STAGE);
   uint64_t* k_full = bars; uint64_t* k_empty = bars + 2; uint64_t* v_full = bars + 4; uint64_t* v_empty = bars + 6;     // [<= 2] each
   uint64_t* s_full = bars + 8;          // [2]
   uint64_t* s_free = bars + 10;         // [2]: the softmax threads are done with the score buffer
@@ -116,11 +120,11 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
     const int r = (warp & 3) * 32 + lane;
     const uint32_t dst = tmem + ((uint32_t)((warp & 3) * 32) << 16) + Q_COL;
     const int t = row_base + (r < R ? r : 0);
-    const bf16* src_nope = a.q_nope + ((size_t)head * a.T + t) * 128;
+    const bf16* src_nope = a.q_nope + ((size_t)head * a.ldt + t) * (KN * 64);
     const bf16* src_rope = a.q_rope + ((size_t)t * a.Hl + head) * 64;
 #pragma unroll 1
-    for (int g = 0; g < 6; ++g) {                  // 16 columns = 32 elements per store
-      const bf16* src = g < 4 ? src_nope + g * 32 : src_rope + (g - 4) * 32;
+    for (int g = 0; g < 2 * NK; ++g) {             // 16 columns = 32 elements per store
+      const bf16* src = (KR == 0 || g < 2 * KN) ? src_nope + g * 32 : src_rope + (g - 2 * KN) * 32;
       uint32_t w[16];
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
@@ -144,10 +148,10 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
       if (!mbar_wait_bounded(&k_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); return false; }
       if (lane == 0) {
         const int row = ctx0 + i * PF_KT;
-        mbar_expect_tx(&k_full[s], PF_K_STAGE);
-        tma_load_3d(sK + s * PF_K_STAGE, &a.kvb_map, &k_full[s], head * 256, row, 0);
-        tma_load_3d(sK + s * PF_K_STAGE + 16384, &a.kvb_map, &k_full[s], head * 256 + 64, row, 0);
-        tma_load_3d(sK + s * PF_K_STAGE + 32768, &a.lat_map, &k_full[s], 512, row, 0);
+        mbar_expect_tx(&k_full[s], K_STAGE);
+#pragma unroll
+        for (int c = 0; c < KN; ++c) tma_load_3d(sK + s * K_STAGE + c * 16384, &a.kvb_map, &k_full[s], head * HEAD_W + c * 64, row, 0);
+        if (KR) tma_load_3d(sK + s * K_STAGE + KN * 16384, &a.lat_map, &k_full[s], 512, row, 0);
       }
       __syncwarp();
       return true;
@@ -159,24 +163,24 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
       if (!mbar_wait_bounded(&v_empty[sv], phv, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, 0x1000 + i); break; }
       if (lane == 0) {
         const int row = ctx0 + i * PF_KT;
-        mbar_expect_tx(&v_full[sv], PF_V_STAGE);
-        tma_load_3d(sV + sv * PF_V_STAGE, &a.kvb_map, &v_full[sv], head * 256 + 128, row, 0);
-        tma_load_3d(sV + sv * PF_V_STAGE + 16384, &a.kvb_map, &v_full[sv], head * 256 + 192, row, 0);
+        mbar_expect_tx(&v_full[sv], V_STAGE);
+#pragma unroll
+        for (int c = 0; c < NV; ++c) tma_load_3d(sV + sv * V_STAGE + c * 16384, &a.kvb_map, &v_full[sv], head * HEAD_W + (KN + c) * 64, row, 0);
       }
       __syncwarp();
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
-    const uint32_t id_s = pf_idesc(PF_KT, 0), id_o = pf_idesc(128, 1);
+    const uint32_t id_s = pf_idesc(PF_KT, 0), id_o = pf_idesc(NV * 64, 1);
     auto issue_scores = [&](int j) -> bool {     // S[j & 1] = Q K(j)^T once the softmax threads have copied tile j - 2 out of it
       const int s = j % PF_NS;
       if (j >= 2 && !mbar_wait_bounded(&s_free[j & 1], ((j - 2) >> 1) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, 0x2000 + j); return false; }
       if (!mbar_wait_bounded(&k_full[s], (j / PF_NS) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, j); return false; }
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t k0 = smem_u32(sK + s * PF_K_STAGE), d = tmem + ((j & 1) ? S1_COL : S0_COL);
+        const uint32_t k0 = smem_u32(sK + s * K_STAGE), d = tmem + ((j & 1) ? S1_COL : S0_COL);
 #pragma unroll
-        for (int kb = 0; kb < 3; ++kb)
+        for (int kb = 0; kb < NK; ++kb)
 #pragma unroll
           for (int k = 0; k < 4; ++k)
             tc_mma_f16_ta(d, tmem + Q_COL + kb * 32 + k * 8, umma_desc_sw128(k0 + kb * 16384) + 2 * k, id_s, (kb | k) ? 1u : 0u);
@@ -194,7 +198,7 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
       if (!mbar_wait_bounded(&v_full[sv], (i / PF_NSV) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, 0x4000 + i); break; }
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t v0 = smem_u32(sV + sv * PF_V_STAGE);
+        const uint32_t v0 = smem_u32(sV + sv * V_STAGE);
 #pragma unroll
         for (int k = 0; k < PF_KT / 16; ++k)       // 16 keys per MMA: P chunk k / 4 (64 keys per 128-byte row), V rows 16 k .. 16 k + 15
           tc_mma_f16(tmem + O_COL, umma_desc_sw128(smem_u32(sP) + (k >> 2) * 16384) + 2 * (k & 3), pf_desc_mn_sw128(v0 + k * 2048, 16384, 1024), id_o,
@@ -297,7 +301,7 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
       tc_fence_after();
       if (i > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {      // warp-uniform: tcgen05.ld/st are warp collectives
 #pragma unroll 1
-        for (int c = 0; c < 8; ++c) {
+        for (int c = 0; c < NV * 4; ++c) {
           uint32_t o[16];
           tmem_ld_x16(tmem + lane_addr + O_COL + c * 16, o);
           tc_wait_ld();
@@ -319,10 +323,11 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
     tc_fence_after();
     if (__all_sync(0xffffffffu, ok)) {
       const int t = row_base + (live ? r : 0);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      bf16* dst = a.out + ((size_t)t * a.Hl + head) * 128;
+      const float inv = (l > 0.f ? 1.f / l : 0.f) * ((a.gate && live) ? a.gate[(size_t)t * a.Hl + head] : 1.f);      // output gate of the head
+      bf16* dst = a.out + (size_t)t * a.ldo + (size_t)head * a.dv;
+      const bool vec = (a.ldo | a.dv) % 8 == 0;
 #pragma unroll 1
-      for (int c = 0; c < 8; ++c) {
+      for (int c = 0; c < NV * 4; ++c) {
         uint32_t o[16];
         if (n_tiles > 0) { tmem_ld_x16(tmem + lane_addr + O_COL + c * 16, o); tc_wait_ld(); }
         else {
@@ -333,8 +338,14 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
         uint32_t w[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) { bf162 hh = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * inv, __uint_as_float(o[2 * j + 1]) * inv); w[j] = *(uint32_t*)&hh; }
-        *(uint4*)(dst + c * 16) = make_uint4(w[0], w[1], w[2], w[3]);
-        *(uint4*)(dst + c * 16 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+        if (vec) {                            // value widths that do not fill their last 64-wide chunk stop at column dv
+          if (c * 16 < a.dv) *(uint4*)(dst + c * 16) = make_uint4(w[0], w[1], w[2], w[3]);
+          if (c * 16 + 8 < a.dv) *(uint4*)(dst + c * 16 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (c * 16 + j < a.dv) dst[c * 16 + j] = ((const bf16*)w)[j];
+        }
       }
     }
   }
@@ -688,17 +699,19 @@ extern "C" int cuteafd_gqa_prefill_attention(const void* q, const void* kv_map, 
 }
 
 // Gathers the latent rows of every sequence's context out of the paged cache into one contiguous buffer:
-// dst[ctx_start[s] + j] = cache[page_table[s][j / 64] * 64 + j % 64] for j < kv_len[s]; rows of 576 bf16 = 72 x 16 bytes.
+// dst[ctx_start[s] + j] = cache[page_table[s][j / 64] * 64 + j % 64] for j < kv_len[s]; rows of w16 16-byte pieces (72: 576 bf16),
+// src16 pieces between two rows of the cache; a block copies blockDim / w16 rows.
 __global__ void mla_gather_ctx_kernel(const uint4* __restrict__ cache, const int* __restrict__ page_table, const int* __restrict__ ctx_start,
-                                      const int* __restrict__ kv_len, uint4* __restrict__ dst, int max_pages, long long n_slots, long long dst_rows, int* status) {
+                                      const int* __restrict__ kv_len, uint4* __restrict__ dst, int max_pages, long long n_slots, long long dst_rows, int w16,
+                                      int src16, int* status) {
   pdl_launch(); pdl_wait();
   const int seq = blockIdx.y;
-  const int j = blockIdx.x * 4 + threadIdx.x / 72, c = threadIdx.x % 72;
+  const int j = blockIdx.x * (blockDim.x / w16) + threadIdx.x / w16, c = threadIdx.x % w16;
   if (j >= kv_len[seq]) return;
   const long long slot = (long long)page_table[(size_t)seq * max_pages + j / 64] * 64 + j % 64;
   const long long row = (long long)ctx_start[seq] + j;
   if (slot < 0 || slot >= n_slots || row < 0 || row >= dst_rows) { if (c == 0) ca_dev_fail(status, CA_DEV_BAD_INDEX, 0xB01); return; }
-  dst[row * 72 + c] = cache[slot * 72 + c];
+  dst[row * w16 + c] = cache[slot * src16 + c];
 }
 
 extern "C" int cuteafd_mla_gather_ctx(const void* cache, const int* page_table, const int* ctx_start, const int* kv_len, void* dst, int n_seq,
@@ -706,8 +719,37 @@ extern "C" int cuteafd_mla_gather_ctx(const void* cache, const int* page_table, 
   CA_REQUIRE(cache && page_table && ctx_start && kv_len && dst, "mla_gather_ctx: null argument");
   if (n_seq <= 0 || max_kv <= 0) return CA_OK;
   CA_LAUNCH_PDL(mla_gather_ctx_kernel, dim3((max_kv + 3) / 4, n_seq), 288, 0, s, (const uint4*)cache, page_table, ctx_start, kv_len, (uint4*)dst, max_pages,
-                n_slots, dst_rows, status);
+                n_slots, dst_rows, 72, 72, status);
   CA_CHECK_LAUNCH("mla_gather_ctx");
+  return CA_OK;
+}
+
+// Rows of `width` bf16 (a multiple of 8, at most 4096) out of a cache whose rows are `row_stride` apart.
+extern "C" int cuteafd_latent_gather_ctx(const void* cache, const int* page_table, const int* ctx_start, const int* kv_len, void* dst, int n_seq,
+                                         int max_kv, int max_pages, long long n_slots, long long dst_rows, int width, int row_stride, int* status,
+                                         cudaStream_t s) {
+  CA_REQUIRE(cache && page_table && ctx_start && kv_len && dst, "latent_gather_ctx: null argument");
+  CA_REQUIRE(width % 8 == 0 && width >= 8 && width <= 4096 && row_stride % 8 == 0 && width <= row_stride, "latent_gather_ctx: bad row width %d / %d", width, row_stride);
+  if (n_seq <= 0 || max_kv <= 0) return CA_OK;
+  const int w16 = width / 8, rpb = w16 >= 256 ? 1 : 256 / w16;
+  CA_LAUNCH_PDL(mla_gather_ctx_kernel, dim3((max_kv + rpb - 1) / rpb, n_seq), w16 * rpb, 0, s, (const uint4*)cache, page_table, ctx_start, kv_len,
+                (uint4*)dst, max_pages, n_slots, dst_rows, w16, row_stride / 8, status);
+  CA_CHECK_LAUNCH("latent_gather_ctx");
+  return CA_OK;
+}
+
+template <int KN, int KR, int NV>
+static int mla_prefill_launch(const MlaPrefillArgs& a, int n_seq, cudaStream_t s) {
+  constexpr int SMEM = PF_P_BYTES + PF_NS * (KN + KR) * 16384 + PF_NSV * NV * 16384 + 256;
+  auto kern = mla_prefill_kernel<KN, KR, NV>;
+  static bool attr_set[64] = {false};
+  int dev = 0; cudaGetDevice(&dev);
+  if (!attr_set[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(mla_prefill)");
+    attr_set[dev & 63] = true;
+  }
+  CA_LAUNCH_PDL(kern, dim3(a.Hl, n_seq * a.max_q_tiles), 192, SMEM, s, a);
   return CA_OK;
 }
 
@@ -726,14 +768,36 @@ extern "C" int cuteafd_mla_prefill_attention(const void* q_nope, const void* q_r
   if (rc) return rc;
   a.q_nope = (const bf16*)q_nope; a.q_rope = (const bf16*)q_rope; a.ctx_start = ctx_start; a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len;
   a.out = (bf16*)out; a.status = status; a.T = T; a.Hl = Hl; a.max_q_tiles = (max_q_len + 127) / 128; a.scale = scale;
-  static bool attr_set[64] = {false};
-  int dev = 0; cudaGetDevice(&dev);
-  if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(mla_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, PF_SMEM);
-    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(mla_prefill)");
-    attr_set[dev & 63] = true;
-  }
-  CA_LAUNCH_PDL(mla_prefill_kernel, dim3(Hl, n_seq * a.max_q_tiles), 192, PF_SMEM, s, a);
+  a.gate = nullptr; a.ldt = T; a.ldo = Hl * 128; a.dv = 128;
+  rc = mla_prefill_launch<2, 1, 2>(a, n_seq, s);
+  if (rc) return rc;
   CA_CHECK_LAUNCH("mla_prefill_attention");
+  return CA_OK;
+}
+
+// The same for latent attention without positions: q [Hl, ldt, dk_pad] head-major (dk_pad 64 / 128 / 192, pad columns zero), kvb
+// [rows, Hl * (dk_pad + dv_pad)] (per head the key columns, then the value columns, each padded to whole 64-wide chunks; dv_pad 64 / 128),
+// out [T, ldo] token-major with head h at column h * dv, `gate` [T, Hl] (or null) multiplied into each head's output.
+extern "C" int cuteafd_latent_prefill_attention(const void* q, const void* kvb, long long rows, const int* ctx_start, const int* kv_len,
+                                                const int* q_start, const int* q_len, const float* gate, void* out, int T, int ldt, int n_seq,
+                                                int max_q_len, int Hl, int dk_pad, int dv_pad, int dv, int ldo, float scale, int* status,
+                                                cudaStream_t s) {
+  CA_REQUIRE(q && kvb && ctx_start && kv_len && q_start && q_len && out && rows > 0, "latent_prefill_attention: null argument");
+  CA_REQUIRE(Hl >= 1 && ldt >= T && dv >= 1 && dv <= dv_pad && ldo >= Hl * dv, "latent_prefill_attention: bad shape");
+  CA_REQUIRE((dk_pad == 64 || dk_pad == 128 || dk_pad == 192) && (dv_pad == 64 || dv_pad == 128), "latent_prefill_attention: head widths %d / %d", dk_pad, dv_pad);
+  if (T <= 0 || n_seq <= 0) return CA_OK;
+  MlaPrefillArgs a;
+  const int hw = dk_pad + dv_pad;
+  int rc = ca_encode_tmap_2d(&a.kvb_map, kvb, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (uint64_t)Hl * hw, (uint64_t)rows, (uint64_t)Hl * hw * 2, 64, PF_KT,
+                             CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return rc;
+  a.lat_map = a.kvb_map;
+  a.q_nope = (const bf16*)q; a.q_rope = nullptr; a.ctx_start = ctx_start; a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len;
+  a.gate = gate; a.out = (bf16*)out; a.status = status; a.T = T; a.Hl = Hl; a.max_q_tiles = (max_q_len + 127) / 128; a.scale = scale;
+  a.ldt = ldt; a.ldo = ldo; a.dv = dv;
+  if (dv_pad == 64) rc = dk_pad == 64 ? mla_prefill_launch<1, 0, 1>(a, n_seq, s) : (dk_pad == 128 ? mla_prefill_launch<2, 0, 1>(a, n_seq, s) : mla_prefill_launch<3, 0, 1>(a, n_seq, s));
+  else rc = dk_pad == 64 ? mla_prefill_launch<1, 0, 2>(a, n_seq, s) : (dk_pad == 128 ? mla_prefill_launch<2, 0, 2>(a, n_seq, s) : mla_prefill_launch<3, 0, 2>(a, n_seq, s));
+  if (rc) return rc;
+  CA_CHECK_LAUNCH("latent_prefill_attention");
   return CA_OK;
 }

@@ -6,6 +6,9 @@
 #include "common.cuh"
 
 enum { SCORE_SIGMOID = 0, SCORE_SOFTMAX = 1, SCORE_SQRTSOFTPLUS = 2 };
+// `scoring` of the selection entry points: the score function, plus this bit when a group is ranked by its best member alone
+// (otherwise by the sum of its two best)
+#define GROUP_BY_MAX 16
 
 // ---------------------------------------------------------------- route packing
 // Inputs: idx [T, k] (expert ids; ids outside [e_lo, e_hi) are skipped - they belong to another expert rank).
@@ -140,7 +143,7 @@ static size_t route_pack_smem(int T, int k, int e_lo, int e_hi) {
 
 // One block per token.  logits fp32 [T, E] (E <= 512).  Selection uses score + bias (bias may be null),
 // optional group-limited routing (top `topk_group` of `n_group` groups ranked by the sum of their two
-// best biased scores); gate weights come from the unbiased scores, normalised over the chosen k and
+// best biased scores, or by their best one: GROUP_BY_MAX); gate weights come from the unbiased scores, normalised over the chosen k and
 // multiplied by route_scale.  Ties resolve to the lowest expert id.
 __global__ void router_select_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ idx,
                                      float* __restrict__ wts, int E, int k, int scoring, int normalize, float route_scale,
@@ -153,6 +156,8 @@ __global__ void router_select_kernel(const float* __restrict__ logits, const flo
   __shared__ int sel[16];
   __shared__ float selw[16];
   const int t = blockIdx.x, tid = threadIdx.x;
+  const bool by_max = (scoring & GROUP_BY_MAX) != 0;
+  scoring &= GROUP_BY_MAX - 1;
   const float* lg = logits + (size_t)t * E;
   float mx = -INFINITY;
   for (int e = tid; e < E; e += blockDim.x) mx = fmaxf(mx, lg[e]);
@@ -178,7 +183,7 @@ __global__ void router_select_kernel(const float* __restrict__ logits, const flo
     if (tid < n_group) {
       float a = -INFINITY, b = -INFINITY;
       for (int j = 0; j < per; ++j) { const float v = choice[tid * per + j]; if (v > a) { b = a; a = v; } else if (v > b) b = v; }
-      gscore[tid] = a + b;
+      gscore[tid] = by_max ? a : a + b;
     }
     __syncthreads();
     if (tid == 0) {
@@ -399,6 +404,8 @@ __device__ __forceinline__ void router_select_warp(const float* lg, const float*
                                                    int scoring, int normalize, float route_scale, int n_group, int topk_group,
                                                    int* idx_out, float* wts_out, int* sel_sh = nullptr) {
   const int lane = threadIdx.x & 31;
+  const bool by_max = (scoring & GROUP_BY_MAX) != 0;
+  scoring &= GROUP_BY_MAX - 1;
   float lv[NQ];                                 // this lane's logits, one trip to L2 for all of them
 #pragma unroll
   for (int q = 0; q < NQ; ++q) lv[q] = (lane + 32 * q < E) ? __ldcg(lg + lane + 32 * q) : -INFINITY;
@@ -428,11 +435,11 @@ __device__ __forceinline__ void router_select_warp(const float* lg, const float*
   __syncwarp();
   if (n_group > 1 && topk_group < n_group) {
     const int per = E / n_group;
-    float gs = -INFINITY;                       // lane g: sum of the two best biased scores of group g
+    float gs = -INFINITY;                       // lane g: sum of the two best biased scores of group g (or the best alone)
     if (lane < n_group) {
       float a = -INFINITY, b = -INFINITY;
       for (int j = 0; j < per; ++j) { const float v = choice[lane * per + j]; if (v > a) { b = a; a = v; } else if (v > b) b = v; }
-      gs = a + b;
+      gs = by_max ? a : a + b;
     }
     unsigned keep = 0;
     for (int r = 0; r < topk_group; ++r) {      // best groups first, lowest group id among equals

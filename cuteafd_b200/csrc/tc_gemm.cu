@@ -63,6 +63,10 @@ struct TcArgs {
   long long* trace;           // optional per-unit time stamps [grid, trace_units, 8] (see cuteafd_tc_trace)
   int ldsfb, ldy, rows_total, N, K, epi, splits, trace_units;
   int w4_tx;                  // KIND_W4A8: bytes one weight tile adds to the stage barrier's transaction count
+  int act;                    // activation of the plain epilogue: 0 none, 1 squared ReLU (experts without a gate projection)
+  // grouped GEMM over head-major operands (row = group * grp_rows + token) with a token-major result: group g writes columns
+  // [g * grp_cols, g * grp_cols + N) of row `token`; grp_rows 0 = the output row is the operand row
+  int grp_rows, grp_cols;
 };
 
 // Per-unit device trace: slot 0/1 producer first/last load issued, 2 MMA thread owns the accumulator, 4 last MMA
@@ -334,7 +338,7 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
     uint32_t tc = 0, stg_uses = 0;
     // staged (transposed) store: plain bf16 output of a 64+-token tile, 16-byte aligned rows
     const bool stage_ok = C::STG_BYTES > 0 && splits == 1 && a.epi != EPI_F32 && a.Y != nullptr && !(QOUT && a.q_out) && !(PEER && a.n_peer) &&
-                          a.ldy % 8 == 0 && a.N % 8 == 0 && ((uintptr_t)a.Y & 15) == 0 && (a.epi != EPI_BF16_RESIDUAL || ((uintptr_t)a.R & 15) == 0);
+                          a.ldy % 8 == 0 && a.N % 8 == 0 && a.grp_cols % 8 == 0 && ((uintptr_t)a.Y & 15) == 0 && (a.epi != EPI_BF16_RESIDUAL || ((uintptr_t)a.R & 15) == 0);
     float* stg = (float*)(smem + C::NSTAGE * C::STAGE_BYTES);
     bool stg_fail = false;
     for (int w = w_begin; w < w_end && !*abortp; ++w, ++tc) {
@@ -352,6 +356,7 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
       const float al2 = (SWIGLU && a.alpha2) ? a.alpha2[g] : al;
       const uint32_t tbase = tmem + ((uint32_t)(q4 * 32) << 16) + acc * C::ACC_COLS;
       float* ws = (splits > 1) ? a.splitk_ws + ((size_t)sp * a.rows_total) * a.N : nullptr;
+      const size_t obase = a.grp_rows > 0 ? (size_t)(row0 - g * a.grp_rows) * a.ldy + (size_t)g * a.grp_cols : (size_t)row0 * a.ldy;
 #pragma unroll 1
       for (int c0 = 0; c0 < TN; c0 += 16) {
         uint32_t r[16], r2[16];
@@ -430,7 +435,7 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
               if (SWIGLU) {
                 const float u = __uint_as_float(r2[j]) * al2;
                 v = v / (1.f + __expf(-v)) * u;
-              }
+              } else if (a.act) { v = fmaxf(v, 0.f); v *= v; }
               buf[j * 128 + et] = v;
             }
             mbar_arrive(&stg_bar);
@@ -445,7 +450,7 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
               if (c < nrows && nn < a.N) {
                 const float4 f0 = *(const float4*)(buf + row * 128 + grp * 8), f1 = *(const float4*)(buf + row * 128 + grp * 8 + 4);
                 float f[8] = {f0.x, f0.y, f0.z, f0.w, f1.x, f1.y, f1.z, f1.w};
-                const size_t o = (size_t)(row0 + c) * a.ldy + nn;
+                const size_t o = obase + (size_t)c * a.ldy + nn;
                 if (a.epi == EPI_BF16_RESIDUAL) {
                   const uint4 rv = *(const uint4*)(a.R + o);
                   const bf16* rb = (const bf16*)&rv;
@@ -472,8 +477,8 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
               if (SWIGLU) {
                 const float u = __uint_as_float(r2[j]) * al2;
                 v = v / (1.f + __expf(-v)) * u;
-              }
-              const size_t o = (size_t)(row0 + c) * a.ldy + n;
+              } else if (a.act) { v = fmaxf(v, 0.f); v *= v; }
+              const size_t o = obase + (size_t)c * a.ldy + n;
               if (splits > 1) ws[(size_t)(row0 + c) * a.N + n] = v;
               else if (a.epi == EPI_F32) ((float*)a.Y)[o] = v;
               else {
@@ -946,8 +951,10 @@ static int cluster_capacity(int splits, int* out) {
 extern "C" int cuteafd_tc_cluster_capacity(int kind, int tn, int splits, int* out) {
   CA_REQUIRE(out && (tn == 16 || tn == 32) && splits >= 1 && splits <= (tn == 16 ? 8 : 4), "tc_cluster_capacity: bad arguments");
   if (kind == KIND_BF16) return tn == 16 ? cluster_capacity<KIND_BF16, 16>(splits, out) : cluster_capacity<KIND_BF16, 32>(splits, out);
+#ifndef CA_TC_BF16_ONLY
   if (kind == KIND_NVFP4) return tn == 16 ? cluster_capacity<KIND_NVFP4, 16>(splits, out) : cluster_capacity<KIND_NVFP4, 32>(splits, out);
   if (kind == KIND_MXFP4) return tn == 16 ? cluster_capacity<KIND_MXFP4, 16>(splits, out) : cluster_capacity<KIND_MXFP4, 32>(splits, out);
+#endif
   return ca_fail(CA_ERR_UNSUPPORTED, "tc_cluster_capacity: no cluster kernel for this kind");
 }
 
@@ -996,8 +1003,12 @@ extern "C" int cuteafd_tc_linear(int kind, int swiglu, int tn, const void* tmA, 
   CA_REQUIRE(splits <= 1 || (!tiles && !swiglu && splitk_ws && splitk_cnt), "tc_linear: split-K is dense, non-swiglu only and needs scratch");
   CA_REQUIRE(epi == EPI_BF16 || epi == EPI_BF16_RESIDUAL || epi == EPI_F32, "tc_linear: bad epilogue %d", epi);
   CA_REQUIRE(epi != EPI_BF16_RESIDUAL || R, "tc_linear: residual epilogue needs R");
+  const int act = extra ? extra->act : 0, grp_rows = extra ? extra->grp_rows : 0, grp_cols = extra ? extra->grp_cols : 0;
+  CA_REQUIRE(act == 0 || (act == 1 && !swiglu && splits <= 1 && !q_out && epi != EPI_BF16_RESIDUAL), "tc_linear: the squared-ReLU epilogue is plain (no SwiGLU, split-K, FP4 output or residual)");
+  CA_REQUIRE(grp_rows == 0 || (grp_rows > 0 && tiles && !swiglu && !q_out && !peer.n && epi != EPI_BF16_RESIDUAL), "tc_linear: token-major output belongs to a plain grouped GEMM");
   if (rows_total <= 0 || N <= 0) return CA_OK;
   TcArgs a;
+  a.act = act; a.grp_rows = grp_rows; a.grp_cols = grp_cols;
   a.tmA = (const CUtensorMap*)tmA; a.tmA2 = (const CUtensorMap*)tmA2; a.tmB = (const CUtensorMap*)tmB;
   a.sfa = (const uint8_t* const*)sfa; a.sfa2 = (const uint8_t* const*)sfa2; a.sfb = (const uint8_t*)sfb;
   a.alpha = alpha; a.alpha2 = alpha2; a.tiles = (const int4*)tiles; a.n_tiles = n_tiles;
@@ -1017,8 +1028,10 @@ extern "C" int cuteafd_tc_linear(int kind, int swiglu, int tn, const void* tmA, 
     {
       const int grid_c = ((rows_total + tn - 1) / tn) * n_nt * a.splits;
       if (kind == KIND_BF16) return tn == 16 ? launch_cluster<KIND_BF16, 16>(a, grid_c, stream) : launch_cluster<KIND_BF16, 32>(a, grid_c, stream);
+#ifndef CA_TC_BF16_ONLY
       if (kind == KIND_NVFP4) return tn == 16 ? launch_cluster<KIND_NVFP4, 16>(a, grid_c, stream) : launch_cluster<KIND_NVFP4, 32>(a, grid_c, stream);
       return tn == 16 ? launch_cluster<KIND_MXFP4, 16>(a, grid_c, stream) : launch_cluster<KIND_MXFP4, 32>(a, grid_c, stream);
+#endif
     }
   }
   long long work = tiles ? (long long)max_tiles * n_nt : (long long)((rows_total + tn - 1) / tn) * n_nt * a.splits;
@@ -1026,7 +1039,11 @@ extern "C" int cuteafd_tc_linear(int kind, int swiglu, int tn, const void* tmA, 
   int grid = (int)(work < cap ? work : cap);
   if (grid < 1) grid = 1;
   if (kind == KIND_BF16) return swiglu ? launch_tn<KIND_BF16, true>(tn, a, grid, stream) : launch_tn<KIND_BF16, false>(tn, a, grid, stream);
+#ifndef CA_TC_BF16_ONLY      // a library built for one family's engine leaves the other operand kinds out
   if (kind == KIND_NVFP4) return swiglu ? launch_tn<KIND_NVFP4, true>(tn, a, grid, stream) : launch_tn<KIND_NVFP4, false>(tn, a, grid, stream);
   if (kind == KIND_W4A8) return swiglu ? launch_tn<KIND_W4A8, true>(tn, a, grid, stream) : launch_tn<KIND_W4A8, false>(tn, a, grid, stream);
   return swiglu ? launch_tn<KIND_MXFP4, true>(tn, a, grid, stream) : launch_tn<KIND_MXFP4, false>(tn, a, grid, stream);
+#else
+  return ca_fail(CA_ERR_UNSUPPORTED, "tc_linear: this build has bf16 operands only");
+#endif
 }

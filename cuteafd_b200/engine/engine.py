@@ -218,6 +218,7 @@ class Engine:
         self.graph_captures = 0
         self.census = GraphCensus()
         self._meta_cap = 0
+        self._meta_copied = None                # event behind the last host-to-device copy of the packed inputs
         self.launches_per_step = 0
 
     # ------------------------------------------------------------------ buffers
@@ -267,6 +268,8 @@ class Engine:
             parts = [context_hashes(self.engram.addr, list(engram_ctx[s]), list(tokens[q_start[s]:q_start[s] + q_len[s]])) for s in range(S)]
             extra = self.engram.set_hashes(np.concatenate(parts, axis=1))
         self._ensure_meta(T)
+        if self._meta_copied is not None:
+            self._meta_copied.synchronize()     # the previous step's copy may still be queued behind its predecessor's kernels
         mh = self.mh
         mh["tokens"][:T] = torch.as_tensor(tokens, dtype=torch.int32)
         mh["positions"][:T] = torch.as_tensor(positions, dtype=torch.int32)
@@ -280,6 +283,9 @@ class Engine:
         for s, row in enumerate(page_table_rows):
             mh["page_table"][s, :len(row)] = torch.as_tensor(row, dtype=torch.int32)
         self.meta_dev.copy_(self.meta_host, non_blocking=True)
+        if self.meta_dev.is_cuda:
+            self._meta_copied = self._meta_copied or torch.cuda.Event()
+            self._meta_copied.record()
         return self.meta_host.numel() * 4 + extra
 
     def set_input_embeds(self, rows, vals: torch.Tensor | None):

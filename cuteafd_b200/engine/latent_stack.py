@@ -1,0 +1,313 @@
+"""Engine of latent-attention layer stacks (the Bedovik design): unequal parallel layers over an fp32 residual, a looped layer range,
+latent attention without positions, squared-ReLU experts.
+
+Runs the generic engine's steps (packed inputs, paged cache, CUDA graphs per shape, head and token selection) with its own layer program:
+
+  token + position rows -> x (fp32)
+  per layer run   [at the start of a pass: x = W_in [x; x0], x += step vector]
+                  h = tanh(alpha x) w + b                              written by whichever kernel produced x
+                  h -> queries | latent | gates | router logits        one product, fp32 output
+                  latent_prepare                                       cache row, head-major queries, gates, logits
+                  decode: q W_uk -> absorbed attention over the latent pages -> W_uv (token-major) -> W_o
+                  prefill chunks: context rows -> keys / values (one product) -> per-head attention -> W_o
+                  routing + packing -> gather -> W_up (squared ReLU in the epilogue) -> W_down
+                  x += ls1 * mixer + ls2 * experts, next h or next [x; x0]     one launch
+  rows that need logits -> final norm -> head
+
+The cache holds one latent row per token and layer RUN (a looped layer keeps one per pass), all runs in one store of a common row width, so
+page bookkeeping, prefix sharing and the host tier treat it like any other paged cache.  With fp32 weights (`QuantSpec.dense = "f32"`) the
+same program runs entirely in fp32: fp32 products, the ordinary-core attention kernel, an fp32 cache.
+"""
+from __future__ import annotations
+
+import math
+import os
+
+import torch
+
+from .. import ops
+from ..models.latent_stack import StackLayer, StackWeights, up
+from ..ops import ActBuffer, KIND_BF16, KIND_F32, native, pick_tn
+from ..ops.native import call, ptr, stream
+from .engine import PAGE, Lane, StepShape
+from .mla import MlaEngine
+
+LANE_CAPS = (16, 32, 64, 256, 1024, 4096, 16384)
+
+
+class StackLane(Lane):
+    """Activation buffers for steps of up to `cap` rows; buffers that depend on a layer's geometry are made on first use per geometry."""
+
+    def __init__(self, eng: "LatentStackEngine", cap: int):
+        self.eng, self.cap, self.dev = eng, cap, eng.device
+        self.dt = torch.float32 if eng.f32 else torch.bfloat16
+        self.kind = KIND_F32 if eng.f32 else KIND_BF16
+        self.tn = pick_tn(min(cap, int(os.environ.get("CUTEAFD_TN", "128"))))
+        Wp = eng.Wp
+        self.x = torch.zeros(cap, Wp, dtype=torch.float32, device=self.dev)
+        self.xn, self.xn_act = self._operand(cap, Wp)
+        self.mix = torch.zeros(cap, Wp, dtype=self.dt, device=self.dev)
+        self.cat = self.cat_act = None
+        if eng.spec.loop is not None:
+            self.cat, self.cat_act = self._operand(cap, 2 * Wp)
+        rows = min(cap, 256)
+        self.xln, self.xln_act = self._operand(rows, Wp)
+        self.logits = torch.zeros(rows, eng.spec.vocab, dtype=torch.float32, device=self.dev)
+        i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=self.dev)
+        self.next_tok, self.tok_status = i32(cap), i32(cap)
+        self._bufs: dict = {}
+
+    def _operand(self, rows: int, K: int, tn: int | None = None):
+        act = ActBuffer.alloc(self.kind, rows, K, tn or self.tn, self.dev)
+        return act.data, act
+
+    def ensure_logits(self, n: int):
+        """Steps that want more logit rows than a lane starts with (whole prompts scored position by position)."""
+        if n > self.logits.shape[0]:
+            rows = min(self.cap, up(n, 256))
+            self.xln, self.xln_act = self._operand(rows, self.eng.Wp)
+            self.logits = torch.zeros(rows, self.eng.spec.vocab, dtype=torch.float32, device=self.dev)
+            self.eng.graphs.clear()                  # captured steps hold the old addresses
+            self.eng.census.invalidate()
+
+    def get(self, key, make):
+        if key not in self._bufs:
+            self._bufs[key] = make()
+        return self._bufs[key]
+
+    def mixer(self, a, n_in: int) -> dict:
+        """Buffers of one mixer geometry (head-major buffers are [heads, cap, .]: head h of row t is row h * cap + t)."""
+        H, dp, rp, cap = a.n_heads, up(a.head_dim, 64), up(a.kv_lora_rank, 64), self.cap
+
+        def make():
+            q, q_act = self._operand(H * cap, dp)
+            o, o_act = self._operand(cap, up(H * a.v_head_dim, 8))
+            return {"proj": torch.zeros(cap, up(n_in, 8), dtype=torch.float32, device=self.dev), "q": q, "q_act": q_act, "o": o, "o_act": o_act,
+                    "gate": torch.zeros(cap, H, dtype=torch.float32, device=self.dev),
+                    "tiles": torch.zeros(H * -(-cap // self.tn), 4, dtype=torch.int32, device=self.dev),
+                    "n_tiles": torch.zeros(1, dtype=torch.int32, device=self.dev), "max_tiles": H * -(-cap // self.tn)}
+        return self.get(("mix", H, a.head_dim, a.v_head_dim, rp, n_in), make)
+
+    def latent(self, H: int, rp: int) -> dict:
+        """Operands of the absorbed form: query and attended rows in the latent space."""
+        def make():
+            q, _ = self._operand(H * self.cap, rp)
+            o, o_act = self._operand(H * self.cap, rp)
+            return {"q": q, "o": o, "o_act": o_act}
+        return self.get(("lat", H, rp), make)
+
+    def experts(self, m) -> dict:
+        E, k, ff, cap = m.n_experts, m.top_k, m.intermediate, self.cap
+
+        def make():
+            rows = cap * k
+            per = max(1, math.ceil(rows / E) * 2)
+            tn = pick_tn(min(per, int(os.environ.get("CUTEAFD_TNG", "32"))))
+            i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=self.dev)
+            xs, xs_act = self._operand(rows, self.eng.Wp, tn)
+            h1, h1_act = self._operand(rows, up(ff, 8), tn)
+            max_tiles = E + rows // tn + 1
+            return {"tn": tn, "max_tiles": max_tiles, "logits": torch.zeros(cap, E, dtype=torch.float32, device=self.dev), "idx": i32(cap, k),
+                    "wts": torch.zeros(cap, k, dtype=torch.float32, device=self.dev), "src": i32(rows), "slot": i32(cap, k), "counts": i32(E),
+                    "offsets": i32(E), "tiles": i32(max_tiles, 4), "n_tiles": i32(1), "n_rows": i32(1), "xs": xs, "xs_act": xs_act, "h1": h1,
+                    "h1_act": h1_act, "y": torch.zeros(rows, self.eng.Wp, dtype=self.dt, device=self.dev)}
+        return self.get(("moe", E, k, ff), make)
+
+
+class LatentStackEngine(MlaEngine):
+    def __init__(self, weights: StackWeights, **kw):
+        spec = weights.spec
+        if not spec.blocks:
+            raise ValueError("LatentStackEngine runs stacks described by ModelSpec.blocks")
+        self.f32, self.Wp = weights.f32, up(spec.hidden, 8)
+        self.runs = spec.layer_runs()
+        for i, b in enumerate(spec.blocks):
+            if b.attn.kv_lora_rank > 1024:
+                raise ValueError(f"layer {i}: latents of up to 1024 values (got {b.attn.kv_lora_rank})")
+            if b.moe is not None and (b.moe.n_experts > 512 or b.moe.top_k > 16 or b.moe.n_group > 32):
+                raise ValueError(f"layer {i}: at most 512 experts, 16 per token, 32 groups")
+        super().__init__(weights, **kw)
+        self.tap = None             # set to a list to collect the residual rows after every layer run of eager steps
+
+    # ------------------------------------------------------------------ cache
+    def _alloc_attention_state(self):
+        spec, n = self.spec, self.n_pages * PAGE
+        self.row = max(up(b.attn.kv_lora_rank, 64) for b in spec.blocks)
+        # [layer runs, slots, row]: zero-filled, so a latent's pad and slots nobody wrote hold finite values
+        self.kv = torch.zeros(len(self.runs), n, self.row, dtype=torch.float32 if self.f32 else torch.bfloat16, device=self.device)
+        self.kv_tmaps = None
+        if not self.f32:
+            host = torch.zeros(len(self.runs), 128, dtype=torch.uint8)
+            for r, (li, _) in enumerate(self.runs):
+                call("cuteafd_tmap_encode_latent_rows", host[r].data_ptr(), self.kv[r].data_ptr(), n, up(spec.blocks[li].attn.kv_lora_rank, 64), self.row)
+            self.kv_tmaps = host.to(self.device)
+        self._pf: dict = {}
+
+    def lane(self, T: int) -> StackLane:
+        cap = next(c for c in LANE_CAPS if T <= c)
+        if cap not in self.lanes:
+            self.lanes[cap] = StackLane(self, cap)
+        return self.lanes[cap]
+
+    def set_inputs(self, tokens, positions, *args, **kw):
+        n = self.spec.learned_positions
+        if n and len(positions) and max(positions) >= n:
+            raise ValueError(f"position {max(positions)} is beyond this model's {n} learned positions")
+        return super().set_inputs(tokens, positions, *args, **kw)
+
+    def set_input_embeds(self, rows, vals):
+        if vals is not None and len(rows):
+            raise NotImplementedError("image / audio rows are not wired for latent-attention stacks")
+
+    def attn_splits_for(self, n_seq: int, max_q_len: int, max_kv: int) -> int:
+        if self.f32 or max_q_len > 16:
+            return 1
+        H = max(b.attn.n_heads for b in self.spec.blocks)
+        ctas = (1 if self.row <= 256 else 2) * n_seq * -(-max_q_len // max(1, 128 // min(H, 128)))
+        tiles = max(1, -(-max_kv // PAGE))
+        fill = self.sm_count * (2 if self.row <= 128 else 1) // ctas            # narrow latents: two CTAs per SM
+        if tiles < min(32, fill):
+            return 1 << (tiles.bit_length() - 1)       # short contexts: powers of two, so a growing context re-captures rarely
+        return max(1, min(32, fill))
+
+    # ------------------------------------------------------------------ layer program
+    def _emit(self, r: int, L: StackLane):
+        """What the producer of the residual rows in front of layer run `r` leaves for it."""
+        if r >= len(self.runs):
+            return None
+        li, opens = self.runs[r]
+        return ops.emit_arg(cat=L.cat) if opens is not None else ops.emit_arg(norm=self.weights.layer(li).norm, xn=L.xn)
+
+    def _forward_single(self, sh: StepShape) -> StackLane:
+        w, T, md = self.weights, sh.T, self.md
+        L = self.lane(T)
+        self.launches_per_step = 0
+        if sh.n_logits > L.logits.shape[0]:
+            L.ensure_logits(sh.n_logits)
+        none = native.EmitArg()
+        ops.stack_embed(md["tokens"], md["positions"], w.embed, w.pos, L.x, L.cat[:, self.Wp:] if L.cat is not None else None, self._emit(0, L) or none, T,
+                        f32=self.f32, status=self.status)
+        for r, (li, opens) in enumerate(self.runs):
+            lw = w.layer(li)
+            if opens is not None:
+                self._dense(w.loop_in, L.cat_act, L.x, T)
+                ops.stack_stream(L.x, ops.emit_arg(norm=lw.norm, xn=L.xn), T, f32=self.f32, vec=w.loop_step[opens])
+                self.launches_per_step += 1
+            self._block(r, li, lw, L, sh)
+            if self.tap is not None:
+                self.tap.append(L.x[:T, :self.spec.hidden].clone())
+        self.launches_per_step += 1
+        if sh.n_logits:
+            ops.stack_stream(L.x, ops.emit_arg(norm=(w.final_norm, w.final_b, w.final_alpha), xn=L.xln), sh.n_logits, f32=self.f32, src_rows=md["logit_rows"])
+            ops.tc_linear(w.lm_head, L.xln_act, L.logits, rows=sh.n_logits, status=self.status)
+            ops.argmax_rows(L.logits, L.next_tok, rows=sh.n_logits, status=L.tok_status)
+            self.launches_per_step += 3
+        return L
+
+    def _splits(self, N, K, T, tn, kind):
+        return 1 if kind == KIND_F32 else super()._splits(N, K, T, tn, kind)
+
+    def _block(self, r: int, li: int, lw: StackLayer, L: StackLane, sh: StepShape):
+        """One parallel layer: mixer and experts read the same rows L.xn; the combine adds both to the residual and prepares run r + 1."""
+        b, T = self.spec.blocks[li], sh.T
+        e = L.experts(b.moe) if b.moe is not None else None
+        self._mixer(r, b.attn, lw, L, sh, e)
+        if e is not None:
+            self._experts(b.moe, lw, L, e, T)
+        ops.stack_combine(L.x, L.mix, lw.ls1, e["y"] if e else None, e["slot"] if e else None, e["wts"] if e else None, lw.ls2, self._emit(r + 1, L), T,
+                          b.moe.top_k if e else 0)
+        self.launches_per_step += 1
+
+    def _mixer(self, r: int, a, lw: StackLayer, L: StackLane, sh: StepShape, e: dict | None):
+        T, md, H, rp, st = sh.T, self.md, a.n_heads, up(a.kv_lora_rank, 64), self.status
+        b = L.mixer(a, lw.w_in.N)
+        self._dense(lw.w_in, L.xn_act, b["proj"], T)
+        gate = b["gate"] if a.out_gate else None
+        ops.latent_prepare(b["proj"], lw.kv_norm, md["slot_map"], b["q"], self.kv[r], gate, e["logits"] if e else None, b["tiles"], b["n_tiles"],
+                           T=T, ldt=L.cap, H=H, d=a.head_dim, r=a.kv_lora_rank, rp=rp, E=e["logits"].shape[1] if e else 0, tn=L.tn, eps=self.spec.rms_eps,
+                           status=st)
+        self.launches_per_step += 1
+        if self._expands(a, sh):
+            self._prefill(r, a, lw, L, b, gate, sh)
+        else:
+            self._absorbed(r, a, lw, L, b, gate, sh)
+        self._dense(lw.wo, b["o_act"], L.mix, T)
+
+    def _absorbed(self, r: int, a, lw: StackLayer, L: StackLane, b: dict, gate, sh: StepShape):
+        T, md, H, rp = sh.T, self.md, a.n_heads, up(a.kv_lora_rank, 64)
+        lat = L.latent(H, rp)
+        per = dict(tiles=b["tiles"], n_tiles=b["n_tiles"], max_tiles=H * -(-T // L.tn), status=self.status)
+        ops.tc_linear(lw.w_uk_t, b["q_act"], lat["q"], rows=H * L.cap, **per)
+        common = dict(T=T, ldt=L.cap, n_seq=sh.n_seq, H=H, rank_pad=rp, scale=a.softmax_scale, status=self.status)
+        if self.f32 or rp > 512 or H > 128:
+            ops.latent_attention_simt(lat["q"], self.kv[r], md["page_table"], md["kv_len"], md["q_start"], md["q_len"], gate, lat["o"], **common)
+        else:
+            po = pml = None
+            if sh.attn_splits > 1:
+                need = sh.attn_splits * T * H
+                if getattr(self, "mla_part_o", None) is None or self.mla_part_o.numel() < need * rp or self.mla_part_ml.numel() < need * 2:
+                    if getattr(self, "mla_part_o", None) is not None:
+                        self.graphs.clear()            # captured steps hold the old scratch
+                        self.census.invalidate()
+                    self.mla_part_o = torch.empty(need * self.row, dtype=torch.float32, device=self.device)
+                    self.mla_part_ml = torch.empty(need * 2, dtype=torch.float32, device=self.device)
+                po, pml = self.mla_part_o, self.mla_part_ml
+                self.launches_per_step += 1
+            ops.latent_attention(lat["q"], self.kv_tmaps[r], md["page_table"], md["kv_len"], md["q_start"], md["q_len"], gate, lat["o"], max_q_len=sh.max_q_len,
+                                 n_splits=sh.attn_splits, part_o=po, part_ml=pml, **common)
+        ops.tc_linear(lw.w_uv, lat["o_act"], b["o"], rows=H * L.cap, token_major=(L.cap, a.v_head_dim), **per)
+        self.launches_per_step += 3
+
+    def _experts(self, m, lw: StackLayer, L: StackLane, e: dict, T: int):
+        E, k = m.n_experts, m.top_k
+        sel = (e["logits"], None, e["idx"], e["wts"], T, k, m.scoring, m.normalize, m.route_scale, m.n_group, m.topk_group)
+        if T * k <= 1024:
+            ops.router_select_pack(*sel, e["src"], e["slot"], e["counts"], e["offsets"], e["tiles"], e["n_tiles"], e["n_rows"], 0, E, e["tn"], e["max_tiles"],
+                                   group_score=m.group_score)
+        else:
+            ops.router_select(*sel, group_score=m.group_score)
+            ops.route_pack(e["idx"], e["src"], e["slot"], e["counts"], e["offsets"], e["tiles"], e["n_tiles"], e["n_rows"], T, k, 0, E, e["tn"], e["max_tiles"])
+            self.launches_per_step += 1
+        rows = T * k
+        call("cuteafd_gather_rows", ptr(L.xn), ptr(e["src"]), ptr(e["n_rows"]), ptr(e["xs"]), rows, self.Wp * L.xn.element_size() // 2, stream())
+        tiles = dict(tiles=e["tiles"], n_tiles=e["n_tiles"], max_tiles=min(e["max_tiles"], E + rows // e["tn"] + 1), status=self.status)
+        ops.tc_linear(lw.w_up, e["xs_act"], e["h1"], rows=rows, act="relu2", **tiles)
+        ops.tc_linear(lw.w_down, e["h1_act"], e["y"], rows=rows, **tiles)
+        self.launches_per_step += 4
+
+    # ------------------------------------------------------------------ prefill chunks: attention over the expanded context
+    def _expands(self, a, sh: StepShape) -> bool:
+        """Chunks whose longest query run fills a 128-row tile expand the context into per-head keys and values (see `MlaEngine`)."""
+        if self.f32 or not self.PREFILL_MIN_Q or sh.max_q_len < self.PREFILL_MIN_Q or sh.uniform or a.head_dim > 192 or a.v_head_dim > 128:
+            return False
+        if torch.cuda.is_current_stream_capturing():
+            return False
+        rows = sum(-(-n // 64) * 64 for n in self.mh["kv_len"][:sh.n_seq].tolist()) + 64
+        return rows * (up(a.kv_lora_rank, 64) + a.n_heads * (up(a.head_dim, 64) + up(a.v_head_dim, 64))) * 2 <= self.PREFILL_MAX_BYTES
+
+    def _pf_buffers(self, rows: int, rp: int, width: int):
+        """Context rows and their expansion (zero-filled: rows no gather ever wrote are multiplied by zero probabilities)."""
+        cap, lat, act = self._pf.get(("lat", rp), (0, None, None))
+        if rows + 64 > cap:
+            cap = max(1024, 1 << (rows + 64 - 1).bit_length())
+            lat = torch.zeros(cap, rp, dtype=torch.bfloat16, device=self.device)
+            act = ActBuffer(KIND_BF16, cap, rp, 256, lat, ops.encode_tmap(lat, 256))
+            self._pf[("lat", rp)] = (cap, lat, act)
+        kcap, kvb = self._pf.get(("kvb", width), (0, None))
+        if kcap < cap:
+            kvb = torch.zeros(cap, width, dtype=torch.bfloat16, device=self.device)
+            self._pf[("kvb", width)] = (cap, kvb)
+        return cap, lat, act, kvb
+
+    def _prefill(self, r: int, a, lw: StackLayer, L: StackLane, b: dict, gate, sh: StepShape):
+        T, md, H, n_seq = sh.T, self.md, a.n_heads, sh.n_seq
+        rp, dp, dvp = up(a.kv_lora_rank, 64), up(a.head_dim, 64), up(a.v_head_dim, 64)
+        kv, rows = self._ctx_plan(sh)
+        cap, lat, act, kvb = self._pf_buffers(rows, rp, H * (dp + dvp))
+        st = ptr(self.status)
+        call("cuteafd_latent_gather_ctx", ptr(self.kv[r]), ptr(md["page_table"]), ptr(self._pf_starts), ptr(md["kv_len"]), ptr(lat), n_seq, max(kv),
+             md["page_table"].shape[1], self.kv.shape[1], cap, rp, self.row, st, stream())
+        ops.tc_linear(lw.ensure_kvb(), act, kvb, rows=rows, status=self.status)
+        call("cuteafd_latent_prefill_attention", ptr(b["q"]), ptr(kvb), cap, ptr(self._pf_starts), ptr(md["kv_len"]), ptr(md["q_start"]), ptr(md["q_len"]),
+             ptr(gate), ptr(b["o"]), T, L.cap, n_seq, sh.max_q_len, H, dp, dvp, a.v_head_dim, b["o"].stride(0), a.softmax_scale, st, stream())
+        self.launches_per_step += 3

@@ -391,19 +391,7 @@ class MlaEngine(Engine):
         attention (`mla_prefill_kernel`), output token-major in b["o_tok"].  Reference: glm_mla_prefill.cu:123-960."""
         a, Hl, dev = self.spec.attn, self.heads_local, self.device
         n_seq, md = sh.n_seq, self.md
-        kv = tuple(self.mh["kv_len"][:n_seq].tolist())
-        plan = getattr(self, "_pf_plan", None)
-        if plan is None or plan[0] != kv:
-            starts, tot = [], 0
-            for n in kv:
-                starts.append(tot)
-                tot += -(-n // 64) * 64
-            host = torch.tensor(starts, dtype=torch.int32).pin_memory()
-            if getattr(self, "_pf_starts", None) is None or self._pf_starts.numel() < n_seq:
-                self._pf_starts = torch.zeros(max(n_seq, self.max_seqs), dtype=torch.int32, device=dev)
-            self._pf_starts[:n_seq].copy_(host, non_blocking=True)
-            self._pf_plan = plan = (kv, tot, host)
-        rows = plan[1]
+        kv, rows = self._ctx_plan(sh)
         cap = getattr(self, "_pf_cap", 0)
         if rows + 64 > cap:                       # zero-filled: rows no gather ever wrote are multiplied by zero probabilities
             cap = max(1024, 1 << (rows + 64 - 1).bit_length())
@@ -420,6 +408,24 @@ class MlaEngine(Engine):
         scale = (a.qk_nope_head_dim + a.qk_rope_head_dim) ** -0.5
         call("cuteafd_mla_prefill_attention", ptr(q_nope), ptr(b["q_rope"]), ptr(self._pf_kvb), ptr(self._pf_lat), self._pf_cap, ptr(self._pf_starts),
              ptr(md["kv_len"]), ptr(md["q_start"]), ptr(md["q_len"]), ptr(b["o_tok"]), sh.T, n_seq, sh.max_q_len, Hl, scale, st, stream())
+
+    def _ctx_plan(self, sh: StepShape) -> tuple:
+        """Where each sequence's context rows go in the contiguous buffers of the expanding prefill path: ((context lengths), total rows);
+        the starts (whole 64-row pages each) are copied to `_pf_starts` when the lengths change."""
+        n_seq, dev = sh.n_seq, self.device
+        kv = tuple(self.mh["kv_len"][:n_seq].tolist())
+        plan = getattr(self, "_pf_plan", None)
+        if plan is None or plan[0] != kv:
+            starts, tot = [], 0
+            for n in kv:
+                starts.append(tot)
+                tot += -(-n // 64) * 64
+            host = torch.tensor(starts, dtype=torch.int32).pin_memory()
+            if getattr(self, "_pf_starts", None) is None or self._pf_starts.numel() < n_seq:
+                self._pf_starts = torch.zeros(max(n_seq, self.max_seqs), dtype=torch.int32, device=dev)
+            self._pf_starts[:n_seq].copy_(host, non_blocking=True)
+            self._pf_plan = plan = (kv, tot, host)
+        return kv, plan[1]
 
     def _attn_in_gs(self, lw):
         return lw.mla.wkv_a.inv_act_gs

@@ -16,12 +16,13 @@ from .native import call, ptr, stream
 
 KIND_BF16, KIND_NVFP4, KIND_MXFP4, KIND_FP8B = 0, 1, 2, 3      # FP8B: E4M3 with fp32 scales per 128 x 128 (weights) / 1 x 128 (activations)
 KIND_W4A8 = 4      # MXFP4 weights x FP8 E4M3 activations, UE8M0 scales per 32 on both (tcgen05 kind::mxf8f6f4)
+KIND_F32 = 5       # plain fp32 operands (csrc/f32_linear.cu): the all-fp32 mode of an engine
 # MXFP4 expert weights run with MXFP4 activations (W4A4) unless CUTEAFD_MXFP4_ACT=fp8 selects FP8 activations (W4A8, the
 # reference's default expert arithmetic; also reachable per model as the "mxfp4_w4a8" format name)
 import os as _os
 MXFP4_ACT = _os.environ.get("CUTEAFD_MXFP4_ACT", "fp4")
 KIND_BY_NAME = {"bf16": KIND_BF16, "nvfp4": KIND_NVFP4, "mxfp4": KIND_W4A8 if MXFP4_ACT == "fp8" else KIND_MXFP4, "mxfp4_w4a4": KIND_MXFP4,
-                "mxfp4_w4a8": KIND_W4A8, "fp8_block128": KIND_FP8B}
+                "mxfp4_w4a8": KIND_W4A8, "fp8_block128": KIND_FP8B, "f32": KIND_F32}
 FP4_KINDS = (KIND_NVFP4, KIND_MXFP4)
 # activation formats the norm kernels (add_rmsnorm, moe_combine with the next layer's norm) can write in the same launch, and the
 # code the native side knows them by
@@ -29,6 +30,7 @@ FUSED_QUANT_KINDS = (KIND_NVFP4, KIND_MXFP4, KIND_FP8B)
 _QKIND = {KIND_NVFP4: 1, KIND_MXFP4: 2, KIND_FP8B: 3}
 EPI_BF16, EPI_BF16_RESIDUAL, EPI_F32 = 0, 1, 3
 SCORING = {"sigmoid": 0, "softmax": 1, "sqrtsoftplus": 2}
+GROUP_BY_MAX = 16      # added to the scoring code: a group of experts is ranked by its best member (default: the sum of its two best)
 
 
 def _chk(t: torch.Tensor, dtype, name: str):
@@ -134,6 +136,8 @@ class TcWeight:
         if kind == KIND_BF16:
             data = w.to(torch.bfloat16).to(device).contiguous()
             return TcWeight(kind, G, N, K, data, encode_tmap(data, 128))
+        if kind == KIND_F32:
+            return TcWeight(kind, G, N, K, w.to(torch.float32).to(device).contiguous(), None)
         if kind == KIND_FP8B:
             qs = [quant.fp8_block_quantize(w[g]) for g in range(G)]
             data = torch.stack([q for q, _ in qs]).to(device).contiguous()
@@ -177,6 +181,8 @@ class TcWeight:
         gen = torch.Generator(device=device).manual_seed(seed)
         lo, hi = groups if groups is not None else (0, G)
         cut = (lambda t: t[lo:hi].clone()) if (lo, hi) != (0, G) else (lambda t: t)
+        if kind == KIND_F32:
+            return TcWeight(kind, hi - lo, N, K, cut(torch.empty(G, N, K, dtype=torch.float32, device=device).normal_(0, std, generator=gen)), None)
         if kind == KIND_BF16:
             data = cut(torch.empty(G, N, K, dtype=torch.bfloat16, device=device).normal_(0, std, generator=gen))
             return TcWeight(kind, hi - lo, N, K, data, encode_tmap(data, 128))
@@ -207,7 +213,7 @@ class TcWeight:
     def dequantize(self) -> torch.Tensor:
         """fp32 [G, N, K] on CPU, without the activation scale folded into alpha (test helper)."""
         from ..ref import quant
-        if self.kind == KIND_BF16:
+        if self.kind in (KIND_BF16, KIND_F32):
             return self.data.float().cpu()
         if self.kind == KIND_FP8B:
             return torch.stack([quant.fp8_block_dequantize(self.data[g].cpu(), self.sf[g].cpu()) for g in range(self.G)])
@@ -241,6 +247,8 @@ class ActBuffer:
         if kind == KIND_BF16:
             data = torch.zeros(rows, K, dtype=torch.bfloat16, device=device)
             return ActBuffer(kind, rows, K, tn, data, encode_tmap(data, tn))
+        if kind == KIND_F32:
+            return ActBuffer(kind, rows, K, tn, torch.zeros(rows, K, dtype=torch.float32, device=device), None)
         if kind == KIND_FP8B:    # E4M3 bytes + one fp32 scale per row and 128 channels
             data = torch.zeros(rows, K, dtype=torch.uint8, device=device)
             return ActBuffer(kind, rows, K, tn, data, encode_tmap(data, tn), torch.zeros(rows, -(-K // 128), dtype=torch.float32, device=device))
@@ -269,14 +277,17 @@ def pick_tn(rows: int, swiglu: bool = False) -> int:
 
 
 _SPLITK_WS: dict = {}
+_SPLITK_KEEP: list = []        # outgrown scratch stays allocated: captured graphs still point at it
 
 
 def _splitk_scratch(device, n_float: int, n_cnt: int):
     key = str(device)
     ws, cnt = _SPLITK_WS.get(key, (None, None))
     if ws is None or ws.numel() < n_float:
+        _SPLITK_KEEP.append(ws)
         ws = torch.empty(max(n_float, 1 << 22), dtype=torch.float32, device=device)
     if cnt is None or cnt.numel() < n_cnt:
+        _SPLITK_KEEP.append(cnt)
         cnt = torch.zeros(max(n_cnt, 1 << 16), dtype=torch.int32, device=device)
     _SPLITK_WS[key] = (ws, cnt)
     return ws, cnt
@@ -285,7 +296,8 @@ def _splitk_scratch(device, n_float: int, n_cnt: int):
 def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | None = None, w_up: TcWeight | None = None,
               residual: torch.Tensor | None = None, tiles: torch.Tensor | None = None, n_tiles: torch.Tensor | None = None,
               max_tiles: int = 0, splits: int = 1, status: torch.Tensor | None = None, max_ctas: int = 0,
-              quant_out: ActBuffer | None = None, inv_gs_out: torch.Tensor | None = None, peer: dict | None = None) -> torch.Tensor | None:
+              quant_out: ActBuffer | None = None, inv_gs_out: torch.Tensor | None = None, peer: dict | None = None, act: str | None = None,
+              token_major: tuple | None = None) -> torch.Tensor | None:
     """y[rows, N] = x[rows, K] @ w[g]^T (per tile's expert g when `tiles` is given).  `w_up` switches on the fused
     SwiGLU epilogue (y = silu(x w^T) * (x w_up^T)).  y is bf16 (optionally + residual) or fp32.  `quant_out` (an FP4
     activation buffer of the operands' kind, K = N) also receives the output quantised for the GEMM that follows
@@ -293,7 +305,10 @@ def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | 
     `peer` fuses the hand-off to other GPUs into the epilogue: {"y": [device addresses of 1-2 peers' bf16 buffers], "ld": row
     pitch in elements, "row_map": int32 tensor or None (row r lands in row_map[r]), "flags": [peer flag addresses],
     "ctl": control block tensor, "done": zeroed uint32 counter tensor}; the flags are released with the step number
-    once the whole output has been stored (y may be None when only the peers need the result)."""
+    once the whole output has been stored (y may be None when only the peers need the result).
+    `act="relu2"`: squared ReLU on the output (an expert without a gate projection).  `token_major=(rows per group, columns per group)`:
+    a GEMM grouped over the heads of head-major operands (operand row = head * rows per group + token) writes head g's N columns of
+    output row `token` at column g * columns per group."""
     rows = x.rows if rows is None else rows
     if w.kind != x.kind or w.K != x.K:
         raise ValueError("tc_linear: operand kinds / K differ")
@@ -309,6 +324,13 @@ def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | 
         call("cuteafd_fp8_linear", x.tn, ptr(w.tmap), ptr(x.tmap), ptr(w.sf), ptr(x.sf), ptr(y), ptr(residual), y.stride(0), rows, w.N, w.K,
              epi, splits, ptr(status), stream())
         return y
+    if w.kind == KIND_F32:
+        if w_up is not None or residual is not None or quant_out is not None or peer is not None or y is None or y.dtype != torch.float32:
+            raise ValueError("tc_linear: the fp32 kernel has a plain fp32 output only")
+        gr, gc = token_major or (0, 0)
+        call("cuteafd_f32_linear", ptr(x.data), x.data.stride(0), ptr(w.data), ptr(y), y.stride(0), ptr(tiles), ptr(n_tiles), max_tiles, rows, w.N, w.K,
+             1 if act == "relu2" else 0, gr, gc, stream())
+        return y
     ws = cnt = None
     if splits > 1:
         n_items = -(-rows // x.tn)
@@ -319,6 +341,12 @@ def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | 
             raise ValueError("tc_linear: quant_out must be an FP4 buffer of the operands' kind with K = N")
         extra = native.TcExtra()
         extra.q_out, extra.sf_out, extra.ldsf_out, extra.inv_gs_out = ptr(quant_out.data), ptr(quant_out.sf), quant_out.sf.shape[1], ptr(inv_gs_out)
+    if act is not None or token_major is not None:
+        if act not in (None, "relu2"):
+            raise ValueError(f"tc_linear: unknown activation {act!r}")
+        extra = extra or native.TcExtra()
+        extra.act = 1 if act == "relu2" else 0
+        extra.grp_rows, extra.grp_cols = token_major or (0, 0)
     if peer is not None:
         ys, fl = list(peer["y"]), list(peer["flags"])
         extra = extra or native.TcExtra()
@@ -461,9 +489,13 @@ def router_logits(x, w: "TcWeight", logits, T: int):
 
 
 # ------------------------------------------------------------------ MoE control
-def router_select(logits, bias, idx, wts, T, k, scoring, normalize, route_scale, n_group=1, topk_group=1):
+def scoring_code(scoring: str, group_score: str = "top2") -> int:
+    return SCORING[scoring] | (GROUP_BY_MAX if group_score == "max" else 0)
+
+
+def router_select(logits, bias, idx, wts, T, k, scoring, normalize, route_scale, n_group=1, topk_group=1, group_score="top2"):
     _chk(logits, torch.float32, "logits")
-    call("cuteafd_router_select", ptr(logits), ptr(bias), ptr(idx), ptr(wts), T, logits.shape[1], k, SCORING[scoring],
+    call("cuteafd_router_select", ptr(logits), ptr(bias), ptr(idx), ptr(wts), T, logits.shape[1], k, scoring_code(scoring, group_score),
          1 if normalize else 0, route_scale, n_group, topk_group, stream())
 
 
@@ -471,13 +503,13 @@ _TICKETS: dict = {}
 
 
 def router_select_pack(logits, bias, idx, wts, T, k, scoring, normalize, route_scale, n_group, topk_group,
-                       src_token, slot_row, counts, offsets, tiles, n_tiles, n_rows, e_lo, e_hi, tn, max_tiles, src_route=None):
+                       src_token, slot_row, counts, offsets, tiles, n_tiles, n_rows, e_lo, e_hi, tn, max_tiles, src_route=None, group_score="top2"):
     """`router_select` followed by `route_pack` in one launch (the select block that finishes last packs)."""
     _chk(logits, torch.float32, "logits")
     dev = logits.device
     if dev not in _TICKETS:
         _TICKETS[dev] = torch.zeros(1, dtype=torch.int32, device=dev)
-    call("cuteafd_router_select_pack", ptr(logits), ptr(bias), ptr(idx), ptr(wts), T, logits.shape[1], k, SCORING[scoring],
+    call("cuteafd_router_select_pack", ptr(logits), ptr(bias), ptr(idx), ptr(wts), T, logits.shape[1], k, scoring_code(scoring, group_score),
          1 if normalize else 0, route_scale, n_group, topk_group, ptr(src_token), ptr(slot_row), ptr(counts), ptr(offsets),
          ptr(tiles), ptr(n_tiles), ptr(n_rows), e_lo, e_hi, tn, max_tiles, ptr(src_route), ptr(_TICKETS[dev]), stream())
 
@@ -669,3 +701,60 @@ def compress_pool(kv, scores, state, state_slot, q_start, q_len, pos0, out_start
     call("cuteafd_compress_pool", ptr(kv), ptr(scores), ptr(state), ptr(state_slot), ptr(q_start), ptr(q_len), ptr(pos0), ptr(out_start),
          ptr(norm_w), ptr(out), n_seq, max_blocks, kv.shape[1], ratio, eps, stream())
     return out
+
+
+# ------------------------------------------------------------------ layer stacks: row kernels between two matrix products
+def emit_arg(norm=None, xn=None, cat=None):
+    """What the row kernels below leave for the next product.  `norm` = (w, b, alpha) of a Dynamic Tanh, written to `xn`; `cat`: buffer
+    whose leading columns take the plain row."""
+    e = native.EmitArg()
+    if norm is not None:
+        e.w, e.b, e.alpha, e.xn, e.ldn = ptr(norm[0]), ptr(norm[1]), float(norm[2]), ptr(xn), xn.stride(0)
+    if cat is not None:
+        e.cat, e.ldc = ptr(cat), cat.stride(0)
+    return e
+
+
+def _f32(t) -> int:
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def stack_embed(tokens, positions, table, pos_table, x, x0, emit, T: int, *, f32: bool, status=None):
+    """x[t] = table[token] + pos_table[position] (fp32 rows); `x0`: view whose rows take the same values as matrix operand."""
+    _chk(tokens, torch.int32, "tokens"); _chk(table, torch.bfloat16, "table"); _chk(x, torch.float32, "x")
+    call("cuteafd_stack_embed", ptr(tokens), ptr(positions), ptr(table), ptr(pos_table), ptr(x), ptr(x0), x0.stride(0) if x0 is not None else 0, T,
+         x.shape[1], table.shape[0], pos_table.shape[0] if pos_table is not None else 0, 1 if f32 else 0, ctypes.byref(emit), ptr(status), stream())
+
+
+def stack_stream(x, emit, T: int, *, f32: bool, vec=None, src_rows=None):
+    """Rows x[t] (+ `vec`, written back), or the rows listed in `src_rows`, handed on by `emit`."""
+    _chk(x, torch.float32, "x")
+    call("cuteafd_stack_stream", ptr(x), ptr(vec), ptr(src_rows), T, x.shape[1], 1 if f32 else 0, ctypes.byref(emit), stream())
+
+
+def stack_combine(x, mix, ls1, y, slot_row, wts, ls2, emit, T: int, k: int):
+    """x += ls1 * mix + ls2 * sum over the token's k routes of wts * y[slot_row]; the new rows are handed on by `emit`."""
+    _chk(x, torch.float32, "x")
+    call("cuteafd_stack_combine", ptr(x), ptr(mix), ptr(ls1), ptr(y), ptr(slot_row), ptr(wts), ptr(ls2), T, x.shape[1], k, _f32(mix),
+         ctypes.byref(emit) if emit is not None else None, stream())
+
+
+def latent_prepare(proj, norm_w, slot_map, q, cache, gate, logits, tiles, n_tiles, *, T, ldt, H, d, r, rp, E, tn, eps, status=None):
+    """Splits the fused projection rows (queries | latent | gates | router logits, fp32): queries head-major [H, ldt, q.shape[-1]], the
+    RMS-normed latent into the paged cache, sigmoid gates, compact router logits, and the tile table of the per-head products."""
+    _chk(proj, torch.float32, "proj")
+    call("cuteafd_latent_prepare", ptr(proj), proj.stride(0), ptr(norm_w), ptr(slot_map), ptr(q), ptr(cache), ptr(gate), ptr(logits), ptr(tiles),
+         ptr(n_tiles), T, ldt, H, d, q.shape[-1], r, rp, cache.stride(0), cache.shape[0], E, tn, eps, _f32(q), ptr(status), stream())
+
+
+def latent_attention(q_lat, kv_map, page_table, kv_len, q_start, q_len, gate, out, *, T, ldt, n_seq, max_q_len, H, rank_pad, n_splits=1, part_o=None,
+                     part_ml=None, scale, status=None):
+    """Absorbed latent attention without positions over the paged cache (tcgen05); q_lat, out: head-major [H, ldt, rank_pad] bf16."""
+    call("cuteafd_latent_attention", ptr(q_lat), ptr(kv_map), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(gate), ptr(out), ptr(part_o),
+         ptr(part_ml), T, ldt, n_seq, max_q_len, H, rank_pad, page_table.shape[1], n_splits, float(scale), ptr(status), stream())
+
+
+def latent_attention_simt(q_lat, cache, page_table, kv_len, q_start, q_len, gate, out, *, T, ldt, n_seq, H, rank_pad, scale, status=None):
+    """The same on the ordinary cores: fp32 operands, latents wider than 512, more than 128 heads."""
+    call("cuteafd_latent_attention_simt", ptr(q_lat), ptr(cache), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(gate), ptr(out), T, ldt,
+         n_seq, H, rank_pad, cache.stride(0), page_table.shape[1], cache.shape[0], float(scale), _f32(q_lat), ptr(status), stream())

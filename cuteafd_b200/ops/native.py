@@ -100,6 +100,16 @@ _PROTOS = {
     "cuteafd_flag_pingpong": [P, P, C.c_uint, I, I, C.c_ulonglong, P, P, P],
     "cuteafd_dispatch_tok_push": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, C.c_uint, P, P],
     "cuteafd_combine_push_lanes": [P, P, P, P, P, P, P, I, I, I, I, I, I, C.c_uint, P, P],
+    "cuteafd_latent_attention": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
+    "cuteafd_tmap_encode_latent_rows": [P, P, U64, U64, U64],
+    "cuteafd_latent_prefill_attention": [P, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
+    "cuteafd_latent_gather_ctx": [P, P, P, P, P, I, I, I, L, L, I, I, P, P],
+    "cuteafd_latent_attention_simt": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
+    "cuteafd_latent_prepare": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P],
+    "cuteafd_stack_embed": [P, P, P, P, P, P, I, I, I, I, I, I, P, P, P],
+    "cuteafd_stack_stream": [P, P, P, I, I, I, P, P],
+    "cuteafd_stack_combine": [P, P, P, P, P, P, P, I, I, I, I, P, P],
+    "cuteafd_f32_linear": [P, I, P, P, I, P, P, I, I, I, I, I, I, I, P],
     "cuteafd_tc_linear": [I, I, I, P, P, P, P, P, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, P, P, P, I, P, P],
 }
 
@@ -117,7 +127,13 @@ class FlagWaitArg(C.Structure):
 class TcExtra(C.Structure):
     """Optional outputs of `cuteafd_tc_linear` (`CaTcExtra` of the C ABI)."""
     _fields_ = [("q_out", P), ("sf_out", P), ("inv_gs_out", P), ("ldsf_out", I), ("n_peer", I), ("peer_y", P * 2), ("peer_flag", P * 2),
-                ("peer_row_map", P), ("peer_ctl", P), ("peer_done", P), ("peer_ld", I), ("reserved", I)]
+                ("peer_row_map", P), ("peer_ctl", P), ("peer_done", P), ("peer_ld", I), ("act", I), ("grp_rows", I), ("grp_cols", I)]
+
+
+class EmitArg(C.Structure):
+    """What a row-producing kernel of a layer stack writes for the next matrix product (`CaEmit` of the C ABI): tanh(alpha x) w + b
+    into `xn`, and / or the plain row into `cat`."""
+    _fields_ = [("w", P), ("b", P), ("xn", P), ("cat", P), ("alpha", F), ("ldn", I), ("ldc", I), ("reserved", I)]
 
 
 def flag_wait(flags_ptr: int, n: int, stride: int, ctl: torch.Tensor, status: torch.Tensor | None, timeout_ns: int = 2_000_000_000) -> FlagWaitArg:

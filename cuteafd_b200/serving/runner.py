@@ -68,6 +68,7 @@ class EngineRunner:
         self._recurrent = bool(getattr(engine, "lin_layers", None))
         self._state_slot: dict = {}
         self._state_pos: dict = {}
+        self.last_lane = None             # the lane of the last step: `.logits` holds its rows that needed logits, in order
         self._deferred = None             # (step shape, [(state id, start position, rows)]) of a speculative step awaiting `commit`
         self._free_slots = list(range(getattr(engine, "max_seqs", 0)))[::-1] if self._recurrent else []
         self._tok_host = torch.zeros(max(64, max_rows), dtype=torch.int32)
@@ -164,7 +165,7 @@ class EngineRunner:
                        attn_splits=eng.attn_splits_for(len(rows), max_q, max(kv_len)) if decode_like else 1, uniform=uniform, defer_state=defer)
         if over_rows:
             eng.set_input_embeds(over_rows, torch.cat(over_vals) if len(over_vals) > 1 else over_vals[0])
-        lane = eng.run(sh, use_graph=decode_like and not over_rows)
+        lane = self.last_lane = eng.run(sh, use_graph=decode_like and not over_rows)
         pending = (sh, [(id(r.state), r.start_pos, len(r.tokens)) for r in rows]) if defer else None
         if self.keep_hidden:
             for r, qs, ql in zip(rows, q_start, q_len):

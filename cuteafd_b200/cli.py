@@ -95,7 +95,7 @@ def build_serving(a):
                             model_max_context=spec.max_context, weights_loaded=True)
         print(f"[serve] capacity: {cap.describe()}", file=sys.stderr)
         n_pages = cap.pool_pages
-    eng = build_engine(spec, weights, n_pages=n_pages, max_seqs=a.max_sequences, max_pages_per_seq=min(n_pages, min(a.max_context, spec.max_context) // 64 + 1))
+    eng = build_engine(spec, weights, n_pages=n_pages, max_seqs=a.max_sequences, max_pages_per_seq=min(n_pages, min(a.max_context, spec.max_context) // 64 + 2))
     pool = PagePool(n_pages)
     runner = attach_pool(EngineRunner(eng, max_rows=a.prefill_batch_tokens), pool)
     host = None
@@ -125,7 +125,7 @@ def build_serving(a):
                                    slice_mb=3 * spec.hidden * m.intermediate * per_weight / 2 ** 20)
     sched = Scheduler(runner, pool, max_seqs=a.max_sequences, prefill_chunk=a.prefill_batch_tokens, decode_share=a.decode_share,
                       prefix=prefix, drafter=drafter, max_draft=a.draft_limit, queue_limit=getattr(a, "http_queue", 64),
-                      queue_wait_s=getattr(a, "queue_wait_s", 0) or None, policy=policy)
+                      queue_wait_s=getattr(a, "queue_wait_s", 0) or None, policy=policy, max_context=spec.learned_positions or None)
     return spec, sched
 
 
@@ -341,6 +341,8 @@ def _golden_masters(model: str):
         raise SystemExit(f"golden windows need fp32 masters: give the tiny model or a snapshot directory, not {model!r}")
     from .loader.checkpoint import read_masters
     spec = spec_from_snapshot(model)
+    if spec.blocks:
+        raise SystemExit("golden windows are sealed from the oracle of the homogeneous families; compare a latent-attention stack with `cuteafd trace`")
     return spec, read_masters(model, spec)
 
 

@@ -94,6 +94,9 @@ def solve(spec: ModelSpec, world: int = 8, gpu_bytes: int = 180 * GIB, reserve_b
         for p in plans:
             if p.shortfall:
                 notes.append(f"rank {p.rank} ({p.role}) is short {p.shortfall / GIB:.1f} GiB")
+    if spec.blocks and dep.world > 1:
+        fits = False
+        notes.append("latent-attention stacks run on one GPU")
     if dep.ep and spec.moe.n_experts % dep.ep:
         notes.append(f"{spec.moe.n_experts} experts over {dep.ep} expert ranks: uneven ranges of "
                      f"{spec.moe.n_experts // dep.ep} or {spec.moe.n_experts // dep.ep + 1} experts")
@@ -106,6 +109,8 @@ def solve_stages(spec: ModelSpec, n_stages: int, gpu_bytes: int = 180 * GIB, res
     and the KV cache of those layers only; the first stage adds the embedding, the last one the head.  The pool is what the tightest
     stage can hold.  (Reference: cuteafd-loader/src/placement/residual.rs: layer ranges per device.)"""
     from ..parallel.pipeline import stage_ranges
+    if spec.blocks:
+        raise NotImplementedError("latent-attention stacks are not cut into layer ranges (a looped range would cross the cut)")
     a = spec.attn
     ranges = stage_ranges(spec.n_layers, n_stages, max(a.full_every or 1, a.linear_every or 1))
     wb = spec.weight_bytes()

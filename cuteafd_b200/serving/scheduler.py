@@ -99,11 +99,12 @@ class NgramDrafter:
 class Scheduler:
     def __init__(self, runner: ModelRunner, pool: PagePool, *, max_seqs: int = 16, prefill_chunk: int = 4096, decode_share: float = 0.2,
                  prefix: PrefixCache | None = None, drafter: Drafter | None = None, policy: DraftPolicy | None = None,
-                 max_draft: int = 3, queue_limit: int = 64, queue_wait_s: float | None = None):
+                 max_draft: int = 3, queue_limit: int = 64, queue_wait_s: float | None = None, max_context: int | None = None):
         self.runner, self.pool = runner, pool
         self.max_seqs, self.prefill_chunk, self.decode_share = max_seqs, prefill_chunk, decode_share
         self.prefix = prefix
         self.drafter, self.policy, self.max_draft = drafter, policy or SimpleDraftPolicy(max_draft), max_draft
+        self.max_context = max_context                        # positions the model has (None: no limit): longer prompts are refused, outputs cut
         self.queue: deque[Request] = deque()
         self.queue_limit = queue_limit
         self.queue_wait_s = queue_wait_s                      # admission wait budget: a request queued longer than this is answered "busy"
@@ -126,6 +127,12 @@ class Scheduler:
         if self.fatal:
             self._finish_unadmitted(req, "unavailable: " + self.fatal)
             return False
+        if self.max_context is not None:
+            if len(req.prompt) > self.max_context:
+                self.stats["rejected"] += 1
+                self._finish_unadmitted(req, f"error: prompt of {len(req.prompt)} tokens exceeds the model's context of {self.max_context}")
+                return False
+            req.max_tokens = min(req.max_tokens, self.max_context - len(req.prompt) + 1)      # the last token is chosen, not run
         if len(self.queue) >= self.queue_limit:
             self.stats["rejected"] += 1
             self._finish_unadmitted(req, "queue full")

@@ -42,7 +42,8 @@ class StackLane(Lane):
         self.eng, self.cap, self.dev = eng, cap, eng.device
         self.dt = torch.float32 if eng.f32 else torch.bfloat16
         self.kind = KIND_F32 if eng.f32 else KIND_BF16
-        self.tn = pick_tn(min(cap, int(os.environ.get("CUTEAFD_TN", "128"))))
+        # no product of these layers pairs two weight tiles, so 256-row token tiles keep both accumulators: prompt-sized lanes take them
+        self.tn = pick_tn(min(cap, int(os.environ.get("CUTEAFD_TN", "256" if cap >= 1024 else "128"))))
         Wp = eng.Wp
         self.x = torch.zeros(cap, Wp, dtype=torch.float32, device=self.dev)
         self.xn, self.xn_act = self._operand(cap, Wp)
@@ -101,8 +102,9 @@ class StackLane(Lane):
 
         def make():
             rows = cap * k
-            per = max(1, math.ceil(rows / E) * 2)
-            tn = pick_tn(min(per, int(os.environ.get("CUTEAFD_TNG", "32"))))
+            # rows per expert of a full lane: whole 256-row tiles where they fill, else about twice the mean
+            mean = max(1, math.ceil(rows / E))
+            tn = pick_tn(min(mean if mean >= 256 else min(2 * mean, 128), int(os.environ.get("CUTEAFD_TNG", "256"))))
             i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=self.dev)
             xs, xs_act = self._operand(rows, self.eng.Wp, tn)
             h1, h1_act = self._operand(rows, up(ff, 8), tn)

@@ -103,12 +103,14 @@ def build_serving(a):
         from .serving.hostcache import attach_host_tier
         host = attach_host_tier(eng, max(0.0, a.host_cache_gib - a.host_cache_headroom_gib), min_tokens=a.host_cache_min_tokens)
     prefix = PrefixCache(pool, max_entries=a.prefix_cache_entries, min_tokens=a.prefix_cache_min_tokens, host=host)
-    recurrent = bool(spec.attn.linear_every)
+    recurrent = bool(spec.attn.linear_every) or spec.stack == "hybrid"
     if recurrent:
-        # gated delta-rule layers carry a recurrent state per sequence: a request cannot resume from cached pages (drafted steps are
-        # fine: they leave the state alone and the accepted rows are replayed into it)
+        # recurrent layers carry a state per sequence: a request cannot resume from cached pages (drafted steps are fine: they leave the
+        # state alone and the accepted rows are replayed into it, or the engine keeps the last positions' states)
         prefix = None
-        print(f"[serve] {spec.name}: linear-attention layers - the prefix cache is off", file=sys.stderr)
+        print(f"[serve] {spec.name}: recurrent layers - the prefix cache is off", file=sys.stderr)
+    depth = getattr(eng, "state_depth", 0)
+    max_draft = min(a.draft_limit, depth - 1) if depth else a.draft_limit
     drafter = None
     if a.draft == "ngram":
         drafter = NgramDrafter()
@@ -124,7 +126,7 @@ def build_serving(a):
         policy = OnlineDraftPolicy(max(a.draft_limit, 1), n_experts=m.n_experts, top_k=m.top_k,
                                    slice_mb=3 * spec.hidden * m.intermediate * per_weight / 2 ** 20)
     sched = Scheduler(runner, pool, max_seqs=a.max_sequences, prefill_chunk=a.prefill_batch_tokens, decode_share=a.decode_share,
-                      prefix=prefix, drafter=drafter, max_draft=a.draft_limit, queue_limit=getattr(a, "http_queue", 64),
+                      prefix=prefix, drafter=drafter, max_draft=max_draft, queue_limit=getattr(a, "http_queue", 64),
                       queue_wait_s=getattr(a, "queue_wait_s", 0) or None, policy=policy, max_context=spec.learned_positions or None)
     return spec, sched
 
@@ -342,7 +344,7 @@ def _golden_masters(model: str):
     from .loader.checkpoint import read_masters
     spec = spec_from_snapshot(model)
     if spec.blocks:
-        raise SystemExit("golden windows are sealed from the oracle of the homogeneous families; compare a latent-attention stack with `cuteafd trace`")
+        raise SystemExit("golden windows are sealed from the oracle of the homogeneous families; compare a layer stack with `cuteafd trace`")
     return spec, read_masters(model, spec)
 
 
@@ -610,7 +612,7 @@ def main(argv=None) -> int:
     _gateway_args(p)
     p.add_argument("--draft-limit", type=int, default=3); p.add_argument("--api-key-file"); p.add_argument("--model-id")
     p.add_argument("--layers", type=int, default=0, help="debug: run only the first N layers of a named shape")
-    p.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="float32: weights, activations and cache in fp32 (latent-attention stacks only)")
+    p.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="float32: weights, activations and cache in fp32 (layer stacks only)")
     p.add_argument("--n-micro", type=int, default=0, help="multi-GPU: micro-batches the attention ranks keep in flight (0 = the layout's default)")
     p.add_argument("--vision", default="auto", help="auto (tower of the snapshot, if it has one) | off | random[:DEPTH]")
     p.add_argument("--gpu-occupancy-percent", type=int, default=0,

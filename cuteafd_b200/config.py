@@ -17,7 +17,9 @@ from typing import Optional
 
 @dataclass(frozen=True)
 class AttentionSpec:
-    kind: str = "gqa"              # "gqa" | "mla" | "latent" (latent attention without positions; per layer, see BlockSpec)
+    # "gqa" | "mla" | per layer of a stack (BlockSpec): "latent" (latent attention without positions), "conv_gqa" (grouped-query attention
+    # whose projections pass a short causal convolution)
+    kind: str = "gqa"
     n_heads: int = 8
     n_kv_heads: int = 2
     head_dim: int = 32
@@ -56,6 +58,13 @@ class AttentionSpec:
     # (0 = head_dim ** -0.5), `out_gate` multiplies each head's output by a sigmoid of the layer's input.
     scale: float = 0.0
     out_gate: bool = False
+    # Kind "conv_gqa": head_dim, v_head_dim, window, qk_norm and scale as above, `conv_taps` of the convolution on q, k and v, the first
+    # `rope_dims` dimensions of a head rotated (interleaved pairs, `rope_theta`, `rope_scaling`), and with kv_from >= 0 the keys and values
+    # of that layer instead of own ones.
+    conv_taps: int = 1
+    rope_dims: int = 0
+    rope_scaling: Optional["RopeScaling"] = None
+    kv_from: int = -1
 
     @property
     def softmax_scale(self) -> float:
@@ -74,7 +83,19 @@ class AttentionSpec:
             return self.kv_lora_rank + self.qk_rope_head_dim
         if self.kind == "latent":
             return self.kv_lora_rank
+        if self.kind == "conv_gqa":
+            return 0 if self.kv_from >= 0 else self.n_kv_heads * (self.head_dim + self.v_head_dim)
         return 2 * self.n_kv_heads * self.head_dim
+
+
+@dataclass(frozen=True)
+class RopeScaling:
+    """YaRN: frequencies that turn fewer than `slow` times over `original` positions are divided by `factor`, those that turn more than
+    `fast` times stay, with a linear ramp over the pairs between; cosine and sine grow by 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
 
 
 @dataclass(frozen=True)
@@ -111,10 +132,32 @@ class QuantSpec:
 
 
 @dataclass(frozen=True)
+class RecurrentSpec:
+    """A recurrent mixer.  "rglru": two branches of `width` channels, one gated by GELU, the other through a convolution of `conv_taps` and a
+    real-gated linear recurrence whose two gates are block-diagonal (`blocks` square blocks)."""
+    kind: str = "rglru"
+    width: int = 256
+    blocks: int = 1
+    conv_taps: int = 4
+
+
+@dataclass(frozen=True)
+class DenseFfnSpec:
+    """A dense feed-forward.  "clamped_glu": gate g = min(., limit), linear half u clamped to [-limit, limit], g sigmoid(1.702 g) (u + 1);
+    biases on all three projections."""
+    intermediate: int
+    limit: float
+    activation: str = "clamped_glu"
+
+
+@dataclass(frozen=True)
 class BlockSpec:
-    """One layer of a stack whose layers differ: its attention and its feed-forward (None = the layer has none)."""
-    attn: AttentionSpec = field(default_factory=lambda: AttentionSpec(kind="latent"))
+    """One layer of a stack whose layers differ: its mixer (attention, or a recurrent one) and its feed-forward (routed experts, dense, or
+    neither: the layer has none)."""
+    attn: Optional[AttentionSpec] = field(default_factory=lambda: AttentionSpec(kind="latent"))
     moe: Optional[MoESpec] = None
+    rec: Optional[RecurrentSpec] = None
+    ffn: Optional[DenseFfnSpec] = None
 
 
 @dataclass(frozen=True)
@@ -151,11 +194,26 @@ class ModelSpec:
     init_std: float = 0.02
     tie_embeddings: bool = False
     max_context: int = 1 << 20
-    # Stacks of unequal layers (`blocks` non-empty; `attn` / `moe` above then describe the first layer of their kind): parallel layers
-    # (one norm, attention and feed-forward read it, both scaled per channel and added to an fp32 residual), Dynamic Tanh for a norm.
+    # Stacks of unequal layers (`blocks` non-empty; `attn` / `moe` above then describe the first layer of their kind), over an fp32 residual.
+    # "latent" stacks: parallel layers (one norm, attention and feed-forward read it, both scaled per channel and added), Dynamic Tanh for a
+    # norm.  "hybrid" stacks: windowed attention and recurrent layers, RMS norms in front of and behind every sub-layer, whose result is
+    # added `residual_mult` times; logits bounded by `logit_softcap` (0 = not).
     blocks: tuple = ()
+    residual_mult: float = 1.0
+    logit_softcap: float = 0.0
     loop: Optional[LoopSpec] = None
     learned_positions: int = 0      # rows of the learned position table (0 = none); also the longest context
+
+    @property
+    def stack(self) -> str:
+        """Which kind of stack `blocks` describes: "latent", "hybrid", or "" for models without blocks."""
+        if not self.blocks:
+            return ""
+        return "latent" if all(b.attn is not None and b.attn.kind == "latent" for b in self.blocks) else "hybrid"
+
+    def kv_layers(self) -> list:
+        """Layers of a hybrid stack that keep keys and values of their own."""
+        return [i for i, b in enumerate(self.blocks) if b.attn is not None and b.attn.kv_from < 0]
 
     def layer_runs(self) -> list:
         """[(layer, pass index where a pass of the loop opens with this run, else None)] in the order the layers run."""
@@ -212,6 +270,8 @@ class ModelSpec:
 
     def attn_params(self, attn: Optional[AttentionSpec] = None) -> int:
         a, h = attn or self.attn, self.hidden
+        if a.kind == "conv_gqa":
+            return h * (a.n_heads * (a.head_dim + a.v_head_dim) + a.kv_token_elems)
         if a.kind == "latent":
             return (h * (a.n_heads * a.head_dim + a.kv_lora_rank + (a.n_heads if a.out_gate else 0)) +
                     a.n_heads * (a.head_dim + a.v_head_dim) * a.kv_lora_rank + a.n_heads * a.v_head_dim * h)
@@ -228,6 +288,12 @@ class ModelSpec:
 
     def weight_bytes(self) -> dict:
         """Bytes per category for the whole model (planner input)."""
+        if self.stack == "hybrid":
+            db = self.bits(self.quant.dense) / 8
+            rec = sum(3 * self.hidden * b.rec.width + 2 * b.rec.width ** 2 // b.rec.blocks for b in self.blocks if b.rec is not None)
+            return {"routed_experts": 0.0, "shared_experts": 0.0, "router": 0.0, "embed_head": self.vocab * self.hidden * (2 + db),
+                    "dense_ffn": sum(3 * self.hidden * b.ffn.intermediate for b in self.blocks if b.ffn is not None) * db,
+                    "attention": (rec + sum(self.attn_params(b.attn) for b in self.blocks if b.attn is not None)) * db}
         if self.blocks:
             eb, db = self.bits(self.quant.experts) / 8, self.bits(self.quant.dense) / 8
             ffs = [b.moe for b in self.blocks if b.moe is not None]
@@ -247,8 +313,26 @@ class ModelSpec:
         return {"routed_experts": routed, "shared_experts": shared, "dense_ffn": dense_ffn,
                 "attention": attn, "router": router, "embed_head": embed}
 
+    def kv_row_elems(self) -> int:
+        """Elements of a cached token's row in a hybrid stack: the widest layer's key heads, then its value heads."""
+        up = lambda n: -(-n // 64) * 64
+        return max((b.attn.n_kv_heads * (up(b.attn.head_dim) + up(b.attn.v_head_dim)) for b in self.blocks if b.attn is not None and b.attn.kv_from < 0), default=0)
+
+    def state_bytes_per_seq(self, depth: int = 8) -> int:
+        """Bytes of one sequence's state slot in a hybrid stack (`engine.hybrid_stack`): convolution inputs and recurrent states of the last
+        positions, `depth` of which can be taken back."""
+        eb, n = 2 if self.quant.dense == "bf16" else 4, 0
+        for b in self.blocks:
+            if b.rec is not None:
+                n += b.rec.width * ((b.rec.conv_taps - 1 + depth) * eb + (depth + 1) * 4)
+            else:
+                n += (b.attn.n_heads * b.attn.head_dim + b.attn.kv_token_elems) * (b.attn.conv_taps - 1 + depth) * eb
+        return n
+
     def kv_bytes_per_token(self) -> float:
         per = {"fp8": 1.0, "f32": 4.0}.get(self.quant.kv, 2.0)
+        if self.stack == "hybrid":  # one row width for every layer with keys of its own, heads in whole 64-element chunks
+            return len(self.kv_layers()) * self.kv_row_elems() * per
         if self.blocks:             # one row width for every layer run (the widest latent, in whole 64-element chunks)
             return len(self.layer_runs()) * max(-(-b.attn.kv_token_elems // 64) * 64 for b in self.blocks) * per
         return self.n_layers * self.attn.kv_token_elems * per
@@ -333,6 +417,23 @@ def bedovik_spec(n_layers: int = 8, heads: int = 32, hidden: int = 4096, rank: i
                      loop=LoopSpec(lo, hi, loop_times) if loop_times > 1 and hi > lo else None, learned_positions=65536, max_context=65536)
 
 
+def tudilix_spec(n_layers: int = 12, hidden: int = 4096, heads: int = 32, kv_heads: int = 4, ff: int = 12288, window: int = 2048, blocks: int = 16) -> ModelSpec:
+    """Tudilix at the size of a real model's layers (synthetic weights): two recurrent layers, then one windowed-attention layer with a dense
+    feed-forward, every second attention layer on the keys and values of the one before it."""
+    rec = BlockSpec(None, rec=RecurrentSpec(width=hidden, blocks=blocks, conv_taps=4))
+    attn = AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, window=window, qk_norm=True, conv_taps=4,
+                         rope_dims=64, rope_scaling=RopeScaling(8.0, 8192, 32.0, 1.0))
+    layers, last = [], -1
+    for i in range(n_layers):
+        if i % 3 != 2:
+            layers.append(rec)
+            continue
+        layers.append(BlockSpec(dataclasses.replace(attn, kv_from=last), ffn=DenseFfnSpec(ff, 7.0)))
+        last = i if last < 0 else -1
+    return ModelSpec(name="tudilix-shape", family="tudilix", vocab=65536, hidden=hidden, n_layers=n_layers, rms_eps=1e-6, attn=attn, moe=MoESpec(n_experts=0, n_shared=0),
+                     quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(layers), residual_mult=0.5, logit_softcap=30.0)
+
+
 NAMED_SPECS = {
     "tiny": tiny_spec,
     "hybrid-gdn": hybrid_gdn_spec,
@@ -341,6 +442,7 @@ NAMED_SPECS = {
     "deepseek-v32": deepseek_v32_spec,
     "qwen3-235b": qwen3_235b_spec,
     "bedovik": bedovik_spec,
+    "tudilix": tudilix_spec,
     "ep-microbench": ep_microbench_spec,
 }
 
@@ -367,6 +469,7 @@ FAMILY_BY_ARCH = {
     "MixtralForCausalLM": "mixtral",
     "Qwen3NextForCausalLM": "hybrid_linear",
     "Bedovik": "bedovik",
+    "Tudilix": "tudilix",
 }
 
 
@@ -420,6 +523,46 @@ def _bedovik_config(cfg: dict) -> ModelSpec:
                      quant=QuantSpec(), blocks=tuple(blocks), loop=loop, learned_positions=n_pos, max_context=n_pos)
 
 
+def _tudilix_config(cfg: dict) -> ModelSpec:
+    """`config.json` of the Tudilix design: every layer names its mixer (windowed attention or a gated linear recurrence) and its
+    feed-forward with their sizes."""
+    blocks = []
+    for i, layer in enumerate(cfg["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        attn = rec = ffn = None
+        if layer["type"] == "rglru":
+            rec = RecurrentSpec(width=int(m["width"]), blocks=int(m["blocks"]), conv_taps=int(m["conv"]))
+            if rec.width % rec.blocks:
+                raise ValueError(f"layer {i}: {rec.width} channels in {rec.blocks} blocks")
+        elif layer["type"] == "attention":
+            rot = m.get("rot") or {"dims": 0, "base": 1e4}
+            sc = rot.get("scaling")
+            attn = AttentionSpec(kind="conv_gqa", n_heads=int(m["heads"]), n_kv_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]),
+                                 scale=float(m["scale"]), window=int((m.get("mask") or {}).get("size") or 0), qk_norm=True, conv_taps=int(m["conv"]),
+                                 rope_dims=int(rot["dims"]), rope_theta=float(rot["base"]),
+                                 rope_scaling=RopeScaling(*(float(sc[k]) for k in ("factor", "original", "fast", "slow"))) if sc else None,
+                                 kv_from=int(m["kv_from"]) if m.get("kv_from") is not None else -1)
+            if attn.n_heads % attn.n_kv_heads:
+                raise ValueError(f"layer {i}: {attn.n_heads} query heads over {attn.n_kv_heads} key heads")
+            if attn.rope_dims % 2 or attn.rope_dims > attn.head_dim:
+                raise ValueError(f"layer {i}: {attn.rope_dims} rotated dimensions of {attn.head_dim}")
+            if attn.kv_from >= 0:
+                src = blocks[attn.kv_from].attn if attn.kv_from < i else None
+                if src is None or src.kv_from >= 0 or (src.n_kv_heads, src.head_dim, src.v_head_dim) != (attn.n_kv_heads, attn.head_dim, attn.v_head_dim):
+                    raise ValueError(f"layer {i}: layer {attn.kv_from} has no keys and values of its shape")
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {layer['type']!r}")
+        if mlp is not None:
+            if mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            ffn = DenseFfnSpec(int(mlp["ff"]), float(mlp["limit"]))
+        blocks.append(BlockSpec(attn, rec=rec, ffn=ffn))
+    first = next((b.attn for b in blocks if b.attn is not None), AttentionSpec(kind="conv_gqa", n_heads=1, n_kv_heads=1))
+    return ModelSpec(name="tudilix", family="tudilix", vocab=int(cfg["vocab"]), hidden=int(cfg["width"]), n_layers=len(blocks), rms_eps=float(cfg["norm"]["eps"]),
+                     attn=first, moe=MoESpec(n_experts=0, n_shared=0), quant=QuantSpec(), blocks=tuple(blocks), residual_mult=float(cfg["residual_mult"]),
+                     logit_softcap=float(cfg.get("logit_softcap") or 0.0))
+
+
 def from_hf_config(cfg: dict | str | Path) -> ModelSpec:
     """Build a ModelSpec from a Hugging Face `config.json` (dict or path)."""
     if not isinstance(cfg, dict):
@@ -432,6 +575,8 @@ def from_hf_config(cfg: dict | str | Path) -> ModelSpec:
         raise ValueError(f"unsupported architecture {archs[0]!r} (supported: {sorted(FAMILY_BY_ARCH)})")
     if family == "bedovik":
         return _bedovik_config(cfg)
+    if family == "tudilix":
+        return _tudilix_config(cfg)
     hidden = cfg["hidden_size"]
     heads = cfg["num_attention_heads"]
     if "kv_lora_rank" in cfg:
@@ -498,12 +643,19 @@ def spec_from_json(d: dict) -> ModelSpec:
     d = dict(d)
     if "engram_layers" in d:
         d["engram_layers"] = tuple(d["engram_layers"])
+    def attn(a: dict) -> AttentionSpec:
+        return AttentionSpec(**dict(a, rope_scaling=RopeScaling(**a["rope_scaling"]) if a.get("rope_scaling") else None))
+
+    def block(b: dict) -> BlockSpec:
+        part = lambda key, make: make(b[key]) if b.get(key) else None
+        return BlockSpec(part("attn", attn), part("moe", lambda m: MoESpec(**m)), part("rec", lambda r: RecurrentSpec(**r)), part("ffn", lambda f: DenseFfnSpec(**f)))
+
     if d.get("blocks"):
-        d["blocks"] = tuple(BlockSpec(AttentionSpec(**b["attn"]), MoESpec(**b["moe"]) if b["moe"] else None) for b in d["blocks"])
+        d["blocks"] = tuple(block(b) for b in d["blocks"])
     d["blocks"] = tuple(d.get("blocks") or ())
     if d.get("loop"):
         d["loop"] = LoopSpec(**d["loop"])
-    return ModelSpec(attn=AttentionSpec(**d.pop("attn")), moe=MoESpec(**d.pop("moe")), quant=QuantSpec(**d.pop("quant")), **d)
+    return ModelSpec(attn=attn(d.pop("attn")), moe=MoESpec(**d.pop("moe")), quant=QuantSpec(**d.pop("quant")), **d)
 
 
 def spec_from_snapshot(path: str | Path) -> ModelSpec:

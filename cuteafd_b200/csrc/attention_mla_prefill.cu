@@ -356,30 +356,39 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
 }
 
 // ------------------------------------------------------------------------------------------------------------
-// The same structure for paged GQA prefill (head_dim 128): a CTA owns 128 query rows of one KV head (row = token_in_tile * G +
+// The same structure for paged GQA prefill, templated on the 64-wide chunks of key (KC) and value (VC) dimensions (head_dim 128: 2, 2): a CTA owns 128 query rows of one KV head (row = token_in_tile * G +
 // head_in_group) and walks the sequence's pages two at a time (128-key tiles), K and V straight from the paged store.  Causal
 // mask, optional sliding window and sink logit as in the decode kernel (attention_tc.cu), no split-KV: a prefill chunk has
 // enough query tiles to fill the GPU.  window < 0 drops the causal mask (bidirectional attention of a vision / audio encoder:
 // every query row sees keys [0, kvlen)).  The 64-key decode kernel spends 8 + 4 tcgen05.mma per 64 keys; this one 8 + 8 per 128 keys.
-#define GQ_K_STAGE 32768          // 2 chunks (64 dims each) x [128 keys x 128 B]
+template <int KC, int VC>
+struct GqaPrefillCfg {
+  static constexpr int K_STAGE = KC * 16384, V_STAGE = VC * 16384;          // chunks (64 dims each) x [128 keys x 128 B]
+  static constexpr int NSV = PF_P_BYTES + PF_NS * K_STAGE + 2 * V_STAGE <= 224 * 1024 ? 2 : 1;
+  static constexpr int SMEM = PF_P_BYTES + PF_NS * K_STAGE + NSV * V_STAGE + 256;
+  static_assert(256 + KC * 32 + VC * 64 <= 512, "scores, query and output exceed tensor memory");
+};
 struct GqaPrefillArgs {
   const bf16* q;
-  const CUtensorMap* kv_map;    // 3-D {128, 2 * Hkv, slots}, box {64, 1, 64}, 128-byte swizzle (the decode kernel's descriptor)
+  const CUtensorMap* k_map; const CUtensorMap* v_map;      // the decode kernel's descriptors; value head h at coordinate v_head0 + h
   const int* page_table; const int* kv_len; const int* q_start; const int* q_len;
   const float* sink;
   bf16* out;
   int* status;
   int q_stride, Hq, Hkv, max_pages, window, max_q_tiles;
+  int v_head0, dv, ldo;
   float scale;
 };
 
+template <int KC, int VC>
 __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_constant__ GqaPrefillArgs a) {
+  using Cf = GqaPrefillCfg<KC, VC>;
   pdl_launch(); pdl_wait();
   extern __shared__ __align__(1024) uint8_t smem[];
   uint8_t* sP = smem;
   uint8_t* sK = sP + PF_P_BYTES;
-  uint8_t* sV = sK + PF_NS * GQ_K_STAGE;
-  uint64_t* bars = (uint64_t*)(sV + PF_NSV * PF_V_STAGE);
+  uint8_t* sV = sK + PF_NS * Cf::K_STAGE;
+  uint64_t* bars = (uint64_t*)(sV + Cf::NSV * Cf::V_STAGE);
   uint64_t* k_full = bars; uint64_t* k_empty = bars + 2; uint64_t* v_full = bars + 4; uint64_t* v_empty = bars + 6;     // [<= 2] each
   uint64_t* s_full = bars + 8;          // [2]
   uint64_t* s_free = bars + 10;         // [2]: the softmax threads are done with the score buffer
@@ -419,15 +428,15 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
   tc_fence_after();
   const uint32_t tmem = tmem_slot;
   volatile int* abortp = &abort_flag;
-  const uint32_t S0_COL = 0, O_COL = 128, S1_COL = 256, Q_COL = 384;
-  // query rows -> tensor memory (row = lane, two bf16 per 32-bit column, 64 columns for the 128-wide head)
+  const uint32_t S0_COL = 0, S1_COL = 128, O_COL = 256, Q_COL = 256 + VC * 64;
+  // query rows -> tensor memory (row = lane, two bf16 per 32-bit column, 32 columns per chunk)
   if (warp >= 2) {
     const int r = (warp & 3) * 32 + lane;
     const uint32_t dst = tmem + ((uint32_t)((warp & 3) * 32) << 16) + Q_COL;
     const int rr = r < R ? r : 0;
-    const bf16* src = a.q + (size_t)(row_base + rr / G) * a.q_stride + (size_t)(kvh * G + rr % G) * 128;
+    const bf16* src = a.q + (size_t)(row_base + rr / G) * a.q_stride + (size_t)(kvh * G + rr % G) * (KC * 64);
 #pragma unroll 1
-    for (int g = 0; g < 4; ++g) {                  // 16 columns = 32 elements per store
+    for (int g = 0; g < KC * 2; ++g) {                  // 16 columns = 32 elements per store
       uint32_t w[16];
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
@@ -455,12 +464,12 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       if (!mbar_wait_bounded(&k_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); return false; }
       if (lane == 0) {
         const int key0 = (tile0 + i) * PF_KT;
-        mbar_expect_tx(&k_full[s], GQ_K_STAGE);
+        mbar_expect_tx(&k_full[s], Cf::K_STAGE);
 #pragma unroll
         for (int p = 0; p < 2; ++p) {
           const int slot0 = page_of(key0 + p * 64) * 64;
-          tma_load_3d(sK + s * GQ_K_STAGE + p * 8192, a.kv_map, &k_full[s], 0, kvh, slot0);
-          tma_load_3d(sK + s * GQ_K_STAGE + 16384 + p * 8192, a.kv_map, &k_full[s], 64, kvh, slot0);
+#pragma unroll
+          for (int c = 0; c < KC; ++c) tma_load_3d(sK + s * Cf::K_STAGE + c * 16384 + p * 8192, a.k_map, &k_full[s], c * 64, kvh, slot0);
         }
       }
       __syncwarp();
@@ -469,32 +478,32 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
     bool okp = n_tiles > 0 ? load_k(0) : true;
     for (int i = 0; okp && i < n_tiles && !*abortp; ++i) {
       if (i + 1 < n_tiles && !load_k(i + 1)) break;
-      const int sv = i % PF_NSV, phv = ((i / PF_NSV) & 1) ^ 1;
+      const int sv = i % Cf::NSV, phv = ((i / Cf::NSV) & 1) ^ 1;
       if (!mbar_wait_bounded(&v_empty[sv], phv, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, 0x1000 + i); break; }
       if (lane == 0) {
         const int key0 = (tile0 + i) * PF_KT;
-        mbar_expect_tx(&v_full[sv], PF_V_STAGE);
+        mbar_expect_tx(&v_full[sv], Cf::V_STAGE);
 #pragma unroll
         for (int p = 0; p < 2; ++p) {
           const int slot0 = page_of(key0 + p * 64) * 64;
-          tma_load_3d(sV + sv * PF_V_STAGE + p * 8192, a.kv_map, &v_full[sv], 0, a.Hkv + kvh, slot0);
-          tma_load_3d(sV + sv * PF_V_STAGE + 16384 + p * 8192, a.kv_map, &v_full[sv], 64, a.Hkv + kvh, slot0);
+#pragma unroll
+          for (int c = 0; c < VC; ++c) tma_load_3d(sV + sv * Cf::V_STAGE + c * 16384 + p * 8192, a.v_map, &v_full[sv], c * 64, a.v_head0 + kvh, slot0);
         }
       }
       __syncwarp();
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
-    const uint32_t id_s = pf_idesc(PF_KT, 0), id_o = pf_idesc(128, 1);
+    const uint32_t id_s = pf_idesc(PF_KT, 0), id_o = pf_idesc(VC * 64, 1);
     auto issue_scores = [&](int j) -> bool {     // S[j & 1] = Q K(j)^T once the softmax threads have copied tile j - 2 out of it
       const int s = j % PF_NS;
       if (j >= 2 && !mbar_wait_bounded(&s_free[j & 1], ((j - 2) >> 1) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, 0x2000 + j); return false; }
       if (!mbar_wait_bounded(&k_full[s], (j / PF_NS) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, j); return false; }
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t k0 = smem_u32(sK + s * GQ_K_STAGE), d = tmem + ((j & 1) ? S1_COL : S0_COL);
+        const uint32_t k0 = smem_u32(sK + s * Cf::K_STAGE), d = tmem + ((j & 1) ? S1_COL : S0_COL);
 #pragma unroll
-        for (int kb = 0; kb < 2; ++kb)
+        for (int kb = 0; kb < KC; ++kb)
 #pragma unroll
           for (int k = 0; k < 4; ++k)
             tc_mma_f16_ta(d, tmem + Q_COL + kb * 32 + k * 8, umma_desc_sw128(k0 + kb * 16384) + 2 * k, id_s, (kb | k) ? 1u : 0u);
@@ -507,12 +516,12 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
     bool ok = true;
     for (int j = 0; ok && j < min(2, n_tiles); ++j) ok = issue_scores(j);
     for (int i = 0; ok && i < n_tiles; ++i) {
-      const int sv = i % PF_NSV;
+      const int sv = i % Cf::NSV;
       if (!mbar_wait_bounded(&p_full, i & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, 0x3000 + i); break; }
-      if (!mbar_wait_bounded(&v_full[sv], (i / PF_NSV) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, 0x4000 + i); break; }
+      if (!mbar_wait_bounded(&v_full[sv], (i / Cf::NSV) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, 0x4000 + i); break; }
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t v0 = smem_u32(sV + sv * PF_V_STAGE);
+        const uint32_t v0 = smem_u32(sV + sv * Cf::V_STAGE);
 #pragma unroll
         for (int k = 0; k < PF_KT / 16; ++k)       // 16 keys per MMA: P chunk k / 4 (64 keys per 128-byte row), V rows 16 k .. 16 k + 15
           tc_mma_f16(tmem + O_COL, umma_desc_sw128(smem_u32(sP) + (k >> 2) * 16384) + 2 * (k & 3), pf_desc_mn_sw128(v0 + k * 2048, 16384, 1024), id_o,
@@ -617,7 +626,7 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       tc_fence_after();
       if (i > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {      // warp-uniform: tcgen05.ld/st are warp collectives
 #pragma unroll 1
-        for (int c = 0; c < 8; ++c) {
+        for (int c = 0; c < VC * 4; ++c) {
           uint32_t o[16];
           tmem_ld_x16(tmem + lane_addr + O_COL + c * 16, o);
           tc_wait_ld();
@@ -648,9 +657,10 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
         lt = l * e1 + __expf(sk - m2); scale_o = e1;
       }
       const float inv = lt > 0.f ? scale_o / lt : 0.f;
-      bf16* dst = a.out + ((size_t)t * a.Hq + h) * 128;
+      bf16* dst = a.out + (size_t)t * a.ldo + (size_t)h * a.dv;
+      const bool vec = ((a.dv | a.ldo) & 7) == 0;
 #pragma unroll 1
-      for (int c = 0; c < 8; ++c) {
+      for (int c = 0; c < VC * 4; ++c) {
         uint32_t o[16];
         if (n_tiles > 0) { tmem_ld_x16(tmem + lane_addr + O_COL + c * 16, o); tc_wait_ld(); }
         else {
@@ -661,8 +671,14 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
         uint32_t w[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) { bf162 hh = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * inv, __uint_as_float(o[2 * j + 1]) * inv); w[j] = *(uint32_t*)&hh; }
-        *(uint4*)(dst + c * 16) = make_uint4(w[0], w[1], w[2], w[3]);
-        *(uint4*)(dst + c * 16 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+        if (vec) {
+          if (c * 16 < a.dv) *(uint4*)(dst + c * 16) = make_uint4(w[0], w[1], w[2], w[3]);
+          if (c * 16 + 8 < a.dv) *(uint4*)(dst + c * 16 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (c * 16 + j < a.dv) dst[c * 16 + j] = ((const bf16*)w)[j];
+        }
       }
     }
   }
@@ -672,6 +688,20 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
   if (warp == 1) tmem_dealloc(tmem, 512);
 }
 
+template <int KC, int VC>
+static int launch_gqa_prefill(const GqaPrefillArgs& a, int n_seq, cudaStream_t s) {
+  const int smem = GqaPrefillCfg<KC, VC>::SMEM;
+  static bool attr_set[64] = {false};
+  int dev = 0; cudaGetDevice(&dev);
+  if (!attr_set[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(gqa_prefill_kernel<KC, VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(gqa_prefill)");
+    attr_set[dev & 63] = true;
+  }
+  CA_LAUNCH_PDL((gqa_prefill_kernel<KC, VC>), dim3(a.Hkv, n_seq * a.max_q_tiles), 192, smem, s, a);
+  CA_CHECK_LAUNCH("gqa_prefill_attention");
+  return CA_OK;
+}
 
 extern "C" int cuteafd_gqa_prefill_attention(const void* q, const void* kv_map, const int* page_table, const int* kv_len, const int* q_start,
                                              const int* q_len, const float* sink, void* out, int T, int n_seq, int max_q_len, int q_stride, int Hq,
@@ -680,22 +710,32 @@ extern "C" int cuteafd_gqa_prefill_attention(const void* q, const void* kv_map, 
   CA_REQUIRE(Hq % Hkv == 0 && 128 % (Hq / Hkv) == 0 && q_stride % 8 == 0, "gqa_prefill_attention: group size %d unsupported", Hq / Hkv);
   if (T <= 0 || n_seq <= 0) return CA_OK;
   GqaPrefillArgs a;
-  a.q = (const bf16*)q; a.kv_map = (const CUtensorMap*)kv_map; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len;
+  a.q = (const bf16*)q; a.k_map = a.v_map = (const CUtensorMap*)kv_map; a.v_head0 = Hkv; a.dv = 128; a.ldo = Hq * 128; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len;
   a.sink = sink; a.out = (bf16*)out; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.window = window;
   a.scale = scale;
   const int tpt = 128 / (Hq / Hkv);
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
-  const int smem = PF_P_BYTES + PF_NS * GQ_K_STAGE + PF_NSV * PF_V_STAGE + 256;
-  static bool attr_set[64] = {false};
-  int dev = 0; cudaGetDevice(&dev);
-  if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(gqa_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(gqa_prefill)");
-    attr_set[dev & 63] = true;
-  }
-  CA_LAUNCH_PDL(gqa_prefill_kernel, dim3(Hkv, n_seq * a.max_q_tiles), 192, smem, s, a);
-  CA_CHECK_LAUNCH("gqa_prefill_attention");
-  return CA_OK;
+  return launch_gqa_prefill<2, 2>(a, n_seq, s);
+}
+
+// The same over a store whose keys and values have widths of their own (layout and maps as `cuteafd_window_attention`); dk_pad + 2 dv_pad
+// of at most 512 fit tensor memory.
+extern "C" int cuteafd_window_prefill_attention(const void* q, const void* maps, const int* page_table, const int* kv_len, const int* q_start, const int* q_len, void* out,
+                                                int T, int n_seq, int max_q_len, int q_stride, int Hq, int Hkv, int dk_pad, int dv_pad, int dv, int ldo, int max_pages,
+                                                int window, float scale, int* status, cudaStream_t s) {
+  CA_REQUIRE(q && maps && page_table && kv_len && q_start && q_len && out, "window_prefill_attention: null argument");
+  CA_REQUIRE(Hkv >= 1 && Hq % Hkv == 0 && Hq / Hkv <= 128 && q_stride % 8 == 0, "window_prefill_attention: group size %d unsupported", Hkv ? Hq / Hkv : 0);
+  CA_REQUIRE(dv >= 1 && dv <= dv_pad && ldo >= Hq * dv && window >= 0 && q_stride >= Hq * dk_pad, "window_prefill_attention: bad shape");
+  if (T <= 0 || n_seq <= 0) return CA_OK;
+  GqaPrefillArgs a = {};
+  a.q = (const bf16*)q; a.k_map = (const CUtensorMap*)maps; a.v_map = a.k_map + 1; a.v_head0 = 0; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
+  a.q_len = q_len; a.sink = nullptr; a.out = (bf16*)out; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.window = window;
+  a.scale = scale; a.dv = dv; a.ldo = ldo;
+  const int tpt = 128 / (Hq / Hkv);
+  a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
+#define WP_CASE(K_, V_) if (dk_pad == K_ * 64 && dv_pad == V_ * 64) return launch_gqa_prefill<K_, V_>(a, n_seq, s);
+  WP_CASE(1, 1) WP_CASE(1, 2) WP_CASE(1, 3) WP_CASE(2, 1) WP_CASE(2, 2) WP_CASE(2, 3) WP_CASE(3, 1) WP_CASE(3, 2) WP_CASE(4, 1) WP_CASE(4, 2)
+  return ca_fail(CA_ERR_UNSUPPORTED, "window_prefill_attention: head widths %d / %d do not fit tensor memory", dk_pad, dv_pad);
 }
 
 // Gathers the latent rows of every sequence's context out of the paged cache into one contiguous buffer:

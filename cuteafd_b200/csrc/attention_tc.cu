@@ -1,5 +1,6 @@
-// Paged GQA attention on the 5th-generation tensor cores (head_dim 128): decode, speculative verify and
-// chunked prefill in one kernel.
+// Paged GQA attention on the 5th-generation tensor cores: decode, speculative verify and chunked prefill in one
+// kernel, templated on the 64-wide chunks of key (KC) and value (VC) dimensions; the sizes below are those of
+// head_dim 128 (KC = VC = 2).
 //
 // A CTA owns up to 128 query rows of one KV head of one sequence (row = token_in_tile * G + head_in_group)
 // and a contiguous range of 64-key pages (split-KV).  Per page:
@@ -28,7 +29,8 @@
 
 struct AttnTcArgs {
   const bf16* q;
-  const CUtensorMap* kv_map;    // 3-D: {D, 2*Hkv, slots}, box {64, 1, 64}, 128-byte swizzle
+  const CUtensorMap* k_map;     // 3-D: {KC * 64, heads, slots}, box {64, 1, 64}, 128-byte swizzle; head h of K at coordinate h
+  const CUtensorMap* v_map;     // {VC * 64, ..}: head h of V at coordinate v_head0 + h (one map of an interleaved store serves both)
   const int* page_table;
   const int* kv_len;
   const int* q_start;
@@ -39,6 +41,7 @@ struct AttnTcArgs {
   float* part_ml;
   int* status;
   int q_stride, Hq, Hkv, max_pages, n_splits, window, max_q_tiles, T;
+  int v_head0, dv, ldo;         // value width of the output (at most VC * 64) and its row pitch: head h at column h * dv
   float scale;
 };
 
@@ -63,12 +66,23 @@ __device__ __forceinline__ void tmem_st_x16(uint32_t addr, const uint32_t* r) {
 }
 __device__ __forceinline__ void tc_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-__global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_constant__ AttnTcArgs a) {
+template <int KC, int VC>
+struct AttnTcCfg {
+  static constexpr int Q_BYTES = KC * 16384, P_BYTES = 16384, K_STAGE = KC * 8192, V_STAGE = VC * 8192;
+  static constexpr int K_OFF = Q_BYTES + P_BYTES, V_OFF = K_OFF + NS * K_STAGE, BAR_OFF = V_OFF + NS * V_STAGE;
+  static constexpr int SMEM = BAR_OFF + 128;
+  static constexpr int TMEM_COLS = 128 + VC * 64 <= 256 ? 256 : 512;         // two score buffers and the output
+  static constexpr int OCC = SMEM <= 115 * 1024 && TMEM_COLS == 256 ? 2 : 1;
+};
+
+template <int KC, int VC>
+__global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_kernel(const __grid_constant__ AttnTcArgs a) {
+  using Cf = AttnTcCfg<KC, VC>;
   pdl_launch(); pdl_wait();
   // All shared memory is dynamic and 1024-byte aligned (operand tiles first, barriers at the tail) so that two
   // CTAs fit on one SM.
   extern __shared__ __align__(1024) uint8_t smem[];
-  uint64_t* bars = (uint64_t*)(smem + 49152 + NS * 32768);
+  uint64_t* bars = (uint64_t*)(smem + Cf::BAR_OFF);
   uint64_t* k_full = bars; uint64_t* k_empty = bars + 2; uint64_t* v_full = bars + 4; uint64_t* v_empty = bars + 6;
   uint64_t* s_full = bars + 8;              // two score buffers
   uint64_t& p_full = bars[10]; uint64_t& o_done = bars[11];
@@ -76,10 +90,10 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
   int& abort_flag = *(int*)(bars + 13);
   uint64_t& x_bar = bars[14];               // column-split softmax: cross-warp exchange barrier
   if (smem_u32(smem) & 1023) { if (threadIdx.x == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0xA11); return; }
-  uint8_t* sQ = smem;                       // 2 x [128 rows x 128 B]
-  uint8_t* sP = smem + 32768;               // [128 rows x 128 B]
-  uint8_t* sK = smem + 49152;               // 2 stages x {lo, hi} x 8 KB
-  uint8_t* sV = smem + 49152 + 32768;       // 2 stages x {lo, hi} x 8 KB
+  uint8_t* sQ = smem;                       // KC x [128 rows x 128 B]
+  uint8_t* sP = smem + Cf::Q_BYTES;         // [128 rows x 128 B]
+  uint8_t* sK = smem + Cf::K_OFF;           // 2 stages x KC x 8 KB
+  uint8_t* sV = smem + Cf::V_OFF;           // 2 stages x VC x 8 KB
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tid = threadIdx.x;
 
   const int G = a.Hq / a.Hkv;
@@ -113,13 +127,13 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
     abort_flag = 0;
     fence_barrier_init();
   }
-  if (warp == 1) { tmem_alloc(&tmem_slot, 256); tmem_relinquish(); }
-  // Q rows -> swizzled K-major operand tiles (two 64-element halves)
-  for (int i = tid; i < 128 * 16; i += 192) {
-    const int r = i >> 4, c = i & 15;                  // 16-byte chunk c of row r
+  if (warp == 1) { tmem_alloc(&tmem_slot, Cf::TMEM_COLS); tmem_relinquish(); }
+  // Q rows -> swizzled K-major operand tiles (64-element chunks)
+  for (int i = tid; i < 128 * KC * 8; i += 192) {
+    const int r = i / (KC * 8), c = i % (KC * 8);      // 16-byte piece c of row r
     uint4 v = make_uint4(0, 0, 0, 0);
     const int qr = rep4 ? (r & 31) : r;                // decode tiles replicate their <= 32 rows into all four lane quarters
-    if (qr < R) v = *(const uint4*)(a.q + (size_t)(row_base + qr / G) * a.q_stride + (size_t)(kvh * G + qr % G) * AD + c * 8);
+    if (qr < R) v = *(const uint4*)(a.q + (size_t)(row_base + qr / G) * a.q_stride + (size_t)(kvh * G + qr % G) * (KC * 64) + c * 8);
     *(uint4*)(sQ + (c >> 3) * 16384 + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
   }
   fence_proxy_async_smem();
@@ -128,7 +142,7 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
   tc_fence_after();
   const uint32_t tmem = tmem_slot;
   volatile int* abortp = &abort_flag;
-  const uint32_t S0_COL = 0, O_COL = 64, S1_COL = 192;
+  const uint32_t S0_COL = 0, O_COL = 64, S1_COL = 64 + VC * 64;
 
   if (warp == 0) {
     // ------------------------------------------------------------------ K/V producer (separate K and V rings:
@@ -140,30 +154,30 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
       const int page = a.page_table[(size_t)seq * a.max_pages + p0 + i];
       if (!mbar_wait_bounded(&k_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); break; }
       if (lane == 0) {
-        mbar_expect_tx(&k_full[s], 16384);
-        tma_load_3d_hint(sK + s * 16384, a.kv_map, &k_full[s], 0, kvh, page * APAGE, kvpol);
-        tma_load_3d_hint(sK + s * 16384 + 8192, a.kv_map, &k_full[s], 64, kvh, page * APAGE, kvpol);
+        mbar_expect_tx(&k_full[s], Cf::K_STAGE);
+#pragma unroll
+        for (int c = 0; c < KC; ++c) tma_load_3d_hint(sK + s * Cf::K_STAGE + c * 8192, a.k_map, &k_full[s], c * 64, kvh, page * APAGE, kvpol);
       }
       if (!mbar_wait_bounded(&v_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); break; }
       if (lane == 0) {
-        mbar_expect_tx(&v_full[s], 16384);
-        tma_load_3d_hint(sV + s * 16384, a.kv_map, &v_full[s], 0, a.Hkv + kvh, page * APAGE, kvpol);
-        tma_load_3d_hint(sV + s * 16384 + 8192, a.kv_map, &v_full[s], 64, a.Hkv + kvh, page * APAGE, kvpol);
+        mbar_expect_tx(&v_full[s], Cf::V_STAGE);
+#pragma unroll
+        for (int c = 0; c < VC; ++c) tma_load_3d_hint(sV + s * Cf::V_STAGE + c * 8192, a.v_map, &v_full[s], c * 64, a.v_head0 + kvh, page * APAGE, kvpol);
       }
       __syncwarp();
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
     // Scores are double-buffered in tensor memory: S(i+1) is computed while the softmax of tile i runs.
-    const uint32_t id_s = idesc_bf16(64, 0), id_o = idesc_bf16(128, 1);
+    const uint32_t id_s = idesc_bf16(64, 0), id_o = idesc_bf16(VC * 64, 1);
     auto issue_scores = [&](int j) -> bool {     // S[j & 1] = Q K(j)^T
       const int s = j & 1;
       if (!mbar_wait_bounded(&k_full[s], (j >> 1) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, j); return false; }
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t k0 = smem_u32(sK + s * 16384), d = tmem + (s ? S1_COL : S0_COL);
+        const uint32_t k0 = smem_u32(sK + s * Cf::K_STAGE), d = tmem + (s ? S1_COL : S0_COL);
 #pragma unroll
-        for (int kb = 0; kb < 2; ++kb)
+        for (int kb = 0; kb < KC; ++kb)
 #pragma unroll
           for (int k = 0; k < 4; ++k)
             tc_mma_f16(d, desc_kmajor_sw128(smem_u32(sQ) + kb * 16384) + 2 * k, desc_kmajor_sw128(k0 + kb * 8192) + 2 * k, id_s, (kb | k) ? 1u : 0u);
@@ -181,7 +195,7 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
       if (!mbar_wait_bounded(&v_full[s], (i >> 1) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_MMA, i); break; }
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t v0 = smem_u32(sV + s * 16384);
+        const uint32_t v0 = smem_u32(sV + s * Cf::V_STAGE);
 #pragma unroll
         for (int k = 0; k < 4; ++k)
           tc_mma_f16(tmem + O_COL, desc_kmajor_sw128(smem_u32(sP)) + 2 * k, desc_mnmajor_sw128(v0 + k * 2048, 8192, 1024), id_o, (i | k) ? 1u : 0u);
@@ -239,7 +253,7 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
         }
         if (q4 == 0 && i > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {     // the real O rows live in lane quarter 0
 #pragma unroll 1
-          for (int c = 0; c < 8; ++c) {
+          for (int c = 0; c < VC * 4; ++c) {
             uint32_t o[16];
             tmem_ld_x16(tmem + O_COL + c * 16, o);
             tc_wait_ld();
@@ -302,7 +316,7 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
       }
       if (i > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
 #pragma unroll 1
-        for (int c = 0; c < 8; ++c) {
+        for (int c = 0; c < VC * 4; ++c) {
           uint32_t o[16];
           tmem_ld_x16(tmem + lane_addr + O_COL + c * 16, o);
           tc_wait_ld();
@@ -345,10 +359,11 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
         lt = l * e1 + __expf(sk - m2); scale_o = e1;
       }
       const float inv = lt > 0.f ? scale_o / lt : 0.f;
-      bf16* dst = a.out + (size_t)t * a.Hq * AD + (size_t)h * AD;
-      float* po = a.n_splits > 1 ? a.part_o + (((size_t)split * a.T + t) * a.Hq + h) * AD : nullptr;
+      bf16* dst = a.out + (size_t)t * a.ldo + (size_t)h * a.dv;
+      const bool vec = ((a.dv | a.ldo) & 7) == 0;      // otherwise heads do not start on 16 bytes
+      float* po = a.n_splits > 1 ? a.part_o + (((size_t)split * a.T + t) * a.Hq + h) * (VC * 64) : nullptr;
 #pragma unroll 1
-      for (int c = 0; c < 8; ++c) {
+      for (int c = 0; c < VC * 4; ++c) {
         uint32_t o[16];
         if (n_tiles > 0) { tmem_ld_x16(tmem + lane_addr + O_COL + c * 16, o); tc_wait_ld(); }   // n_tiles is CTA-uniform
         else {
@@ -360,8 +375,14 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
           uint32_t w[8];
 #pragma unroll
           for (int j = 0; j < 8; ++j) { bf162 hh = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * inv, __uint_as_float(o[2 * j + 1]) * inv); w[j] = *(uint32_t*)&hh; }
-          *(uint4*)(dst + c * 16) = make_uint4(w[0], w[1], w[2], w[3]);
-          *(uint4*)(dst + c * 16 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+          if (vec) {
+            if (c * 16 < a.dv) *(uint4*)(dst + c * 16) = make_uint4(w[0], w[1], w[2], w[3]);
+            if (c * 16 + 8 < a.dv) *(uint4*)(dst + c * 16 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (c * 16 + j < a.dv) dst[c * 16 + j] = ((const bf16*)w)[j];
+          }
         } else {
 #pragma unroll
           for (int j = 0; j < 4; ++j) *(uint4*)(po + c * 16 + j * 4) = make_uint4(o[4 * j], o[4 * j + 1], o[4 * j + 2], o[4 * j + 3]);
@@ -376,7 +397,24 @@ __global__ void __launch_bounds__(192, 2) paged_attn_tc_kernel(const __grid_cons
   if (*abortp && warp == 0) { const uint64_t t0 = globaltimer_ns(); while (globaltimer_ns() - t0 < 200000) __nanosleep(1000); }
   tc_fence_before();
   __syncthreads();
-  if (warp == 1) tmem_dealloc(tmem, 256);
+  if (warp == 1) tmem_dealloc(tmem, Cf::TMEM_COLS);
+}
+
+template <int KC, int VC>
+static int launch_attn_tc(const AttnTcArgs& a, int n_seq, cudaStream_t s) {
+  const int smem = AttnTcCfg<KC, VC>::SMEM;
+  static bool attr_set[64] = {false};
+  int dev = 0; cudaGetDevice(&dev);
+  if (!attr_set[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(paged_attn_tc_kernel<KC, VC>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(paged_attn_tc)");
+    attr_set[dev & 63] = true;
+  }
+  // No pre-fill of the (m, l) partials: every CTA writes them for all of its live rows, also when its split
+  // holds no key (m = -inf, l = 0), and a CTA that gives up reports through the status word.
+  CA_LAUNCH_PDL((paged_attn_tc_kernel<KC, VC>), dim3(a.n_splits, a.Hkv, n_seq * a.max_q_tiles), 192, smem, s, a);
+  CA_CHECK_LAUNCH("paged_attention_tc");
+  return CA_OK;
 }
 
 // Context split (a long context whose KV pages live on several GPUs): every owner runs the attention over ITS pages
@@ -393,7 +431,7 @@ extern "C" int cuteafd_attn_merge(const float* part_o, const float* part_ml, con
                                   cudaStream_t s) {
   CA_REQUIRE(part_o && part_ml && out && n_parts >= 1, "attn_merge: needs partials");
   if (T <= 0) return CA_OK;
-  CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * AD / 8 + 127) / 128), 128, 0, s, part_o, part_ml, sink, (bf16*)out, T, Hq, (int)AD, n_parts,
+  CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * AD / 8 + 127) / 128), 128, 0, s, part_o, part_ml, sink, (bf16*)out, T, Hq, (int)AD, (int)AD, Hq * AD, n_parts,
                 (uint8_t*)nullptr, (uint8_t*)nullptr, 0, (const float*)nullptr, 0);
   CA_CHECK_LAUNCH("attn_merge");
   return CA_OK;
@@ -415,26 +453,15 @@ extern "C" int cuteafd_paged_attention_tc(const void* q, const void* kv_map, con
   CA_REQUIRE(!partials_only || n_splits >= 2, "paged_attention_tc: partials-only needs at least two splits");
   if (T <= 0 || n_seq <= 0) return CA_OK;
   AttnTcArgs a;
-  a.q = (const bf16*)q; a.kv_map = (const CUtensorMap*)kv_map; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
+  a.q = (const bf16*)q; a.k_map = a.v_map = (const CUtensorMap*)kv_map; a.v_head0 = Hkv; a.dv = AD; a.ldo = Hq * AD; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
   a.q_len = q_len; a.sink = sink; a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.status = status;
   a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.n_splits = n_splits; a.window = window; a.T = T; a.scale = scale;
   const int tpt = 128 / (Hq / Hkv);
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
-  const int smem = 49152 + NS * 32768 + 128;
-  static bool attr_set[64] = {false};
-  int dev = 0; cudaGetDevice(&dev);
-  if (!attr_set[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(paged_attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(paged_attn_tc)");
-    attr_set[dev & 63] = true;
-  }
-  // No pre-fill of the (m, l) partials: every CTA writes them for all of its live rows, also when its split
-  // holds no key (m = -inf, l = 0), and a CTA that gives up reports through the status word.
-  dim3 grid(n_splits, Hkv, n_seq * a.max_q_tiles);
-  CA_LAUNCH_PDL(paged_attn_tc_kernel, grid, 192, smem, s, a);
-  CA_CHECK_LAUNCH("paged_attention_tc");
+  const int rc = launch_attn_tc<2, 2>(a, n_seq, s);
+  if (rc != CA_OK) return rc;
   if (n_splits > 1 && !partials_only) {
-    CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * AD / 8 + 127) / 128), 128, 0, s, part_o, part_ml, sink, (bf16*)out, T, Hq, (int)AD, n_splits,
+    CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * AD / 8 + 127) / 128), 128, 0, s, part_o, part_ml, sink, (bf16*)out, T, Hq, (int)AD, (int)AD, Hq * AD, n_splits,
                   (uint8_t*)q_out, (uint8_t*)sf_out, ldsf, inv_gs, qkind);
     CA_CHECK_LAUNCH("attn_merge");
   }
@@ -446,6 +473,49 @@ extern "C" int cuteafd_tmap_encode_kv(void* out128, const void* base, int Hkv, u
   CUtensorMap m;
   int rc = ca_encode_tmap_3d(&m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, AD, 2 * (uint64_t)Hkv, n_slots, AD * 2,
                              (uint64_t)2 * Hkv * AD * 2, 64, 1, 64, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (rc) return rc;
+  memcpy(out128, &m, sizeof(m));
+  return CA_OK;
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// The same kernel over a store whose keys and values have widths of their own: row = Hkv key heads of dk_pad elements, then Hkv value
+// heads of dv_pad (each 64, 128, 192 or 256; pad columns of q are zero, pads of K and V finite), any group of up to 128 query heads.
+// q [T, q_stride] (head h at h * dk_pad), out [T, ldo] (head h at h * dv).  maps: the key and the value descriptor
+// (`cuteafd_tmap_encode_heads`), 128 bytes each.
+extern "C" int cuteafd_window_attention(const void* q, const void* maps, const int* page_table, const int* kv_len, const int* q_start, const int* q_len, void* out,
+                                        float* part_o, float* part_ml, int T, int n_seq, int max_q_len, int q_stride, int Hq, int Hkv, int dk_pad, int dv_pad, int dv,
+                                        int ldo, int max_pages, int n_splits, int window, float scale, int* status, cudaStream_t s) {
+  CA_REQUIRE(q && maps && page_table && kv_len && q_start && q_len && out, "window_attention: null argument");
+  CA_REQUIRE(Hkv >= 1 && Hq % Hkv == 0 && Hq / Hkv <= 128 && q_stride % 8 == 0, "window_attention: group size %d unsupported", Hkv ? Hq / Hkv : 0);
+  CA_REQUIRE(dv >= 1 && dv <= dv_pad && ldo >= Hq * dv && window >= 0 && q_stride >= Hq * dk_pad, "window_attention: bad shape");
+  CA_REQUIRE(n_splits >= 1 && (n_splits == 1 || (part_o && part_ml)), "window_attention: split-KV needs scratch");
+  if (T <= 0 || n_seq <= 0) return CA_OK;
+  AttnTcArgs a = {};
+  a.q = (const bf16*)q; a.k_map = (const CUtensorMap*)maps; a.v_map = a.k_map + 1; a.v_head0 = 0; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
+  a.q_len = q_len; a.sink = nullptr; a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv;
+  a.max_pages = max_pages; a.n_splits = n_splits; a.window = window; a.T = T; a.scale = scale; a.dv = dv; a.ldo = ldo;
+  const int tpt = 128 / (Hq / Hkv);
+  a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
+  int rc = CA_ERR_UNSUPPORTED;
+#define WA_CASE(K_, V_) if (dk_pad == K_ * 64 && dv_pad == V_ * 64) rc = launch_attn_tc<K_, V_>(a, n_seq, s);
+#define WA_ROW(K_) WA_CASE(K_, 1) WA_CASE(K_, 2) WA_CASE(K_, 3) WA_CASE(K_, 4)
+  WA_ROW(1) WA_ROW(2) WA_ROW(3) WA_ROW(4)
+  if (rc == CA_ERR_UNSUPPORTED) return ca_fail(rc, "window_attention: head widths %d / %d (64, 128, 192 or 256)", dk_pad, dv_pad);
+  if (rc != CA_OK) return rc;
+  if (n_splits > 1) {
+    CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * dv_pad / 8 + 127) / 128), 128, 0, s, part_o, part_ml, (const float*)nullptr, (bf16*)out, T, Hq, dv_pad, dv, ldo, n_splits,
+                  (uint8_t*)nullptr, (uint8_t*)nullptr, 0, (const float*)nullptr, 0);
+    CA_CHECK_LAUNCH("attn_merge");
+  }
+  return CA_OK;
+}
+
+// Descriptor of `heads` heads of `width` bf16 each (a multiple of 64) that start at `base` in rows `row_elems` apart.
+extern "C" int cuteafd_tmap_encode_heads(void* out128, const void* base, int width, int heads, uint64_t row_elems, uint64_t n_slots) {
+  CA_REQUIRE(width > 0 && width % 64 == 0 && heads >= 1 && row_elems % 8 == 0 && ((uintptr_t)base & 15) == 0, "tmap_encode_heads: bad geometry");
+  CUtensorMap m;
+  int rc = ca_encode_tmap_3d(&m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, width, heads, n_slots, (uint64_t)width * 2, row_elems * 2, 64, 1, 64, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
   memcpy(out128, &m, sizeof(m));
   return CA_OK;

@@ -26,10 +26,10 @@ static __global__ void attn_merge_kernel(const float* __restrict__ part_o, const
   }
 }
 
-// Same merge, eight output elements per thread, optionally also writing the merged row quantised to FP4 for the
+// Same merge, eight output elements per thread (the first Dout of a head's D columns, head h at column h * Dout of rows ldo apart), optionally also writing the merged row quantised to FP4 for the
 // output projection that follows (qkind 1 NVFP4 / 2 MXFP4; needs Hq * D % 256 == 0).  grid (T, ceil(Hq * D / 8 / 128)).
 static __global__ void attn_merge8_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ sink,
-                                          bf16* __restrict__ out, int T, int Hq, int D, int n_splits, uint8_t* __restrict__ q,
+                                          bf16* __restrict__ out, int T, int Hq, int D, int Dout, int ldo, int n_splits, uint8_t* __restrict__ q,
                                           uint8_t* __restrict__ sf, int ldsf, const float* __restrict__ inv_gs_ptr, int qkind) {
   pdl_launch(); pdl_wait();
   const int t = blockIdx.x, vi = blockIdx.y * blockDim.x + threadIdx.x, vpr = D / 8;
@@ -78,7 +78,12 @@ static __global__ void attn_merge8_kernel(const float* __restrict__ part_o, cons
   bf16 ob[8];
 #pragma unroll
   for (int j = 0; j < 8; ++j) ob[j] = __float2bfloat16(o[j] * inv);
-  *(uint4*)(out + ((size_t)t * Hq + h) * D + d0) = *(uint4*)ob;
+  bf16* dst = out + (size_t)t * ldo + (size_t)h * Dout + d0;
+  if (((Dout | ldo) & 7) == 0) { if (d0 < Dout) *(uint4*)dst = *(uint4*)ob; }
+  else {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) if (d0 + j < Dout) dst[j] = ob[j];
+  }
   if (qkind) {
     float f[8];
 #pragma unroll

@@ -444,7 +444,8 @@ struct CaFlagWaitArg {        // in-kernel wait in front of a consumer of peer d
 struct CaTcExtra {            // tc_linear: FP4 copy of the output and/or stores of the output tile into peers' memory
   void* q_out; void* sf_out; const float* inv_gs_out; int ldsf_out; int n_peer;
   void* peer_y[2]; void* peer_flag[2]; const int* peer_row_map; void* peer_ctl; void* peer_done; int peer_ld;
-  int act, grp_rows, grp_cols;      // squared-ReLU epilogue; token-major output of a GEMM grouped over heads
+  int act, grp_rows, grp_cols;      // activation (1 squared ReLU, 2 soft cap, 3 clamped GLU); token-major output of a GEMM grouped over heads
+  float act_p; const float* bias; const float* bias2;      // soft cap / GLU limit; biases of the GLU's two halves
 };
 static inline FlagWait ca_flag_wait_from(const CaFlagWaitArg* a) {
   FlagWait w = {nullptr, nullptr, nullptr, 0ull, 0, 0};

@@ -1,0 +1,714 @@
+// Kernels of the hybrid recurrent / windowed-attention stacks (fp32 residual rows, RMS norms in front of and behind every sub-layer):
+//   norm_rows        embedding, residual += mult * norm(sub-layer output + bias), or a gather of rows - each also leaves the next product's
+//                    normalised operand row
+//   rope_table       cosine / sine of the step's positions, once per rotation
+//   conv_qkv         projected queries, keys and values -> short causal convolution -> head norm -> rotation -> query rows, paged cache
+//   rglru_conv       x branch -> short causal convolution -> block-major operand of the gate product (and its tile table)
+//   lru_scan         the real-gated linear recurrence: one pass over short runs, chunk aggregates + carried rescan over long ones
+//   glu_rows         clamped GLU over two projected rows (all-fp32 mode; bf16 products do it in their epilogue)
+//   window_attn_simt paged grouped-query attention on the ordinary cores (fp32, and shapes the tcgen05 kernels do not take)
+// Everything a sequence carries from step to step is addressed by absolute position: convolution inputs live in a ring of
+// taps - 1 + depth rows, recurrent states in a ring of depth + 1, so a step that is repeated, or the last `depth` tokens that are taken back
+// (rejected drafts), need no restore - later positions overwrite them.  T is the operand type: bf16, or float for the all-fp32 mode.
+// (No counterpart in the reference, which has no such family; the recurrence's kernel is the sibling of linear_attn.cu.)
+#include "stack_rows.cuh"
+
+#define HS_TILE 16          // tokens of a sequence one block of the convolution kernels walks (at least taps - 1)
+#define HS_MAX_TAPS 16
+#define HS_CHUNK 64         // tokens of a chunk of the recurrence
+
+// ---------------------------------------------------------------- residual rows and their norms
+enum { ROWS_EMBED = 0, ROWS_ADD = 1, ROWS_GATHER = 2 };
+
+template <typename T>
+struct NormRows {
+  float* x; int W, Wp;                                      // residual rows, Wp apart; norms average over W
+  const int* tokens; const bf16* table; int vocab;          // ROWS_EMBED
+  const T* add; const float* bias; const float* post; float mult;      // ROWS_ADD: bias and post (gain of the norm behind) may be null
+  const int* src_rows;                                      // ROWS_GATHER
+  const float* gain; T* xn; int ldn;                        // next operand: rows normalised by `gain`, or null
+  float eps; int* status;
+};
+
+template <typename T, int NCH, int MODE>
+__global__ void norm_rows_kernel(const NormRows<T> a) {
+  pdl_launch(); pdl_wait();
+  __shared__ float red[32];
+  const int t = blockIdx.x, nt = blockDim.x;
+  float v[NCH][8];
+  size_t row = t;
+  if (MODE == ROWS_GATHER) row = (size_t)a.src_rows[t];
+  int tok = 0;
+  if (MODE == ROWS_EMBED) {
+    tok = a.tokens[t];
+    if (tok < 0 || tok >= a.vocab) { if (threadIdx.x == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, t); tok = 0; }
+  }
+#pragma unroll
+  for (int c = 0; c < NCH; ++c) {
+    const int i = (threadIdx.x + c * nt) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[c][j] = 0.f;
+    if (i >= a.Wp) continue;
+    if (MODE == ROWS_EMBED) load8<bf16>(a.table + (size_t)tok * a.Wp + i, v[c]);
+    else load8<float>(a.x + row * a.Wp + i, v[c]);
+  }
+  if (MODE == ROWS_ADD) {
+    float m[NCH][8], ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+      const int i = (threadIdx.x + c * nt) * 8;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) m[c][j] = 0.f;
+      if (i >= a.Wp) continue;
+      load8<T>(a.add + (size_t)t * a.Wp + i, m[c]);
+      if (a.bias) {
+        float b[8];
+        load8<float>(a.bias + i, b);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) m[c][j] += b[j];
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(m[c][j], m[c][j], ss);
+    }
+    const float inv = a.post ? rsqrtf(block_sum(ss, red) / (float)a.W + a.eps) : 1.f;
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+      const int i = (threadIdx.x + c * nt) * 8;
+      if (i >= a.Wp) continue;
+      float g[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
+      if (a.post) load8<float>(a.post + i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[c][j] = fmaf(a.mult, m[c][j] * inv * g[j], v[c][j]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < NCH; ++c) {
+    const int i = (threadIdx.x + c * nt) * 8;
+    if (i >= a.Wp) continue;
+    if (MODE != ROWS_GATHER) store8<float>(a.x + (size_t)t * a.Wp + i, v[c]);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(v[c][j], v[c][j], ss);
+  }
+  if (!a.xn) return;
+  const float inv = rsqrtf(block_sum(ss, red) / (float)a.W + a.eps);
+#pragma unroll
+  for (int c = 0; c < NCH; ++c) {
+    const int i = (threadIdx.x + c * nt) * 8;
+    if (i >= a.Wp) continue;
+    float g[8], y[8];
+    load8<float>(a.gain + i, g);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) y[j] = v[c][j] * inv * g[j];
+    store8<T>(a.xn + (size_t)t * a.ldn + i, y);
+  }
+}
+
+// ---------------------------------------------------------------- rotation
+// freq: [2, pairs] - the fp32 angle per position and what fp32 rounded off it, so that angles of far positions keep full accuracy.
+__global__ void rope_table_kernel(const int* __restrict__ positions, const float* __restrict__ freq, float amp, int pairs, float2* __restrict__ out) {
+  pdl_launch(); pdl_wait();
+  const int t = blockIdx.x;
+  const float p = (float)positions[t];
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    const float f = freq[i], a = p * f, lo = fmaf(p, f, -a) + p * freq[pairs + i];
+    float s, c;
+    sincosf(a, &s, &c);
+    out[(size_t)t * pairs + i] = make_float2(amp * fmaf(-s, lo, c), amp * fmaf(c, lo, s));
+  }
+}
+
+// ---------------------------------------------------------------- short convolution in front of attention
+template <typename T>
+struct ConvQkv {
+  const T* proj; int ldp;                       // [T, ldp]: H * dim queries | G * dim keys | G * vdim values
+  const float* w;                               // [taps, C]
+  const float* q_norm; const float* k_norm;     // gains of the head norms
+  const float2* rope;                           // [T, pairs]
+  T* ring;                                      // [slots, R, C] projected rows by position
+  const int* state_slot; const int* q_start; const int* q_len; const int* kv_len; const int* slot_map;
+  T* q; int q_stride;                           // [T, H * dp]
+  T* cache; int row_stride, n_slots;            // paged rows: G * dp keys, then G * dvp values
+  int H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state;
+  float eps; int* status;
+};
+
+template <typename T> __device__ __forceinline__ float2 load_pair(const T* p, bool two, bool vec);
+template <> __device__ __forceinline__ float2 load_pair<bf16>(const bf16* p, bool two, bool vec) {
+  if (vec) return __bfloat1622float2(*(const bf162*)p);
+  return make_float2(to_f(p[0]), two ? to_f(p[1]) : 0.f);
+}
+template <> __device__ __forceinline__ float2 load_pair<float>(const float* p, bool two, bool vec) {
+  if (vec) return *(const float2*)p;
+  return make_float2(p[0], two ? p[1] : 0.f);
+}
+template <typename T> __device__ __forceinline__ void store_pair(T* p, float2 v, bool two, bool vec);
+template <> __device__ __forceinline__ void store_pair<bf16>(bf16* p, float2 v, bool two, bool vec) {
+  if (vec) { *(bf162*)p = __floats2bfloat162_rn(v.x, v.y); return; }
+  p[0] = __float2bfloat16(v.x);
+  if (two) p[1] = __float2bfloat16(v.y);
+}
+template <> __device__ __forceinline__ void store_pair<float>(float* p, float2 v, bool two, bool vec) {
+  if (vec) { *(float2*)p = v; return; }
+  p[0] = v.x;
+  if (two) p[1] = v.y;
+}
+
+// One warp per (head, tile of HS_TILE tokens); a lane owns the dimension pairs lane, lane + 32, ... of the head (NC of them).  TAPS > 0: the
+// last inputs and the weights stay in registers; 0: any number of taps, inputs re-read.
+template <typename T, int NC, int TAPS>
+__global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvQkv<T> a) {
+  pdl_launch(); pdl_wait();
+  const int lane = threadIdx.x & 31, unit = blockIdx.x * 4 + (threadIdx.x >> 5), seq = blockIdx.z;
+  const int n = a.q_len[seq], i0 = blockIdx.y * HS_TILE;
+  if (unit >= a.H + 2 * a.G || i0 >= n) return;
+  const int row0 = a.q_start[seq], p0 = a.kv_len[seq] - n, slot = a.state_slot[seq], i1 = min(n, i0 + HS_TILE);
+  if (slot < 0 || slot >= a.n_state) { if (lane == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6E1); return; }
+  const bool is_q = unit < a.H, is_v = unit >= a.H + a.G;
+  const int d = is_v ? a.vdim : a.dim, head = is_q ? unit : (is_v ? unit - a.H - a.G : unit - a.H);
+  const int ch = is_v ? (a.H + a.G) * a.dim + head * a.vdim : unit * a.dim;
+  const int taps = TAPS ? TAPS : a.taps;
+  T* ring = a.ring + (size_t)slot * a.R * a.C + ch;
+  bool has[NC], two[NC], vec[NC], rvec[NC];
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int e = 2 * (lane + 32 * c);
+    has[c] = e < d; two[c] = e + 1 < d;
+    vec[c] = two[c] && ((ch | a.ldp) & 1) == 0;
+    rvec[c] = vec[c] && (a.C & 1) == 0;
+  }
+  // input row i of this run (i < 0: what the sequence fed before, nothing in front of its start)
+  auto input = [&](int i, int c) -> float2 {
+    const int e = 2 * (lane + 32 * c);
+    if (!has[c]) return make_float2(0.f, 0.f);
+    if (i >= 0) return load_pair<T>(a.proj + (size_t)(row0 + i) * a.ldp + ch + e, two[c], vec[c]);
+    const int pos = p0 + i;
+    if (pos < 0) return make_float2(0.f, 0.f);
+    return load_pair<T>(ring + (size_t)(pos % a.R) * a.C + e, two[c], rvec[c]);
+  };
+  auto weight = [&](int j, int c) -> float2 {
+    const float* w = a.w + (size_t)j * a.C + ch + 2 * (lane + 32 * c);
+    return make_float2(has[c] ? w[0] : 0.f, two[c] ? w[1] : 0.f);
+  };
+  constexpr int NH = TAPS > 1 ? TAPS - 1 : 1, NW = TAPS ? TAPS : 1;
+  float2 hist[NH][NC], wr[NW][NC], gain[NC];
+  const float* norm = is_q ? a.q_norm : a.k_norm;
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int e = 2 * (lane + 32 * c);
+    gain[c] = is_v ? make_float2(1.f, 1.f) : make_float2(has[c] ? norm[e] : 0.f, two[c] ? norm[e + 1] : 0.f);
+    if (TAPS) {
+#pragma unroll
+      for (int j = 0; j < NW; ++j) wr[j][c] = weight(j, c);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) hist[j][c] = input(i0 - (TAPS - 1) + j, c);
+    }
+  }
+  const bool keep = n <= a.R - (taps - 1);              // short runs leave every input (a single tile), long ones the last taps - 1
+  for (int i = i0; i < i1; ++i) {
+    const int row = row0 + i;
+    float2 y[NC];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const float2 cur = input(i, c);
+      float2 s = make_float2(0.f, 0.f);
+      if (TAPS) {
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) { s.x = fmaf(wr[j][c].x, hist[j][c].x, s.x); s.y = fmaf(wr[j][c].y, hist[j][c].y, s.y); }
+        s.x = fmaf(wr[NW - 1][c].x, cur.x, s.x); s.y = fmaf(wr[NW - 1][c].y, cur.y, s.y);
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][c] = hist[j + 1][c];
+        if (TAPS > 1) hist[NH - 1][c] = cur;
+      } else {
+        for (int j = 0; j < taps; ++j) {
+          const float2 u = j == taps - 1 ? cur : input(i - (taps - 1) + j, c), w = weight(j, c);
+          s.x = fmaf(w.x, u.x, s.x); s.y = fmaf(w.y, u.y, s.y);
+        }
+      }
+      if (keep && has[c]) store_pair<T>(ring + (size_t)((p0 + i) % a.R) * a.C + 2 * (lane + 32 * c), cur, two[c], rvec[c]);
+      y[c] = s;
+      ss = fmaf(s.x, s.x, fmaf(s.y, s.y, ss));
+    }
+    T* dst;
+    if (is_q) dst = a.q + (size_t)row * a.q_stride + (size_t)head * a.dp;
+    else {
+      const int cs = a.slot_map[row];
+      if (cs < 0 || cs >= a.n_slots) { if (lane == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, row); continue; }     // warp-uniform
+      dst = a.cache + (size_t)cs * a.row_stride + (is_v ? (size_t)a.G * a.dp + (size_t)head * a.dvp : (size_t)head * a.dp);
+    }
+    if (!is_v) {
+      const float inv = rsqrtf(warp_sum(ss) / (float)d + a.eps);
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        y[c].x *= inv * gain[c].x; y[c].y *= inv * gain[c].y;
+        const int pr = lane + 32 * c;
+        if (pr < a.pairs) {
+          const float2 cs = a.rope[(size_t)row * a.pairs + pr];
+          y[c] = make_float2(y[c].x * cs.x - y[c].y * cs.y, y[c].y * cs.x + y[c].x * cs.y);
+        }
+      }
+    }
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+      if (has[c]) store_pair<T>(dst + 2 * (lane + 32 * c), y[c], two[c], two[c]);       // head starts are multiples of 64 elements
+  }
+  if (!keep && i0 == 0)          // this block read the old ring rows of these channels above: it may overwrite them now
+    for (int i = max(0, n - (taps - 1)); i < n; ++i)
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+        if (has[c]) store_pair<T>(ring + (size_t)((p0 + i) % a.R) * a.C + 2 * (lane + 32 * c), input(i, c), two[c], rvec[c]);
+}
+
+// ---------------------------------------------------------------- short convolution in front of the recurrence
+template <typename T>
+struct RecConv {
+  const T* proj; int ldp;                       // rows whose columns [0, C) are the x branch
+  const float* x_b; const float* w; const float* w_b;       // [C], [taps, C], [C]
+  T* ring;                                      // [slots, R, C] projected rows (without x_b) by position
+  const int* state_slot; const int* q_start; const int* q_len; const int* kv_len;
+  T* u; int ldt, sq, sqp;                       // block-major operand: channel b * sq + j of row t at ((b * ldt) + t) * sqp + j
+  int4* tiles; int* n_tiles;                    // tile table of the gate product: {block, first operand row, rows, 0}
+  int T_rows, tn, C, taps, R, n_state;
+  int* status;
+};
+
+template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, float* v) {
+  if constexpr (V == 4 && sizeof(T) == 2) {
+    const uint2 q = *(const uint2*)p;
+    const float2 x = __bfloat1622float2(*(const bf162*)&q.x), y = __bfloat1622float2(*(const bf162*)&q.y);
+    v[0] = x.x; v[1] = x.y; v[2] = y.x; v[3] = y.y;
+  } else if constexpr (V == 4) {
+    const float4 q = *(const float4*)p;
+    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+  } else if constexpr (V == 2 && sizeof(T) == 2) {
+    const float2 x = __bfloat1622float2(*(const bf162*)p);
+    v[0] = x.x; v[1] = x.y;
+  } else if constexpr (V == 2) {
+    const float2 x = *(const float2*)p;
+    v[0] = x.x; v[1] = x.y;
+  } else {
+    v[0] = to_f(p[0]);
+  }
+}
+template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const float* v) {
+  if constexpr (V == 4 && sizeof(T) == 2) {
+    const bf162 x = __floats2bfloat162_rn(v[0], v[1]), y = __floats2bfloat162_rn(v[2], v[3]);
+    *(uint2*)p = make_uint2(*(const uint32_t*)&x, *(const uint32_t*)&y);
+  } else if constexpr (V == 4) {
+    *(float4*)p = make_float4(v[0], v[1], v[2], v[3]);
+  } else if constexpr (V == 2 && sizeof(T) == 2) {
+    *(bf162*)p = __floats2bfloat162_rn(v[0], v[1]);
+  } else if constexpr (V == 2) {
+    *(float2*)p = make_float2(v[0], v[1]);
+  } else {
+    p[0] = to_t<T>(v[0]);
+  }
+}
+
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(128) rglru_conv_kernel(const RecConv<T> a) {
+  pdl_launch(); pdl_wait();
+  if (blockIdx.x == 0 && blockIdx.y == 0 && blockIdx.z == 0 && a.tiles) {
+    const int per = (a.T_rows + a.tn - 1) / a.tn, nt = a.C / a.sq * per;
+    for (int i = threadIdx.x; i < nt; i += blockDim.x) {
+      const int b = i / per, r0 = (i % per) * a.tn;
+      a.tiles[i] = make_int4(b, b * a.ldt + r0, min(a.tn, a.T_rows - r0), 0);
+    }
+    if (threadIdx.x == 0) *a.n_tiles = nt;
+  }
+  const int ch = (blockIdx.x * blockDim.x + threadIdx.x) * V, seq = blockIdx.z;
+  const int n = a.q_len[seq], i0 = blockIdx.y * HS_TILE;
+  if (ch >= a.C || i0 >= n) return;
+  const int row0 = a.q_start[seq], p0 = a.kv_len[seq] - n, slot = a.state_slot[seq], i1 = min(n, i0 + HS_TILE);
+  if (slot < 0 || slot >= a.n_state) { if (ch == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6E2); return; }
+  const int taps = TAPS ? TAPS : a.taps;
+  T* ring = a.ring + (size_t)slot * a.R * a.C + ch;
+  T* u = a.u + ((size_t)(ch / a.sq) * a.ldt + row0) * a.sqp + ch % a.sq;
+  float xb[V], wb[V];
+  load_v<float, V>(a.x_b + ch, xb); load_v<float, V>(a.w_b + ch, wb);
+  auto raw = [&](int i, float* v) { load_v<T, V>(a.proj + (size_t)(row0 + i) * a.ldp + ch, v); };
+  auto input = [&](int i, float* v) {
+    const int pos = p0 + i;
+    if (pos < 0) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) v[k] = 0.f;
+      return;
+    }
+    if (i >= 0) raw(i, v);
+    else load_v<T, V>(ring + (size_t)(pos % a.R) * a.C, v);
+#pragma unroll
+    for (int k = 0; k < V; ++k) v[k] += xb[k];
+  };
+  constexpr int NH = TAPS > 1 ? TAPS - 1 : 1, NW = TAPS ? TAPS : 1;
+  float hist[NH][V], wr[NW][V];
+  if (TAPS) {
+#pragma unroll
+    for (int j = 0; j < NW; ++j) load_v<float, V>(a.w + (size_t)j * a.C + ch, wr[j]);
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) input(i0 - (TAPS - 1) + j, hist[j]);
+  }
+  const bool keep = n <= a.R - (taps - 1);
+  for (int i = i0; i < i1; ++i) {
+    float cur[V], y[V], r[V];
+    raw(i, r);
+    if (keep) store_v<T, V>(ring + (size_t)((p0 + i) % a.R) * a.C, r);
+#pragma unroll
+    for (int k = 0; k < V; ++k) { cur[k] = r[k] + xb[k]; y[k] = wb[k]; }
+    if (TAPS) {
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[k] = fmaf(wr[j][k], hist[j][k], y[k]);
+#pragma unroll
+      for (int k = 0; k < V; ++k) y[k] = fmaf(wr[NW - 1][k], cur[k], y[k]);
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS - 1; ++j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) hist[j][k] = hist[j + 1][k];
+      if (TAPS > 1)
+#pragma unroll
+        for (int k = 0; k < V; ++k) hist[NH - 1][k] = cur[k];
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        float w[V], s[V];
+        load_v<float, V>(a.w + (size_t)j * a.C + ch, w);
+        input(i - (taps - 1) + j, s);
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[k] = fmaf(w[k], s[k], y[k]);
+      }
+    }
+    store_v<T, V>(u + (size_t)i * a.sqp, y);
+  }
+  if (!keep && i0 == 0)
+    for (int i = max(0, n - (taps - 1)); i < n; ++i) {
+      float r[V];
+      raw(i, r);
+      store_v<T, V>(ring + (size_t)((p0 + i) % a.R) * a.C, r);
+    }
+}
+
+// ---------------------------------------------------------------- real-gated linear recurrence
+//   log a = decay * sigmoid(zr),  S <- a S + sqrt(1 - a^2) sigmoid(zi) u,  out = S * gelu(y)
+template <typename T>
+struct LruScan {
+  const T* u; int ldt, sq, sqp;                 // block-major operand of the gate product
+  const float* gates; int ldg;                  // [T, ldg]: block b's decay gate at columns [2 b sq, + sq), input gate at the next sq
+  const float* gates_b; const float* decay;     // the same order; [C]
+  const T* y; int ldy; const float* y_b;        // y branch rows and bias
+  float* state;                                 // [slots, depth + 1, C] states by position
+  const int* state_slot; const int* q_start; const int* q_len; const int* kv_len;
+  float2* agg;                                  // chunk aggregates [.., C]: first chunk {state in front, state behind}, later ones {decay, sum}
+  T* out; int ldo;
+  int C, depth, n_state;
+  int* status;
+};
+
+// PASS 0: aggregates of every chunk but a run's last one; 1: outputs and states.
+template <typename T, int V, int PASS>
+__global__ void __launch_bounds__(128) lru_scan_kernel(const LruScan<T> a) {
+  pdl_launch(); pdl_wait();
+  constexpr int NB = 4;                         // rows loaded together: nothing but the state depends on the row before
+  const int ch = (blockIdx.x * blockDim.x + threadIdx.x) * V, c = blockIdx.y, seq = blockIdx.z;
+  const int n = a.q_len[seq], chunks = (n + HS_CHUNK - 1) / HS_CHUNK;
+  if (ch >= a.C || c >= chunks || (PASS == 0 && c == chunks - 1)) return;
+  const int row0 = a.q_start[seq], p0 = a.kv_len[seq] - n, slot = a.state_slot[seq];
+  if (slot < 0 || slot >= a.n_state) { if (ch == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6E3); return; }
+  const int b = ch / a.sq, j0 = ch % a.sq, gc = 2 * b * a.sq + j0;
+  const T* u = a.u + ((size_t)b * a.ldt + row0) * a.sqp + j0;
+  const float* g = a.gates + (size_t)row0 * a.ldg + gc;
+  float* st = a.state + (size_t)slot * (a.depth + 1) * a.C + ch;
+  // aggregates of a run's chunks are consecutive rows; q_start / CHUNK + seq keeps the runs of a step apart
+  float2* agg = a.agg + (size_t)(row0 / HS_CHUNK + seq) * a.C + ch;
+  float rb[V], ib[V], dk[V], yb[V], h[V], A[V], h0[V];
+  load_v<float, V>(a.gates_b + gc, rb); load_v<float, V>(a.gates_b + gc + a.sq, ib); load_v<float, V>(a.decay + ch, dk);
+  if (PASS == 1) load_v<float, V>(a.y_b + ch, yb);
+#pragma unroll
+  for (int k = 0; k < V; ++k) { h[k] = 0.f; A[k] = 1.f; }
+  if (c == 0 && (PASS == 0 || chunks == 1)) {
+    if (p0 > 0) load_v<float, V>(st + (size_t)((p0 - 1) % (a.depth + 1)) * a.C, h);
+  } else if (PASS == 1) {
+    // the first chunk's entry holds both its ends, so no block reads the ring that the last chunk's block writes
+#pragma unroll
+    for (int k = 0; k < V; ++k) { const float2 f = agg[k]; h[k] = c == 0 ? f.x : f.y; }
+    for (int q0 = 1; q0 < c; q0 += 8) {
+      float2 f[8][V];
+#pragma unroll
+      for (int q = 0; q < 8; ++q)
+#pragma unroll
+        for (int k = 0; k < V; ++k) f[q][k] = q0 + q < c ? agg[(size_t)(q0 + q) * a.C + k] : make_float2(1.f, 0.f);
+#pragma unroll
+      for (int q = 0; q < 8; ++q)
+#pragma unroll
+        for (int k = 0; k < V; ++k) h[k] = fmaf(f[q][k].x, h[k], f[q][k].y);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < V; ++k) h0[k] = h[k];
+  const int i1 = min(n, (c + 1) * HS_CHUNK);
+  for (int i0 = c * HS_CHUNK; i0 < i1; i0 += NB) {
+    float zr[NB][V], zi[NB][V], us[NB][V], ys[NB][V];
+#pragma unroll
+    for (int q = 0; q < NB; ++q) {
+      const int i = min(i0 + q, i1 - 1);
+      load_v<float, V>(g + (size_t)i * a.ldg, zr[q]); load_v<float, V>(g + (size_t)i * a.ldg + a.sq, zi[q]);
+      load_v<T, V>(u + (size_t)i * a.sqp, us[q]);
+      if (PASS == 1) load_v<T, V>(a.y + (size_t)(row0 + i) * a.ldy + ch, ys[q]);
+    }
+#pragma unroll
+    for (int q = 0; q < NB; ++q) {
+      const int i = i0 + q;
+      if (i >= i1) break;
+      float o[V];
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        const float la = dk[k] / (1.f + expf(-(zr[q][k] + rb[k]))), gate = 1.f / (1.f + expf(-(zi[q][k] + ib[k])));
+        // with m = a - 1: a S = S + m S and 1 - a^2 = -m (m + 2), both exact to rounding where a is close to 1 (long memories)
+        const float m = expm1f(la);
+        h[k] = fmaf(m, h[k], h[k]) + sqrtf(-m * (m + 2.f)) * gate * us[q][k];
+        if (PASS == 0) A[k] = fmaf(m, A[k], A[k]);
+        if (PASS == 1) {
+          const float z = ys[q][k] + yb[k];
+          o[k] = h[k] * z / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z)));      // 0.5 (1 + tanh(w)) = sigmoid(2 w)
+        }
+      }
+      if (PASS == 1) {
+        store_v<T, V>(a.out + (size_t)(row0 + i) * a.ldo + ch, o);
+        if (n <= a.depth || i == n - 1) store_v<float, V>(st + (size_t)((p0 + i) % (a.depth + 1)) * a.C, h);
+      }
+    }
+  }
+  if (PASS == 0)
+#pragma unroll
+    for (int k = 0; k < V; ++k) agg[(size_t)c * a.C + k] = make_float2(c == 0 ? h0[k] : A[k], h[k]);
+}
+
+// ---------------------------------------------------------------- clamped GLU over two projected rows
+template <typename T>
+__global__ void glu_rows_kernel(const T* __restrict__ g, const T* __restrict__ u, const float* __restrict__ gb, const float* __restrict__ ub, T* __restrict__ out,
+                                int ldi, int ldo, int N, float limit) {
+  pdl_launch(); pdl_wait();
+  const int t = blockIdx.x;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < N; i += gridDim.y * blockDim.x) {
+    const float gv = fminf(to_f(g[(size_t)t * ldi + i]) + gb[i], limit), uv = fminf(fmaxf(to_f(u[(size_t)t * ldi + i]) + ub[i], -limit), limit);
+    out[(size_t)t * ldo + i] = to_t<T>(gv / (1.f + expf(-1.702f * gv)) * (uv + 1.f));
+  }
+}
+
+// ---------------------------------------------------------------- windowed grouped-query attention on the ordinary cores
+// One block per (query row, head): scores of a page of keys (a warp takes 16 of them), online softmax, weighted sum of the page's values
+// (a thread owns columns tid, tid + 128, ...).
+#define WA_COLS 4
+template <typename T>
+__global__ void __launch_bounds__(128) window_attn_simt_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ cache, const int* __restrict__ page_table,
+                                                               const int* __restrict__ kv_len, const int* __restrict__ q_start, const int* __restrict__ q_len,
+                                                               T* __restrict__ out, int ldo, int n_seq, int G, int group, int dp, int dvp, int dv, int row_stride,
+                                                               int max_pages, int n_slots, int window, float scale, int* status) {
+  pdl_launch(); pdl_wait();
+  extern __shared__ float qs[];
+  __shared__ float sc[64];
+  const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, kh = h / group;
+  int seq = -1;
+  for (int s = 0; s < n_seq; ++s) if (t >= q_start[s] && t < q_start[s] + q_len[s]) { seq = s; break; }
+  if (seq < 0) return;
+  const int pos = kv_len[seq] - q_len[seq] + t - q_start[seq], lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const T* qr = q + (size_t)t * q_stride + (size_t)h * dp;
+  for (int i = tid; i < dp; i += 128) qs[i] = to_f(qr[i]);
+  __syncthreads();
+  float m = -INFINITY, l = 0.f, o[WA_COLS];
+#pragma unroll
+  for (int j = 0; j < WA_COLS; ++j) o[j] = 0.f;
+  for (int k0 = lo / 64 * 64; k0 <= pos; k0 += 64) {
+    int slot0 = page_table[(size_t)seq * max_pages + k0 / 64] * 64;
+    if (slot0 < 0 || slot0 + 64 > n_slots) { if (tid == 0) ca_dev_fail(status, CA_DEV_BAD_INDEX, t); slot0 = 0; }
+    const T* kb = cache + (size_t)slot0 * row_stride + (size_t)kh * dp;
+    const T* vb = cache + (size_t)slot0 * row_stride + (size_t)G * dp + (size_t)kh * dvp;
+    const int n = min(64, pos + 1 - k0), first = max(0, lo - k0);
+    for (int j = warp * 16; j < warp * 16 + 16; ++j) {
+      float s = 0.f;
+      const bool in = j >= first && j < n;
+      if (in) for (int i = lane; i < dp; i += 32) s = fmaf(qs[i], to_f(kb[(size_t)j * row_stride + i]), s);
+      s = warp_sum(s);
+      if (lane == 0) sc[j] = in ? s * scale : -INFINITY;
+    }
+    __syncthreads();
+    const float s0 = sc[lane], s1 = sc[lane + 32];
+    const float mn = fmaxf(m, warp_max(fmaxf(s0, s1)));             // every page of the loop holds a visible key, so mn is finite
+    const float al = m == -INFINITY ? 0.f : expf(m - mn);
+    const float e0 = expf(s0 - mn), e1 = expf(s1 - mn);
+    l = l * al + warp_sum(e0 + e1);
+    m = mn;
+    __syncthreads();
+    if (warp == 0) { sc[lane] = e0; sc[lane + 32] = e1; }
+    __syncthreads();
+#pragma unroll
+    for (int c = 0; c < WA_COLS; ++c) {
+      const int i = tid + c * 128;
+      if (i < dv) {
+        float acc = o[c] * al;
+        for (int j = first; j < n; ++j) acc = fmaf(sc[j], to_f(vb[(size_t)j * row_stride + i]), acc);
+        o[c] = acc;
+      }
+    }
+    __syncthreads();
+  }
+  const float f = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+  for (int c = 0; c < WA_COLS; ++c) {
+    const int i = tid + c * 128;
+    if (i < dv) out[(size_t)t * ldo + (size_t)h * dv + i] = to_t<T>(o[c] * f);
+  }
+}
+
+// ---------------------------------------------------------------- C ABI
+struct CaNormRows {
+  float* x; const int* tokens; const void* table; const void* add; const float* bias; const float* post; const int* src_rows; const float* gain; void* xn; int* status;
+  int W, Wp, vocab, ldn; float mult, eps;
+};
+
+template <typename T, int MODE>
+static int norm_rows_launch(const CaNormRows* c, int rows, cudaStream_t s) {
+  const NormRows<T> a{c->x, c->W, c->Wp, c->tokens, (const bf16*)c->table, c->vocab, (const T*)c->add, c->bias, c->post, c->mult, c->src_rows, c->gain, (T*)c->xn, c->ldn, c->eps, c->status};
+  const int chunks = c->Wp / 8, most = rows <= 2 * ca_sm_count() ? 1024 : 256;
+  int nt = chunks <= most ? (chunks + 31) / 32 * 32 : most;
+  if ((chunks + nt - 1) / nt > 8) nt = 1024;
+  const int nch = (chunks + nt - 1) / nt;
+  if (nch == 1) CA_LAUNCH_PDL((norm_rows_kernel<T, 1, MODE>), rows, nt, 0, s, a);
+  else if (nch == 2) CA_LAUNCH_PDL((norm_rows_kernel<T, 2, MODE>), rows, nt, 0, s, a);
+  else if (nch <= 4) CA_LAUNCH_PDL((norm_rows_kernel<T, 4, MODE>), rows, nt, 0, s, a);
+  else if (nch <= 8) CA_LAUNCH_PDL((norm_rows_kernel<T, 8, MODE>), rows, nt, 0, s, a);
+  else return ca_fail(CA_ERR_ARG, "norm_rows: rows of %d elements (at most 65536)", c->Wp);
+  CA_CHECK_LAUNCH("norm_rows");
+  return CA_OK;
+}
+
+extern "C" int cuteafd_norm_rows(const CaNormRows* c, int mode, int rows, int f32, cudaStream_t s) {
+  CA_REQUIRE(c && c->x && c->W >= 1 && c->Wp >= c->W && c->Wp % 8 == 0 && (!c->xn || (c->gain && c->ldn % 8 == 0 && c->ldn >= c->Wp)), "norm_rows: bad arguments");
+  CA_REQUIRE(mode == ROWS_EMBED ? c->tokens && c->table && c->vocab > 0 : mode == ROWS_ADD ? c->add != nullptr : mode == ROWS_GATHER && c->src_rows && c->xn, "norm_rows: mode %d without its inputs", mode);
+  if (rows <= 0) return CA_OK;
+  if (mode == ROWS_EMBED) return f32 ? norm_rows_launch<float, ROWS_EMBED>(c, rows, s) : norm_rows_launch<bf16, ROWS_EMBED>(c, rows, s);
+  if (mode == ROWS_ADD) return f32 ? norm_rows_launch<float, ROWS_ADD>(c, rows, s) : norm_rows_launch<bf16, ROWS_ADD>(c, rows, s);
+  return f32 ? norm_rows_launch<float, ROWS_GATHER>(c, rows, s) : norm_rows_launch<bf16, ROWS_GATHER>(c, rows, s);
+}
+
+extern "C" int cuteafd_rope_table(const int* positions, const float* freq, float amp, int pairs, void* out, int T, cudaStream_t s) {
+  CA_REQUIRE(positions && freq && out && pairs >= 1, "rope_table: bad arguments");
+  if (T <= 0) return CA_OK;
+  CA_LAUNCH_PDL(rope_table_kernel, T, pairs < 128 ? (pairs + 31) / 32 * 32 : 128, 0, s, positions, freq, amp, pairs, (float2*)out);
+  CA_CHECK_LAUNCH("rope_table");
+  return CA_OK;
+}
+
+struct CaConvQkv {
+  const void* proj; const float* w; const float* q_norm; const float* k_norm; const void* rope; void* ring; const int* state_slot; const int* q_start; const int* q_len;
+  const int* kv_len; const int* slot_map; void* q; void* cache; int* status;
+  int ldp, q_stride, row_stride, n_slots, H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state, n_seq, max_q_len; float eps;
+};
+
+template <typename T, int NC>
+static int conv_qkv_launch(const CaConvQkv* c, cudaStream_t s) {
+  const ConvQkv<T> a{(const T*)c->proj, c->ldp, c->w, c->q_norm, c->k_norm, (const float2*)c->rope, (T*)c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len, c->slot_map,
+                     (T*)c->q, c->q_stride, (T*)c->cache, c->row_stride, c->n_slots, c->H, c->G, c->dim, c->dp, c->vdim, c->dvp, c->pairs, c->taps, c->R, c->C, c->n_state,
+                     c->eps, c->status};
+  const dim3 grid((c->H + 2 * c->G + 3) / 4, (c->max_q_len + HS_TILE - 1) / HS_TILE, c->n_seq);
+  if (c->taps == 2) CA_LAUNCH_PDL((conv_qkv_kernel<T, NC, 2>), grid, 128, 0, s, a);
+  else if (c->taps == 3) CA_LAUNCH_PDL((conv_qkv_kernel<T, NC, 3>), grid, 128, 0, s, a);
+  else if (c->taps == 4) CA_LAUNCH_PDL((conv_qkv_kernel<T, NC, 4>), grid, 128, 0, s, a);
+  else CA_LAUNCH_PDL((conv_qkv_kernel<T, NC, 0>), grid, 128, 0, s, a);
+  CA_CHECK_LAUNCH("conv_qkv");
+  return CA_OK;
+}
+
+extern "C" int cuteafd_conv_qkv(const CaConvQkv* c, int f32, cudaStream_t s) {
+  CA_REQUIRE(c && c->proj && c->w && c->q_norm && c->ring && c->state_slot && c->q_start && c->q_len && c->kv_len && c->slot_map && c->q, "conv_qkv: null argument");
+  CA_REQUIRE(c->H >= 1 && c->G >= 0 && (c->G == 0 || (c->k_norm && c->cache)) && c->taps >= 1 && c->taps <= HS_MAX_TAPS && c->R >= c->taps, "conv_qkv: bad geometry");
+  CA_REQUIRE(c->dim >= 1 && c->dim <= 256 && c->vdim <= 256 && c->dp % 8 == 0 && c->dvp % 8 == 0 && c->dim <= c->dp && c->vdim <= c->dvp && c->row_stride % 8 == 0, "conv_qkv: heads of up to 256 dimensions");
+  CA_REQUIRE(c->C == (c->H + c->G) * c->dim + c->G * c->vdim && c->ldp >= c->C && c->q_stride >= c->H * c->dp && (c->G == 0 || c->row_stride >= c->G * (c->dp + c->dvp)), "conv_qkv: row too short");
+  CA_REQUIRE(c->pairs >= 0 && 2 * c->pairs <= c->dim && (c->pairs == 0 || c->rope) && c->R - (c->taps - 1) <= HS_TILE, "conv_qkv: bad rotation or ring");
+  if (c->n_seq <= 0 || c->max_q_len <= 0) return CA_OK;
+  CA_REQUIRE(c->n_seq <= 65535 && (c->max_q_len + HS_TILE - 1) / HS_TILE <= 65535, "conv_qkv: step too large");
+  const int nc = ((c->dim > c->vdim || c->G == 0 ? c->dim : c->vdim) + 63) / 64;
+  if (nc <= 1) return f32 ? conv_qkv_launch<float, 1>(c, s) : conv_qkv_launch<bf16, 1>(c, s);
+  if (nc <= 2) return f32 ? conv_qkv_launch<float, 2>(c, s) : conv_qkv_launch<bf16, 2>(c, s);
+  return f32 ? conv_qkv_launch<float, 4>(c, s) : conv_qkv_launch<bf16, 4>(c, s);
+}
+
+struct CaRecurrence {          // one recurrent layer's step: shared by its convolution and its scan
+  const void* x; const void* y; const float* x_b; const float* y_b; const float* conv; const float* conv_b; void* ring; float* state; void* u; const float* gates;
+  const float* gates_b; const float* decay; void* agg; void* out; void* tiles; int* n_tiles; const int* state_slot; const int* q_start; const int* q_len; const int* kv_len;
+  int* status;
+  int ldp, ldt, sq, sqp, ldg, ldo, tn, T, C, taps, depth, n_state, n_seq, max_q_len, agg_rows;
+};
+
+template <typename T, int V>
+static int rglru_conv_launch(const CaRecurrence* c, cudaStream_t s) {
+  const RecConv<T> a{(const T*)c->x, c->ldp, c->x_b, c->conv, c->conv_b, (T*)c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len, (T*)c->u, c->ldt, c->sq, c->sqp,
+                     (int4*)c->tiles, c->n_tiles, c->T, c->tn, c->C, c->taps, c->taps - 1 + c->depth, c->n_state, c->status};
+  const dim3 grid((c->C / V + 127) / 128, (c->max_q_len + HS_TILE - 1) / HS_TILE, c->n_seq);
+  if (c->taps == 2) CA_LAUNCH_PDL((rglru_conv_kernel<T, V, 2>), grid, 128, 0, s, a);
+  else if (c->taps == 3) CA_LAUNCH_PDL((rglru_conv_kernel<T, V, 3>), grid, 128, 0, s, a);
+  else if (c->taps == 4) CA_LAUNCH_PDL((rglru_conv_kernel<T, V, 4>), grid, 128, 0, s, a);
+  else CA_LAUNCH_PDL((rglru_conv_kernel<T, V, 0>), grid, 128, 0, s, a);
+  CA_CHECK_LAUNCH("rglru_conv");
+  return CA_OK;
+}
+
+template <typename T, int V>
+static int lru_scan_launch(const CaRecurrence* c, cudaStream_t s) {
+  const LruScan<T> a{(const T*)c->u, c->ldt, c->sq, c->sqp, c->gates, c->ldg, c->gates_b, c->decay, (const T*)c->y, c->ldp, c->y_b, c->state, c->state_slot, c->q_start,
+                     c->q_len, c->kv_len, (float2*)c->agg, (T*)c->out, c->ldo, c->C, c->depth, c->n_state, c->status};
+  const int chunks = (c->max_q_len + HS_CHUNK - 1) / HS_CHUNK;
+  const dim3 grid((c->C / V + 127) / 128, chunks, c->n_seq);
+  if (chunks > 1) {
+    CA_LAUNCH_PDL((lru_scan_kernel<T, V, 0>), dim3(grid.x, chunks - 1, c->n_seq), 128, 0, s, a);
+    CA_CHECK_LAUNCH("lru_scan aggregates");
+  }
+  CA_LAUNCH_PDL((lru_scan_kernel<T, V, 1>), grid, 128, 0, s, a);
+  CA_CHECK_LAUNCH("lru_scan");
+  return CA_OK;
+}
+
+static bool recurrence_ok(const CaRecurrence* c) {
+  return c && c->state_slot && c->q_start && c->q_len && c->kv_len && c->u && c->C >= 1 && c->sq >= 1 && c->C % c->sq == 0 && c->sqp >= c->sq && c->ldt >= c->T &&
+         c->taps >= 1 && c->taps <= HS_MAX_TAPS && c->depth >= 1 && c->depth <= HS_TILE && c->n_state >= 1 && c->n_seq <= 65535 && c->max_q_len <= 65535 * HS_TILE;
+}
+
+extern "C" int cuteafd_rglru_conv(const CaRecurrence* c, int f32, cudaStream_t s) {
+  CA_REQUIRE(recurrence_ok(c) && c->x && c->x_b && c->conv && c->conv_b && c->ring && (!c->tiles || (c->n_tiles && c->tn >= 1)) && c->ldp >= c->C, "rglru_conv: bad arguments");
+  if (c->n_seq <= 0 || c->max_q_len <= 0) return CA_OK;
+  const bool v4 = c->sq % 4 == 0 && c->sqp % 4 == 0 && c->ldp % 4 == 0 && ((uintptr_t)c->x & 15) == 0;
+  if (v4) return f32 ? rglru_conv_launch<float, 4>(c, s) : rglru_conv_launch<bf16, 4>(c, s);
+  return f32 ? rglru_conv_launch<float, 1>(c, s) : rglru_conv_launch<bf16, 1>(c, s);
+}
+
+extern "C" int cuteafd_lru_scan(const CaRecurrence* c, int f32, cudaStream_t s) {
+  CA_REQUIRE(recurrence_ok(c) && c->gates && c->gates_b && c->decay && c->y && c->y_b && c->state && c->out && c->ldg >= 2 * c->C && c->ldo >= c->C && c->ldp >= c->C, "lru_scan: bad arguments");
+  if (c->n_seq <= 0 || c->max_q_len <= 0) return CA_OK;
+  CA_REQUIRE(c->max_q_len <= HS_CHUNK || (c->agg && c->agg_rows >= c->T / HS_CHUNK + c->n_seq + 1), "lru_scan: runs of more than %d tokens need room for their aggregates", HS_CHUNK);
+  const bool v2 = c->sq % 2 == 0 && c->sqp % 2 == 0 && c->ldp % 2 == 0 && c->ldo % 2 == 0 && c->ldg % 2 == 0 && ((uintptr_t)c->y & 7) == 0;
+  if (v2) return f32 ? lru_scan_launch<float, 2>(c, s) : lru_scan_launch<bf16, 2>(c, s);
+  return f32 ? lru_scan_launch<float, 1>(c, s) : lru_scan_launch<bf16, 1>(c, s);
+}
+
+extern "C" int cuteafd_glu_rows(const void* g, const void* u, const float* gb, const float* ub, void* out, int T, int ldi, int ldo, int N, float limit, int f32, cudaStream_t s) {
+  CA_REQUIRE(g && u && gb && ub && out && N >= 1 && ldi >= N && ldo >= N, "glu_rows: bad arguments");
+  if (T <= 0) return CA_OK;
+  const dim3 grid(T, (N + 1023) / 1024);
+  if (f32) CA_LAUNCH_PDL(glu_rows_kernel<float>, grid, 256, 0, s, (const float*)g, (const float*)u, gb, ub, (float*)out, ldi, ldo, N, limit);
+  else CA_LAUNCH_PDL(glu_rows_kernel<bf16>, grid, 256, 0, s, (const bf16*)g, (const bf16*)u, gb, ub, (bf16*)out, ldi, ldo, N, limit);
+  CA_CHECK_LAUNCH("glu_rows");
+  return CA_OK;
+}
+
+extern "C" int cuteafd_window_attention_simt(const void* q, int q_stride, const void* cache, const int* page_table, const int* kv_len, const int* q_start, const int* q_len,
+                                             void* out, int ldo, int T, int n_seq, int Hq, int Hkv, int dp, int dvp, int dv, int row_stride, int max_pages, int n_slots,
+                                             int window, float scale, int f32, int* status, cudaStream_t s) {
+  CA_REQUIRE(q && cache && page_table && kv_len && q_start && q_len && out, "window_attention_simt: null argument");
+  CA_REQUIRE(Hkv >= 1 && Hq % Hkv == 0 && Hq <= 65535 && dv >= 1 && dv <= dvp && dv <= 128 * WA_COLS && dp >= 1 && dp <= 4096 && row_stride >= Hkv * (dp + dvp) && ldo >= Hq * dv,
+             "window_attention_simt: bad shape");
+  if (T <= 0 || n_seq <= 0) return CA_OK;
+  if (f32) CA_LAUNCH_PDL(window_attn_simt_kernel<float>, dim3(T, Hq), 128, dp * sizeof(float), s, (const float*)q, q_stride, (const float*)cache, page_table, kv_len, q_start, q_len, (float*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, max_pages, n_slots, window, scale, status);
+  else CA_LAUNCH_PDL(window_attn_simt_kernel<bf16>, dim3(T, Hq), 128, dp * sizeof(float), s, (const bf16*)q, q_stride, (const bf16*)cache, page_table, kv_len, q_start, q_len, (bf16*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, max_pages, n_slots, window, scale, status);
+  CA_CHECK_LAUNCH("window_attention_simt");
+  return CA_OK;
+}

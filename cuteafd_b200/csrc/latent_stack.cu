@@ -9,35 +9,7 @@
 //   latent_attn_simt absorbed attention for what the tcgen05 kernels do not take (fp32, ranks above 512, more than 128 heads)
 // T is the type of the matrix-product operands and of the cache: bf16, or float for the all-fp32 mode.  Rows are padded to multiples of
 // 8 elements (pad weights are zero).  (No counterpart in the reference, which has no such family; the fused shapes follow moe.cu.)
-#include "common.cuh"
-
-template <typename T> __device__ __forceinline__ void load8(const T* p, float* v);
-template <> __device__ __forceinline__ void load8<bf16>(const bf16* p, float* v) {
-  const uint4 q = *(const uint4*)p;
-  const bf162* h = (const bf162*)&q;
-#pragma unroll
-  for (int j = 0; j < 4; ++j) { const float2 f = __bfloat1622float2(h[j]); v[2 * j] = f.x; v[2 * j + 1] = f.y; }
-}
-template <> __device__ __forceinline__ void load8<float>(const float* p, float* v) {
-  const float4 a = *(const float4*)p, b = *(const float4*)(p + 4);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-template <typename T> __device__ __forceinline__ void store8(T* p, const float* v);
-template <> __device__ __forceinline__ void store8<bf16>(bf16* p, const float* v) {
-  uint32_t w[4];
-#pragma unroll
-  for (int j = 0; j < 4; ++j) { const bf162 h = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]); w[j] = *(const uint32_t*)&h; }
-  *(uint4*)p = make_uint4(w[0], w[1], w[2], w[3]);
-}
-template <> __device__ __forceinline__ void store8<float>(float* p, const float* v) {
-  *(float4*)p = make_float4(v[0], v[1], v[2], v[3]);
-  *(float4*)(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
-}
-template <typename T> __device__ __forceinline__ T to_t(float v);
-template <> __device__ __forceinline__ bf16 to_t<bf16>(float v) { return __float2bfloat16(v); }
-template <> __device__ __forceinline__ float to_t<float>(float v) { return v; }
-__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
-__device__ __forceinline__ float to_f(float v) { return v; }
+#include "stack_rows.cuh"
 
 // What a row-producing kernel hands to the next matrix product: tanh(alpha x) w + b -> xn and / or the plain row -> cat.
 template <typename T>

@@ -63,7 +63,12 @@ struct TcArgs {
   long long* trace;           // optional per-unit time stamps [grid, trace_units, 8] (see cuteafd_tc_trace)
   int ldsfb, ldy, rows_total, N, K, epi, splits, trace_units;
   int w4_tx;                  // KIND_W4A8: bytes one weight tile adds to the stage barrier's transaction count
-  int act;                    // activation of the plain epilogue: 0 none, 1 squared ReLU (experts without a gate projection)
+  // activation: 0 none (SWIGLU mode: silu(g) * u), 1 squared ReLU (experts without a gate projection); XACT instantiations only:
+  // 2 soft cap act_p * tanh(v / act_p) (logits), 3 SWIGLU mode's clamped GLU with biases and limit act_p
+  int act;
+  float act_p;
+  const float* bias;          // act 3: [N] of the gate and of the linear half
+  const float* bias2;
   // grouped GEMM over head-major operands (row = group * grp_rows + token) with a token-major result: group g writes columns
   // [g * grp_cols, g * grp_cols + N) of row `token`; grp_rows 0 = the output row is the operand row
   int grp_rows, grp_cols;
@@ -156,9 +161,17 @@ __device__ __forceinline__ void peer_store(const TcArgs& a, int row, int n, bf16
   if (a.n_peer > 1) ((bf16*)a.peer_y1)[prow * a.peer_ld + n] = v;
 }
 
+// Values of an XACT instantiation: bounded logits, or g = min(g + b, p), u = clamp(u + b2, -p, p) -> g * sigmoid(1.702 g) * (u + 1).
+__device__ __forceinline__ float epi_softcap(const TcArgs& a, float v) { return a.act == 2 ? a.act_p * tanhf(v / a.act_p) : v; }
+__device__ __forceinline__ float epi_clamped_glu(const TcArgs& a, float g, float u, float b, float b2) {
+  g = fminf(g + b, a.act_p); u = fminf(fmaxf(u + b2, -a.act_p), a.act_p);
+  return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+}
+
 // PEER instantiations carry the peer-store epilogue; the others are the plain local kernels (the extra code costs
 // ~1.5 us per launch even when switched off at run time, so it is compiled in only where it is used).
-template <int KIND, int TN, bool SWIGLU, bool PEER, bool QOUT>
+// (XACT: the epilogues with biases or a soft cap, for the same reason.)
+template <int KIND, int TN, bool SWIGLU, bool PEER, bool QOUT, bool XACT>
 __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_kernel(const __grid_constant__ TcArgs a) {
   using C = TcCfg<KIND, TN, SWIGLU>;
   extern __shared__ uint8_t smem_raw[];
@@ -356,6 +369,7 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
       const float al2 = (SWIGLU && a.alpha2) ? a.alpha2[g] : al;
       const uint32_t tbase = tmem + ((uint32_t)(q4 * 32) << 16) + acc * C::ACC_COLS;
       float* ws = (splits > 1) ? a.splitk_ws + ((size_t)sp * a.rows_total) * a.N : nullptr;
+      const float xb = (XACT && SWIGLU && n_ok) ? a.bias[n] : 0.f, xb2 = (XACT && SWIGLU && n_ok) ? a.bias2[n] : 0.f;
       const size_t obase = a.grp_rows > 0 ? (size_t)(row0 - g * a.grp_rows) * a.ldy + (size_t)g * a.grp_cols : (size_t)row0 * a.ldy;
 #pragma unroll 1
       for (int c0 = 0; c0 < TN; c0 += 16) {
@@ -434,8 +448,9 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
               float v = __uint_as_float(r[j]) * al;
               if (SWIGLU) {
                 const float u = __uint_as_float(r2[j]) * al2;
-                v = v / (1.f + __expf(-v)) * u;
-              } else if (a.act) { v = fmaxf(v, 0.f); v *= v; }
+                v = XACT ? epi_clamped_glu(a, v, u, xb, xb2) : v / (1.f + __expf(-v)) * u;
+              } else if (XACT) v = epi_softcap(a, v);
+              else if (a.act) { v = fmaxf(v, 0.f); v *= v; }
               buf[j * 128 + et] = v;
             }
             mbar_arrive(&stg_bar);
@@ -476,8 +491,9 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
               float v = __uint_as_float(r[j]) * al;
               if (SWIGLU) {
                 const float u = __uint_as_float(r2[j]) * al2;
-                v = v / (1.f + __expf(-v)) * u;
-              } else if (a.act) { v = fmaxf(v, 0.f); v *= v; }
+                v = XACT ? epi_clamped_glu(a, v, u, xb, xb2) : v / (1.f + __expf(-v)) * u;
+              } else if (XACT) v = epi_softcap(a, v);
+              else if (a.act) { v = fmaxf(v, 0.f); v *= v; }
               const size_t o = obase + (size_t)c * a.ldy + n;
               if (splits > 1) ws[(size_t)(row0 + c) * a.N + n] = v;
               else if (a.epi == EPI_F32) ((float*)a.Y)[o] = v;
@@ -561,10 +577,10 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
   if (warp == 1) tmem_dealloc(tmem, C::TMEM_COLS);
 }
 
-template <int KIND, int TN, bool SWIGLU, bool PEER, bool QOUT>
+template <int KIND, int TN, bool SWIGLU, bool PEER, bool QOUT, bool XACT = false>
 static int launch_p(const TcArgs& a, int grid, cudaStream_t stream) {
   using C = TcCfg<KIND, TN, SWIGLU>;
-  auto kern = tc_linear_kernel<KIND, TN, SWIGLU, PEER, QOUT>;
+  auto kern = tc_linear_kernel<KIND, TN, SWIGLU, PEER, QOUT, XACT>;
   static bool attr_set[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -579,6 +595,7 @@ static int launch_p(const TcArgs& a, int grid, cudaStream_t stream) {
 
 template <int KIND, int TN, bool SWIGLU>
 static int launch(const TcArgs& a, int grid, cudaStream_t stream) {
+  if constexpr (KIND == KIND_BF16) { if (a.act >= 2) return launch_p<KIND, TN, SWIGLU, false, false, true>(a, grid, stream); }
   if constexpr (!SWIGLU) { if (a.n_peer) return launch_p<KIND, TN, false, true, false>(a, grid, stream); }
   if constexpr (SWIGLU && KIND != KIND_BF16) { if (a.q_out) return launch_p<KIND, TN, true, false, true>(a, grid, stream); }
   return launch_p<KIND, TN, SWIGLU, false, false>(a, grid, stream);
@@ -1004,11 +1021,14 @@ extern "C" int cuteafd_tc_linear(int kind, int swiglu, int tn, const void* tmA, 
   CA_REQUIRE(epi == EPI_BF16 || epi == EPI_BF16_RESIDUAL || epi == EPI_F32, "tc_linear: bad epilogue %d", epi);
   CA_REQUIRE(epi != EPI_BF16_RESIDUAL || R, "tc_linear: residual epilogue needs R");
   const int act = extra ? extra->act : 0, grp_rows = extra ? extra->grp_rows : 0, grp_cols = extra ? extra->grp_cols : 0;
-  CA_REQUIRE(act == 0 || (act == 1 && !swiglu && splits <= 1 && !q_out && epi != EPI_BF16_RESIDUAL), "tc_linear: the squared-ReLU epilogue is plain (no SwiGLU, split-K, FP4 output or residual)");
+  CA_REQUIRE(act == 0 || (act >= 1 && act <= 3 && splits <= 1 && !q_out && epi != EPI_BF16_RESIDUAL && (act == 3) == (swiglu != 0)),
+             "tc_linear: squared ReLU and soft cap are plain epilogues, the clamped GLU one of two weights (no split-K, FP4 output or residual)");
+  CA_REQUIRE(act < 2 || (kind == KIND_BF16 && !peer.n && extra->act_p > 0.f && (act == 2 || (extra->bias && extra->bias2))),
+             "tc_linear: soft cap and clamped GLU take bf16 operands, a positive bound and (GLU) two biases");
   CA_REQUIRE(grp_rows == 0 || (grp_rows > 0 && tiles && !swiglu && !q_out && !peer.n && epi != EPI_BF16_RESIDUAL), "tc_linear: token-major output belongs to a plain grouped GEMM");
   if (rows_total <= 0 || N <= 0) return CA_OK;
   TcArgs a;
-  a.act = act; a.grp_rows = grp_rows; a.grp_cols = grp_cols;
+  a.act = act; a.act_p = extra ? extra->act_p : 0.f; a.bias = extra ? extra->bias : nullptr; a.bias2 = extra ? extra->bias2 : nullptr; a.grp_rows = grp_rows; a.grp_cols = grp_cols;
   a.tmA = (const CUtensorMap*)tmA; a.tmA2 = (const CUtensorMap*)tmA2; a.tmB = (const CUtensorMap*)tmB;
   a.sfa = (const uint8_t* const*)sfa; a.sfa2 = (const uint8_t* const*)sfa2; a.sfb = (const uint8_t*)sfb;
   a.alpha = alpha; a.alpha2 = alpha2; a.tiles = (const int4*)tiles; a.n_tiles = n_tiles;

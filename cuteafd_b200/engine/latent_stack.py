@@ -27,54 +27,19 @@ import torch
 
 from .. import ops
 from ..models.latent_stack import StackLayer, StackWeights, up
-from ..ops import ActBuffer, KIND_BF16, KIND_F32, native, pick_tn
+from ..ops import ActBuffer, KIND_BF16, native, pick_tn
 from ..ops.native import call, ptr, stream
-from .engine import PAGE, Lane, StepShape
+from .engine import PAGE, StepShape
 from .mla import MlaEngine
+from .stack import StackBase, StackLane
 
-LANE_CAPS = (16, 32, 64, 256, 1024, 4096, 16384)
 
-
-class StackLane(Lane):
-    """Activation buffers for steps of up to `cap` rows; buffers that depend on a layer's geometry are made on first use per geometry."""
-
+class LatentLane(StackLane):
     def __init__(self, eng: "LatentStackEngine", cap: int):
-        self.eng, self.cap, self.dev = eng, cap, eng.device
-        self.dt = torch.float32 if eng.f32 else torch.bfloat16
-        self.kind = KIND_F32 if eng.f32 else KIND_BF16
-        # no product of these layers pairs two weight tiles, so 256-row token tiles keep both accumulators: prompt-sized lanes take them
-        self.tn = pick_tn(min(cap, int(os.environ.get("CUTEAFD_TN", "256" if cap >= 1024 else "128"))))
-        Wp = eng.Wp
-        self.x = torch.zeros(cap, Wp, dtype=torch.float32, device=self.dev)
-        self.xn, self.xn_act = self._operand(cap, Wp)
-        self.mix = torch.zeros(cap, Wp, dtype=self.dt, device=self.dev)
+        super().__init__(eng, cap)
         self.cat = self.cat_act = None
         if eng.spec.loop is not None:
-            self.cat, self.cat_act = self._operand(cap, 2 * Wp)
-        rows = min(cap, 256)
-        self.xln, self.xln_act = self._operand(rows, Wp)
-        self.logits = torch.zeros(rows, eng.spec.vocab, dtype=torch.float32, device=self.dev)
-        i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=self.dev)
-        self.next_tok, self.tok_status = i32(cap), i32(cap)
-        self._bufs: dict = {}
-
-    def _operand(self, rows: int, K: int, tn: int | None = None):
-        act = ActBuffer.alloc(self.kind, rows, K, tn or self.tn, self.dev)
-        return act.data, act
-
-    def ensure_logits(self, n: int):
-        """Steps that want more logit rows than a lane starts with (whole prompts scored position by position)."""
-        if n > self.logits.shape[0]:
-            rows = min(self.cap, up(n, 256))
-            self.xln, self.xln_act = self._operand(rows, self.eng.Wp)
-            self.logits = torch.zeros(rows, self.eng.spec.vocab, dtype=torch.float32, device=self.dev)
-            self.eng.graphs.clear()                  # captured steps hold the old addresses
-            self.eng.census.invalidate()
-
-    def get(self, key, make):
-        if key not in self._bufs:
-            self._bufs[key] = make()
-        return self._bufs[key]
+            self.cat, self.cat_act = self._operand(cap, 2 * eng.Wp)
 
     def mixer(self, a, n_in: int) -> dict:
         """Buffers of one mixer geometry (head-major buffers are [heads, cap, .]: head h of row t is row h * cap + t)."""
@@ -116,12 +81,13 @@ class StackLane(Lane):
         return self.get(("moe", E, k, ff), make)
 
 
-class LatentStackEngine(MlaEngine):
+class LatentStackEngine(StackBase, MlaEngine):
+    LANE = LatentLane
+
     def __init__(self, weights: StackWeights, **kw):
         spec = weights.spec
-        if not spec.blocks:
-            raise ValueError("LatentStackEngine runs stacks described by ModelSpec.blocks")
-        self.f32, self.Wp = weights.f32, up(spec.hidden, 8)
+        if spec.stack != "latent":
+            raise ValueError("LatentStackEngine runs latent-attention stacks described by ModelSpec.blocks")
         self.runs = spec.layer_runs()
         for i, b in enumerate(spec.blocks):
             if b.attn.kv_lora_rank > 1024:
@@ -129,7 +95,6 @@ class LatentStackEngine(MlaEngine):
             if b.moe is not None and (b.moe.n_experts > 512 or b.moe.top_k > 16 or b.moe.n_group > 32):
                 raise ValueError(f"layer {i}: at most 512 experts, 16 per token, 32 groups")
         super().__init__(weights, **kw)
-        self.tap = None             # set to a list to collect the residual rows after every layer run of eager steps
 
     # ------------------------------------------------------------------ cache
     def _alloc_attention_state(self):
@@ -145,21 +110,11 @@ class LatentStackEngine(MlaEngine):
             self.kv_tmaps = host.to(self.device)
         self._pf: dict = {}
 
-    def lane(self, T: int) -> StackLane:
-        cap = next(c for c in LANE_CAPS if T <= c)
-        if cap not in self.lanes:
-            self.lanes[cap] = StackLane(self, cap)
-        return self.lanes[cap]
-
     def set_inputs(self, tokens, positions, *args, **kw):
         n = self.spec.learned_positions
         if n and len(positions) and max(positions) >= n:
             raise ValueError(f"position {max(positions)} is beyond this model's {n} learned positions")
         return super().set_inputs(tokens, positions, *args, **kw)
-
-    def set_input_embeds(self, rows, vals):
-        if vals is not None and len(rows):
-            raise NotImplementedError("image / audio rows are not wired for latent-attention stacks")
 
     def attn_splits_for(self, n_seq: int, max_q_len: int, max_kv: int) -> int:
         if self.f32 or max_q_len > 16:
@@ -173,14 +128,14 @@ class LatentStackEngine(MlaEngine):
         return max(1, min(32, fill))
 
     # ------------------------------------------------------------------ layer program
-    def _emit(self, r: int, L: StackLane):
+    def _emit(self, r: int, L: LatentLane):
         """What the producer of the residual rows in front of layer run `r` leaves for it."""
         if r >= len(self.runs):
             return None
         li, opens = self.runs[r]
         return ops.emit_arg(cat=L.cat) if opens is not None else ops.emit_arg(norm=self.weights.layer(li).norm, xn=L.xn)
 
-    def _forward_single(self, sh: StepShape) -> StackLane:
+    def _forward_single(self, sh: StepShape) -> LatentLane:
         w, T, md = self.weights, sh.T, self.md
         L = self.lane(T)
         self.launches_per_step = 0
@@ -206,10 +161,7 @@ class LatentStackEngine(MlaEngine):
             self.launches_per_step += 3
         return L
 
-    def _splits(self, N, K, T, tn, kind):
-        return 1 if kind == KIND_F32 else super()._splits(N, K, T, tn, kind)
-
-    def _block(self, r: int, li: int, lw: StackLayer, L: StackLane, sh: StepShape):
+    def _block(self, r: int, li: int, lw: StackLayer, L: LatentLane, sh: StepShape):
         """One parallel layer: mixer and experts read the same rows L.xn; the combine adds both to the residual and prepares run r + 1."""
         b, T = self.spec.blocks[li], sh.T
         e = L.experts(b.moe) if b.moe is not None else None
@@ -220,7 +172,7 @@ class LatentStackEngine(MlaEngine):
                           b.moe.top_k if e else 0)
         self.launches_per_step += 1
 
-    def _mixer(self, r: int, a, lw: StackLayer, L: StackLane, sh: StepShape, e: dict | None):
+    def _mixer(self, r: int, a, lw: StackLayer, L: LatentLane, sh: StepShape, e: dict | None):
         T, md, H, rp, st = sh.T, self.md, a.n_heads, up(a.kv_lora_rank, 64), self.status
         b = L.mixer(a, lw.w_in.N)
         self._dense(lw.w_in, L.xn_act, b["proj"], T)
@@ -235,7 +187,7 @@ class LatentStackEngine(MlaEngine):
             self._absorbed(r, a, lw, L, b, gate, sh)
         self._dense(lw.wo, b["o_act"], L.mix, T)
 
-    def _absorbed(self, r: int, a, lw: StackLayer, L: StackLane, b: dict, gate, sh: StepShape):
+    def _absorbed(self, r: int, a, lw: StackLayer, L: LatentLane, b: dict, gate, sh: StepShape):
         T, md, H, rp = sh.T, self.md, a.n_heads, up(a.kv_lora_rank, 64)
         lat = L.latent(H, rp)
         per = dict(tiles=b["tiles"], n_tiles=b["n_tiles"], max_tiles=H * -(-T // L.tn), status=self.status)
@@ -260,7 +212,7 @@ class LatentStackEngine(MlaEngine):
         ops.tc_linear(lw.w_uv, lat["o_act"], b["o"], rows=H * L.cap, token_major=(L.cap, a.v_head_dim), **per)
         self.launches_per_step += 3
 
-    def _experts(self, m, lw: StackLayer, L: StackLane, e: dict, T: int):
+    def _experts(self, m, lw: StackLayer, L: LatentLane, e: dict, T: int):
         E, k = m.n_experts, m.top_k
         sel = (e["logits"], None, e["idx"], e["wts"], T, k, m.scoring, m.normalize, m.route_scale, m.n_group, m.topk_group)
         if T * k <= 1024:
@@ -301,7 +253,7 @@ class LatentStackEngine(MlaEngine):
             self._pf[("kvb", width)] = (cap, kvb)
         return cap, lat, act, kvb
 
-    def _prefill(self, r: int, a, lw: StackLayer, L: StackLane, b: dict, gate, sh: StepShape):
+    def _prefill(self, r: int, a, lw: StackLayer, L: LatentLane, b: dict, gate, sh: StepShape):
         T, md, H, n_seq = sh.T, self.md, a.n_heads, sh.n_seq
         rp, dp, dvp = up(a.kv_lora_rank, 64), up(a.head_dim, 64), up(a.v_head_dim, 64)
         kv, rows = self._ctx_plan(sh)

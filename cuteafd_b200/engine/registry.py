@@ -11,7 +11,7 @@ DTYPES = {"bfloat16": "bf16", "float32": "f32"}
 
 
 def model_spec(model: str, *, layers: int = 0, dtype: str = "bfloat16") -> ModelSpec:
-    """`layers` > 0 keeps that many layers of a named shape; `dtype` "float32" runs everything in fp32 (latent-attention stacks only)."""
+    """`layers` > 0 keeps that many layers of a named shape; `dtype` "float32" runs everything in fp32 (layer stacks only)."""
     if model in NAMED_SPECS:
         spec = spec_by_name(model)
         if layers:
@@ -24,7 +24,7 @@ def model_spec(model: str, *, layers: int = 0, dtype: str = "bfloat16") -> Model
         if dtype not in DTYPES:
             raise ValueError(f"dtype {dtype!r}: one of {sorted(DTYPES)}")
         if not spec.blocks:
-            raise ValueError(f"{spec.name}: only latent-attention stacks run in {dtype}")
+            raise ValueError(f"{spec.name}: only layer stacks run in {dtype}")
         k = DTYPES[dtype]
         spec = spec.replace(quant=dataclasses.replace(spec.quant, dense=k, experts=k, kv=k))
     return spec
@@ -34,6 +34,12 @@ def load_weights(model: str, spec: ModelSpec, device, seed: int = 1):
     """Weights of a snapshot in the forms the kernels consume, or synthetic ones for a named shape."""
     from ..models.weights import DeviceWeights
     snapshot = os.path.isdir(model)
+    if spec.stack == "hybrid":
+        from ..models.hybrid_stack import hybrid_weights_from_masters, hybrid_weights_random
+        if snapshot:
+            from ..loader.stack_checkpoint import read_hybrid_masters
+            return hybrid_weights_from_masters(spec, read_hybrid_masters(model, spec), device)
+        return hybrid_weights_random(spec, device, seed=seed)
     if spec.blocks:
         from ..models.latent_stack import stack_weights_from_masters, stack_weights_random
         if snapshot:
@@ -56,6 +62,9 @@ def load_weights(model: str, spec: ModelSpec, device, seed: int = 1):
 
 
 def engine_class(spec: ModelSpec):
+    if spec.stack == "hybrid":
+        from .hybrid_stack import HybridStackEngine
+        return HybridStackEngine
     if spec.blocks:
         from .latent_stack import LatentStackEngine
         return LatentStackEngine

@@ -72,7 +72,7 @@ def solve(spec: ModelSpec, world: int = 8, gpu_bytes: int = 180 * GIB, reserve_b
         if is_exp:
             p.weights["routed_experts"] = int(routed_share)
         plans.append(p)
-    kv_tok_rank = spec.kv_bytes_per_token() / (dep.tp if spec.attn.kind == "gqa" else 1)    # MLA latent is replicated over TP
+    kv_tok_rank = spec.kv_bytes_per_token() / (dep.tp if spec.attn.kind == "gqa" else 1) or 1.0    # a stack without attention caches nothing; MLA latent is replicated over TP
     tokens_fit = []
     for p in plans:
         free = gpu_bytes - p.weight_bytes - p.workspace - p.reserve
@@ -96,7 +96,7 @@ def solve(spec: ModelSpec, world: int = 8, gpu_bytes: int = 180 * GIB, reserve_b
                 notes.append(f"rank {p.rank} ({p.role}) is short {p.shortfall / GIB:.1f} GiB")
     if spec.blocks and dep.world > 1:
         fits = False
-        notes.append("latent-attention stacks run on one GPU")
+        notes.append("layer stacks run on one GPU")
     if dep.ep and spec.moe.n_experts % dep.ep:
         notes.append(f"{spec.moe.n_experts} experts over {dep.ep} expert ranks: uneven ranges of "
                      f"{spec.moe.n_experts // dep.ep} or {spec.moe.n_experts // dep.ep + 1} experts")
@@ -110,7 +110,7 @@ def solve_stages(spec: ModelSpec, n_stages: int, gpu_bytes: int = 180 * GIB, res
     stage can hold.  (Reference: cuteafd-loader/src/placement/residual.rs: layer ranges per device.)"""
     from ..parallel.pipeline import stage_ranges
     if spec.blocks:
-        raise NotImplementedError("latent-attention stacks are not cut into layer ranges (a looped range would cross the cut)")
+        raise NotImplementedError("layer stacks are not cut into layer ranges (looped ranges and shared keys would cross the cut)")
     a = spec.attn
     ranges = stage_ranges(spec.n_layers, n_stages, max(a.full_every or 1, a.linear_every or 1))
     wb = spec.weight_bytes()

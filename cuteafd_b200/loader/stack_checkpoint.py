@@ -1,7 +1,12 @@
-"""Snapshots of latent-attention layer stacks (the Bedovik design): tensor names <-> the masters `models.latent_stack` packs.
+"""Snapshots of layer stacks: tensor names <-> the masters `models.latent_stack` and `models.hybrid_stack` pack.  Matrices are [out, in].
 
-Layer i's tensors start with `l<i>.`: `norm1` (+ `.b`, `.alpha`), `mix.{q,dkv,dkv.norm,uk,uv,g,o}`, `mlp.router`, `mlp.e<j>.{up,down}`,
-`ls1`, `ls2`; the stack has `embed`, `pos`, `loop.in`, `loop.step`, `final.norm` (+ `.b`, `.alpha`) and `head`.  Matrices are [out, in].
+Latent-attention stacks (the Bedovik design): layer i's tensors start with `l<i>.`: `norm1` (+ `.b`, `.alpha`), `mix.{q,dkv,dkv.norm,uk,uv,g,o}`, `mlp.router`, `mlp.e<j>.{up,down}`,
+`ls1`, `ls2`; the stack has `embed`, `pos`, `loop.in`, `loop.step`, `final.norm` (+ `.b`, `.alpha`) and `head`.
+
+Hybrid recurrent / windowed-attention stacks (the Tudilix design): `l<i>.norm1`, `norm1b` and, with a feed-forward, `norm2`, `norm2b`,
+`mlp.{gate,up,down}` (+ `.b`); attention has `mix.{q,k,v,o}`, `mix.{q,k,v}.conv`, `mix.{q,k}.norm` (no `k` and `v` where the layer uses
+another layer's); the recurrence has `mix.{y,x}` (+ `.b`), `mix.conv` (+ `.b`), `mix.{ra,ri}` (+ `.b`), `mix.lam`, `mix.o`; the stack has
+`embed`, `final.norm` and `head`.
 """
 from __future__ import annotations
 
@@ -13,8 +18,8 @@ from ..config import ModelSpec
 from .safetensors_io import catalog, read_tensor
 
 
-def read_stack_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
-    """Weights of a snapshot in their stored dtype, checked against the shapes the configuration implies."""
+def _reader(snapshot: str | Path):
+    """get(name, *shape): a tensor of the snapshot in its stored dtype, refused when its shape is not the one the configuration implies."""
     cat = catalog(snapshot)
 
     def get(name: str, *shape: int) -> torch.Tensor:
@@ -24,7 +29,12 @@ def read_stack_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
         if t.numel() != torch.Size(shape).numel() or (t.dim() > 1 and tuple(t.shape) != shape):
             raise ValueError(f"tensor {name}: shape {tuple(t.shape)}, the configuration implies {shape}")
         return t.reshape(shape)
+    return get
 
+
+def read_stack_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
+    """Weights of a snapshot in their stored dtype, checked against the shapes the configuration implies."""
+    get = _reader(snapshot)
     W = spec.hidden
 
     def norm(name: str) -> tuple:
@@ -51,3 +61,37 @@ def read_stack_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
         w["loop_in"], w["loop_step"] = get("loop.in", W, 2 * W), get("loop.step", spec.loop.times, W)
     w["layers"] = [layer(i, b) for i, b in enumerate(spec.blocks)]
     return w
+
+
+def read_hybrid_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
+    """Weights of a hybrid stack's snapshot in their stored dtype, checked against the shapes the configuration implies."""
+    get, W = _reader(snapshot), spec.hidden
+
+    def layer(i: int, b) -> dict:
+        p = f"l{i}"
+        lw = {"norm1": get(f"{p}.norm1", W), "norm1b": get(f"{p}.norm1b", W)}
+        if b.rec is not None:
+            n, nb, sq = b.rec.width, b.rec.blocks, b.rec.width // b.rec.blocks
+            for k in ("y", "x"):
+                lw[f"w{k}"], lw[f"{k}_b"] = get(f"{p}.mix.{k}", n, W), get(f"{p}.mix.{k}.b", n)
+            lw["conv"], lw["conv_b"], lw["lam"] = get(f"{p}.mix.conv", n, b.rec.conv_taps), get(f"{p}.mix.conv.b", n), get(f"{p}.mix.lam", n)
+            for k in ("ra", "ri"):
+                lw[k], lw[f"{k}_b"] = get(f"{p}.mix.{k}", nb, sq, sq), get(f"{p}.mix.{k}.b", nb, sq)
+            lw["wo"] = get(f"{p}.mix.o", W, n)
+        else:
+            a = b.attn
+            sizes = {"q": a.n_heads * a.head_dim, "k": a.n_kv_heads * a.head_dim, "v": a.n_kv_heads * a.v_head_dim}
+            for k in ("q", "k", "v") if a.kv_from < 0 else ("q",):
+                lw[f"w{k}"], lw[f"{k}_conv"] = get(f"{p}.mix.{k}", sizes[k], W), get(f"{p}.mix.{k}.conv", sizes[k], a.conv_taps)
+                if k != "v":
+                    lw[f"{k}_norm"] = get(f"{p}.mix.{k}.norm", a.head_dim)
+            lw["wo"] = get(f"{p}.mix.o", W, a.n_heads * a.v_head_dim)
+        if b.ffn is not None:
+            ff = b.ffn.intermediate
+            lw["norm2"], lw["norm2b"] = get(f"{p}.norm2", W), get(f"{p}.norm2b", W)
+            for k, n, d in (("gate", ff, W), ("up", ff, W), ("down", W, ff)):
+                lw[f"w_{k}"], lw[f"{k}_b"] = get(f"{p}.mlp.{k}", n, d), get(f"{p}.mlp.{k}.b", n)
+        return lw
+
+    return {"embed": get("embed", spec.vocab, W), "lm_head": get("head", spec.vocab, W), "final_norm": get("final.norm", W),
+            "layers": [layer(i, b) for i, b in enumerate(spec.blocks)]}

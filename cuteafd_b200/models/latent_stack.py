@@ -83,7 +83,7 @@ def _pad(t: torch.Tensor, *shape: int) -> torch.Tensor:
 
 def stack_kind(spec: ModelSpec) -> str:
     if spec.quant.dense not in ("bf16", "f32") or spec.quant.experts != spec.quant.dense:
-        raise ValueError("latent-attention stacks run with bf16 or fp32 weights (dense and experts alike)")
+        raise ValueError("layer stacks run with bf16 or fp32 weights (dense and experts alike)")
     return spec.quant.dense
 
 

@@ -30,6 +30,7 @@ FUSED_QUANT_KINDS = (KIND_NVFP4, KIND_MXFP4, KIND_FP8B)
 _QKIND = {KIND_NVFP4: 1, KIND_MXFP4: 2, KIND_FP8B: 3}
 EPI_BF16, EPI_BF16_RESIDUAL, EPI_F32 = 0, 1, 3
 SCORING = {"sigmoid": 0, "softmax": 1, "sqrtsoftplus": 2}
+ACTIVATIONS = {None: 0, "relu2": 1, "softcap": 2, "clamped_glu": 3}      # of a product's epilogue
 GROUP_BY_MAX = 16      # added to the scoring code: a group of experts is ranked by its best member (default: the sum of its two best)
 
 
@@ -297,7 +298,7 @@ def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | 
               residual: torch.Tensor | None = None, tiles: torch.Tensor | None = None, n_tiles: torch.Tensor | None = None,
               max_tiles: int = 0, splits: int = 1, status: torch.Tensor | None = None, max_ctas: int = 0,
               quant_out: ActBuffer | None = None, inv_gs_out: torch.Tensor | None = None, peer: dict | None = None, act: str | None = None,
-              token_major: tuple | None = None) -> torch.Tensor | None:
+              token_major: tuple | None = None, bound: float = 0.0, biases: tuple | None = None) -> torch.Tensor | None:
     """y[rows, N] = x[rows, K] @ w[g]^T (per tile's expert g when `tiles` is given).  `w_up` switches on the fused
     SwiGLU epilogue (y = silu(x w^T) * (x w_up^T)).  y is bf16 (optionally + residual) or fp32.  `quant_out` (an FP4
     activation buffer of the operands' kind, K = N) also receives the output quantised for the GEMM that follows
@@ -306,7 +307,9 @@ def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | 
     pitch in elements, "row_map": int32 tensor or None (row r lands in row_map[r]), "flags": [peer flag addresses],
     "ctl": control block tensor, "done": zeroed uint32 counter tensor}; the flags are released with the step number
     once the whole output has been stored (y may be None when only the peers need the result).
-    `act="relu2"`: squared ReLU on the output (an expert without a gate projection).  `token_major=(rows per group, columns per group)`:
+    `act="relu2"`: squared ReLU on the output (an expert without a gate projection); `act="softcap"`: bound * tanh(y / bound);
+    `act="clamped_glu"` (with `w_up`): gate and linear half with `biases` (fp32 [N] each), bounded by `bound`, g sigmoid(1.702 g) (u + 1)
+    instead of SwiGLU.  `token_major=(rows per group, columns per group)`:
     a GEMM grouped over the heads of head-major operands (operand row = head * rows per group + token) writes head g's N columns of
     output row `token` at column g * columns per group."""
     rows = x.rows if rows is None else rows
@@ -329,7 +332,7 @@ def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | 
             raise ValueError("tc_linear: the fp32 kernel has a plain fp32 output only")
         gr, gc = token_major or (0, 0)
         call("cuteafd_f32_linear", ptr(x.data), x.data.stride(0), ptr(w.data), ptr(y), y.stride(0), ptr(tiles), ptr(n_tiles), max_tiles, rows, w.N, w.K,
-             1 if act == "relu2" else 0, gr, gc, stream())
+             ACTIVATIONS[act], float(bound), gr, gc, stream())
         return y
     ws = cnt = None
     if splits > 1:
@@ -342,10 +345,11 @@ def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | 
         extra = native.TcExtra()
         extra.q_out, extra.sf_out, extra.ldsf_out, extra.inv_gs_out = ptr(quant_out.data), ptr(quant_out.sf), quant_out.sf.shape[1], ptr(inv_gs_out)
     if act is not None or token_major is not None:
-        if act not in (None, "relu2"):
-            raise ValueError(f"tc_linear: unknown activation {act!r}")
         extra = extra or native.TcExtra()
-        extra.act = 1 if act == "relu2" else 0
+        extra.act, extra.act_p = ACTIVATIONS[act], float(bound)
+        if biases is not None:
+            _chk(biases[0], torch.float32, "biases"); _chk(biases[1], torch.float32, "biases")
+            extra.bias, extra.bias2 = ptr(biases[0]), ptr(biases[1])
         extra.grp_rows, extra.grp_cols = token_major or (0, 0)
     if peer is not None:
         ys, fl = list(peer["y"]), list(peer["flags"])
@@ -758,3 +762,107 @@ def latent_attention_simt(q_lat, cache, page_table, kv_len, q_start, q_len, gate
     """The same on the ordinary cores: fp32 operands, latents wider than 512, more than 128 heads."""
     call("cuteafd_latent_attention_simt", ptr(q_lat), ptr(cache), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(gate), ptr(out), T, ldt,
          n_seq, H, rank_pad, cache.stride(0), page_table.shape[1], cache.shape[0], float(scale), _f32(q_lat), ptr(status), stream())
+
+
+# ------------------------------------------------------------------ hybrid stacks: norms around sub-layers, short convolutions, recurrence, windows
+ROWS_EMBED, ROWS_ADD, ROWS_GATHER = 0, 1, 2
+
+
+def norm_rows(x, W: int, rows: int, *, f32: bool, eps: float, gain=None, xn=None, tokens=None, table=None, add=None, bias=None, post=None, mult: float = 1.0,
+              src_rows=None, status=None):
+    """Residual rows (fp32 [., Wp], norms average over W): x = table[token] with `tokens`; x += mult * norm(add + bias) with `add` (`post`: gain of
+    that norm, None = no norm); the rows listed in `src_rows` otherwise.  `xn` receives the rows RMS-normed with `gain`."""
+    _chk(x, torch.float32, "x")
+    a = native.NormRows()
+    a.x, a.W, a.Wp, a.eps, a.mult, a.status = ptr(x), W, x.shape[1], eps, mult, ptr(status)
+    a.gain, a.xn, a.ldn = ptr(gain), ptr(xn), xn.stride(0) if xn is not None else 0
+    mode = ROWS_GATHER
+    if tokens is not None:
+        _chk(tokens, torch.int32, "tokens"); _chk(table, torch.bfloat16, "table")
+        if table.shape[1] != x.shape[1]:
+            raise ValueError("norm_rows: table and residual rows differ in width")
+        mode, a.tokens, a.table, a.vocab = ROWS_EMBED, ptr(tokens), ptr(table), table.shape[0]
+    elif add is not None:
+        if add.shape[1] != x.shape[1]:
+            raise ValueError("norm_rows: added rows and residual rows differ in width")
+        mode, a.add, a.bias, a.post = ROWS_ADD, ptr(add), ptr(bias), ptr(post)
+    else:
+        a.src_rows = ptr(src_rows)
+    call("cuteafd_norm_rows", ctypes.addressof(a), mode, rows, 1 if f32 else 0, stream())
+
+
+def rope_table(positions, freq, amp: float, out, T: int):
+    """Cosine / sine rows [T, pairs] of the step's positions; `freq` fp32 [2, pairs] (value, rounding error)."""
+    _chk(positions, torch.int32, "positions"); _chk(freq, torch.float32, "freq")
+    call("cuteafd_rope_table", ptr(positions), ptr(freq), float(amp), freq.shape[1], ptr(out), T, stream())
+
+
+def conv_qkv(proj, w, q_norm, k_norm, rope, ring, q, cache, meta: dict, *, H, G, dim, dp, vdim, dvp, pairs, eps, n_seq, max_q_len, status=None):
+    """Short causal convolution over projected query / key / value rows, head norms, rotation; queries to `q` [., H * dp], keys and values to the
+    paged `cache` rows.  `ring` [slots, depth + taps - 1, channels]: inputs by position.  `meta`: the step's device inputs.  G = 0: queries only."""
+    _chk(w, torch.float32, "w")
+    a = native.ConvQkv()
+    a.proj, a.w, a.q_norm, a.k_norm, a.rope, a.ring, a.q, a.cache, a.status = (ptr(t) for t in (proj, w, q_norm, k_norm, rope, ring, q, cache, status))
+    for n in ("state_slot", "q_start", "q_len", "kv_len", "slot_map"):
+        setattr(a, n, ptr(meta[n]))
+    a.ldp, a.q_stride, a.H, a.G, a.dim, a.dp, a.vdim, a.dvp, a.pairs, a.eps = proj.stride(0), q.stride(0), H, G, dim, dp, vdim, dvp, pairs, eps
+    a.row_stride, a.n_slots = (cache.stride(0), cache.shape[0]) if cache is not None else (8, 0)
+    a.taps, (a.n_state, a.R, a.C), a.n_seq, a.max_q_len = w.shape[0], ring.shape, n_seq, max_q_len
+    if w.shape[1] != ring.shape[2] or not ring.is_contiguous():
+        raise ValueError("conv_qkv: convolution weights and ring differ in channels")
+    call("cuteafd_conv_qkv", ctypes.addressof(a), _f32(proj), stream())
+
+
+def recurrence_arg(x, y, x_b, y_b, conv, conv_b, ring, state, u, gates, gates_b, decay, agg, out, meta: dict, *, blocks, T, ldt, tiles, n_tiles, tn, n_seq, max_q_len,
+                   status=None):
+    """Arguments of one recurrent layer's step (`rglru_conv`, the gate product, `lru_scan`): x, y column views of one projection buffer; u block-major
+    [blocks * ldt, n_pad]; `ring` [slots, depth + taps - 1, width], `state` [slots, depth + 1, width] by position."""
+    a = native.Recurrence()
+    for n, t in dict(x=x, y=y, x_b=x_b, y_b=y_b, conv=conv, conv_b=conv_b, ring=ring, state=state, u=u, gates=gates, gates_b=gates_b, decay=decay, agg=agg, out=out,
+                     tiles=tiles, n_tiles=n_tiles, status=status, **{k: meta[k] for k in ("state_slot", "q_start", "q_len", "kv_len")}).items():
+        setattr(a, n, ptr(t))
+    a.n_state, a.depth, a.C = state.shape[0], state.shape[1] - 1, state.shape[2]
+    a.taps, a.sq, a.sqp = conv.shape[0], a.C // blocks, u.shape[-1]
+    if ring.shape != (a.n_state, a.taps - 1 + a.depth, a.C) or x.stride(0) != y.stride(0):
+        raise ValueError("recurrence: ring, state and projection do not belong together")
+    a.ldp, a.ldt, a.ldg, a.ldo, a.tn, a.T, a.n_seq, a.max_q_len = x.stride(0), ldt, gates.stride(0), out.stride(0), tn, T, n_seq, max_q_len
+    a.agg_rows = agg.shape[0] if agg is not None else 0
+    return a
+
+
+def rglru_conv(a, *, f32: bool):
+    call("cuteafd_rglru_conv", ctypes.addressof(a), 1 if f32 else 0, stream())
+
+
+def lru_scan(a, *, f32: bool):
+    call("cuteafd_lru_scan", ctypes.addressof(a), 1 if f32 else 0, stream())
+
+
+def glu_rows(g, u, gate_b, up_b, out, rows: int, limit: float):
+    """out = clamped GLU of two projected rows with biases (`tc_linear`'s clamped_glu epilogue as a pass of its own)."""
+    call("cuteafd_glu_rows", ptr(g), ptr(u), ptr(gate_b), ptr(up_b), ptr(out), rows, g.stride(0), out.stride(0), g.shape[1], float(limit), _f32(g), stream())
+
+
+def encode_window_maps(rows: torch.Tensor, Hkv: int, dp: int, dvp: int) -> torch.Tensor:
+    """TMA descriptors (uint8 [2, 128]: keys, values) of one layer's store [slots, row]: Hkv key heads of dp elements, then Hkv value heads of dvp."""
+    host = torch.zeros(2, 128, dtype=torch.uint8)
+    call("cuteafd_tmap_encode_heads", host[0].data_ptr(), rows.data_ptr(), dp, Hkv, rows.stride(0), rows.shape[0])
+    call("cuteafd_tmap_encode_heads", host[1].data_ptr(), rows.data_ptr() + Hkv * dp * rows.element_size(), dvp, Hkv, rows.stride(0), rows.shape[0])
+    return host.to(rows.device)
+
+
+def window_attention(q, maps, page_table, kv_len, q_start, q_len, out, *, T, n_seq, max_q_len, Hq, Hkv, dp, dvp, dv, n_splits=1, part_o=None, part_ml=None, window=0, scale,
+                     prefill=False, status=None):
+    """Windowed paged GQA on the tensor cores (key / value heads of their own, padded widths); `prefill`: the 128-key kernel (dp + 2 dvp <= 512)."""
+    head = (ptr(q), ptr(maps), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(out))
+    shape = (T, n_seq, max_q_len, q.stride(0), Hq, Hkv, dp, dvp, dv, out.stride(0), page_table.shape[1])
+    if prefill:
+        call("cuteafd_window_prefill_attention", *head, *shape, window, float(scale), ptr(status), stream())
+    else:
+        call("cuteafd_window_attention", *head, ptr(part_o), ptr(part_ml), *shape, n_splits, window, float(scale), ptr(status), stream())
+
+
+def window_attention_simt(q, cache, page_table, kv_len, q_start, q_len, out, *, T, n_seq, Hq, Hkv, dp, dvp, dv, window=0, scale, status=None):
+    """The same on the ordinary cores: fp32, heads wider than 256, groups of more than 128."""
+    call("cuteafd_window_attention_simt", ptr(q), q.stride(0), ptr(cache), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(out), out.stride(0), T, n_seq, Hq,
+         Hkv, dp, dvp, dv, cache.stride(0), page_table.shape[1], cache.shape[0], window, float(scale), _f32(q), ptr(status), stream())

@@ -109,7 +109,17 @@ _PROTOS = {
     "cuteafd_stack_embed": [P, P, P, P, P, P, I, I, I, I, I, I, P, P, P],
     "cuteafd_stack_stream": [P, P, P, I, I, I, P, P],
     "cuteafd_stack_combine": [P, P, P, P, P, P, P, I, I, I, I, P, P],
-    "cuteafd_f32_linear": [P, I, P, P, I, P, P, I, I, I, I, I, I, I, P],
+    "cuteafd_f32_linear": [P, I, P, P, I, P, P, I, I, I, I, I, F, I, I, P],
+    "cuteafd_norm_rows": [P, I, I, I, P],
+    "cuteafd_rope_table": [P, P, F, I, P, I, P],
+    "cuteafd_conv_qkv": [P, I, P],
+    "cuteafd_rglru_conv": [P, I, P],
+    "cuteafd_lru_scan": [P, I, P],
+    "cuteafd_glu_rows": [P, P, P, P, P, I, I, I, I, F, I, P],
+    "cuteafd_window_attention_simt": [P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P],
+    "cuteafd_window_attention": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P],
+    "cuteafd_window_prefill_attention": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P],
+    "cuteafd_tmap_encode_heads": [P, P, I, I, U64, U64],
     "cuteafd_tc_linear": [I, I, I, P, P, P, P, P, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, P, P, P, I, P, P],
 }
 
@@ -127,13 +137,35 @@ class FlagWaitArg(C.Structure):
 class TcExtra(C.Structure):
     """Optional outputs of `cuteafd_tc_linear` (`CaTcExtra` of the C ABI)."""
     _fields_ = [("q_out", P), ("sf_out", P), ("inv_gs_out", P), ("ldsf_out", I), ("n_peer", I), ("peer_y", P * 2), ("peer_flag", P * 2),
-                ("peer_row_map", P), ("peer_ctl", P), ("peer_done", P), ("peer_ld", I), ("act", I), ("grp_rows", I), ("grp_cols", I)]
+                ("peer_row_map", P), ("peer_ctl", P), ("peer_done", P), ("peer_ld", I), ("act", I), ("grp_rows", I), ("grp_cols", I),
+                ("act_p", F), ("bias", P), ("bias2", P)]
 
 
 class EmitArg(C.Structure):
     """What a row-producing kernel of a layer stack writes for the next matrix product (`CaEmit` of the C ABI): tanh(alpha x) w + b
     into `xn`, and / or the plain row into `cat`."""
     _fields_ = [("w", P), ("b", P), ("xn", P), ("cat", P), ("alpha", F), ("ldn", I), ("ldc", I), ("reserved", I)]
+
+
+def _fields(pointers: str, ints: str, floats: str = "") -> list:
+    return [(n, P) for n in pointers.split()] + [(n, I) for n in ints.split()] + [(n, F) for n in floats.split()]
+
+
+class NormRows(C.Structure):
+    """`cuteafd_norm_rows` (`CaNormRows` of the C ABI)."""
+    _fields_ = _fields("x tokens table add bias post src_rows gain xn status", "W Wp vocab ldn", "mult eps")
+
+
+class ConvQkv(C.Structure):
+    """`cuteafd_conv_qkv` (`CaConvQkv` of the C ABI)."""
+    _fields_ = _fields("proj w q_norm k_norm rope ring state_slot q_start q_len kv_len slot_map q cache status",
+                       "ldp q_stride row_stride n_slots H G dim dp vdim dvp pairs taps R C n_state n_seq max_q_len", "eps")
+
+
+class Recurrence(C.Structure):
+    """One recurrent layer's step: `cuteafd_rglru_conv`, then `cuteafd_lru_scan` (`CaRecurrence` of the C ABI)."""
+    _fields_ = _fields("x y x_b y_b conv conv_b ring state u gates gates_b decay agg out tiles n_tiles state_slot q_start q_len kv_len status",
+                       "ldp ldt sq sqp ldg ldo tn T C taps depth n_state n_seq max_q_len agg_rows")
 
 
 def flag_wait(flags_ptr: int, n: int, stride: int, ctl: torch.Tensor, status: torch.Tensor | None, timeout_ns: int = 2_000_000_000) -> FlagWaitArg:

@@ -64,10 +64,14 @@ class EngineRunner:
         # MTP drafter pairs with the next tokens (serving.mtp_drafter)
         self.keep_hidden = False
         self.records: dict = {}
-        # hybrid stacks (linear-attention layers): every live sequence owns one recurrent-state slot of the engine
-        self._recurrent = bool(getattr(engine, "lin_layers", None))
+        # hybrid stacks: every live sequence owns one recurrent-state slot of the engine.  Linear-attention layers keep one state, so drafted
+        # steps are deferred and replayed; engines with a `state_depth` keep the states of the last positions and simply go on from an
+        # earlier one
+        self._depth = getattr(engine, "state_depth", 0)
+        self._recurrent = bool(getattr(engine, "lin_layers", None)) or self._depth > 0
         self._state_slot: dict = {}
         self._state_pos: dict = {}
+        self._state_back: dict = {}       # rows of the sequence's last step that can be taken back
         self.last_lane = None             # the lane of the last step: `.logits` holds its rows that needed logits, in order
         self._deferred = None             # (step shape, [(state id, start position, rows)]) of a speculative step awaiting `commit`
         self._free_slots = list(range(getattr(engine, "max_seqs", 0)))[::-1] if self._recurrent else []
@@ -83,6 +87,7 @@ class EngineRunner:
         """The scheduler finished this sequence: its recurrent-state slot and hidden records are free again."""
         slot = self._state_slot.pop(id(state), None)
         self._state_pos.pop(id(state), None)
+        self._state_back.pop(id(state), None)
         if slot is not None:
             self._free_slots.append(slot)
         self.records.pop(id(state), None)
@@ -94,14 +99,15 @@ class EngineRunner:
             if slot is None or r.start_pos == 0:
                 if slot is None:
                     if r.start_pos != 0:
-                        raise RuntimeError("a linear-attention stack cannot resume a sequence from cached pages: run it without the prefix cache")
+                        raise RuntimeError("a recurrent stack cannot resume a sequence from cached pages: run it without the prefix cache")
                     if not self._free_slots:
                         raise RuntimeError("more live sequences than recurrent-state slots (engine max_seqs)")
                     slot = self._state_slot[id(r.state)] = self._free_slots.pop()
                 fresh.append(slot)
-            elif r.start_pos != self._state_pos.get(id(r.state)):      # the recurrent state sits at another position
-                raise RuntimeError("a linear-attention stack cannot step back (was a speculative step left uncommitted?)")
+            elif not 0 <= self._state_pos.get(id(r.state)) - r.start_pos <= self._state_back.get(id(r.state), 0):      # the recurrent state sits at another position
+                raise RuntimeError("a recurrent stack cannot step back this far (was a speculative step left uncommitted?)")
             self._state_pos[id(r.state)] = r.start_pos + len(r.tokens)
+            self._state_back[id(r.state)] = len(r.tokens) if len(r.tokens) <= self._depth else 0
             out.append(slot)
         self.eng.reset_state_slots(fresh)
         return out
@@ -160,7 +166,7 @@ class EngineRunner:
         # micro-batches by a multi-GPU engine
         uniform = decode_like and all(q == max_q for q in q_len) and (not logit_rows or logit_rows == list(range(len(tokens))))
         # drafted rows over recurrent layers: the step leaves their state alone, `commit` absorbs what the scheduler accepts
-        defer = self._recurrent and decode_like and any(len(r.tokens) > 1 and len(r.want_logits) == len(r.tokens) for r in rows)
+        defer = self._recurrent and not self._depth and decode_like and any(len(r.tokens) > 1 and len(r.want_logits) == len(r.tokens) for r in rows)
         sh = StepShape(T=len(tokens), n_seq=len(rows), max_q_len=max_q, n_logits=len(logit_rows),
                        attn_splits=eng.attn_splits_for(len(rows), max_q, max(kv_len)) if decode_like else 1, uniform=uniform, defer_state=defer)
         if over_rows:

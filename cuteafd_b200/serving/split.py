@@ -38,7 +38,7 @@ def build_split_serving(a, world: int):
         dist.init_process_group("nccl", device_id=torch.device("cuda", local))
     spec = spec_by_name(a.model) if a.model in NAMED_SPECS else spec_from_snapshot(a.model)
     if spec.blocks:
-        raise NotImplementedError(f"{spec.name}: latent-attention stacks are served on one GPU")
+        raise NotImplementedError(f"{spec.name}: layer stacks are served on one GPU")
     if getattr(a, "layers", 0):
         spec = spec.replace(n_layers=a.layers)
     masters = None

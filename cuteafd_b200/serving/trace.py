@@ -50,6 +50,9 @@ class TraceReplay:
         out = None
         if rows:
             self.runner.run(rows)
+            commit = getattr(self.runner, "commit", None)
+            if commit is not None:
+                commit([(r.state, len(r.tokens)) for r in rows])        # every token given is kept
             for r in rows:
                 r.state.req.prompt += r.tokens
                 r.state.seq.length += len(r.tokens)
@@ -70,7 +73,8 @@ def ensure_kernels(model: str):
         return
     from .. import build
     from ..config import spec_from_snapshot
-    os.environ["CUTEAFD_LIB"] = str(build.ensure("latent_stack" if spec_from_snapshot(model).blocks else None))
+    stack = spec_from_snapshot(model).stack
+    os.environ["CUTEAFD_LIB"] = str(build.ensure(f"{stack}_stack" if stack else None))
 
 
 def add_arguments(ap):

@@ -114,7 +114,8 @@ __global__ void rope_table_kernel(const int* __restrict__ positions, const float
     const float f = freq[i], a = p * f, lo = fmaf(p, f, -a) + p * freq[pairs + i];
     float s, c;
     sincosf(a, &s, &c);
-    out[(size_t)t * pairs + i] = make_float2(amp * fmaf(-s, lo, c), amp * fmaf(c, lo, s));
+    const float cl = fmaf(-0.5f * lo, lo, 1.f), sl = lo * fmaf(lo * lo, -1.f / 6.f, 1.f);      // lo is at most half an ulp of a
+    out[(size_t)t * pairs + i] = make_float2(amp * (c * cl - s * sl), amp * (s * cl + c * sl));
   }
 }
 

@@ -135,11 +135,13 @@ class HybridStackEngine(StackBase, Engine):
         return best
 
     def _scratch(self, n_o: int, n_ml: int):
-        if getattr(self, "part_o", None) is None or self.part_o.numel() < n_o or self.part_ml.numel() < n_ml:
-            if getattr(self, "part_o", None) is not None:
+        """Partial outputs and (max, sum) pairs of split attention: grows to the largest need of any layer, in the eager run of a new shape."""
+        o, ml = (t.numel() if t is not None else 0 for t in (getattr(self, "part_o", None), getattr(self, "part_ml", None)))
+        if o < n_o or ml < n_ml:
+            if o:
                 self.drop_graphs()                         # captured steps hold the old scratch
-            self.part_o = torch.empty(n_o, dtype=torch.float32, device=self.device)
-            self.part_ml = torch.empty(n_ml, dtype=torch.float32, device=self.device)
+            self.part_o = torch.empty(max(o, n_o), dtype=torch.float32, device=self.device)
+            self.part_ml = torch.empty(max(ml, n_ml), dtype=torch.float32, device=self.device)
 
     # ------------------------------------------------------------------ layer program
     def _forward_single(self, sh: StepShape) -> HybridLane:

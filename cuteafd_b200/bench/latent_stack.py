@@ -26,8 +26,7 @@ from ..config import AttentionSpec, ModelSpec, QuantSpec, bedovik_spec
 from ..engine.engine import PAGE, StepShape
 from ..engine.generate import BatchGenerator
 from ..engine.kv import PagePool, SeqKV
-from ..engine.registry import build_engine
-from ..models.latent_stack import stack_weights_random
+from ..engine.registry import build_engine, load_weights
 from ..ops import native
 
 # hidden, heads, latent rank, experts, squared-ReLU width, layers (the middle half of them twice)
@@ -47,11 +46,11 @@ def specs(size: str) -> tuple[ModelSpec, ModelSpec]:
 
 def make_engine(spec: ModelSpec, pages: int, seqs: int, per_seq: int):
     dev = torch.device("cuda", 0)
-    if spec.blocks:
-        w = stack_weights_random(spec, dev)
-    else:
+    if spec.attn.kind == "mla":
         from ..engine.mla import mla_weights_random
         w = mla_weights_random(spec, dev, distinct_moe_layers=4, seed=1)
+    else:
+        w = load_weights(spec.name, spec, dev)
     eng = build_engine(spec, w, n_pages=pages, max_seqs=seqs, max_pages_per_seq=per_seq)
     eng.kv.normal_(0, 1)
     return eng
@@ -185,7 +184,7 @@ def roofline(spec: ModelSpec, T: int, pairs: int, kv_rows: int, site: tuple, pre
     return None
 
 
-def kernel_table(eng, sh, pairs: int, kv_rows: int, prefill: bool, peaks: dict) -> dict:
+def kernel_table(eng, sh, pairs: int, kv_rows: int, prefill: bool, peaks: dict, roofline=roofline) -> dict:
     out: dict = {}
     for s, (count, ms) in launch_times(eng, sh).items():
         r = roofline(eng.spec, sh.T, pairs, kv_rows, s, prefill, peaks)
@@ -199,7 +198,10 @@ def kernel_table(eng, sh, pairs: int, kv_rows: int, prefill: bool, peaks: dict) 
 
 
 # ------------------------------------------------------------------ workloads
-def measure(spec: ModelSpec, *, batches, context: int, chunks, steps: int, warmup: int, kernels: bool, peaks: dict) -> dict:
+def measure(spec: ModelSpec, *, batches, context: int, chunks, steps: int, warmup: int, kernels: bool, peaks: dict, roofline=roofline) -> dict:
+    """`roofline`: what a launch has to compute and move, for the per-launch table (windowed layers see the last `attn.window` keys only)."""
+    win = spec.attn.window or 1 << 40
+    seen = lambda lo, hi: sum(min(p + 1, win) for p in range(lo, hi))            # (query, key) pairs of positions [lo, hi)
     longest = max([context] + [c for _, c in chunks])
     per = longest // PAGE + 3
     pages = max(max(batches) * (context // PAGE + 2), per) + 2
@@ -214,7 +216,7 @@ def measure(spec: ModelSpec, *, batches, context: int, chunks, steps: int, warmu
         row = {"batch": b, "context": context, "ms_per_step": round(ms, 4), "tokens_per_s": round(b / ms * 1e3, 1), "us_per_layer_run": round(1e3 * ms / res["layer_runs"], 1),
                "launches_per_step": eng.launches_per_step}
         if kernels:
-            row["kernels"] = kernel_table(eng, sh, b * (context + 1), b * (context + 1), False, peaks)
+            row["kernels"] = kernel_table(eng, sh, b * seen(context, context + 1), b * min(context + 1, win), False, peaks, roofline)
         res["decode"].append(row)
         eng.check_status()
     for chunk, ctx in chunks:
@@ -224,7 +226,7 @@ def measure(spec: ModelSpec, *, batches, context: int, chunks, steps: int, warmu
         row = {"chunk": chunk, "context": ctx, "ms_per_chunk": round(ms, 3), "tokens_per_s": round(chunk / ms * 1e3, 1), "us_per_layer_run": round(1e3 * ms / res["layer_runs"], 1)}
         if kernels:
             off = ctx - chunk
-            row["kernels"] = kernel_table(eng, sh, chunk * off + chunk * (chunk + 1) // 2, ctx, True, peaks)
+            row["kernels"] = kernel_table(eng, sh, seen(off, ctx), min(ctx, chunk + win), True, peaks, roofline)
         res["prefill"].append(row)
         eng.check_status()
     res["gpu_launches"] = launches

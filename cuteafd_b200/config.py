@@ -417,10 +417,11 @@ def bedovik_spec(n_layers: int = 8, heads: int = 32, hidden: int = 4096, rank: i
                      loop=LoopSpec(lo, hi, loop_times) if loop_times > 1 and hi > lo else None, learned_positions=65536, max_context=65536)
 
 
-def tudilix_spec(n_layers: int = 12, hidden: int = 4096, heads: int = 32, kv_heads: int = 4, ff: int = 12288, window: int = 2048, blocks: int = 16) -> ModelSpec:
-    """Tudilix at the size of a real model's layers (synthetic weights): two recurrent layers, then one windowed-attention layer with a dense
-    feed-forward, every second attention layer on the keys and values of the one before it."""
-    rec = BlockSpec(None, rec=RecurrentSpec(width=hidden, blocks=blocks, conv_taps=4))
+def tudilix_spec(n_layers: int = 12, hidden: int = 4096, heads: int = 32, kv_heads: int = 4, ff: int = 12288, window: int = 2048, blocks: int = 16,
+                 ffn_everywhere: bool = False) -> ModelSpec:
+    """Tudilix at the size of a real model's layers (synthetic weights): two recurrent layers, then one windowed-attention layer, every second
+    attention layer on the keys and values of the one before it; dense feed-forwards behind the attention layers, or behind every layer."""
+    rec = BlockSpec(None, rec=RecurrentSpec(width=hidden, blocks=blocks, conv_taps=4), ffn=DenseFfnSpec(ff, 7.0) if ffn_everywhere else None)
     attn = AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, window=window, qk_norm=True, conv_taps=4,
                          rope_dims=64, rope_scaling=RopeScaling(8.0, 8192, 32.0, 1.0))
     layers, last = [], -1

@@ -134,148 +134,10 @@ struct ConvQkv {
   float eps; int* status;
 };
 
-template <typename T> __device__ __forceinline__ float2 load_pair(const T* p, bool two, bool vec);
-template <> __device__ __forceinline__ float2 load_pair<bf16>(const bf16* p, bool two, bool vec) {
-  if (vec) return __bfloat1622float2(*(const bf162*)p);
-  return make_float2(to_f(p[0]), two ? to_f(p[1]) : 0.f);
-}
-template <> __device__ __forceinline__ float2 load_pair<float>(const float* p, bool two, bool vec) {
-  if (vec) return *(const float2*)p;
-  return make_float2(p[0], two ? p[1] : 0.f);
-}
-template <typename T> __device__ __forceinline__ void store_pair(T* p, float2 v, bool two, bool vec);
-template <> __device__ __forceinline__ void store_pair<bf16>(bf16* p, float2 v, bool two, bool vec) {
-  if (vec) { *(bf162*)p = __floats2bfloat162_rn(v.x, v.y); return; }
-  p[0] = __float2bfloat16(v.x);
-  if (two) p[1] = __float2bfloat16(v.y);
-}
-template <> __device__ __forceinline__ void store_pair<float>(float* p, float2 v, bool two, bool vec) {
-  if (vec) { *(float2*)p = v; return; }
-  p[0] = v.x;
-  if (two) p[1] = v.y;
-}
-
-// One warp per (head, tile of HS_TILE tokens); a lane owns the dimension pairs lane, lane + 32, ... of the head (NC of them).  TAPS > 0: the
-// last inputs and the weights stay in registers; 0: any number of taps, inputs re-read.
-template <typename T, int NC, int TAPS>
-__global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvQkv<T> a) {
-  pdl_launch(); pdl_wait();
-  const int lane = threadIdx.x & 31, unit = blockIdx.x * 4 + (threadIdx.x >> 5), seq = blockIdx.z;
-  const int n = a.q_len[seq], i0 = blockIdx.y * HS_TILE;
-  if (unit >= a.H + 2 * a.G || i0 >= n) return;
-  const int row0 = a.q_start[seq], p0 = a.kv_len[seq] - n, slot = a.state_slot[seq], i1 = min(n, i0 + HS_TILE);
-  if (slot < 0 || slot >= a.n_state) { if (lane == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6E1); return; }
-  const bool is_q = unit < a.H, is_v = unit >= a.H + a.G;
-  const int d = is_v ? a.vdim : a.dim, head = is_q ? unit : (is_v ? unit - a.H - a.G : unit - a.H);
-  const int ch = is_v ? (a.H + a.G) * a.dim + head * a.vdim : unit * a.dim;
-  const int taps = TAPS ? TAPS : a.taps;
-  T* ring = a.ring + (size_t)slot * a.R * a.C + ch;
-  bool has[NC], two[NC], vec[NC], rvec[NC];
-#pragma unroll
-  for (int c = 0; c < NC; ++c) {
-    const int e = 2 * (lane + 32 * c);
-    has[c] = e < d; two[c] = e + 1 < d;
-    vec[c] = two[c] && ((ch | a.ldp) & 1) == 0;
-    rvec[c] = vec[c] && (a.C & 1) == 0;
-  }
-  // input row i of this run (i < 0: what the sequence fed before, nothing in front of its start)
-  auto input = [&](int i, int c) -> float2 {
-    const int e = 2 * (lane + 32 * c);
-    if (!has[c]) return make_float2(0.f, 0.f);
-    if (i >= 0) return load_pair<T>(a.proj + (size_t)(row0 + i) * a.ldp + ch + e, two[c], vec[c]);
-    const int pos = p0 + i;
-    if (pos < 0) return make_float2(0.f, 0.f);
-    return load_pair<T>(ring + (size_t)(pos % a.R) * a.C + e, two[c], rvec[c]);
-  };
-  auto weight = [&](int j, int c) -> float2 {
-    const float* w = a.w + (size_t)j * a.C + ch + 2 * (lane + 32 * c);
-    return make_float2(has[c] ? w[0] : 0.f, two[c] ? w[1] : 0.f);
-  };
-  constexpr int NH = TAPS > 1 ? TAPS - 1 : 1, NW = TAPS ? TAPS : 1;
-  float2 hist[NH][NC], wr[NW][NC], gain[NC];
-  const float* norm = is_q ? a.q_norm : a.k_norm;
-#pragma unroll
-  for (int c = 0; c < NC; ++c) {
-    const int e = 2 * (lane + 32 * c);
-    gain[c] = is_v ? make_float2(1.f, 1.f) : make_float2(has[c] ? norm[e] : 0.f, two[c] ? norm[e + 1] : 0.f);
-    if (TAPS) {
-#pragma unroll
-      for (int j = 0; j < NW; ++j) wr[j][c] = weight(j, c);
-#pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) hist[j][c] = input(i0 - (TAPS - 1) + j, c);
-    }
-  }
-  const bool keep = n <= a.R - (taps - 1);              // short runs leave every input (a single tile), long ones the last taps - 1
-  for (int i = i0; i < i1; ++i) {
-    const int row = row0 + i;
-    float2 y[NC];
-    float ss = 0.f;
-#pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const float2 cur = input(i, c);
-      float2 s = make_float2(0.f, 0.f);
-      if (TAPS) {
-#pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) { s.x = fmaf(wr[j][c].x, hist[j][c].x, s.x); s.y = fmaf(wr[j][c].y, hist[j][c].y, s.y); }
-        s.x = fmaf(wr[NW - 1][c].x, cur.x, s.x); s.y = fmaf(wr[NW - 1][c].y, cur.y, s.y);
-#pragma unroll
-        for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][c] = hist[j + 1][c];
-        if (TAPS > 1) hist[NH - 1][c] = cur;
-      } else {
-        for (int j = 0; j < taps; ++j) {
-          const float2 u = j == taps - 1 ? cur : input(i - (taps - 1) + j, c), w = weight(j, c);
-          s.x = fmaf(w.x, u.x, s.x); s.y = fmaf(w.y, u.y, s.y);
-        }
-      }
-      if (keep && has[c]) store_pair<T>(ring + (size_t)((p0 + i) % a.R) * a.C + 2 * (lane + 32 * c), cur, two[c], rvec[c]);
-      y[c] = s;
-      ss = fmaf(s.x, s.x, fmaf(s.y, s.y, ss));
-    }
-    T* dst;
-    if (is_q) dst = a.q + (size_t)row * a.q_stride + (size_t)head * a.dp;
-    else {
-      const int cs = a.slot_map[row];
-      if (cs < 0 || cs >= a.n_slots) { if (lane == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, row); continue; }     // warp-uniform
-      dst = a.cache + (size_t)cs * a.row_stride + (is_v ? (size_t)a.G * a.dp + (size_t)head * a.dvp : (size_t)head * a.dp);
-    }
-    if (!is_v) {
-      const float inv = rsqrtf(warp_sum(ss) / (float)d + a.eps);
-#pragma unroll
-      for (int c = 0; c < NC; ++c) {
-        y[c].x *= inv * gain[c].x; y[c].y *= inv * gain[c].y;
-        const int pr = lane + 32 * c;
-        if (pr < a.pairs) {
-          const float2 cs = a.rope[(size_t)row * a.pairs + pr];
-          y[c] = make_float2(y[c].x * cs.x - y[c].y * cs.y, y[c].y * cs.x + y[c].x * cs.y);
-        }
-      }
-    }
-#pragma unroll
-    for (int c = 0; c < NC; ++c)
-      if (has[c]) store_pair<T>(dst + 2 * (lane + 32 * c), y[c], two[c], two[c]);       // head starts are multiples of 64 elements
-  }
-  if (!keep && i0 == 0)          // this block read the old ring rows of these channels above: it may overwrite them now
-    for (int i = max(0, n - (taps - 1)); i < n; ++i)
-#pragma unroll
-      for (int c = 0; c < NC; ++c)
-        if (has[c]) store_pair<T>(ring + (size_t)((p0 + i) % a.R) * a.C + 2 * (lane + 32 * c), input(i, c), two[c], rvec[c]);
-}
-
-// ---------------------------------------------------------------- short convolution in front of the recurrence
-template <typename T>
-struct RecConv {
-  const T* proj; int ldp;                       // rows whose columns [0, C) are the x branch
-  const float* x_b; const float* w; const float* w_b;       // [C], [taps, C], [C]
-  T* ring;                                      // [slots, R, C] projected rows (without x_b) by position
-  const int* state_slot; const int* q_start; const int* q_len; const int* kv_len;
-  T* u; int ldt, sq, sqp;                       // block-major operand: channel b * sq + j of row t at ((b * ldt) + t) * sqp + j
-  int4* tiles; int* n_tiles;                    // tile table of the gate product: {block, first operand row, rows, 0}
-  int T_rows, tn, C, taps, R, n_state;
-  int* status;
-};
-
 template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, float* v) {
-  if constexpr (V == 4 && sizeof(T) == 2) {
+  if constexpr (V == 8) {
+    load8<T>(p, v);
+  } else if constexpr (V == 4 && sizeof(T) == 2) {
     const uint2 q = *(const uint2*)p;
     const float2 x = __bfloat1622float2(*(const bf162*)&q.x), y = __bfloat1622float2(*(const bf162*)&q.y);
     v[0] = x.x; v[1] = x.y; v[2] = y.x; v[3] = y.y;
@@ -293,7 +155,9 @@ template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, 
   }
 }
 template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const float* v) {
-  if constexpr (V == 4 && sizeof(T) == 2) {
+  if constexpr (V == 8) {
+    store8<T>(p, v);
+  } else if constexpr (V == 4 && sizeof(T) == 2) {
     const bf162 x = __floats2bfloat162_rn(v[0], v[1]), y = __floats2bfloat162_rn(v[2], v[3]);
     *(uint2*)p = make_uint2(*(const uint32_t*)&x, *(const uint32_t*)&y);
   } else if constexpr (V == 4) {
@@ -306,6 +170,129 @@ template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const
     p[0] = to_t<T>(v[0]);
   }
 }
+// The first n of V elements (the others read as zero, or stay), with one access where `vec` says that all are there and aligned.
+template <typename T, int V> __device__ __forceinline__ void load_n(const T* p, int n, bool vec, float* v) {
+  if (vec) { load_v<T, V>(p, v); return; }
+#pragma unroll
+  for (int k = 0; k < V; ++k) v[k] = k < n ? to_f(p[k]) : 0.f;
+}
+template <typename T, int V> __device__ __forceinline__ void store_n(T* p, int n, bool vec, const float* v) {
+  if (vec) { store_v<T, V>(p, v); return; }
+#pragma unroll
+  for (int k = 0; k < V; ++k) if (k < n) p[k] = to_t<T>(v[k]);
+}
+
+// One warp per (head, tile of HS_TILE tokens); a lane owns V neighbouring dimensions of the head (whole rotated pairs).  TAPS > 0: the last
+// inputs and the weights stay in registers; 0: any number of taps, inputs re-read.
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvQkv<T> a) {
+  pdl_launch(); pdl_wait();
+  const int lane = threadIdx.x & 31, unit = blockIdx.x * 4 + (threadIdx.x >> 5), seq = blockIdx.z;
+  const int n = a.q_len[seq], i0 = blockIdx.y * HS_TILE;
+  if (unit >= a.H + 2 * a.G || i0 >= n) return;
+  const int row0 = a.q_start[seq], p0 = a.kv_len[seq] - n, slot = a.state_slot[seq], i1 = min(n, i0 + HS_TILE);
+  if (slot < 0 || slot >= a.n_state) { if (lane == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6E1); return; }
+  const bool is_q = unit < a.H, is_v = unit >= a.H + a.G;
+  const int d = is_v ? a.vdim : a.dim, head = is_q ? unit : (is_v ? unit - a.H - a.G : unit - a.H), e = lane * V;
+  const int ch = (is_v ? (a.H + a.G) * a.dim + head * a.vdim : unit * a.dim) + e;
+  const int taps = TAPS ? TAPS : a.taps, own = max(0, min(V, d - e));      // dimensions of this lane
+  const bool vec = own == V && ch % V == 0 && a.ldp % V == 0, wvec = own == V && ch % V == 0 && a.C % V == 0;
+  T* ring = a.ring + (size_t)slot * a.R * a.C + ch;
+  // input row i of this run (i < 0: what the sequence fed before, nothing in front of its start)
+  auto fresh = [&](int i, float* v) { load_n<T, V>(a.proj + (size_t)(row0 + i) * a.ldp + ch, own, vec, v); };
+  auto input = [&](int i, float* v) {
+    const int pos = p0 + i;
+    if (i >= 0) fresh(i, v);
+    else load_n<T, V>(ring + (size_t)((pos + a.R) % a.R) * a.C, pos < 0 ? 0 : own, pos >= 0 && wvec, v);
+  };
+  auto weight = [&](int j, float* v) { load_n<float, V>(a.w + (size_t)j * a.C + ch, own, wvec, v); };
+  constexpr int NH = TAPS > 1 ? TAPS - 1 : 1, NW = TAPS ? TAPS : 1;
+  float hist[NH][V], wr[NW][V], gain[V];
+  const float* norm = is_q ? a.q_norm : a.k_norm;
+#pragma unroll
+  for (int k = 0; k < V; ++k) gain[k] = is_v ? 1.f : (k < own ? norm[e + k] : 0.f);
+  if (TAPS) {
+#pragma unroll
+    for (int j = 0; j < NW; ++j) weight(j, wr[j]);
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) input(i0 - (TAPS - 1) + j, hist[j]);
+  }
+  const bool keep = n <= a.R - (taps - 1);              // short runs leave every input (a single tile), long ones the last taps - 1
+  for (int i = i0; i < i1; ++i) {
+    const int row = row0 + i;
+    float cur[V], y[V], ss = 0.f;
+    fresh(i, cur);
+    float2 turn[V / 2];
+#pragma unroll
+    for (int k = 0; k < V / 2; ++k) {
+      const int pr = e / 2 + k;
+      turn[k] = !is_v && pr < a.pairs ? a.rope[(size_t)row * a.pairs + pr] : make_float2(1.f, 0.f);
+    }
+    if (keep && own) store_n<T, V>(ring + (size_t)((p0 + i) % a.R) * a.C, own, wvec, cur);
+#pragma unroll
+    for (int k = 0; k < V; ++k) y[k] = 0.f;
+    if (TAPS) {
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[k] = fmaf(wr[j][k], hist[j][k], y[k]);
+#pragma unroll
+      for (int k = 0; k < V; ++k) y[k] = fmaf(wr[NW - 1][k], cur[k], y[k]);
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS - 1; ++j)
+#pragma unroll
+        for (int k = 0; k < V; ++k) hist[j][k] = hist[j + 1][k];
+      if (TAPS > 1)
+#pragma unroll
+        for (int k = 0; k < V; ++k) hist[NH - 1][k] = cur[k];
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        float u[V], w[V];
+        input(i - (taps - 1) + j, u);
+        weight(j, w);
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[k] = fmaf(w[k], u[k], y[k]);
+      }
+    }
+    T* dst;
+    if (is_q) dst = a.q + (size_t)row * a.q_stride + (size_t)head * a.dp;
+    else {
+      const int cs = a.slot_map[row];
+      if (cs < 0 || cs >= a.n_slots) { if (lane == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, row); continue; }     // warp-uniform
+      dst = a.cache + (size_t)cs * a.row_stride + (is_v ? (size_t)a.G * a.dp + (size_t)head * a.dvp : (size_t)head * a.dp);
+    }
+    if (!is_v) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) ss = fmaf(y[k], y[k], ss);
+      const float inv = rsqrtf(warp_sum(ss) / (float)d + a.eps);
+#pragma unroll
+      for (int k = 0; k < V / 2; ++k) {
+        const float u = y[2 * k] * inv * gain[2 * k], v = y[2 * k + 1] * inv * gain[2 * k + 1];
+        y[2 * k] = u * turn[k].x - v * turn[k].y; y[2 * k + 1] = v * turn[k].x + u * turn[k].y;
+      }
+    }
+    if (own) store_n<T, V>(dst + e, own, own == V, y);          // head starts are multiples of 64 elements
+  }
+  if (!keep && i0 == 0 && own)          // this block read the old ring rows of these channels above: it may overwrite them now
+    for (int i = max(0, n - (taps - 1)); i < n; ++i) {
+      float v[V];
+      fresh(i, v);
+      store_n<T, V>(ring + (size_t)((p0 + i) % a.R) * a.C, own, wvec, v);
+    }
+}
+
+// ---------------------------------------------------------------- short convolution in front of the recurrence
+template <typename T>
+struct RecConv {
+  const T* proj; int ldp;                       // rows whose columns [0, C) are the x branch
+  const float* x_b; const float* w; const float* w_b;       // [C], [taps, C], [C]
+  T* ring;                                      // [slots, R, C] projected rows (without x_b) by position
+  const int* state_slot; const int* q_start; const int* q_len; const int* kv_len;
+  T* u; int ldt, sq, sqp;                       // block-major operand: channel b * sq + j of row t at ((b * ldt) + t) * sqp + j
+  int4* tiles; int* n_tiles;                    // tile table of the gate product: {block, first operand row, rows, 0}
+  int T_rows, tn, C, taps, R, n_state;
+  int* status;
+};
 
 template <typename T, int V, int TAPS>
 __global__ void __launch_bounds__(128) rglru_conv_kernel(const RecConv<T> a) {
@@ -350,9 +337,17 @@ __global__ void __launch_bounds__(128) rglru_conv_kernel(const RecConv<T> a) {
     for (int j = 0; j < TAPS - 1; ++j) input(i0 - (TAPS - 1) + j, hist[j]);
   }
   const bool keep = n <= a.R - (taps - 1);
-  for (int i = i0; i < i1; ++i) {
-    float cur[V], y[V], r[V];
-    raw(i, r);
+  constexpr int NB = 4;                                 // rows loaded together
+  for (int ib = i0; ib < i1; ib += NB) {
+   float rows[NB][V];
+#pragma unroll
+   for (int q = 0; q < NB; ++q) raw(min(ib + q, i1 - 1), rows[q]);
+#pragma unroll
+   for (int q = 0; q < NB; ++q) {
+    const int i = ib + q;
+    if (i >= i1) break;
+    float cur[V], y[V];
+    const float* r = rows[q];
     if (keep) store_v<T, V>(ring + (size_t)((p0 + i) % a.R) * a.C, r);
 #pragma unroll
     for (int k = 0; k < V; ++k) { cur[k] = r[k] + xb[k]; y[k] = wb[k]; }
@@ -380,6 +375,7 @@ __global__ void __launch_bounds__(128) rglru_conv_kernel(const RecConv<T> a) {
       }
     }
     store_v<T, V>(u + (size_t)i * a.sqp, y);
+   }
   }
   if (!keep && i0 == 0)
     for (int i = max(0, n - (taps - 1)); i < n; ++i) {
@@ -394,7 +390,8 @@ __global__ void __launch_bounds__(128) rglru_conv_kernel(const RecConv<T> a) {
 template <typename T>
 struct LruScan {
   const T* u; int ldt, sq, sqp;                 // block-major operand of the gate product
-  const float* gates; int ldg;                  // [T, ldg]: block b's decay gate at columns [2 b sq, + sq), input gate at the next sq
+  float* gates; int ldg;                        // [T, ldg]: block b's decay gate at columns [2 b sq, + sq), input gate at the next sq; the
+                                                // aggregate pass leaves {a - 1, input of the recurrence} in their places
   const float* gates_b; const float* decay;     // the same order; [C]
   const T* y; int ldy; const float* y_b;        // y branch rows and bias
   float* state;                                 // [slots, depth + 1, C] states by position
@@ -404,6 +401,29 @@ struct LruScan {
   int C, depth, n_state;
   int* status;
 };
+
+// fp32 results either way; beside bf16 operands the hardware's approximations (a few units in the last place) do.
+template <typename T> __device__ __forceinline__ float sigmoid_t(float z);
+template <> __device__ __forceinline__ float sigmoid_t<float>(float z) { return 1.f / (1.f + expf(-z)); }
+template <> __device__ __forceinline__ float sigmoid_t<bf16>(float z) { return __fdividef(1.f, 1.f + __expf(-fmaxf(z, -80.f))); }
+// two at the price of one reciprocal
+template <typename T> __device__ __forceinline__ void sigmoid2_t(float x, float y, float& sx, float& sy);
+template <> __device__ __forceinline__ void sigmoid2_t<float>(float x, float y, float& sx, float& sy) { sx = sigmoid_t<float>(x); sy = sigmoid_t<float>(y); }
+template <> __device__ __forceinline__ void sigmoid2_t<bf16>(float x, float y, float& sx, float& sy) {
+  const float ex = 1.f + __expf(-fmaxf(x, -40.f)), ey = 1.f + __expf(-fmaxf(y, -40.f)), inv = __fdividef(1.f, ex * ey);
+  sx = inv * ey; sy = inv * ex;
+}
+// e^z - 1 for z <= 0: near zero the Taylor series (seven terms: relative error below 1e-7 down to z = -1/4), elsewhere the difference
+template <typename T> __device__ __forceinline__ float expm1_t(float z);
+template <> __device__ __forceinline__ float expm1_t<float>(float z) { return expm1f(z); }
+template <> __device__ __forceinline__ float expm1_t<bf16>(float z) {
+  float p = fmaf(z, 1.f / 7.f, 1.f);
+  p = fmaf(z * (1.f / 6.f), p, 1.f); p = fmaf(z * 0.2f, p, 1.f); p = fmaf(z * 0.25f, p, 1.f); p = fmaf(z * (1.f / 3.f), p, 1.f); p = fmaf(z * 0.5f, p, 1.f);
+  return z > -0.25f ? z * p : __expf(z) - 1.f;
+}
+template <typename T> __device__ __forceinline__ float sqrt_t(float z);
+template <> __device__ __forceinline__ float sqrt_t<float>(float z) { return sqrtf(z); }
+template <> __device__ __forceinline__ float sqrt_t<bf16>(float z) { return z * rsqrtf(fmaxf(z, 1e-30f)); }
 
 // PASS 0: aggregates of every chunk but a run's last one; 1: outputs and states.
 template <typename T, int V, int PASS>
@@ -417,7 +437,7 @@ __global__ void __launch_bounds__(128) lru_scan_kernel(const LruScan<T> a) {
   if (slot < 0 || slot >= a.n_state) { if (ch == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6E3); return; }
   const int b = ch / a.sq, j0 = ch % a.sq, gc = 2 * b * a.sq + j0;
   const T* u = a.u + ((size_t)b * a.ldt + row0) * a.sqp + j0;
-  const float* g = a.gates + (size_t)row0 * a.ldg + gc;
+  float* g = a.gates + (size_t)row0 * a.ldg + gc;
   float* st = a.state + (size_t)slot * (a.depth + 1) * a.C + ch;
   // aggregates of a run's chunks are consecutive rows; q_start / CHUNK + seq keeps the runs of a step apart
   float2* agg = a.agg + (size_t)(row0 / HS_CHUNK + seq) * a.C + ch;
@@ -447,30 +467,42 @@ __global__ void __launch_bounds__(128) lru_scan_kernel(const LruScan<T> a) {
 #pragma unroll
   for (int k = 0; k < V; ++k) h0[k] = h[k];
   const int i1 = min(n, (c + 1) * HS_CHUNK);
+  const bool ready = PASS == 1 && c < chunks - 1;       // the aggregate pass has been here
   for (int i0 = c * HS_CHUNK; i0 < i1; i0 += NB) {
     float zr[NB][V], zi[NB][V], us[NB][V], ys[NB][V];
 #pragma unroll
     for (int q = 0; q < NB; ++q) {
       const int i = min(i0 + q, i1 - 1);
       load_v<float, V>(g + (size_t)i * a.ldg, zr[q]); load_v<float, V>(g + (size_t)i * a.ldg + a.sq, zi[q]);
-      load_v<T, V>(u + (size_t)i * a.sqp, us[q]);
+      if (!ready) load_v<T, V>(u + (size_t)i * a.sqp, us[q]);
       if (PASS == 1) load_v<T, V>(a.y + (size_t)(row0 + i) * a.ldy + ch, ys[q]);
     }
 #pragma unroll
     for (int q = 0; q < NB; ++q) {
       const int i = i0 + q;
       if (i >= i1) break;
-      float o[V];
+      float o[V], m[V], in[V];
+      if (ready) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) { m[k] = zr[q][k]; in[k] = zi[q][k]; }
+      } else {
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+          float la, gate;
+          sigmoid2_t<T>(zr[q][k] + rb[k], zi[q][k] + ib[k], la, gate);
+          // with m = a - 1: a S = S + m S and 1 - a^2 = -m (m + 2), both exact to rounding where a is close to 1 (long memories)
+          m[k] = expm1_t<T>(la * dk[k]);
+          in[k] = sqrt_t<T>(-m[k] * (m[k] + 2.f)) * gate * us[q][k];
+        }
+      }
+      if (PASS == 0) { store_v<float, V>(g + (size_t)i * a.ldg, m); store_v<float, V>(g + (size_t)i * a.ldg + a.sq, in); }
 #pragma unroll
       for (int k = 0; k < V; ++k) {
-        const float la = dk[k] / (1.f + expf(-(zr[q][k] + rb[k]))), gate = 1.f / (1.f + expf(-(zi[q][k] + ib[k])));
-        // with m = a - 1: a S = S + m S and 1 - a^2 = -m (m + 2), both exact to rounding where a is close to 1 (long memories)
-        const float m = expm1f(la);
-        h[k] = fmaf(m, h[k], h[k]) + sqrtf(-m * (m + 2.f)) * gate * us[q][k];
-        if (PASS == 0) A[k] = fmaf(m, A[k], A[k]);
+        h[k] = fmaf(m[k], h[k], h[k]) + in[k];
+        if (PASS == 0) A[k] = fmaf(m[k], A[k], A[k]);
         if (PASS == 1) {
           const float z = ys[q][k] + yb[k];
-          o[k] = h[k] * z / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z)));      // 0.5 (1 + tanh(w)) = sigmoid(2 w)
+          o[k] = h[k] * z * sigmoid_t<T>(1.5957691216057308f * fmaf(0.044715f * z * z, z, z));      // 0.5 (1 + tanh(w)) = sigmoid(2 w)
         }
       }
       if (PASS == 1) {
@@ -606,16 +638,16 @@ struct CaConvQkv {
   int ldp, q_stride, row_stride, n_slots, H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state, n_seq, max_q_len; float eps;
 };
 
-template <typename T, int NC>
+template <typename T, int V>
 static int conv_qkv_launch(const CaConvQkv* c, cudaStream_t s) {
   const ConvQkv<T> a{(const T*)c->proj, c->ldp, c->w, c->q_norm, c->k_norm, (const float2*)c->rope, (T*)c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len, c->slot_map,
                      (T*)c->q, c->q_stride, (T*)c->cache, c->row_stride, c->n_slots, c->H, c->G, c->dim, c->dp, c->vdim, c->dvp, c->pairs, c->taps, c->R, c->C, c->n_state,
                      c->eps, c->status};
   const dim3 grid((c->H + 2 * c->G + 3) / 4, (c->max_q_len + HS_TILE - 1) / HS_TILE, c->n_seq);
-  if (c->taps == 2) CA_LAUNCH_PDL((conv_qkv_kernel<T, NC, 2>), grid, 128, 0, s, a);
-  else if (c->taps == 3) CA_LAUNCH_PDL((conv_qkv_kernel<T, NC, 3>), grid, 128, 0, s, a);
-  else if (c->taps == 4) CA_LAUNCH_PDL((conv_qkv_kernel<T, NC, 4>), grid, 128, 0, s, a);
-  else CA_LAUNCH_PDL((conv_qkv_kernel<T, NC, 0>), grid, 128, 0, s, a);
+  if (c->taps == 2) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 2>), grid, 128, 0, s, a);
+  else if (c->taps == 3) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 3>), grid, 128, 0, s, a);
+  else if (c->taps == 4) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 4>), grid, 128, 0, s, a);
+  else CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 0>), grid, 128, 0, s, a);
   CA_CHECK_LAUNCH("conv_qkv");
   return CA_OK;
 }
@@ -629,13 +661,13 @@ extern "C" int cuteafd_conv_qkv(const CaConvQkv* c, int f32, cudaStream_t s) {
   if (c->n_seq <= 0 || c->max_q_len <= 0) return CA_OK;
   CA_REQUIRE(c->n_seq <= 65535 && (c->max_q_len + HS_TILE - 1) / HS_TILE <= 65535, "conv_qkv: step too large");
   const int nc = ((c->dim > c->vdim || c->G == 0 ? c->dim : c->vdim) + 63) / 64;
-  if (nc <= 1) return f32 ? conv_qkv_launch<float, 1>(c, s) : conv_qkv_launch<bf16, 1>(c, s);
-  if (nc <= 2) return f32 ? conv_qkv_launch<float, 2>(c, s) : conv_qkv_launch<bf16, 2>(c, s);
-  return f32 ? conv_qkv_launch<float, 4>(c, s) : conv_qkv_launch<bf16, 4>(c, s);
+  if (nc <= 1) return f32 ? conv_qkv_launch<float, 2>(c, s) : conv_qkv_launch<bf16, 2>(c, s);
+  if (nc <= 2) return f32 ? conv_qkv_launch<float, 4>(c, s) : conv_qkv_launch<bf16, 4>(c, s);
+  return f32 ? conv_qkv_launch<float, 8>(c, s) : conv_qkv_launch<bf16, 8>(c, s);
 }
 
 struct CaRecurrence {          // one recurrent layer's step: shared by its convolution and its scan
-  const void* x; const void* y; const float* x_b; const float* y_b; const float* conv; const float* conv_b; void* ring; float* state; void* u; const float* gates;
+  const void* x; const void* y; const float* x_b; const float* y_b; const float* conv; const float* conv_b; void* ring; float* state; void* u; float* gates;
   const float* gates_b; const float* decay; void* agg; void* out; void* tiles; int* n_tiles; const int* state_slot; const int* q_start; const int* q_len; const int* kv_len;
   int* status;
   int ldp, ldt, sq, sqp, ldg, ldo, tn, T, C, taps, depth, n_state, n_seq, max_q_len, agg_rows;

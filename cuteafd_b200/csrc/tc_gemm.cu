@@ -162,10 +162,13 @@ __device__ __forceinline__ void peer_store(const TcArgs& a, int row, int n, bf16
 }
 
 // Values of an XACT instantiation: bounded logits, or g = min(g + b, p), u = clamp(u + b2, -p, p) -> g * sigmoid(1.702 g) * (u + 1).
-__device__ __forceinline__ float epi_softcap(const TcArgs& a, float v) { return a.act == 2 ? a.act_p * tanhf(v / a.act_p) : v; }
+// (p tanh(v / p) = p - 2 p / (1 + e^(2 v / p)): absolute error of a few 1e-7 p, in short code - it is unrolled over the tile's columns.)
+__device__ __forceinline__ float epi_softcap(const TcArgs& a, float v) {
+  return a.act == 2 ? a.act_p - __fdividef(2.f * a.act_p, 1.f + __expf(__fdividef(2.f * v, a.act_p))) : v;
+}
 __device__ __forceinline__ float epi_clamped_glu(const TcArgs& a, float g, float u, float b, float b2) {
   g = fminf(g + b, a.act_p); u = fminf(fmaxf(u + b2, -a.act_p), a.act_p);
-  return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+  return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
 }
 
 // PEER instantiations carry the peer-store epilogue; the others are the plain local kernels (the extra code costs
@@ -349,8 +352,8 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
     const int q4 = warp & 3;                 // tensor-memory lane quarter this warp may read
     const int et = q4 * 32 + lane;           // 0..127: weight row inside the tile
     uint32_t tc = 0, stg_uses = 0;
-    // staged (transposed) store: plain bf16 output of a 64+-token tile, 16-byte aligned rows
-    const bool stage_ok = C::STG_BYTES > 0 && splits == 1 && a.epi != EPI_F32 && a.Y != nullptr && !(QOUT && a.q_out) && !(PEER && a.n_peer) &&
+    // staged (transposed) store: plain bf16 or fp32 output of a 64+-token tile, 16-byte aligned rows
+    const bool stage_ok = C::STG_BYTES > 0 && splits == 1 && a.Y != nullptr && !(QOUT && a.q_out) && !(PEER && a.n_peer) &&
                           a.ldy % 8 == 0 && a.N % 8 == 0 && a.grp_cols % 8 == 0 && ((uintptr_t)a.Y & 15) == 0 && (a.epi != EPI_BF16_RESIDUAL || ((uintptr_t)a.R & 15) == 0);
     float* stg = (float*)(smem + C::NSTAGE * C::STAGE_BYTES);
     bool stg_fail = false;
@@ -456,8 +459,15 @@ __global__ void __launch_bounds__(192, TcCfg<KIND, TN, SWIGLU>::OCC) tc_linear_k
             mbar_arrive(&stg_bar);
             if (!mbar_wait_bounded(&stg_bar, stg_uses & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_EPILOGUE, 0x7000 + w); stg_fail = true; break; }
             ++stg_uses;
-            // 16 rows x 16 groups of 8 features; thread -> (row, group), two per thread.  A buffer is rewritten two chunks
-            // later, after every warp has passed the NEXT chunk's barrier, i.e. finished these reads.
+            // 16 rows x 16 groups of 8 features; thread -> (row, group), two per thread (fp32: 32 groups of 4, whole 512-byte rows per
+            // warp).  A buffer is rewritten two chunks later, after every warp has passed the NEXT chunk's barrier, i.e. finished these reads.
+            if (a.epi == EPI_F32) {
+#pragma unroll
+              for (int h = 0; h < 4; ++h) {
+                const int row = (warp - 2) + h * 4, c = c0 + row, nn = nt * 128 + lane * 4;
+                if (c < nrows && nn < a.N) *(float4*)((float*)a.Y + obase + (size_t)c * a.ldy + nn) = *(const float4*)(buf + row * 128 + lane * 4);
+              }
+            } else
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
               const int idx = (warp - 2) * 32 + lane + h * 128, row = idx >> 4, grp = idx & 15;

@@ -68,7 +68,7 @@ class HybridLane(StackLane):
 
     def ffn(self, width: int) -> dict:
         def make():
-            h, h_act = self._operand(self.cap, up(width, 8), min(self.tn, 128) if not self.eng.f32 else None)
+            h, h_act = self._operand(self.cap, up(width, 8))
             return {"h": h, "h_act": h_act, **({"g": torch.zeros_like(h), "u": torch.zeros_like(h)} if self.eng.f32 else {})}
         return self.get(("ffn", width), make)
 

@@ -173,7 +173,7 @@ class HybridStackEngine(StackBase, Engine):
         if sh.n_logits:
             ops.norm_rows(L.x, spec.hidden, sh.n_logits, src_rows=md["logit_rows"], gain=w.final_norm, xn=L.xln, **rows)
             cap = spec.logit_softcap
-            ops.tc_linear(w.lm_head, L.xln_act, L.logits, rows=sh.n_logits, act="softcap" if cap else None, bound=cap, status=st)
+            ops.tc_linear(w.lm_head, L.head_operand(sh.n_logits), L.logits, rows=sh.n_logits, act="softcap" if cap else None, bound=cap, status=st)
             ops.argmax_rows(L.logits, L.next_tok, rows=sh.n_logits, status=L.tok_status)
             self.launches_per_step += 3
         return L

@@ -156,7 +156,7 @@ class LatentStackEngine(StackBase, MlaEngine):
         self.launches_per_step += 1
         if sh.n_logits:
             ops.stack_stream(L.x, ops.emit_arg(norm=(w.final_norm, w.final_b, w.final_alpha), xn=L.xln), sh.n_logits, f32=self.f32, src_rows=md["logit_rows"])
-            ops.tc_linear(w.lm_head, L.xln_act, L.logits, rows=sh.n_logits, status=self.status)
+            ops.tc_linear(w.lm_head, L.head_operand(sh.n_logits), L.logits, rows=sh.n_logits, status=self.status)
             ops.argmax_rows(L.logits, L.next_tok, rows=sh.n_logits, status=L.tok_status)
             self.launches_per_step += 3
         return L

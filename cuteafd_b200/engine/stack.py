@@ -5,6 +5,7 @@ import os
 
 import torch
 
+from .. import ops
 from ..models.latent_stack import up
 from ..ops import ActBuffer, KIND_BF16, KIND_F32, pick_tn
 from .engine import Lane
@@ -27,6 +28,7 @@ class StackLane(Lane):
         self.mix = torch.zeros(cap, Wp, dtype=self.dt, device=self.dev)
         rows = min(cap, 256)
         self.xln, self.xln_act = self._operand(rows, Wp)
+        self._head_acts: dict = {}
         self.logits = torch.zeros(rows, eng.spec.vocab, dtype=torch.float32, device=self.dev)
         i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=self.dev)
         self.next_tok, self.tok_status = i32(cap), i32(cap)
@@ -42,7 +44,17 @@ class StackLane(Lane):
             rows = min(self.cap, up(n, 256))
             self.xln, self.xln_act = self._operand(rows, self.eng.Wp)
             self.logits = torch.zeros(rows, self.eng.spec.vocab, dtype=torch.float32, device=self.dev)
+            self._head_acts.clear()
             self.eng.drop_graphs()                   # captured steps hold the old addresses
+
+    def head_operand(self, n: int) -> ActBuffer:
+        """The head's operand in token tiles that fit the `n` rows it multiplies (a prompt's step has few)."""
+        tn = pick_tn(min(n, self.tn))
+        if self.eng.f32 or tn == self.xln_act.tn:
+            return self.xln_act
+        if tn not in self._head_acts:
+            self._head_acts[tn] = ActBuffer(self.kind, self.xln.shape[0], self.eng.Wp, tn, self.xln, ops.encode_tmap(self.xln, tn))
+        return self._head_acts[tn]
 
     def get(self, key, make):
         if key not in self._bufs:

@@ -423,7 +423,7 @@ def tudilix_spec(n_layers: int = 12, hidden: int = 4096, heads: int = 32, kv_hea
     attention layer on the keys and values of the one before it; dense feed-forwards behind the attention layers, or behind every layer."""
     rec = BlockSpec(None, rec=RecurrentSpec(width=hidden, blocks=blocks, conv_taps=4), ffn=DenseFfnSpec(ff, 7.0) if ffn_everywhere else None)
     attn = AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, window=window, qk_norm=True, conv_taps=4,
-                         rope_dims=64, rope_scaling=RopeScaling(8.0, 8192, 32.0, 1.0))
+                         rope_dims=64, rope_scaling=RopeScaling(4.0, 16384, 24.0, 1.0))
     layers, last = [], -1
     for i in range(n_layers):
         if i % 3 != 2:
@@ -432,7 +432,7 @@ def tudilix_spec(n_layers: int = 12, hidden: int = 4096, heads: int = 32, kv_hea
         layers.append(BlockSpec(dataclasses.replace(attn, kv_from=last), ffn=DenseFfnSpec(ff, 7.0)))
         last = i if last < 0 else -1
     return ModelSpec(name="tudilix-shape", family="tudilix", vocab=65536, hidden=hidden, n_layers=n_layers, rms_eps=1e-6, attn=attn, moe=MoESpec(n_experts=0, n_shared=0),
-                     quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(layers), residual_mult=0.5, logit_softcap=30.0)
+                     quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(layers), residual_mult=0.5, logit_softcap=40.0)
 
 
 NAMED_SPECS = {

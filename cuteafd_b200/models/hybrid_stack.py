@@ -2,7 +2,7 @@
 
 Everything that reads the same row is one matrix (`w_in`): queries, keys and values of an attention layer, or the two branches of a
 recurrent one.  The two block-diagonal gates of a recurrence are one product grouped over the blocks (`w_gates`, per block the decay
-gate's rows, then the input gate's).  Norm weights stored around zero become plain gains, lambda becomes the log decay at an open gate.
+gate's rows, then the input gate's).  Norm weights (stored as distances from one) become plain gains, lambda becomes the log decay at an open gate.
 
 Widths are padded so that every operand row starts on a 16-byte boundary (multiples of 8); pads are zero in the weights, so they stay
 zero in the activations.

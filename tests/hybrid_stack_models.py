@@ -29,7 +29,7 @@ MIXED = {"architecture": "Tudilix", "vocab": 301, "width": 200, "norm": {"eps": 
          "layers": [rglru(120, 3, 3, ff=72, limit=0.8), attention(6, 2, 40, 24, 70, 4, 12, 0.3, scaling=yarn(4.0, 64)), rglru(96, 2, 4),
                     attention(4, 2, 40, 24, 33, 2, 12, 0.25, scaling=yarn(4.0, 64), ff=100, limit=1.3, kv_from=1), attention(3, 1, 72, 136, 128, 3, 72, 0.2, base=500.0)]}
 # odd widths everywhere (rows and heads that do not start on 16 bytes), one tap and many, windows of one token and of whole pages
-ODD = {"architecture": "Tudilix", "vocab": 97, "width": 90, "norm": {"eps": 1e-5}, "residual_mult": 1.0, "logit_softcap": 30.0,
+ODD = {"architecture": "Tudilix", "vocab": 97, "width": 90, "norm": {"eps": 1e-5}, "residual_mult": 1.0, "logit_softcap": 26.0,
        "layers": [attention(7, 7, 33, 45, 64, 5, 10, 0.4, scaling=yarn(2.0, 32, fast=4.0), ff=27, limit=2.0), rglru(45, 3, 1), attention(5, 1, 20, 13, 1, 1, 20, 0.3),
                   rglru(35, 1, 6, ff=36), attention(14, 7, 33, 45, 65, 2, 10, 0.3, scaling=yarn(2.0, 32, fast=4.0), kv_from=0)]}
 # every width class of the attention kernels, groups that do not divide a tile of rows

@@ -257,7 +257,7 @@ class Paged:
         self.table = self.table.to(DEV)
 
 
-@pytest.mark.parametrize("H,G,dim,vdim,window,splits", [(8, 1, 128, 80, 96, 2), (3, 3, 40, 24, 1, 1), (6, 2, 64, 64, 64, 3), (9, 1, 200, 256, 65, 1), (5, 1, 192, 33, 63, 4), (40, 1, 100, 192, 130, 1),
+@pytest.mark.parametrize("H,G,dim,vdim,window,splits", [(10, 1, 128, 72, 90, 2), (3, 3, 40, 24, 1, 1), (6, 2, 64, 64, 64, 3), (9, 1, 200, 256, 65, 1), (5, 1, 192, 33, 63, 4), (40, 1, 100, 192, 130, 1),
                                                         (12, 4, 256, 128, 0, 5), (128, 1, 16, 48, 200, 2), (4, 2, 130, 136, 4096, 7), (96, 1, 64, 130, 70, 1)])
 def test_window_attention(H, G, dim, vdim, window, splits):
     """Ragged batch (prompt portions, decoded tokens, a first token) on scattered pages; rows point at the first key of their window, at the one

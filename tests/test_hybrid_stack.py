@@ -73,7 +73,7 @@ def test_plan_reads_the_family(tmp_path):
 
 
 # ------------------------------------------------------------------ the oracle, mechanism by mechanism
-def test_oracle_norm_is_stored_around_zero():
+def test_oracle_norm_weights_are_distances_from_one():
     y = oracle.centred_norm(torch.tensor([[3.0, 4.0]]), torch.tensor([0.0, 1.0]), 0.5)
     assert torch.allclose(y, torch.tensor([[3.0, 8.0]]) / math.sqrt(12.5 + 0.5))
 

@@ -13,6 +13,8 @@ Only token ids / status words return to the host.
 """
 from __future__ import annotations
 
+import contextlib
+import gc
 import math
 import os
 from dataclasses import dataclass
@@ -36,6 +38,20 @@ PREFILL_ATTN_MIN_Q = int(os.environ.get("CUTEAFD_PREFILL_ATTN_MIN_Q", "64"))
 FP8_FUSE_GATE_UP = os.environ.get("CUTEAFD_FP8_FUSE_GATE_UP", "1") != "0"      # FP8 dense FFNs: gate and up projections as one GEMM
 CLUSTER_KINDS = (KIND_BF16,) + tuple(FP4_KINDS)       # operand kinds with a cluster split-K kernel besides FP8
 ROUTER_FUSED = os.environ.get("CUTEAFD_ROUTER_FUSED", "0") == "1"
+
+
+@contextlib.contextmanager
+def graph_capture(graph: torch.cuda.CUDAGraph):
+    """`torch.cuda.graph` without the cyclic garbage collector: were it to run meanwhile and find graphs of an engine that is gone, their
+    release would invalidate the capture."""
+    collecting = gc.isenabled()
+    gc.disable()
+    try:
+        with torch.cuda.graph(graph):
+            yield
+    finally:
+        if collecting:
+            gc.enable()
 
 
 @dataclass
@@ -648,7 +664,6 @@ class Engine:
         else:
             self.launches_per_step += stage.receive(L.x, T)         # the residual rows arrive from the stage before
         self._hc_pending = "init" if spec.hyper_streams else None
-        import contextlib
         from ..utils.trace import nvtx
         timed = self.layer_clock is not None and not torch.cuda.is_current_stream_capturing()
         for li in range(spec.n_layers):
@@ -744,7 +759,7 @@ class Engine:
             self.on_mtp_step = None                          # the capture launches nothing: nobody must be told
             try:
                 graph = torch.cuda.CUDAGraph()
-                with torch.cuda.graph(graph):
+                with graph_capture(graph):
                     lane = self.mtp_forward(depth, sh, buf)
             finally:
                 if hook is not None:
@@ -800,7 +815,7 @@ class Engine:
 
     def _capture(self, sh: StepShape):
         graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(graph):
+        with graph_capture(graph):
             lane = self.forward(sh)
         self.graphs[sh.key()] = (graph, lane, self.launches_per_step)
         self.graph_captures += 1

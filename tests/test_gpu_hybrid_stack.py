@@ -589,3 +589,24 @@ def test_trace_program_end_to_end(tmp_path):
     read = lambda n, rows: torch.frombuffer(bytearray((out / f"{n}.f32").read_bytes()), dtype=torch.float32).reshape(rows, cfg["vocab"])
     check(torch.cat([read(1, 4), read(2, 1)]), torch.stack([wa[70], wa[71], wb[4], wb[0], wa[79]]), "float32")
     assert sorted(x.name for x in out.iterdir()) == ["1.f32", "2.f32"]
+
+
+def test_a_capture_survives_garbage_from_an_engine_that_is_gone(tmp_path):
+    """Captured graphs of a dropped engine sit in reference cycles; the collector must not release them in the middle of another capture."""
+    import gc
+    toks = tokens(PLAIN, 12, 70)
+    old, _ = build(PLAIN, tmp_path / "a", "bfloat16")
+    for n in (1, 2, 3):
+        run_portions(old, f"r{n}", toks, [n])
+    assert old.engine.graph_captures >= 3
+    rep, t = build(PLAIN, tmp_path / "b", "bfloat16")
+    run_portions(rep, "warm", toks, [12])
+    before = gc.get_threshold()
+    try:
+        old.engine.self_reference = old.engine
+        del old
+        gc.set_threshold(1, 1, 1)                            # collect at every opportunity
+        check(run_portions(rep, "x", toks, [1]), logits(PLAIN, t, toks), "bfloat16")
+    finally:
+        gc.set_threshold(*before)
+    assert rep.engine.graph_captures >= 1

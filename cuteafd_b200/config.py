@@ -65,6 +65,25 @@ class AttentionSpec:
     rope_dims: int = 0
     rope_scaling: Optional["RopeScaling"] = None
     kv_from: int = -1
+    # Kind "conv_gqa" in hyper-connected stacks, besides: `keep_first` keys of the sequence stay visible behind the window; `sink`; one norm over
+    # all heads of q (and of k) at once; keys that are also the values (as they leave the convolution, no value projection); biases of the
+    # projections; an output gate with one number per head (`out_gate`) or, with `gate_values`, one per output value.
+    keep_first: int = 0
+    qk_norm_whole: bool = False
+    values_are_keys: bool = False
+    qkv_bias: bool = False
+    out_bias: bool = False
+    gate_values: bool = False
+
+    @property
+    def gate_width(self) -> int:
+        """Numbers of the output gate per token."""
+        return 0 if not self.out_gate else (self.n_heads * self.v_head_dim if self.gate_values else self.n_heads)
+
+    @property
+    def conv_channels(self) -> int:
+        """Projected channels in front of the convolution (kind "conv_gqa")."""
+        return self.n_heads * self.head_dim + (self.kv_token_elems if not self.values_are_keys else self.n_kv_heads * self.head_dim)
 
     @property
     def softmax_scale(self) -> float:
@@ -134,30 +153,53 @@ class QuantSpec:
 @dataclass(frozen=True)
 class RecurrentSpec:
     """A recurrent mixer.  "rglru": two branches of `width` channels, one gated by GELU, the other through a convolution of `conv_taps` and a
-    real-gated linear recurrence whose two gates are block-diagonal (`blocks` square blocks)."""
+    real-gated linear recurrence whose two gates are block-diagonal (`blocks` square blocks).
+    Linear attention of `heads` heads with a state of `dim` x `vdim` each: "retention" (a constant decay per head, `decay`; the first `rope_dims`
+    dimensions of q and k rotated, i with i + rope_dims / 2) and "gla" (a decay per key channel and token, the sigmoid of a projection of rank
+    `rank` to the power 1 / `tau`; rank 0: as wide as the snapshot's tensors)."""
     kind: str = "rglru"
     width: int = 256
     blocks: int = 1
     conv_taps: int = 4
+    heads: int = 0
+    dim: int = 0
+    vdim: int = 0
+    decay: tuple = ()
+    rope_dims: int = 0
+    rope_theta: float = 10000.0
+    tau: float = 1.0
+    rank: int = 0
 
 
 @dataclass(frozen=True)
 class DenseFfnSpec:
     """A dense feed-forward.  "clamped_glu": gate g = min(., limit), linear half u clamped to [-limit, limit], g sigmoid(1.702 g) (u + 1);
-    biases on all three projections."""
+    biases on all three projections.  "silu_glu": silu(g) u, no biases."""
     intermediate: int
-    limit: float
+    limit: float = 0.0
     activation: str = "clamped_glu"
 
 
 @dataclass(frozen=True)
 class BlockSpec:
     """One layer of a stack whose layers differ: its mixer (attention, or a recurrent one) and its feed-forward (routed experts, dense, or
-    neither: the layer has none)."""
+    neither: the layer has none).  A layer with both mixers runs them side by side on the same input and adds their outputs, `merge_scales`
+    times each, with `merge_norm` behind an RMS norm each."""
     attn: Optional[AttentionSpec] = field(default_factory=lambda: AttentionSpec(kind="latent"))
     moe: Optional[MoESpec] = None
     rec: Optional[RecurrentSpec] = None
     ffn: Optional[DenseFfnSpec] = None
+    merge_scales: tuple = (1.0, 1.0)
+    merge_norm: bool = False
+
+
+@dataclass(frozen=True)
+class PairTableSpec:
+    """A table added to the token embedding, addressed by the token and the one before it: row (previous * mul_prev + token * mul_cur) mod buckets;
+    the row behind the last starts a sequence."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
 
 
 @dataclass(frozen=True)
@@ -197,8 +239,11 @@ class ModelSpec:
     # Stacks of unequal layers (`blocks` non-empty; `attn` / `moe` above then describe the first layer of their kind), over an fp32 residual.
     # "latent" stacks: parallel layers (one norm, attention and feed-forward read it, both scaled per channel and added), Dynamic Tanh for a
     # norm.  "hybrid" stacks: windowed attention and recurrent layers, RMS norms in front of and behind every sub-layer, whose result is
-    # added `residual_mult` times; logits bounded by `logit_softcap` (0 = not).
+    # added `residual_mult` times; logits bounded by `logit_softcap` (0 = not).  "hyper" stacks (`streams` > 0): that many residual streams with
+    # constant weights per sub-layer (how it reads them, how its output and the old streams make the new ones); mixers alone or side by side.
     blocks: tuple = ()
+    streams: int = 0
+    pair_table: Optional[PairTableSpec] = None
     residual_mult: float = 1.0
     logit_softcap: float = 0.0
     loop: Optional[LoopSpec] = None
@@ -206,13 +251,15 @@ class ModelSpec:
 
     @property
     def stack(self) -> str:
-        """Which kind of stack `blocks` describes: "latent", "hybrid", or "" for models without blocks."""
+        """Which kind of stack `blocks` describes: "latent", "hybrid", "hyper", or "" for models without blocks."""
         if not self.blocks:
             return ""
+        if self.streams:
+            return "hyper"
         return "latent" if all(b.attn is not None and b.attn.kind == "latent" for b in self.blocks) else "hybrid"
 
     def kv_layers(self) -> list:
-        """Layers of a hybrid stack that keep keys and values of their own."""
+        """Layers of a hybrid or hyper-connected stack that keep keys and values of their own."""
         return [i for i, b in enumerate(self.blocks) if b.attn is not None and b.attn.kv_from < 0]
 
     def layer_runs(self) -> list:
@@ -271,7 +318,7 @@ class ModelSpec:
     def attn_params(self, attn: Optional[AttentionSpec] = None) -> int:
         a, h = attn or self.attn, self.hidden
         if a.kind == "conv_gqa":
-            return h * (a.n_heads * (a.head_dim + a.v_head_dim) + a.kv_token_elems)
+            return h * (a.conv_channels + a.gate_width + a.n_heads * a.v_head_dim)
         if a.kind == "latent":
             return (h * (a.n_heads * a.head_dim + a.kv_lora_rank + (a.n_heads if a.out_gate else 0)) +
                     a.n_heads * (a.head_dim + a.v_head_dim) * a.kv_lora_rank + a.n_heads * a.v_head_dim * h)
@@ -288,10 +335,12 @@ class ModelSpec:
 
     def weight_bytes(self) -> dict:
         """Bytes per category for the whole model (planner input)."""
-        if self.stack == "hybrid":
-            db = self.bits(self.quant.dense) / 8
-            rec = sum(3 * self.hidden * b.rec.width + 2 * b.rec.width ** 2 // b.rec.blocks for b in self.blocks if b.rec is not None)
-            return {"routed_experts": 0.0, "shared_experts": 0.0, "router": 0.0, "embed_head": self.vocab * self.hidden * (2 + db),
+        if self.stack in ("hybrid", "hyper"):
+            db, eb, moes = self.bits(self.quant.dense) / 8, self.bits(self.quant.experts) / 8, [b.moe for b in self.blocks if b.moe is not None]
+            rec = sum(self.recurrent_params(b.rec) for b in self.blocks if b.rec is not None)
+            return {"routed_experts": sum(3 * self.hidden * m.intermediate * m.n_experts for m in moes) * eb,
+                    "shared_experts": sum(3 * self.hidden * m.shared_inter for m in moes if m.n_shared) * db, "router": sum(m.n_experts for m in moes) * self.hidden * db,
+                    "embed_head": self.vocab * self.hidden * (2 + db) + (2 * (self.pair_table.buckets + 1) * self.hidden if self.pair_table else 0),
                     "dense_ffn": sum(3 * self.hidden * b.ffn.intermediate for b in self.blocks if b.ffn is not None) * db,
                     "attention": (rec + sum(self.attn_params(b.attn) for b in self.blocks if b.attn is not None)) * db}
         if self.blocks:
@@ -313,25 +362,34 @@ class ModelSpec:
         return {"routed_experts": routed, "shared_experts": shared, "dense_ffn": dense_ffn,
                 "attention": attn, "router": router, "embed_head": embed}
 
+    def recurrent_params(self, r: RecurrentSpec) -> int:
+        if r.kind == "rglru":
+            return 3 * self.hidden * r.width + 2 * r.width ** 2 // r.blocks
+        return self.hidden * r.heads * (2 * r.dim + 3 * r.vdim) + r.rank * (self.hidden + r.heads * r.dim)
+
     def kv_row_elems(self) -> int:
-        """Elements of a cached token's row in a hybrid stack: the widest layer's key heads, then its value heads."""
+        """Elements of a cached token's row in a hybrid or hyper-connected stack: the widest layer's key heads, then its value heads."""
         up = lambda n: -(-n // 64) * 64
         return max((b.attn.n_kv_heads * (up(b.attn.head_dim) + up(b.attn.v_head_dim)) for b in self.blocks if b.attn is not None and b.attn.kv_from < 0), default=0)
 
     def state_bytes_per_seq(self, depth: int = 8) -> int:
-        """Bytes of one sequence's state slot in a hybrid stack (`engine.hybrid_stack`): convolution inputs and recurrent states of the last
-        positions, `depth` of which can be taken back."""
-        eb, n = 2 if self.quant.dense == "bf16" else 4, 0
+        """Bytes of one sequence's state slot in a hybrid or hyper-connected stack (`engine.hybrid_stack`, `engine.hyper_stack`): convolution
+        inputs and recurrent states of the last positions, `depth` of which can be taken back."""
+        eb, n = 2 if self.quant.dense == "bf16" else 4, 4 * (depth + 1) if self.pair_table is not None else 0
         for b in self.blocks:
-            if b.rec is not None:
-                n += b.rec.width * ((b.rec.conv_taps - 1 + depth) * eb + (depth + 1) * 4)
-            else:
-                n += (b.attn.n_heads * b.attn.head_dim + b.attn.kv_token_elems) * (b.attn.conv_taps - 1 + depth) * eb
+            r, a = b.rec, b.attn
+            if r is not None and r.kind == "rglru":
+                n += r.width * ((r.conv_taps - 1 + depth) * eb + (depth + 1) * 4)
+            elif r is not None:         # two states, the last inputs of the recurrence, two positions per head
+                vp = -(-r.vdim // 4) * 4
+                n += r.heads * (4 * (2 * r.dim * vp + depth * (2 * r.dim + vp)) + 8)
+            if a is not None and not (self.streams and a.conv_taps == 1):
+                n += a.conv_channels * (a.conv_taps - 1 + depth) * eb
         return n
 
     def kv_bytes_per_token(self) -> float:
         per = {"fp8": 1.0, "f32": 4.0}.get(self.quant.kv, 2.0)
-        if self.stack == "hybrid":  # one row width for every layer with keys of its own, heads in whole 64-element chunks
+        if self.stack in ("hybrid", "hyper"):  # one row width for every layer with keys of its own, heads in whole 64-element chunks
             return len(self.kv_layers()) * self.kv_row_elems() * per
         if self.blocks:             # one row width for every layer run (the widest latent, in whole 64-element chunks)
             return len(self.layer_runs()) * max(-(-b.attn.kv_token_elems // 64) * 64 for b in self.blocks) * per
@@ -435,6 +493,28 @@ def tudilix_spec(n_layers: int = 12, hidden: int = 4096, heads: int = 32, kv_hea
                      quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(layers), residual_mult=0.5, logit_softcap=40.0)
 
 
+def vozetar_spec(n_layers: int = 6, hidden: int = 4096, heads: int = 32, kv_heads: int = 4, ff: int = 12288, window: int = 2048, rec_heads: int = 16, rec_dim: int = 128,
+                 rec_vdim: int = 256, experts: int = 0, expert_ff: int = 1536, streams: int = 4, mixers: str = "PGA") -> ModelSpec:
+    """Vozetar at the size of a real model's layers (synthetic weights).  `mixers` repeats over the layers: P windowed attention beside retention, G
+    windowed attention (values are the keys) beside gated linear attention, A full attention.  `experts` > 0: routed experts (with a shared one)
+    instead of a dense feed-forward in every second layer."""
+    base = AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, rope_dims=128)
+    windowed = dataclasses.replace(base, window=window, keep_first=4, rope_dims=64, rope_theta=1e6)
+    rec = RecurrentSpec(kind="retention", heads=rec_heads, dim=rec_dim, vdim=rec_vdim, decay=tuple(1.0 - 2.0 ** (-5 - 7.0 * i / rec_heads) for i in range(rec_heads)), rope_dims=rec_dim)
+    kinds = {"P": (dataclasses.replace(windowed, qkv_bias=True, sink=True), rec, (1.2, 1.1), False),
+             "G": (dataclasses.replace(windowed, values_are_keys=True, conv_taps=3, qk_norm_whole=True, out_gate=True), dataclasses.replace(rec, kind="gla", decay=(), rope_dims=0, tau=16.0, rank=16),
+                   (0.5, 0.5), True),
+             "A": (dataclasses.replace(base, rope_interleaved=False, conv_taps=4, qkv_bias=True, out_bias=True, sink=True, out_gate=True, gate_values=True), None, (1.0, 1.0), False)}
+    moe = MoESpec(n_experts=experts, top_k=8, intermediate=expert_ff, n_shared=1, shared_intermediate=expert_ff, scoring="sigmoid", normalize=False, n_group=8, topk_group=4) if experts else None
+    blocks = []
+    for i in range(n_layers):
+        attn, r, scales, norm = kinds[mixers[i % len(mixers)]]
+        routed = moe is not None and i % 2 == 1
+        blocks.append(BlockSpec(attn, moe if routed else None, r, None if routed else DenseFfnSpec(ff, activation="silu_glu"), scales, norm))
+    return ModelSpec(name="vozetar-shape", family="vozetar", vocab=65536, hidden=hidden, n_layers=n_layers, rms_eps=1e-5, attn=blocks[0].attn, moe=moe or MoESpec(n_experts=0, n_shared=0),
+                     quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(blocks), streams=streams, pair_table=PairTableSpec(65521, 31, 17))
+
+
 NAMED_SPECS = {
     "tiny": tiny_spec,
     "hybrid-gdn": hybrid_gdn_spec,
@@ -444,6 +524,7 @@ NAMED_SPECS = {
     "qwen3-235b": qwen3_235b_spec,
     "bedovik": bedovik_spec,
     "tudilix": tudilix_spec,
+    "vozetar": vozetar_spec,
     "ep-microbench": ep_microbench_spec,
 }
 
@@ -471,6 +552,7 @@ FAMILY_BY_ARCH = {
     "Qwen3NextForCausalLM": "hybrid_linear",
     "Bedovik": "bedovik",
     "Tudilix": "tudilix",
+    "Vozetar": "vozetar",
 }
 
 
@@ -564,6 +646,66 @@ def _tudilix_config(cfg: dict) -> ModelSpec:
                      logit_softcap=float(cfg.get("logit_softcap") or 0.0))
 
 
+def _vozetar_attention(i: int, m: dict, **kw) -> AttentionSpec:
+    rot, mask = m.get("rot") or {"dims": 0, "base": 1e4}, m.get("mask") or {}
+    a = AttentionSpec(kind="conv_gqa", n_heads=int(m["heads"]), n_kv_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]), scale=float(m["scale"]),
+                      window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0), conv_taps=int(m.get("conv") or 1), rope_dims=int(rot["dims"]),
+                      rope_theta=float(rot["base"]), **kw)
+    if a.n_heads % a.n_kv_heads:
+        raise ValueError(f"layer {i}: {a.n_heads} query heads over {a.n_kv_heads} key heads")
+    if a.rope_dims % 2 or a.rope_dims > a.head_dim:
+        raise ValueError(f"layer {i}: {a.rope_dims} rotated dimensions of {a.head_dim}")
+    if a.values_are_keys and a.v_head_dim != a.head_dim:
+        raise ValueError(f"layer {i}: values are the keys, but {a.v_head_dim} is not {a.head_dim}")
+    return a
+
+
+def _vozetar_config(cfg: dict) -> ModelSpec:
+    """`config.json` of the Vozetar design: every layer names its mixer (attention, or attention beside a linear one) and its feed-forward with
+    their sizes."""
+    blocks = []
+    for i, layer in enumerate(cfg["layers"]):
+        m, mlp, kind = layer["mixer"], layer.get("mlp"), layer["type"]
+        rec, moe, ffn, scales = None, None, None, (1.0, 1.0)
+        if kind == "attention":
+            attn = _vozetar_attention(i, m, rope_interleaved=False, qkv_bias=True, out_bias=True, sink=True, out_gate=True, gate_values=True)
+        elif kind == "parallel":
+            attn = _vozetar_attention(i, m["left"], qkv_bias=True, sink=True)
+            r = m["right"]
+            rot = r.get("rot") or {"dims": 0, "base": 1e4}
+            rec = RecurrentSpec(kind="retention", heads=int(r["heads"]), dim=int(r["dim"]), vdim=int(r["vdim"]), decay=tuple(float(x) for x in r["decay"]), rope_dims=int(rot["dims"]),
+                                rope_theta=float(rot["base"]))
+            if len(rec.decay) != rec.heads or rec.rope_dims % 2 or rec.rope_dims > rec.dim:
+                raise ValueError(f"layer {i}: {len(rec.decay)} decays of {rec.heads} heads, {rec.rope_dims} rotated dimensions of {rec.dim}")
+            scales = (float(m["left_scale"]), float(m["right_scale"]))
+        elif kind == "parallel_2":
+            attn = _vozetar_attention(i, m["left"], values_are_keys=True, qk_norm_whole=True, out_gate=True)
+            r = m["right"]
+            rec = RecurrentSpec(kind="gla", heads=int(r["heads"]), dim=int(r["dim"]), vdim=int(r["vdim"]), tau=float(r["tau"]))
+            scales = (0.5, 0.5)
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+        if mlp is not None and mlp["kind"] == "dense":
+            ffn = DenseFfnSpec(int(mlp["ff"]), activation="silu_glu")
+        elif mlp is not None and mlp["kind"] == "moe":
+            r, shared = mlp["router"], mlp.get("shared")
+            groups = r.get("groups") or {"count": 1, "keep": 1}
+            moe = MoESpec(n_experts=int(r["experts"]), top_k=int(r["top"]), intermediate=int(mlp["expert"]["ff"]), n_shared=1 if shared else 0,
+                          shared_intermediate=int(shared["ff"]) if shared else 0, scoring="sigmoid", normalize=False, n_group=int(groups["count"]), topk_group=int(groups["keep"]))
+            if moe.n_experts % moe.n_group or not 1 <= moe.topk_group <= moe.n_group or moe.top_k > moe.n_experts // moe.n_group * moe.topk_group:
+                raise ValueError(f"layer {i}: {moe.n_experts} experts in {moe.n_group} groups, {moe.topk_group} kept, top {moe.top_k}: not a routing")
+        elif mlp is not None:
+            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        blocks.append(BlockSpec(attn, moe, rec, ffn, scales, kind == "parallel_2"))
+    pairs = (cfg.get("embedding") or {}).get("bigram")
+    streams = int(cfg["streams"])
+    if streams < 1:
+        raise ValueError(f"{streams} residual streams")
+    return ModelSpec(name="vozetar", family="vozetar", vocab=int(cfg["vocab"]), hidden=int(cfg["width"]), n_layers=len(blocks), rms_eps=float(cfg["norm"]["eps"]),
+                     attn=blocks[0].attn, moe=next((b.moe for b in blocks if b.moe is not None), MoESpec(n_experts=0, n_shared=0)), quant=QuantSpec(), blocks=tuple(blocks),
+                     streams=streams, pair_table=PairTableSpec(int(pairs["buckets"]), int(pairs["mul_prev"]), int(pairs["mul_cur"])) if pairs else None)
+
+
 def from_hf_config(cfg: dict | str | Path) -> ModelSpec:
     """Build a ModelSpec from a Hugging Face `config.json` (dict or path)."""
     if not isinstance(cfg, dict):
@@ -578,6 +720,8 @@ def from_hf_config(cfg: dict | str | Path) -> ModelSpec:
         return _bedovik_config(cfg)
     if family == "tudilix":
         return _tudilix_config(cfg)
+    if family == "vozetar":
+        return _vozetar_config(cfg)
     hidden = cfg["hidden_size"]
     heads = cfg["num_attention_heads"]
     if "kv_lora_rank" in cfg:
@@ -649,13 +793,16 @@ def spec_from_json(d: dict) -> ModelSpec:
 
     def block(b: dict) -> BlockSpec:
         part = lambda key, make: make(b[key]) if b.get(key) else None
-        return BlockSpec(part("attn", attn), part("moe", lambda m: MoESpec(**m)), part("rec", lambda r: RecurrentSpec(**r)), part("ffn", lambda f: DenseFfnSpec(**f)))
+        return BlockSpec(part("attn", attn), part("moe", lambda m: MoESpec(**m)), part("rec", lambda r: RecurrentSpec(**dict(r, decay=tuple(r.get("decay") or ())))),
+                         part("ffn", lambda f: DenseFfnSpec(**f)), tuple(b.get("merge_scales") or (1.0, 1.0)), bool(b.get("merge_norm")))
 
     if d.get("blocks"):
         d["blocks"] = tuple(block(b) for b in d["blocks"])
     d["blocks"] = tuple(d.get("blocks") or ())
     if d.get("loop"):
         d["loop"] = LoopSpec(**d["loop"])
+    if d.get("pair_table"):
+        d["pair_table"] = PairTableSpec(**d["pair_table"])
     return ModelSpec(attn=attn(d.pop("attn")), moe=MoESpec(**d.pop("moe")), quant=QuantSpec(**d.pop("quant")), **d)
 
 

@@ -25,6 +25,7 @@
 
 #define CA_PDL_CLASS 2
 #include "common.cuh"
+#include "attn_extras.cuh"
 
 #define PF_KT 128                 // keys per tile
 #define PF_NS 2                   // K stages
@@ -372,7 +373,7 @@ struct GqaPrefillArgs {
   const bf16* q;
   const CUtensorMap* k_map; const CUtensorMap* v_map;      // the decode kernel's descriptors; value head h at coordinate v_head0 + h
   const int* page_table; const int* kv_len; const int* q_start; const int* q_len;
-  const float* sink;
+  AttnExtras<bf16> x;                                      // sink, kept first keys, output gate
   bf16* out;
   int* status;
   int q_stride, Hq, Hkv, max_pages, window, max_q_tiles;
@@ -413,7 +414,9 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
   const int hi = bidir ? kvlen : first_pos + ntok;
   const int lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
   const int tile0 = lo / PF_KT;
-  const int n_tiles = max(0, (hi + PF_KT - 1) / PF_KT - tile0);
+  // tiles of kept first keys in front of the window, then the window's
+  const int kept = a.x.kept_tiles(tile0, PF_KT), n_tiles = kept + max(0, (hi + PF_KT - 1) / PF_KT - tile0);
+  auto tile_at = [&](int i) { return i < kept ? i : i - kept + tile0; };
 
   if (tid == 0) {
     for (int s = 0; s < 2; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
@@ -463,7 +466,7 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       const int s = i % PF_NS, ph = ((i / PF_NS) & 1) ^ 1;
       if (!mbar_wait_bounded(&k_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); return false; }
       if (lane == 0) {
-        const int key0 = (tile0 + i) * PF_KT;
+        const int key0 = tile_at(i) * PF_KT;
         mbar_expect_tx(&k_full[s], Cf::K_STAGE);
 #pragma unroll
         for (int p = 0; p < 2; ++p) {
@@ -481,7 +484,7 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       const int sv = i % Cf::NSV, phv = ((i / Cf::NSV) & 1) ^ 1;
       if (!mbar_wait_bounded(&v_empty[sv], phv, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, 0x1000 + i); break; }
       if (lane == 0) {
-        const int key0 = (tile0 + i) * PF_KT;
+        const int key0 = tile_at(i) * PF_KT;
         mbar_expect_tx(&v_full[sv], Cf::V_STAGE);
 #pragma unroll
         for (int p = 0; p < 2; ++p) {
@@ -546,9 +549,9 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       if (!mbar_wait_bounded(&s_full[i & 1], (i >> 1) & 1, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_EPILOGUE, i); ok = false; break; }
       tc_fence_after();
       const uint32_t s_addr = tmem + lane_addr + ((i & 1) ? S1_COL : S0_COL);
-      const int key0 = (tile0 + i) * PF_KT;
+      const int key0 = tile_at(i) * PF_KT;
       // CTA-uniform: every key of the tile is visible to every live row (below the diagonal and inside every row's window)
-      const bool all_visible = key0 + PF_KT - 1 <= first_pos && (a.window <= 0 || key0 > first_pos + ntok - 1 - a.window);
+      const bool all_visible = key0 + PF_KT - 1 <= first_pos && (a.window <= 0 || key0 > first_pos + ntok - 1 - a.window || key0 + PF_KT <= a.x.keep_first);
       // two passes over the tile's 128 score columns: row maximum, then exponentials packed to bf16 pairs (64 registers).
       // Tiles below the diagonal need no mask (CTA-uniform test), which is all but the last one or two of a long context.
       float mx = -INFINITY;
@@ -594,7 +597,7 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const int kp = key0 + c * 32 + j;
-            if (live && kp <= qpos && kp > wlo) mx = fmaxf(mx, __uint_as_float(sr[j]) * sc2);
+            if (live && kp <= qpos && (kp > wlo || kp < a.x.keep_first)) mx = fmaxf(mx, __uint_as_float(sr[j]) * sc2);
           }
         }
         if (mx > m_ref + 8.f) {
@@ -610,8 +613,8 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int kp = key0 + c * 32 + 2 * j;
-            const float e0 = (live && kp <= qpos && kp > wlo) ? exp2f(fmaf(__uint_as_float(sr[2 * j]), sc2, -m_ref)) : 0.f;
-            const float e1 = (live && kp + 1 <= qpos && kp + 1 > wlo) ? exp2f(fmaf(__uint_as_float(sr[2 * j + 1]), sc2, -m_ref)) : 0.f;
+            const float e0 = (live && kp <= qpos && (kp > wlo || kp < a.x.keep_first)) ? exp2f(fmaf(__uint_as_float(sr[2 * j]), sc2, -m_ref)) : 0.f;
+            const float e1 = (live && kp + 1 <= qpos && (kp + 1 > wlo || kp + 1 < a.x.keep_first)) ? exp2f(fmaf(__uint_as_float(sr[2 * j + 1]), sc2, -m_ref)) : 0.f;
             psum += e0 + e1;
             bf162 h = __floats2bfloat162_rn(e0, e1);
             pk[c * 16 + j] = *(uint32_t*)&h;
@@ -650,13 +653,14 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       const int rr = live ? r : 0;
       const int t = row_base + rr / G, h = kvh * G + rr % G;
       float scale_o = 1.f, lt = l;
-      if (a.sink) {                                     // learned sink logit: one more softmax term with a zero value
+      if (a.x.sink) {                                   // learned sink logit: one more softmax term with a zero value
         const float m_nat = (m_ref == -INFINITY) ? -INFINITY : m_ref * 0.6931471805599453f;
-        const float sk = a.sink[h], m2 = fmaxf(m_nat, sk);
+        const float sk = a.x.sink[h], m2 = fmaxf(m_nat, sk);
         const float e1 = (m_nat == -INFINITY) ? 0.f : __expf(m_nat - m2);
         lt = l * e1 + __expf(sk - m2); scale_o = e1;
       }
-      const float inv = lt > 0.f ? scale_o / lt : 0.f;
+      const float inv = (lt > 0.f ? scale_o / lt : 0.f) * a.x.head_factor(t, h);
+      const bool gated = a.x.gate && a.x.gate_values;
       bf16* dst = a.out + (size_t)t * a.ldo + (size_t)h * a.dv;
       const bool vec = ((a.dv | a.ldo) & 7) == 0;
 #pragma unroll 1
@@ -668,6 +672,11 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
           for (int j = 0; j < 16; ++j) o[j] = 0;
         }
         if (!live) continue;
+        if (gated) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            if (c * 16 + j < a.dv) o[j] = __float_as_uint(__uint_as_float(o[j]) * a.x.value_factor(t, h * a.dv + c * 16 + j));
+        }
         uint32_t w[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) { bf162 hh = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * inv, __uint_as_float(o[2 * j + 1]) * inv); w[j] = *(uint32_t*)&hh; }
@@ -711,7 +720,7 @@ extern "C" int cuteafd_gqa_prefill_attention(const void* q, const void* kv_map, 
   if (T <= 0 || n_seq <= 0) return CA_OK;
   GqaPrefillArgs a;
   a.q = (const bf16*)q; a.k_map = a.v_map = (const CUtensorMap*)kv_map; a.v_head0 = Hkv; a.dv = 128; a.ldo = Hq * 128; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len;
-  a.sink = sink; a.out = (bf16*)out; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.window = window;
+  a.x = attn_extras<bf16>(nullptr, 0); a.x.sink = sink; a.out = (bf16*)out; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.window = window;
   a.scale = scale;
   const int tpt = 128 / (Hq / Hkv);
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
@@ -722,14 +731,15 @@ extern "C" int cuteafd_gqa_prefill_attention(const void* q, const void* kv_map, 
 // of at most 512 fit tensor memory.
 extern "C" int cuteafd_window_prefill_attention(const void* q, const void* maps, const int* page_table, const int* kv_len, const int* q_start, const int* q_len, void* out,
                                                 int T, int n_seq, int max_q_len, int q_stride, int Hq, int Hkv, int dk_pad, int dv_pad, int dv, int ldo, int max_pages,
-                                                int window, float scale, int* status, cudaStream_t s) {
+                                                int window, float scale, const CaAttnExtras* extras, int* status, cudaStream_t s) {
   CA_REQUIRE(q && maps && page_table && kv_len && q_start && q_len && out, "window_prefill_attention: null argument");
   CA_REQUIRE(Hkv >= 1 && Hq % Hkv == 0 && Hq / Hkv <= 128 && q_stride % 8 == 0, "window_prefill_attention: group size %d unsupported", Hkv ? Hq / Hkv : 0);
   CA_REQUIRE(dv >= 1 && dv <= dv_pad && ldo >= Hq * dv && window >= 0 && q_stride >= Hq * dk_pad, "window_prefill_attention: bad shape");
+  CA_REQUIRE(!extras || !extras->gate || extras->ldg >= (extras->gate_values ? Hq * dv : Hq), "window_prefill_attention: gate rows too short");
   if (T <= 0 || n_seq <= 0) return CA_OK;
   GqaPrefillArgs a = {};
   a.q = (const bf16*)q; a.k_map = (const CUtensorMap*)maps; a.v_map = a.k_map + 1; a.v_head0 = 0; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
-  a.q_len = q_len; a.sink = nullptr; a.out = (bf16*)out; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.window = window;
+  a.q_len = q_len; a.x = attn_extras<bf16>(extras, window); a.out = (bf16*)out; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.window = window;
   a.scale = scale; a.dv = dv; a.ldo = ldo;
   const int tpt = 128 / (Hq / Hkv);
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;

@@ -22,6 +22,7 @@
 #define CA_PDL_CLASS 2
 #include "common.cuh"
 #include "attn_common.cuh"
+#include "attn_extras.cuh"
 
 #define APAGE 64
 #define AD 128
@@ -35,7 +36,7 @@ struct AttnTcArgs {
   const int* kv_len;
   const int* q_start;
   const int* q_len;
-  const float* sink;
+  AttnExtras<bf16> x;           // sink, kept first keys, output gate
   bf16* out;
   float* part_o;
   float* part_ml;
@@ -110,9 +111,12 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
   const int hi = first_pos + ntok;                      // keys [lo, hi) can be visible
   const int lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
   const int first_page = lo / APAGE, last_page = (hi + APAGE - 1) / APAGE;
-  const int per = (last_page - first_page + a.n_splits - 1) / a.n_splits;
-  const int p0 = first_page + split * per, p1 = min(last_page, p0 + per);
+  // the pages that count: those of kept first keys in front of the window, then the window's; a split takes a run of them
+  const int kept = a.x.kept_tiles(first_page, APAGE), n_pages = kept + last_page - first_page;
+  const int per = (n_pages + a.n_splits - 1) / a.n_splits;
+  const int p0 = split * per, p1 = min(n_pages, p0 + per);
   const int n_tiles = max(0, p1 - p0);
+  auto page_at = [&](int i) { const int j = p0 + i; return j < kept ? j : j - kept + first_page; };
 
   // Decode-shaped tiles (<= 32 real rows) replicate the rows into every 32-lane quarter of the MMA tile so that
   // the four softmax warps each take 16 of the 64 score columns of the SAME rows (4x shorter per-tile chain).
@@ -151,7 +155,7 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
     const uint64_t kvpol = a.max_q_tiles == 1 ? l2_policy_stream() : l2_policy_normal();
     for (int i = 0; i < n_tiles && !*abortp; ++i) {
       const int s = i & 1, ph = ((i >> 1) & 1) ^ 1;
-      const int page = a.page_table[(size_t)seq * a.max_pages + p0 + i];
+      const int page = a.page_table[(size_t)seq * a.max_pages + page_at(i)];
       if (!mbar_wait_bounded(&k_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); break; }
       if (lane == 0) {
         mbar_expect_tx(&k_full[s], Cf::K_STAGE);
@@ -229,12 +233,12 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
         uint32_t sr[16];
         tmem_ld_x16(tmem + lane_addr + ((i & 1) ? S1_COL : S0_COL) + col0, sr);
         tc_wait_ld();
-        const int key0 = (p0 + i) * APAGE + col0;
+        const int key0 = page_at(i) * APAGE + col0;
         float mx = -INFINITY;
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           const int kp = key0 + j;
-          const bool vis = rlive && kp <= rq && kp < kvlen && (a.window <= 0 || kp > rq - a.window);
+          const bool vis = rlive && kp <= rq && kp < kvlen && (a.window <= 0 || kp > rq - a.window || kp < a.x.keep_first);
           const float v = vis ? __uint_as_float(sr[j]) * sc2 : -INFINITY;
           sr[j] = __float_as_uint(v);
           mx = fmaxf(mx, v);
@@ -293,12 +297,12 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld_x16(tmem + lane_addr + ((i & 1) ? S1_COL : S0_COL) + c * 16, sr + c * 16);
       tc_wait_ld();
-      const int key0 = (p0 + i) * APAGE;
+      const int key0 = page_at(i) * APAGE;
       float mx = -INFINITY;
 #pragma unroll
       for (int j = 0; j < 64; ++j) {
         const int kp = key0 + j;
-        const bool vis = live && kp <= qpos && kp < kvlen && (a.window <= 0 || kp > qpos - a.window);
+        const bool vis = live && kp <= qpos && kp < kvlen && (a.window <= 0 || kp > qpos - a.window || kp < a.x.keep_first);
         const float v = vis ? __uint_as_float(sr[j]) * sc2 : -INFINITY;
         sr[j] = __float_as_uint(v);
         mx = fmaxf(mx, v);
@@ -353,12 +357,13 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
       const int t = row_base + rr / G, h = kvh * G + rr % G;
       const float m_nat = (m_ref == -INFINITY) ? -INFINITY : m_ref * 0.6931471805599453f;
       float scale_o = 1.f, lt = l;
-      if (a.n_splits == 1 && a.sink) {
-        const float sk = a.sink[h], m2 = fmaxf(m_nat, sk);
+      if (a.n_splits == 1 && a.x.sink) {
+        const float sk = a.x.sink[h], m2 = fmaxf(m_nat, sk);
         const float e1 = (m_nat == -INFINITY) ? 0.f : __expf(m_nat - m2);
         lt = l * e1 + __expf(sk - m2); scale_o = e1;
       }
-      const float inv = lt > 0.f ? scale_o / lt : 0.f;
+      const float inv = (lt > 0.f ? scale_o / lt : 0.f) * (a.n_splits == 1 ? a.x.head_factor(t, h) : 1.f);      // splits: the merge applies it
+      const bool gated = a.x.gate && a.x.gate_values;
       bf16* dst = a.out + (size_t)t * a.ldo + (size_t)h * a.dv;
       const bool vec = ((a.dv | a.ldo) & 7) == 0;      // otherwise heads do not start on 16 bytes
       float* po = a.n_splits > 1 ? a.part_o + (((size_t)split * a.T + t) * a.Hq + h) * (VC * 64) : nullptr;
@@ -372,6 +377,11 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
         }
         if (!live) continue;
         if (a.n_splits == 1) {
+          if (gated) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              if (c * 16 + j < a.dv) o[j] = __float_as_uint(__uint_as_float(o[j]) * a.x.value_factor(t, h * a.dv + c * 16 + j));
+          }
           uint32_t w[8];
 #pragma unroll
           for (int j = 0; j < 8; ++j) { bf162 hh = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * inv, __uint_as_float(o[2 * j + 1]) * inv); w[j] = *(uint32_t*)&hh; }
@@ -398,6 +408,12 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
   tc_fence_before();
   __syncthreads();
   if (warp == 1) tmem_dealloc(tmem, Cf::TMEM_COLS);
+}
+
+static AttnExtras<bf16> sink_only(const float* sink) {
+  AttnExtras<bf16> x = attn_extras<bf16>(nullptr, 0);
+  x.sink = sink;
+  return x;
 }
 
 template <int KC, int VC>
@@ -431,7 +447,7 @@ extern "C" int cuteafd_attn_merge(const float* part_o, const float* part_ml, con
                                   cudaStream_t s) {
   CA_REQUIRE(part_o && part_ml && out && n_parts >= 1, "attn_merge: needs partials");
   if (T <= 0) return CA_OK;
-  CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * AD / 8 + 127) / 128), 128, 0, s, part_o, part_ml, sink, (bf16*)out, T, Hq, (int)AD, (int)AD, Hq * AD, n_parts,
+  CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * AD / 8 + 127) / 128), 128, 0, s, part_o, part_ml, sink_only(sink), (bf16*)out, T, Hq, (int)AD, (int)AD, Hq * AD, n_parts,
                 (uint8_t*)nullptr, (uint8_t*)nullptr, 0, (const float*)nullptr, 0);
   CA_CHECK_LAUNCH("attn_merge");
   return CA_OK;
@@ -454,14 +470,14 @@ extern "C" int cuteafd_paged_attention_tc(const void* q, const void* kv_map, con
   if (T <= 0 || n_seq <= 0) return CA_OK;
   AttnTcArgs a;
   a.q = (const bf16*)q; a.k_map = a.v_map = (const CUtensorMap*)kv_map; a.v_head0 = Hkv; a.dv = AD; a.ldo = Hq * AD; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
-  a.q_len = q_len; a.sink = sink; a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.status = status;
+  a.q_len = q_len; a.x = sink_only(sink); a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.status = status;
   a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv; a.max_pages = max_pages; a.n_splits = n_splits; a.window = window; a.T = T; a.scale = scale;
   const int tpt = 128 / (Hq / Hkv);
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
   const int rc = launch_attn_tc<2, 2>(a, n_seq, s);
   if (rc != CA_OK) return rc;
   if (n_splits > 1 && !partials_only) {
-    CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * AD / 8 + 127) / 128), 128, 0, s, part_o, part_ml, sink, (bf16*)out, T, Hq, (int)AD, (int)AD, Hq * AD, n_splits,
+    CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * AD / 8 + 127) / 128), 128, 0, s, part_o, part_ml, sink_only(sink), (bf16*)out, T, Hq, (int)AD, (int)AD, Hq * AD, n_splits,
                   (uint8_t*)q_out, (uint8_t*)sf_out, ldsf, inv_gs, qkind);
     CA_CHECK_LAUNCH("attn_merge");
   }
@@ -485,15 +501,16 @@ extern "C" int cuteafd_tmap_encode_kv(void* out128, const void* base, int Hkv, u
 // (`cuteafd_tmap_encode_heads`), 128 bytes each.
 extern "C" int cuteafd_window_attention(const void* q, const void* maps, const int* page_table, const int* kv_len, const int* q_start, const int* q_len, void* out,
                                         float* part_o, float* part_ml, int T, int n_seq, int max_q_len, int q_stride, int Hq, int Hkv, int dk_pad, int dv_pad, int dv,
-                                        int ldo, int max_pages, int n_splits, int window, float scale, int* status, cudaStream_t s) {
+                                        int ldo, int max_pages, int n_splits, int window, float scale, const CaAttnExtras* extras, int* status, cudaStream_t s) {
   CA_REQUIRE(q && maps && page_table && kv_len && q_start && q_len && out, "window_attention: null argument");
   CA_REQUIRE(Hkv >= 1 && Hq % Hkv == 0 && Hq / Hkv <= 128 && q_stride % 8 == 0, "window_attention: group size %d unsupported", Hkv ? Hq / Hkv : 0);
   CA_REQUIRE(dv >= 1 && dv <= dv_pad && ldo >= Hq * dv && window >= 0 && q_stride >= Hq * dk_pad, "window_attention: bad shape");
   CA_REQUIRE(n_splits >= 1 && (n_splits == 1 || (part_o && part_ml)), "window_attention: split-KV needs scratch");
+  CA_REQUIRE(!extras || !extras->gate || extras->ldg >= (extras->gate_values ? Hq * dv : Hq), "window_attention: gate rows too short");
   if (T <= 0 || n_seq <= 0) return CA_OK;
   AttnTcArgs a = {};
   a.q = (const bf16*)q; a.k_map = (const CUtensorMap*)maps; a.v_map = a.k_map + 1; a.v_head0 = 0; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
-  a.q_len = q_len; a.sink = nullptr; a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv;
+  a.q_len = q_len; a.x = attn_extras<bf16>(extras, window); a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.status = status; a.q_stride = q_stride; a.Hq = Hq; a.Hkv = Hkv;
   a.max_pages = max_pages; a.n_splits = n_splits; a.window = window; a.T = T; a.scale = scale; a.dv = dv; a.ldo = ldo;
   const int tpt = 128 / (Hq / Hkv);
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
@@ -504,7 +521,7 @@ extern "C" int cuteafd_window_attention(const void* q, const void* maps, const i
   if (rc == CA_ERR_UNSUPPORTED) return ca_fail(rc, "window_attention: head widths %d / %d (64, 128, 192 or 256)", dk_pad, dv_pad);
   if (rc != CA_OK) return rc;
   if (n_splits > 1) {
-    CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * dv_pad / 8 + 127) / 128), 128, 0, s, part_o, part_ml, (const float*)nullptr, (bf16*)out, T, Hq, dv_pad, dv, ldo, n_splits,
+    CA_LAUNCH_PDL(attn_merge8_kernel, dim3(T, (Hq * dv_pad / 8 + 127) / 128), 128, 0, s, part_o, part_ml, a.x, (bf16*)out, T, Hq, dv_pad, dv, ldo, n_splits,
                   (uint8_t*)nullptr, (uint8_t*)nullptr, 0, (const float*)nullptr, 0);
     CA_CHECK_LAUNCH("attn_merge");
   }

@@ -1,6 +1,7 @@
 // Split-KV partial merge shared by the SIMT and the tensor-core paged attention kernels.
 #pragma once
 #include "common.cuh"
+#include "attn_extras.cuh"
 
 // Merge split partials: out = sum_s o_s * exp(m_s - M) / sum_s l_s * exp(m_s - M)  (+ sink term).
 // Splits that saw no key carry m = -inf, l = 0 and drop out.  Partials of rows a split never touched are
@@ -28,7 +29,7 @@ static __global__ void attn_merge_kernel(const float* __restrict__ part_o, const
 
 // Same merge, eight output elements per thread (the first Dout of a head's D columns, head h at column h * Dout of rows ldo apart), optionally also writing the merged row quantised to FP4 for the
 // output projection that follows (qkind 1 NVFP4 / 2 MXFP4; needs Hq * D % 256 == 0).  grid (T, ceil(Hq * D / 8 / 128)).
-static __global__ void attn_merge8_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ sink,
+static __global__ void attn_merge8_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const AttnExtras<bf16> x,
                                           bf16* __restrict__ out, int T, int Hq, int D, int Dout, int ldo, int n_splits, uint8_t* __restrict__ q,
                                           uint8_t* __restrict__ sf, int ldsf, const float* __restrict__ inv_gs_ptr, int qkind) {
   pdl_launch(); pdl_wait();
@@ -38,7 +39,7 @@ static __global__ void attn_merge8_kernel(const float* __restrict__ part_o, cons
   // Up to eight splits at a time, every load issued before the first use: the (m, l) pairs and the partial rows of all splits are
   // in flight together (a loop that reads m, branches, then loads the row is one L2 round trip per split on a decode step's
   // critical path).  Partial rows of empty splits (m = -inf) are loaded but not used; the buffers always cover every split.
-  const float sk = sink ? sink[h] : -INFINITY;
+  const float sk = x.sink ? x.sink[h] : -INFINITY;
   float M = sk, L = 0.f;
   float o[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
   for (int s0 = 0; s0 < n_splits; s0 += 8) {
@@ -55,7 +56,7 @@ static __global__ void attn_merge8_kernel(const float* __restrict__ part_o, cons
 #pragma unroll
     for (int j = 0; j < 8; ++j) if (s0 + j < n_splits) Mn = fmaxf(Mn, ml[j].x);
     if (s0 == 0) {
-      if (sink) L = __expf(sk - Mn);                  // the sink's share first, as the one-pass form adds it
+      if (x.sink) L = __expf(sk - Mn);                  // the sink's share first, as the one-pass form adds it
     } else if (Mn != M && M != -INFINITY) {           // a later batch raised the maximum: rescale what was accumulated
       const float r = __expf(M - Mn);
       L *= r;
@@ -74,8 +75,12 @@ static __global__ void attn_merge8_kernel(const float* __restrict__ part_o, cons
     }
   }
 
-  const float inv = L > 0.f ? 1.f / L : 0.f;
+  const float inv = (L > 0.f ? 1.f / L : 0.f) * x.head_factor(t, h);
   bf16 ob[8];
+  if (x.gate && x.gate_values) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) if (d0 + j < Dout) o[j] *= x.value_factor(t, h * Dout + d0 + j);
+  }
 #pragma unroll
   for (int j = 0; j < 8; ++j) ob[j] = __float2bfloat16(o[j] * inv);
   bf16* dst = out + (size_t)t * ldo + (size_t)h * Dout + d0;

@@ -2,16 +2,19 @@
 //   norm_rows        embedding, residual += mult * norm(sub-layer output + bias), or a gather of rows - each also leaves the next product's
 //                    normalised operand row
 //   rope_table       cosine / sine of the step's positions, once per rotation
-//   conv_qkv         projected queries, keys and values -> short causal convolution -> head norm -> rotation -> query rows, paged cache
+//   conv_qkv         projected queries, keys and values (+ bias) -> short causal convolution -> norm (per head, over the whole projection, or
+//                    none) -> rotation (neighbouring or half-apart pairs) -> query rows, paged cache; values may be the keys in front of the norm
 //   rglru_conv       x branch -> short causal convolution -> block-major operand of the gate product (and its tile table)
 //   lru_scan         the real-gated linear recurrence: one pass over short runs, chunk aggregates + carried rescan over long ones
 //   glu_rows         clamped GLU over two projected rows (all-fp32 mode; bf16 products do it in their epilogue)
-//   window_attn_simt paged grouped-query attention on the ordinary cores (fp32, and shapes the tcgen05 kernels do not take)
+//   window_attn_simt paged grouped-query attention on the ordinary cores (fp32, and shapes the tcgen05 kernels do not take): windows with kept
+//                    first keys, sinks, output gates
 // Everything a sequence carries from step to step is addressed by absolute position: convolution inputs live in a ring of
 // taps - 1 + depth rows, recurrent states in a ring of depth + 1, so a step that is repeated, or the last `depth` tokens that are taken back
 // (rejected drafts), need no restore - later positions overwrite them.  T is the operand type: bf16, or float for the all-fp32 mode.
 // (No counterpart in the reference, which has no such family; the recurrence's kernel is the sibling of linear_attn.cu.)
 #include "stack_rows.cuh"
+#include "attn_extras.cuh"
 
 #define HS_TILE 16          // tokens of a sequence one block of the convolution kernels walks (at least taps - 1)
 #define HS_MAX_TAPS 16
@@ -120,17 +123,20 @@ __global__ void rope_table_kernel(const int* __restrict__ positions, const float
 }
 
 // ---------------------------------------------------------------- short convolution in front of attention
+enum { QK_NORM_NONE = 0, QK_NORM_HEAD = 1, QK_NORM_WHOLE = 2 };
+
 template <typename T>
 struct ConvQkv {
-  const T* proj; int ldp;                       // [T, ldp]: H * dim queries | G * dim keys | G * vdim values
-  const float* w;                               // [taps, C]
-  const float* q_norm; const float* k_norm;     // gains of the head norms
+  const T* proj; int ldp;                       // [T, ldp]: H * dim queries | G * dim keys | G * vdim values (none with v_from_k)
+  const float* w;                               // [taps, C]; null with one tap: no convolution
+  const float* bias;                            // [C] of the projection, or null
+  const float* q_norm; const float* k_norm;     // gains: [dim] of the head norms, [H * dim] and [G * dim] of the whole ones
   const float2* rope;                           // [T, pairs]
-  T* ring;                                      // [slots, R, C] projected rows by position
+  T* ring;                                      // [slots, R, C] projected rows (without bias) by position; null with one tap
   const int* state_slot; const int* q_start; const int* q_len; const int* kv_len; const int* slot_map;
   T* q; int q_stride;                           // [T, H * dp]
   T* cache; int row_stride, n_slots;            // paged rows: G * dp keys, then G * dvp values
-  int H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state;
+  int H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state, norm, v_from_k;
   float eps; int* status;
 };
 
@@ -182,55 +188,65 @@ template <typename T, int V> __device__ __forceinline__ void store_n(T* p, int n
   for (int k = 0; k < V; ++k) if (k < n) p[k] = to_t<T>(v[k]);
 }
 
-// One warp per (head, tile of HS_TILE tokens); a lane owns V neighbouring dimensions of the head (whole rotated pairs).  TAPS > 0: the last
-// inputs and the weights stay in registers; 0: any number of taps, inputs re-read.
-template <typename T, int V, int TAPS>
-__global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvQkv<T> a) {
-  pdl_launch(); pdl_wait();
-  const int lane = threadIdx.x & 31, unit = blockIdx.x * 4 + (threadIdx.x >> 5), seq = blockIdx.z;
-  const int n = a.q_len[seq], i0 = blockIdx.y * HS_TILE;
-  if (unit >= a.H + 2 * a.G || i0 >= n) return;
-  const int row0 = a.q_start[seq], p0 = a.kv_len[seq] - n, slot = a.state_slot[seq], i1 = min(n, i0 + HS_TILE);
-  if (slot < 0 || slot >= a.n_state) { if (lane == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6E1); return; }
+// One warp takes one head of a tile of HS_TILE tokens; a lane owns V neighbouring dimensions of the head (whole rotated pairs when neighbours
+// turn together; with HALF the partner is half a rotation away and comes through `xch`).  TAPS > 0: the last inputs and the weights stay in
+// registers; 0: any number of taps, inputs re-read.  STATS: only the sums of squares of the tile's rows, left in stats[i - i0]; otherwise
+// `inv` holds the tile's factors of a norm over the whole projection (null: the norm is per head, or there is none).
+template <typename T, int V, int TAPS, bool HALF, bool STATS>
+__device__ __forceinline__ void conv_qkv_tile(const ConvQkv<T>& a, int unit, int seq, int i0, int i1, int slot, float* xch, float* stats, const float* inv) {
+  const int lane = threadIdx.x & 31, n = a.q_len[seq], row0 = a.q_start[seq], p0 = a.kv_len[seq] - n;
   const bool is_q = unit < a.H, is_v = unit >= a.H + a.G;
   const int d = is_v ? a.vdim : a.dim, head = is_q ? unit : (is_v ? unit - a.H - a.G : unit - a.H), e = lane * V;
   const int ch = (is_v ? (a.H + a.G) * a.dim + head * a.vdim : unit * a.dim) + e;
   const int taps = TAPS ? TAPS : a.taps, own = max(0, min(V, d - e));      // dimensions of this lane
   const bool vec = own == V && ch % V == 0 && a.ldp % V == 0, wvec = own == V && ch % V == 0 && a.C % V == 0;
-  T* ring = a.ring + (size_t)slot * a.R * a.C + ch;
+  T* ring = a.ring ? a.ring + (size_t)slot * a.R * a.C + ch : nullptr;
+  float bias[V];
+#pragma unroll
+  for (int k = 0; k < V; ++k) bias[k] = a.bias && k < own ? a.bias[ch + k] : 0.f;
   // input row i of this run (i < 0: what the sequence fed before, nothing in front of its start)
   auto fresh = [&](int i, float* v) { load_n<T, V>(a.proj + (size_t)(row0 + i) * a.ldp + ch, own, vec, v); };
   auto input = [&](int i, float* v) {
     const int pos = p0 + i;
     if (i >= 0) fresh(i, v);
     else load_n<T, V>(ring + (size_t)((pos + a.R) % a.R) * a.C, pos < 0 ? 0 : own, pos >= 0 && wvec, v);
+    if (pos >= 0)
+#pragma unroll
+      for (int k = 0; k < V; ++k) v[k] += bias[k];
   };
   auto weight = [&](int j, float* v) { load_n<float, V>(a.w + (size_t)j * a.C + ch, own, wvec, v); };
   constexpr int NH = TAPS > 1 ? TAPS - 1 : 1, NW = TAPS ? TAPS : 1;
   float hist[NH][V], wr[NW][V], gain[V];
-  const float* norm = is_q ? a.q_norm : a.k_norm;
+  const float* norm = (is_q ? a.q_norm : a.k_norm) + (a.norm == QK_NORM_WHOLE ? head * a.dim : 0);
 #pragma unroll
-  for (int k = 0; k < V; ++k) gain[k] = is_v ? 1.f : (k < own ? norm[e + k] : 0.f);
+  for (int k = 0; k < V; ++k) gain[k] = is_v || a.norm == QK_NORM_NONE ? 1.f : (k < own ? norm[e + k] : 0.f);
   if (TAPS) {
 #pragma unroll
-    for (int j = 0; j < NW; ++j) weight(j, wr[j]);
+    for (int j = 0; j < NW; ++j) {
+      if (a.w) weight(j, wr[j]);
+      else
+#pragma unroll
+        for (int k = 0; k < V; ++k) wr[j][k] = 1.f;
+    }
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j) input(i0 - (TAPS - 1) + j, hist[j]);
   }
-  const bool keep = n <= a.R - (taps - 1);              // short runs leave every input (a single tile), long ones the last taps - 1
+  const bool keep = ring && n <= a.R - (taps - 1);      // short runs leave every input (a single tile), long ones the last taps - 1
   for (int i = i0; i < i1; ++i) {
     const int row = row0 + i;
     float cur[V], y[V], ss = 0.f;
     fresh(i, cur);
-    float2 turn[V / 2];
+    constexpr int NT = HALF ? V : V / 2;
+    float2 turn[NT];
+    if (!STATS)
 #pragma unroll
-    for (int k = 0; k < V / 2; ++k) {
-      const int pr = e / 2 + k;
-      turn[k] = !is_v && pr < a.pairs ? a.rope[(size_t)row * a.pairs + pr] : make_float2(1.f, 0.f);
-    }
-    if (keep && own) store_n<T, V>(ring + (size_t)((p0 + i) % a.R) * a.C, own, wvec, cur);
+      for (int k = 0; k < NT; ++k) {
+        const int pr = HALF ? (e + k < a.pairs ? e + k : e + k - a.pairs) : e / 2 + k;
+        turn[k] = !is_v && pr < a.pairs ? a.rope[(size_t)row * a.pairs + pr] : make_float2(1.f, 0.f);
+      }
+    if (!STATS && keep && own) store_n<T, V>(ring + (size_t)((p0 + i) % a.R) * a.C, own, wvec, cur);
 #pragma unroll
-    for (int k = 0; k < V; ++k) y[k] = 0.f;
+    for (int k = 0; k < V; ++k) { y[k] = 0.f; cur[k] += bias[k]; }
     if (TAPS) {
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j)
@@ -254,31 +270,88 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(const ConvQkv<T> a) {
         for (int k = 0; k < V; ++k) y[k] = fmaf(w[k], u[k], y[k]);
       }
     }
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(y[k], y[k], ss);
+    if (STATS) {
+      ss = warp_sum(ss);
+      if (lane == 0) stats[i - i0] += ss;
+      continue;
+    }
     T* dst;
     if (is_q) dst = a.q + (size_t)row * a.q_stride + (size_t)head * a.dp;
     else {
       const int cs = a.slot_map[row];
       if (cs < 0 || cs >= a.n_slots) { if (lane == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, row); continue; }     // warp-uniform
-      dst = a.cache + (size_t)cs * a.row_stride + (is_v ? (size_t)a.G * a.dp + (size_t)head * a.dvp : (size_t)head * a.dp);
+      T* line = a.cache + (size_t)cs * a.row_stride;
+      dst = line + (is_v ? (size_t)a.G * a.dp + (size_t)head * a.dvp : (size_t)head * a.dp);
+      if (!is_v && a.v_from_k && own) store_n<T, V>(line + (size_t)a.G * a.dp + (size_t)head * a.dvp + e, own, own == V, y);
     }
     if (!is_v) {
+      const float f = inv ? inv[i - i0] : (a.norm == QK_NORM_HEAD ? rsqrtf(warp_sum(ss) / (float)d + a.eps) : 1.f);
 #pragma unroll
-      for (int k = 0; k < V; ++k) ss = fmaf(y[k], y[k], ss);
-      const float inv = rsqrtf(warp_sum(ss) / (float)d + a.eps);
+      for (int k = 0; k < V; ++k) y[k] *= f * gain[k];
+      if constexpr (HALF) {
+        if (a.pairs) {
 #pragma unroll
-      for (int k = 0; k < V / 2; ++k) {
-        const float u = y[2 * k] * inv * gain[2 * k], v = y[2 * k + 1] * inv * gain[2 * k + 1];
-        y[2 * k] = u * turn[k].x - v * turn[k].y; y[2 * k + 1] = v * turn[k].x + u * turn[k].y;
+          for (int k = 0; k < V; ++k) xch[e + k] = y[k];
+          __syncwarp();
+#pragma unroll
+          for (int k = 0; k < V; ++k) {
+            const int j = e + k;
+            if (j < a.pairs) y[k] = y[k] * turn[k].x - xch[j + a.pairs] * turn[k].y;
+            else if (j < 2 * a.pairs) y[k] = y[k] * turn[k].x + xch[j - a.pairs] * turn[k].y;
+          }
+          __syncwarp();
+        }
+      } else {
+#pragma unroll
+        for (int k = 0; k < V / 2; ++k) {
+          const float u = y[2 * k], v = y[2 * k + 1];
+          y[2 * k] = u * turn[k].x - v * turn[k].y; y[2 * k + 1] = v * turn[k].x + u * turn[k].y;
+        }
       }
     }
     if (own) store_n<T, V>(dst + e, own, own == V, y);          // head starts are multiples of 64 elements
   }
-  if (!keep && i0 == 0 && own)          // this block read the old ring rows of these channels above: it may overwrite them now
+  if (!STATS && ring && !keep && i0 == 0 && own)          // this block read the old ring rows of these channels above: it may overwrite them now
     for (int i = max(0, n - (taps - 1)); i < n; ++i) {
       float v[V];
       fresh(i, v);
       store_n<T, V>(ring + (size_t)((p0 + i) % a.R) * a.C, own, wvec, v);
     }
+}
+
+// Norms per head (or none): a warp per (head, tile).  WHOLE: a block per tile, its warps share the heads out - sums of squares first, then
+// everything else with the convolution once more (inputs are in L1).
+#define HS_WHOLE_WARPS 16
+template <typename T, int V, int TAPS, bool HALF, bool WHOLE>
+__global__ void __launch_bounds__(WHOLE ? HS_WHOLE_WARPS * 32 : 128) conv_qkv_kernel(const ConvQkv<T> a) {
+  pdl_launch(); pdl_wait();
+  constexpr int NWARP = WHOLE ? HS_WHOLE_WARPS : 4;
+  __shared__ float xch[HALF ? NWARP : 1][HALF ? 32 * V : 1];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, seq = blockIdx.z, units = a.H + (a.v_from_k ? 1 : 2) * a.G;
+  const int n = a.q_len[seq], i0 = blockIdx.y * HS_TILE, i1 = min(n, i0 + HS_TILE), slot = a.state_slot[seq];
+  if (i0 >= n) return;
+  if (slot < 0 || slot >= a.n_state) { if (threadIdx.x == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6E1); return; }
+  float* x = xch[HALF ? warp : 0];
+  if constexpr (!WHOLE) {
+    const int unit = blockIdx.x * NWARP + warp;
+    if (unit < units) conv_qkv_tile<T, V, TAPS, HALF, false>(a, unit, seq, i0, i1, slot, x, nullptr, nullptr);
+  } else {
+    __shared__ float part[2][NWARP][HS_TILE], inv[2][HS_TILE];
+    for (int i = lane; i < 2 * HS_TILE; i += 32) part[i / HS_TILE][warp][i % HS_TILE] = 0.f;
+    __syncwarp();
+    for (int u = warp; u < a.H + a.G; u += NWARP) conv_qkv_tile<T, V, TAPS, HALF, true>(a, u, seq, i0, i1, slot, x, part[u < a.H ? 0 : 1][warp], nullptr);
+    __syncthreads();
+    if (threadIdx.x < 2 * HS_TILE) {
+      const int which = threadIdx.x / HS_TILE, i = threadIdx.x % HS_TILE;
+      float s = 0.f;
+      for (int w = 0; w < NWARP; ++w) s += part[which][w][i];
+      inv[which][i] = rsqrtf(s / (float)((which ? a.G : a.H) * a.dim) + a.eps);
+    }
+    __syncthreads();
+    for (int u = warp; u < units; u += NWARP) conv_qkv_tile<T, V, TAPS, HALF, false>(a, u, seq, i0, i1, slot, x, nullptr, u < a.H + a.G ? inv[u < a.H ? 0 : 1] : nullptr);
+  }
 }
 
 // ---------------------------------------------------------------- short convolution in front of the recurrence
@@ -536,7 +609,7 @@ template <typename T>
 __global__ void __launch_bounds__(128) window_attn_simt_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ cache, const int* __restrict__ page_table,
                                                                const int* __restrict__ kv_len, const int* __restrict__ q_start, const int* __restrict__ q_len,
                                                                T* __restrict__ out, int ldo, int n_seq, int G, int group, int dp, int dvp, int dv, int row_stride,
-                                                               int max_pages, int n_slots, int window, float scale, int* status) {
+                                                               int max_pages, int n_slots, int window, float scale, const AttnExtras<T> x, int* status) {
   pdl_launch(); pdl_wait();
   extern __shared__ float qs[];
   __shared__ float sc[64];
@@ -551,15 +624,18 @@ __global__ void __launch_bounds__(128) window_attn_simt_kernel(const T* __restri
   float m = -INFINITY, l = 0.f, o[WA_COLS];
 #pragma unroll
   for (int j = 0; j < WA_COLS; ++j) o[j] = 0.f;
-  for (int k0 = lo / 64 * 64; k0 <= pos; k0 += 64) {
+  // pages of kept first keys that lie in front of the window, then the window's
+  const int kept = x.kept_tiles(lo / 64, 64), pages = kept + pos / 64 - lo / 64 + 1;
+  for (int pi = 0; pi < pages; ++pi) {
+    const int k0 = (pi < kept ? pi : pi - kept + lo / 64) * 64;
     int slot0 = page_table[(size_t)seq * max_pages + k0 / 64] * 64;
     if (slot0 < 0 || slot0 + 64 > n_slots) { if (tid == 0) ca_dev_fail(status, CA_DEV_BAD_INDEX, t); slot0 = 0; }
     const T* kb = cache + (size_t)slot0 * row_stride + (size_t)kh * dp;
     const T* vb = cache + (size_t)slot0 * row_stride + (size_t)G * dp + (size_t)kh * dvp;
-    const int n = min(64, pos + 1 - k0), first = max(0, lo - k0);
+    const int n = min(64, pos + 1 - k0);
     for (int j = warp * 16; j < warp * 16 + 16; ++j) {
       float s = 0.f;
-      const bool in = j >= first && j < n;
+      const bool in = j < n && (k0 + j >= lo || k0 + j < x.keep_first);
       if (in) for (int i = lane; i < dp; i += 32) s = fmaf(qs[i], to_f(kb[(size_t)j * row_stride + i]), s);
       s = warp_sum(s);
       if (lane == 0) sc[j] = in ? s * scale : -INFINITY;
@@ -579,17 +655,18 @@ __global__ void __launch_bounds__(128) window_attn_simt_kernel(const T* __restri
       const int i = tid + c * 128;
       if (i < dv) {
         float acc = o[c] * al;
-        for (int j = first; j < n; ++j) acc = fmaf(sc[j], to_f(vb[(size_t)j * row_stride + i]), acc);
+        for (int j = 0; j < n; ++j) acc = fmaf(sc[j], to_f(vb[(size_t)j * row_stride + i]), acc);         // keys out of sight weigh zero
         o[c] = acc;
       }
     }
     __syncthreads();
   }
-  const float f = l > 0.f ? 1.f / l : 0.f;
+  if (x.sink) l += expf(x.sink[h] - m);
+  const float f = (l > 0.f ? 1.f / l : 0.f) * x.head_factor(t, h);
 #pragma unroll
   for (int c = 0; c < WA_COLS; ++c) {
     const int i = tid + c * 128;
-    if (i < dv) out[(size_t)t * ldo + (size_t)h * dv + i] = to_t<T>(o[c] * f);
+    if (i < dv) out[(size_t)t * ldo + (size_t)h * dv + i] = to_t<T>(o[c] * f * x.value_factor(t, h * dv + i));
   }
 }
 
@@ -633,37 +710,48 @@ extern "C" int cuteafd_rope_table(const int* positions, const float* freq, float
 }
 
 struct CaConvQkv {
-  const void* proj; const float* w; const float* q_norm; const float* k_norm; const void* rope; void* ring; const int* state_slot; const int* q_start; const int* q_len;
-  const int* kv_len; const int* slot_map; void* q; void* cache; int* status;
-  int ldp, q_stride, row_stride, n_slots, H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state, n_seq, max_q_len; float eps;
+  const void* proj; const float* w; const float* bias; const float* q_norm; const float* k_norm; const void* rope; void* ring; const int* state_slot; const int* q_start;
+  const int* q_len; const int* kv_len; const int* slot_map; void* q; void* cache; int* status;
+  int ldp, q_stride, row_stride, n_slots, H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state, n_seq, max_q_len, norm, half, v_from_k; float eps;
 };
 
-template <typename T, int V>
+template <typename T, int V, bool HALF, bool WHOLE>
 static int conv_qkv_launch(const CaConvQkv* c, cudaStream_t s) {
-  const ConvQkv<T> a{(const T*)c->proj, c->ldp, c->w, c->q_norm, c->k_norm, (const float2*)c->rope, (T*)c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len, c->slot_map,
-                     (T*)c->q, c->q_stride, (T*)c->cache, c->row_stride, c->n_slots, c->H, c->G, c->dim, c->dp, c->vdim, c->dvp, c->pairs, c->taps, c->R, c->C, c->n_state,
-                     c->eps, c->status};
-  const dim3 grid((c->H + 2 * c->G + 3) / 4, (c->max_q_len + HS_TILE - 1) / HS_TILE, c->n_seq);
-  if (c->taps == 2) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 2>), grid, 128, 0, s, a);
-  else if (c->taps == 3) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 3>), grid, 128, 0, s, a);
-  else if (c->taps == 4) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 4>), grid, 128, 0, s, a);
-  else CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 0>), grid, 128, 0, s, a);
+  const ConvQkv<T> a{(const T*)c->proj, c->ldp, c->w, c->bias, c->q_norm, c->k_norm, (const float2*)c->rope, (T*)c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len,
+                     c->slot_map, (T*)c->q, c->q_stride, (T*)c->cache, c->row_stride, c->n_slots, c->H, c->G, c->dim, c->dp, c->vdim, c->dvp, c->pairs, c->taps, c->R, c->C,
+                     c->n_state, c->norm, c->v_from_k, c->eps, c->status};
+  const int units = c->H + (c->v_from_k ? 1 : 2) * c->G;
+  const dim3 grid(WHOLE ? 1 : (units + 3) / 4, (c->max_q_len + HS_TILE - 1) / HS_TILE, c->n_seq);
+  const int nt = WHOLE ? HS_WHOLE_WARPS * 32 : 128;
+  if (c->taps == 1) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 1, HALF, WHOLE>), grid, nt, 0, s, a);
+  else if (c->taps == 2) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 2, HALF, WHOLE>), grid, nt, 0, s, a);
+  else if (c->taps == 3) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 3, HALF, WHOLE>), grid, nt, 0, s, a);
+  else if (c->taps == 4) CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 4, HALF, WHOLE>), grid, nt, 0, s, a);
+  else CA_LAUNCH_PDL((conv_qkv_kernel<T, V, 0, HALF, WHOLE>), grid, nt, 0, s, a);
   CA_CHECK_LAUNCH("conv_qkv");
   return CA_OK;
 }
 
+template <typename T, int V>
+static int conv_qkv_modes(const CaConvQkv* c, cudaStream_t s) {
+  if (c->norm == QK_NORM_WHOLE) return c->half ? conv_qkv_launch<T, V, true, true>(c, s) : conv_qkv_launch<T, V, false, true>(c, s);
+  return c->half ? conv_qkv_launch<T, V, true, false>(c, s) : conv_qkv_launch<T, V, false, false>(c, s);
+}
+
 extern "C" int cuteafd_conv_qkv(const CaConvQkv* c, int f32, cudaStream_t s) {
-  CA_REQUIRE(c && c->proj && c->w && c->q_norm && c->ring && c->state_slot && c->q_start && c->q_len && c->kv_len && c->slot_map && c->q, "conv_qkv: null argument");
-  CA_REQUIRE(c->H >= 1 && c->G >= 0 && (c->G == 0 || (c->k_norm && c->cache)) && c->taps >= 1 && c->taps <= HS_MAX_TAPS && c->R >= c->taps, "conv_qkv: bad geometry");
+  CA_REQUIRE(c && c->proj && c->state_slot && c->q_start && c->q_len && c->kv_len && c->slot_map && c->q, "conv_qkv: null argument");
+  CA_REQUIRE(c->taps >= 1 && c->taps <= HS_MAX_TAPS && (c->taps == 1 || (c->w && c->ring)) && (!c->ring || c->R >= c->taps), "conv_qkv: convolution without its weights or inputs");
+  CA_REQUIRE(c->norm >= QK_NORM_NONE && c->norm <= QK_NORM_WHOLE && (c->norm == QK_NORM_NONE || (c->q_norm && (c->G == 0 || c->k_norm))), "conv_qkv: norm without its gains");
+  CA_REQUIRE(c->H >= 1 && c->G >= 0 && (c->G == 0 || c->cache) && (!c->v_from_k || c->vdim == c->dim), "conv_qkv: bad geometry");
   CA_REQUIRE(c->dim >= 1 && c->dim <= 256 && c->vdim <= 256 && c->dp % 8 == 0 && c->dvp % 8 == 0 && c->dim <= c->dp && c->vdim <= c->dvp && c->row_stride % 8 == 0, "conv_qkv: heads of up to 256 dimensions");
-  CA_REQUIRE(c->C == (c->H + c->G) * c->dim + c->G * c->vdim && c->ldp >= c->C && c->q_stride >= c->H * c->dp && (c->G == 0 || c->row_stride >= c->G * (c->dp + c->dvp)), "conv_qkv: row too short");
-  CA_REQUIRE(c->pairs >= 0 && 2 * c->pairs <= c->dim && (c->pairs == 0 || c->rope) && c->R - (c->taps - 1) <= HS_TILE, "conv_qkv: bad rotation or ring");
+  CA_REQUIRE(c->C == (c->H + c->G) * c->dim + (c->v_from_k ? 0 : c->G * c->vdim) && c->ldp >= c->C && c->q_stride >= c->H * c->dp && (c->G == 0 || c->row_stride >= c->G * (c->dp + c->dvp)), "conv_qkv: row too short");
+  CA_REQUIRE(c->pairs >= 0 && 2 * c->pairs <= c->dim && (c->pairs == 0 || c->rope) && (!c->ring || c->R - (c->taps - 1) <= HS_TILE), "conv_qkv: bad rotation or ring");
   if (c->n_seq <= 0 || c->max_q_len <= 0) return CA_OK;
   CA_REQUIRE(c->n_seq <= 65535 && (c->max_q_len + HS_TILE - 1) / HS_TILE <= 65535, "conv_qkv: step too large");
   const int nc = ((c->dim > c->vdim || c->G == 0 ? c->dim : c->vdim) + 63) / 64;
-  if (nc <= 1) return f32 ? conv_qkv_launch<float, 2>(c, s) : conv_qkv_launch<bf16, 2>(c, s);
-  if (nc <= 2) return f32 ? conv_qkv_launch<float, 4>(c, s) : conv_qkv_launch<bf16, 4>(c, s);
-  return f32 ? conv_qkv_launch<float, 8>(c, s) : conv_qkv_launch<bf16, 8>(c, s);
+  if (nc <= 1) return f32 ? conv_qkv_modes<float, 2>(c, s) : conv_qkv_modes<bf16, 2>(c, s);
+  if (nc <= 2) return f32 ? conv_qkv_modes<float, 4>(c, s) : conv_qkv_modes<bf16, 4>(c, s);
+  return f32 ? conv_qkv_modes<float, 8>(c, s) : conv_qkv_modes<bf16, 8>(c, s);
 }
 
 struct CaRecurrence {          // one recurrent layer's step: shared by its convolution and its scan
@@ -735,13 +823,13 @@ extern "C" int cuteafd_glu_rows(const void* g, const void* u, const float* gb, c
 
 extern "C" int cuteafd_window_attention_simt(const void* q, int q_stride, const void* cache, const int* page_table, const int* kv_len, const int* q_start, const int* q_len,
                                              void* out, int ldo, int T, int n_seq, int Hq, int Hkv, int dp, int dvp, int dv, int row_stride, int max_pages, int n_slots,
-                                             int window, float scale, int f32, int* status, cudaStream_t s) {
+                                             int window, float scale, int f32, const CaAttnExtras* extras, int* status, cudaStream_t s) {
   CA_REQUIRE(q && cache && page_table && kv_len && q_start && q_len && out, "window_attention_simt: null argument");
   CA_REQUIRE(Hkv >= 1 && Hq % Hkv == 0 && Hq <= 65535 && dv >= 1 && dv <= dvp && dv <= 128 * WA_COLS && dp >= 1 && dp <= 4096 && row_stride >= Hkv * (dp + dvp) && ldo >= Hq * dv,
              "window_attention_simt: bad shape");
   if (T <= 0 || n_seq <= 0) return CA_OK;
-  if (f32) CA_LAUNCH_PDL(window_attn_simt_kernel<float>, dim3(T, Hq), 128, dp * sizeof(float), s, (const float*)q, q_stride, (const float*)cache, page_table, kv_len, q_start, q_len, (float*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, max_pages, n_slots, window, scale, status);
-  else CA_LAUNCH_PDL(window_attn_simt_kernel<bf16>, dim3(T, Hq), 128, dp * sizeof(float), s, (const bf16*)q, q_stride, (const bf16*)cache, page_table, kv_len, q_start, q_len, (bf16*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, max_pages, n_slots, window, scale, status);
+  if (f32) CA_LAUNCH_PDL(window_attn_simt_kernel<float>, dim3(T, Hq), 128, dp * sizeof(float), s, (const float*)q, q_stride, (const float*)cache, page_table, kv_len, q_start, q_len, (float*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, max_pages, n_slots, window, scale, attn_extras<float>(extras, window), status);
+  else CA_LAUNCH_PDL(window_attn_simt_kernel<bf16>, dim3(T, Hq), 128, dp * sizeof(float), s, (const bf16*)q, q_stride, (const bf16*)cache, page_table, kv_len, q_start, q_len, (bf16*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, max_pages, n_slots, window, scale, attn_extras<bf16>(extras, window), status);
   CA_CHECK_LAUNCH("window_attention_simt");
   return CA_OK;
 }

@@ -183,7 +183,7 @@ __global__ void router_select_kernel(const float* __restrict__ logits, const flo
     if (tid < n_group) {
       float a = -INFINITY, b = -INFINITY;
       for (int j = 0; j < per; ++j) { const float v = choice[tid * per + j]; if (v > a) { b = a; a = v; } else if (v > b) b = v; }
-      gscore[tid] = by_max ? a : a + b;
+      gscore[tid] = by_max || per == 1 ? a : a + b;
     }
     __syncthreads();
     if (tid == 0) {
@@ -439,7 +439,7 @@ __device__ __forceinline__ void router_select_warp(const float* lg, const float*
     if (lane < n_group) {
       float a = -INFINITY, b = -INFINITY;
       for (int j = 0; j < per; ++j) { const float v = choice[lane * per + j]; if (v > a) { b = a; a = v; } else if (v > b) b = v; }
-      gs = by_max ? a : a + b;
+      gs = by_max || per == 1 ? a : a + b;
     }
     unsigned keep = 0;
     for (int r = 0; r < topk_group; ++r) {      // best groups first, lowest group id among equals

@@ -79,7 +79,10 @@ class HybridStackEngine(StackBase, Engine):
     PREFILL_MIN_Q = 64          # query rows of a sequence from which attention takes the 128-key kernel
 
     def __init__(self, weights: HybridWeights, **kw):
-        spec = weights.spec
+        self._check(weights.spec)
+        super().__init__(weights, **kw)
+
+    def _check(self, spec):
         if spec.stack != "hybrid":
             raise ValueError("HybridStackEngine runs hybrid stacks described by ModelSpec.blocks")
         for i, b in enumerate(spec.blocks):
@@ -88,7 +91,6 @@ class HybridStackEngine(StackBase, Engine):
                 raise ValueError(f"layer {i}: convolutions of 1 to {MAX_TAPS} taps (got {taps})")
             if b.attn is not None and max(b.attn.head_dim, b.attn.v_head_dim) > 256:
                 raise ValueError(f"layer {i}: heads of up to 256 dimensions (got {b.attn.head_dim} / {b.attn.v_head_dim})")
-        super().__init__(weights, **kw)
 
     # ------------------------------------------------------------------ cache and state
     def _alloc_attention_state(self):
@@ -105,18 +107,26 @@ class HybridStackEngine(StackBase, Engine):
             for i in owners:
                 a = spec.blocks[i].attn
                 self.maps[self.plane[i]] = ops.encode_window_maps(self.kv[self.plane[i]], a.n_kv_heads, up(a.head_dim, 64), up(a.v_head_dim, 64))
-        self.rings, self.states = [], []
-        for i, b in enumerate(spec.blocks):
+        self.rings = []
+        for i in range(spec.n_layers):
             conv = self.weights.layer(i).conv
-            self.rings.append(torch.zeros(self.max_seqs, conv.shape[0] - 1 + self.state_depth, conv.shape[1], dtype=dt, device=dev))
-            self.states.append(torch.zeros(self.max_seqs, self.state_depth + 1, b.rec.width, dtype=torch.float32, device=dev) if b.rec is not None else None)
+            self.rings.append(torch.zeros(self.max_seqs, conv.shape[0] - 1 + self.state_depth, conv.shape[1], dtype=dt, device=dev) if conv is not None else None)
+        self._alloc_states()
         with LEDGER.scope("kv"):
-            LEDGER.charge(sum(t.numel() * t.element_size() for t in self.rings + self.states if t is not None), "sequence state slots")
+            LEDGER.charge(sum(t.numel() * t.element_size() for t in self.state_buffers()), "sequence state slots")
+
+    def _alloc_states(self):
+        """What the recurrent layers carry per state slot."""
+        self.states = [torch.zeros(self.max_seqs, self.state_depth + 1, b.rec.width, dtype=torch.float32, device=self.device) if b.rec is not None else None
+                       for b in self.spec.blocks]
+
+    def state_buffers(self) -> list:
+        return [t for t in self.rings + self.states if t is not None]
 
     @staticmethod
     def _visible_pages(a: AttentionSpec, rows: int) -> int:
-        """Pages a run of `rows` queries can see at most through the layer's window (a large number without one)."""
-        return (a.window + rows - 1 + PAGE - 2) // PAGE + 1 if a.window else 1 << 20
+        """Pages a run of `rows` queries can see at most through the layer's window and among kept first keys (a large number without a window)."""
+        return (a.window + rows - 1 + PAGE - 2) // PAGE + 1 + -(-a.keep_first // PAGE) if a.window else 1 << 20
 
     def attn_splits_for(self, n_seq: int, max_q_len: int, max_kv: int) -> int:
         """The largest split count a layer of the step wants (each takes no more than its window has pages)."""
@@ -179,14 +189,21 @@ class HybridStackEngine(StackBase, Engine):
         return L
 
     def _attention(self, li: int, a: AttentionSpec, lw: HybridLayer, L: HybridLane, sh: StepShape):
+        b = L.attention(a, lw.w_in.N)
+        self._dense(lw.w_in, L.xn_act, b["proj"], sh.T)
+        self._attend(li, a, lw, L, b, b["o"], sh)
+        self._dense(lw.wo, b["o_act"], L.mix, sh.T)
+
+    def _attend(self, li: int, a: AttentionSpec, lw: HybridLayer, L: HybridLane, b: dict, out: torch.Tensor, sh: StepShape, *, bias=None, extras=None):
+        """Projected rows b["proj"] -> convolution, norms, rotation, cache -> attended rows `out`."""
         T, md, H, G, plane = sh.T, self.md, a.n_heads, a.n_kv_heads, self.plane[li]
         dp, dvp, dv = up(a.head_dim, 64), up(a.v_head_dim, 64), a.v_head_dim
-        b = L.attention(a, lw.w_in.N)
-        self._dense(lw.w_in, L.xn_act, b["proj"], T)
         ops.conv_qkv(b["proj"], lw.conv, lw.q_norm, lw.k_norm, L.rope.get(rope_key(a)), self.rings[li], b["q"], self.kv[plane], md, H=H, G=G if a.kv_from < 0 else 0,
-                     dim=a.head_dim, dp=dp, vdim=dv, dvp=dvp, pairs=a.rope_dims // 2, eps=self.spec.rms_eps, n_seq=sh.n_seq, max_q_len=sh.max_q_len, status=self.status)
-        where = (md["page_table"], md["kv_len"], md["q_start"], md["q_len"], b["o"])
-        shape = dict(T=T, n_seq=sh.n_seq, Hq=H, Hkv=G, dp=dp, dvp=dvp, dv=dv, window=a.window, scale=a.softmax_scale, status=self.status)
+                     dim=a.head_dim, dp=dp, vdim=dv, dvp=dvp, pairs=a.rope_dims // 2, eps=self.spec.rms_eps, n_seq=sh.n_seq, max_q_len=sh.max_q_len, bias=bias,
+                     norm="whole" if a.qk_norm_whole else ("head" if a.qk_norm else ""), half=not a.rope_interleaved, values_are_keys=a.values_are_keys,
+                     n_slots=self.max_seqs, status=self.status)
+        where = (md["page_table"], md["kv_len"], md["q_start"], md["q_len"], out)
+        shape = dict(T=T, n_seq=sh.n_seq, Hq=H, Hkv=G, dp=dp, dvp=dvp, dv=dv, window=a.window, scale=a.softmax_scale, extras=extras, status=self.status)
         if self.f32 or H // G > 128:
             ops.window_attention_simt(b["q"], self.kv[plane], *where, **shape)
         elif sh.max_q_len >= self.PREFILL_MIN_Q and dp + 2 * dvp <= 512:
@@ -198,7 +215,6 @@ class HybridStackEngine(StackBase, Engine):
                 self.launches_per_step += 1
             ops.window_attention(b["q"], self.maps[plane], *where, max_q_len=sh.max_q_len, n_splits=splits, part_o=self.part_o if splits > 1 else None,
                                  part_ml=self.part_ml if splits > 1 else None, **shape)
-        self._dense(lw.wo, b["o_act"], L.mix, T)
         self.launches_per_step += 2
 
     def _recurrence(self, li: int, r: RecurrentSpec, lw: HybridLayer, L: HybridLane, sh: StepShape):

@@ -20,14 +20,11 @@ same program runs entirely in fp32: fp32 products, the ordinary-core attention k
 """
 from __future__ import annotations
 
-import math
-import os
-
 import torch
 
 from .. import ops
 from ..models.latent_stack import StackLayer, StackWeights, up
-from ..ops import ActBuffer, KIND_BF16, native, pick_tn
+from ..ops import ActBuffer, KIND_BF16, native
 from ..ops.native import call, ptr, stream
 from .engine import PAGE, StepShape
 from .mla import MlaEngine
@@ -61,24 +58,6 @@ class LatentLane(StackLane):
             o, o_act = self._operand(H * self.cap, rp)
             return {"q": q, "o": o, "o_act": o_act}
         return self.get(("lat", H, rp), make)
-
-    def experts(self, m) -> dict:
-        E, k, ff, cap = m.n_experts, m.top_k, m.intermediate, self.cap
-
-        def make():
-            rows = cap * k
-            # rows per expert of a full lane: whole 256-row tiles where they fill, else about twice the mean
-            mean = max(1, math.ceil(rows / E))
-            tn = pick_tn(min(mean if mean >= 256 else min(2 * mean, 128), int(os.environ.get("CUTEAFD_TNG", "256"))))
-            i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=self.dev)
-            xs, xs_act = self._operand(rows, self.eng.Wp, tn)
-            h1, h1_act = self._operand(rows, up(ff, 8), tn)
-            max_tiles = E + rows // tn + 1
-            return {"tn": tn, "max_tiles": max_tiles, "logits": torch.zeros(cap, E, dtype=torch.float32, device=self.dev), "idx": i32(cap, k),
-                    "wts": torch.zeros(cap, k, dtype=torch.float32, device=self.dev), "src": i32(rows), "slot": i32(cap, k), "counts": i32(E),
-                    "offsets": i32(E), "tiles": i32(max_tiles, 4), "n_tiles": i32(1), "n_rows": i32(1), "xs": xs, "xs_act": xs_act, "h1": h1,
-                    "h1_act": h1_act, "y": torch.zeros(rows, self.eng.Wp, dtype=self.dt, device=self.dev)}
-        return self.get(("moe", E, k, ff), make)
 
 
 class LatentStackEngine(StackBase, MlaEngine):
@@ -211,23 +190,6 @@ class LatentStackEngine(StackBase, MlaEngine):
                                  n_splits=sh.attn_splits, part_o=po, part_ml=pml, **common)
         ops.tc_linear(lw.w_uv, lat["o_act"], b["o"], rows=H * L.cap, token_major=(L.cap, a.v_head_dim), **per)
         self.launches_per_step += 3
-
-    def _experts(self, m, lw: StackLayer, L: LatentLane, e: dict, T: int):
-        E, k = m.n_experts, m.top_k
-        sel = (e["logits"], None, e["idx"], e["wts"], T, k, m.scoring, m.normalize, m.route_scale, m.n_group, m.topk_group)
-        if T * k <= 1024:
-            ops.router_select_pack(*sel, e["src"], e["slot"], e["counts"], e["offsets"], e["tiles"], e["n_tiles"], e["n_rows"], 0, E, e["tn"], e["max_tiles"],
-                                   group_score=m.group_score)
-        else:
-            ops.router_select(*sel, group_score=m.group_score)
-            ops.route_pack(e["idx"], e["src"], e["slot"], e["counts"], e["offsets"], e["tiles"], e["n_tiles"], e["n_rows"], T, k, 0, E, e["tn"], e["max_tiles"])
-            self.launches_per_step += 1
-        rows = T * k
-        call("cuteafd_gather_rows", ptr(L.xn), ptr(e["src"]), ptr(e["n_rows"]), ptr(e["xs"]), rows, self.Wp * L.xn.element_size() // 2, stream())
-        tiles = dict(tiles=e["tiles"], n_tiles=e["n_tiles"], max_tiles=min(e["max_tiles"], E + rows // e["tn"] + 1), status=self.status)
-        ops.tc_linear(lw.w_up, e["xs_act"], e["h1"], rows=rows, act="relu2", **tiles)
-        ops.tc_linear(lw.w_down, e["h1_act"], e["y"], rows=rows, **tiles)
-        self.launches_per_step += 4
 
     # ------------------------------------------------------------------ prefill chunks: attention over the expanded context
     def _expands(self, a, sh: StepShape) -> bool:

@@ -34,6 +34,12 @@ def load_weights(model: str, spec: ModelSpec, device, seed: int = 1):
     """Weights of a snapshot in the forms the kernels consume, or synthetic ones for a named shape."""
     from ..models.weights import DeviceWeights
     snapshot = os.path.isdir(model)
+    if spec.stack == "hyper":
+        from ..models.hyper_stack import hyper_weights_from_masters, hyper_weights_random
+        if snapshot:
+            from ..loader.stack_checkpoint import read_hyper_masters
+            return hyper_weights_from_masters(spec, read_hyper_masters(model, spec), device)
+        return hyper_weights_random(spec, device, seed=seed)
     if spec.stack == "hybrid":
         from ..models.hybrid_stack import hybrid_weights_from_masters, hybrid_weights_random
         if snapshot:
@@ -62,6 +68,9 @@ def load_weights(model: str, spec: ModelSpec, device, seed: int = 1):
 
 
 def engine_class(spec: ModelSpec):
+    if spec.stack == "hyper":
+        from .hyper_stack import HyperStackEngine
+        return HyperStackEngine
     if spec.stack == "hybrid":
         from .hybrid_stack import HybridStackEngine
         return HybridStackEngine

@@ -1,6 +1,8 @@
-"""What the engines of layer stacks share: a lane over fp32 residual rows, bf16 or fp32 operands, lanes of prompt size, lazily made buffers."""
+"""What the engines of layer stacks share: a lane over fp32 residual rows, bf16 or fp32 operands, lanes of prompt size, lazily made buffers, routed
+experts."""
 from __future__ import annotations
 
+import math
 import os
 
 import torch
@@ -8,6 +10,7 @@ import torch
 from .. import ops
 from ..models.latent_stack import up
 from ..ops import ActBuffer, KIND_BF16, KIND_F32, pick_tn
+from ..ops.native import call, ptr, stream
 from .engine import Lane
 
 LANE_CAPS = (16, 32, 64, 256, 1024, 4096, 16384)
@@ -23,7 +26,7 @@ class StackLane(Lane):
         # products of one weight tile keep both accumulators with 256-row token tiles: prompt-sized lanes take them
         self.tn = pick_tn(min(cap, int(os.environ.get("CUTEAFD_TN", "256" if cap >= 1024 else "128"))))
         Wp = eng.Wp
-        self.x = torch.zeros(cap, Wp, dtype=torch.float32, device=self.dev)
+        self.x = torch.zeros(cap, *eng.residual_shape, dtype=torch.float32, device=self.dev)
         self.xn, self.xn_act = self._operand(cap, Wp)
         self.mix = torch.zeros(cap, Wp, dtype=self.dt, device=self.dev)
         rows = min(cap, 256)
@@ -56,6 +59,27 @@ class StackLane(Lane):
             self._head_acts[tn] = ActBuffer(self.kind, self.xln.shape[0], self.eng.Wp, tn, self.xln, ops.encode_tmap(self.xln, tn))
         return self._head_acts[tn]
 
+    def experts(self, m) -> dict:
+        E, k, ff, cap = m.n_experts, m.top_k, m.intermediate, self.cap
+        glu = m.activation == "swiglu"
+
+        def make():
+            rows = cap * k
+            # rows per expert of a full lane: whole 256-row tiles where they fill, else about twice the mean (a product of two weight tiles
+            # takes at most 128)
+            mean = max(1, math.ceil(rows / E))
+            tn = pick_tn(min(mean if mean >= 256 else min(2 * mean, 128), int(os.environ.get("CUTEAFD_TNG", "256"))), swiglu=glu)
+            i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=self.dev)
+            xs, xs_act = self._operand(rows, self.eng.Wp, tn)
+            h1, h1_act = self._operand(rows, up(ff, 8), tn)
+            max_tiles = E + rows // tn + 1
+            return {"tn": tn, "max_tiles": max_tiles, "logits": torch.zeros(cap, E, dtype=torch.float32, device=self.dev), "idx": i32(cap, k),
+                    "wts": torch.zeros(cap, k, dtype=torch.float32, device=self.dev), "src": i32(rows), "slot": i32(cap, k), "counts": i32(E),
+                    "offsets": i32(E), "tiles": i32(max_tiles, 4), "n_tiles": i32(1), "n_rows": i32(1), "xs": xs, "xs_act": xs_act, "h1": h1,
+                    "h1_act": h1_act, "y": torch.zeros(rows, self.eng.Wp, dtype=self.dt, device=self.dev),
+                    **({"g": torch.zeros_like(h1), "u": torch.zeros_like(h1)} if glu and self.eng.f32 else {})}
+        return self.get(("moe", E, k, ff, m.activation), make)
+
     def get(self, key, make):
         if key not in self._bufs:
             self._bufs[key] = make()
@@ -70,6 +94,11 @@ class StackBase:
         self.f32, self.Wp = weights.f32, up(weights.spec.hidden, 8)
         self.tap = None             # set to a list to collect the residual rows after every layer run of eager steps
         super().__init__(weights, **kw)
+
+    @property
+    def residual_shape(self) -> tuple:
+        """Shape of a token's residual rows."""
+        return (self.Wp,)
 
     def lane(self, T: int) -> StackLane:
         cap = next(c for c in LANE_CAPS if T <= c)
@@ -87,3 +116,28 @@ class StackBase:
 
     def _splits(self, N, K, T, tn, kind):
         return 1 if kind == KIND_F32 else super()._splits(N, K, T, tn, kind)
+
+    def _experts(self, m, lw, L: StackLane, e: dict, T: int):
+        """Routing, packing, gather and the experts' products of the rows L.xn, from router logits in e["logits"]: weighted rows stay in e."""
+        E, k = m.n_experts, m.top_k
+        sel = (e["logits"], None, e["idx"], e["wts"], T, k, m.scoring, m.normalize, m.route_scale, m.n_group, m.topk_group)
+        if T * k <= 1024:
+            ops.router_select_pack(*sel, e["src"], e["slot"], e["counts"], e["offsets"], e["tiles"], e["n_tiles"], e["n_rows"], 0, E, e["tn"], e["max_tiles"],
+                                   group_score=m.group_score)
+        else:
+            ops.router_select(*sel, group_score=m.group_score)
+            ops.route_pack(e["idx"], e["src"], e["slot"], e["counts"], e["offsets"], e["tiles"], e["n_tiles"], e["n_rows"], T, k, 0, E, e["tn"], e["max_tiles"])
+            self.launches_per_step += 1
+        rows = T * k
+        call("cuteafd_gather_rows", ptr(L.xn), ptr(e["src"]), ptr(e["n_rows"]), ptr(e["xs"]), rows, self.Wp * L.xn.element_size() // 2, stream())
+        tiles = dict(tiles=e["tiles"], n_tiles=e["n_tiles"], max_tiles=min(e["max_tiles"], E + rows // e["tn"] + 1), status=self.status)
+        if m.activation == "relu2":
+            ops.tc_linear(lw.w_up, e["xs_act"], e["h1"], rows=rows, act="relu2", **tiles)
+        elif self.f32:
+            ops.tc_linear(lw.w_gate, e["xs_act"], e["g"], rows=rows, **tiles)
+            ops.tc_linear(lw.w_up, e["xs_act"], e["u"], rows=rows, **tiles)
+            ops.silu_rows(e["g"], e["u"], e["h1"], rows)
+        else:
+            ops.tc_linear(lw.w_gate, e["xs_act"], e["h1"], rows=rows, w_up=lw.w_up, **tiles)
+        ops.tc_linear(lw.w_down, e["h1_act"], e["y"], rows=rows, **tiles)
+        self.launches_per_step += 4

@@ -1,4 +1,4 @@
-"""Snapshots of layer stacks: tensor names <-> the masters `models.latent_stack` and `models.hybrid_stack` pack.  Matrices are [out, in].
+"""Snapshots of layer stacks: tensor names <-> the masters `models.latent_stack`, `models.hybrid_stack` and `models.hyper_stack` pack.  Matrices are [out, in].
 
 Latent-attention stacks (the Bedovik design): layer i's tensors start with `l<i>.`: `norm1` (+ `.b`, `.alpha`), `mix.{q,dkv,dkv.norm,uk,uv,g,o}`, `mlp.router`, `mlp.e<j>.{up,down}`,
 `ls1`, `ls2`; the stack has `embed`, `pos`, `loop.in`, `loop.step`, `final.norm` (+ `.b`, `.alpha`) and `head`.
@@ -7,6 +7,11 @@ Hybrid recurrent / windowed-attention stacks (the Tudilix design): `l<i>.norm1`,
 `mlp.{gate,up,down}` (+ `.b`); attention has `mix.{q,k,v,o}`, `mix.{q,k,v}.conv`, `mix.{q,k}.norm` (no `k` and `v` where the layer uses
 another layer's); the recurrence has `mix.{y,x}` (+ `.b`), `mix.conv` (+ `.b`), `mix.{ra,ri}` (+ `.b`), `mix.lam`, `mix.o`; the stack has
 `embed`, `final.norm` and `head`.
+
+Hyper-connected stacks (the Vozetar design): `l<i>.norm1`, `hc1.{in,out,mix}` and, with a feed-forward, `norm2`, `hc2.*`, `mlp.{gate,up,down}` or
+`mlp.router`, `mlp.e<j>.{gate,up,down}`, `mlp.shared.{gate,up,down}`; attention has `{q,k,v,o}` (+ `.b`, `.conv`, `.norm`), `sink` and `g` as its kind
+has them, under `mix.` or - beside a linear mixer with `right.{q,k,v,g,o}`, `right.{a1,a2,a2.b,norm}` - under `mix.left.`; normalised mixers have
+`mix.{left,right}.out`; the stack has `embed`, `bigram`, `final.norm` and `head`.
 """
 from __future__ import annotations
 
@@ -19,13 +24,16 @@ from .safetensors_io import catalog, read_tensor
 
 
 def _reader(snapshot: str | Path):
-    """get(name, *shape): a tensor of the snapshot in its stored dtype, refused when its shape is not the one the configuration implies."""
+    """get(name, *shape): a tensor of the snapshot in its stored dtype, refused when its shape is not the one the configuration implies (0: a size
+    that only the tensor tells)."""
     cat = catalog(snapshot)
 
     def get(name: str, *shape: int) -> torch.Tensor:
         if name not in cat:
             raise KeyError(f"tensor {name} missing from the snapshot")
         t = read_tensor(cat[name])
+        if t.dim() == len(shape):
+            shape = tuple(n or m for n, m in zip(shape, t.shape))
         if t.numel() != torch.Size(shape).numel() or (t.dim() > 1 and tuple(t.shape) != shape):
             raise ValueError(f"tensor {name}: shape {tuple(t.shape)}, the configuration implies {shape}")
         return t.reshape(shape)
@@ -95,3 +103,55 @@ def read_hybrid_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
 
     return {"embed": get("embed", spec.vocab, W), "lm_head": get("head", spec.vocab, W), "final_norm": get("final.norm", W),
             "layers": [layer(i, b) for i, b in enumerate(spec.blocks)]}
+
+
+def read_hyper_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
+    """Weights of a hyper-connected stack's snapshot in their stored dtype, checked against the shapes the configuration implies."""
+    get, W, S = _reader(snapshot), spec.hidden, spec.streams
+
+    def layer(i: int, b) -> dict:
+        a, r, m = b.attn, b.rec, b.moe
+        p = f"l{i}.mix" + (".left" if r is not None else "")
+        hc = lambda q: (get(f"l{i}.hc{q}.in", S), get(f"l{i}.hc{q}.out", S), get(f"l{i}.hc{q}.mix", S, S))
+        lw = {"norm1": get(f"l{i}.norm1", W), "hc1": hc(1), "wo": get(f"{p}.o", W, a.n_heads * a.v_head_dim)}
+        sizes = {"q": a.n_heads * a.head_dim, "k": a.n_kv_heads * a.head_dim, "v": a.n_kv_heads * a.v_head_dim}
+        for k in ("q", "k") if a.values_are_keys else ("q", "k", "v"):
+            lw[f"w{k}"] = get(f"{p}.{k}", sizes[k], W)
+            if a.qkv_bias:
+                lw[f"{k}_b"] = get(f"{p}.{k}.b", sizes[k])
+            if a.conv_taps > 1:
+                lw[f"{k}_conv"] = get(f"{p}.{k}.conv", sizes[k], a.conv_taps)
+            if a.qk_norm_whole and k != "v":
+                lw[f"{k}_norm"] = get(f"{p}.{k}.norm", sizes[k])
+        if a.out_bias:
+            lw["o_b"] = get(f"{p}.o.b", W)
+        if a.sink:
+            lw["sink"] = get(f"{p}.sink", a.n_heads)
+        if a.out_gate:
+            lw["wg"] = get(f"{p}.g", a.gate_width, W)
+        if r is not None:
+            p, hk, hv = f"l{i}.mix.right", r.heads * r.dim, r.heads * r.vdim
+            lw.update(rq=get(f"{p}.q", hk, W), rk=get(f"{p}.k", hk, W), rv=get(f"{p}.v", hv, W), rg=get(f"{p}.g", hv, W), r_o=get(f"{p}.o", W, hv))
+            if r.kind == "gla":
+                lw["a1"] = get(f"{p}.a1", r.rank, W)
+                lw["a2"], lw["a2_b"], lw["r_norm"] = get(f"{p}.a2", hk, lw["a1"].shape[0]), get(f"{p}.a2.b", hk), get(f"{p}.norm", r.vdim)
+        if b.merge_norm:
+            lw["merge_norms"] = (get(f"l{i}.mix.left.out", W), get(f"l{i}.mix.right.out", W))
+        if m is None and b.ffn is None:
+            return lw
+        p, glu = f"l{i}.mlp", lambda p, ff: (get(f"{p}.gate", ff, W), get(f"{p}.up", ff, W), get(f"{p}.down", W, ff))
+        lw["norm2"], lw["hc2"] = get(f"l{i}.norm2", W), hc(2)
+        if b.ffn is not None:
+            lw["ws_gate"], lw["ws_up"], lw["ws_down"] = glu(p, b.ffn.intermediate)
+            return lw
+        lw["router"] = get(f"{p}.router", m.n_experts, W)
+        lw["w_gate"], lw["w_up"], lw["w_down"] = (torch.stack(ts) for ts in zip(*[glu(f"{p}.e{j}", m.intermediate) for j in range(m.n_experts)]))
+        if m.n_shared:
+            lw["ws_gate"], lw["ws_up"], lw["ws_down"] = glu(f"{p}.shared", m.shared_inter)
+        return lw
+
+    w = {"embed": get("embed", spec.vocab, W), "lm_head": get("head", spec.vocab, W), "final_norm": get("final.norm", W)}
+    if spec.pair_table is not None:
+        w["pairs"] = get("bigram", spec.pair_table.buckets + 1, W)
+    w["layers"] = [layer(i, b) for i, b in enumerate(spec.blocks)]
+    return w

@@ -16,7 +16,7 @@ import torch
 import torch.nn.functional as F
 
 from .. import ops
-from ..config import AttentionSpec, ModelSpec
+from ..config import AttentionSpec, ModelSpec, RecurrentSpec
 from ..ops import KIND_BF16, KIND_F32, TcWeight
 from .latent_stack import _pad, stack_kind, up
 from .weights import DeviceWeights, LayerWeights
@@ -53,13 +53,13 @@ class HybridWeights(DeviceWeights):
         return self.lm_head.kind == KIND_F32
 
 
-def rope_key(a: AttentionSpec) -> tuple:
-    return (a.rope_dims, a.rope_theta, a.rope_scaling)
+def rope_key(a: AttentionSpec | RecurrentSpec) -> tuple:
+    return (a.rope_dims, a.rope_theta, getattr(a, "rope_scaling", None))
 
 
-def rope_frequencies(a: AttentionSpec) -> tuple[list, float]:
+def rope_frequencies(a: AttentionSpec | RecurrentSpec) -> tuple[list, float]:
     """Angle per position of every rotated pair, and the factor on cosine and sine."""
-    n, s = a.rope_dims, a.rope_scaling
+    n, s = a.rope_dims, getattr(a, "rope_scaling", None)
     freq = [a.rope_theta ** (-2.0 * i / n) for i in range(n // 2)]
     if s is None:
         return freq, 1.0
@@ -71,13 +71,13 @@ def rope_frequencies(a: AttentionSpec) -> tuple[list, float]:
 
 def rope_tables(spec: ModelSpec, device) -> dict:
     out = {}
-    for b in spec.blocks:
-        if b.attn is None or not b.attn.rope_dims or rope_key(b.attn) in out:
+    for m in [m for b in spec.blocks for m in (b.attn, b.rec) if m is not None]:
+        if not m.rope_dims or rope_key(m) in out:
             continue
-        freq, amp = rope_frequencies(b.attn)
+        freq, amp = rope_frequencies(m)
         f = torch.tensor(freq, dtype=torch.float64)
         hi = f.float()
-        out[rope_key(b.attn)] = (torch.stack([hi, (f - hi.double()).float()]).to(device).contiguous(), amp)
+        out[rope_key(m)] = (torch.stack([hi, (f - hi.double()).float()]).to(device).contiguous(), amp)
     return out
 
 

@@ -797,19 +797,29 @@ def rope_table(positions, freq, amp: float, out, T: int):
     call("cuteafd_rope_table", ptr(positions), ptr(freq), float(amp), freq.shape[1], ptr(out), T, stream())
 
 
-def conv_qkv(proj, w, q_norm, k_norm, rope, ring, q, cache, meta: dict, *, H, G, dim, dp, vdim, dvp, pairs, eps, n_seq, max_q_len, status=None):
-    """Short causal convolution over projected query / key / value rows, head norms, rotation; queries to `q` [., H * dp], keys and values to the
-    paged `cache` rows.  `ring` [slots, depth + taps - 1, channels]: inputs by position.  `meta`: the step's device inputs.  G = 0: queries only."""
-    _chk(w, torch.float32, "w")
+QK_NORMS = {"": 0, "head": 1, "whole": 2}
+
+
+def conv_qkv(proj, w, q_norm, k_norm, rope, ring, q, cache, meta: dict, *, H, G, dim, dp, vdim, dvp, pairs, eps, n_seq, max_q_len, bias=None, norm: str = "head",
+             half: bool = False, values_are_keys: bool = False, n_slots: int = 0, status=None):
+    """Short causal convolution over projected query / key / value rows (+ `bias`), norms, rotation; queries to `q` [., H * dp], keys and values to
+    the paged `cache` rows.  `w` None: no convolution.  `ring` [slots, depth + taps - 1, channels]: inputs by position (None with one tap: give the
+    number of state slots).  `norm`: "head" (gains [dim]), "whole" (over all heads at once, gains [H * dim] / [G * dim]) or "".  `half`: dimensions i
+    and i + pairs turn together instead of neighbours.  `values_are_keys`: no value channels, the keys in front of norm and rotation are the values.
+    `meta`: the step's device inputs.  G = 0: queries only."""
+    if w is not None:
+        _chk(w, torch.float32, "w")
     a = native.ConvQkv()
-    a.proj, a.w, a.q_norm, a.k_norm, a.rope, a.ring, a.q, a.cache, a.status = (ptr(t) for t in (proj, w, q_norm, k_norm, rope, ring, q, cache, status))
+    a.proj, a.w, a.bias, a.q_norm, a.k_norm, a.rope, a.ring, a.q, a.cache, a.status = (ptr(t) for t in (proj, w, bias, q_norm, k_norm, rope, ring, q, cache, status))
+    a.norm, a.half, a.v_from_k = QK_NORMS[norm], 1 if half else 0, 1 if values_are_keys else 0
     for n in ("state_slot", "q_start", "q_len", "kv_len", "slot_map"):
         setattr(a, n, ptr(meta[n]))
     a.ldp, a.q_stride, a.H, a.G, a.dim, a.dp, a.vdim, a.dvp, a.pairs, a.eps = proj.stride(0), q.stride(0), H, G, dim, dp, vdim, dvp, pairs, eps
     a.row_stride, a.n_slots = (cache.stride(0), cache.shape[0]) if cache is not None else (8, 0)
-    a.taps, (a.n_state, a.R, a.C), a.n_seq, a.max_q_len = w.shape[0], ring.shape, n_seq, max_q_len
-    if w.shape[1] != ring.shape[2] or not ring.is_contiguous():
-        raise ValueError("conv_qkv: convolution weights and ring differ in channels")
+    a.taps, a.C, a.n_seq, a.max_q_len = w.shape[0] if w is not None else 1, (H + G) * dim + (0 if values_are_keys else G * vdim), n_seq, max_q_len
+    a.n_state, a.R = ring.shape[:2] if ring is not None else (n_slots, a.taps)
+    if (w is not None and w.shape[1] != a.C) or (ring is not None and (ring.shape[2] != a.C or not ring.is_contiguous())):
+        raise ValueError("conv_qkv: convolution weights, ring and heads differ in channels")
     call("cuteafd_conv_qkv", ctypes.addressof(a), _f32(proj), stream())
 
 
@@ -851,18 +861,107 @@ def encode_window_maps(rows: torch.Tensor, Hkv: int, dp: int, dvp: int) -> torch
     return host.to(rows.device)
 
 
+def attn_extras(sink=None, gate=None, per_value: bool = False, keep_first: int = 0, out_scale: float = 1.0):
+    """What an attention layer has besides: a `sink` logit per head (fp32 [Hq]); `gate` logits (column view of the projection rows: one per head, or
+    `per_value` one per output value) whose sigmoid multiplies the output; the sequence's first `keep_first` keys visible behind the window; a
+    constant factor on the output."""
+    x = native.AttnExtras()
+    x.sink, x.gate, x.ldg = ptr(sink), ptr(gate), gate.stride(0) if gate is not None else 0
+    x.gate_values, x.keep_first, x.out_scale = 1 if per_value else 0, keep_first, float(out_scale)
+    return x
+
+
+def _extras(x):
+    return ctypes.addressof(x) if x is not None else None
+
+
 def window_attention(q, maps, page_table, kv_len, q_start, q_len, out, *, T, n_seq, max_q_len, Hq, Hkv, dp, dvp, dv, n_splits=1, part_o=None, part_ml=None, window=0, scale,
-                     prefill=False, status=None):
-    """Windowed paged GQA on the tensor cores (key / value heads of their own, padded widths); `prefill`: the 128-key kernel (dp + 2 dvp <= 512)."""
+                     prefill=False, extras=None, status=None):
+    """Windowed paged GQA on the tensor cores (key / value heads of their own, padded widths); `prefill`: the 128-key kernel (dp + 2 dvp <= 512);
+    `extras`: see `attn_extras`."""
     head = (ptr(q), ptr(maps), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(out))
     shape = (T, n_seq, max_q_len, q.stride(0), Hq, Hkv, dp, dvp, dv, out.stride(0), page_table.shape[1])
     if prefill:
-        call("cuteafd_window_prefill_attention", *head, *shape, window, float(scale), ptr(status), stream())
+        call("cuteafd_window_prefill_attention", *head, *shape, window, float(scale), _extras(extras), ptr(status), stream())
     else:
-        call("cuteafd_window_attention", *head, ptr(part_o), ptr(part_ml), *shape, n_splits, window, float(scale), ptr(status), stream())
+        call("cuteafd_window_attention", *head, ptr(part_o), ptr(part_ml), *shape, n_splits, window, float(scale), _extras(extras), ptr(status), stream())
 
 
-def window_attention_simt(q, cache, page_table, kv_len, q_start, q_len, out, *, T, n_seq, Hq, Hkv, dp, dvp, dv, window=0, scale, status=None):
+def window_attention_simt(q, cache, page_table, kv_len, q_start, q_len, out, *, T, n_seq, Hq, Hkv, dp, dvp, dv, window=0, scale, extras=None, status=None):
     """The same on the ordinary cores: fp32, heads wider than 256, groups of more than 128."""
     call("cuteafd_window_attention_simt", ptr(q), q.stride(0), ptr(cache), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(out), out.stride(0), T, n_seq, Hq,
-         Hkv, dp, dvp, dv, cache.stride(0), page_table.shape[1], cache.shape[0], window, float(scale), _f32(q), ptr(status), stream())
+         Hkv, dp, dvp, dv, cache.stride(0), page_table.shape[1], cache.shape[0], window, float(scale), _f32(q), _extras(extras), ptr(status), stream())
+
+
+# ------------------------------------------------------------------ hyper-connected stacks: stream boundaries, linear attention with a decay
+HYPER_EMBED, HYPER_ADD, HYPER_GATHER = 0, 1, 2
+
+
+def hyper_rows(x, W: int, rows: int, *, f32: bool, eps: float, next_in=None, gain=None, xn=None, tokens=None, table=None, pairs=None, meta=None, n_seq: int = 0, out=None,
+               mix=None, a=None, b=None, bias=None, norms=None, scales=(1.0, 1.0), routed=None, src_rows=None, status=None):
+    """Residual streams x (fp32 [., S, Wp], norms average over W) at a sub-layer boundary.
+
+    With `tokens`: every stream = table[token] + the pair table's row; `pairs` = (rows, mul_prev, mul_cur, recent): the row number is
+    (previous token * mul_prev + token * mul_cur) mod buckets, the row behind the last starts a sequence; `recent` int32 [slots, R] keeps the
+    tokens fed by position, `meta` and `n_seq` are the step's sequences.
+    With `out` / `mix`: x_t = sum_s mix[s, t] x_s + out[t] y, where y = scales[0] * (a + bias) + scales[1] * b (with `norms` = two gains, each
+    RMS-normed first) + the weighted rows of `routed` = (y, slot_row, wts, k).
+    Otherwise the rows listed in `src_rows`, collapsed by summing the streams.
+    `xn` receives the collapsed rows (weights `next_in`) RMS-normed with `gain`."""
+    _chk(x, torch.float32, "x")
+    r = native.HyperRows()
+    r.x, r.S, r.W, r.Wp, r.eps, r.status = ptr(x), x.shape[1], W, x.shape[2], eps, ptr(status)
+    r.next_in, r.gain, r.xn, r.ldn = ptr(next_in), ptr(gain), ptr(xn), xn.stride(0) if xn is not None else 0
+    mode = HYPER_GATHER
+    for t in (table, a, b):
+        if t is not None and t.shape[1] != x.shape[2]:
+            raise ValueError("hyper_rows: rows and residual streams differ in width")
+    if tokens is not None:
+        _chk(tokens, torch.int32, "tokens"); _chk(table, torch.bfloat16, "table")
+        mode, r.tokens, r.table, r.vocab = HYPER_EMBED, ptr(tokens), ptr(table), table.shape[0]
+        if pairs is not None:
+            rows_, r.mul_prev, r.mul_cur, recent = pairs
+            _chk(rows_, torch.bfloat16, "pairs"); _chk(recent, torch.int32, "recent")
+            r.pair_rows, r.buckets, r.recent, r.R, r.n_seq, r.n_state = ptr(rows_), rows_.shape[0] - 1, ptr(recent), recent.shape[1], n_seq, recent.shape[0]
+            for n in ("state_slot", "q_start", "q_len", "kv_len"):
+                setattr(r, n, ptr(meta[n]))
+    elif mix is not None:
+        mode, r.out, r.mix, r.a, r.b, r.bias = HYPER_ADD, ptr(out), ptr(mix), ptr(a), ptr(b), ptr(bias)
+        r.sa, r.sb = float(scales[0]), float(scales[1])
+        if norms is not None:
+            r.ga, r.gb = ptr(norms[0]), ptr(norms[1])
+        if routed is not None:
+            y, slot_row, wts, r.k = routed
+            r.y, r.slot_row, r.wts = ptr(y), ptr(slot_row), ptr(wts)
+    else:
+        r.src_rows = ptr(src_rows)
+    call("cuteafd_hyper_rows", ctypes.addressof(r), mode, rows, 1 if f32 else 0, stream())
+
+
+def decay_scan_arg(q, k, v, g, state, tags, ring, out, meta: dict, *, H, dim, vdim, n_seq, max_q_len, eps, rope=None, pairs=0, q_scale=1.0, k_scale=1.0, decay=None, low_rank=None,
+                   tau=1.0, norm=None, out_scale=1.0, status=None):
+    """Arguments of `decay_scan`: q, k, v, g column views of one projection buffer; `decay` fp32 [H] (constant) or `low_rank` = (a1 column view, a2 fp32
+    [H * dim, rank], bias fp32 [H * dim]): decay sigmoid(a2 a1 + bias) ** (1 / tau) per key channel; `state` [slots, 2, H, dim, vp] with `tags`
+    [slots, H, 2] (positions), `ring` [slots, depth, H, 2 dim + vp]."""
+    a = native.DecayScan()
+    for n, t in dict(q=q, k=k, v=v, g=g, rope=rope, decay=decay, norm=norm, state=state, tags=tags, ring=ring, out=out, status=status,
+                     **{m: meta[m] for m in ("state_slot", "q_start", "q_len", "kv_len")}).items():
+        setattr(a, n, ptr(t))
+    if low_rank is not None:
+        a.a1, a.a2, a.a2_b, a.rank = ptr(low_rank[0]), ptr(low_rank[1]), ptr(low_rank[2]), low_rank[1].shape[1]
+    if not q.stride(0) == k.stride(0) == v.stride(0) == g.stride(0):
+        raise ValueError("decay_scan: q, k, v and gate are columns of one buffer")
+    a.ldp, a.pairs, a.ldo, a.H, a.dim, a.vdim, a.vp, a.depth, a.n_state = q.stride(0), pairs, out.stride(0), H, dim, vdim, state.shape[-1], ring.shape[1], state.shape[0]
+    a.n_seq, a.max_q_len, a.q_scale, a.k_scale, a.inv_tau, a.eps, a.out_scale = n_seq, max_q_len, q_scale, k_scale, 1.0 / tau, eps, out_scale
+    if state.shape[1:4] != (2, H, dim) or ring.shape[2:] != (H, 2 * dim + a.vp) or tags.shape != (a.n_state, H, 2):
+        raise ValueError("decay_scan: state, tags and ring do not belong together")
+    return a
+
+
+def decay_scan(a, *, f32: bool):
+    call("cuteafd_decay_scan", ctypes.addressof(a), 1 if f32 else 0, stream())
+
+
+def silu_rows(g, u, out, rows: int):
+    """out = silu(g) * u over two projected rows (`tc_linear`'s SwiGLU epilogue as a pass of its own)."""
+    call("cuteafd_silu_rows", ptr(g), ptr(u), ptr(out), rows, g.stride(0), out.stride(0), g.shape[1], _f32(g), stream())

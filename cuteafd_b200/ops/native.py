@@ -116,9 +116,12 @@ _PROTOS = {
     "cuteafd_rglru_conv": [P, I, P],
     "cuteafd_lru_scan": [P, I, P],
     "cuteafd_glu_rows": [P, P, P, P, P, I, I, I, I, F, I, P],
-    "cuteafd_window_attention_simt": [P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P],
-    "cuteafd_window_attention": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P],
-    "cuteafd_window_prefill_attention": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P],
+    "cuteafd_window_attention_simt": [P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P],
+    "cuteafd_window_attention": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P, P],
+    "cuteafd_window_prefill_attention": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P, P],
+    "cuteafd_hyper_rows": [P, I, I, I, P],
+    "cuteafd_decay_scan": [P, I, P],
+    "cuteafd_silu_rows": [P, P, P, I, I, I, I, I, P],
     "cuteafd_tmap_encode_heads": [P, P, I, I, U64, U64],
     "cuteafd_tc_linear": [I, I, I, P, P, P, P, P, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, P, P, P, I, P, P],
 }
@@ -158,8 +161,25 @@ class NormRows(C.Structure):
 
 class ConvQkv(C.Structure):
     """`cuteafd_conv_qkv` (`CaConvQkv` of the C ABI)."""
-    _fields_ = _fields("proj w q_norm k_norm rope ring state_slot q_start q_len kv_len slot_map q cache status",
-                       "ldp q_stride row_stride n_slots H G dim dp vdim dvp pairs taps R C n_state n_seq max_q_len", "eps")
+    _fields_ = _fields("proj w bias q_norm k_norm rope ring state_slot q_start q_len kv_len slot_map q cache status",
+                       "ldp q_stride row_stride n_slots H G dim dp vdim dvp pairs taps R C n_state n_seq max_q_len norm half v_from_k", "eps")
+
+
+class AttnExtras(C.Structure):
+    """Sink, output gate, kept first keys and output factor of a windowed attention call (`CaAttnExtras` of the C ABI)."""
+    _fields_ = _fields("sink gate", "ldg gate_values keep_first", "out_scale")
+
+
+class HyperRows(C.Structure):
+    """`cuteafd_hyper_rows` (`CaHyperRows` of the C ABI)."""
+    _fields_ = (_fields("x next_in gain xn status tokens table pair_rows recent state_slot q_start q_len kv_len a b bias ga gb y slot_row wts out mix src_rows", "") +
+                [("mul_prev", L), ("mul_cur", L)] + _fields("", "S W Wp ldn vocab buckets R n_seq n_state k", "eps sa sb"))
+
+
+class DecayScan(C.Structure):
+    """`cuteafd_decay_scan` (`CaDecayScan` of the C ABI)."""
+    _fields_ = _fields("q k v g rope decay a1 a2 a2_b norm state tags ring state_slot q_start q_len kv_len out status",
+                       "ldp pairs rank ldo H dim vdim vp depth n_state n_seq max_q_len", "q_scale k_scale inv_tau eps out_scale")
 
 
 class Recurrence(C.Structure):

@@ -27,7 +27,7 @@ SUBSETS = {"latent_stack": (["runtime", "elementwise", "moe", "sampling", "tc_ge
                             ["-DCA_TC_BF16_ONLY"]),
            "hybrid_stack": (["runtime", "elementwise", "sampling", "tc_gemm", "attention_tc", "attention_mla_prefill", "hybrid_stack", "f32_linear"],
                             ["-DCA_TC_BF16_ONLY"]),
-           "hyper_stack": (["runtime", "elementwise", "moe", "sampling", "tc_gemm", "attention_tc", "attention_mla_prefill", "hybrid_stack", "hyper_stack", "f32_linear"],
+           "hyper_stack": (["runtime", "elementwise", "moe", "sampling", "tc_gemm", "attention_tc", "attention_mla_prefill", "hybrid_stack", "hyper_stack", "decay_scan", "f32_linear"],
                            ["-DCA_TC_BF16_ONLY"])}
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

@@ -65,7 +65,7 @@ class AttentionSpec:
     rope_dims: int = 0
     rope_scaling: Optional["RopeScaling"] = None
     kv_from: int = -1
-    # Kind "conv_gqa" in hyper-connected stacks, besides: `keep_first` keys of the sequence stay visible behind the window; `sink`; one norm over
+    # Kind "conv_gqa" in hyper-connected stacks, besides: no convolution with `conv_taps` 0; `keep_first` keys of the sequence stay visible behind the window; `sink`; one norm over
     # all heads of q (and of k) at once; keys that are also the values (as they leave the convolution, no value projection); biases of the
     # projections; an output gate with one number per head (`out_gate`) or, with `gate_values`, one per output value.
     keep_first: int = 0
@@ -383,7 +383,7 @@ class ModelSpec:
             elif r is not None:         # two states, the last inputs of the recurrence, two positions per head
                 vp = -(-r.vdim // 4) * 4
                 n += r.heads * (4 * (2 * r.dim * vp + depth * (2 * r.dim + vp)) + 8)
-            if a is not None and not (self.streams and a.conv_taps == 1):
+            if a is not None and a.conv_taps:
                 n += a.conv_channels * (a.conv_taps - 1 + depth) * eb
         return n
 
@@ -498,7 +498,7 @@ def vozetar_spec(n_layers: int = 6, hidden: int = 4096, heads: int = 32, kv_head
     """Vozetar at the size of a real model's layers (synthetic weights).  `mixers` repeats over the layers: P windowed attention beside retention, G
     windowed attention (values are the keys) beside gated linear attention, A full attention.  `experts` > 0: routed experts (with a shared one)
     instead of a dense feed-forward in every second layer."""
-    base = AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, rope_dims=128)
+    base = AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, rope_dims=128, conv_taps=0)
     windowed = dataclasses.replace(base, window=window, keep_first=4, rope_dims=64, rope_theta=1e6)
     rec = RecurrentSpec(kind="retention", heads=rec_heads, dim=rec_dim, vdim=rec_vdim, decay=tuple(1.0 - 2.0 ** (-5 - 7.0 * i / rec_heads) for i in range(rec_heads)), rope_dims=rec_dim)
     kinds = {"P": (dataclasses.replace(windowed, qkv_bias=True, sink=True), rec, (1.2, 1.1), False),
@@ -649,7 +649,7 @@ def _tudilix_config(cfg: dict) -> ModelSpec:
 def _vozetar_attention(i: int, m: dict, **kw) -> AttentionSpec:
     rot, mask = m.get("rot") or {"dims": 0, "base": 1e4}, m.get("mask") or {}
     a = AttentionSpec(kind="conv_gqa", n_heads=int(m["heads"]), n_kv_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]), scale=float(m["scale"]),
-                      window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0), conv_taps=int(m.get("conv") or 1), rope_dims=int(rot["dims"]),
+                      window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0), conv_taps=int(m.get("conv") or 0), rope_dims=int(rot["dims"]),
                       rope_theta=float(rot["base"]), **kw)
     if a.n_heads % a.n_kv_heads:
         raise ValueError(f"layer {i}: {a.n_heads} query heads over {a.n_kv_heads} key heads")

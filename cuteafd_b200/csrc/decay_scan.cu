@@ -1,0 +1,752 @@
+// Linear attention with a decay per head or per key channel (retention, gated linear attention): the mixers that hyper-connected stacks run
+// beside their attention.
+//   S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   out_t = norm(o_t) * silu(g_t)
+// Two forms.  Runs of up to DS_GROUP tokens (decoding, drafts, short portions; every run in the all-fp32 mode): one block per (head, sequence), the
+// state crosses HBM once for the whole group.  Longer runs in chunks of DC_TOK tokens, all chunks of all heads in parallel:
+//   chunk_states   D_c = sum_j decay(j -> end of chunk) k_j v_j^T          one tcgen05 product per (head, chunk), and the chunk's decays
+//   chunk_scan     state in front of every chunk, state behind the run     elementwise over the chunks
+//   chunk_out      o = (q k^T, decayed, causal) v + decay(start -> i) q S  three tcgen05 products per (head, chunk), output norm, gate
+// Everything that is not a projection enters the products as two bf16 terms (value and rounding error, 16 bits of mantissa together), with fp32
+// accumulators in tensor memory; the states stay fp32.  Per-channel decays are folded into q and k relative to the middle of the chunk; a chunk
+// whose decays span more than 2^80 on the way takes its scores from the ordinary cores instead.
+// (Sibling of linear_attn.cu, whose delta rule has no such form yet; the reference's linear-attention programs are AOT exports without sources.)
+#define CA_PDL_CLASS 2
+#include "stack_rows.cuh"
+#include <climits>
+
+// A state slot holds two states per head, each with the position it belongs to (-1: the zero state in front of a sequence).  A run starts from
+// the state right in front of it and leaves its last state in the other place, so a repeated step repeats its writes.  Runs of up to `depth`
+// tokens also leave their keys, decays and values (`ring`, by position): when some of them are taken back, the next run starts from the
+// earlier state and absorbs the kept ones again.
+#define DS_THREADS 256
+#define DS_GROUP 16         // tokens of one pass over the state (at least 2 depth - 1)
+#define DS_ROWS 4           // state rows a thread has in flight
+
+template <typename T>
+struct DecayScan {
+  const T* q; const T* k; const T* v; const T* g; int ldp;  // column views of the projection rows: [H * dim], [H * dim], [H * vdim], [H * vdim]
+  const float2* rope; int pairs;                            // [T, pairs], dimensions i and i + pairs turn together; null = none
+  float q_scale, k_scale;
+  const float* decay;                                       // [H] constant decays; null: alpha = sigmoid(a2 a1 + a2_b)^(1 / tau) per key channel
+  const T* a1; const float* a2; const float* a2_b;          // [rank] columns of the projection rows, [H * dim, rank], [H * dim]
+  int rank; float inv_tau;
+  const float* norm; float eps, out_scale;                  // gain of the output norm [vdim], or null
+  float* state; int* tags; float* ring;                     // [slots, 2, H, dim, vp], [slots, H, 2], [slots, depth, H, 2 dim + vp]
+  const int* state_slot; const int* q_start; const int* q_len; const int* kv_len;
+  T* out; int ldo;
+  int H, dim, vdim, vp, depth, n_state;
+  int long_from;                                            // runs of more tokens take the chunk kernels (bf16): only their replay is done here
+  float* chunk_state; float* chunk_decay;                   // [chunks, H, dim, vp], [chunks, H, dim]; a run's chunks are consecutive, from q_start / DC_TOK + sequence
+  int* status;
+};
+
+// log alpha of a channel from its logit
+__device__ __forceinline__ float log_decay(float z, float inv_tau) { return -(fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau; }
+
+struct ScanBase { int place, pos, replay; };               // where a run starts: which of the two states, its position, tokens to absorb again
+__device__ __forceinline__ ScanBase scan_base(const int* tags, int p0) {
+  if (p0 == 0) return ScanBase{0, -1, 0};
+  const int c0 = tags[0] < p0 ? tags[0] : -2, c1 = tags[1] < p0 ? tags[1] : -2;
+  const int pos = max(c0, c1);
+  return ScanBase{c1 > c0 ? 1 : 0, pos, p0 - 1 - pos};
+}
+
+struct ScanTile { float* q; float* k; float* al; float* v; float* red; float* o; };
+
+// One pass over the state for `cnt` (<= NT) tokens of the tile, the first `replay` of which only advance it; partial outputs of this thread's
+// rows stay in acc.
+template <int NT>
+__device__ __forceinline__ void scan_pass(const ScanTile& sm, const float* src, float* dst, float* mid, int cnt, int replay, int dim, int vp, int rg, int RG, int c4, float4 (&acc)[NT]) {
+#pragma unroll
+  for (int t = 0; t < NT; ++t) acc[t] = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int r0 = rg; r0 < dim; r0 += RG * DS_ROWS) {
+    float4 S[DS_ROWS];
+#pragma unroll
+    for (int i = 0; i < DS_ROWS; ++i) {
+      const int r = r0 + i * RG;
+      S[i] = src && r < dim ? *(const float4*)(src + (size_t)r * vp + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int t = 0; t < NT; ++t) {
+      if (t >= cnt) break;
+      const float4 v = *(const float4*)(sm.v + t * vp + c4);
+#pragma unroll
+      for (int i = 0; i < DS_ROWS; ++i) {
+        const int r = min(r0 + i * RG, dim - 1);
+        const float al = sm.al[t * dim + r], k = sm.k[t * dim + r], q = sm.q[t * dim + r];
+        S[i].x = fmaf(al, S[i].x, k * v.x); S[i].y = fmaf(al, S[i].y, k * v.y); S[i].z = fmaf(al, S[i].z, k * v.z); S[i].w = fmaf(al, S[i].w, k * v.w);
+        if (r0 + i * RG < dim) {
+          acc[t].x = fmaf(q, S[i].x, acc[t].x); acc[t].y = fmaf(q, S[i].y, acc[t].y); acc[t].z = fmaf(q, S[i].z, acc[t].z); acc[t].w = fmaf(q, S[i].w, acc[t].w);
+        }
+      }
+      if (mid && t == replay - 1) {
+#pragma unroll
+        for (int i = 0; i < DS_ROWS; ++i) if (r0 + i * RG < dim) *(float4*)(mid + (size_t)(r0 + i * RG) * vp + c4) = S[i];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < DS_ROWS; ++i) if (r0 + i * RG < dim) *(float4*)(dst + (size_t)(r0 + i * RG) * vp + c4) = S[i];
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(const DecayScan<T> a, int cap) {
+  pdl_launch(); pdl_wait();
+  extern __shared__ float ds_smem[];
+  __shared__ float red32[32];
+  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, dim = a.dim, vp = a.vp;
+  const int n = a.q_len[seq], p0 = a.kv_len[seq] - n, row0 = a.q_start[seq], slot = a.state_slot[seq];
+  if (n <= 0) return;
+  if (slot < 0 || slot >= a.n_state) { if (tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F2); return; }
+  ScanTile sm;
+  sm.v = ds_smem; sm.red = sm.v + cap * vp; sm.o = sm.red + 4 * DS_THREADS;            // four at a time: multiples of 4 first
+  sm.q = sm.o + vp; sm.k = sm.q + cap * dim; sm.al = sm.k + cap * dim;
+  int* tags = a.tags + ((size_t)slot * a.H + h) * 2;
+  const ScanBase b = scan_base(tags, p0);
+  if (b.pos < -1 || b.replay >= a.depth) { if (tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F3); return; }
+  const size_t one = (size_t)dim * vp;
+  float* base = a.state + (((size_t)slot * 2 + b.place) * a.H + h) * one;
+  float* last = a.state + (((size_t)slot * 2 + 1 - b.place) * a.H + h) * one;
+  const int rw = 2 * dim + vp;
+  float* ring = a.ring + ((size_t)slot * a.depth * a.H + h) * rw;           // entry of position p: + (p % depth) * H * rw
+  const int CG = vp / 4, RG = DS_THREADS / CG, c4 = (tid % CG) * 4, rg = tid / CG;
+  const bool works = rg < RG;
+  const float decay = a.decay ? a.decay[h] : 0.f;
+  const bool only_replay = n > a.long_from;
+  if (only_replay && !b.replay) return;
+
+  for (int done = 0, first = 1; first || done < n; first = 0) {
+    const int replay = first ? b.replay : 0, cnt = only_replay ? replay : min(cap, replay + n - done), fresh = cnt - replay;
+    __syncthreads();
+    for (int i = tid; i < cnt * dim; i += DS_THREADS) {
+      const int t = i / dim, r = i % dim;
+      if (t < replay) {
+        const float* e = ring + (size_t)((b.pos + 1 + t) % a.depth) * a.H * rw;
+        sm.k[i] = e[r]; sm.al[i] = e[dim + r]; sm.q[i] = 0.f;
+        continue;
+      }
+      const int row = row0 + done + t - replay;
+      const T* qr = a.q + (size_t)row * a.ldp + h * dim;
+      const T* kr = a.k + (size_t)row * a.ldp + h * dim;
+      float q = to_f(qr[r]), k = to_f(kr[r]);
+      if (a.rope && r < 2 * a.pairs) {
+        const bool lo = r < a.pairs;
+        const int pr = lo ? r : r - a.pairs, o = lo ? r + a.pairs : pr;
+        const float2 cs = a.rope[(size_t)row * a.pairs + pr];
+        const float q2 = to_f(qr[o]), k2 = to_f(kr[o]);
+        q = lo ? q * cs.x - q2 * cs.y : q * cs.x + q2 * cs.y;
+        k = lo ? k * cs.x - k2 * cs.y : k * cs.x + k2 * cs.y;
+      }
+      float al = decay;
+      if (!a.decay) {
+        float z = a.a2_b[h * dim + r];
+        const T* ar = a.a1 + (size_t)row * a.ldp;
+        const float* wr = a.a2 + (size_t)(h * dim + r) * a.rank;
+        for (int j = 0; j < a.rank; ++j) z = fmaf(wr[j], to_f(ar[j]), z);
+        al = expf(log_decay(z, a.inv_tau));
+      }
+      sm.q[i] = q * a.q_scale; sm.k[i] = k * a.k_scale; sm.al[i] = al;
+    }
+    for (int i = tid; i < cnt * vp; i += DS_THREADS) {
+      const int t = i / vp, c = i % vp;
+      if (t < replay) sm.v[i] = ring[(size_t)((b.pos + 1 + t) % a.depth) * a.H * rw + 2 * dim + c];
+      else sm.v[i] = c < a.vdim ? to_f(a.v[(size_t)(row0 + done + t - replay) * a.ldp + h * a.vdim + c]) : 0.f;
+    }
+    __syncthreads();                                        // the tile is there, and the ring entries that were needed have been read
+    if (n >= 2 && n <= a.depth) {
+      for (int i = tid; i < fresh * rw; i += DS_THREADS) {
+        const int t = i / rw, c = i % rw, s = replay + t;
+        ring[(size_t)((p0 + t) % a.depth) * a.H * rw + c] = c < dim ? sm.k[s * dim + c] : (c < 2 * dim ? sm.al[s * dim + c - dim] : sm.v[s * vp + c - 2 * dim]);
+      }
+    }
+    if (only_replay) {                                      // the state moves up to the run's start, in its own place
+      float4 acc[DS_GROUP];
+      if (works) scan_pass<DS_GROUP>(sm, b.pos >= 0 ? base : nullptr, base, nullptr, cnt, 0, dim, vp, rg, RG, c4, acc);
+      if (tid == 0) tags[b.place] = p0 - 1;
+      return;
+    }
+    const float* src = first ? (b.pos >= 0 ? base : nullptr) : last;
+    float* mid = replay ? base : nullptr;
+    // outputs of one token: sum over the row groups, norm, gate
+    auto finish = [&](int t, const float4& part) {
+      __syncthreads();
+      if (works) *(float4*)(sm.red + rg * vp + c4) = part;
+      __syncthreads();
+      float ss = 0.f;
+      for (int c = tid; c < a.vdim; c += DS_THREADS) {
+        float o = 0.f;
+        for (int g = 0; g < RG; ++g) o += sm.red[g * vp + c];
+        sm.o[c] = o;
+        ss = fmaf(o, o, ss);
+      }
+      const float inv = rsqrtf(block_sum(ss, red32) / (float)a.vdim + a.eps) * a.out_scale;
+      const size_t row = row0 + done + t - replay;
+      for (int c = tid; c < a.vdim; c += DS_THREADS) {
+        const float g = to_f(a.g[row * a.ldp + h * a.vdim + c]);
+        a.out[row * a.ldo + h * a.vdim + c] = to_t<T>(sm.o[c] * inv * (a.norm ? a.norm[c] : 1.f) * (g / (1.f + expf(-g))));
+      }
+    };
+    if (cnt == 1) {
+      float4 acc[1];
+      if (works) scan_pass<1>(sm, src, last, mid, cnt, replay, dim, vp, rg, RG, c4, acc);
+      finish(0, acc[0]);
+    } else {
+      float4 acc[DS_GROUP];
+      if (works) scan_pass<DS_GROUP>(sm, src, last, mid, cnt, replay, dim, vp, rg, RG, c4, acc);
+#pragma unroll
+      for (int t = 0; t < DS_GROUP; ++t) if (t >= replay && t < cnt) finish(t, acc[t]);
+    }
+    done += fresh;
+  }
+  if (tid == 0) {
+    tags[b.place] = b.replay ? p0 - 1 : b.pos;
+    tags[1 - b.place] = p0 + n - 1;
+  }
+}
+
+// ---------------------------------------------------------------- long runs in chunks
+#define DC_TOK 128
+#define DC_THREADS 256
+#define DC_SPAN 80.f        // most binary digits a chunk's decays may span on either side of its middle
+
+// Operand tiles: 64 columns x 128 rows in 128-byte rows, 128-byte swizzle.  DB 64-wide blocks of key dimensions; value tiles have up to 4 blocks.
+template <int DB>
+struct ChunkSmem {
+  static constexpr int TILE = 16384, HL = 2 * DB * TILE;               // an operand of key dimensions: values, then rounding errors
+  static constexpr int SMALL = 4096;                                   // vectors, barrier, flags
+  static constexpr int X = 4 * TILE;                                   // decays [128, 64 DB] fp32, then the value tiles, then state tiles
+  static constexpr int P = 4 * TILE;                                   // keys, then probabilities (two terms of two blocks), then state tiles
+  static constexpr int STATES = HL + X + SMALL, OUT = HL + P + X + SMALL;
+};
+
+struct ChunkRun { int n, p0, row, len, ci, chunks; };                  // run, first row and length of the block's chunk, its place in the scratch
+__device__ __forceinline__ bool chunk_of(const DecayScan<bf16>& a, int c, int seq, ChunkRun& r) {
+  r.n = a.q_len[seq];
+  r.chunks = (r.n + DC_TOK - 1) / DC_TOK;
+  if (r.n <= a.long_from || c >= r.chunks) return false;
+  const int row0 = a.q_start[seq];
+  r.p0 = a.kv_len[seq] - r.n; r.row = row0 + c * DC_TOK; r.len = min(DC_TOK, r.n - c * DC_TOK); r.ci = row0 / DC_TOK + seq + c;
+  return true;
+}
+
+__device__ __forceinline__ uint64_t dc_desc_mn(uint32_t saddr, uint32_t lbo) {      // MN-major, 128-byte swizzle: 64-wide blocks `lbo` bytes apart, 8-row groups 1024
+  return (uint64_t)((saddr & 0x3FFFF) >> 4) | (uint64_t)(lbo >> 4) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
+}
+__device__ __forceinline__ uint32_t dc_idesc(int n, int a_mn, int b_mn) {
+  return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)a_mn << 15) | ((uint32_t)b_mn << 16) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
+}
+// Eight values at (row, column) of a tile set whose 64-wide blocks are `block` bytes apart.
+__device__ __forceinline__ uint32_t tile_at(int row, int col, int block) { return (col >> 6) * block + row * 128 + ((((col >> 3) & 7) ^ (row & 7)) << 4); }
+__device__ __forceinline__ void put8(uint8_t* tile, uint32_t at, const float* v) {
+  uint32_t w[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) { const bf162 h = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]); w[j] = *(const uint32_t*)&h; }
+  *(uint4*)(tile + at) = make_uint4(w[0], w[1], w[2], w[3]);
+}
+// A value and what bf16 rounds off it, `lo` bytes apart.
+__device__ __forceinline__ void put8_two(uint8_t* tile, uint32_t at, int lo, const float* v) {
+  float r[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) r[j] = v[j] - __bfloat162float(__float2bfloat16(v[j]));
+  put8(tile, at, v);
+  put8(tile + lo, at, r);
+}
+
+// Eight neighbouring dimensions of a head's projected row (zero past `dim`), rotated and scaled.  `vec`: rows and rotation allow 16-byte pieces.
+__device__ __forceinline__ void head8(const bf16* row, int d0, int dim, const float2* cs, int pairs, float scale, bool vec, float* v) {
+  if (d0 >= dim) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = 0.f;
+    return;
+  }
+  if (vec) {
+    load8<bf16>(row + d0, v);
+    if (cs && d0 < 2 * pairs) {
+      const bool lo = d0 < pairs;
+      const int p0 = lo ? d0 : d0 - pairs;
+      float u[8];
+      load8<bf16>(row + (lo ? d0 + pairs : p0), u);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) { const float2 c = cs[p0 + j]; v[j] = lo ? v[j] * c.x - u[j] * c.y : v[j] * c.x + u[j] * c.y; }
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int d = d0 + j;
+      v[j] = d < dim ? to_f(row[d]) : 0.f;
+      if (cs && d < 2 * pairs) {
+        const bool lo = d < pairs;
+        const int pr = lo ? d : d - pairs;
+        const float2 c = cs[pr];
+        const float u = to_f(row[lo ? d + pairs : pr]);
+        v[j] = lo ? v[j] * c.x - u * c.y : v[j] * c.x + u * c.y;
+      }
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 8; ++j) v[j] *= scale;
+}
+
+// log2 of the chunk's per-channel decays -> X [128, DP] (zero past the run's end and past `dim`); `stage`: 8 KB.
+template <int DP>
+__device__ __forceinline__ void chunk_logs(const DecayScan<bf16>& a, int h, const ChunkRun& r, float* X, float* stage) {
+  const int tid = threadIdx.x, c = tid % DP;
+  const float b = c < a.dim ? a.a2_b[h * a.dim + c] : 0.f;
+  for (int r0 = 0; r0 < a.rank; r0 += 16) {
+    __syncthreads();
+    for (int i = tid; i < DC_TOK * 16; i += DC_THREADS) {
+      const int t = i >> 4, q = r0 + (i & 15);
+      stage[i] = t < r.len && q < a.rank ? to_f(a.a1[(size_t)(r.row + t) * a.ldp + q]) : 0.f;
+    }
+    float w[16];
+#pragma unroll
+    for (int q = 0; q < 16; ++q) w[q] = c < a.dim && r0 + q < a.rank ? a.a2[(size_t)(h * a.dim + c) * a.rank + r0 + q] : 0.f;
+    __syncthreads();
+    for (int t = tid / DP; t < DC_TOK; t += DC_THREADS / DP) {
+      float z = r0 ? X[t * DP + c] : b;
+#pragma unroll
+      for (int q = 0; q < 16; q += 4) {
+        const float4 s = *(const float4*)(stage + t * 16 + q);
+        z = fmaf(w[q], s.x, z); z = fmaf(w[q + 1], s.y, z); z = fmaf(w[q + 2], s.z, z); z = fmaf(w[q + 3], s.w, z);
+      }
+      X[t * DP + c] = r0 + 16 < a.rank ? z : (t < r.len && c < a.dim ? log_decay(z, a.inv_tau) * 1.4426950408889634f : 0.f);
+    }
+  }
+  __syncthreads();
+}
+
+__device__ __forceinline__ void load_values(const DecayScan<bf16>& a, int h, const ChunkRun& r, uint8_t* sV, int VB) {
+  const bool vec = ((a.vdim | a.ldp) & 7) == 0 && ((uintptr_t)a.v & 15) == 0;
+  for (int i = threadIdx.x; i < DC_TOK * VB * 8; i += DC_THREADS) {
+    const int t = i / (VB * 8), c0 = (i % (VB * 8)) * 8;
+    uint4 w = make_uint4(0, 0, 0, 0);
+    if (t < r.len && c0 < a.vdim) {
+      const bf16* src = a.v + (size_t)(r.row + t) * a.ldp + h * a.vdim + c0;
+      if (vec) w = *(const uint4*)src;
+      else {
+        bf16 e[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) e[j] = c0 + j < a.vdim ? src[j] : __float2bfloat16(0.f);
+        w = *(const uint4*)e;
+      }
+    }
+    *(uint4*)(sV + tile_at(t, c0, 16384)) = w;
+  }
+}
+
+__device__ __forceinline__ float decay_log2(float d) { return fmaxf(log2f(d), -1e30f); }      // (a decay of zero forgets everything but the token itself)
+
+// Barrier, tensor memory and the end of a chunk block.
+struct ChunkSync {
+  uint64_t* bar; int* abortp; uint32_t tmem; int ph; int* status;
+  // All threads: wait for the products committed last.
+  __device__ __forceinline__ void wait(int where) {
+    if (!mbar_wait_bounded(bar, ph, (volatile int*)abortp)) ca_dev_fail(status, CA_DEV_TIMEOUT_EPILOGUE, where);
+    ph ^= 1;
+    tc_fence_after();
+  }
+  __device__ __forceinline__ void publish() { fence_proxy_async_smem(); tc_fence_before(); __syncthreads(); tc_fence_after(); }
+};
+__device__ __forceinline__ ChunkSync chunk_begin(uint8_t* small, int cols, int* status) {
+  uint64_t* bar = (uint64_t*)small;
+  uint32_t* slot = (uint32_t*)(small + 8);
+  int* abortp = (int*)(small + 16);
+  if (threadIdx.x == 0) { mbar_init(bar, 1); *abortp = 0; fence_barrier_init(); }
+  if (threadIdx.x >> 5 == 1) { tmem_alloc(slot, cols); tmem_relinquish(); }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  return ChunkSync{bar, abortp, *slot, 0, status};
+}
+__device__ __forceinline__ void chunk_end(const ChunkSync& y, int cols) {
+  if (*(volatile int*)y.abortp && threadIdx.x < 32) { const uint64_t t0 = globaltimer_ns(); while (globaltimer_ns() - t0 < 200000) __nanosleep(1000); }
+  tc_fence_before();
+  __syncthreads();
+  if (threadIdx.x >> 5 == 1) tmem_dealloc(y.tmem, cols);
+}
+
+// D_c = sum_j decay(j -> end) k_j v_j^T of one head and chunk, rows of key dimensions; the decays of the whole chunk.
+template <int DB, bool GLA>
+__global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __grid_constant__ DecayScan<bf16> a) {
+  pdl_launch(); pdl_wait();
+  using Sm = ChunkSmem<DB>;
+  constexpr int DP = DB * 64;
+  extern __shared__ __align__(1024) uint8_t dc_smem[];
+  const int h = blockIdx.x, tid = threadIdx.x;
+  ChunkRun r;
+  if (!chunk_of(a, blockIdx.y, blockIdx.z, r)) return;                // block-uniform
+  if (smem_u32(dc_smem) & 1023) { if (tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F4); return; }
+  uint8_t* sK = dc_smem; uint8_t* sX = sK + Sm::HL; uint8_t* small = sX + Sm::X;
+  float* X = (float*)sX; float* rest = (float*)(small + 64); float* total = rest + DP;      // [DP] decay of the second half, of the chunk
+  ChunkSync y = chunk_begin(small, 256, a.status);
+  const int VB = (a.vp + 63) / 64;
+  const bool vec = ((a.dim | a.ldp | (a.rope ? a.pairs : 0)) & 7) == 0 && ((uintptr_t)a.k & 15) == 0;
+  const float l2 = GLA ? 0.f : decay_log2(a.decay[h]);
+  if (GLA) {
+    chunk_logs<DP>(a, h, r, X, (float*)sK);
+    if (tid < 2 * DP) {                                               // decays behind every token, within its half
+      const int c = tid % DP, half = tid / DP;
+      float s = 0.f;
+      for (int t = half * 64 + 63; t >= half * 64; --t) { const float l = X[t * DP + c]; X[t * DP + c] = s; s += l; }
+      (half ? rest : total)[c] = s;
+    }
+    __syncthreads();
+    if (tid < DP) {
+      total[tid] += rest[tid];
+      if (tid < a.dim) a.chunk_decay[((size_t)r.ci * a.H + h) * a.dim + tid] = exp2f(total[tid]);
+    }
+  } else if (tid < a.dim) {
+    a.chunk_decay[((size_t)r.ci * a.H + h) * a.dim + tid] = exp2f(l2 * (float)r.len);
+  }
+  for (int i = tid; i < DC_TOK * DB * 8; i += DC_THREADS) {
+    const int t = i / (DB * 8), d0 = (i % (DB * 8)) * 8;
+    float v[8];
+    if (t < r.len) {
+      const size_t row = r.row + t;
+      head8(a.k + row * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + row * a.pairs : nullptr, a.pairs, a.k_scale, vec, v);
+      const float f = GLA ? 0.f : exp2f(l2 * (float)(r.len - 1 - t));
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] *= GLA ? exp2f(X[t * DP + d0 + j] + (t < 64 ? rest[d0 + j] : 0.f)) : f;
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] = 0.f;
+    }
+    put8_two(sK, tile_at(t, d0, Sm::TILE), DB * Sm::TILE, v);
+  }
+  __syncthreads();                                                    // the decays have been read: values take their place
+  load_values(a, h, r, sX, VB);
+  y.publish();
+  if (tid == 0) {
+    const uint32_t id = dc_idesc(VB * 64, 1, 1);
+    for (int part = 0; part < 2; ++part)
+      for (int k = 0; k < DC_TOK / 16; ++k)
+        tc_mma_f16(y.tmem, dc_desc_mn(smem_u32(sK) + part * DB * Sm::TILE + k * 2048, Sm::TILE), dc_desc_mn(smem_u32(sX) + k * 2048, Sm::TILE), id, (part | k) ? 1u : 0u);
+    tc_commit(y.bar);
+  }
+  __syncwarp();
+  y.wait(0x6F5);
+  const int warp = tid >> 5, row = (warp & 3) * 32 + (tid & 31);
+  float* dst = a.chunk_state + (((size_t)r.ci * a.H + h) * a.dim + (row < a.dim ? row : 0)) * a.vp;
+  for (int c = (warp >> 2) * VB * 32; c < ((warp >> 2) + 1) * VB * 32; c += 16) {
+    uint32_t o[16];
+    tmem_ld_x16(y.tmem + ((uint32_t)((warp & 3) * 32) << 16) + c, o);
+    tc_wait_ld();
+    if (row < a.dim)
+#pragma unroll
+      for (int j = 0; j < 16; j += 4)
+        if (c + j < a.vp) *(uint4*)(dst + c + j) = make_uint4(o[j], o[j + 1], o[j + 2], o[j + 3]);
+  }
+  chunk_end(y, 256);
+}
+
+// The chunks' contributions become the states in front of the chunks; the state behind the run goes to the slot.
+template <bool GLA>
+__global__ void __launch_bounds__(128) chunk_scan_kernel(const DecayScan<bf16> a) {
+  pdl_launch(); pdl_wait();
+  const int h = blockIdx.y, seq = blockIdx.z, e = (blockIdx.x * 128 + threadIdx.x) * 4, one = a.dim * a.vp;
+  ChunkRun r;
+  if (!chunk_of(a, 0, seq, r) || e >= one) return;
+  const int slot = a.state_slot[seq];
+  if (slot < 0 || slot >= a.n_state) { if (e == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F2); return; }
+  const ScanBase b = scan_base(a.tags + ((size_t)slot * a.H + h) * 2, r.p0);
+  if (b.pos < -1 || b.replay) { if (e == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F3); return; }
+  float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (b.pos >= 0) S = *(const float4*)(a.state + (((size_t)slot * 2 + b.place) * a.H + h) * one + e);
+  float* D = a.chunk_state + ((size_t)r.ci * a.H + h) * one + e;
+  const float* dec = a.chunk_decay + ((size_t)r.ci * a.H + h) * a.dim + e / a.vp;
+  const size_t step = (size_t)a.H * one, dstep = (size_t)a.H * a.dim;
+  for (int c0 = 0; c0 < r.chunks; c0 += 8) {
+    float4 d[8]; float f[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = min(c0 + j, r.chunks - 1);
+      d[j] = *(const float4*)(D + c * step); f[j] = dec[c * dstep];
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (c0 + j >= r.chunks) break;
+      *(float4*)(D + (c0 + j) * step) = S;
+      S.x = fmaf(f[j], S.x, d[j].x); S.y = fmaf(f[j], S.y, d[j].y); S.z = fmaf(f[j], S.z, d[j].z); S.w = fmaf(f[j], S.w, d[j].w);
+    }
+  }
+  *(float4*)(a.state + (((size_t)slot * 2 + 1 - b.place) * a.H + h) * one + e) = S;
+}
+
+template <int DB, bool GLA>
+__global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_constant__ DecayScan<bf16> a) {
+  pdl_launch(); pdl_wait();
+  using Sm = ChunkSmem<DB>;
+  constexpr int DP = DB * 64, T = Sm::TILE;
+  extern __shared__ __align__(1024) uint8_t dc_smem[];
+  const int h = blockIdx.x, seq = blockIdx.z, tid = threadIdx.x;
+  ChunkRun r;
+  if (!chunk_of(a, blockIdx.y, seq, r)) return;                       // block-uniform
+  const int slot = a.state_slot[seq];
+  if (slot < 0 || slot >= a.n_state || (smem_u32(dc_smem) & 1023)) { if (tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F6); return; }
+  uint8_t* sQ = dc_smem; uint8_t* sP = sQ + Sm::HL; uint8_t* sX = sP + Sm::P; uint8_t* small = sX + Sm::X;
+  float* X = (float*)sX; float* mid = (float*)(small + 64); float* ssum = mid + DP;      // [DP] log2 decay up to the reference, [2, 128]
+  ChunkSync y = chunk_begin(small, 512, a.status);
+  const uint32_t O1 = 0, O2 = 256, SC = 256;                          // scores stand where the state's share is accumulated later
+  const int VB = (a.vp + 63) / 64, warp = tid >> 5, half = warp >> 2, row = (warp & 3) * 32 + (tid & 31);
+  const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
+  const bool vec = ((a.dim | a.ldp | (a.rope ? a.pairs : 0)) & 7) == 0 && (((uintptr_t)a.q | (uintptr_t)a.k) & 15) == 0;
+  const float l2 = GLA ? 0.f : decay_log2(a.decay[h]);
+  bool wide = false;                                                  // decays that span too much for a common reference
+  if (GLA) {
+    chunk_logs<DP>(a, h, r, X, (float*)sQ);
+    bool far = false;
+    if (tid < 2 * DP) {                                               // relative to the chunk's middle: in front of it up to 63 (positive), behind it (negative)
+      const int c = tid % DP;
+      float s = 0.f;
+      if (tid < DP) {
+        for (int t = 63; t >= 0; --t) { const float l = X[t * DP + c]; X[t * DP + c] = -s; s += l; }
+        mid[c] = s;
+      } else {
+        for (int t = 64; t < DC_TOK; ++t) { s += X[t * DP + c]; X[t * DP + c] = s; }
+      }
+      far = s < -DC_SPAN;
+    }
+    wide = __syncthreads_or(far);
+  }
+  for (int i = tid; i < DC_TOK * DB * 8; i += DC_THREADS) {
+    const int t = i / (DB * 8), d0 = (i % (DB * 8)) * 8;
+    float q[8], k[8];
+    if (t < r.len) {
+      const size_t gr = r.row + t;
+      const float2* cs = a.rope ? a.rope + gr * a.pairs : nullptr;
+      head8(a.q + gr * a.ldp + h * a.dim, d0, a.dim, cs, a.pairs, a.q_scale, vec, q);
+      head8(a.k + gr * a.ldp + h * a.dim, d0, a.dim, cs, a.pairs, a.k_scale, vec, k);
+      if (GLA) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const float x = X[t * DP + d0 + j];
+          if (wide) q[j] *= exp2f(x + mid[d0 + j]);                   // from the chunk's start: for the state alone
+          else { q[j] *= exp2f(x); k[j] *= exp2f(-x); }
+        }
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) q[j] = k[j] = 0.f;
+    }
+    put8_two(sQ, tile_at(t, d0, T), DB * T, q);
+    if (!wide) put8_two(sP, tile_at(t, d0, T), DB * T, k);
+  }
+  float sc[64];                                                       // this thread's scores: its row, keys [64 half, + 64)
+  if (!wide) {
+    y.publish();
+    if (tid == 0) {
+      const uint32_t id = dc_idesc(DC_TOK, 0, 0), q0 = smem_u32(sQ), k0 = smem_u32(sP);
+      for (int part = 0; part < 3; ++part) {                          // value x value, value x error, error x value
+        const uint32_t qa = q0 + (part == 2 ? DB * T : 0), kb = k0 + (part == 1 ? DB * T : 0);
+        for (int b = 0; b < DB; ++b)
+          for (int k = 0; k < 4; ++k) tc_mma_f16(y.tmem + SC, umma_desc_sw128(qa + b * T) + 2 * k, umma_desc_sw128(kb + b * T) + 2 * k, id, (part | b | k) ? 1u : 0u);
+      }
+      tc_commit(y.bar);
+    }
+    __syncwarp();
+    load_values(a, h, r, sX, VB);                                     // (every thread is past its decays)
+    y.wait(0x6F7);
+#pragma unroll
+    for (int c = 0; c < 64; c += 16) {
+      uint32_t o[16];
+      tmem_ld_x16(y.tmem + lanes + SC + half * 64 + c, o);
+      tc_wait_ld();
+#pragma unroll
+      for (int j = 0; j < 16; ++j) {
+        const int back = row - (half * 64 + c + j);
+        sc[c + j] = back < 0 ? 0.f : __uint_as_float(o[j]) * (GLA ? 1.f : exp2f(l2 * (float)back));
+      }
+    }
+  } else {
+    // pairwise, from the projected rows: the decays between two tokens as the difference of their sums
+    for (int j = 0; j < 64; ++j) {
+      const int key = half * 64 + j;
+      float s = 0.f;
+      if (key <= row && row < r.len) {
+        const size_t gq = r.row + row, gk = r.row + key;
+        for (int d0 = 0; d0 < a.dim; d0 += 8) {
+          float q[8], k[8];
+          head8(a.q + gq * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + gq * a.pairs : nullptr, a.pairs, a.q_scale, vec, q);
+          head8(a.k + gk * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + gk * a.pairs : nullptr, a.pairs, a.k_scale, vec, k);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) s = fmaf(q[e] * k[e], exp2f(X[row * DP + d0 + e] - X[key * DP + d0 + e]), s);
+        }
+      }
+      sc[j] = s;
+    }
+    __syncthreads();                                                  // the decays have been read
+    load_values(a, h, r, sX, VB);
+  }
+  tc_fence_before();
+  __syncthreads();                                                    // keys and scores have been read
+  tc_fence_after();
+#pragma unroll
+  for (int c = 0; c < 64; c += 8) put8_two(sP, tile_at(row, half * 64 + c, T), 2 * T, sc + c);
+  y.publish();
+  if (tid == 0) {
+    const uint32_t id = dc_idesc(VB * 64, 0, 1), p0 = smem_u32(sP), v0 = smem_u32(sX);
+    for (int part = 0; part < 2; ++part)
+      for (int k = 0; k < DC_TOK / 16; ++k)
+        tc_mma_f16(y.tmem + O1, umma_desc_sw128(p0 + part * 2 * T + (k >> 2) * T) + 2 * (k & 3), dc_desc_mn(v0 + k * 2048, T), id, (part | k) ? 1u : 0u);
+    tc_commit(y.bar);
+  }
+  __syncwarp();
+  y.wait(0x6F8);
+  // the state in front of the chunk takes the place of probabilities and values
+  const float* S = a.chunk_state + ((size_t)r.ci * a.H + h) * a.dim * a.vp;
+  for (int i = tid; i < DP * VB * 8; i += DC_THREADS) {
+    const int d = i / (VB * 8), c0 = (i % (VB * 8)) * 8;
+    float v[8];
+    const float f = GLA && !wide ? exp2f(mid[d]) : 1.f;
+#pragma unroll
+    for (int j = 0; j < 8; j += 4) {
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (d < a.dim && c0 + j < a.vp) x = *(const float4*)(S + (size_t)d * a.vp + c0 + j);
+      v[j] = x.x * f; v[j + 1] = x.y * f; v[j + 2] = x.z * f; v[j + 3] = x.w * f;
+    }
+    float e[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) e[j] = v[j] - __bfloat162float(__float2bfloat16(v[j]));
+    const uint32_t at = tile_at(d, c0, DP * 128);
+    put8(sP, at, v);
+    put8(sX, at, e);
+  }
+  y.publish();
+  if (tid == 0) {
+    const uint32_t id = dc_idesc(VB * 64, 0, 1), q0 = smem_u32(sQ);
+    for (int part = 0; part < 3; ++part) {
+      const uint32_t qa = q0 + (part == 2 ? DB * T : 0), sb = smem_u32(part == 1 ? sX : sP);
+      for (int k = 0; k < DP / 16; ++k) tc_mma_f16(y.tmem + O2, umma_desc_sw128(qa + (k >> 2) * T) + 2 * (k & 3), dc_desc_mn(sb + k * 2048, DP * 128), id, (part | k) ? 1u : 0u);
+    }
+    tc_commit(y.bar);
+  }
+  __syncwarp();
+  y.wait(0x6F9);
+  // output norm and gate: a thread has its token's columns [half * VB * 32, + VB * 32)
+  const float f2 = GLA ? 1.f : exp2f(l2 * (float)(row + 1));
+  const int c_lo = half * VB * 32, c_hi = c_lo + VB * 32;
+  float ss = 0.f;
+  for (int c = c_lo; c < c_hi; c += 16) {
+    uint32_t o[16], s[16];
+    tmem_ld_x16(y.tmem + lanes + O1 + c, o);
+    tmem_ld_x16(y.tmem + lanes + O2 + c, s);
+    tc_wait_ld();
+#pragma unroll
+    for (int j = 0; j < 16; ++j) { const float v = fmaf(f2, __uint_as_float(s[j]), __uint_as_float(o[j])); ss = fmaf(v, v, ss); }       // columns past vdim are zero
+  }
+  ssum[half * 128 + row] = ss;
+  __syncthreads();
+  const float inv = rsqrtf((ssum[row] + ssum[128 + row]) / (float)a.vdim + a.eps) * a.out_scale;
+  const bool vout = ((a.vdim | a.ldp | a.ldo) & 7) == 0 && (((uintptr_t)a.g | (uintptr_t)a.out) & 15) == 0;
+  const size_t gr = r.row + min(row, r.len - 1);
+  const bf16* g = a.g + gr * a.ldp + h * a.vdim;
+  bf16* dst = a.out + gr * a.ldo + h * a.vdim;
+  for (int c = c_lo; c < c_hi; c += 16) {
+    uint32_t o[16], s[16];
+    tmem_ld_x16(y.tmem + lanes + O1 + c, o);
+    tmem_ld_x16(y.tmem + lanes + O2 + c, s);
+    tc_wait_ld();
+    if (row >= r.len) continue;
+#pragma unroll
+    for (int p = 0; p < 16; p += 8) {
+      if (c + p >= a.vdim) continue;
+      float gv[8], v[8];
+      if (vout) load8<bf16>(g + c + p, gv);
+      else
+#pragma unroll
+        for (int j = 0; j < 8; ++j) gv[j] = c + p + j < a.vdim ? to_f(g[c + p + j]) : 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float x = fmaf(f2, __uint_as_float(s[p + j]), __uint_as_float(o[p + j])) * inv;
+        v[j] = x * (a.norm && c + p + j < a.vdim ? a.norm[c + p + j] : 1.f) * __fdividef(gv[j], 1.f + __expf(-fmaxf(gv[j], -80.f)));
+      }
+      if (vout) store8<bf16>(dst + c + p, v);
+      else
+#pragma unroll
+        for (int j = 0; j < 8; ++j) if (c + p + j < a.vdim) dst[c + p + j] = __float2bfloat16(v[j]);
+    }
+  }
+  if (tid == 0 && (int)blockIdx.y == r.chunks - 1) {                  // no other block of this launch reads the tags
+    int* tags = a.tags + ((size_t)slot * a.H + h) * 2;
+    const ScanBase b = scan_base(tags, r.p0);
+    tags[b.place] = b.pos; tags[1 - b.place] = r.p0 + r.n - 1;
+  }
+  chunk_end(y, 512);
+}
+
+// ---------------------------------------------------------------- C ABI
+struct CaDecayScan {
+  const void* q; const void* k; const void* v; const void* g; const void* rope; const float* decay; const void* a1; const float* a2; const float* a2_b; const float* norm;
+  float* state; int* tags; float* ring; const int* state_slot; const int* q_start; const int* q_len; const int* kv_len; void* out; float* chunk_state; float* chunk_decay; int* status;
+  int ldp, pairs, rank, ldo, H, dim, vdim, vp, depth, n_state, n_seq, max_q_len, T, chunks; float q_scale, k_scale, inv_tau, eps, out_scale;
+};
+
+template <typename T>
+static DecayScan<T> decay_scan_args(const CaDecayScan* c, bool chunked) {
+  return DecayScan<T>{(const T*)c->q, (const T*)c->k, (const T*)c->v, (const T*)c->g, c->ldp, (const float2*)c->rope, c->pairs, c->q_scale, c->k_scale, c->decay, (const T*)c->a1, c->a2,
+                      c->a2_b, c->rank, c->inv_tau, c->norm, c->eps, c->out_scale, c->state, c->tags, c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len, (T*)c->out, c->ldo,
+                      c->H, c->dim, c->vdim, c->vp, c->depth, c->n_state, chunked ? DS_GROUP : INT_MAX, c->chunk_state, c->chunk_decay, c->status};
+}
+
+template <typename K>
+static int dynamic_smem(K kern, int bytes, bool (&done)[64]) {
+  int dev = 0; cudaGetDevice(&dev);
+  if (!done[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return ca_cuda(e, "cudaFuncSetAttribute(decay_scan)");
+    done[dev & 63] = true;
+  }
+  return CA_OK;
+}
+
+template <typename T>
+static int decay_scan_launch(const CaDecayScan* c, bool chunked, cudaStream_t s) {
+  const int longest = chunked ? DS_GROUP : c->max_q_len;
+  const int cap = longest + c->depth - 1 < DS_GROUP ? longest + c->depth - 1 : DS_GROUP;
+  const size_t smem = ((size_t)cap * (3 * c->dim + c->vp) + 4 * DS_THREADS + c->vp) * sizeof(float);
+  static bool attr_set[64] = {false};
+  const int rc = dynamic_smem(decay_scan_kernel<T>, 200 * 1024, attr_set);
+  if (rc) return rc;
+  CA_REQUIRE(smem <= 200 * 1024, "decay_scan: heads of %d x %d do not fit shared memory", c->dim, c->vdim);
+  CA_LAUNCH_PDL((decay_scan_kernel<T>), dim3(c->H, c->n_seq), DS_THREADS, smem, s, decay_scan_args<T>(c, chunked), cap);
+  CA_CHECK_LAUNCH("decay_scan");
+  return CA_OK;
+}
+
+template <int DB, bool GLA>
+static int chunk_launch(const CaDecayScan* c, cudaStream_t s) {
+  const DecayScan<bf16> a = decay_scan_args<bf16>(c, true);
+  const int chunks = (c->max_q_len + DC_TOK - 1) / DC_TOK;
+  const dim3 grid(c->H, chunks, c->n_seq);
+  static bool states_set[64] = {false}, out_set[64] = {false};
+  int rc = dynamic_smem(chunk_states_kernel<DB, GLA>, ChunkSmem<DB>::STATES, states_set);
+  if (!rc) rc = dynamic_smem(chunk_out_kernel<DB, GLA>, ChunkSmem<DB>::OUT, out_set);
+  if (rc) return rc;
+  CA_LAUNCH_PDL((chunk_states_kernel<DB, GLA>), grid, DC_THREADS, ChunkSmem<DB>::STATES, s, a);
+  CA_CHECK_LAUNCH("decay_scan chunk states");
+  CA_LAUNCH_PDL((chunk_scan_kernel<GLA>), dim3((c->dim * c->vp / 4 + 127) / 128, c->H, c->n_seq), 128, 0, s, a);
+  CA_CHECK_LAUNCH("decay_scan chunk scan");
+  CA_LAUNCH_PDL((chunk_out_kernel<DB, GLA>), grid, DC_THREADS, ChunkSmem<DB>::OUT, s, a);
+  CA_CHECK_LAUNCH("decay_scan chunk outputs");
+  return CA_OK;
+}
+
+// Whether the chunk kernels take a step's long runs.
+static bool chunkable(const CaDecayScan* c, int f32) { return !f32 && c->chunk_state && c->chunk_decay && c->dim <= 128 && c->vdim <= 256 && c->max_q_len > DS_GROUP; }
+
+extern "C" int cuteafd_decay_scan(const CaDecayScan* c, int f32, cudaStream_t s) {
+  CA_REQUIRE(c && c->q && c->k && c->v && c->g && c->state && c->tags && c->ring && c->state_slot && c->q_start && c->q_len && c->kv_len && c->out, "decay_scan: null argument");
+  CA_REQUIRE(c->decay || (c->a1 && c->a2 && c->a2_b && c->rank >= 1), "decay_scan: neither constant decays nor a projection of them");
+  CA_REQUIRE(c->H >= 1 && c->dim >= 1 && c->dim <= 512 && c->vdim >= 1 && c->vp % 4 == 0 && c->vp >= c->vdim && c->vp <= 4 * DS_THREADS, "decay_scan: heads of %d x %d (at most 512 x %d)", c->dim, c->vdim, 4 * DS_THREADS);
+  CA_REQUIRE(c->pairs >= 0 && 2 * c->pairs <= c->dim && (c->pairs == 0 || c->rope) && c->depth >= 1 && 2 * c->depth - 1 <= DS_GROUP && c->n_state >= 1, "decay_scan: bad rotation or depth");
+  CA_REQUIRE(c->ldo >= c->H * c->vdim && c->ldp >= c->H * c->vdim && c->ldp >= c->H * c->dim, "decay_scan: rows too short");
+  if (c->n_seq <= 0 || c->max_q_len <= 0) return CA_OK;
+  CA_REQUIRE(c->n_seq <= 65535, "decay_scan: too many sequences");
+  if (f32) return decay_scan_launch<float>(c, false, s);
+  const bool chunked = chunkable(c, f32);
+  CA_REQUIRE(!chunked || (c->chunks >= c->T / DC_TOK + c->n_seq + 1 && c->vp <= 256 && c->max_q_len <= 65535 * DC_TOK), "decay_scan: room for %d chunks is too little", c->chunks);
+  const int rc = decay_scan_launch<bf16>(c, chunked, s);
+  if (rc || !chunked) return rc;
+  if (c->dim <= 64) return c->decay ? chunk_launch<1, false>(c, s) : chunk_launch<1, true>(c, s);
+  return c->decay ? chunk_launch<2, false>(c, s) : chunk_launch<2, true>(c, s);
+}

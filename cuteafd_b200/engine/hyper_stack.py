@@ -9,7 +9,7 @@ program on the hybrid stacks' attention; every arrow between two products is one
   mixer          h -> queries | keys | values | gate | linear mixer's queries, keys, values, gate, decay input       one product
                  conv_qkv: bias, convolution, norm, rotation -> query rows, paged cache rows, ring of inputs
                  paged attention (window, kept first keys, sink, gate) -> columns of the output operand
-                 decay_scan: rotation, decays, recurrence, output norm, gate -> the columns behind them
+                 decay_scan: rotation, decays, recurrence, output norm, gate -> the columns behind them (prompts: four launches, in chunks)
                  -> W_o          (one product over both, or one each where the outputs are normalised before they are added)
   streams <- constants x (streams, mixer), h = norm(collapsed streams)                                               one launch
   feed-forward   h -> SwiGLU in the product's epilogue -> W_down;  routed: router -> selection + packing -> gather -> grouped products
@@ -17,7 +17,7 @@ program on the hybrid stacks' attention; every arrow between two products is one
   rows that need logits: sum of the streams -> final norm -> head
 
 Keys and values live in the paged cache like the hybrid stacks'.  What a sequence carries besides sits in its state slot: convolution inputs and
-fed tokens in rings addressed by position, the linear mixers' states in two places tagged with their positions (see `csrc/hyper_stack.cu`).  A
+fed tokens in rings addressed by position, the linear mixers' states in two places tagged with their positions (see `csrc/decay_scan.cu`).  A
 slot needs no reset, a repeated step repeats its writes, and up to `state_depth` tokens can be taken back by continuing from an earlier
 position.  With fp32 weights (`QuantSpec.dense = "f32"`) the same program runs entirely in fp32.
 """
@@ -26,7 +26,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from ..config import BlockSpec, MoESpec
+from ..config import BlockSpec, MoESpec, RecurrentSpec
 from ..models.hybrid_stack import rope_key
 from ..models.hyper_stack import HyperLayer, check_blocks
 from ..models.latent_stack import up
@@ -54,6 +54,14 @@ class HyperLane(HybridLane):
                 d["r"], d["r_act"] = self._operand(cap, K2)
             return d
         return self.get(("mix", a.n_heads, a.head_dim, a.v_head_dim, K2, b.merge_norm, n_in), make)
+
+
+    def scan_chunks(self, r: RecurrentSpec) -> tuple | None:
+        """Scratch of a linear mixer's long runs (none in the all-fp32 mode, for decode-sized lanes and for heads the chunk kernels do not take)."""
+        if self.eng.f32 or self.cap <= 16 or r.dim > 128 or r.vdim > 256:
+            return None
+        n, f32 = self.cap // ops.SCAN_CHUNK + self.eng.max_seqs + 1, dict(dtype=torch.float32, device=self.dev)
+        return self.get(("scan", r.heads, r.dim, r.vdim), lambda: (torch.zeros(n, r.heads, r.dim, up(r.vdim, 4), **f32), torch.zeros(n, r.heads, r.dim, **f32)))
 
 
 class HyperStackEngine(HybridStackEngine):
@@ -138,9 +146,9 @@ class HyperStackEngine(HybridStackEngine):
                                      n_seq=sh.n_seq, max_q_len=sh.max_q_len, eps=self.spec.rms_eps, rope=L.rope[rope_key(r)] if r.rope_dims else None,
                                      pairs=r.rope_dims // 2, q_scale=r.dim ** -0.5 if gla else 1.0, k_scale=1.0 if gla else r.dim ** -0.5, decay=lw.lin_decay,
                                      low_rank=(column("a1"), lw.lin_a2, lw.lin_a2_b) if gla else None, tau=r.tau, norm=lw.lin_norm,
-                                     out_scale=b.merge_scales[1] if merged else 1.0, status=self.status)
+                                     out_scale=b.merge_scales[1] if merged else 1.0, chunks=L.scan_chunks(r), T=T, status=self.status)
             ops.decay_scan(arg, f32=self.f32)
-            self.launches_per_step += 1
+            self.launches_per_step += 4 if arg.chunks and sh.max_q_len > 16 else 1
         self._dense(lw.wo, m["o_act"], L.mix, T)
         if not b.merge_norm:
             return dict(a=L.mix, bias=lw.wo_b)

@@ -119,7 +119,7 @@ def read_hyper_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
             lw[f"w{k}"] = get(f"{p}.{k}", sizes[k], W)
             if a.qkv_bias:
                 lw[f"{k}_b"] = get(f"{p}.{k}.b", sizes[k])
-            if a.conv_taps > 1:
+            if a.conv_taps:
                 lw[f"{k}_conv"] = get(f"{p}.{k}.conv", sizes[k], a.conv_taps)
             if a.qk_norm_whole and k != "v":
                 lw[f"{k}_norm"] = get(f"{p}.{k}.norm", sizes[k])

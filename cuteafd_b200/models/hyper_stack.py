@@ -67,8 +67,8 @@ def check_blocks(spec: ModelSpec):
         a, r, m = b.attn, b.rec, b.moe
         if a is None or (r is not None and r.kind not in ("retention", "gla")):
             raise ValueError(f"layer {i}: hyper-connected stacks have attention, alone or beside retention or gated linear attention")
-        if not 1 <= a.conv_taps <= 16 or max(a.head_dim, a.v_head_dim) > 256:
-            raise ValueError(f"layer {i}: convolutions of 1 to 16 taps and heads of up to 256 dimensions (got {a.conv_taps} and {a.head_dim} / {a.v_head_dim})")
+        if not 0 <= a.conv_taps <= 16 or max(a.head_dim, a.v_head_dim) > 256:
+            raise ValueError(f"layer {i}: convolutions of up to 16 taps and heads of up to 256 dimensions (got {a.conv_taps} and {a.head_dim} / {a.v_head_dim})")
         if r is not None and (r.dim > 512 or r.vdim > 1024):
             raise ValueError(f"layer {i}: recurrent heads of up to 512 x 1024 (got {r.dim} x {r.vdim})")
         if m is not None and (m.n_experts > 512 or m.top_k > 16 or m.n_group > 32):
@@ -106,7 +106,7 @@ def hyper_weights_from_masters(spec: ModelSpec, masters: dict, device) -> HyperW
                 wo = torch.cat([_pad(wo, W, K1), _pad(lw["r_o"], W, K2)], 1)
         out = HyperLayer(attn_norm=vec(lw["norm1"], Wp), ffn_norm=None, wqkv=None, wo=mat(wo, Wp, up(wo.shape[1], 8)), columns=cols, w_in=mat(w, rows, Wp), wo2=wo2,
                          hc1=tuple(f32(t) for t in lw["hc1"]))
-        if a.conv_taps > 1:
+        if a.conv_taps:
             out.conv = f32(torch.cat([lw[f"{k}_conv"] for k in qkv]).float().T)
         if a.qkv_bias:
             out.qkv_b = f32(torch.cat([lw[f"{k}_b"] for k in qkv]))
@@ -169,7 +169,7 @@ def hyper_weights_random(spec: ModelSpec, device, seed: int = 1) -> HyperWeights
         H, G, K1 = a.n_heads, a.n_kv_heads, up(a.n_heads * a.v_head_dim, 8)
         K2 = up(r.heads * r.vdim, 8) if r is not None else 0
         out = HyperLayer(attn_norm=ones(W), ffn_norm=None, wqkv=None, wo=R(1, W, K1 if b.merge_norm else K1 + K2), columns=cols, w_in=R(1, rows, W), hc1=constants())
-        out.conv = nrm(a.conv_taps, a.conv_channels, std=0.5) if a.conv_taps > 1 else None
+        out.conv = nrm(a.conv_taps, a.conv_channels, std=0.5) if a.conv_taps else None
         out.qkv_b = nrm(a.conv_channels, std=0.1) if a.qkv_bias else None
         out.wo_b = nrm(W, std=0.1) if a.out_bias else None
         out.sink = nrm(H, std=1.0) if a.sink else None

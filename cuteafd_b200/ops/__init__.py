@@ -895,6 +895,7 @@ def window_attention_simt(q, cache, page_table, kv_len, q_start, q_len, out, *, 
 
 # ------------------------------------------------------------------ hyper-connected stacks: stream boundaries, linear attention with a decay
 HYPER_EMBED, HYPER_ADD, HYPER_GATHER = 0, 1, 2
+SCAN_CHUNK = 128            # tokens of a chunk of `decay_scan`'s long form
 
 
 def hyper_rows(x, W: int, rows: int, *, f32: bool, eps: float, next_in=None, gain=None, xn=None, tokens=None, table=None, pairs=None, meta=None, n_seq: int = 0, out=None,
@@ -939,11 +940,16 @@ def hyper_rows(x, W: int, rows: int, *, f32: bool, eps: float, next_in=None, gai
 
 
 def decay_scan_arg(q, k, v, g, state, tags, ring, out, meta: dict, *, H, dim, vdim, n_seq, max_q_len, eps, rope=None, pairs=0, q_scale=1.0, k_scale=1.0, decay=None, low_rank=None,
-                   tau=1.0, norm=None, out_scale=1.0, status=None):
+                   tau=1.0, norm=None, out_scale=1.0, chunks=None, T: int = 0, status=None):
     """Arguments of `decay_scan`: q, k, v, g column views of one projection buffer; `decay` fp32 [H] (constant) or `low_rank` = (a1 column view, a2 fp32
     [H * dim, rank], bias fp32 [H * dim]): decay sigmoid(a2 a1 + bias) ** (1 / tau) per key channel; `state` [slots, 2, H, dim, vp] with `tags`
-    [slots, H, 2] (positions), `ring` [slots, depth, H, 2 dim + vp]."""
+    [slots, H, 2] (positions), `ring` [slots, depth, H, 2 dim + vp].  `chunks` = (states [n, H, dim, vp], decays [n, H, dim]) fp32 scratch with which
+    long runs of a step of `T` rows take the chunk kernels (bf16, heads of up to 128 x 256; n >= T / SCAN_CHUNK + sequences + 1)."""
     a = native.DecayScan()
+    if chunks is not None:
+        a.chunk_state, a.chunk_decay, a.chunks, a.T = ptr(chunks[0]), ptr(chunks[1]), chunks[0].shape[0], T
+        if chunks[0].shape[1:] != (H, dim, state.shape[-1]) or chunks[1].shape != chunks[0].shape[:3]:
+            raise ValueError("decay_scan: chunk scratch of another geometry")
     for n, t in dict(q=q, k=k, v=v, g=g, rope=rope, decay=decay, norm=norm, state=state, tags=tags, ring=ring, out=out, status=status,
                      **{m: meta[m] for m in ("state_slot", "q_start", "q_len", "kv_len")}).items():
         setattr(a, n, ptr(t))

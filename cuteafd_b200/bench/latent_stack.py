@@ -198,8 +198,9 @@ def kernel_table(eng, sh, pairs: int, kv_rows: int, prefill: bool, peaks: dict, 
 
 
 # ------------------------------------------------------------------ workloads
-def measure(spec: ModelSpec, *, batches, context: int, chunks, steps: int, warmup: int, kernels: bool, peaks: dict, roofline=roofline) -> dict:
-    """`roofline`: what a launch has to compute and move, for the per-launch table (windowed layers see the last `attn.window` keys only)."""
+def measure(spec: ModelSpec, *, batches, context: int, chunks, steps: int, warmup: int, kernels: bool, peaks: dict, roofline=roofline, at_position=lambda eng, pos: None) -> dict:
+    """`roofline`: what a launch has to compute and move, for the per-launch table (windowed layers see the last `attn.window` keys only).
+    `at_position(engine, position)`: puts recurrent states that know their position in front of the step's first one."""
     win = spec.attn.window or 1 << 40
     seen = lambda lo, hi: sum(min(p + 1, win) for p in range(lo, hi))            # (query, key) pairs of positions [lo, hi)
     longest = max([context] + [c for _, c in chunks])
@@ -211,6 +212,7 @@ def measure(spec: ModelSpec, *, batches, context: int, chunks, steps: int, warmu
     for b in batches:
         pool = PagePool(pages)
         gen, sh = decode_shape(eng, b, context, pool)
+        at_position(eng, context)
         ms = timed(lambda: eng.run(sh), steps, warmup)
         launches += eng.launches_per_step * steps
         row = {"batch": b, "context": context, "ms_per_step": round(ms, 4), "tokens_per_s": round(b / ms * 1e3, 1), "us_per_layer_run": round(1e3 * ms / res["layer_runs"], 1),
@@ -221,6 +223,7 @@ def measure(spec: ModelSpec, *, batches, context: int, chunks, steps: int, warmu
         eng.check_status()
     for chunk, ctx in chunks:
         s, sh = prefill_shape(eng, chunk, ctx, PagePool(pages))
+        at_position(eng, ctx - chunk)
         ms = timed(lambda: eng.run(sh, use_graph=False), max(3, steps // 4), warmup)
         launches += eng.launches_per_step * max(3, steps // 4)
         row = {"chunk": chunk, "context": ctx, "ms_per_chunk": round(ms, 3), "tokens_per_s": round(chunk / ms * 1e3, 1), "us_per_layer_run": round(1e3 * ms / res["layer_runs"], 1)}

@@ -494,10 +494,10 @@ def tudilix_spec(n_layers: int = 12, hidden: int = 4096, heads: int = 32, kv_hea
 
 
 def vozetar_spec(n_layers: int = 6, hidden: int = 4096, heads: int = 32, kv_heads: int = 4, ff: int = 12288, window: int = 2048, rec_heads: int = 16, rec_dim: int = 128,
-                 rec_vdim: int = 256, experts: int = 0, expert_ff: int = 1536, streams: int = 4, mixers: str = "PGA") -> ModelSpec:
+                 rec_vdim: int = 256, experts: int = 0, expert_ff: int = 1536, streams: int = 4, mixers: str = "PGA", moe_every: int = 2) -> ModelSpec:
     """Vozetar at the size of a real model's layers (synthetic weights).  `mixers` repeats over the layers: P windowed attention beside retention, G
     windowed attention (values are the keys) beside gated linear attention, A full attention.  `experts` > 0: routed experts (with a shared one)
-    instead of a dense feed-forward in every second layer."""
+    instead of a dense feed-forward in every `moe_every`-th layer."""
     base = AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, rope_dims=128, conv_taps=0)
     windowed = dataclasses.replace(base, window=window, keep_first=4, rope_dims=64, rope_theta=1e6)
     rec = RecurrentSpec(kind="retention", heads=rec_heads, dim=rec_dim, vdim=rec_vdim, decay=tuple(1.0 - 2.0 ** (-5 - 7.0 * i / rec_heads) for i in range(rec_heads)), rope_dims=rec_dim)
@@ -509,7 +509,7 @@ def vozetar_spec(n_layers: int = 6, hidden: int = 4096, heads: int = 32, kv_head
     blocks = []
     for i in range(n_layers):
         attn, r, scales, norm = kinds[mixers[i % len(mixers)]]
-        routed = moe is not None and i % 2 == 1
+        routed = moe is not None and i % moe_every == moe_every - 1
         blocks.append(BlockSpec(attn, moe if routed else None, r, None if routed else DenseFfnSpec(ff, activation="silu_glu"), scales, norm))
     return ModelSpec(name="vozetar-shape", family="vozetar", vocab=65536, hidden=hidden, n_layers=n_layers, rms_eps=1e-5, attn=blocks[0].attn, moe=moe or MoESpec(n_experts=0, n_shared=0),
                      quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(blocks), streams=streams, pair_table=PairTableSpec(65521, 31, 17))

@@ -4,7 +4,7 @@
 // Two forms.  Runs of up to DS_GROUP tokens (decoding, drafts, short portions; every run in the all-fp32 mode): one block per (head, sequence), the
 // state crosses HBM once for the whole group.  Longer runs in chunks of DC_TOK tokens, all chunks of all heads in parallel:
 //   chunk_states   D_c = sum_j decay(j -> end of chunk) k_j v_j^T          one tcgen05 product per (head, chunk), and the chunk's decays
-//   chunk_scan     state in front of every chunk, state behind the run     elementwise over the chunks
+//   chunk_scan     state in front of every chunk (operand tiles), state behind the run     elementwise over the chunks
 //   chunk_out      o = (q k^T, decayed, causal) v + decay(start -> i) q S  three tcgen05 products per (head, chunk), output norm, gate
 // Everything that is not a projection enters the products as two bf16 terms (value and rounding error, 16 bits of mantissa together), with fp32
 // accumulators in tensor memory; the states stay fp32.  Per-channel decays are folded into q and k relative to the middle of the chunk; a chunk
@@ -20,7 +20,6 @@
 // earlier state and absorbs the kept ones again.
 #define DS_THREADS 256
 #define DS_GROUP 16         // tokens of one pass over the state (at least 2 depth - 1)
-#define DS_ROWS 4           // state rows a thread has in flight
 
 template <typename T>
 struct DecayScan {
@@ -36,7 +35,10 @@ struct DecayScan {
   T* out; int ldo;
   int H, dim, vdim, vp, depth, n_state;
   int long_from;                                            // runs of more tokens take the chunk kernels (bf16): only their replay is done here
-  float* chunk_state; float* chunk_decay;                   // [chunks, H, dim, vp], [chunks, H, dim]; a run's chunks are consecutive, from q_start / DC_TOK + sequence
+  // scratch of the long form, a run's chunks consecutive from q_start / DC_TOK + sequence: contributions [chunks, H, dim, vp], factors
+  // [chunks, H, 2 dim + 1] (decays of the chunk; what puts the state in front of it on the scale of the chunk's queries; whether the decays span too
+  // much for a common reference), states as operand tiles [chunks, H, tile set]
+  float* chunk_state; float* chunk_decay; uint8_t* chunk_tiles;
   int* status;
 };
 
@@ -51,12 +53,16 @@ __device__ __forceinline__ ScanBase scan_base(const int* tags, int p0) {
   return ScanBase{c1 > c0 ? 1 : 0, pos, p0 - 1 - pos};
 }
 
-struct ScanTile { float* q; float* k; float* al; float* v; float* red; float* o; };
+struct ScanTile {
+  float* q; float* k; float* al; float* v; float* red; float* o;
+  __device__ __forceinline__ ScanTile from(int t, int dim, int vp) const { return ScanTile{q + t * dim, k + t * dim, al + t * dim, v + t * vp, red, o}; }
+};
 
 // One pass over the state for `cnt` (<= NT) tokens of the tile, the first `replay` of which only advance it; partial outputs of this thread's
 // rows stay in acc.
 template <int NT>
 __device__ __forceinline__ void scan_pass(const ScanTile& sm, const float* src, float* dst, float* mid, int cnt, int replay, int dim, int vp, int rg, int RG, int c4, float4 (&acc)[NT]) {
+  constexpr int DS_ROWS = NT == 1 ? 8 : 4;                   // state rows a thread has in flight
 #pragma unroll
   for (int t = 0; t < NT; ++t) acc[t] = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int r0 = rg; r0 < dim; r0 += RG * DS_ROWS) {
@@ -89,8 +95,9 @@ __device__ __forceinline__ void scan_pass(const ScanTile& sm, const float* src, 
   }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(const DecayScan<T> a, int cap) {
+// NT: tokens of a pass over the state.  One: decoding (several blocks per SM; kept rows of a drafted step are absorbed one by one in place).
+template <typename T, int NT>
+__global__ void __launch_bounds__(DS_THREADS, NT == 1 ? 3 : 1) decay_scan_kernel(const DecayScan<T> a, int cap) {
   pdl_launch(); pdl_wait();
   extern __shared__ float ds_smem[];
   __shared__ float red32[32];
@@ -160,8 +167,9 @@ __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(const DecayScan<
       }
     }
     if (only_replay) {                                      // the state moves up to the run's start, in its own place
-      float4 acc[DS_GROUP];
-      if (works) scan_pass<DS_GROUP>(sm, b.pos >= 0 ? base : nullptr, base, nullptr, cnt, 0, dim, vp, rg, RG, c4, acc);
+      float4 acc[NT];
+      if (works)
+        for (int t = 0; t < cnt; t += NT) scan_pass<NT>(sm.from(t, dim, vp), t || b.pos >= 0 ? base : nullptr, base, nullptr, min(NT, cnt - t), 0, dim, vp, rg, RG, c4, acc);
       if (tid == 0) tags[b.place] = p0 - 1;
       return;
     }
@@ -186,15 +194,17 @@ __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(const DecayScan<
         a.out[row * a.ldo + h * a.vdim + c] = to_t<T>(sm.o[c] * inv * (a.norm ? a.norm[c] : 1.f) * (g / (1.f + expf(-g))));
       }
     };
-    if (cnt == 1) {
-      float4 acc[1];
-      if (works) scan_pass<1>(sm, src, last, mid, cnt, replay, dim, vp, rg, RG, c4, acc);
-      finish(0, acc[0]);
+    float4 acc[NT];
+    if constexpr (NT == 1) {
+      for (int t = 0; t < cnt; ++t) {                       // a thread's part of the state is its own: no barrier between the passes
+        const float* from = t == 0 ? src : (t <= replay ? base : last);
+        if (works) scan_pass<1>(sm.from(t, dim, vp), from, t < replay ? base : last, nullptr, 1, 0, dim, vp, rg, RG, c4, acc);
+        if (t >= replay) finish(t, acc[0]);
+      }
     } else {
-      float4 acc[DS_GROUP];
-      if (works) scan_pass<DS_GROUP>(sm, src, last, mid, cnt, replay, dim, vp, rg, RG, c4, acc);
+      if (works) scan_pass<NT>(sm, src, last, mid, cnt, replay, dim, vp, rg, RG, c4, acc);
 #pragma unroll
-      for (int t = 0; t < DS_GROUP; ++t) if (t >= replay && t < cnt) finish(t, acc[t]);
+      for (int t = 0; t < NT; ++t) if (t >= replay && t < cnt) finish(t, acc[t]);
     }
     done += fresh;
   }
@@ -206,7 +216,8 @@ __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(const DecayScan<
 
 // ---------------------------------------------------------------- long runs in chunks
 #define DC_TOK 128
-#define DC_THREADS 256
+#define DC_THREADS 512
+#define DC_PARTS (DC_THREADS / 128)      // threads that share a row of an accumulator
 #define DC_SPAN 80.f        // most binary digits a chunk's decays may span on either side of its middle
 
 // Operand tiles: 64 columns x 128 rows in 128-byte rows, 128-byte swizzle.  DB 64-wide blocks of key dimensions; value tiles have up to 4 blocks.
@@ -252,6 +263,18 @@ __device__ __forceinline__ void put8_two(uint8_t* tile, uint32_t at, int lo, con
   put8(tile + lo, at, r);
 }
 
+// Rows no kernel of the launch writes: loads may pass the stores in front of them.
+__device__ __forceinline__ void ldg8(const bf16* p, float* v) {
+  const uint4 q = __ldg((const uint4*)p);
+  const bf162* h = (const bf162*)&q;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) { const float2 f = __bfloat1622float2(h[j]); v[2 * j] = f.x; v[2 * j + 1] = f.y; }
+}
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
 // Eight neighbouring dimensions of a head's projected row (zero past `dim`), rotated and scaled.  `vec`: rows and rotation allow 16-byte pieces.
 __device__ __forceinline__ void head8(const bf16* row, int d0, int dim, const float2* cs, int pairs, float scale, bool vec, float* v) {
   if (d0 >= dim) {
@@ -260,14 +283,18 @@ __device__ __forceinline__ void head8(const bf16* row, int d0, int dim, const fl
     return;
   }
   if (vec) {
-    load8<bf16>(row + d0, v);
+    ldg8(row + d0, v);
     if (cs && d0 < 2 * pairs) {
       const bool lo = d0 < pairs;
       const int p0 = lo ? d0 : d0 - pairs;
       float u[8];
-      load8<bf16>(row + (lo ? d0 + pairs : p0), u);
+      ldg8(row + (lo ? d0 + pairs : p0), u);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) { const float2 c = cs[p0 + j]; v[j] = lo ? v[j] * c.x - u[j] * c.y : v[j] * c.x + u[j] * c.y; }
+      for (int j = 0; j < 8; j += 2) {                      // (cosine, sine) of two pairs
+        const float4 c = __ldg((const float4*)(cs + p0 + j));
+        v[j] = lo ? v[j] * c.x - u[j] * c.y : v[j] * c.x + u[j] * c.y;
+        v[j + 1] = lo ? v[j + 1] * c.z - u[j + 1] * c.w : v[j + 1] * c.z + u[j + 1] * c.w;
+      }
     }
   } else {
 #pragma unroll
@@ -319,18 +346,14 @@ __device__ __forceinline__ void load_values(const DecayScan<bf16>& a, int h, con
   const bool vec = ((a.vdim | a.ldp) & 7) == 0 && ((uintptr_t)a.v & 15) == 0;
   for (int i = threadIdx.x; i < DC_TOK * VB * 8; i += DC_THREADS) {
     const int t = i / (VB * 8), c0 = (i % (VB * 8)) * 8;
-    uint4 w = make_uint4(0, 0, 0, 0);
-    if (t < r.len && c0 < a.vdim) {
-      const bf16* src = a.v + (size_t)(r.row + t) * a.ldp + h * a.vdim + c0;
-      if (vec) w = *(const uint4*)src;
-      else {
-        bf16 e[8];
+    const bool in = t < r.len && c0 < a.vdim;
+    const bf16* src = a.v + (size_t)(r.row + t) * a.ldp + h * a.vdim + c0;
+    uint8_t* dst = sV + tile_at(t, c0, 16384);
+    if (in && vec) { cp_async16(dst, src); continue; }      // (the caller waits for the copies)
+    float e[8];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) e[j] = c0 + j < a.vdim ? src[j] : __float2bfloat16(0.f);
-        w = *(const uint4*)e;
-      }
-    }
-    *(uint4*)(sV + tile_at(t, c0, 16384)) = w;
+    for (int j = 0; j < 8; ++j) e[j] = in && c0 + j < a.vdim ? to_f(src[j]) : 0.f;
+    put8(dst, 0, e);
   }
 }
 
@@ -377,27 +400,30 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __gri
   if (!chunk_of(a, blockIdx.y, blockIdx.z, r)) return;                // block-uniform
   if (smem_u32(dc_smem) & 1023) { if (tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F4); return; }
   uint8_t* sK = dc_smem; uint8_t* sX = sK + Sm::HL; uint8_t* small = sX + Sm::X;
-  float* X = (float*)sX; float* rest = (float*)(small + 64); float* total = rest + DP;      // [DP] decay of the second half, of the chunk
+  float* X = (float*)sX; float* rest = (float*)(small + 64); float* first = rest + DP;      // [DP] log2 decays of the second and the first half
   ChunkSync y = chunk_begin(small, 256, a.status);
   const int VB = (a.vp + 63) / 64;
   const bool vec = ((a.dim | a.ldp | (a.rope ? a.pairs : 0)) & 7) == 0 && ((uintptr_t)a.k & 15) == 0;
   const float l2 = GLA ? 0.f : decay_log2(a.decay[h]);
+  float* factors = a.chunk_decay + ((size_t)r.ci * a.H + h) * (2 * a.dim + 1);
   if (GLA) {
     chunk_logs<DP>(a, h, r, X, (float*)sK);
+    bool far = false;
     if (tid < 2 * DP) {                                               // decays behind every token, within its half
       const int c = tid % DP, half = tid / DP;
       float s = 0.f;
       for (int t = half * 64 + 63; t >= half * 64; --t) { const float l = X[t * DP + c]; X[t * DP + c] = s; s += l; }
-      (half ? rest : total)[c] = s;
+      (half ? rest : first)[c] = s;
+      far = s < -DC_SPAN;
     }
-    __syncthreads();
-    if (tid < DP) {
-      total[tid] += rest[tid];
-      if (tid < a.dim) a.chunk_decay[((size_t)r.ci * a.H + h) * a.dim + tid] = exp2f(total[tid]);
-    }
-  } else if (tid < a.dim) {
-    a.chunk_decay[((size_t)r.ci * a.H + h) * a.dim + tid] = exp2f(l2 * (float)r.len);
+    const bool wide = __syncthreads_or(far);
+    if (tid == 0) factors[2 * a.dim] = wide ? 1.f : 0.f;
+    if (tid < a.dim) { factors[tid] = exp2f(first[tid] + rest[tid]); factors[a.dim + tid] = wide ? 1.f : exp2f(first[tid]); }
+  } else {
+    load_values(a, h, r, sX, VB);
+    if (tid < a.dim) { factors[tid] = exp2f(l2 * (float)r.len); factors[a.dim + tid] = 1.f; }
   }
+#pragma unroll 4
   for (int i = tid; i < DC_TOK * DB * 8; i += DC_THREADS) {
     const int t = i / (DB * 8), d0 = (i % (DB * 8)) * 8;
     float v[8];
@@ -413,8 +439,11 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __gri
     }
     put8_two(sK, tile_at(t, d0, Sm::TILE), DB * Sm::TILE, v);
   }
-  __syncthreads();                                                    // the decays have been read: values take their place
-  load_values(a, h, r, sX, VB);
+  if (GLA) {
+    __syncthreads();                                                  // the decays have been read: values take their place
+    load_values(a, h, r, sX, VB);
+  }
+  cp_async_wait();
   y.publish();
   if (tid == 0) {
     const uint32_t id = dc_idesc(VB * 64, 1, 1);
@@ -427,7 +456,8 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __gri
   y.wait(0x6F5);
   const int warp = tid >> 5, row = (warp & 3) * 32 + (tid & 31);
   float* dst = a.chunk_state + (((size_t)r.ci * a.H + h) * a.dim + (row < a.dim ? row : 0)) * a.vp;
-  for (int c = (warp >> 2) * VB * 32; c < ((warp >> 2) + 1) * VB * 32; c += 16) {
+  constexpr int PW = 64 / DC_PARTS;                                   // columns of a 64-wide block that a thread takes
+  for (int c = (warp >> 2) * VB * PW; c < ((warp >> 2) + 1) * VB * PW; c += 16) {
     uint32_t o[16];
     tmem_ld_x16(y.tmem + ((uint32_t)((warp & 3) * 32) << 16) + c, o);
     tc_wait_ld();
@@ -439,8 +469,9 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __gri
   chunk_end(y, 256);
 }
 
-// The chunks' contributions become the states in front of the chunks; the state behind the run goes to the slot.
-template <bool GLA>
+// The chunks' contributions become the states in front of the chunks, as the operand tiles (values, then rounding errors) of the output kernel; the
+// state behind the run goes to the slot.
+template <int DB>
 __global__ void __launch_bounds__(128) chunk_scan_kernel(const DecayScan<bf16> a) {
   pdl_launch(); pdl_wait();
   const int h = blockIdx.y, seq = blockIdx.z, e = (blockIdx.x * 128 + threadIdx.x) * 4, one = a.dim * a.vp;
@@ -452,20 +483,27 @@ __global__ void __launch_bounds__(128) chunk_scan_kernel(const DecayScan<bf16> a
   if (b.pos < -1 || b.replay) { if (e == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F3); return; }
   float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
   if (b.pos >= 0) S = *(const float4*)(a.state + (((size_t)slot * 2 + b.place) * a.H + h) * one + e);
-  float* D = a.chunk_state + ((size_t)r.ci * a.H + h) * one + e;
-  const float* dec = a.chunk_decay + ((size_t)r.ci * a.H + h) * a.dim + e / a.vp;
-  const size_t step = (size_t)a.H * one, dstep = (size_t)a.H * a.dim;
+  const int row = e / a.vp, col = e % a.vp, half = (a.vp + 63) / 64 * DB * 64 * 128;
+  const float* D = a.chunk_state + ((size_t)r.ci * a.H + h) * one + e;
+  const float* dec = a.chunk_decay + ((size_t)r.ci * a.H + h) * (2 * a.dim + 1) + row;
+  uint8_t* tile = a.chunk_tiles + ((size_t)r.ci * a.H + h) * 2 * half + tile_at(row, col, DB * 64 * 128) + (col & 7) * 2;
+  const size_t step = (size_t)a.H * one, dstep = (size_t)a.H * (2 * a.dim + 1), tstep = (size_t)a.H * 2 * half;
   for (int c0 = 0; c0 < r.chunks; c0 += 8) {
-    float4 d[8]; float f[8];
+    float4 d[8]; float f[8], m[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const int c = min(c0 + j, r.chunks - 1);
-      d[j] = *(const float4*)(D + c * step); f[j] = dec[c * dstep];
+      d[j] = __ldg((const float4*)(D + c * step)); f[j] = __ldg(dec + c * dstep); m[j] = __ldg(dec + c * dstep + a.dim);
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       if (c0 + j >= r.chunks) break;
-      *(float4*)(D + (c0 + j) * step) = S;
+      const float v[4] = {S.x * m[j], S.y * m[j], S.z * m[j], S.w * m[j]};
+      float lo[4];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) lo[q] = v[q] - __bfloat162float(__float2bfloat16(v[q]));
+      store4<bf16>((bf16*)(tile + (c0 + j) * tstep), v);
+      store4<bf16>((bf16*)(tile + (c0 + j) * tstep + half), lo);
       S.x = fmaf(f[j], S.x, d[j].x); S.y = fmaf(f[j], S.y, d[j].y); S.z = fmaf(f[j], S.z, d[j].z); S.w = fmaf(f[j], S.w, d[j].w);
     }
   }
@@ -484,17 +522,21 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
   const int slot = a.state_slot[seq];
   if (slot < 0 || slot >= a.n_state || (smem_u32(dc_smem) & 1023)) { if (tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F6); return; }
   uint8_t* sQ = dc_smem; uint8_t* sP = sQ + Sm::HL; uint8_t* sX = sP + Sm::P; uint8_t* small = sX + Sm::X;
-  float* X = (float*)sX; float* mid = (float*)(small + 64); float* ssum = mid + DP;      // [DP] log2 decay up to the reference, [2, 128]
+  float* X = (float*)sX; float* mid = (float*)(small + 64); float* ssum = mid + DP;      // [DP] log2 decay up to the reference, [DC_PARTS, 128]
+  uint64_t* tiles_bar = (uint64_t*)(small + 32);
+  if (tid == 0) mbar_init(tiles_bar, 1);
   ChunkSync y = chunk_begin(small, 512, a.status);
   const uint32_t O1 = 0, O2 = 256, SC = 256;                          // scores stand where the state's share is accumulated later
-  const int VB = (a.vp + 63) / 64, warp = tid >> 5, half = warp >> 2, row = (warp & 3) * 32 + (tid & 31);
+  constexpr int KW = DC_TOK / DC_PARTS, PW = 64 / DC_PARTS;             // keys, and columns of a 64-wide block of values, that a thread takes of its row
+  const int VB = (a.vp + 63) / 64, warp = tid >> 5, part = warp >> 2, row = (warp & 3) * 32 + (tid & 31);
   const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
   const bool vec = ((a.dim | a.ldp | (a.rope ? a.pairs : 0)) & 7) == 0 && (((uintptr_t)a.q | (uintptr_t)a.k) & 15) == 0;
   const float l2 = GLA ? 0.f : decay_log2(a.decay[h]);
   bool wide = false;                                                  // decays that span too much for a common reference
+  if (!GLA) load_values(a, h, r, sX, VB);
   if (GLA) {
     chunk_logs<DP>(a, h, r, X, (float*)sQ);
-    bool far = false;
+    wide = a.chunk_decay[((size_t)r.ci * a.H + h) * (2 * a.dim + 1) + 2 * a.dim] != 0.f;
     if (tid < 2 * DP) {                                               // relative to the chunk's middle: in front of it up to 63 (positive), behind it (negative)
       const int c = tid % DP;
       float s = 0.f;
@@ -504,10 +546,10 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
       } else {
         for (int t = 64; t < DC_TOK; ++t) { s += X[t * DP + c]; X[t * DP + c] = s; }
       }
-      far = s < -DC_SPAN;
     }
-    wide = __syncthreads_or(far);
+    __syncthreads();
   }
+#pragma unroll 2
   for (int i = tid; i < DC_TOK * DB * 8; i += DC_THREADS) {
     const int t = i / (DB * 8), d0 = (i % (DB * 8)) * 8;
     float q[8], k[8];
@@ -531,7 +573,7 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
     put8_two(sQ, tile_at(t, d0, T), DB * T, q);
     if (!wide) put8_two(sP, tile_at(t, d0, T), DB * T, k);
   }
-  float sc[64];                                                       // this thread's scores: its row, keys [64 half, + 64)
+  float sc[KW];                                                       // this thread's scores: its row, keys [part * KW, + KW)
   if (!wide) {
     y.publish();
     if (tid == 0) {
@@ -544,23 +586,23 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
       tc_commit(y.bar);
     }
     __syncwarp();
-    load_values(a, h, r, sX, VB);                                     // (every thread is past its decays)
+    if (GLA) load_values(a, h, r, sX, VB);                            // (every thread is past its decays)
     y.wait(0x6F7);
 #pragma unroll
-    for (int c = 0; c < 64; c += 16) {
+    for (int c = 0; c < KW; c += 16) {
       uint32_t o[16];
-      tmem_ld_x16(y.tmem + lanes + SC + half * 64 + c, o);
+      tmem_ld_x16(y.tmem + lanes + SC + part * KW + c, o);
       tc_wait_ld();
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
-        const int back = row - (half * 64 + c + j);
+        const int back = row - (part * KW + c + j);
         sc[c + j] = back < 0 ? 0.f : __uint_as_float(o[j]) * (GLA ? 1.f : exp2f(l2 * (float)back));
       }
     }
   } else {
     // pairwise, from the projected rows: the decays between two tokens as the difference of their sums
-    for (int j = 0; j < 64; ++j) {
-      const int key = half * 64 + j;
+    for (int j = 0; j < KW; ++j) {
+      const int key = part * KW + j;
       float s = 0.f;
       if (key <= row && row < r.len) {
         const size_t gq = r.row + row, gk = r.row + key;
@@ -581,7 +623,8 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
   __syncthreads();                                                    // keys and scores have been read
   tc_fence_after();
 #pragma unroll
-  for (int c = 0; c < 64; c += 8) put8_two(sP, tile_at(row, half * 64 + c, T), 2 * T, sc + c);
+  for (int c = 0; c < KW; c += 8) put8_two(sP, tile_at(row, part * KW + c, T), 2 * T, sc + c);
+  cp_async_wait();
   y.publish();
   if (tid == 0) {
     const uint32_t id = dc_idesc(VB * 64, 0, 1), p0 = smem_u32(sP), v0 = smem_u32(sX);
@@ -593,26 +636,13 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
   __syncwarp();
   y.wait(0x6F8);
   // the state in front of the chunk takes the place of probabilities and values
-  const float* S = a.chunk_state + ((size_t)r.ci * a.H + h) * a.dim * a.vp;
-  for (int i = tid; i < DP * VB * 8; i += DC_THREADS) {
-    const int d = i / (VB * 8), c0 = (i % (VB * 8)) * 8;
-    float v[8];
-    const float f = GLA && !wide ? exp2f(mid[d]) : 1.f;
-#pragma unroll
-    for (int j = 0; j < 8; j += 4) {
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (d < a.dim && c0 + j < a.vp) x = *(const float4*)(S + (size_t)d * a.vp + c0 + j);
-      v[j] = x.x * f; v[j + 1] = x.y * f; v[j + 2] = x.z * f; v[j + 3] = x.w * f;
-    }
-    float e[8];
-#pragma unroll
-    for (int j = 0; j < 8; ++j) e[j] = v[j] - __bfloat162float(__float2bfloat16(v[j]));
-    const uint32_t at = tile_at(d, c0, DP * 128);
-    put8(sP, at, v);
-    put8(sX, at, e);
-  }
-  y.publish();
   if (tid == 0) {
+    const uint32_t bytes = VB * DP * 128;
+    const uint8_t* S = a.chunk_tiles + ((size_t)r.ci * a.H + h) * 2 * bytes;
+    mbar_expect_tx(tiles_bar, 2 * bytes);
+    bulk_load_1d(sP, S, bytes, tiles_bar);
+    bulk_load_1d(sX, S + bytes, bytes, tiles_bar);
+    if (!mbar_wait_bounded(tiles_bar, 0, (volatile int*)y.abortp)) ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, 0x6FA);
     const uint32_t id = dc_idesc(VB * 64, 0, 1), q0 = smem_u32(sQ);
     for (int part = 0; part < 3; ++part) {
       const uint32_t qa = q0 + (part == 2 ? DB * T : 0), sb = smem_u32(part == 1 ? sX : sP);
@@ -621,10 +651,32 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
     tc_commit(y.bar);
   }
   __syncwarp();
+  // the gates arrive under these products: a thread has its token's columns [c_lo, c_hi)
+  const int c_lo = part * VB * PW, c_hi = c_lo + VB * PW;
+  const bool vout = ((a.vdim | a.ldp | a.ldo) & 7) == 0 && (((uintptr_t)a.g | (uintptr_t)a.out) & 15) == 0;
+  const size_t gr = r.row + min(row, r.len - 1);
+  const bf16* g = a.g + gr * a.ldp + h * a.vdim;
+  bf16* dst = a.out + gr * a.ldo + h * a.vdim;
+  constexpr int NG = 4 * PW / 8;
+  uint4 gates[NG];
+#pragma unroll
+  for (int p = 0; p < NG; ++p) {
+    const int c = c_lo + p * 8;
+    if (c >= c_hi || c >= a.vdim) gates[p] = make_uint4(0, 0, 0, 0);
+    else if (vout) gates[p] = __ldg((const uint4*)(g + c));
+    else {
+      bf16 e[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) e[j] = c + j < a.vdim ? g[c + j] : __float2bfloat16(0.f);
+      uint32_t w[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) { const bf162 b2 = __halves2bfloat162(e[2 * j], e[2 * j + 1]); w[j] = *(const uint32_t*)&b2; }
+      gates[p] = make_uint4(w[0], w[1], w[2], w[3]);
+    }
+  }
   y.wait(0x6F9);
-  // output norm and gate: a thread has its token's columns [half * VB * 32, + VB * 32)
+  // output norm and gate
   const float f2 = GLA ? 1.f : exp2f(l2 * (float)(row + 1));
-  const int c_lo = half * VB * 32, c_hi = c_lo + VB * 32;
   float ss = 0.f;
   for (int c = c_lo; c < c_hi; c += 16) {
     uint32_t o[16], s[16];
@@ -634,14 +686,16 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
 #pragma unroll
     for (int j = 0; j < 16; ++j) { const float v = fmaf(f2, __uint_as_float(s[j]), __uint_as_float(o[j])); ss = fmaf(v, v, ss); }       // columns past vdim are zero
   }
-  ssum[half * 128 + row] = ss;
+  ssum[part * 128 + row] = ss;
   __syncthreads();
-  const float inv = rsqrtf((ssum[row] + ssum[128 + row]) / (float)a.vdim + a.eps) * a.out_scale;
-  const bool vout = ((a.vdim | a.ldp | a.ldo) & 7) == 0 && (((uintptr_t)a.g | (uintptr_t)a.out) & 15) == 0;
-  const size_t gr = r.row + min(row, r.len - 1);
-  const bf16* g = a.g + gr * a.ldp + h * a.vdim;
-  bf16* dst = a.out + gr * a.ldo + h * a.vdim;
-  for (int c = c_lo; c < c_hi; c += 16) {
+  ss = 0.f;
+#pragma unroll
+  for (int p = 0; p < DC_PARTS; ++p) ss += ssum[p * 128 + row];
+  const float inv = rsqrtf(ss / (float)a.vdim + a.eps) * a.out_scale;
+#pragma unroll
+  for (int b = 0; b < NG / 2; ++b) {
+    const int c = c_lo + b * 16;
+    if (c >= c_hi) break;                                             // block-uniform
     uint32_t o[16], s[16];
     tmem_ld_x16(y.tmem + lanes + O1 + c, o);
     tmem_ld_x16(y.tmem + lanes + O2 + c, s);
@@ -650,15 +704,14 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
 #pragma unroll
     for (int p = 0; p < 16; p += 8) {
       if (c + p >= a.vdim) continue;
-      float gv[8], v[8];
-      if (vout) load8<bf16>(g + c + p, gv);
-      else
-#pragma unroll
-        for (int j = 0; j < 8; ++j) gv[j] = c + p + j < a.vdim ? to_f(g[c + p + j]) : 0.f;
+      const bf162* gp = (const bf162*)&gates[b * 2 + p / 8];
+      float v[8];
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
+        const float2 g2 = __bfloat1622float2(gp[j / 2]);
+        const float gv = j & 1 ? g2.y : g2.x;
         const float x = fmaf(f2, __uint_as_float(s[p + j]), __uint_as_float(o[p + j])) * inv;
-        v[j] = x * (a.norm && c + p + j < a.vdim ? a.norm[c + p + j] : 1.f) * __fdividef(gv[j], 1.f + __expf(-fmaxf(gv[j], -80.f)));
+        v[j] = x * (a.norm && c + p + j < a.vdim ? __ldg(a.norm + c + p + j) : 1.f) * __fdividef(gv, 1.f + __expf(-fmaxf(gv, -80.f)));
       }
       if (vout) store8<bf16>(dst + c + p, v);
       else
@@ -677,7 +730,7 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
 // ---------------------------------------------------------------- C ABI
 struct CaDecayScan {
   const void* q; const void* k; const void* v; const void* g; const void* rope; const float* decay; const void* a1; const float* a2; const float* a2_b; const float* norm;
-  float* state; int* tags; float* ring; const int* state_slot; const int* q_start; const int* q_len; const int* kv_len; void* out; float* chunk_state; float* chunk_decay; int* status;
+  float* state; int* tags; float* ring; const int* state_slot; const int* q_start; const int* q_len; const int* kv_len; void* out; float* chunk_state; float* chunk_decay; void* chunk_tiles; int* status;
   int ldp, pairs, rank, ldo, H, dim, vdim, vp, depth, n_state, n_seq, max_q_len, T, chunks; float q_scale, k_scale, inv_tau, eps, out_scale;
 };
 
@@ -685,7 +738,7 @@ template <typename T>
 static DecayScan<T> decay_scan_args(const CaDecayScan* c, bool chunked) {
   return DecayScan<T>{(const T*)c->q, (const T*)c->k, (const T*)c->v, (const T*)c->g, c->ldp, (const float2*)c->rope, c->pairs, c->q_scale, c->k_scale, c->decay, (const T*)c->a1, c->a2,
                       c->a2_b, c->rank, c->inv_tau, c->norm, c->eps, c->out_scale, c->state, c->tags, c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len, (T*)c->out, c->ldo,
-                      c->H, c->dim, c->vdim, c->vp, c->depth, c->n_state, chunked ? DS_GROUP : INT_MAX, c->chunk_state, c->chunk_decay, c->status};
+                      c->H, c->dim, c->vdim, c->vp, c->depth, c->n_state, chunked ? DS_GROUP : INT_MAX, c->chunk_state, c->chunk_decay, (uint8_t*)c->chunk_tiles, c->status};
 }
 
 template <typename K>
@@ -699,16 +752,16 @@ static int dynamic_smem(K kern, int bytes, bool (&done)[64]) {
   return CA_OK;
 }
 
-template <typename T>
+template <typename T, int NT>
 static int decay_scan_launch(const CaDecayScan* c, bool chunked, cudaStream_t s) {
   const int longest = chunked ? DS_GROUP : c->max_q_len;
   const int cap = longest + c->depth - 1 < DS_GROUP ? longest + c->depth - 1 : DS_GROUP;
   const size_t smem = ((size_t)cap * (3 * c->dim + c->vp) + 4 * DS_THREADS + c->vp) * sizeof(float);
   static bool attr_set[64] = {false};
-  const int rc = dynamic_smem(decay_scan_kernel<T>, 200 * 1024, attr_set);
+  const int rc = dynamic_smem(decay_scan_kernel<T, NT>, 200 * 1024, attr_set);
   if (rc) return rc;
   CA_REQUIRE(smem <= 200 * 1024, "decay_scan: heads of %d x %d do not fit shared memory", c->dim, c->vdim);
-  CA_LAUNCH_PDL((decay_scan_kernel<T>), dim3(c->H, c->n_seq), DS_THREADS, smem, s, decay_scan_args<T>(c, chunked), cap);
+  CA_LAUNCH_PDL((decay_scan_kernel<T, NT>), dim3(c->H, c->n_seq), DS_THREADS, smem, s, decay_scan_args<T>(c, chunked), cap);
   CA_CHECK_LAUNCH("decay_scan");
   return CA_OK;
 }
@@ -724,7 +777,7 @@ static int chunk_launch(const CaDecayScan* c, cudaStream_t s) {
   if (rc) return rc;
   CA_LAUNCH_PDL((chunk_states_kernel<DB, GLA>), grid, DC_THREADS, ChunkSmem<DB>::STATES, s, a);
   CA_CHECK_LAUNCH("decay_scan chunk states");
-  CA_LAUNCH_PDL((chunk_scan_kernel<GLA>), dim3((c->dim * c->vp / 4 + 127) / 128, c->H, c->n_seq), 128, 0, s, a);
+  CA_LAUNCH_PDL((chunk_scan_kernel<DB>), dim3((c->dim * c->vp / 4 + 127) / 128, c->H, c->n_seq), 128, 0, s, a);
   CA_CHECK_LAUNCH("decay_scan chunk scan");
   CA_LAUNCH_PDL((chunk_out_kernel<DB, GLA>), grid, DC_THREADS, ChunkSmem<DB>::OUT, s, a);
   CA_CHECK_LAUNCH("decay_scan chunk outputs");
@@ -732,7 +785,7 @@ static int chunk_launch(const CaDecayScan* c, cudaStream_t s) {
 }
 
 // Whether the chunk kernels take a step's long runs.
-static bool chunkable(const CaDecayScan* c, int f32) { return !f32 && c->chunk_state && c->chunk_decay && c->dim <= 128 && c->vdim <= 256 && c->max_q_len > DS_GROUP; }
+static bool chunkable(const CaDecayScan* c, int f32) { return !f32 && c->chunk_state && c->chunk_decay && c->chunk_tiles && c->dim <= 128 && c->vdim <= 256 && c->max_q_len > DS_GROUP; }
 
 extern "C" int cuteafd_decay_scan(const CaDecayScan* c, int f32, cudaStream_t s) {
   CA_REQUIRE(c && c->q && c->k && c->v && c->g && c->state && c->tags && c->ring && c->state_slot && c->q_start && c->q_len && c->kv_len && c->out, "decay_scan: null argument");
@@ -742,10 +795,11 @@ extern "C" int cuteafd_decay_scan(const CaDecayScan* c, int f32, cudaStream_t s)
   CA_REQUIRE(c->ldo >= c->H * c->vdim && c->ldp >= c->H * c->vdim && c->ldp >= c->H * c->dim, "decay_scan: rows too short");
   if (c->n_seq <= 0 || c->max_q_len <= 0) return CA_OK;
   CA_REQUIRE(c->n_seq <= 65535, "decay_scan: too many sequences");
-  if (f32) return decay_scan_launch<float>(c, false, s);
+  if (f32) return c->max_q_len == 1 ? decay_scan_launch<float, 1>(c, false, s) : decay_scan_launch<float, DS_GROUP>(c, false, s);
+  if (c->max_q_len == 1) return decay_scan_launch<bf16, 1>(c, false, s);
   const bool chunked = chunkable(c, f32);
   CA_REQUIRE(!chunked || (c->chunks >= c->T / DC_TOK + c->n_seq + 1 && c->vp <= 256 && c->max_q_len <= 65535 * DC_TOK), "decay_scan: room for %d chunks is too little", c->chunks);
-  const int rc = decay_scan_launch<bf16>(c, chunked, s);
+  const int rc = decay_scan_launch<bf16, DS_GROUP>(c, chunked, s);
   if (rc || !chunked) return rc;
   if (c->dim <= 64) return c->decay ? chunk_launch<1, false>(c, s) : chunk_launch<1, true>(c, s);
   return c->decay ? chunk_launch<2, false>(c, s) : chunk_launch<2, true>(c, s);

@@ -60,8 +60,7 @@ class HyperLane(HybridLane):
         """Scratch of a linear mixer's long runs (none in the all-fp32 mode, for decode-sized lanes and for heads the chunk kernels do not take)."""
         if self.eng.f32 or self.cap <= 16 or r.dim > 128 or r.vdim > 256:
             return None
-        n, f32 = self.cap // ops.SCAN_CHUNK + self.eng.max_seqs + 1, dict(dtype=torch.float32, device=self.dev)
-        return self.get(("scan", r.heads, r.dim, r.vdim), lambda: (torch.zeros(n, r.heads, r.dim, up(r.vdim, 4), **f32), torch.zeros(n, r.heads, r.dim, **f32)))
+        return self.get(("scan", r.heads, r.dim, r.vdim), lambda: ops.scan_scratch(self.cap, self.eng.max_seqs, r.heads, r.dim, r.vdim, self.dev))
 
 
 class HyperStackEngine(HybridStackEngine):
@@ -172,7 +171,7 @@ class HyperStackEngine(HybridStackEngine):
             ops.router_logits(L.xn, lw.router, e["logits"], T)
             self.launches_per_step += 1
         else:
-            self._dense(lw.router, L.xn_act, e["logits"], T)
+            self._dense(lw.router, L.xn_glu, e["logits"], T)      # (narrow products spread better over 128-row tiles)
 
     def _silu_ffn(self, width: int, lw: HyperLayer, L: HyperLane, T: int):
         """Dense feed-forward or shared expert: L.xn -> L.mix."""

@@ -943,12 +943,12 @@ def decay_scan_arg(q, k, v, g, state, tags, ring, out, meta: dict, *, H, dim, vd
                    tau=1.0, norm=None, out_scale=1.0, chunks=None, T: int = 0, status=None):
     """Arguments of `decay_scan`: q, k, v, g column views of one projection buffer; `decay` fp32 [H] (constant) or `low_rank` = (a1 column view, a2 fp32
     [H * dim, rank], bias fp32 [H * dim]): decay sigmoid(a2 a1 + bias) ** (1 / tau) per key channel; `state` [slots, 2, H, dim, vp] with `tags`
-    [slots, H, 2] (positions), `ring` [slots, depth, H, 2 dim + vp].  `chunks` = (states [n, H, dim, vp], decays [n, H, dim]) fp32 scratch with which
-    long runs of a step of `T` rows take the chunk kernels (bf16, heads of up to 128 x 256; n >= T / SCAN_CHUNK + sequences + 1)."""
+    [slots, H, 2] (positions), `ring` [slots, depth, H, 2 dim + vp].  `chunks`: scratch of `scan_scratch`, with which long runs of a step of
+    `T` rows take the chunk kernels (bf16, heads of up to 128 x 256)."""
     a = native.DecayScan()
     if chunks is not None:
-        a.chunk_state, a.chunk_decay, a.chunks, a.T = ptr(chunks[0]), ptr(chunks[1]), chunks[0].shape[0], T
-        if chunks[0].shape[1:] != (H, dim, state.shape[-1]) or chunks[1].shape != chunks[0].shape[:3]:
+        a.chunk_state, a.chunk_decay, a.chunk_tiles, a.chunks, a.T = ptr(chunks[0]), ptr(chunks[1]), ptr(chunks[2]), chunks[0].shape[0], T
+        if chunks[0].shape[1:] != (H, dim, state.shape[-1]) or any(c.shape[0] != a.chunks for c in chunks):
             raise ValueError("decay_scan: chunk scratch of another geometry")
     for n, t in dict(q=q, k=k, v=v, g=g, rope=rope, decay=decay, norm=norm, state=state, tags=tags, ring=ring, out=out, status=status,
                      **{m: meta[m] for m in ("state_slot", "q_start", "q_len", "kv_len")}).items():
@@ -962,6 +962,13 @@ def decay_scan_arg(q, k, v, g, state, tags, ring, out, meta: dict, *, H, dim, vd
     if state.shape[1:4] != (2, H, dim) or ring.shape[2:] != (H, 2 * dim + a.vp) or tags.shape != (a.n_state, H, 2):
         raise ValueError("decay_scan: state, tags and ring do not belong together")
     return a
+
+
+def scan_scratch(rows: int, n_seq: int, H: int, dim: int, vdim: int, device) -> tuple:
+    """Scratch of `decay_scan`'s chunk kernels for steps of up to `rows` rows of up to `n_seq` sequences (zeroed: pads of the operand tiles stay zero)."""
+    n, up = rows // SCAN_CHUNK + n_seq + 1, lambda v, m: -(-v // m) * m
+    return (torch.zeros(n, H, dim, up(vdim, 4), dtype=torch.float32, device=device), torch.zeros(n, H, 2 * dim + 1, dtype=torch.float32, device=device),
+            torch.zeros(n, H, 2, up(dim, 64) * up(vdim, 64), dtype=torch.bfloat16, device=device))
 
 
 def decay_scan(a, *, f32: bool):

@@ -178,7 +178,7 @@ class HyperRows(C.Structure):
 
 class DecayScan(C.Structure):
     """`cuteafd_decay_scan` (`CaDecayScan` of the C ABI)."""
-    _fields_ = _fields("q k v g rope decay a1 a2 a2_b norm state tags ring state_slot q_start q_len kv_len out chunk_state chunk_decay status",
+    _fields_ = _fields("q k v g rope decay a1 a2 a2_b norm state tags ring state_slot q_start q_len kv_len out chunk_state chunk_decay chunk_tiles status",
                        "ldp pairs rank ldo H dim vdim vp depth n_state n_seq max_q_len T chunks", "q_scale k_scale inv_tau eps out_scale")
 
 

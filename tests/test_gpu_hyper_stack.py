@@ -248,7 +248,9 @@ def test_linear_attention_across_portions(kind, H, d, dv, rot, tau, rank, harsh,
     dec, a2d, a2bd, nd = dev(decay), dev(a2), dev(a2b), dev(norm)
     state, tags, ring = scan_buffers(H, d, dv)
     st = status_word()
-    scratch = (torch.full((12, H, d, state.shape[-1]), float("nan"), device=DEV), torch.full((12, H, d), float("nan"), device=DEV)) if form == CHUNKS else None
+    scratch = ops.scan_scratch(600, 3, H, d, dv, DEV) if form == CHUNKS else None
+    if scratch:
+        scratch[0].fill_(float("nan")); scratch[1].fill_(float("nan"))
     back = [[(194, 8), (79, 8), (221, 8)], [(195, 30), (86, 9), (222, 1)]]                   # long runs behind rejected rows
     for runs in STEPS + back + [[(0, 1), (0, 17), (0, 400)]] + [r for r in LONG_STEPS]:
         T = sum(n for _, n in runs)

@@ -501,7 +501,7 @@ def vozetar_spec(n_layers: int = 6, hidden: int = 4096, heads: int = 32, kv_head
     base = AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, rope_dims=128, conv_taps=0)
     windowed = dataclasses.replace(base, window=window, keep_first=4, rope_dims=64, rope_theta=1e6)
     rec = RecurrentSpec(kind="retention", heads=rec_heads, dim=rec_dim, vdim=rec_vdim, decay=tuple(1.0 - 2.0 ** (-5 - 7.0 * i / rec_heads) for i in range(rec_heads)), rope_dims=rec_dim)
-    kinds = {"P": (dataclasses.replace(windowed, qkv_bias=True, sink=True), rec, (1.2, 1.1), False),
+    kinds = {"P": (dataclasses.replace(windowed, qkv_bias=True, sink=True), rec, (1.0, 0.8), False),
              "G": (dataclasses.replace(windowed, values_are_keys=True, conv_taps=3, qk_norm_whole=True, out_gate=True), dataclasses.replace(rec, kind="gla", decay=(), rope_dims=0, tau=16.0, rank=16),
                    (0.5, 0.5), True),
              "A": (dataclasses.replace(base, rope_interleaved=False, conv_taps=4, qkv_bias=True, out_bias=True, sink=True, out_gate=True, gate_values=True), None, (1.0, 1.0), False)}
@@ -512,7 +512,7 @@ def vozetar_spec(n_layers: int = 6, hidden: int = 4096, heads: int = 32, kv_head
         routed = moe is not None and i % moe_every == moe_every - 1
         blocks.append(BlockSpec(attn, moe if routed else None, r, None if routed else DenseFfnSpec(ff, activation="silu_glu"), scales, norm))
     return ModelSpec(name="vozetar-shape", family="vozetar", vocab=65536, hidden=hidden, n_layers=n_layers, rms_eps=1e-5, attn=blocks[0].attn, moe=moe or MoESpec(n_experts=0, n_shared=0),
-                     quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(blocks), streams=streams, pair_table=PairTableSpec(65521, 31, 17))
+                     quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(blocks), streams=streams, pair_table=PairTableSpec(65521, 40503, 9973))
 
 
 NAMED_SPECS = {

@@ -28,7 +28,9 @@ SUBSETS = {"latent_stack": (["runtime", "elementwise", "moe", "sampling", "tc_ge
            "hybrid_stack": (["runtime", "elementwise", "sampling", "tc_gemm", "attention_tc", "attention_mla_prefill", "hybrid_stack", "f32_linear"],
                             ["-DCA_TC_BF16_ONLY"]),
            "hyper_stack": (["runtime", "elementwise", "moe", "sampling", "tc_gemm", "attention_tc", "attention_mla_prefill", "hybrid_stack", "hyper_stack", "decay_scan", "f32_linear"],
-                           ["-DCA_TC_BF16_ONLY"])}
+                           ["-DCA_TC_BF16_ONLY"]),
+           "mixed_stack": (["runtime", "elementwise", "sampling", "tc_gemm", "attention_tc", "attention_mla", "attention_mla_prefill", "hybrid_stack", "latent_stack", "hyper_stack", "decay_scan",
+                            "mixed_stack", "f32_linear"], ["-DCA_TC_BF16_ONLY"])}
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "--use_fast_math=false", "-Xptxas", "-v"]

@@ -103,7 +103,7 @@ def build_serving(a):
         from .serving.hostcache import attach_host_tier
         host = attach_host_tier(eng, max(0.0, a.host_cache_gib - a.host_cache_headroom_gib), min_tokens=a.host_cache_min_tokens)
     prefix = PrefixCache(pool, max_entries=a.prefix_cache_entries, min_tokens=a.prefix_cache_min_tokens, host=host)
-    recurrent = bool(spec.attn.linear_every) or spec.stack in ("hybrid", "hyper")
+    recurrent = bool(spec.attn.linear_every) or spec.stack in ("hybrid", "hyper", "mixed")
     if recurrent:
         # recurrent layers carry a state per sequence: a request cannot resume from cached pages (drafted steps are fine: they leave the
         # state alone and the accepted rows are replayed into it, or the engine keeps the last positions' states)

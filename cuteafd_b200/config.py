@@ -74,6 +74,24 @@ class AttentionSpec:
     qkv_bias: bool = False
     out_bias: bool = False
     gate_values: bool = False
+    # Kind "conv_gqa" in mixed stacks, besides: one key and value for each block of `pool` tokens that lies wholly in front of the window (the means of
+    # the tokens' cached keys and values); queries and keys over their root mean square per head, without gains; every angle of the rotation divided by
+    # `rope_divisor`.
+    # Kind "latent" in mixed stacks, besides: queries through a latent of their own (`q_lora_rank` > 0), a rotated part of `rope_dims` dimensions behind
+    # the `head_dim` unrotated ones (one rotated key part shared by the heads, cached beside the latent), `sink`.
+    pool: int = 0
+    qk_norm_unit: bool = False
+    rope_divisor: float = 1.0
+
+    @property
+    def latent_row(self) -> int:
+        """Elements of a cached row of kind "latent": latent and rotated key part in whole 64-element chunks."""
+        return -(-self.kv_lora_rank // 64) * 64 + -(-self.rope_dims // 64) * 64
+
+    @property
+    def pooled_page_rows(self) -> int:
+        """Rows of pooled blocks that belong to a page of 64 tokens: whole strips of eight blocks, each with the page of its first token."""
+        return 8 * -(-8 // self.pool) if self.pool else 0
 
     @property
     def gate_width(self) -> int:
@@ -101,7 +119,7 @@ class AttentionSpec:
         if self.kind == "mla":
             return self.kv_lora_rank + self.qk_rope_head_dim
         if self.kind == "latent":
-            return self.kv_lora_rank
+            return self.kv_lora_rank + self.rope_dims
         if self.kind == "conv_gqa":
             return 0 if self.kv_from >= 0 else self.n_kv_heads * (self.head_dim + self.v_head_dim)
         return 2 * self.n_kv_heads * self.head_dim
@@ -156,7 +174,8 @@ class RecurrentSpec:
     real-gated linear recurrence whose two gates are block-diagonal (`blocks` square blocks).
     Linear attention of `heads` heads with a state of `dim` x `vdim` each: "retention" (a constant decay per head, `decay`; the first `rope_dims`
     dimensions of q and k rotated, i with i + rope_dims / 2) and "gla" (a decay per key channel and token, the sigmoid of a projection of rank
-    `rank` to the power 1 / `tau`; rank 0: as wide as the snapshot's tensors)."""
+    `rank` to the power 1 / `tau`; rank 0: as wide as the snapshot's tensors).  "hgrn2" writes with what its forget gate gives up: a gate per channel
+    between a learned lower bound and one is the decay, one minus it the key; SiLU on q, an output norm, no output gate."""
     kind: str = "rglru"
     width: int = 256
     blocks: int = 1
@@ -204,11 +223,13 @@ class PairTableSpec:
 
 @dataclass(frozen=True)
 class LoopSpec:
-    """Layers [start, stop) run `times` times in a row with the same weights and a cache of their own per pass; each pass opens with a
-    projection of [x; embedding output] and a learned vector of the pass."""
+    """Layers [start, stop) run `times` times in a row with the same weights and a cache (and state) of their own per pass.  With entry "project" each
+    pass opens with a projection of [x; embedding output] and a learned vector of the pass; with "add" every pass but the first opens by adding the
+    embedding output to x."""
     start: int
     stop: int
     times: int
+    entry: str = "project"
 
 
 @dataclass(frozen=True)
@@ -241,7 +262,13 @@ class ModelSpec:
     # norm.  "hybrid" stacks: windowed attention and recurrent layers, RMS norms in front of and behind every sub-layer, whose result is
     # added `residual_mult` times; logits bounded by `logit_softcap` (0 = not).  "hyper" stacks (`streams` > 0): that many residual streams with
     # constant weights per sub-layer (how it reads them, how its output and the old streams make the new ones); mixers alone or side by side.
+    # "mixed" stacks (`mixed`): parallel layers of attention with pooled blocks, rotated latent attention and HGRN2; mixer and feed-forward read the same
+    # RMS-normed row, each times a number of its own; behind a layer the token's part of a second table (`side_dim` values per layer, gated by the
+    # residual) is projected, normalised and added; the embedding is multiplied by `embed_scale`.
     blocks: tuple = ()
+    mixed: bool = False
+    embed_scale: float = 1.0
+    side_dim: int = 0
     streams: int = 0
     pair_table: Optional[PairTableSpec] = None
     residual_mult: float = 1.0
@@ -251,9 +278,11 @@ class ModelSpec:
 
     @property
     def stack(self) -> str:
-        """Which kind of stack `blocks` describes: "latent", "hybrid", "hyper", or "" for models without blocks."""
+        """Which kind of stack `blocks` describes: "latent", "hybrid", "hyper", "mixed", or "" for models without blocks."""
         if not self.blocks:
             return ""
+        if self.mixed:
+            return "mixed"
         if self.streams:
             return "hyper"
         return "latent" if all(b.attn is not None and b.attn.kind == "latent" for b in self.blocks) else "hybrid"
@@ -269,6 +298,10 @@ class ModelSpec:
             return [(i, None) for i in range(n)]
         return ([(i, None) for i in range(lp.start)] + [(i, t if i == lp.start else None) for t in range(lp.times) for i in range(lp.start, lp.stop)] +
                 [(i, None) for i in range(lp.stop, n)])
+
+    def attention_runs(self, kind: str) -> list:
+        """Layer runs (their numbers in `layer_runs`) whose mixer is attention of this kind: each keeps a cache plane of its own in a mixed stack."""
+        return [r for r, (i, _) in enumerate(self.layer_runs()) if self.blocks[i].attn is not None and self.blocks[i].attn.kind == kind]
 
     def replace(self, **kw) -> "ModelSpec":
         return dataclasses.replace(self, **kw)
@@ -320,7 +353,8 @@ class ModelSpec:
         if a.kind == "conv_gqa":
             return h * (a.conv_channels + a.gate_width + a.n_heads * a.v_head_dim)
         if a.kind == "latent":
-            return (h * (a.n_heads * a.head_dim + a.kv_lora_rank + (a.n_heads if a.out_gate else 0)) +
+            qd = a.n_heads * (a.head_dim + a.rope_dims)
+            return ((h * a.q_lora_rank + a.q_lora_rank * qd if a.q_lora_rank else h * qd) + h * (a.kv_lora_rank + a.rope_dims + (a.n_heads if a.out_gate else 0)) +
                     a.n_heads * (a.head_dim + a.v_head_dim) * a.kv_lora_rank + a.n_heads * a.v_head_dim * h)
         if a.kind == "mla":
             qk = a.qk_nope_head_dim + a.qk_rope_head_dim
@@ -335,12 +369,13 @@ class ModelSpec:
 
     def weight_bytes(self) -> dict:
         """Bytes per category for the whole model (planner input)."""
-        if self.stack in ("hybrid", "hyper"):
+        if self.stack in ("hybrid", "hyper", "mixed"):
             db, eb, moes = self.bits(self.quant.dense) / 8, self.bits(self.quant.experts) / 8, [b.moe for b in self.blocks if b.moe is not None]
             rec = sum(self.recurrent_params(b.rec) for b in self.blocks if b.rec is not None)
             return {"routed_experts": sum(3 * self.hidden * m.intermediate * m.n_experts for m in moes) * eb,
                     "shared_experts": sum(3 * self.hidden * m.shared_inter for m in moes if m.n_shared) * db, "router": sum(m.n_experts for m in moes) * self.hidden * db,
-                    "embed_head": self.vocab * self.hidden * (2 + db) + (2 * (self.pair_table.buckets + 1) * self.hidden if self.pair_table else 0),
+                    "embed_head": self.vocab * self.hidden * (2 + db) + (2 * (self.pair_table.buckets + 1) * self.hidden if self.pair_table else 0) +
+                                  self.n_layers * self.side_dim * (2 * self.vocab + 2 * self.hidden * db),
                     "dense_ffn": sum(3 * self.hidden * b.ffn.intermediate for b in self.blocks if b.ffn is not None) * db,
                     "attention": (rec + sum(self.attn_params(b.attn) for b in self.blocks if b.attn is not None)) * db}
         if self.blocks:
@@ -365,25 +400,32 @@ class ModelSpec:
     def recurrent_params(self, r: RecurrentSpec) -> int:
         if r.kind == "rglru":
             return 3 * self.hidden * r.width + 2 * r.width ** 2 // r.blocks
+        if r.kind == "hgrn2":
+            return 2 * self.hidden * r.heads * (r.dim + r.vdim)
         return self.hidden * r.heads * (2 * r.dim + 3 * r.vdim) + r.rank * (self.hidden + r.heads * r.dim)
 
     def kv_row_elems(self) -> int:
-        """Elements of a cached token's row in a hybrid or hyper-connected stack: the widest layer's key heads, then its value heads."""
+        """Elements of a cached token's row in a hybrid, hyper-connected or mixed stack: the widest layer's key heads, then its value heads."""
         up = lambda n: -(-n // 64) * 64
-        return max((b.attn.n_kv_heads * (up(b.attn.head_dim) + up(b.attn.v_head_dim)) for b in self.blocks if b.attn is not None and b.attn.kv_from < 0), default=0)
+        return max((b.attn.n_kv_heads * (up(b.attn.head_dim) + up(b.attn.v_head_dim)) for b in self.blocks
+                    if b.attn is not None and b.attn.kind == "conv_gqa" and b.attn.kv_from < 0), default=0)
+
+    def latent_row_elems(self) -> int:
+        """Elements of a cached token's latent row in a mixed stack: the widest layer's."""
+        return max((b.attn.latent_row for b in self.blocks if b.attn is not None and b.attn.kind == "latent"), default=0)
 
     def state_bytes_per_seq(self, depth: int = 8) -> int:
-        """Bytes of one sequence's state slot in a hybrid or hyper-connected stack (`engine.hybrid_stack`, `engine.hyper_stack`): convolution
-        inputs and recurrent states of the last positions, `depth` of which can be taken back."""
+        """Bytes of one sequence's state slot in a hybrid, hyper-connected or mixed stack (`engine.hybrid_stack`, `engine.hyper_stack`,
+        `engine.mixed_stack`): convolution inputs and recurrent states of the last positions, `depth` of which can be taken back."""
         eb, n = 2 if self.quant.dense == "bf16" else 4, 4 * (depth + 1) if self.pair_table is not None else 0
-        for b in self.blocks:
+        for b in (self.blocks[i] for i, _ in self.layer_runs()):
             r, a = b.rec, b.attn
             if r is not None and r.kind == "rglru":
                 n += r.width * ((r.conv_taps - 1 + depth) * eb + (depth + 1) * 4)
             elif r is not None:         # two states, the last inputs of the recurrence, two positions per head
                 vp = -(-r.vdim // 4) * 4
                 n += r.heads * (4 * (2 * r.dim * vp + depth * (2 * r.dim + vp)) + 8)
-            if a is not None and a.conv_taps:
+            if a is not None and a.kind == "conv_gqa" and a.conv_taps:
                 n += a.conv_channels * (a.conv_taps - 1 + depth) * eb
         return n
 
@@ -391,6 +433,10 @@ class ModelSpec:
         per = {"fp8": 1.0, "f32": 4.0}.get(self.quant.kv, 2.0)
         if self.stack in ("hybrid", "hyper"):  # one row width for every layer with keys of its own, heads in whole 64-element chunks
             return len(self.kv_layers()) * self.kv_row_elems() * per
+        if self.stack == "mixed":   # keys and values with their pooled blocks, and latents: a plane per layer run
+            runs = [self.blocks[i].attn for i, _ in self.layer_runs()]
+            pooled = sum(a.pooled_page_rows / 64 * a.n_kv_heads * (-(-a.head_dim // 64) * 64 + -(-a.v_head_dim // 64) * 64) for a in runs if a is not None and a.pool)
+            return (len(self.attention_runs("conv_gqa")) * self.kv_row_elems() + len(self.attention_runs("latent")) * self.latent_row_elems() + pooled) * per
         if self.blocks:             # one row width for every layer run (the widest latent, in whole 64-element chunks)
             return len(self.layer_runs()) * max(-(-b.attn.kv_token_elems // 64) * 64 for b in self.blocks) * per
         return self.n_layers * self.attn.kv_token_elems * per
@@ -515,6 +561,22 @@ def vozetar_spec(n_layers: int = 6, hidden: int = 4096, heads: int = 32, kv_head
                      quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=tuple(blocks), streams=streams, pair_table=PairTableSpec(65521, 40503, 9973))
 
 
+def sikazen_spec(n_layers: int = 6, hidden: int = 4096, heads: int = 32, kv_heads: int = 4, ff: int = 12288, window: int = 2048, pool: int = 16, rank: int = 512, q_rank: int = 1536,
+                 rec_heads: int = 16, rec_dim: int = 128, rec_vdim: int = 256, side: int = 256, mixers: str = "LHA", loop: tuple | None = None) -> ModelSpec:
+    """Sikazen at the size of a real model's layers (synthetic weights).  `mixers` repeats over the layers: L rotated latent attention with sinks, H HGRN2,
+    A windowed attention with pooled blocks.  `loop`: (start, stop, times)."""
+    kinds = {"L": (AttentionSpec(kind="latent", n_heads=heads, n_kv_heads=heads, head_dim=128, v_head_dim=128, kv_lora_rank=rank, q_lora_rank=q_rank, rope_dims=64, rope_theta=1e6,
+                                 scale=192 ** -0.5, sink=True), None),
+             "H": (None, RecurrentSpec(kind="hgrn2", heads=rec_heads, dim=rec_dim, vdim=rec_vdim)),
+             "A": (AttentionSpec(kind="conv_gqa", n_heads=heads, n_kv_heads=kv_heads, head_dim=128, v_head_dim=128, scale=128 ** -0.5, window=window, pool=pool, conv_taps=0, rope_dims=128,
+                                 rope_interleaved=False, rope_divisor=4.0, qk_norm_unit=True, qkv_bias=True), None)}
+    blocks = tuple(BlockSpec(a, rec=r, ffn=DenseFfnSpec(ff, activation="silu_glu")) for a, r in (kinds[mixers[i % len(mixers)]] for i in range(n_layers)))
+    return ModelSpec(name="sikazen-shape", family="sikazen", vocab=65536, hidden=hidden, n_layers=n_layers, rms_eps=1e-5,
+                     attn=next((b.attn for b in blocks if b.attn is not None), AttentionSpec(kind="conv_gqa", n_heads=1, n_kv_heads=1)), moe=MoESpec(n_experts=0, n_shared=0),
+                     quant=QuantSpec(experts="bf16", dense="bf16", kv="bf16"), blocks=blocks, mixed=True, embed_scale=hidden ** 0.5, side_dim=side,
+                     loop=LoopSpec(*loop, entry="add") if loop else None)
+
+
 NAMED_SPECS = {
     "tiny": tiny_spec,
     "hybrid-gdn": hybrid_gdn_spec,
@@ -525,6 +587,7 @@ NAMED_SPECS = {
     "bedovik": bedovik_spec,
     "tudilix": tudilix_spec,
     "vozetar": vozetar_spec,
+    "sikazen": sikazen_spec,
     "ep-microbench": ep_microbench_spec,
 }
 
@@ -553,6 +616,7 @@ FAMILY_BY_ARCH = {
     "Bedovik": "bedovik",
     "Tudilix": "tudilix",
     "Vozetar": "vozetar",
+    "Sikazen": "sikazen",
 }
 
 
@@ -706,6 +770,51 @@ def _vozetar_config(cfg: dict) -> ModelSpec:
                      streams=streams, pair_table=PairTableSpec(int(pairs["buckets"]), int(pairs["mul_prev"]), int(pairs["mul_cur"])) if pairs else None)
 
 
+def _sikazen_config(cfg: dict) -> ModelSpec:
+    """`config.json` of the Sikazen design: every layer names its mixer (attention with pooled blocks, rotated latent attention, HGRN2) and its
+    feed-forward with their sizes."""
+    blocks = []
+    for i, layer in enumerate(cfg["layers"]):
+        m, mlp, kind = layer["mixer"], layer.get("mlp"), layer["type"]
+        attn = rec = ffn = None
+        rot = m.get("rot") or {"dims": 0, "base": 1e4}
+        turn = dict(rope_theta=float(rot["base"]), rope_divisor=float((rot.get("scaling") or {}).get("factor", 1.0)))
+        if kind == "attention":
+            mask = m.get("mask") or {}
+            attn = AttentionSpec(kind="conv_gqa", n_heads=int(m["heads"]), n_kv_heads=int(m["kv_heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]), scale=float(m["scale"]),
+                                 window=int(mask.get("size") or 0), pool=int(mask.get("pool") or 0) if mask.get("size") else 0, conv_taps=0, rope_dims=int(rot["dims"]),
+                                 rope_interleaved=False, qk_norm_unit=True, qkv_bias=True, **turn)
+            if attn.n_heads % attn.n_kv_heads:
+                raise ValueError(f"layer {i}: {attn.n_heads} query heads over {attn.n_kv_heads} key heads")
+            if attn.rope_dims % 2 or attn.rope_dims > attn.head_dim:
+                raise ValueError(f"layer {i}: {attn.rope_dims} rotated dimensions of {attn.head_dim}")
+            if attn.window < 0 or attn.pool < 0:
+                raise ValueError(f"layer {i}: window of {attn.window} tokens, blocks of {attn.pool}")
+        elif kind == "latent_attention":
+            attn = AttentionSpec(kind="latent", n_heads=int(m["heads"]), n_kv_heads=int(m["heads"]), head_dim=int(m["dim"]), v_head_dim=int(m["vdim"]), kv_lora_rank=int(m["kv_rank"]),
+                                 q_lora_rank=int(m["q_rank"]), rope_dims=int(m["rot_dim"]), scale=float(m["scale"]), sink=True, **turn)
+            if attn.rope_dims % 2 or int(rot["dims"]) != attn.rope_dims:
+                raise ValueError(f"layer {i}: rotation over {rot['dims']} dimensions of a rotated part of {attn.rope_dims}")
+        elif kind == "hgrn2":
+            rec = RecurrentSpec(kind="hgrn2", heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+        if mlp is not None:
+            if mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            ffn = DenseFfnSpec(int(mlp["ff"]), activation="silu_glu")
+        blocks.append(BlockSpec(attn, rec=rec, ffn=ffn))
+    loop = None
+    if cfg.get("loop"):
+        loop = LoopSpec(int(cfg["loop"]["start"]), int(cfg["loop"]["stop"]), int(cfg["loop"]["times"]), "add")
+        if not (0 <= loop.start < loop.stop <= len(blocks) and loop.times >= 1):
+            raise ValueError(f"loop {cfg['loop']} does not fit {len(blocks)} layers")
+    first = next((b.attn for b in blocks if b.attn is not None), AttentionSpec(kind="conv_gqa", n_heads=1, n_kv_heads=1))
+    return ModelSpec(name="sikazen", family="sikazen", vocab=int(cfg["vocab"]), hidden=int(cfg["width"]), n_layers=len(blocks), rms_eps=float(cfg["norm"]["eps"]), attn=first,
+                     moe=MoESpec(n_experts=0, n_shared=0), quant=QuantSpec(), blocks=tuple(blocks), mixed=True, embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
+                     side_dim=int((cfg.get("token_side") or {}).get("dim") or 0), loop=loop)
+
+
 def from_hf_config(cfg: dict | str | Path) -> ModelSpec:
     """Build a ModelSpec from a Hugging Face `config.json` (dict or path)."""
     if not isinstance(cfg, dict):
@@ -722,6 +831,8 @@ def from_hf_config(cfg: dict | str | Path) -> ModelSpec:
         return _tudilix_config(cfg)
     if family == "vozetar":
         return _vozetar_config(cfg)
+    if family == "sikazen":
+        return _sikazen_config(cfg)
     hidden = cfg["hidden_size"]
     heads = cfg["num_attention_heads"]
     if "kv_lora_rank" in cfg:

@@ -34,7 +34,9 @@
 
 struct MlaArgs {
   const bf16* q_lat;        // [Hl * T, 512] head-major
-  const bf16* q_rope;       // [T, Hl, 64]
+  const bf16* q_rope;       // rotated parts, 64 wide: row (t, h) at t * qr_t + h * qr_h
+  const float* sink;        // [Hl], or null
+  int qr_t, qr_h;
   const CUtensorMap* kv_map;    // 2-D (as 3-D): {576, slots, 1}, box {64, 32, 1}, 128-byte swizzle
   const int* page_table; const int* kv_len; const int* q_start; const int* q_len;
   bf16* out;                // [Hl, T, 512] head-major
@@ -137,7 +139,7 @@ __global__ void __launch_bounds__(192, MlaGeo<NC, NL>::OCC) mla_attn_kernel(cons
     if (r < R) {
       const int t = row_base + r / a.Hl, h = r % a.Hl;
       v = (NC == NL || c < NL * 8) ? *(const uint4*)(a.q_lat + ((size_t)h * a.ldt + t) * LAT + c * 8)
-                                   : *(const uint4*)(a.q_rope + ((size_t)t * a.Hl + h) * 64 + (c - NL * 8) * 8);
+                                   : *(const uint4*)(a.q_rope + (size_t)t * a.qr_t + (size_t)h * a.qr_h + (c - NL * 8) * 8);
     }
     *(uint4*)(sQ + ((c >> 3) - G::QT) * 16384 + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
   }
@@ -154,13 +156,16 @@ __global__ void __launch_bounds__(192, MlaGeo<NC, NL>::OCC) mla_attn_kernel(cons
   if (warp >= 2) {
     const int r = (warp & 3) * 32 + lane;
     const uint32_t dst = tmem + ((uint32_t)((warp & 3) * 32) << 16) + QT_COL;
-    const bf16* src = a.q_lat + ((size_t)((r < R ? r : 0) % a.Hl) * a.ldt + row_base + (r < R ? r : 0) / a.Hl) * LAT;
+    const int rt = row_base + (r < R ? r : 0) / a.Hl, rh = (r < R ? r : 0) % a.Hl;
+    const bf16* lat = a.q_lat + ((size_t)rh * a.ldt + rt) * LAT;
+    const bf16* rot = NC > NL ? a.q_rope + (size_t)rt * a.qr_t + (size_t)rh * a.qr_h : lat;
 #pragma unroll 1
     for (int g = 0; g < G::QT * 2; ++g) {                // 16 columns = 32 elements per store
+      const bf16* src = g < 2 * NL ? lat + g * 32 : rot + (g - 2 * NL) * 32;
       uint32_t w[16];
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const uint4 v = r < R ? *(const uint4*)(src + g * 32 + j * 8) : make_uint4(0, 0, 0, 0);
+        const uint4 v = r < R ? *(const uint4*)(src + j * 8) : make_uint4(0, 0, 0, 0);
         w[4 * j] = v.x; w[4 * j + 1] = v.y; w[4 * j + 2] = v.z; w[4 * j + 3] = v.w;
       }
       mla_tmem_st_x16(dst + g * 16, w);
@@ -318,7 +323,12 @@ __global__ void __launch_bounds__(192, MlaGeo<NC, NL>::OCC) mla_attn_kernel(cons
       const int rr = live ? r : 0;
       const int t = row_base + rr / a.Hl, h = rr % a.Hl;
       const float m_nat = (m_ref == -INFINITY) ? -INFINITY : m_ref * 0.6931471805599453f;
-      const float inv = (l > 0.f ? 1.f / l : 0.f) * ((a.gate && live) ? a.gate[(size_t)t * a.Hl + h] : 1.f);      // output gate of the head
+      float scale_o = 1.f, lt = l;
+      if (a.n_splits == 1 && a.sink) {                        // learned sink logit: one more softmax term with a zero value (splits: the merge adds it)
+        const float sk = a.sink[h], m2 = fmaxf(m_nat, sk), e1 = (m_nat == -INFINITY) ? 0.f : __expf(m_nat - m2);
+        lt = l * e1 + __expf(sk - m2); scale_o = e1;
+      }
+      const float inv = (lt > 0.f ? scale_o / lt : 0.f) * ((a.gate && live) ? a.gate[(size_t)t * a.Hl + h] : 1.f);      // output gate of the head
       bf16* dst = a.out + ((size_t)h * a.ldt + t) * LAT + vh * (G::VCH * 64);
       float* po = a.n_splits > 1 ? a.part_o + (((size_t)split * a.T + t) * a.Hl + h) * LAT + vh * (G::VCH * 64) : nullptr;
 #pragma unroll 1
@@ -691,7 +701,7 @@ __global__ void __launch_bounds__(192, 1) mla_attn_pair_kernel(const __grid_cons
 }
 
 // out[h, t, :] = sum_s o_s * exp(m_s - M) / sum_s l_s * exp(m_s - M); partials are token-major, the output head-major.
-__global__ void __launch_bounds__(128) mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ gate,
+__global__ void __launch_bounds__(128) mla_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ gate, const float* __restrict__ sink,
                                                         bf16* __restrict__ out, int T, int ldt, int Hl, int D, int n_splits) {
   // One block per (token, head), four output columns per thread (D / 4 threads, at least a warp).  The (m, l) pairs of all splits are read at once by
   // one warp (weights exp(m - M) and the denominator land in shared memory); the partial rows then come eight splits at a time,
@@ -708,7 +718,7 @@ __global__ void __launch_bounds__(128) mla_merge_kernel(const float* __restrict_
       const int sidx = lane + 32 * j;
       v[j] = sidx < n_splits ? *(const float2*)(part_ml + (((size_t)sidx * T + t) * Hl + h) * 2) : make_float2(-INFINITY, 0.f);
     }
-    const float M = warp_max(fmaxf(v[0].x, v[1].x));
+    const float sk = sink ? sink[h] : -INFINITY, M = fmaxf(warp_max(fmaxf(v[0].x, v[1].x)), sk);
     float l = 0.f;
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -717,7 +727,7 @@ __global__ void __launch_bounds__(128) mla_merge_kernel(const float* __restrict_
       l += v[j].y * w;
     }
     l = warp_sum(l);
-    if (lane == 0) Lsh = l;
+    if (lane == 0) Lsh = l + (sink ? __expf(sk - M) : 0.f);
   }
   __syncthreads();
   const int d0 = threadIdx.x * 4;
@@ -772,6 +782,7 @@ extern "C" int cuteafd_mla_attention(const void* q_lat, const void* q_rope, cons
   a.q_lat = (const bf16*)q_lat; a.q_rope = (const bf16*)q_rope; a.kv_map = (const CUtensorMap*)kv_map; a.page_table = page_table;
   a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len; a.out = (bf16*)out; a.part_o = part_o; a.part_ml = part_ml; a.status = status;
   a.Hl = Hl; a.max_pages = max_pages; a.n_splits = n_splits; a.T = T; a.ldt = T; a.gate = nullptr; a.scale = scale;
+  a.sink = nullptr; a.qr_t = Hl * 64; a.qr_h = 64;
   const int tpt = 128 / Hl;
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
   int dev = 0; cudaGetDevice(&dev);
@@ -808,16 +819,17 @@ extern "C" int cuteafd_mla_attention(const void* q_lat, const void* q_rope, cons
   }
   CA_CHECK_LAUNCH("mla_attention");
   if (n_splits > 1) {
-    CA_LAUNCH_PDL(mla_merge_kernel, dim3(T, Hl), 128, 0, s, part_o, part_ml, (const float*)nullptr, (bf16*)out, T, T, Hl, DV, n_splits);
+    CA_LAUNCH_PDL(mla_merge_kernel, dim3(T, Hl), 128, 0, s, part_o, part_ml, (const float*)nullptr, (const float*)nullptr, (bf16*)out, T, T, Hl, DV, n_splits);
     CA_CHECK_LAUNCH("mla_merge");
   }
   return CA_OK;
 }
 
-// Latent attention without positions: the absorbed kernel over cache rows of `rank_pad` values (a multiple of 64, 64..512; the pad of a
+// Latent attention of other sizes: the absorbed kernel over cache rows of `rank_pad` values (a multiple of 64, 64..512; the pad of a
 // narrower latent is zero in the cache and in the queries).  q_lat, out: head-major [Hl, ldt, rank_pad]; any Hl <= 128 (a query tile
-// takes 128 / Hl whole tokens).  `gate` [T, Hl] multiplies each head's output (null: none).
-extern "C" int cuteafd_latent_attention(const void* q_lat, const void* kv_map, const int* page_table, const int* kv_len, const int* q_start,
+// takes 128 / Hl whole tokens).  `q_rope` (null: attention without positions): rotated parts [Hl, ldt, 64], whose key part stands in the 64 columns
+// behind the latent's.  `gate` [T, Hl] multiplies each head's output, `sink` [Hl] is one more logit per head (null: none).
+extern "C" int cuteafd_latent_attention(const void* q_lat, const void* q_rope, const float* sink, const void* kv_map, const int* page_table, const int* kv_len, const int* q_start,
                                         const int* q_len, const float* gate, void* out, float* part_o, float* part_ml, int T, int ldt, int n_seq,
                                         int max_q_len, int Hl, int rank_pad, int max_pages, int n_splits, float scale, int* status, cudaStream_t s) {
   CA_REQUIRE(q_lat && kv_map && page_table && kv_len && q_start && q_len && out, "latent_attention: null argument");
@@ -826,28 +838,20 @@ extern "C" int cuteafd_latent_attention(const void* q_lat, const void* kv_map, c
   CA_REQUIRE(n_splits >= 1 && n_splits <= 64 && (n_splits == 1 || (part_o && part_ml)), "latent_attention: 1..64 KV splits, and split-KV needs scratch");
   if (T <= 0 || n_seq <= 0) return CA_OK;
   MlaArgs a;
-  a.q_lat = (const bf16*)q_lat; a.q_rope = nullptr; a.kv_map = (const CUtensorMap*)kv_map; a.page_table = page_table;
+  a.q_lat = (const bf16*)q_lat; a.q_rope = (const bf16*)q_rope; a.sink = sink; a.qr_t = 64; a.qr_h = ldt * 64; a.kv_map = (const CUtensorMap*)kv_map; a.page_table = page_table;
   a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len; a.gate = n_splits > 1 ? nullptr : gate; a.out = (bf16*)out; a.part_o = part_o;
   a.part_ml = part_ml; a.status = status; a.Hl = Hl; a.max_pages = max_pages; a.n_splits = n_splits; a.T = T; a.ldt = ldt; a.scale = scale;
   const int tpt = 128 / Hl, nl = rank_pad / 64;
   a.max_q_tiles = (max_q_len + tpt - 1) / tpt;
   const dim3 grid(n_splits, nl <= 4 ? 1 : 2, n_seq * a.max_q_tiles);
-  int rc;
-  switch (nl) {
-    case 1: rc = mla_launch<1, 1>(a, grid, s); break;
-    case 2: rc = mla_launch<2, 2>(a, grid, s); break;
-    case 3: rc = mla_launch<3, 3>(a, grid, s); break;
-    case 4: rc = mla_launch<4, 4>(a, grid, s); break;
-    case 5: rc = mla_launch<5, 5>(a, grid, s); break;
-    case 6: rc = mla_launch<6, 6>(a, grid, s); break;
-    case 7: rc = mla_launch<7, 7>(a, grid, s); break;
-    default: rc = mla_launch<8, 8>(a, grid, s); break;
-  }
+  int rc = CA_ERR_UNSUPPORTED;
+#define LA_CASE(N_) if (nl == N_) rc = q_rope ? mla_launch<N_ + 1, N_>(a, grid, s) : mla_launch<N_, N_>(a, grid, s);
+  LA_CASE(1) LA_CASE(2) LA_CASE(3) LA_CASE(4) LA_CASE(5) LA_CASE(6) LA_CASE(7) LA_CASE(8)
   if (rc) return rc;
   CA_CHECK_LAUNCH("latent_attention");
   if (n_splits > 1) {
     const int threads = rank_pad / 4 < 32 ? 32 : rank_pad / 4;
-    CA_LAUNCH_PDL(mla_merge_kernel, dim3(T, Hl), threads, 0, s, part_o, part_ml, gate, (bf16*)out, T, ldt, Hl, rank_pad, n_splits);
+    CA_LAUNCH_PDL(mla_merge_kernel, dim3(T, Hl), threads, 0, s, part_o, part_ml, gate, sink, (bf16*)out, T, ldt, Hl, rank_pad, n_splits);
     CA_CHECK_LAUNCH("mla_merge");
   }
   return CA_OK;

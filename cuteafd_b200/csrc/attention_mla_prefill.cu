@@ -36,7 +36,8 @@
 
 struct MlaPrefillArgs {
   const bf16* q_nope;           // [Hl, T, 128] head-major
-  const bf16* q_rope;           // [T, Hl, 64]
+  const bf16* q_rope;           // rotated parts, 64 wide: row (t, head) at t * qr_t + head * qr_h
+  const float* sink;            // [Hl], or null
   CUtensorMap kvb_map;          // {Hl * 256, rows, 1}, box {64, 128, 1}, 128-byte swizzle (encoded with rank 3: loads pass z = 0)
   CUtensorMap lat_map;          // {576, rows, 1}, box {64, 128, 1}, 128-byte swizzle
   const int* ctx_start;         // [n_seq] first row of the sequence's context in the two buffers
@@ -47,6 +48,7 @@ struct MlaPrefillArgs {
   bf16* out;                    // [T, ldo] token-major, head h at column h * dv
   int* status;
   int T, Hl, max_q_tiles;
+  int qr_t, qr_h, rope_col;     // (rope_col: column of the latent rows where the rotated key part starts)
   int ldt, ldo, dv;             // rows between two heads of q_nope, output row stride, value width
   float scale;
 };
@@ -122,7 +124,7 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
     const uint32_t dst = tmem + ((uint32_t)((warp & 3) * 32) << 16) + Q_COL;
     const int t = row_base + (r < R ? r : 0);
     const bf16* src_nope = a.q_nope + ((size_t)head * a.ldt + t) * (KN * 64);
-    const bf16* src_rope = a.q_rope + ((size_t)t * a.Hl + head) * 64;
+    const bf16* src_rope = a.q_rope + (size_t)t * a.qr_t + (size_t)head * a.qr_h;
 #pragma unroll 1
     for (int g = 0; g < 2 * NK; ++g) {             // 16 columns = 32 elements per store
       const bf16* src = (KR == 0 || g < 2 * KN) ? src_nope + g * 32 : src_rope + (g - 2 * KN) * 32;
@@ -152,7 +154,7 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
         mbar_expect_tx(&k_full[s], K_STAGE);
 #pragma unroll
         for (int c = 0; c < KN; ++c) tma_load_3d(sK + s * K_STAGE + c * 16384, &a.kvb_map, &k_full[s], head * HEAD_W + c * 64, row, 0);
-        if (KR) tma_load_3d(sK + s * K_STAGE + KN * 16384, &a.lat_map, &k_full[s], 512, row, 0);
+        if (KR) tma_load_3d(sK + s * K_STAGE + KN * 16384, &a.lat_map, &k_full[s], a.rope_col, row, 0);
       }
       __syncwarp();
       return true;
@@ -324,7 +326,13 @@ __global__ void __launch_bounds__(192, 1) mla_prefill_kernel(const __grid_consta
     tc_fence_after();
     if (__all_sync(0xffffffffu, ok)) {
       const int t = row_base + (live ? r : 0);
-      const float inv = (l > 0.f ? 1.f / l : 0.f) * ((a.gate && live) ? a.gate[(size_t)t * a.Hl + head] : 1.f);      // output gate of the head
+      float scale_o = 1.f, lt = l;
+      if (a.sink) {                                     // learned sink logit: one more softmax term with a zero value
+        const float m_nat = (m_ref == -INFINITY) ? -INFINITY : m_ref * 0.6931471805599453f, sk = a.sink[head], m2 = fmaxf(m_nat, sk);
+        const float e1 = (m_nat == -INFINITY) ? 0.f : __expf(m_nat - m2);
+        lt = l * e1 + __expf(sk - m2); scale_o = e1;
+      }
+      const float inv = (lt > 0.f ? scale_o / lt : 0.f) * ((a.gate && live) ? a.gate[(size_t)t * a.Hl + head] : 1.f);      // output gate of the head
       bf16* dst = a.out + (size_t)t * a.ldo + (size_t)head * a.dv;
       const bool vec = (a.ldo | a.dv) % 8 == 0;
 #pragma unroll 1
@@ -414,9 +422,10 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
   const int hi = bidir ? kvlen : first_pos + ntok;
   const int lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
   const int tile0 = lo / PF_KT;
-  // tiles of kept first keys in front of the window, then the window's
-  const int kept = a.x.kept_tiles(tile0, PF_KT), n_tiles = kept + max(0, (hi + PF_KT - 1) / PF_KT - tile0);
+  // tiles of kept first keys or of pooled blocks in front of the window, then the window's
+  const int kept = a.x.lead_tiles(tile0, PF_KT, hi - 1, a.window), n_tiles = kept + max(0, (hi + PF_KT - 1) / PF_KT - tile0);
   auto tile_at = [&](int i) { return i < kept ? i : i - kept + tile0; };
+  auto pooled_at = [&](int i) { return a.x.pool > 0 && i < kept; };
 
   if (tid == 0) {
     for (int s = 0; s < 2; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
@@ -462,10 +471,20 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       const int pi = key / 64;
       return pi < a.max_pages ? a.page_table[(size_t)seq * a.max_pages + pi] : 0;
     };
+    // lane l's strip of a tile of pooled blocks (past the last one: that one again, masked)
+    auto strip_of = [&](int i) { return a.x.strip_row(min(tile_at(i) * 16 + (lane & 15), (a.x.blocks_seen(hi - 1, a.window) - 1) >> 3), a.page_table + (size_t)seq * a.max_pages); };
     auto load_k = [&](int i) -> bool {
       const int s = i % PF_NS, ph = ((i / PF_NS) & 1) ^ 1;
       if (!mbar_wait_bounded(&k_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); return false; }
-      if (lane == 0) {
+      if (pooled_at(i)) {
+        const int row = strip_of(i);
+        if (lane == 0) mbar_expect_tx(&k_full[s], Cf::K_STAGE);
+        __syncwarp();
+        if (lane < 16) {
+#pragma unroll
+          for (int c = 0; c < KC; ++c) tma_load_3d(sK + s * Cf::K_STAGE + c * 16384 + lane * 1024, a.x.pool_maps, &k_full[s], c * 64, kvh, row);
+        }
+      } else if (lane == 0) {
         const int key0 = tile_at(i) * PF_KT;
         mbar_expect_tx(&k_full[s], Cf::K_STAGE);
 #pragma unroll
@@ -483,7 +502,15 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       if (i + 1 < n_tiles && !load_k(i + 1)) break;
       const int sv = i % Cf::NSV, phv = ((i / Cf::NSV) & 1) ^ 1;
       if (!mbar_wait_bounded(&v_empty[sv], phv, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, 0x1000 + i); break; }
-      if (lane == 0) {
+      if (pooled_at(i)) {
+        const int row = strip_of(i);
+        if (lane == 0) mbar_expect_tx(&v_full[sv], Cf::V_STAGE);
+        __syncwarp();
+        if (lane < 16) {
+#pragma unroll
+          for (int c = 0; c < VC; ++c) tma_load_3d(sV + sv * Cf::V_STAGE + c * 16384 + lane * 1024, a.x.pool_maps + 1, &v_full[sv], c * 64, kvh, row);
+        }
+      } else if (lane == 0) {
         const int key0 = tile_at(i) * PF_KT;
         mbar_expect_tx(&v_full[sv], Cf::V_STAGE);
 #pragma unroll
@@ -542,6 +569,7 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
     const bool live = r < R;
     const int qpos = live ? (bidir ? first_pos : first_pos + r / G) : -1;
     const int wlo = a.window > 0 ? qpos - a.window : -1;           // keys at or below this position are outside the row's window
+    const int blocks = live ? a.x.blocks_seen(qpos, a.window) : 0;
     const float sc2 = a.scale * 1.4426950408889634f;
     float m_ref = -INFINITY, l = 0.f;
     bool ok = true;
@@ -551,7 +579,11 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
       const uint32_t s_addr = tmem + lane_addr + ((i & 1) ? S1_COL : S0_COL);
       const int key0 = tile_at(i) * PF_KT;
       // CTA-uniform: every key of the tile is visible to every live row (below the diagonal and inside every row's window)
-      const bool all_visible = key0 + PF_KT - 1 <= first_pos && (a.window <= 0 || key0 > first_pos + ntok - 1 - a.window || key0 + PF_KT <= a.x.keep_first);
+      // (tiles of pooled blocks: of the blocks that a row sees)
+      const bool pooled = pooled_at(i);
+      const bool all_visible = pooled ? key0 + PF_KT <= a.x.blocks_seen(first_pos, a.window)
+                                      : key0 + PF_KT - 1 <= first_pos && (a.window <= 0 || key0 > first_pos + ntok - 1 - a.window || key0 + PF_KT <= a.x.keep_first);
+      auto sees = [&](int kp) { return pooled ? kp < blocks : live && kp <= qpos && (kp > wlo || kp < a.x.keep_first); };
       // two passes over the tile's 128 score columns: row maximum, then exponentials packed to bf16 pairs (64 registers).
       // Tiles below the diagonal need no mask (CTA-uniform test), which is all but the last one or two of a long context.
       float mx = -INFINITY;
@@ -597,7 +629,7 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const int kp = key0 + c * 32 + j;
-            if (live && kp <= qpos && (kp > wlo || kp < a.x.keep_first)) mx = fmaxf(mx, __uint_as_float(sr[j]) * sc2);
+            if (sees(kp)) mx = fmaxf(mx, __uint_as_float(sr[j]) * sc2);
           }
         }
         if (mx > m_ref + 8.f) {
@@ -613,8 +645,8 @@ __global__ void __launch_bounds__(192, 1) gqa_prefill_kernel(const __grid_consta
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const int kp = key0 + c * 32 + 2 * j;
-            const float e0 = (live && kp <= qpos && (kp > wlo || kp < a.x.keep_first)) ? exp2f(fmaf(__uint_as_float(sr[2 * j]), sc2, -m_ref)) : 0.f;
-            const float e1 = (live && kp + 1 <= qpos && (kp + 1 > wlo || kp + 1 < a.x.keep_first)) ? exp2f(fmaf(__uint_as_float(sr[2 * j + 1]), sc2, -m_ref)) : 0.f;
+            const float e0 = sees(kp) ? exp2f(fmaf(__uint_as_float(sr[2 * j]), sc2, -m_ref)) : 0.f;
+            const float e1 = sees(kp + 1) ? exp2f(fmaf(__uint_as_float(sr[2 * j + 1]), sc2, -m_ref)) : 0.f;
             psum += e0 + e1;
             bf162 h = __floats2bfloat162_rn(e0, e1);
             pk[c * 16 + j] = *(uint32_t*)&h;
@@ -736,6 +768,7 @@ extern "C" int cuteafd_window_prefill_attention(const void* q, const void* maps,
   CA_REQUIRE(Hkv >= 1 && Hq % Hkv == 0 && Hq / Hkv <= 128 && q_stride % 8 == 0, "window_prefill_attention: group size %d unsupported", Hkv ? Hq / Hkv : 0);
   CA_REQUIRE(dv >= 1 && dv <= dv_pad && ldo >= Hq * dv && window >= 0 && q_stride >= Hq * dk_pad, "window_prefill_attention: bad shape");
   CA_REQUIRE(!extras || !extras->gate || extras->ldg >= (extras->gate_values ? Hq * dv : Hq), "window_prefill_attention: gate rows too short");
+  CA_REQUIRE(attn_extras_ok(extras, true), "window_prefill_attention: pooled blocks without their rows, or beside kept keys");
   if (T <= 0 || n_seq <= 0) return CA_OK;
   GqaPrefillArgs a = {};
   a.q = (const bf16*)q; a.k_map = (const CUtensorMap*)maps; a.v_map = a.k_map + 1; a.v_head0 = 0; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
@@ -818,22 +851,25 @@ extern "C" int cuteafd_mla_prefill_attention(const void* q_nope, const void* q_r
   if (rc) return rc;
   a.q_nope = (const bf16*)q_nope; a.q_rope = (const bf16*)q_rope; a.ctx_start = ctx_start; a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len;
   a.out = (bf16*)out; a.status = status; a.T = T; a.Hl = Hl; a.max_q_tiles = (max_q_len + 127) / 128; a.scale = scale;
-  a.gate = nullptr; a.ldt = T; a.ldo = Hl * 128; a.dv = 128;
+  a.gate = nullptr; a.ldt = T; a.ldo = Hl * 128; a.dv = 128; a.sink = nullptr; a.qr_t = Hl * 64; a.qr_h = 64; a.rope_col = 512;
   rc = mla_prefill_launch<2, 1, 2>(a, n_seq, s);
   if (rc) return rc;
   CA_CHECK_LAUNCH("mla_prefill_attention");
   return CA_OK;
 }
 
-// The same for latent attention without positions: q [Hl, ldt, dk_pad] head-major (dk_pad 64 / 128 / 192, pad columns zero), kvb
+// The same for latent attention of other sizes: q [Hl, ldt, dk_pad] head-major (dk_pad 64 / 128 / 192, pad columns zero), kvb
 // [rows, Hl * (dk_pad + dv_pad)] (per head the key columns, then the value columns, each padded to whole 64-wide chunks; dv_pad 64 / 128),
-// out [T, ldo] token-major with head h at column h * dv, `gate` [T, Hl] (or null) multiplied into each head's output.
-extern "C" int cuteafd_latent_prefill_attention(const void* q, const void* kvb, long long rows, const int* ctx_start, const int* kv_len,
+// out [T, ldo] token-major with head h at column h * dv, `gate` [T, Hl] (or null) multiplied into each head's output, `sink` [Hl] (or null) one more
+// logit per head.  With a rotated part (q_rope, null: attention without positions) of up to 64 dimensions: q_rope [Hl, ldt, 64] and, in the
+// gathered context rows `lat` [rows, lat_width], 64 columns from `rope_col` on, shared by the heads; pad columns of q_rope are zero.
+extern "C" int cuteafd_latent_prefill_attention(const void* q, const void* q_rope, const void* kvb, const void* lat, int lat_width, int rope_col, const float* sink, long long rows, const int* ctx_start, const int* kv_len,
                                                 const int* q_start, const int* q_len, const float* gate, void* out, int T, int ldt, int n_seq,
                                                 int max_q_len, int Hl, int dk_pad, int dv_pad, int dv, int ldo, float scale, int* status,
                                                 cudaStream_t s) {
   CA_REQUIRE(q && kvb && ctx_start && kv_len && q_start && q_len && out && rows > 0, "latent_prefill_attention: null argument");
   CA_REQUIRE(Hl >= 1 && ldt >= T && dv >= 1 && dv <= dv_pad && ldo >= Hl * dv, "latent_prefill_attention: bad shape");
+  CA_REQUIRE(!q_rope || (lat && rope_col % 64 == 0 && rope_col + 64 <= lat_width && lat_width % 8 == 0), "latent_prefill_attention: rotated part outside the context rows");
   CA_REQUIRE((dk_pad == 64 || dk_pad == 128 || dk_pad == 192) && (dv_pad == 64 || dv_pad == 128), "latent_prefill_attention: head widths %d / %d", dk_pad, dv_pad);
   if (T <= 0 || n_seq <= 0) return CA_OK;
   MlaPrefillArgs a;
@@ -842,11 +878,17 @@ extern "C" int cuteafd_latent_prefill_attention(const void* q, const void* kvb, 
                              CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
   a.lat_map = a.kvb_map;
-  a.q_nope = (const bf16*)q; a.q_rope = nullptr; a.ctx_start = ctx_start; a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len;
+  if (q_rope) {
+    rc = ca_encode_tmap_2d(&a.lat_map, lat, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, (uint64_t)lat_width, (uint64_t)rows, (uint64_t)lat_width * 2, 64, PF_KT, CU_TENSOR_MAP_SWIZZLE_128B);
+    if (rc) return rc;
+  }
+  a.sink = sink; a.qr_t = 64; a.qr_h = ldt * 64; a.rope_col = rope_col;
+  a.q_nope = (const bf16*)q; a.q_rope = (const bf16*)q_rope; a.ctx_start = ctx_start; a.kv_len = kv_len; a.q_start = q_start; a.q_len = q_len;
   a.gate = gate; a.out = (bf16*)out; a.status = status; a.T = T; a.Hl = Hl; a.max_q_tiles = (max_q_len + 127) / 128; a.scale = scale;
   a.ldt = ldt; a.ldo = ldo; a.dv = dv;
-  if (dv_pad == 64) rc = dk_pad == 64 ? mla_prefill_launch<1, 0, 1>(a, n_seq, s) : (dk_pad == 128 ? mla_prefill_launch<2, 0, 1>(a, n_seq, s) : mla_prefill_launch<3, 0, 1>(a, n_seq, s));
-  else rc = dk_pad == 64 ? mla_prefill_launch<1, 0, 2>(a, n_seq, s) : (dk_pad == 128 ? mla_prefill_launch<2, 0, 2>(a, n_seq, s) : mla_prefill_launch<3, 0, 2>(a, n_seq, s));
+#define LP_CASE(K_, R_, V_) if (dk_pad == K_ * 64 && dv_pad == V_ * 64 && (q_rope != nullptr) == (R_ != 0)) rc = mla_prefill_launch<K_, R_, V_>(a, n_seq, s);
+#define LP_ROW(R_, V_) LP_CASE(1, R_, V_) LP_CASE(2, R_, V_) LP_CASE(3, R_, V_)
+  LP_ROW(0, 1) LP_ROW(0, 2) LP_ROW(1, 1) LP_ROW(1, 2)
   if (rc) return rc;
   CA_CHECK_LAUNCH("latent_prefill_attention");
   return CA_OK;

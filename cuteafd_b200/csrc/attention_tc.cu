@@ -111,12 +111,13 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
   const int hi = first_pos + ntok;                      // keys [lo, hi) can be visible
   const int lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
   const int first_page = lo / APAGE, last_page = (hi + APAGE - 1) / APAGE;
-  // the pages that count: those of kept first keys in front of the window, then the window's; a split takes a run of them
-  const int kept = a.x.kept_tiles(first_page, APAGE), n_pages = kept + last_page - first_page;
+  // the pages that count: those of kept first keys (or tiles of pooled blocks) in front of the window, then the window's; a split takes a run of them
+  const int kept = a.x.lead_tiles(first_page, APAGE, hi - 1, a.window), n_pages = kept + last_page - first_page;
   const int per = (n_pages + a.n_splits - 1) / a.n_splits;
   const int p0 = split * per, p1 = min(n_pages, p0 + per);
   const int n_tiles = max(0, p1 - p0);
   auto page_at = [&](int i) { const int j = p0 + i; return j < kept ? j : j - kept + first_page; };
+  auto pooled_at = [&](int i) { return a.x.pool > 0 && p0 + i < kept; };
 
   // Decode-shaped tiles (<= 32 real rows) replicate the rows into every 32-lane quarter of the MMA tile so that
   // the four softmax warps each take 16 of the 64 score columns of the SAME rows (4x shorter per-tile chain).
@@ -155,7 +156,27 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
     const uint64_t kvpol = a.max_q_tiles == 1 ? l2_policy_stream() : l2_policy_normal();
     for (int i = 0; i < n_tiles && !*abortp; ++i) {
       const int s = i & 1, ph = ((i >> 1) & 1) ^ 1;
-      const int page = a.page_table[(size_t)seq * a.max_pages + page_at(i)];
+      const int* table = a.page_table + (size_t)seq * a.max_pages;
+      if (pooled_at(i)) {                                  // eight strips of eight blocks (past the last one: that one again, masked)
+        const int last = (a.x.blocks_seen(hi - 1, a.window) - 1) >> 3, row = a.x.strip_row(min(page_at(i) * 8 + (lane & 7), last), table);
+        if (!mbar_wait_bounded(&k_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); break; }
+        if (lane == 0) mbar_expect_tx(&k_full[s], Cf::K_STAGE);
+        __syncwarp();
+        if (lane < 8) {
+#pragma unroll
+          for (int c = 0; c < KC; ++c) tma_load_3d(sK + s * Cf::K_STAGE + c * 8192 + lane * 1024, a.x.pool_maps, &k_full[s], c * 64, kvh, row);
+        }
+        if (!mbar_wait_bounded(&v_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); break; }
+        if (lane == 0) mbar_expect_tx(&v_full[s], Cf::V_STAGE);
+        __syncwarp();
+        if (lane < 8) {
+#pragma unroll
+          for (int c = 0; c < VC; ++c) tma_load_3d(sV + s * Cf::V_STAGE + c * 8192 + lane * 1024, a.x.pool_maps + 1, &v_full[s], c * 64, kvh, row);
+        }
+        __syncwarp();
+        continue;
+      }
+      const int page = table[page_at(i)];
       if (!mbar_wait_bounded(&k_empty[s], ph, abortp)) { ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, i); break; }
       if (lane == 0) {
         mbar_expect_tx(&k_full[s], Cf::K_STAGE);
@@ -217,6 +238,7 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
     const uint32_t lane_addr = (uint32_t)(q4 * 32) << 16;
     const bool live = r < R;                  // in the replicated layout quarter 0 (r = lane) holds the real rows
     const int qpos = live ? first_pos + r / G : -1;
+    const int seen = live ? a.x.blocks_seen(qpos, a.window) : 0;
     const float sc2 = a.scale * 1.4426950408889634f;
     float m_ref = -INFINITY, l = 0.f;
     bool ok = true;
@@ -224,6 +246,7 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
       // ---- column-split path: thread (q4, lane) owns row `lane`, score columns [16*q4, 16*q4 + 16)
       const bool rlive = lane < R;
       const int rq = rlive ? first_pos + lane / G : -1;
+      const int blocks = rlive ? a.x.blocks_seen(rq, a.window) : 0;
       float* xchg = (float*)(sP + 8192);                 // [2][4][32] row maxima (P rows >= 64 are never read back)
       float* lsum = xchg + 256;                          // [4][32]
       const int col0 = 16 * q4;
@@ -234,11 +257,12 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
         tmem_ld_x16(tmem + lane_addr + ((i & 1) ? S1_COL : S0_COL) + col0, sr);
         tc_wait_ld();
         const int key0 = page_at(i) * APAGE + col0;
+        const bool pooled = pooled_at(i);
         float mx = -INFINITY;
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           const int kp = key0 + j;
-          const bool vis = rlive && kp <= rq && kp < kvlen && (a.window <= 0 || kp > rq - a.window || kp < a.x.keep_first);
+          const bool vis = pooled ? kp < blocks : rlive && kp <= rq && kp < kvlen && (a.window <= 0 || kp > rq - a.window || kp < a.x.keep_first);
           const float v = vis ? __uint_as_float(sr[j]) * sc2 : -INFINITY;
           sr[j] = __float_as_uint(v);
           mx = fmaxf(mx, v);
@@ -298,11 +322,12 @@ __global__ void __launch_bounds__(192, AttnTcCfg<KC, VC>::OCC) paged_attn_tc_ker
       for (int c = 0; c < 4; ++c) tmem_ld_x16(tmem + lane_addr + ((i & 1) ? S1_COL : S0_COL) + c * 16, sr + c * 16);
       tc_wait_ld();
       const int key0 = page_at(i) * APAGE;
+      const bool pooled = pooled_at(i);
       float mx = -INFINITY;
 #pragma unroll
       for (int j = 0; j < 64; ++j) {
         const int kp = key0 + j;
-        const bool vis = live && kp <= qpos && kp < kvlen && (a.window <= 0 || kp > qpos - a.window || kp < a.x.keep_first);
+        const bool vis = pooled ? kp < seen : live && kp <= qpos && kp < kvlen && (a.window <= 0 || kp > qpos - a.window || kp < a.x.keep_first);
         const float v = vis ? __uint_as_float(sr[j]) * sc2 : -INFINITY;
         sr[j] = __float_as_uint(v);
         mx = fmaxf(mx, v);
@@ -507,6 +532,7 @@ extern "C" int cuteafd_window_attention(const void* q, const void* maps, const i
   CA_REQUIRE(dv >= 1 && dv <= dv_pad && ldo >= Hq * dv && window >= 0 && q_stride >= Hq * dk_pad, "window_attention: bad shape");
   CA_REQUIRE(n_splits >= 1 && (n_splits == 1 || (part_o && part_ml)), "window_attention: split-KV needs scratch");
   CA_REQUIRE(!extras || !extras->gate || extras->ldg >= (extras->gate_values ? Hq * dv : Hq), "window_attention: gate rows too short");
+  CA_REQUIRE(attn_extras_ok(extras, true), "window_attention: pooled blocks without their rows, or beside kept keys");
   if (T <= 0 || n_seq <= 0) return CA_OK;
   AttnTcArgs a = {};
   a.q = (const bf16*)q; a.k_map = (const CUtensorMap*)maps; a.v_map = a.k_map + 1; a.v_head0 = 0; a.page_table = page_table; a.kv_len = kv_len; a.q_start = q_start;
@@ -528,11 +554,12 @@ extern "C" int cuteafd_window_attention(const void* q, const void* maps, const i
   return CA_OK;
 }
 
-// Descriptor of `heads` heads of `width` bf16 each (a multiple of 64) that start at `base` in rows `row_elems` apart.
-extern "C" int cuteafd_tmap_encode_heads(void* out128, const void* base, int width, int heads, uint64_t row_elems, uint64_t n_slots) {
-  CA_REQUIRE(width > 0 && width % 64 == 0 && heads >= 1 && row_elems % 8 == 0 && ((uintptr_t)base & 15) == 0, "tmap_encode_heads: bad geometry");
+// Descriptor of `heads` heads of `width` bf16 each (a multiple of 64) that start at `base` in rows `row_elems` apart; boxes of `box_rows` rows (64: a
+// page, 8: a strip of pooled blocks).
+extern "C" int cuteafd_tmap_encode_heads(void* out128, const void* base, int width, int heads, uint64_t row_elems, uint64_t n_slots, int box_rows) {
+  CA_REQUIRE((box_rows == 64 || box_rows == 8) && width > 0 && width % 64 == 0 && heads >= 1 && row_elems % 8 == 0 && ((uintptr_t)base & 15) == 0, "tmap_encode_heads: bad geometry");
   CUtensorMap m;
-  int rc = ca_encode_tmap_3d(&m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, width, heads, n_slots, (uint64_t)width * 2, row_elems * 2, 64, 1, 64, CU_TENSOR_MAP_SWIZZLE_128B);
+  int rc = ca_encode_tmap_3d(&m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, width, heads, n_slots, (uint64_t)width * 2, row_elems * 2, 64, 1, box_rows, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
   memcpy(out128, &m, sizeof(m));
   return CA_OK;

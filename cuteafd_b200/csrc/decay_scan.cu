@@ -1,6 +1,8 @@
-// Linear attention with a decay per head or per key channel (retention, gated linear attention): the mixers that hyper-connected stacks run
-// beside their attention.
+// Linear attention with a decay per head or per key channel: retention and gated linear attention, which hyper-connected stacks run beside their
+// attention, and HGRN2, a mixer of the mixed stacks.
 //   S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   out_t = norm(o_t) * silu(g_t)
+// HGRN2 has no keys and no output gate: its forget gate f = l + (1 - l) sigmoid(z + b), with a learned lower bound l per channel, is the decay, and the
+// key is what the gate gives up, 1 - f = (1 - l) sigmoid(-z - b); queries pass SiLU.
 // Two forms.  Runs of up to DS_GROUP tokens (decoding, drafts, short portions; every run in the all-fp32 mode): one block per (head, sequence), the
 // state crosses HBM once for the whole group.  Longer runs in chunks of DC_TOK tokens, all chunks of all heads in parallel:
 //   chunk_states   D_c = sum_j decay(j -> end of chunk) k_j v_j^T          one tcgen05 product per (head, chunk), and the chunk's decays
@@ -8,7 +10,7 @@
 //   chunk_out      o = (q k^T, decayed, causal) v + decay(start -> i) q S  three tcgen05 products per (head, chunk), output norm, gate
 // Everything that is not a projection enters the products as two bf16 terms (value and rounding error, 16 bits of mantissa together), with fp32
 // accumulators in tensor memory; the states stay fp32.  Per-channel decays are folded into q and k relative to the middle of the chunk; a chunk
-// whose decays span more than 2^80 on the way takes its scores from the ordinary cores instead.
+// whose decays span more than 2^80 on the way takes its scores from the ordinary cores instead, pair by pair.
 // (Sibling of linear_attn.cu, whose delta rule has no such form yet; the reference's linear-attention programs are AOT exports without sources.)
 #define CA_PDL_CLASS 2
 #include "stack_rows.cuh"
@@ -29,6 +31,7 @@ struct DecayScan {
   const float* decay;                                       // [H] constant decays; null: alpha = sigmoid(a2 a1 + a2_b)^(1 / tau) per key channel
   const T* a1; const float* a2; const float* a2_b;          // [rank] columns of the projection rows, [H * dim, rank], [H * dim]
   int rank; float inv_tau;
+  const float* forget_b; const float* lower;                // HGRN2 (null otherwise): bias and lower bound of the forget gate [H * dim], whose logits are k
   const float* norm; float eps, out_scale;                  // gain of the output norm [vdim], or null
   float* state; int* tags; float* ring;                     // [slots, 2, H, dim, vp], [slots, H, 2], [slots, depth, H, 2 dim + vp]
   const int* state_slot; const int* q_start; const int* q_len; const int* kv_len;
@@ -41,6 +44,15 @@ struct DecayScan {
   float* chunk_state; float* chunk_decay; uint8_t* chunk_tiles;
   int* status;
 };
+
+// HGRN2: (decay, key) of a channel from the forget gate's logit z (bias added) and lower bound l
+__device__ __forceinline__ float2 forget_gate(float z, float l) {
+  const float e = expf(-fabsf(z)), s = 1.f / (1.f + e), big = s, small = e * s;      // sigmoids of |z| and -|z|
+  return make_float2(fmaf(1.f - l, z >= 0.f ? big : small, l), (1.f - l) * (z >= 0.f ? small : big));
+}
+// and the binary logarithm of that decay
+__device__ __forceinline__ float forget_log2(float2 f) { return f.y < 0.5f ? log1pf(-f.y) * 1.4426950408889634f : log2f(fmaxf(f.x, 1e-38f)); }
+__device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.f + __expf(-fmaxf(z, -80.f))); }
 
 // log alpha of a channel from its logit
 __device__ __forceinline__ float log_decay(float z, float inv_tau) { return -(fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau; }
@@ -145,7 +157,10 @@ __global__ void __launch_bounds__(DS_THREADS, NT == 1 ? 3 : 1) decay_scan_kernel
         k = lo ? k * cs.x - k2 * cs.y : k * cs.x + k2 * cs.y;
       }
       float al = decay;
-      if (!a.decay) {
+      if (a.lower) {
+        const float2 f = forget_gate(k + a.forget_b[h * dim + r], a.lower[h * dim + r]);
+        al = f.x; k = f.y; q = q / (1.f + expf(-q));
+      } else if (!a.decay) {
         float z = a.a2_b[h * dim + r];
         const T* ar = a.a1 + (size_t)row * a.ldp;
         const float* wr = a.a2 + (size_t)(h * dim + r) * a.rank;
@@ -190,8 +205,8 @@ __global__ void __launch_bounds__(DS_THREADS, NT == 1 ? 3 : 1) decay_scan_kernel
       const float inv = rsqrtf(block_sum(ss, red32) / (float)a.vdim + a.eps) * a.out_scale;
       const size_t row = row0 + done + t - replay;
       for (int c = tid; c < a.vdim; c += DS_THREADS) {
-        const float g = to_f(a.g[row * a.ldp + h * a.vdim + c]);
-        a.out[row * a.ldo + h * a.vdim + c] = to_t<T>(sm.o[c] * inv * (a.norm ? a.norm[c] : 1.f) * (g / (1.f + expf(-g))));
+        const float g = a.g ? to_f(a.g[row * a.ldp + h * a.vdim + c]) : 0.f;
+        a.out[row * a.ldo + h * a.vdim + c] = to_t<T>(sm.o[c] * inv * (a.norm ? a.norm[c] : 1.f) * (a.g ? g / (1.f + expf(-g)) : 1.f));
       }
     };
     float4 acc[NT];
@@ -314,6 +329,45 @@ __device__ __forceinline__ void head8(const bf16* row, int d0, int dim, const fl
   for (int j = 0; j < 8; ++j) v[j] *= scale;
 }
 
+// How the chunk kernels get their decays: a constant per head, from a low-rank projection, from HGRN2's forget gate.
+enum { DECAY_HEAD = 0, DECAY_LOW_RANK = 1, DECAY_FORGET = 2 };
+
+template <int MODE>
+__device__ __forceinline__ void query8(const DecayScan<bf16>& a, int h, size_t row, int d0, bool vec, float* v) {
+  head8(a.q + row * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + row * a.pairs : nullptr, a.pairs, a.q_scale, vec, v);
+  if (MODE == DECAY_FORGET)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = silu_f(v[j]);
+}
+template <int MODE>
+__device__ __forceinline__ void key8(const DecayScan<bf16>& a, int h, size_t row, int d0, bool vec, float* v) {
+  head8(a.k + row * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + row * a.pairs : nullptr, a.pairs, a.k_scale, vec, v);
+  if (MODE == DECAY_FORGET)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = h * a.dim + d0 + j;
+      v[j] = d0 + j < a.dim ? (1.f - __ldg(a.lower + c)) * __fdividef(1.f, 1.f + __expf(fminf(v[j] + __ldg(a.forget_b + c), 80.f))) : 0.f;
+    }
+}
+
+// log2 of the forget gate's decays -> X [128, DP] (zero past the run's end and past `dim`).
+template <int DP>
+__device__ __forceinline__ void chunk_forget(const DecayScan<bf16>& a, int h, const ChunkRun& r, bool vec, float* X) {
+  for (int i = threadIdx.x; i < DC_TOK * DP / 8; i += DC_THREADS) {
+    const int t = i / (DP / 8), d0 = (i % (DP / 8)) * 8;
+    float z[8];
+    head8(a.k + (size_t)(r.row + min(t, r.len - 1)) * a.ldp + h * a.dim, d0, a.dim, nullptr, 0, 1.f, vec, z);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = h * a.dim + d0 + j;
+      z[j] = t < r.len && d0 + j < a.dim ? forget_log2(forget_gate(z[j] + __ldg(a.forget_b + c), __ldg(a.lower + c))) : 0.f;
+    }
+    *(float4*)(X + t * DP + d0) = make_float4(z[0], z[1], z[2], z[3]);
+    *(float4*)(X + t * DP + d0 + 4) = make_float4(z[4], z[5], z[6], z[7]);
+  }
+  __syncthreads();
+}
+
 // log2 of the chunk's per-channel decays -> X [128, DP] (zero past the run's end and past `dim`); `stage`: 8 KB.
 template <int DP>
 __device__ __forceinline__ void chunk_logs(const DecayScan<bf16>& a, int h, const ChunkRun& r, float* X, float* stage) {
@@ -389,10 +443,11 @@ __device__ __forceinline__ void chunk_end(const ChunkSync& y, int cols) {
 }
 
 // D_c = sum_j decay(j -> end) k_j v_j^T of one head and chunk, rows of key dimensions; the decays of the whole chunk.
-template <int DB, bool GLA>
+template <int DB, int MODE>
 __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __grid_constant__ DecayScan<bf16> a) {
   pdl_launch(); pdl_wait();
   using Sm = ChunkSmem<DB>;
+  constexpr bool GLA = MODE != DECAY_HEAD;                            // a decay per key channel
   constexpr int DP = DB * 64;
   extern __shared__ __align__(1024) uint8_t dc_smem[];
   const int h = blockIdx.x, tid = threadIdx.x;
@@ -407,7 +462,8 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __gri
   const float l2 = GLA ? 0.f : decay_log2(a.decay[h]);
   float* factors = a.chunk_decay + ((size_t)r.ci * a.H + h) * (2 * a.dim + 1);
   if (GLA) {
-    chunk_logs<DP>(a, h, r, X, (float*)sK);
+    if (MODE == DECAY_FORGET) chunk_forget<DP>(a, h, r, vec, X);
+    else chunk_logs<DP>(a, h, r, X, (float*)sK);
     bool far = false;
     if (tid < 2 * DP) {                                               // decays behind every token, within its half
       const int c = tid % DP, half = tid / DP;
@@ -429,7 +485,7 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __gri
     float v[8];
     if (t < r.len) {
       const size_t row = r.row + t;
-      head8(a.k + row * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + row * a.pairs : nullptr, a.pairs, a.k_scale, vec, v);
+      key8<MODE>(a, h, row, d0, vec, v);
       const float f = GLA ? 0.f : exp2f(l2 * (float)(r.len - 1 - t));
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[j] *= GLA ? exp2f(X[t * DP + d0 + j] + (t < 64 ? rest[d0 + j] : 0.f)) : f;
@@ -510,10 +566,11 @@ __global__ void __launch_bounds__(128) chunk_scan_kernel(const DecayScan<bf16> a
   *(float4*)(a.state + (((size_t)slot * 2 + 1 - b.place) * a.H + h) * one + e) = S;
 }
 
-template <int DB, bool GLA>
+template <int DB, int MODE>
 __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_constant__ DecayScan<bf16> a) {
   pdl_launch(); pdl_wait();
   using Sm = ChunkSmem<DB>;
+  constexpr bool GLA = MODE != DECAY_HEAD;                            // a decay per key channel
   constexpr int DP = DB * 64, T = Sm::TILE;
   extern __shared__ __align__(1024) uint8_t dc_smem[];
   const int h = blockIdx.x, seq = blockIdx.z, tid = threadIdx.x;
@@ -535,7 +592,8 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
   bool wide = false;                                                  // decays that span too much for a common reference
   if (!GLA) load_values(a, h, r, sX, VB);
   if (GLA) {
-    chunk_logs<DP>(a, h, r, X, (float*)sQ);
+    if (MODE == DECAY_FORGET) chunk_forget<DP>(a, h, r, vec, X);
+    else chunk_logs<DP>(a, h, r, X, (float*)sQ);
     wide = a.chunk_decay[((size_t)r.ci * a.H + h) * (2 * a.dim + 1) + 2 * a.dim] != 0.f;
     if (tid < 2 * DP) {                                               // relative to the chunk's middle: in front of it up to 63 (positive), behind it (negative)
       const int c = tid % DP;
@@ -555,9 +613,8 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
     float q[8], k[8];
     if (t < r.len) {
       const size_t gr = r.row + t;
-      const float2* cs = a.rope ? a.rope + gr * a.pairs : nullptr;
-      head8(a.q + gr * a.ldp + h * a.dim, d0, a.dim, cs, a.pairs, a.q_scale, vec, q);
-      head8(a.k + gr * a.ldp + h * a.dim, d0, a.dim, cs, a.pairs, a.k_scale, vec, k);
+      query8<MODE>(a, h, gr, d0, vec, q);
+      key8<MODE>(a, h, gr, d0, vec, k);
       if (GLA) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
@@ -571,7 +628,7 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
       for (int j = 0; j < 8; ++j) q[j] = k[j] = 0.f;
     }
     put8_two(sQ, tile_at(t, d0, T), DB * T, q);
-    if (!wide) put8_two(sP, tile_at(t, d0, T), DB * T, k);
+    put8_two(sP, tile_at(t, d0, T), DB * T, k);                       // (wide: as they are)
   }
   float sc[KW];                                                       // this thread's scores: its row, keys [part * KW, + KW)
   if (!wide) {
@@ -600,22 +657,29 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
       }
     }
   } else {
-    // pairwise, from the projected rows: the decays between two tokens as the difference of their sums
-    for (int j = 0; j < KW; ++j) {
-      const int key = part * KW + j;
-      float s = 0.f;
-      if (key <= row && row < r.len) {
-        const size_t gq = r.row + row, gk = r.row + key;
-        for (int d0 = 0; d0 < a.dim; d0 += 8) {
-          float q[8], k[8];
-          head8(a.q + gq * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + gq * a.pairs : nullptr, a.pairs, a.q_scale, vec, q);
-          head8(a.k + gk * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + gk * a.pairs : nullptr, a.pairs, a.k_scale, vec, k);
+    // pairwise: the decays between two tokens as the difference of their sums
+    __syncthreads();                                                  // the keys are there
 #pragma unroll
-          for (int e = 0; e < 8; ++e) s = fmaf(q[e] * k[e], exp2f(X[row * DP + d0 + e] - X[key * DP + d0 + e]), s);
+    for (int j = 0; j < KW; ++j) sc[j] = 0.f;
+    if (part * KW <= (warp & 3) * 32 + 31)                            // warp-uniform: some key is not behind every row of the warp
+      for (int d0 = 0; d0 < a.dim; d0 += 8) {
+        float q[8], x[8];
+        query8<MODE>(a, h, r.row + min(row, r.len - 1), d0, vec, q);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = X[row * DP + d0 + e];
+#pragma unroll
+        for (int j = 0; j < KW; ++j) {
+          const int key = part * KW + j;
+          const uint8_t* at = sP + tile_at(key, d0, T);
+          float k[8], lo[8];
+          load8<bf16>((const bf16*)at, k);
+          load8<bf16>((const bf16*)(at + DB * T), lo);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) sc[j] = fmaf(q[e] * (k[e] + lo[e]), exp2f(x[e] - X[key * DP + d0 + e]), sc[j]);
         }
       }
-      sc[j] = s;
-    }
+#pragma unroll
+    for (int j = 0; j < KW; ++j) if (part * KW + j > row || row >= r.len) sc[j] = 0.f;         // (may not be a number)
     __syncthreads();                                                  // the decays have been read
     load_values(a, h, r, sX, VB);
   }
@@ -655,14 +719,14 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
   const int c_lo = part * VB * PW, c_hi = c_lo + VB * PW;
   const bool vout = ((a.vdim | a.ldp | a.ldo) & 7) == 0 && (((uintptr_t)a.g | (uintptr_t)a.out) & 15) == 0;
   const size_t gr = r.row + min(row, r.len - 1);
-  const bf16* g = a.g + gr * a.ldp + h * a.vdim;
+  const bf16* g = a.g ? a.g + gr * a.ldp + h * a.vdim : nullptr;
   bf16* dst = a.out + gr * a.ldo + h * a.vdim;
   constexpr int NG = 4 * PW / 8;
   uint4 gates[NG];
 #pragma unroll
   for (int p = 0; p < NG; ++p) {
     const int c = c_lo + p * 8;
-    if (c >= c_hi || c >= a.vdim) gates[p] = make_uint4(0, 0, 0, 0);
+    if (!g || c >= c_hi || c >= a.vdim) gates[p] = make_uint4(0, 0, 0, 0);
     else if (vout) gates[p] = __ldg((const uint4*)(g + c));
     else {
       bf16 e[8];
@@ -711,7 +775,7 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
         const float2 g2 = __bfloat1622float2(gp[j / 2]);
         const float gv = j & 1 ? g2.y : g2.x;
         const float x = fmaf(f2, __uint_as_float(s[p + j]), __uint_as_float(o[p + j])) * inv;
-        v[j] = x * (a.norm && c + p + j < a.vdim ? __ldg(a.norm + c + p + j) : 1.f) * __fdividef(gv, 1.f + __expf(-fmaxf(gv, -80.f)));
+        v[j] = x * (a.norm && c + p + j < a.vdim ? __ldg(a.norm + c + p + j) : 1.f) * (g ? silu_f(gv) : 1.f);
       }
       if (vout) store8<bf16>(dst + c + p, v);
       else
@@ -730,14 +794,14 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
 // ---------------------------------------------------------------- C ABI
 struct CaDecayScan {
   const void* q; const void* k; const void* v; const void* g; const void* rope; const float* decay; const void* a1; const float* a2; const float* a2_b; const float* norm;
-  float* state; int* tags; float* ring; const int* state_slot; const int* q_start; const int* q_len; const int* kv_len; void* out; float* chunk_state; float* chunk_decay; void* chunk_tiles; int* status;
+  float* state; int* tags; float* ring; const int* state_slot; const int* q_start; const int* q_len; const int* kv_len; void* out; float* chunk_state; float* chunk_decay; void* chunk_tiles; int* status; const float* forget_b; const float* lower;
   int ldp, pairs, rank, ldo, H, dim, vdim, vp, depth, n_state, n_seq, max_q_len, T, chunks; float q_scale, k_scale, inv_tau, eps, out_scale;
 };
 
 template <typename T>
 static DecayScan<T> decay_scan_args(const CaDecayScan* c, bool chunked) {
   return DecayScan<T>{(const T*)c->q, (const T*)c->k, (const T*)c->v, (const T*)c->g, c->ldp, (const float2*)c->rope, c->pairs, c->q_scale, c->k_scale, c->decay, (const T*)c->a1, c->a2,
-                      c->a2_b, c->rank, c->inv_tau, c->norm, c->eps, c->out_scale, c->state, c->tags, c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len, (T*)c->out, c->ldo,
+                      c->a2_b, c->rank, c->inv_tau, c->forget_b, c->lower, c->norm, c->eps, c->out_scale, c->state, c->tags, c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len, (T*)c->out, c->ldo,
                       c->H, c->dim, c->vdim, c->vp, c->depth, c->n_state, chunked ? DS_GROUP : INT_MAX, c->chunk_state, c->chunk_decay, (uint8_t*)c->chunk_tiles, c->status};
 }
 
@@ -766,20 +830,20 @@ static int decay_scan_launch(const CaDecayScan* c, bool chunked, cudaStream_t s)
   return CA_OK;
 }
 
-template <int DB, bool GLA>
+template <int DB, int MODE>
 static int chunk_launch(const CaDecayScan* c, cudaStream_t s) {
   const DecayScan<bf16> a = decay_scan_args<bf16>(c, true);
   const int chunks = (c->max_q_len + DC_TOK - 1) / DC_TOK;
   const dim3 grid(c->H, chunks, c->n_seq);
   static bool states_set[64] = {false}, out_set[64] = {false};
-  int rc = dynamic_smem(chunk_states_kernel<DB, GLA>, ChunkSmem<DB>::STATES, states_set);
-  if (!rc) rc = dynamic_smem(chunk_out_kernel<DB, GLA>, ChunkSmem<DB>::OUT, out_set);
+  int rc = dynamic_smem(chunk_states_kernel<DB, MODE>, ChunkSmem<DB>::STATES, states_set);
+  if (!rc) rc = dynamic_smem(chunk_out_kernel<DB, MODE>, ChunkSmem<DB>::OUT, out_set);
   if (rc) return rc;
-  CA_LAUNCH_PDL((chunk_states_kernel<DB, GLA>), grid, DC_THREADS, ChunkSmem<DB>::STATES, s, a);
+  CA_LAUNCH_PDL((chunk_states_kernel<DB, MODE>), grid, DC_THREADS, ChunkSmem<DB>::STATES, s, a);
   CA_CHECK_LAUNCH("decay_scan chunk states");
   CA_LAUNCH_PDL((chunk_scan_kernel<DB>), dim3((c->dim * c->vp / 4 + 127) / 128, c->H, c->n_seq), 128, 0, s, a);
   CA_CHECK_LAUNCH("decay_scan chunk scan");
-  CA_LAUNCH_PDL((chunk_out_kernel<DB, GLA>), grid, DC_THREADS, ChunkSmem<DB>::OUT, s, a);
+  CA_LAUNCH_PDL((chunk_out_kernel<DB, MODE>), grid, DC_THREADS, ChunkSmem<DB>::OUT, s, a);
   CA_CHECK_LAUNCH("decay_scan chunk outputs");
   return CA_OK;
 }
@@ -788,8 +852,9 @@ static int chunk_launch(const CaDecayScan* c, cudaStream_t s) {
 static bool chunkable(const CaDecayScan* c, int f32) { return !f32 && c->chunk_state && c->chunk_decay && c->chunk_tiles && c->dim <= 128 && c->vdim <= 256 && c->max_q_len > DS_GROUP; }
 
 extern "C" int cuteafd_decay_scan(const CaDecayScan* c, int f32, cudaStream_t s) {
-  CA_REQUIRE(c && c->q && c->k && c->v && c->g && c->state && c->tags && c->ring && c->state_slot && c->q_start && c->q_len && c->kv_len && c->out, "decay_scan: null argument");
-  CA_REQUIRE(c->decay || (c->a1 && c->a2 && c->a2_b && c->rank >= 1), "decay_scan: neither constant decays nor a projection of them");
+  CA_REQUIRE(c && c->q && c->k && c->v && (c->g || c->lower) && c->state && c->tags && c->ring && c->state_slot && c->q_start && c->q_len && c->kv_len && c->out, "decay_scan: null argument");
+  CA_REQUIRE(!c->lower || (c->forget_b && !c->decay && !c->a1 && c->pairs == 0), "decay_scan: a forget gate has a bias, and no other decays or rotation");
+  CA_REQUIRE(c->lower || c->decay || (c->a1 && c->a2 && c->a2_b && c->rank >= 1), "decay_scan: neither constant decays nor a projection of them");
   CA_REQUIRE(c->H >= 1 && c->dim >= 1 && c->dim <= 512 && c->vdim >= 1 && c->vp % 4 == 0 && c->vp >= c->vdim && c->vp <= 4 * DS_THREADS, "decay_scan: heads of %d x %d (at most 512 x %d)", c->dim, c->vdim, 4 * DS_THREADS);
   CA_REQUIRE(c->pairs >= 0 && 2 * c->pairs <= c->dim && (c->pairs == 0 || c->rope) && c->depth >= 1 && 2 * c->depth - 1 <= DS_GROUP && c->n_state >= 1, "decay_scan: bad rotation or depth");
   CA_REQUIRE(c->ldo >= c->H * c->vdim && c->ldp >= c->H * c->vdim && c->ldp >= c->H * c->dim, "decay_scan: rows too short");
@@ -801,6 +866,7 @@ extern "C" int cuteafd_decay_scan(const CaDecayScan* c, int f32, cudaStream_t s)
   CA_REQUIRE(!chunked || (c->chunks >= c->T / DC_TOK + c->n_seq + 1 && c->vp <= 256 && c->max_q_len <= 65535 * DC_TOK), "decay_scan: room for %d chunks is too little", c->chunks);
   const int rc = decay_scan_launch<bf16, DS_GROUP>(c, chunked, s);
   if (rc || !chunked) return rc;
-  if (c->dim <= 64) return c->decay ? chunk_launch<1, false>(c, s) : chunk_launch<1, true>(c, s);
-  return c->decay ? chunk_launch<2, false>(c, s) : chunk_launch<2, true>(c, s);
+  if (c->lower) return c->dim <= 64 ? chunk_launch<1, DECAY_FORGET>(c, s) : chunk_launch<2, DECAY_FORGET>(c, s);
+  if (c->dim <= 64) return c->decay ? chunk_launch<1, DECAY_HEAD>(c, s) : chunk_launch<1, DECAY_LOW_RANK>(c, s);
+  return c->decay ? chunk_launch<2, DECAY_HEAD>(c, s) : chunk_launch<2, DECAY_LOW_RANK>(c, s);
 }

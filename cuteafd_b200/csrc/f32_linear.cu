@@ -10,7 +10,7 @@
 
 struct F32Args {
   const float* X; const float* W; float* Y;
-  const int4* tiles; const int* n_tiles;
+  const int4* tiles; const int* n_tiles; const float* alpha;      // [G] output factors, or null
   int ldx, ldy, rows, N, K, act, grp_rows, grp_cols;      // act: 1 squared ReLU, 2 soft cap at act_p
   float act_p;
 };
@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(256) f32_linear_kernel(const F32Args a) {
       for (int j = 0; j < 4; ++j) {
         const int n = n0 + tx * 4 + j;
         if (n >= a.N) continue;
-        float v = acc[i][j];
+        float v = a.alpha ? acc[i][j] * a.alpha[g] : acc[i][j];
         if (a.act == 1) { v = fmaxf(v, 0.f); v *= v; }
         if (a.act == 2) v = a.act_p * tanhf(v / a.act_p);
         a.Y[o + n] = v;
@@ -69,11 +69,11 @@ __global__ void __launch_bounds__(256) f32_linear_kernel(const F32Args a) {
 }
 
 extern "C" int cuteafd_f32_linear(const float* X, int ldx, const float* W, float* Y, int ldy, const void* tiles, const int* n_tiles, int max_tiles, int rows,
-                                  int N, int K, int act, float act_p, int grp_rows, int grp_cols, cudaStream_t s) {
+                                  int N, int K, int act, float act_p, int grp_rows, int grp_cols, const float* alpha, cudaStream_t s) {
   CA_REQUIRE(X && W && Y && (!tiles || (n_tiles && max_tiles > 0 && max_tiles <= 65535)) && act >= 0 && act <= 2 && (act != 2 || act_p > 0.f), "f32_linear: bad arguments");
   CA_REQUIRE(grp_rows == 0 || tiles, "f32_linear: token-major output belongs to a grouped product");
   if (rows <= 0 || N <= 0) return CA_OK;
-  const F32Args a{X, W, Y, (const int4*)tiles, n_tiles, ldx, ldy, rows, N, K, act, grp_rows, grp_cols, act_p};
+  const F32Args a{X, W, Y, (const int4*)tiles, n_tiles, alpha, ldx, ldy, rows, N, K, act, grp_rows, grp_cols, act_p};
   const int m = tiles ? max_tiles : (rows + FL_T - 1) / FL_T;
   CA_REQUIRE(m <= 65535, "f32_linear: too many row tiles");
   CA_LAUNCH_PDL(f32_linear_kernel, dim3((N + FL_T - 1) / FL_T, m), 256, 0, s, a);

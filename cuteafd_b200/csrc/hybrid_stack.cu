@@ -1,14 +1,16 @@
 // Kernels of the hybrid recurrent / windowed-attention stacks (fp32 residual rows, RMS norms in front of and behind every sub-layer):
-//   norm_rows        embedding, residual += mult * norm(sub-layer output + bias), or a gather of rows - each also leaves the next product's
-//                    normalised operand row
+//   norm_rows        embedding, residual += mult * norm(sub-layer output + bias) (+ the embedding row once more), or a gather of rows - each also
+//                    leaves the next product's operand row, normalised or as it is
 //   rope_table       cosine / sine of the step's positions, once per rotation
 //   conv_qkv         projected queries, keys and values (+ bias) -> short causal convolution -> norm (per head, over the whole projection, or
-//                    none) -> rotation (neighbouring or half-apart pairs) -> query rows, paged cache; values may be the keys in front of the norm
+//                    none) -> rotation (neighbouring or half-apart pairs) -> query rows, paged cache; values may be the keys in front of the norm;
+//                    short runs also leave the blocks they complete as pooled rows
+//   pool_kv          cached rows -> means of the blocks that a long run completes
 //   rglru_conv       x branch -> short causal convolution -> block-major operand of the gate product (and its tile table)
 //   lru_scan         the real-gated linear recurrence: one pass over short runs, chunk aggregates + carried rescan over long ones
 //   glu_rows         clamped GLU over two projected rows (all-fp32 mode; bf16 products do it in their epilogue)
 //   window_attn_simt paged grouped-query attention on the ordinary cores (fp32, and shapes the tcgen05 kernels do not take): windows with kept
-//                    first keys, sinks, output gates
+//                    first keys or pooled blocks, sinks, output gates
 // Everything a sequence carries from step to step is addressed by absolute position: convolution inputs live in a ring of
 // taps - 1 + depth rows, recurrent states in a ring of depth + 1, so a step that is repeated, or the last `depth` tokens that are taken back
 // (rejected drafts), need no restore - later positions overwrite them.  T is the operand type: bf16, or float for the all-fp32 mode.
@@ -26,10 +28,11 @@ enum { ROWS_EMBED = 0, ROWS_ADD = 1, ROWS_GATHER = 2 };
 template <typename T>
 struct NormRows {
   float* x; int W, Wp;                                      // residual rows, Wp apart; norms average over W
-  const int* tokens; const bf16* table; int vocab;          // ROWS_EMBED
+  const int* tokens; const bf16* table; int vocab; float scale;        // ROWS_EMBED: scale times the token's row (ROWS_ADD with a table: added behind the rest)
   const T* add; const float* bias; const float* post; float mult;      // ROWS_ADD: bias and post (gain of the norm behind) may be null
   const int* src_rows;                                      // ROWS_GATHER
-  const float* gain; T* xn; int ldn;                        // next operand: rows normalised by `gain`, or null
+  const float* gain; T* xn; int ldn;                        // next operand: rows normalised by `gain` (null: without gains), or null
+  int raw;                                                  // next operand: the rows as they are
   float eps; int* status;
 };
 
@@ -42,7 +45,7 @@ __global__ void norm_rows_kernel(const NormRows<T> a) {
   size_t row = t;
   if (MODE == ROWS_GATHER) row = (size_t)a.src_rows[t];
   int tok = 0;
-  if (MODE == ROWS_EMBED) {
+  if (MODE == ROWS_EMBED || (MODE == ROWS_ADD && a.table)) {
     tok = a.tokens[t];
     if (tok < 0 || tok >= a.vocab) { if (threadIdx.x == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, t); tok = 0; }
   }
@@ -52,8 +55,11 @@ __global__ void norm_rows_kernel(const NormRows<T> a) {
 #pragma unroll
     for (int j = 0; j < 8; ++j) v[c][j] = 0.f;
     if (i >= a.Wp) continue;
-    if (MODE == ROWS_EMBED) load8<bf16>(a.table + (size_t)tok * a.Wp + i, v[c]);
-    else load8<float>(a.x + row * a.Wp + i, v[c]);
+    if (MODE == ROWS_EMBED) {
+      load8<bf16>(a.table + (size_t)tok * a.Wp + i, v[c]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[c][j] *= a.scale;
+    } else load8<float>(a.x + row * a.Wp + i, v[c]);
   }
   if (MODE == ROWS_ADD) {
     float m[NCH][8], ss = 0.f;
@@ -82,6 +88,12 @@ __global__ void norm_rows_kernel(const NormRows<T> a) {
       if (a.post) load8<float>(a.post + i, g);
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[c][j] = fmaf(a.mult, m[c][j] * inv * g[j], v[c][j]);
+      if (a.table) {
+        float e[8];
+        load8<bf16>(a.table + (size_t)tok * a.Wp + i, e);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[c][j] = fmaf(a.scale, e[j], v[c][j]);
+      }
     }
   }
   float ss = 0.f;
@@ -94,13 +106,13 @@ __global__ void norm_rows_kernel(const NormRows<T> a) {
     for (int j = 0; j < 8; ++j) ss = fmaf(v[c][j], v[c][j], ss);
   }
   if (!a.xn) return;
-  const float inv = rsqrtf(block_sum(ss, red) / (float)a.W + a.eps);
+  const float inv = a.raw ? 1.f : rsqrtf(block_sum(ss, red) / (float)a.W + a.eps);
 #pragma unroll
   for (int c = 0; c < NCH; ++c) {
     const int i = (threadIdx.x + c * nt) * 8;
     if (i >= a.Wp) continue;
-    float g[8], y[8];
-    load8<float>(a.gain + i, g);
+    float g[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f}, y[8];
+    if (a.gain) load8<float>(a.gain + i, g);
 #pragma unroll
     for (int j = 0; j < 8; ++j) y[j] = v[c][j] * inv * g[j];
     store8<T>(a.xn + (size_t)t * a.ldn + i, y);
@@ -130,7 +142,8 @@ struct ConvQkv {
   const T* proj; int ldp;                       // [T, ldp]: H * dim queries | G * dim keys | G * vdim values (none with v_from_k)
   const float* w;                               // [taps, C]; null with one tap: no convolution
   const float* bias;                            // [C] of the projection, or null
-  const float* q_norm; const float* k_norm;     // gains: [dim] of the head norms, [H * dim] and [G * dim] of the whole ones
+  const float* q_norm; const float* k_norm;     // gains: [dim] of the head norms, [H * dim] and [G * dim] of the whole ones; null: none.  (A norm without
+                                                // gains is the same in front of the rotation and behind it: rotations keep a head's sum of squares.)
   const float2* rope;                           // [T, pairs]
   T* ring;                                      // [slots, R, C] projected rows (without bias) by position; null with one tap
   const int* state_slot; const int* q_start; const int* q_len; const int* kv_len; const int* slot_map;
@@ -138,6 +151,8 @@ struct ConvQkv {
   T* cache; int row_stride, n_slots;            // paged rows: G * dp keys, then G * dvp values
   int H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state, norm, v_from_k;
   float eps; int* status;
+  AttnExtras<T> pool;                           // blocks of pooled tokens (0: none); rows of `pooled` pool_stride apart
+  T* pooled; const int* page_table; int max_pages, pool_stride, n_pooled;
 };
 
 template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, float* v) {
@@ -217,9 +232,10 @@ __device__ __forceinline__ void conv_qkv_tile(const ConvQkv<T>& a, int unit, int
   auto weight = [&](int j, float* v) { load_n<float, V>(a.w + (size_t)j * a.C + ch, own, wvec, v); };
   constexpr int NH = TAPS > 1 ? TAPS - 1 : 1, NW = TAPS ? TAPS : 1;
   float hist[NH][V], wr[NW][V], gain[V];
-  const float* norm = (is_q ? a.q_norm : a.k_norm) + (a.norm == QK_NORM_WHOLE ? head * a.dim : 0);
+  const float* gains = is_q ? a.q_norm : a.k_norm;
+  const float* norm = gains + (a.norm == QK_NORM_WHOLE ? head * a.dim : 0);
 #pragma unroll
-  for (int k = 0; k < V; ++k) gain[k] = is_v || a.norm == QK_NORM_NONE ? 1.f : (k < own ? norm[e + k] : 0.f);
+  for (int k = 0; k < V; ++k) gain[k] = is_v || a.norm == QK_NORM_NONE || !gains ? 1.f : (k < own ? norm[e + k] : 0.f);
   if (TAPS) {
 #pragma unroll
     for (int j = 0; j < NW; ++j) {
@@ -312,6 +328,28 @@ __device__ __forceinline__ void conv_qkv_tile(const ConvQkv<T>& a, int unit, int
       }
     }
     if (own) store_n<T, V>(dst + e, own, own == V, y);          // head starts are multiples of 64 elements
+    if (!STATS && a.pooled && !is_q && own && n <= HS_TILE && (p0 + i + 1) % a.pool.pool == 0) {
+      // the run is one tile: the block's rows are this lane's own, or of earlier steps
+      const int P = a.pool.pool, b = (p0 + i) / P, *table = a.page_table + (size_t)seq * a.max_pages;
+      const size_t off = (is_v ? (size_t)a.G * a.dp + (size_t)head * a.dvp : (size_t)head * a.dp) + e;
+      const int row_b = a.pool.strip_row(b >> 3, table) + (b & 7);
+      float m[V];
+#pragma unroll
+      for (int k = 0; k < V; ++k) m[k] = 0.f;
+      bool ok = row_b >= 0 && row_b < a.n_pooled;
+      for (int p = b * P; p < (b + 1) * P && ok; ++p) {
+        const int cs = table[p / 64] * 64 + p % 64;
+        if (cs < 0 || cs >= a.n_slots) { ok = false; break; }
+        float u[V];
+        load_n<T, V>(a.cache + (size_t)cs * a.row_stride + off, own, own == V, u);
+#pragma unroll
+        for (int k = 0; k < V; ++k) m[k] += u[k];
+      }
+      if (!ok) { ca_dev_fail(a.status, CA_DEV_BAD_INDEX, row); continue; }
+#pragma unroll
+      for (int k = 0; k < V; ++k) m[k] /= (float)P;
+      store_n<T, V>(a.pooled + (size_t)row_b * a.pool_stride + off, own, own == V, m);
+    }
   }
   if (!STATS && ring && !keep && i0 == 0 && own)          // this block read the old ring rows of these channels above: it may overwrite them now
     for (int i = max(0, n - (taps - 1)); i < n; ++i) {
@@ -351,6 +389,39 @@ __global__ void __launch_bounds__(WHOLE ? HS_WHOLE_WARPS * 32 : 128) conv_qkv_ke
     }
     __syncthreads();
     for (int u = warp; u < units; u += NWARP) conv_qkv_tile<T, V, TAPS, HALF, false>(a, u, seq, i0, i1, slot, x, nullptr, u < a.H + a.G ? inv[u < a.H ? 0 : 1] : nullptr);
+  }
+}
+
+// ---------------------------------------------------------------- pooled blocks of long runs
+// grid (blocks a run may complete, sequence): means of P cached rows, eight elements a thread.
+template <typename T>
+__global__ void __launch_bounds__(128) pool_kv_kernel(const T* __restrict__ cache, int row_stride, int n_slots, T* __restrict__ pooled, int pool_stride, int n_pooled, int width,
+                                                      const AttnExtras<T> x, const int* __restrict__ page_table, int max_pages, const int* __restrict__ kv_len,
+                                                      const int* __restrict__ q_len, int* status) {
+  pdl_launch(); pdl_wait();
+  const int seq = blockIdx.y, P = x.pool, kv = kv_len[seq], n = q_len[seq], b = (kv - n) / P + blockIdx.x;
+  if (n <= HS_TILE || (long long)(b + 1) * P > kv) return;                // (short runs have left theirs)
+  const int* table = page_table + (size_t)seq * max_pages;
+  const int row_b = x.strip_row(b >> 3, table) + (b & 7);
+  if (row_b < 0 || row_b >= n_pooled) { if (threadIdx.x == 0) ca_dev_fail(status, CA_DEV_BAD_INDEX, b & 0xFFFF); return; }
+  for (int i = threadIdx.x * 8; i < width; i += 1024) {
+    float m[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    for (int p0 = b * P; p0 < (b + 1) * P; p0 += 4) {
+      float u[4][8];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const int p = min(p0 + q, (b + 1) * P - 1), cs = min(max(table[p / 64] * 64 + p % 64, 0), n_slots - 1);
+        load8<T>(cache + (size_t)cs * row_stride + i, u[q]);
+      }
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
+        if (p0 + q < (b + 1) * P)
+#pragma unroll
+          for (int k = 0; k < 8; ++k) m[k] += u[q][k];
+    }
+#pragma unroll
+    for (int k = 0; k < 8; ++k) m[k] /= (float)P;
+    store8<T>(pooled + (size_t)row_b * pool_stride + i, m);
   }
 }
 
@@ -608,7 +679,7 @@ __global__ void glu_rows_kernel(const T* __restrict__ g, const T* __restrict__ u
 template <typename T>
 __global__ void __launch_bounds__(128) window_attn_simt_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ cache, const int* __restrict__ page_table,
                                                                const int* __restrict__ kv_len, const int* __restrict__ q_start, const int* __restrict__ q_len,
-                                                               T* __restrict__ out, int ldo, int n_seq, int G, int group, int dp, int dvp, int dv, int row_stride,
+                                                               T* __restrict__ out, int ldo, int n_seq, int G, int group, int dp, int dvp, int dv, int row_stride, int pool_stride,
                                                                int max_pages, int n_slots, int window, float scale, const AttnExtras<T> x, int* status) {
   pdl_launch(); pdl_wait();
   extern __shared__ float qs[];
@@ -624,19 +695,31 @@ __global__ void __launch_bounds__(128) window_attn_simt_kernel(const T* __restri
   float m = -INFINITY, l = 0.f, o[WA_COLS];
 #pragma unroll
   for (int j = 0; j < WA_COLS; ++j) o[j] = 0.f;
-  // pages of kept first keys that lie in front of the window, then the window's
-  const int kept = x.kept_tiles(lo / 64, 64), pages = kept + pos / 64 - lo / 64 + 1;
+  // pages of kept first keys that lie in front of the window, or tiles of pooled blocks, then the window's
+  const int kept = x.lead_tiles(lo / 64, 64, pos, window), pages = kept + pos / 64 - lo / 64 + 1, blocks = x.blocks_seen(pos, window);
+  __shared__ int strip[8];
   for (int pi = 0; pi < pages; ++pi) {
+    const bool pooled = x.pool > 0 && pi < kept;
     const int k0 = (pi < kept ? pi : pi - kept + lo / 64) * 64;
-    int slot0 = page_table[(size_t)seq * max_pages + k0 / 64] * 64;
-    if (slot0 < 0 || slot0 + 64 > n_slots) { if (tid == 0) ca_dev_fail(status, CA_DEV_BAD_INDEX, t); slot0 = 0; }
-    const T* kb = cache + (size_t)slot0 * row_stride + (size_t)kh * dp;
-    const T* vb = cache + (size_t)slot0 * row_stride + (size_t)G * dp + (size_t)kh * dvp;
-    const int n = min(64, pos + 1 - k0);
+    int slot0 = 0;
+    if (pooled) {
+      if (tid < 8) strip[tid] = x.strip_row(min(k0 / 8 + tid, (blocks - 1) >> 3), page_table + (size_t)seq * max_pages);
+      __syncthreads();
+    } else {
+      slot0 = page_table[(size_t)seq * max_pages + k0 / 64] * 64;
+      if (slot0 < 0 || slot0 + 64 > n_slots) { if (tid == 0) ca_dev_fail(status, CA_DEV_BAD_INDEX, t); slot0 = 0; }
+    }
+    auto row_of = [&](int j) -> const T* {
+      return pooled ? x.pooled + (size_t)(strip[j >> 3] + (j & 7)) * pool_stride : cache + (size_t)(slot0 + j) * row_stride;
+    };
+    const int n = min(64, pooled ? blocks - k0 : pos + 1 - k0);
     for (int j = warp * 16; j < warp * 16 + 16; ++j) {
       float s = 0.f;
-      const bool in = j < n && (k0 + j >= lo || k0 + j < x.keep_first);
-      if (in) for (int i = lane; i < dp; i += 32) s = fmaf(qs[i], to_f(kb[(size_t)j * row_stride + i]), s);
+      const bool in = j < n && (pooled || k0 + j >= lo || k0 + j < x.keep_first);
+      if (in) {
+        const T* kb = row_of(j) + (size_t)kh * dp;
+        for (int i = lane; i < dp; i += 32) s = fmaf(qs[i], to_f(kb[i]), s);
+      }
       s = warp_sum(s);
       if (lane == 0) sc[j] = in ? s * scale : -INFINITY;
     }
@@ -655,7 +738,7 @@ __global__ void __launch_bounds__(128) window_attn_simt_kernel(const T* __restri
       const int i = tid + c * 128;
       if (i < dv) {
         float acc = o[c] * al;
-        for (int j = 0; j < n; ++j) acc = fmaf(sc[j], to_f(vb[(size_t)j * row_stride + i]), acc);         // keys out of sight weigh zero
+        for (int j = 0; j < n; ++j) acc = fmaf(sc[j], to_f(row_of(j)[(size_t)G * dp + (size_t)kh * dvp + i]), acc);         // keys out of sight weigh zero
         o[c] = acc;
       }
     }
@@ -673,12 +756,12 @@ __global__ void __launch_bounds__(128) window_attn_simt_kernel(const T* __restri
 // ---------------------------------------------------------------- C ABI
 struct CaNormRows {
   float* x; const int* tokens; const void* table; const void* add; const float* bias; const float* post; const int* src_rows; const float* gain; void* xn; int* status;
-  int W, Wp, vocab, ldn; float mult, eps;
+  int W, Wp, vocab, ldn, raw; float mult, eps, scale;
 };
 
 template <typename T, int MODE>
 static int norm_rows_launch(const CaNormRows* c, int rows, cudaStream_t s) {
-  const NormRows<T> a{c->x, c->W, c->Wp, c->tokens, (const bf16*)c->table, c->vocab, (const T*)c->add, c->bias, c->post, c->mult, c->src_rows, c->gain, (T*)c->xn, c->ldn, c->eps, c->status};
+  const NormRows<T> a{c->x, c->W, c->Wp, c->tokens, (const bf16*)c->table, c->vocab, c->scale, (const T*)c->add, c->bias, c->post, c->mult, c->src_rows, c->gain, (T*)c->xn, c->ldn, c->raw, c->eps, c->status};
   const int chunks = c->Wp / 8, most = rows <= 2 * ca_sm_count() ? 1024 : 256;
   int nt = chunks <= most ? (chunks + 31) / 32 * 32 : most;
   if ((chunks + nt - 1) / nt > 8) nt = 1024;
@@ -693,8 +776,8 @@ static int norm_rows_launch(const CaNormRows* c, int rows, cudaStream_t s) {
 }
 
 extern "C" int cuteafd_norm_rows(const CaNormRows* c, int mode, int rows, int f32, cudaStream_t s) {
-  CA_REQUIRE(c && c->x && c->W >= 1 && c->Wp >= c->W && c->Wp % 8 == 0 && (!c->xn || (c->gain && c->ldn % 8 == 0 && c->ldn >= c->Wp)), "norm_rows: bad arguments");
-  CA_REQUIRE(mode == ROWS_EMBED ? c->tokens && c->table && c->vocab > 0 : mode == ROWS_ADD ? c->add != nullptr : mode == ROWS_GATHER && c->src_rows && c->xn, "norm_rows: mode %d without its inputs", mode);
+  CA_REQUIRE(c && c->x && c->W >= 1 && c->Wp >= c->W && c->Wp % 8 == 0 && (!c->xn || (c->ldn % 8 == 0 && c->ldn >= c->Wp)), "norm_rows: bad arguments");
+  CA_REQUIRE(mode == ROWS_EMBED ? c->tokens && c->table && c->vocab > 0 : mode == ROWS_ADD ? c->add && (!c->table || (c->tokens && c->vocab > 0)) : mode == ROWS_GATHER && c->src_rows && c->xn, "norm_rows: mode %d without its inputs", mode);
   if (rows <= 0) return CA_OK;
   if (mode == ROWS_EMBED) return f32 ? norm_rows_launch<float, ROWS_EMBED>(c, rows, s) : norm_rows_launch<bf16, ROWS_EMBED>(c, rows, s);
   if (mode == ROWS_ADD) return f32 ? norm_rows_launch<float, ROWS_ADD>(c, rows, s) : norm_rows_launch<bf16, ROWS_ADD>(c, rows, s);
@@ -711,15 +794,22 @@ extern "C" int cuteafd_rope_table(const int* positions, const float* freq, float
 
 struct CaConvQkv {
   const void* proj; const float* w; const float* bias; const float* q_norm; const float* k_norm; const void* rope; void* ring; const int* state_slot; const int* q_start;
-  const int* q_len; const int* kv_len; const int* slot_map; void* q; void* cache; int* status;
-  int ldp, q_stride, row_stride, n_slots, H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state, n_seq, max_q_len, norm, half, v_from_k; float eps;
+  const int* q_len; const int* kv_len; const int* slot_map; void* q; void* cache; int* status; void* pooled; const int* page_table;
+  int ldp, q_stride, row_stride, n_slots, H, G, dim, dp, vdim, dvp, pairs, taps, R, C, n_state, n_seq, max_q_len, norm, half, v_from_k, pool, pool_rows, pool_stride, n_pooled, max_pages; float eps;
 };
+
+template <typename T>
+static AttnExtras<T> pool_extras(int pool, int pool_rows) {
+  AttnExtras<T> x = attn_extras<T>(nullptr, 0);
+  x.pool = pool; x.pool_rows = pool_rows;
+  return x;
+}
 
 template <typename T, int V, bool HALF, bool WHOLE>
 static int conv_qkv_launch(const CaConvQkv* c, cudaStream_t s) {
   const ConvQkv<T> a{(const T*)c->proj, c->ldp, c->w, c->bias, c->q_norm, c->k_norm, (const float2*)c->rope, (T*)c->ring, c->state_slot, c->q_start, c->q_len, c->kv_len,
                      c->slot_map, (T*)c->q, c->q_stride, (T*)c->cache, c->row_stride, c->n_slots, c->H, c->G, c->dim, c->dp, c->vdim, c->dvp, c->pairs, c->taps, c->R, c->C,
-                     c->n_state, c->norm, c->v_from_k, c->eps, c->status};
+                     c->n_state, c->norm, c->v_from_k, c->eps, c->status, pool_extras<T>(c->pool, c->pool_rows), (T*)c->pooled, c->page_table, c->max_pages, c->pool_stride, c->n_pooled};
   const int units = c->H + (c->v_from_k ? 1 : 2) * c->G;
   const dim3 grid(WHOLE ? 1 : (units + 3) / 4, (c->max_q_len + HS_TILE - 1) / HS_TILE, c->n_seq);
   const int nt = WHOLE ? HS_WHOLE_WARPS * 32 : 128;
@@ -741,7 +831,9 @@ static int conv_qkv_modes(const CaConvQkv* c, cudaStream_t s) {
 extern "C" int cuteafd_conv_qkv(const CaConvQkv* c, int f32, cudaStream_t s) {
   CA_REQUIRE(c && c->proj && c->state_slot && c->q_start && c->q_len && c->kv_len && c->slot_map && c->q, "conv_qkv: null argument");
   CA_REQUIRE(c->taps >= 1 && c->taps <= HS_MAX_TAPS && (c->taps == 1 || (c->w && c->ring)) && (!c->ring || c->R >= c->taps), "conv_qkv: convolution without its weights or inputs");
-  CA_REQUIRE(c->norm >= QK_NORM_NONE && c->norm <= QK_NORM_WHOLE && (c->norm == QK_NORM_NONE || (c->q_norm && (c->G == 0 || c->k_norm))), "conv_qkv: norm without its gains");
+  CA_REQUIRE(c->norm >= QK_NORM_NONE && c->norm <= QK_NORM_WHOLE && (c->norm != QK_NORM_WHOLE || (c->q_norm && (c->G == 0 || c->k_norm))) && (c->G == 0 || !c->q_norm == !c->k_norm), "conv_qkv: norm without its gains");
+  CA_REQUIRE(!c->pooled || (c->pool >= 1 && c->pool_rows == (8 + c->pool - 1) / c->pool * 8 && c->page_table && !c->v_from_k && c->G >= 1 && c->pool_stride >= c->G * (c->dp + c->dvp) && c->pool_stride % 8 == 0),
+             "conv_qkv: pooled blocks without their rows and pages");
   CA_REQUIRE(c->H >= 1 && c->G >= 0 && (c->G == 0 || c->cache) && (!c->v_from_k || c->vdim == c->dim), "conv_qkv: bad geometry");
   CA_REQUIRE(c->dim >= 1 && c->dim <= 256 && c->vdim <= 256 && c->dp % 8 == 0 && c->dvp % 8 == 0 && c->dim <= c->dp && c->vdim <= c->dvp && c->row_stride % 8 == 0, "conv_qkv: heads of up to 256 dimensions");
   CA_REQUIRE(c->C == (c->H + c->G) * c->dim + (c->v_from_k ? 0 : c->G * c->vdim) && c->ldp >= c->C && c->q_stride >= c->H * c->dp && (c->G == 0 || c->row_stride >= c->G * (c->dp + c->dvp)), "conv_qkv: row too short");
@@ -752,6 +844,20 @@ extern "C" int cuteafd_conv_qkv(const CaConvQkv* c, int f32, cudaStream_t s) {
   if (nc <= 1) return f32 ? conv_qkv_modes<float, 2>(c, s) : conv_qkv_modes<bf16, 2>(c, s);
   if (nc <= 2) return f32 ? conv_qkv_modes<float, 4>(c, s) : conv_qkv_modes<bf16, 4>(c, s);
   return f32 ? conv_qkv_modes<float, 8>(c, s) : conv_qkv_modes<bf16, 8>(c, s);
+}
+
+// Blocks that runs of more than HS_TILE tokens complete (shorter runs: `cuteafd_conv_qkv` leaves them).
+extern "C" int cuteafd_pool_kv(const void* cache, int row_stride, int n_slots, void* pooled, int pool_stride, int n_pooled, int width, int pool, int pool_rows, const int* page_table,
+                               int max_pages, const int* kv_len, const int* q_len, int n_seq, int max_q_len, int f32, int* status, cudaStream_t s) {
+  CA_REQUIRE(cache && pooled && page_table && kv_len && q_len && pool >= 1 && pool_rows == (8 + pool - 1) / pool * 8, "pool_kv: bad arguments");
+  CA_REQUIRE(width % 8 == 0 && width <= row_stride && width <= pool_stride && row_stride % 8 == 0 && pool_stride % 8 == 0 && n_slots >= 1, "pool_kv: rows too short");
+  if (n_seq <= 0 || max_q_len <= HS_TILE) return CA_OK;
+  CA_REQUIRE(n_seq <= 65535, "pool_kv: too many sequences");
+  const dim3 grid(max_q_len / pool + 1, n_seq);
+  if (f32) CA_LAUNCH_PDL(pool_kv_kernel<float>, grid, 128, 0, s, (const float*)cache, row_stride, n_slots, (float*)pooled, pool_stride, n_pooled, width, pool_extras<float>(pool, pool_rows), page_table, max_pages, kv_len, q_len, status);
+  else CA_LAUNCH_PDL(pool_kv_kernel<bf16>, grid, 128, 0, s, (const bf16*)cache, row_stride, n_slots, (bf16*)pooled, pool_stride, n_pooled, width, pool_extras<bf16>(pool, pool_rows), page_table, max_pages, kv_len, q_len, status);
+  CA_CHECK_LAUNCH("pool_kv");
+  return CA_OK;
 }
 
 struct CaRecurrence {          // one recurrent layer's step: shared by its convolution and its scan
@@ -822,14 +928,15 @@ extern "C" int cuteafd_glu_rows(const void* g, const void* u, const float* gb, c
 }
 
 extern "C" int cuteafd_window_attention_simt(const void* q, int q_stride, const void* cache, const int* page_table, const int* kv_len, const int* q_start, const int* q_len,
-                                             void* out, int ldo, int T, int n_seq, int Hq, int Hkv, int dp, int dvp, int dv, int row_stride, int max_pages, int n_slots,
+                                             void* out, int ldo, int T, int n_seq, int Hq, int Hkv, int dp, int dvp, int dv, int row_stride, int pool_stride, int max_pages, int n_slots,
                                              int window, float scale, int f32, const CaAttnExtras* extras, int* status, cudaStream_t s) {
   CA_REQUIRE(q && cache && page_table && kv_len && q_start && q_len && out, "window_attention_simt: null argument");
   CA_REQUIRE(Hkv >= 1 && Hq % Hkv == 0 && Hq <= 65535 && dv >= 1 && dv <= dvp && dv <= 128 * WA_COLS && dp >= 1 && dp <= 4096 && row_stride >= Hkv * (dp + dvp) && ldo >= Hq * dv,
              "window_attention_simt: bad shape");
+  CA_REQUIRE(attn_extras_ok(extras, false) && (!extras || !extras->pool || pool_stride >= Hkv * (dp + dvp)), "window_attention_simt: pooled blocks without their rows, or beside kept keys");
   if (T <= 0 || n_seq <= 0) return CA_OK;
-  if (f32) CA_LAUNCH_PDL(window_attn_simt_kernel<float>, dim3(T, Hq), 128, dp * sizeof(float), s, (const float*)q, q_stride, (const float*)cache, page_table, kv_len, q_start, q_len, (float*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, max_pages, n_slots, window, scale, attn_extras<float>(extras, window), status);
-  else CA_LAUNCH_PDL(window_attn_simt_kernel<bf16>, dim3(T, Hq), 128, dp * sizeof(float), s, (const bf16*)q, q_stride, (const bf16*)cache, page_table, kv_len, q_start, q_len, (bf16*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, max_pages, n_slots, window, scale, attn_extras<bf16>(extras, window), status);
+  if (f32) CA_LAUNCH_PDL(window_attn_simt_kernel<float>, dim3(T, Hq), 128, dp * sizeof(float), s, (const float*)q, q_stride, (const float*)cache, page_table, kv_len, q_start, q_len, (float*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, pool_stride, max_pages, n_slots, window, scale, attn_extras<float>(extras, window), status);
+  else CA_LAUNCH_PDL(window_attn_simt_kernel<bf16>, dim3(T, Hq), 128, dp * sizeof(float), s, (const bf16*)q, q_stride, (const bf16*)cache, page_table, kv_len, q_start, q_len, (bf16*)out, ldo, n_seq, Hkv, Hq / Hkv, dp, dvp, dv, row_stride, pool_stride, max_pages, n_slots, window, scale, attn_extras<bf16>(extras, window), status);
   CA_CHECK_LAUNCH("window_attention_simt");
   return CA_OK;
 }

@@ -6,6 +6,8 @@
 //   stack_combine    residual += ls1 * mixer output + ls2 * weighted sum of the routed experts' rows
 //   latent_prepare   fused input projection (fp32: queries | latent | head gates | router logits) -> head-major queries, RMS-normed
 //                    latent row in the paged cache, sigmoid gates, router logits, tile table of the per-head matrix products
+//   latent_down      fused down-projections (fp32: queries' latent | latent, rotated key part) -> RMS-normed operand of the query expansion, cache row
+//   latent_split     expanded queries -> head-major unrotated parts, rotated parts, tile table of the per-head products
 //   latent_attn_simt absorbed attention for what the tcgen05 kernels do not take (fp32, ranks above 512, more than 128 heads)
 // T is the type of the matrix-product operands and of the cache: bf16, or float for the all-fp32 mode.  Rows are padded to multiples of
 // 8 elements (pad weights are zero).  (No counterpart in the reference, which has no such family; the fused shapes follow moe.cu.)
@@ -162,12 +164,94 @@ __global__ void __launch_bounds__(256) latent_prepare_kernel(const LatentPrep a,
   }
 }
 
+// ---------------------------------------------------------------- queries through a latent, rotated parts
+struct LatentDown {
+  const float* proj; int ldp, q_col, kv_col;     // [T, ldp] fp32: q_rank columns from q_col on; r latent, then rot rotated columns from kv_col on
+  const float* q_norm; const float* kv_norm;     // [q_rank], [r]
+  const float2* rope;                            // [T, rot / 2], neighbouring dimensions turn together
+  const int* slot_map;
+  int q_rank, ldq, r, rp, rot, rotp, row_stride, n_slots;       // cache row: latent in rp columns, rotated part in the rotp behind them
+  float eps; int* status;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) latent_down_kernel(const LatentDown a, T* __restrict__ cq, T* __restrict__ cache) {
+  pdl_launch(); pdl_wait();
+  __shared__ float red[32];
+  const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, slot = a.slot_map[t];
+  const float* q = a.proj + (size_t)t * a.ldp + a.q_col;
+  const float* kv = a.proj + (size_t)t * a.ldp + a.kv_col;
+  const bool ok = slot >= 0 && slot < a.n_slots;
+  if (!ok && tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, t);
+  float sq = 0.f, sk = 0.f;
+  for (int i = tid; i < a.q_rank; i += nt) sq = fmaf(q[i], q[i], sq);
+  for (int i = tid; i < a.r; i += nt) sk = fmaf(kv[i], kv[i], sk);
+  const float fq = rsqrtf(block_sum(sq, red) / (float)a.q_rank + a.eps), fk = rsqrtf(block_sum(sk, red) / (float)a.r + a.eps);
+  for (int i = tid; i < a.q_rank; i += nt) cq[(size_t)t * a.ldq + i] = to_t<T>(q[i] * fq * a.q_norm[i]);
+  if (!ok) return;
+  T* dst = cache + (size_t)slot * a.row_stride;
+  for (int i = tid; i < a.rp; i += nt) dst[i] = to_t<T>(i < a.r ? kv[i] * fk * a.kv_norm[i] : 0.f);
+  for (int i = tid; i < a.rotp; i += nt) {
+    float v = 0.f;
+    if (i < a.rot) {
+      const float2 cs = a.rope[(size_t)t * (a.rot / 2) + i / 2];
+      const float x = kv[a.r + i], y = kv[a.r + (i ^ 1)];
+      v = i & 1 ? x * cs.x + y * cs.y : x * cs.x - y * cs.y;
+    }
+    dst[a.rp + i] = to_t<T>(v);
+  }
+}
+
+struct LatentSplit {
+  const float2* rope; int T, ldt, H, d, dp, rot, rotp, ldq;     // rows of H * (d + rot) queries; [H, ldt, dp] and [H, ldt, rotp], whose pads stay as they are
+  int4* tiles; int* n_tiles; int tn;
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) latent_split_kernel(const LatentSplit a, const T* __restrict__ q, T* __restrict__ qn, T* __restrict__ qr) {
+  pdl_launch(); pdl_wait();
+  const int t = blockIdx.x, w = a.d + a.rot, tid = threadIdx.x, nt = blockDim.x;
+  const T* row = q + (size_t)t * a.ldq;
+  const float2* cs = a.rope + (size_t)t * (a.rot / 2);
+  for (int i = tid * V; i < a.H * w; i += nt * V) {
+    const int h = i / w, j = i % w;
+    if constexpr (V == 8) {
+      float v[8];
+      load8<T>(row + i, v);
+      if (j < a.d) { store8<T>(qn + ((size_t)h * a.ldt + t) * a.dp + j, v); continue; }
+      const int p = (j - a.d) / 2;
+      float o[8];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 c = cs[p + k];
+        o[2 * k] = v[2 * k] * c.x - v[2 * k + 1] * c.y; o[2 * k + 1] = v[2 * k + 1] * c.x + v[2 * k] * c.y;
+      }
+      store8<T>(qr + ((size_t)h * a.ldt + t) * a.rotp + j - a.d, o);
+    } else {
+      const float x = to_f(row[i]);
+      if (j < a.d) { qn[((size_t)h * a.ldt + t) * a.dp + j] = to_t<T>(x); continue; }
+      const int r = j - a.d;
+      const float2 c = cs[r / 2];
+      const float y = to_f(row[i - r + (r ^ 1)]);
+      qr[((size_t)h * a.ldt + t) * a.rotp + r] = to_t<T>(r & 1 ? x * c.x + y * c.y : x * c.x - y * c.y);
+    }
+  }
+  if (a.tiles) {
+    const int per = (a.T + a.tn - 1) / a.tn, n = a.H * per;
+    for (int i = t * nt + tid; i < n; i += a.T * nt) {
+      const int h = i / per, r0 = (i % per) * a.tn;
+      a.tiles[i] = make_int4(h, h * a.ldt + r0, min(a.tn, a.T - r0), 0);
+    }
+    if (t == 0 && tid == 0) *a.n_tiles = n;
+  }
+}
+
 // ---------------------------------------------------------------- absorbed latent attention on the ordinary cores
 // One block per (query row, head): scores of a page of keys (a warp takes 16 of them), online softmax, weighted sum of the page's
 // latent rows (a thread owns columns tid, tid + 128, ...).
 #define LS_COLS 8
 template <typename T>
-__global__ void __launch_bounds__(128) latent_attn_simt_kernel(const T* __restrict__ q_lat, const T* __restrict__ cache, const int* __restrict__ page_table,
+__global__ void __launch_bounds__(128) latent_attn_simt_kernel(const T* __restrict__ q_lat, const T* __restrict__ q_rope, int rotp, const float* __restrict__ sink, const T* __restrict__ cache, const int* __restrict__ page_table,
                                                                const int* __restrict__ kv_len, const int* __restrict__ q_start, const int* __restrict__ q_len,
                                                                const float* __restrict__ gate, T* __restrict__ out, int ldt, int n_seq, int H, int rp,
                                                                int row_stride, int max_pages, int n_slots, float scale, int* status) {
@@ -181,6 +265,7 @@ __global__ void __launch_bounds__(128) latent_attn_simt_kernel(const T* __restri
   const int pos = kv_len[seq] - q_len[seq] + t - q_start[seq];
   const T* qr = q_lat + ((size_t)h * ldt + t) * rp;
   for (int i = tid; i < rp; i += 128) qs[i] = to_f(qr[i]);
+  for (int i = tid; i < rotp; i += 128) qs[rp + i] = to_f(q_rope[((size_t)h * ldt + t) * rotp + i]);
   __syncthreads();
   float m = -INFINITY, l = 0.f, o[LS_COLS];
 #pragma unroll
@@ -192,7 +277,7 @@ __global__ void __launch_bounds__(128) latent_attn_simt_kernel(const T* __restri
     const int n = min(64, pos + 1 - k0);
     for (int j = warp * 16; j < warp * 16 + 16; ++j) {
       float d = 0.f;
-      if (j < n) for (int i = lane; i < rp; i += 32) d = fmaf(qs[i], to_f(base[(size_t)j * row_stride + i]), d);
+      if (j < n) for (int i = lane; i < rp + rotp; i += 32) d = fmaf(qs[i], to_f(base[(size_t)j * row_stride + i]), d);
       d = warp_sum(d);
       if (lane == 0) sc[j] = j < n ? d * scale : -INFINITY;
     }
@@ -217,6 +302,7 @@ __global__ void __launch_bounds__(128) latent_attn_simt_kernel(const T* __restri
     }
     __syncthreads();
   }
+  if (sink) l += expf(sink[h] - m);
   const float f = (l > 0.f ? 1.f / l : 0.f) * (gate ? gate[(size_t)t * H + h] : 1.f);
 #pragma unroll
   for (int c = 0; c < LS_COLS; ++c) {
@@ -281,14 +367,47 @@ extern "C" int cuteafd_latent_prepare(const float* proj, int ldp, const float* n
   return CA_OK;
 }
 
-extern "C" int cuteafd_latent_attention_simt(const void* q_lat, const void* cache, const int* page_table, const int* kv_len, const int* q_start,
+struct CaLatentDown {
+  const float* proj; const float* q_norm; const float* kv_norm; const void* rope; const int* slot_map; void* cq; void* cache; int* status;
+  int ldp, q_col, kv_col, q_rank, ldq, r, rp, rot, rotp, row_stride, n_slots, T; float eps;
+};
+
+extern "C" int cuteafd_latent_down(const CaLatentDown* c, int f32, cudaStream_t s) {
+  CA_REQUIRE(c && c->proj && c->q_norm && c->kv_norm && c->slot_map && c->cq && c->cache && (c->rot == 0 || c->rope), "latent_down: null argument");
+  CA_REQUIRE(c->q_rank >= 1 && c->q_rank <= c->ldq && c->r >= 1 && c->r <= c->rp && c->rot % 2 == 0 && c->rot <= c->rotp && c->rp + c->rotp <= c->row_stride && c->q_col + c->q_rank <= c->ldp &&
+             c->kv_col + c->r + c->rot <= c->ldp && c->q_col >= 0 && c->kv_col >= 0, "latent_down: bad shape");
+  if (c->T <= 0) return CA_OK;
+  const LatentDown a{c->proj, c->ldp, c->q_col, c->kv_col, c->q_norm, c->kv_norm, (const float2*)c->rope, c->slot_map, c->q_rank, c->ldq, c->r, c->rp, c->rot, c->rotp, c->row_stride,
+                     c->n_slots, c->eps, c->status};
+  if (f32) CA_LAUNCH_PDL(latent_down_kernel<float>, c->T, 256, 0, s, a, (float*)c->cq, (float*)c->cache);
+  else CA_LAUNCH_PDL(latent_down_kernel<bf16>, c->T, 256, 0, s, a, (bf16*)c->cq, (bf16*)c->cache);
+  CA_CHECK_LAUNCH("latent_down");
+  return CA_OK;
+}
+
+extern "C" int cuteafd_latent_split(const void* q, int ldq, const void* rope, void* qn, void* qr, void* tiles, int* n_tiles, int T, int ldt, int H, int d, int dp, int rot, int rotp, int tn,
+                                    int f32, cudaStream_t s) {
+  CA_REQUIRE(q && qn && (rot == 0 || (rope && qr)) && (!tiles || (n_tiles && tn >= 1)), "latent_split: null argument");
+  CA_REQUIRE(H >= 1 && d >= 1 && d <= dp && rot % 2 == 0 && rot >= 0 && rot <= rotp && ldq >= H * (d + rot) && ldt >= T && dp % 8 == 0 && rotp % 8 == 0, "latent_split: bad shape");
+  if (T <= 0) return CA_OK;
+  const LatentSplit a{(const float2*)rope, T, ldt, H, d, dp, rot, rotp, ldq, (int4*)tiles, n_tiles, tn};
+  const bool v8 = ((d | rot | ldq) & 7) == 0 && (((uintptr_t)q | (uintptr_t)qn | (uintptr_t)qr) & 15) == 0;
+#define LS_GO(T_, V_) CA_LAUNCH_PDL((latent_split_kernel<T_, V_>), T, 256, 0, s, a, (const T_*)q, (T_*)qn, (T_*)qr)
+  if (f32) { if (v8) LS_GO(float, 8); else LS_GO(float, 1); }
+  else if (v8) LS_GO(bf16, 8);
+  else LS_GO(bf16, 1);
+  CA_CHECK_LAUNCH("latent_split");
+  return CA_OK;
+}
+
+extern "C" int cuteafd_latent_attention_simt(const void* q_lat, const void* q_rope, int rotp, const float* sink, const void* cache, const int* page_table, const int* kv_len, const int* q_start,
                                              const int* q_len, const float* gate, void* out, int T, int ldt, int n_seq, int H, int rp, int row_stride,
                                              int max_pages, int n_slots, float scale, int f32, int* status, cudaStream_t s) {
   CA_REQUIRE(q_lat && cache && page_table && kv_len && q_start && q_len && out, "latent_attention_simt: null argument");
-  CA_REQUIRE(H >= 1 && H <= 65535 && rp >= 1 && rp <= 128 * LS_COLS && rp <= row_stride && ldt >= T, "latent_attention_simt: latent width %d (at most %d)", rp, 128 * LS_COLS);
+  CA_REQUIRE(H >= 1 && H <= 65535 && rp >= 1 && rp <= 128 * LS_COLS && rotp >= 0 && rotp <= 1024 && (rotp == 0 || q_rope) && rp + rotp <= row_stride && ldt >= T, "latent_attention_simt: latent width %d (at most %d)", rp, 128 * LS_COLS);
   if (T <= 0 || n_seq <= 0) return CA_OK;
-  if (f32) CA_LAUNCH_PDL(latent_attn_simt_kernel<float>, dim3(T, H), 128, rp * sizeof(float), s, (const float*)q_lat, (const float*)cache, page_table, kv_len, q_start, q_len, gate, (float*)out, ldt, n_seq, H, rp, row_stride, max_pages, n_slots, scale, status);
-  else CA_LAUNCH_PDL(latent_attn_simt_kernel<bf16>, dim3(T, H), 128, rp * sizeof(float), s, (const bf16*)q_lat, (const bf16*)cache, page_table, kv_len, q_start, q_len, gate, (bf16*)out, ldt, n_seq, H, rp, row_stride, max_pages, n_slots, scale, status);
+  if (f32) CA_LAUNCH_PDL(latent_attn_simt_kernel<float>, dim3(T, H), 128, (rp + rotp) * sizeof(float), s, (const float*)q_lat, (const float*)q_rope, rotp, sink, (const float*)cache, page_table, kv_len, q_start, q_len, gate, (float*)out, ldt, n_seq, H, rp, row_stride, max_pages, n_slots, scale, status);
+  else CA_LAUNCH_PDL(latent_attn_simt_kernel<bf16>, dim3(T, H), 128, (rp + rotp) * sizeof(float), s, (const bf16*)q_lat, (const bf16*)q_rope, rotp, sink, (const bf16*)cache, page_table, kv_len, q_start, q_len, gate, (bf16*)out, ldt, n_seq, H, rp, row_stride, max_pages, n_slots, scale, status);
   CA_CHECK_LAUNCH("latent_attention_simt");
   return CA_OK;
 }

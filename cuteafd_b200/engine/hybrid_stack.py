@@ -35,6 +35,7 @@ from .stack import StackBase, StackLane
 
 SCAN_CHUNK = 64             # tokens of a chunk of the recurrence's long-run form
 MAX_TAPS = 16
+POOL_ROWS = 16              # runs of up to this many tokens leave the blocks they complete in the launch that writes their keys and values
 
 
 class HybridLane(StackLane):
@@ -124,9 +125,10 @@ class HybridStackEngine(StackBase, Engine):
         return [t for t in self.rings + self.states if t is not None]
 
     @staticmethod
-    def _visible_pages(a: AttentionSpec, rows: int) -> int:
-        """Pages a run of `rows` queries can see at most through the layer's window and among kept first keys (a large number without a window)."""
-        return (a.window + rows - 1 + PAGE - 2) // PAGE + 1 + -(-a.keep_first // PAGE) if a.window else 1 << 20
+    def _visible_pages(a: AttentionSpec, rows: int, max_kv: int = 1 << 40) -> int:
+        """Pages a run of `rows` queries can see at most through the layer's window, among kept first keys and pooled blocks of a context of up to
+        `max_kv` tokens (a large number without a window)."""
+        return min(1 << 20, (a.window + rows - 1 + PAGE - 2) // PAGE + 1 + -(-a.keep_first // PAGE) + (-(-max_kv // (a.pool * PAGE)) if a.pool else 0)) if a.window else 1 << 20
 
     def attn_splits_for(self, n_seq: int, max_q_len: int, max_kv: int) -> int:
         """The largest split count a layer of the step wants (each takes no more than its window has pages)."""
@@ -134,24 +136,15 @@ class HybridStackEngine(StackBase, Engine):
             return 1
         best = 1
         for b in self.spec.blocks:
-            if b.attn is None:
+            if b.attn is None or b.attn.kind != "conv_gqa":
                 continue
             ctas = b.attn.n_kv_heads * n_seq * -(-max_q_len // max(1, 128 // (b.attn.n_heads // b.attn.n_kv_heads)))
-            pages = min(max(1, -(-max_kv // PAGE)), self._visible_pages(b.attn, max_q_len))
+            pages = min(max(1, -(-max_kv // PAGE)), self._visible_pages(b.attn, max_q_len, max_kv))
             want = max(1, min(32, 2 * self.sm_count // ctas, pages))
             if want == pages and not (b.attn.window and max_kv > b.attn.window):
                 want = 1 << (want.bit_length() - 1)        # a growing context re-captures rarely
             best = max(best, want)
         return best
-
-    def _scratch(self, n_o: int, n_ml: int):
-        """Partial outputs and (max, sum) pairs of split attention: grows to the largest need of any layer, in the eager run of a new shape."""
-        o, ml = (t.numel() if t is not None else 0 for t in (getattr(self, "part_o", None), getattr(self, "part_ml", None)))
-        if o < n_o or ml < n_ml:
-            if o:
-                self.drop_graphs()                         # captured steps hold the old scratch
-            self.part_o = torch.empty(max(o, n_o), dtype=torch.float32, device=self.device)
-            self.part_ml = torch.empty(max(ml, n_ml), dtype=torch.float32, device=self.device)
 
     # ------------------------------------------------------------------ layer program
     def _forward_single(self, sh: StepShape) -> HybridLane:
@@ -194,18 +187,21 @@ class HybridStackEngine(StackBase, Engine):
         self._attend(li, a, lw, L, b, b["o"], sh)
         self._dense(lw.wo, b["o_act"], L.mix, sh.T)
 
-    def _attend(self, li: int, a: AttentionSpec, lw: HybridLayer, L: HybridLane, b: dict, out: torch.Tensor, sh: StepShape, *, bias=None, extras=None):
-        """Projected rows b["proj"] -> convolution, norms, rotation, cache -> attended rows `out`."""
+    def _attend(self, li: int, a: AttentionSpec, lw: HybridLayer, L: HybridLane, b: dict, out: torch.Tensor, sh: StepShape, *, bias=None, extras=None, pooled=None):
+        """Projected rows b["proj"] -> convolution, norms, rotation, cache (and `pooled` blocks) -> attended rows `out`."""
         T, md, H, G, plane = sh.T, self.md, a.n_heads, a.n_kv_heads, self.plane[li]
         dp, dvp, dv = up(a.head_dim, 64), up(a.v_head_dim, 64), a.v_head_dim
         ops.conv_qkv(b["proj"], lw.conv, lw.q_norm, lw.k_norm, L.rope.get(rope_key(a)), self.rings[li], b["q"], self.kv[plane], md, H=H, G=G if a.kv_from < 0 else 0,
                      dim=a.head_dim, dp=dp, vdim=dv, dvp=dvp, pairs=a.rope_dims // 2, eps=self.spec.rms_eps, n_seq=sh.n_seq, max_q_len=sh.max_q_len, bias=bias,
-                     norm="whole" if a.qk_norm_whole else ("head" if a.qk_norm else ""), half=not a.rope_interleaved, values_are_keys=a.values_are_keys,
-                     n_slots=self.max_seqs, status=self.status)
+                     norm="whole" if a.qk_norm_whole else ("head" if a.qk_norm or a.qk_norm_unit else ""), half=not a.rope_interleaved, values_are_keys=a.values_are_keys,
+                     n_slots=self.max_seqs, pooled=pooled, pool=a.pool, status=self.status)
+        if pooled is not None and sh.max_q_len > POOL_ROWS:
+            ops.pool_kv(self.kv[plane], pooled, a.pool, md["page_table"], md["kv_len"], md["q_len"], width=G * (dp + dvp), n_seq=sh.n_seq, max_q_len=sh.max_q_len, status=self.status)
+            self.launches_per_step += 1
         where = (md["page_table"], md["kv_len"], md["q_start"], md["q_len"], out)
         shape = dict(T=T, n_seq=sh.n_seq, Hq=H, Hkv=G, dp=dp, dvp=dvp, dv=dv, window=a.window, scale=a.softmax_scale, extras=extras, status=self.status)
         if self.f32 or H // G > 128:
-            ops.window_attention_simt(b["q"], self.kv[plane], *where, **shape)
+            ops.window_attention_simt(b["q"], self.kv[plane], *where, pool_stride=pooled.stride(0) if pooled is not None else 0, **shape)
         elif sh.max_q_len >= self.PREFILL_MIN_Q and dp + 2 * dvp <= 512:
             ops.window_attention(b["q"], self.maps[plane], *where, max_q_len=sh.max_q_len, prefill=True, **shape)
         else:

@@ -51,17 +51,108 @@ class LatentLane(StackLane):
                     "n_tiles": torch.zeros(1, dtype=torch.int32, device=self.dev), "max_tiles": H * -(-cap // self.tn)}
         return self.get(("mix", H, a.head_dim, a.v_head_dim, rp, n_in), make)
 
-    def latent(self, H: int, rp: int) -> dict:
-        """Operands of the absorbed form: query and attended rows in the latent space."""
-        def make():
-            q, _ = self._operand(H * self.cap, rp)
-            o, o_act = self._operand(H * self.cap, rp)
-            return {"q": q, "o": o, "o_act": o_act}
-        return self.get(("lat", H, rp), make)
+
+class LatentAttention:
+    """Attention over paged latent rows, for engines on `StackBase`: absorbed over the rows themselves (decoding, short runs, fp32), or - long runs -
+    per head over keys and values that the context's rows are expanded to.  Optional: a rotated part behind the latent (`AttentionSpec.rope_dims`;
+    queries' parts in b["qr"]), sinks, output gates.  `b`: the lane's buffers (`q` head-major unrotated queries, `o` attended rows, `tiles`)."""
+    _ctx_plan = MlaEngine._ctx_plan
+    PREFILL_MAX_BYTES = MlaEngine.PREFILL_MAX_BYTES
+
+    @property
+    def latent_prefill_min_q(self) -> int:
+        """Query rows of a sequence from which the context is expanded (0: never)."""
+        return MlaEngine.PREFILL_MIN_Q
+
+    def _latent_fill(self, a, n_seq: int, max_q_len: int) -> int:
+        """Splits of a layer's absorbed attention that fill the machine once."""
+        rp, H = up(a.kv_lora_rank, 64), a.n_heads
+        ctas = (1 if rp <= 256 else 2) * n_seq * -(-max_q_len // max(1, 128 // min(H, 128)))
+        return max(1, self.sm_count * (2 if rp <= 128 else 1) // ctas)            # narrow latents: two CTAs per SM
+
+    def _latent_splits(self, a, n_seq: int, max_q_len: int, max_kv: int) -> int:
+        tiles, fill = max(1, -(-max_kv // PAGE)), self._latent_fill(a, n_seq, max_q_len)
+        if tiles < min(32, fill):
+            return 1 << (tiles.bit_length() - 1)       # short contexts: powers of two, so a growing context re-captures rarely
+        return max(1, min(32, fill))
+
+    def _latent_maps(self, planes: torch.Tensor, attns: list) -> torch.Tensor:
+        """TMA descriptors of the planes [., slots, row] of layers of these kinds."""
+        host = torch.zeros(len(attns), 128, dtype=torch.uint8)
+        for r, a in enumerate(attns):
+            call("cuteafd_tmap_encode_latent_rows", host[r].data_ptr(), planes[r].data_ptr(), planes.shape[1], a.latent_row, planes.shape[2])
+        return host.to(self.device)
+
+    def _latent_attention(self, a, lw, L, b: dict, rows: torch.Tensor, tmap, gate, sh: StepShape):
+        if self._expands(a, sh):
+            self._expanded(a, lw, L, b, rows, gate, sh)
+        else:
+            self._absorbed(a, lw, L, b, rows, tmap, gate, sh)
+
+    def _absorbed(self, a, lw, L, b: dict, rows: torch.Tensor, tmap, gate, sh: StepShape):
+        T, md, H, rp = sh.T, self.md, a.n_heads, up(a.kv_lora_rank, 64)
+        lat = L.latent(H, rp)
+        per = dict(tiles=b["tiles"], n_tiles=b["n_tiles"], max_tiles=H * -(-T // L.tn), status=self.status)
+        ops.tc_linear(lw.w_uk_t, b["q_act"], lat["q"], rows=H * L.cap, **per)
+        common = dict(T=T, ldt=L.cap, n_seq=sh.n_seq, H=H, rank_pad=rp, scale=a.softmax_scale, q_rope=b.get("qr"), sink=lw.sink, status=self.status)
+        where = (md["page_table"], md["kv_len"], md["q_start"], md["q_len"], gate, lat["o"])
+        if self.f32 or rp > 512 or H > 128 or a.rope_dims > 64:
+            ops.latent_attention_simt(lat["q"], rows, *where, **common)
+        else:
+            splits = min(sh.attn_splits, self._latent_fill(a, sh.n_seq, sh.max_q_len))
+            if splits > 1:
+                self._scratch(splits * T * H * rp, splits * T * H * 2)
+                self.launches_per_step += 1
+            ops.latent_attention(lat["q"], tmap, *where, max_q_len=sh.max_q_len, n_splits=splits, part_o=self.part_o if splits > 1 else None,
+                                 part_ml=self.part_ml if splits > 1 else None, **common)
+        ops.tc_linear(lw.w_uv, lat["o_act"], b["o"], rows=H * L.cap, token_major=(L.cap, a.v_head_dim), **per)
+        self.launches_per_step += 3
+
+    def _expands(self, a, sh: StepShape) -> bool:
+        """Chunks whose longest query run fills a 128-row tile expand the context into per-head keys and values (see `MlaEngine`)."""
+        least = self.latent_prefill_min_q
+        if self.f32 or not least or sh.max_q_len < least or sh.uniform or a.head_dim > 192 or a.v_head_dim > 128 or a.rope_dims > 64:
+            return False
+        if torch.cuda.is_current_stream_capturing():
+            return False
+        rows = sum(-(-n // 64) * 64 for n in self.mh["kv_len"][:sh.n_seq].tolist()) + 64
+        return rows * (a.latent_row + a.n_heads * (up(a.head_dim, 64) + up(a.v_head_dim, 64))) * 2 <= self.PREFILL_MAX_BYTES
+
+    def _pf_buffers(self, rows: int, rp: int, row: int, width: int):
+        """Context rows and their expansion (zero-filled: rows no gather ever wrote are multiplied by zero probabilities)."""
+        cap, lat, act = self._pf.get(("lat", rp, row), (0, None, None))
+        if rows + 64 > cap:
+            cap = max(1024, 1 << (rows + 64 - 1).bit_length())
+            lat = torch.zeros(cap, row, dtype=torch.bfloat16, device=self.device)
+            view = lat[:, :rp]
+            act = ActBuffer(KIND_BF16, cap, rp, 256, view, ops.encode_tmap(view, 256))
+            self._pf[("lat", rp, row)] = (cap, lat, act)
+        kcap, kvb = self._pf.get(("kvb", width), (0, None))
+        if kcap < cap:
+            kvb = torch.zeros(cap, width, dtype=torch.bfloat16, device=self.device)
+            self._pf[("kvb", width)] = (cap, kvb)
+        return cap, lat, act, kvb
+
+    def _expanded(self, a, lw, L, b: dict, rows_: torch.Tensor, gate, sh: StepShape):
+        T, md, H, n_seq = sh.T, self.md, a.n_heads, sh.n_seq
+        rp, dp, dvp, row = up(a.kv_lora_rank, 64), up(a.head_dim, 64), up(a.v_head_dim, 64), a.latent_row
+        kv, rows = self._ctx_plan(sh)
+        cap, lat, act, kvb = self._pf_buffers(rows, rp, row, H * (dp + dvp))
+        st = ptr(self.status)
+        call("cuteafd_latent_gather_ctx", ptr(rows_), ptr(md["page_table"]), ptr(self._pf_starts), ptr(md["kv_len"]), ptr(lat), n_seq, max(kv),
+             md["page_table"].shape[1], rows_.shape[0], cap, row, rows_.stride(0), st, stream())
+        ops.tc_linear(lw.ensure_kvb(), act, kvb, rows=rows, status=self.status)
+        call("cuteafd_latent_prefill_attention", ptr(b["q"]), ptr(b.get("qr")), ptr(kvb), ptr(lat), row, rp, ptr(lw.sink), cap, ptr(self._pf_starts), ptr(md["kv_len"]), ptr(md["q_start"]),
+             ptr(md["q_len"]), ptr(gate), ptr(b["o"]), T, L.cap, n_seq, sh.max_q_len, H, dp, dvp, a.v_head_dim, b["o"].stride(0), a.softmax_scale, st, stream())
+        self.launches_per_step += 3
 
 
-class LatentStackEngine(StackBase, MlaEngine):
+class LatentStackEngine(LatentAttention, StackBase, MlaEngine):
     LANE = LatentLane
+
+    @property
+    def latent_prefill_min_q(self) -> int:
+        return self.PREFILL_MIN_Q
 
     def __init__(self, weights: StackWeights, **kw):
         spec = weights.spec
@@ -83,10 +174,7 @@ class LatentStackEngine(StackBase, MlaEngine):
         self.kv = torch.zeros(len(self.runs), n, self.row, dtype=torch.float32 if self.f32 else torch.bfloat16, device=self.device)
         self.kv_tmaps = None
         if not self.f32:
-            host = torch.zeros(len(self.runs), 128, dtype=torch.uint8)
-            for r, (li, _) in enumerate(self.runs):
-                call("cuteafd_tmap_encode_latent_rows", host[r].data_ptr(), self.kv[r].data_ptr(), n, up(spec.blocks[li].attn.kv_lora_rank, 64), self.row)
-            self.kv_tmaps = host.to(self.device)
+            self.kv_tmaps = self._latent_maps(self.kv, [spec.blocks[li].attn for li, _ in self.runs])
         self._pf: dict = {}
 
     def set_inputs(self, tokens, positions, *args, **kw):
@@ -98,13 +186,7 @@ class LatentStackEngine(StackBase, MlaEngine):
     def attn_splits_for(self, n_seq: int, max_q_len: int, max_kv: int) -> int:
         if self.f32 or max_q_len > 16:
             return 1
-        H = max(b.attn.n_heads for b in self.spec.blocks)
-        ctas = (1 if self.row <= 256 else 2) * n_seq * -(-max_q_len // max(1, 128 // min(H, 128)))
-        tiles = max(1, -(-max_kv // PAGE))
-        fill = self.sm_count * (2 if self.row <= 128 else 1) // ctas            # narrow latents: two CTAs per SM
-        if tiles < min(32, fill):
-            return 1 << (tiles.bit_length() - 1)       # short contexts: powers of two, so a growing context re-captures rarely
-        return max(1, min(32, fill))
+        return max(self._latent_splits(b.attn, n_seq, max_q_len, max_kv) for b in self.spec.blocks)
 
     # ------------------------------------------------------------------ layer program
     def _emit(self, r: int, L: LatentLane):
@@ -160,70 +242,5 @@ class LatentStackEngine(StackBase, MlaEngine):
                            T=T, ldt=L.cap, H=H, d=a.head_dim, r=a.kv_lora_rank, rp=rp, E=e["logits"].shape[1] if e else 0, tn=L.tn, eps=self.spec.rms_eps,
                            status=st)
         self.launches_per_step += 1
-        if self._expands(a, sh):
-            self._prefill(r, a, lw, L, b, gate, sh)
-        else:
-            self._absorbed(r, a, lw, L, b, gate, sh)
+        self._latent_attention(a, lw, L, b, self.kv[r], self.kv_tmaps[r] if self.kv_tmaps is not None else None, gate, sh)
         self._dense(lw.wo, b["o_act"], L.mix, T)
-
-    def _absorbed(self, r: int, a, lw: StackLayer, L: LatentLane, b: dict, gate, sh: StepShape):
-        T, md, H, rp = sh.T, self.md, a.n_heads, up(a.kv_lora_rank, 64)
-        lat = L.latent(H, rp)
-        per = dict(tiles=b["tiles"], n_tiles=b["n_tiles"], max_tiles=H * -(-T // L.tn), status=self.status)
-        ops.tc_linear(lw.w_uk_t, b["q_act"], lat["q"], rows=H * L.cap, **per)
-        common = dict(T=T, ldt=L.cap, n_seq=sh.n_seq, H=H, rank_pad=rp, scale=a.softmax_scale, status=self.status)
-        if self.f32 or rp > 512 or H > 128:
-            ops.latent_attention_simt(lat["q"], self.kv[r], md["page_table"], md["kv_len"], md["q_start"], md["q_len"], gate, lat["o"], **common)
-        else:
-            po = pml = None
-            if sh.attn_splits > 1:
-                need = sh.attn_splits * T * H
-                if getattr(self, "mla_part_o", None) is None or self.mla_part_o.numel() < need * rp or self.mla_part_ml.numel() < need * 2:
-                    if getattr(self, "mla_part_o", None) is not None:
-                        self.graphs.clear()            # captured steps hold the old scratch
-                        self.census.invalidate()
-                    self.mla_part_o = torch.empty(need * self.row, dtype=torch.float32, device=self.device)
-                    self.mla_part_ml = torch.empty(need * 2, dtype=torch.float32, device=self.device)
-                po, pml = self.mla_part_o, self.mla_part_ml
-                self.launches_per_step += 1
-            ops.latent_attention(lat["q"], self.kv_tmaps[r], md["page_table"], md["kv_len"], md["q_start"], md["q_len"], gate, lat["o"], max_q_len=sh.max_q_len,
-                                 n_splits=sh.attn_splits, part_o=po, part_ml=pml, **common)
-        ops.tc_linear(lw.w_uv, lat["o_act"], b["o"], rows=H * L.cap, token_major=(L.cap, a.v_head_dim), **per)
-        self.launches_per_step += 3
-
-    # ------------------------------------------------------------------ prefill chunks: attention over the expanded context
-    def _expands(self, a, sh: StepShape) -> bool:
-        """Chunks whose longest query run fills a 128-row tile expand the context into per-head keys and values (see `MlaEngine`)."""
-        if self.f32 or not self.PREFILL_MIN_Q or sh.max_q_len < self.PREFILL_MIN_Q or sh.uniform or a.head_dim > 192 or a.v_head_dim > 128:
-            return False
-        if torch.cuda.is_current_stream_capturing():
-            return False
-        rows = sum(-(-n // 64) * 64 for n in self.mh["kv_len"][:sh.n_seq].tolist()) + 64
-        return rows * (up(a.kv_lora_rank, 64) + a.n_heads * (up(a.head_dim, 64) + up(a.v_head_dim, 64))) * 2 <= self.PREFILL_MAX_BYTES
-
-    def _pf_buffers(self, rows: int, rp: int, width: int):
-        """Context rows and their expansion (zero-filled: rows no gather ever wrote are multiplied by zero probabilities)."""
-        cap, lat, act = self._pf.get(("lat", rp), (0, None, None))
-        if rows + 64 > cap:
-            cap = max(1024, 1 << (rows + 64 - 1).bit_length())
-            lat = torch.zeros(cap, rp, dtype=torch.bfloat16, device=self.device)
-            act = ActBuffer(KIND_BF16, cap, rp, 256, lat, ops.encode_tmap(lat, 256))
-            self._pf[("lat", rp)] = (cap, lat, act)
-        kcap, kvb = self._pf.get(("kvb", width), (0, None))
-        if kcap < cap:
-            kvb = torch.zeros(cap, width, dtype=torch.bfloat16, device=self.device)
-            self._pf[("kvb", width)] = (cap, kvb)
-        return cap, lat, act, kvb
-
-    def _prefill(self, r: int, a, lw: StackLayer, L: LatentLane, b: dict, gate, sh: StepShape):
-        T, md, H, n_seq = sh.T, self.md, a.n_heads, sh.n_seq
-        rp, dp, dvp = up(a.kv_lora_rank, 64), up(a.head_dim, 64), up(a.v_head_dim, 64)
-        kv, rows = self._ctx_plan(sh)
-        cap, lat, act, kvb = self._pf_buffers(rows, rp, H * (dp + dvp))
-        st = ptr(self.status)
-        call("cuteafd_latent_gather_ctx", ptr(self.kv[r]), ptr(md["page_table"]), ptr(self._pf_starts), ptr(md["kv_len"]), ptr(lat), n_seq, max(kv),
-             md["page_table"].shape[1], self.kv.shape[1], cap, rp, self.row, st, stream())
-        ops.tc_linear(lw.ensure_kvb(), act, kvb, rows=rows, status=self.status)
-        call("cuteafd_latent_prefill_attention", ptr(b["q"]), ptr(kvb), cap, ptr(self._pf_starts), ptr(md["kv_len"]), ptr(md["q_start"]), ptr(md["q_len"]),
-             ptr(gate), ptr(b["o"]), T, L.cap, n_seq, sh.max_q_len, H, dp, dvp, a.v_head_dim, b["o"].stride(0), a.softmax_scale, st, stream())
-        self.launches_per_step += 3

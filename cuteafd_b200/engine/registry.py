@@ -34,6 +34,12 @@ def load_weights(model: str, spec: ModelSpec, device, seed: int = 1):
     """Weights of a snapshot in the forms the kernels consume, or synthetic ones for a named shape."""
     from ..models.weights import DeviceWeights
     snapshot = os.path.isdir(model)
+    if spec.stack == "mixed":
+        from ..models.mixed_stack import mixed_weights_from_masters, mixed_weights_random
+        if snapshot:
+            from ..loader.stack_checkpoint import read_mixed_masters
+            return mixed_weights_from_masters(spec, read_mixed_masters(model, spec), device)
+        return mixed_weights_random(spec, device, seed=seed)
     if spec.stack == "hyper":
         from ..models.hyper_stack import hyper_weights_from_masters, hyper_weights_random
         if snapshot:
@@ -68,6 +74,9 @@ def load_weights(model: str, spec: ModelSpec, device, seed: int = 1):
 
 
 def engine_class(spec: ModelSpec):
+    if spec.stack == "mixed":
+        from .mixed_stack import MixedStackEngine
+        return MixedStackEngine
     if spec.stack == "hyper":
         from .hyper_stack import HyperStackEngine
         return HyperStackEngine

@@ -80,6 +80,14 @@ class StackLane(Lane):
                     **({"g": torch.zeros_like(h1), "u": torch.zeros_like(h1)} if glu and self.eng.f32 else {})}
         return self.get(("moe", E, k, ff, m.activation), make)
 
+    def latent(self, H: int, rp: int) -> dict:
+        """Operands of the absorbed form: query and attended rows in the latent space."""
+        def make():
+            q, _ = self._operand(H * self.cap, rp)
+            o, o_act = self._operand(H * self.cap, rp)
+            return {"q": q, "o": o, "o_act": o_act}
+        return self.get(("lat", H, rp), make)
+
     def get(self, key, make):
         if key not in self._bufs:
             self._bufs[key] = make()
@@ -109,6 +117,19 @@ class StackBase:
     def drop_graphs(self):
         self.graphs.clear()
         self.census.invalidate()
+
+    def cache_buffers(self) -> list:
+        """What the paged cache consists of."""
+        return [self.kv]
+
+    def _scratch(self, n_o: int, n_ml: int):
+        """Partial outputs and (max, sum) pairs of split attention: grows to the largest need of any layer, in the eager run of a new shape."""
+        o, ml = (t.numel() if t is not None else 0 for t in (getattr(self, "part_o", None), getattr(self, "part_ml", None)))
+        if o < n_o or ml < n_ml:
+            if o:
+                self.drop_graphs()                         # captured steps hold the old scratch
+            self.part_o = torch.empty(max(o, n_o), dtype=torch.float32, device=self.device)
+            self.part_ml = torch.empty(max(ml, n_ml), dtype=torch.float32, device=self.device)
 
     def set_input_embeds(self, rows, vals):
         if vals is not None and len(rows):

@@ -1,4 +1,4 @@
-"""Snapshots of layer stacks: tensor names <-> the masters `models.latent_stack`, `models.hybrid_stack` and `models.hyper_stack` pack.  Matrices are [out, in].
+"""Snapshots of layer stacks: tensor names <-> the masters `models.latent_stack`, `models.hybrid_stack`, `models.hyper_stack` and `models.mixed_stack` pack.  Matrices are [out, in].
 
 Latent-attention stacks (the Bedovik design): layer i's tensors start with `l<i>.`: `norm1` (+ `.b`, `.alpha`), `mix.{q,dkv,dkv.norm,uk,uv,g,o}`, `mlp.router`, `mlp.e<j>.{up,down}`,
 `ls1`, `ls2`; the stack has `embed`, `pos`, `loop.in`, `loop.step`, `final.norm` (+ `.b`, `.alpha`) and `head`.
@@ -12,6 +12,10 @@ Hyper-connected stacks (the Vozetar design): `l<i>.norm1`, `hc1.{in,out,mix}` an
 `mlp.router`, `mlp.e<j>.{gate,up,down}`, `mlp.shared.{gate,up,down}`; attention has `{q,k,v,o}` (+ `.b`, `.conv`, `.norm`), `sink` and `g` as its kind
 has them, under `mix.` or - beside a linear mixer with `right.{q,k,v,g,o}`, `right.{a1,a2,a2.b,norm}` - under `mix.left.`; normalised mixers have
 `mix.{left,right}.out`; the stack has `embed`, `bigram`, `final.norm` and `head`.
+
+Mixed stacks (the Sikazen design): `l<i>.norm1` and, with a feed-forward, `norm2` (a number each), `mlp.{gate,up,down}`, with a side input
+`side.{gate,proj,norm}`; under `mix.` attention has `{q,k,v}` (+ `.b`) and `o`, latent attention `dq` (+ `.norm`), `uq`, `dkv` (+ `.norm`), `uk`, `uv`,
+`sink`, `o`, HGRN2 `q`, `f` (+ `.b`), `lower`, `v`, `norm`, `o`; the stack has `embed`, `side.embed`, `final.norm` (a number) and `head`.
 """
 from __future__ import annotations
 
@@ -154,4 +158,38 @@ def read_hyper_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
     if spec.pair_table is not None:
         w["pairs"] = get("bigram", spec.pair_table.buckets + 1, W)
     w["layers"] = [layer(i, b) for i, b in enumerate(spec.blocks)]
+    return w
+
+
+def read_mixed_masters(snapshot: str | Path, spec: ModelSpec) -> dict:
+    """Weights of a mixed stack's snapshot in their stored dtype, checked against the shapes the configuration implies."""
+    get, W, sd = _reader(snapshot), spec.hidden, spec.side_dim
+
+    def layer(i: int, b) -> dict:
+        a, r, p = b.attn, b.rec, f"l{i}.mix"
+        lw = {"norm1": float(get(f"l{i}.norm1"))}
+        if r is not None:
+            hk, hv = r.heads * r.dim, r.heads * r.vdim
+            lw.update(rq=get(f"{p}.q", hk, W), rf=get(f"{p}.f", hk, W), f_b=get(f"{p}.f.b", hk), lower=get(f"{p}.lower", hk), rv=get(f"{p}.v", hv, W), r_norm=get(f"{p}.norm", r.vdim),
+                      wo=get(f"{p}.o", W, hv))
+        elif a.kind == "latent":
+            H, d, dv, rk, dr = a.n_heads, a.head_dim, a.v_head_dim, a.kv_lora_rank, a.rope_dims
+            lw.update(dq=get(f"{p}.dq", a.q_lora_rank, W), dq_norm=get(f"{p}.dq.norm", a.q_lora_rank), uq=get(f"{p}.uq", H * (d + dr), a.q_lora_rank), dkv=get(f"{p}.dkv", rk + dr, W),
+                      dkv_norm=get(f"{p}.dkv.norm", rk), w_uk=get(f"{p}.uk", H * d, rk), w_uv=get(f"{p}.uv", H * dv, rk), sink=get(f"{p}.sink", H), wo=get(f"{p}.o", W, H * dv))
+        else:
+            for k, n in (("q", a.n_heads * a.head_dim), ("k", a.n_kv_heads * a.head_dim), ("v", a.n_kv_heads * a.v_head_dim)):
+                lw[f"w{k}"], lw[f"{k}_b"] = get(f"{p}.{k}", n, W), get(f"{p}.{k}.b", n)
+            lw["wo"] = get(f"{p}.o", W, a.n_heads * a.v_head_dim)
+        if b.ffn is not None:
+            ff, p = b.ffn.intermediate, f"l{i}.mlp"
+            lw.update(norm2=float(get(f"l{i}.norm2")), ws_gate=get(f"{p}.gate", ff, W), ws_up=get(f"{p}.up", ff, W), ws_down=get(f"{p}.down", W, ff))
+        if sd:
+            p = f"l{i}.side"
+            lw.update(side_gate=get(f"{p}.gate", sd, W), side_proj=get(f"{p}.proj", W, sd), side_norm=get(f"{p}.norm", W))
+        return lw
+
+    w = {"embed": get("embed", spec.vocab, W), "lm_head": get("head", spec.vocab, W), "final_norm": float(get("final.norm")),
+         "layers": [layer(i, b) for i, b in enumerate(spec.blocks)]}
+    if sd:
+        w["side"] = get("side.embed", spec.vocab, spec.n_layers * sd)
     return w

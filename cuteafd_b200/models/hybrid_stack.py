@@ -54,13 +54,13 @@ class HybridWeights(DeviceWeights):
 
 
 def rope_key(a: AttentionSpec | RecurrentSpec) -> tuple:
-    return (a.rope_dims, a.rope_theta, getattr(a, "rope_scaling", None))
+    return (a.rope_dims, a.rope_theta, getattr(a, "rope_scaling", None), getattr(a, "rope_divisor", 1.0))
 
 
 def rope_frequencies(a: AttentionSpec | RecurrentSpec) -> tuple[list, float]:
     """Angle per position of every rotated pair, and the factor on cosine and sine."""
     n, s = a.rope_dims, getattr(a, "rope_scaling", None)
-    freq = [a.rope_theta ** (-2.0 * i / n) for i in range(n // 2)]
+    freq = [a.rope_theta ** (-2.0 * i / n) / getattr(a, "rope_divisor", 1.0) for i in range(n // 2)]
     if s is None:
         return freq, 1.0
     edge = lambda turns: n * math.log(s.original / (2.0 * math.pi * turns)) / (2.0 * math.log(a.rope_theta))

@@ -119,7 +119,7 @@ class TcWeight:
     tmap: torch.Tensor              # uint8 [G, 128]
     sf: torch.Tensor | None = None  # uint8 [G, swizzled bytes]
     sf_ptrs: torch.Tensor | None = None
-    alpha: torch.Tensor | None = None   # fp32 [G]: weight global scale x activation global scale
+    alpha: torch.Tensor | None = None   # fp32 [G]: weight global scale x activation global scale (bf16, fp32: an output factor)
     inv_act_gs: torch.Tensor | None = None  # fp32 [1]: 1 / activation global scale (NVFP4)
 
     @property
@@ -332,7 +332,7 @@ def tc_linear(w: TcWeight, x: ActBuffer, y: torch.Tensor | None, *, rows: int | 
             raise ValueError("tc_linear: the fp32 kernel has a plain fp32 output only")
         gr, gc = token_major or (0, 0)
         call("cuteafd_f32_linear", ptr(x.data), x.data.stride(0), ptr(w.data), ptr(y), y.stride(0), ptr(tiles), ptr(n_tiles), max_tiles, rows, w.N, w.K,
-             ACTIVATIONS[act], float(bound), gr, gc, stream())
+             ACTIVATIONS[act], float(bound), gr, gc, ptr(w.alpha), stream())
         return y
     ws = cnt = None
     if splits > 1:
@@ -752,16 +752,35 @@ def latent_prepare(proj, norm_w, slot_map, q, cache, gate, logits, tiles, n_tile
 
 
 def latent_attention(q_lat, kv_map, page_table, kv_len, q_start, q_len, gate, out, *, T, ldt, n_seq, max_q_len, H, rank_pad, n_splits=1, part_o=None,
-                     part_ml=None, scale, status=None):
-    """Absorbed latent attention without positions over the paged cache (tcgen05); q_lat, out: head-major [H, ldt, rank_pad] bf16."""
-    call("cuteafd_latent_attention", ptr(q_lat), ptr(kv_map), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(gate), ptr(out), ptr(part_o),
+                     part_ml=None, scale, q_rope=None, sink=None, status=None):
+    """Absorbed latent attention over the paged cache (tcgen05); q_lat, out: head-major [H, ldt, rank_pad] bf16.  `q_rope` [H, ldt, 64]: rotated parts
+    (the rows' 64 columns behind the latent are the rotated key); `sink` fp32 [H]: one more logit per head."""
+    call("cuteafd_latent_attention", ptr(q_lat), ptr(q_rope), ptr(sink), ptr(kv_map), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(gate), ptr(out), ptr(part_o),
          ptr(part_ml), T, ldt, n_seq, max_q_len, H, rank_pad, page_table.shape[1], n_splits, float(scale), ptr(status), stream())
 
 
-def latent_attention_simt(q_lat, cache, page_table, kv_len, q_start, q_len, gate, out, *, T, ldt, n_seq, H, rank_pad, scale, status=None):
-    """The same on the ordinary cores: fp32 operands, latents wider than 512, more than 128 heads."""
-    call("cuteafd_latent_attention_simt", ptr(q_lat), ptr(cache), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(gate), ptr(out), T, ldt,
+def latent_attention_simt(q_lat, cache, page_table, kv_len, q_start, q_len, gate, out, *, T, ldt, n_seq, H, rank_pad, scale, q_rope=None, sink=None, status=None):
+    """The same on the ordinary cores: fp32 operands, latents wider than 512, more than 128 heads, rotated parts [H, ldt, any multiple of 8]."""
+    call("cuteafd_latent_attention_simt", ptr(q_lat), ptr(q_rope), q_rope.shape[-1] if q_rope is not None else 0, ptr(sink), ptr(cache), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(gate), ptr(out), T, ldt,
          n_seq, H, rank_pad, cache.stride(0), page_table.shape[1], cache.shape[0], float(scale), _f32(q_lat), ptr(status), stream())
+
+
+def latent_down(proj, q_col: int, kv_col: int, q_norm, kv_norm, rope, slot_map, cq, cache, *, T, r, rp, rot, eps, status=None):
+    """Splits fused down-projection rows (fp32: the queries' latent from column `q_col`, the latent and the rotated key part from `kv_col`): the RMS-normed
+    queries' latent into `cq` [., q_rank_pad], the normed latent and the rotated part (neighbouring pairs) into the paged cache rows."""
+    _chk(proj, torch.float32, "proj")
+    a = native.LatentDown()
+    a.proj, a.q_norm, a.kv_norm, a.rope, a.slot_map, a.cq, a.cache, a.status = (ptr(t) for t in (proj, q_norm, kv_norm, rope, slot_map, cq, cache, status))
+    a.ldp, a.q_col, a.kv_col, a.q_rank, a.ldq, a.r, a.rp, a.rot, a.rotp = proj.stride(0), q_col, kv_col, q_norm.numel(), cq.stride(0), r, rp, rot, -(-rot // 64) * 64
+    a.row_stride, a.n_slots, a.T, a.eps = cache.stride(0), cache.shape[0], T, eps
+    call("cuteafd_latent_down", ctypes.addressof(a), _f32(cq), stream())
+
+
+def latent_split(q, rope, qn, qr, tiles, n_tiles, *, T, ldt, H, d, rot, tn):
+    """Expanded query rows [T, H * (d + rot)] -> head-major unrotated parts [H, ldt, qn.shape[-1]], rotated parts [H, ldt, qr.shape[-1]] (neighbouring
+    pairs) and the tile table of the products grouped over heads."""
+    call("cuteafd_latent_split", ptr(q), q.stride(0), ptr(rope), ptr(qn), ptr(qr), ptr(tiles), ptr(n_tiles), T, ldt, H, d, qn.shape[-1], rot, qr.shape[-1] if qr is not None else 0, tn,
+         _f32(q), stream())
 
 
 # ------------------------------------------------------------------ hybrid stacks: norms around sub-layers, short convolutions, recurrence, windows
@@ -769,24 +788,25 @@ ROWS_EMBED, ROWS_ADD, ROWS_GATHER = 0, 1, 2
 
 
 def norm_rows(x, W: int, rows: int, *, f32: bool, eps: float, gain=None, xn=None, tokens=None, table=None, add=None, bias=None, post=None, mult: float = 1.0,
-              src_rows=None, status=None):
-    """Residual rows (fp32 [., Wp], norms average over W): x = table[token] with `tokens`; x += mult * norm(add + bias) with `add` (`post`: gain of
-    that norm, None = no norm); the rows listed in `src_rows` otherwise.  `xn` receives the rows RMS-normed with `gain`."""
+              src_rows=None, scale: float = 1.0, raw: bool = False, status=None):
+    """Residual rows (fp32 [., Wp], norms average over W): x += mult * norm(add + bias) with `add` (`post`: gain of that norm, None = no norm), and with
+    `tokens` and `table` besides + scale * table[token]; x = scale * table[token] with `tokens` alone; the rows listed in `src_rows` otherwise.  `xn`
+    receives the rows RMS-normed with `gain` (None: without gains), or as they are (`raw`)."""
     _chk(x, torch.float32, "x")
     a = native.NormRows()
     a.x, a.W, a.Wp, a.eps, a.mult, a.status = ptr(x), W, x.shape[1], eps, mult, ptr(status)
-    a.gain, a.xn, a.ldn = ptr(gain), ptr(xn), xn.stride(0) if xn is not None else 0
+    a.gain, a.xn, a.ldn, a.scale, a.raw = ptr(gain), ptr(xn), xn.stride(0) if xn is not None else 0, float(scale), 1 if raw else 0
     mode = ROWS_GATHER
     if tokens is not None:
         _chk(tokens, torch.int32, "tokens"); _chk(table, torch.bfloat16, "table")
         if table.shape[1] != x.shape[1]:
             raise ValueError("norm_rows: table and residual rows differ in width")
         mode, a.tokens, a.table, a.vocab = ROWS_EMBED, ptr(tokens), ptr(table), table.shape[0]
-    elif add is not None:
+    if add is not None:
         if add.shape[1] != x.shape[1]:
             raise ValueError("norm_rows: added rows and residual rows differ in width")
         mode, a.add, a.bias, a.post = ROWS_ADD, ptr(add), ptr(bias), ptr(post)
-    else:
+    elif tokens is None:
         a.src_rows = ptr(src_rows)
     call("cuteafd_norm_rows", ctypes.addressof(a), mode, rows, 1 if f32 else 0, stream())
 
@@ -801,11 +821,12 @@ QK_NORMS = {"": 0, "head": 1, "whole": 2}
 
 
 def conv_qkv(proj, w, q_norm, k_norm, rope, ring, q, cache, meta: dict, *, H, G, dim, dp, vdim, dvp, pairs, eps, n_seq, max_q_len, bias=None, norm: str = "head",
-             half: bool = False, values_are_keys: bool = False, n_slots: int = 0, status=None):
+             half: bool = False, values_are_keys: bool = False, n_slots: int = 0, pooled=None, pool: int = 0, status=None):
     """Short causal convolution over projected query / key / value rows (+ `bias`), norms, rotation; queries to `q` [., H * dp], keys and values to
     the paged `cache` rows.  `w` None: no convolution.  `ring` [slots, depth + taps - 1, channels]: inputs by position (None with one tap: give the
-    number of state slots).  `norm`: "head" (gains [dim]), "whole" (over all heads at once, gains [H * dim] / [G * dim]) or "".  `half`: dimensions i
+    number of state slots).  `norm`: "head" (gains [dim], None: without), "whole" (over all heads at once, gains [H * dim] / [G * dim]) or "".  `half`: dimensions i
     and i + pairs turn together instead of neighbours.  `values_are_keys`: no value channels, the keys in front of norm and rotation are the values.
+    `pooled`, `pool`: rows of the pooled blocks of that many tokens (see `pool_kv`), of which short runs leave those that they complete.
     `meta`: the step's device inputs.  G = 0: queries only."""
     if w is not None:
         _chk(w, torch.float32, "w")
@@ -818,9 +839,24 @@ def conv_qkv(proj, w, q_norm, k_norm, rope, ring, q, cache, meta: dict, *, H, G,
     a.row_stride, a.n_slots = (cache.stride(0), cache.shape[0]) if cache is not None else (8, 0)
     a.taps, a.C, a.n_seq, a.max_q_len = w.shape[0] if w is not None else 1, (H + G) * dim + (0 if values_are_keys else G * vdim), n_seq, max_q_len
     a.n_state, a.R = ring.shape[:2] if ring is not None else (n_slots, a.taps)
+    if pooled is not None:
+        table = meta["page_table"]
+        a.pooled, a.page_table, a.pool, a.pool_rows, a.pool_stride, a.n_pooled, a.max_pages = ptr(pooled), ptr(table), pool, pooled_page_rows(pool), pooled.stride(0), pooled.shape[0], table.shape[1]
     if (w is not None and w.shape[1] != a.C) or (ring is not None and (ring.shape[2] != a.C or not ring.is_contiguous())):
         raise ValueError("conv_qkv: convolution weights, ring and heads differ in channels")
     call("cuteafd_conv_qkv", ctypes.addressof(a), _f32(proj), stream())
+
+
+def pooled_page_rows(pool: int) -> int:
+    """Pooled rows that belong to a page of 64 tokens: whole strips of eight blocks, each with the page of its first token."""
+    return 8 * -(-8 // pool)
+
+
+def pool_kv(cache, pooled, pool: int, page_table, kv_len, q_len, *, width: int, n_seq: int, max_q_len: int, status=None):
+    """Means over blocks of `pool` cached rows (`width` elements each) for every block that a run of more than 16 tokens completes; `pooled`
+    [pages * pooled_page_rows(pool), .] is addressed through the page table (see `csrc/attn_extras.cuh`)."""
+    call("cuteafd_pool_kv", ptr(cache), cache.stride(0), cache.shape[0], ptr(pooled), pooled.stride(0), pooled.shape[0], width, pool, pooled_page_rows(pool), ptr(page_table),
+         page_table.shape[1], ptr(kv_len), ptr(q_len), n_seq, max_q_len, _f32(cache), ptr(status), stream())
 
 
 def recurrence_arg(x, y, x_b, y_b, conv, conv_b, ring, state, u, gates, gates_b, decay, agg, out, meta: dict, *, blocks, T, ldt, tiles, n_tiles, tn, n_seq, max_q_len,
@@ -853,21 +889,25 @@ def glu_rows(g, u, gate_b, up_b, out, rows: int, limit: float):
     call("cuteafd_glu_rows", ptr(g), ptr(u), ptr(gate_b), ptr(up_b), ptr(out), rows, g.stride(0), out.stride(0), g.shape[1], float(limit), _f32(g), stream())
 
 
-def encode_window_maps(rows: torch.Tensor, Hkv: int, dp: int, dvp: int) -> torch.Tensor:
-    """TMA descriptors (uint8 [2, 128]: keys, values) of one layer's store [slots, row]: Hkv key heads of dp elements, then Hkv value heads of dvp."""
+def encode_window_maps(rows: torch.Tensor, Hkv: int, dp: int, dvp: int, box_rows: int = 64) -> torch.Tensor:
+    """TMA descriptors (uint8 [2, 128]: keys, values) of one layer's store [slots, row]: Hkv key heads of dp elements, then Hkv value heads of dvp;
+    `box_rows` 8: of its pooled blocks."""
     host = torch.zeros(2, 128, dtype=torch.uint8)
-    call("cuteafd_tmap_encode_heads", host[0].data_ptr(), rows.data_ptr(), dp, Hkv, rows.stride(0), rows.shape[0])
-    call("cuteafd_tmap_encode_heads", host[1].data_ptr(), rows.data_ptr() + Hkv * dp * rows.element_size(), dvp, Hkv, rows.stride(0), rows.shape[0])
+    call("cuteafd_tmap_encode_heads", host[0].data_ptr(), rows.data_ptr(), dp, Hkv, rows.stride(0), rows.shape[0], box_rows)
+    call("cuteafd_tmap_encode_heads", host[1].data_ptr(), rows.data_ptr() + Hkv * dp * rows.element_size(), dvp, Hkv, rows.stride(0), rows.shape[0], box_rows)
     return host.to(rows.device)
 
 
-def attn_extras(sink=None, gate=None, per_value: bool = False, keep_first: int = 0, out_scale: float = 1.0):
+def attn_extras(sink=None, gate=None, per_value: bool = False, keep_first: int = 0, out_scale: float = 1.0, pooled=None, pool_maps=None, pool: int = 0):
     """What an attention layer has besides: a `sink` logit per head (fp32 [Hq]); `gate` logits (column view of the projection rows: one per head, or
-    `per_value` one per output value) whose sigmoid multiplies the output; the sequence's first `keep_first` keys visible behind the window; a
-    constant factor on the output."""
+    `per_value` one per output value) whose sigmoid multiplies the output; the sequence's first `keep_first` keys visible behind the window; or one key
+    and value for each block of `pool` tokens wholly in front of it (`pooled`: rows of the blocks, `pool_maps`: their descriptors); a constant factor
+    on the output."""
     x = native.AttnExtras()
     x.sink, x.gate, x.ldg = ptr(sink), ptr(gate), gate.stride(0) if gate is not None else 0
     x.gate_values, x.keep_first, x.out_scale = 1 if per_value else 0, keep_first, float(out_scale)
+    if pool:
+        x.pooled, x.pool_maps, x.pool, x.pool_rows = ptr(pooled), ptr(pool_maps), pool, pooled_page_rows(pool)
     return x
 
 
@@ -887,10 +927,10 @@ def window_attention(q, maps, page_table, kv_len, q_start, q_len, out, *, T, n_s
         call("cuteafd_window_attention", *head, ptr(part_o), ptr(part_ml), *shape, n_splits, window, float(scale), _extras(extras), ptr(status), stream())
 
 
-def window_attention_simt(q, cache, page_table, kv_len, q_start, q_len, out, *, T, n_seq, Hq, Hkv, dp, dvp, dv, window=0, scale, extras=None, status=None):
-    """The same on the ordinary cores: fp32, heads wider than 256, groups of more than 128."""
+def window_attention_simt(q, cache, page_table, kv_len, q_start, q_len, out, *, T, n_seq, Hq, Hkv, dp, dvp, dv, window=0, scale, extras=None, pool_stride=0, status=None):
+    """The same on the ordinary cores: fp32, heads wider than 256, groups of more than 128; `pool_stride`: elements between two pooled rows."""
     call("cuteafd_window_attention_simt", ptr(q), q.stride(0), ptr(cache), ptr(page_table), ptr(kv_len), ptr(q_start), ptr(q_len), ptr(out), out.stride(0), T, n_seq, Hq,
-         Hkv, dp, dvp, dv, cache.stride(0), page_table.shape[1], cache.shape[0], window, float(scale), _f32(q), _extras(extras), ptr(status), stream())
+         Hkv, dp, dvp, dv, cache.stride(0), pool_stride, page_table.shape[1], cache.shape[0], window, float(scale), _f32(q), _extras(extras), ptr(status), stream())
 
 
 # ------------------------------------------------------------------ hyper-connected stacks: stream boundaries, linear attention with a decay
@@ -939,10 +979,11 @@ def hyper_rows(x, W: int, rows: int, *, f32: bool, eps: float, next_in=None, gai
     call("cuteafd_hyper_rows", ctypes.addressof(r), mode, rows, 1 if f32 else 0, stream())
 
 
-def decay_scan_arg(q, k, v, g, state, tags, ring, out, meta: dict, *, H, dim, vdim, n_seq, max_q_len, eps, rope=None, pairs=0, q_scale=1.0, k_scale=1.0, decay=None, low_rank=None,
+def decay_scan_arg(q, k, v, g, state, tags, ring, out, meta: dict, *, H, dim, vdim, n_seq, max_q_len, eps, rope=None, pairs=0, q_scale=1.0, k_scale=1.0, decay=None, low_rank=None, forget=None,
                    tau=1.0, norm=None, out_scale=1.0, chunks=None, T: int = 0, status=None):
     """Arguments of `decay_scan`: q, k, v, g column views of one projection buffer; `decay` fp32 [H] (constant) or `low_rank` = (a1 column view, a2 fp32
-    [H * dim, rank], bias fp32 [H * dim]): decay sigmoid(a2 a1 + bias) ** (1 / tau) per key channel; `state` [slots, 2, H, dim, vp] with `tags`
+    [H * dim, rank], bias fp32 [H * dim]): decay sigmoid(a2 a1 + bias) ** (1 / tau) per key channel, or `forget` = (bias, lower bound; fp32 [H * dim]):
+    HGRN2, where k are the forget gate's logits and q passes SiLU; g None: no output gate; `state` [slots, 2, H, dim, vp] with `tags`
     [slots, H, 2] (positions), `ring` [slots, depth, H, 2 dim + vp].  `chunks`: scratch of `scan_scratch`, with which long runs of a step of
     `T` rows take the chunk kernels (bf16, heads of up to 128 x 256)."""
     a = native.DecayScan()
@@ -955,7 +996,9 @@ def decay_scan_arg(q, k, v, g, state, tags, ring, out, meta: dict, *, H, dim, vd
         setattr(a, n, ptr(t))
     if low_rank is not None:
         a.a1, a.a2, a.a2_b, a.rank = ptr(low_rank[0]), ptr(low_rank[1]), ptr(low_rank[2]), low_rank[1].shape[1]
-    if not q.stride(0) == k.stride(0) == v.stride(0) == g.stride(0):
+    if forget is not None:
+        a.forget_b, a.lower = ptr(forget[0]), ptr(forget[1])
+    if not q.stride(0) == k.stride(0) == v.stride(0) == (g.stride(0) if g is not None else v.stride(0)):
         raise ValueError("decay_scan: q, k, v and gate are columns of one buffer")
     a.ldp, a.pairs, a.ldo, a.H, a.dim, a.vdim, a.vp, a.depth, a.n_state = q.stride(0), pairs, out.stride(0), H, dim, vdim, state.shape[-1], ring.shape[1], state.shape[0]
     a.n_seq, a.max_q_len, a.q_scale, a.k_scale, a.inv_tau, a.eps, a.out_scale = n_seq, max_q_len, q_scale, k_scale, 1.0 / tau, eps, out_scale
@@ -973,6 +1016,12 @@ def scan_scratch(rows: int, n_seq: int, H: int, dim: int, vdim: int, device) -> 
 
 def decay_scan(a, *, f32: bool):
     call("cuteafd_decay_scan", ctypes.addressof(a), 1 if f32 else 0, stream())
+
+
+def side_gate(z, tokens, table, col: int, n: int, out, rows: int, *, status=None):
+    """out[t, :n] = gelu_tanh(z[t, :n]) * table[token, col : col + n] (z fp32, the table bf16)."""
+    _chk(z, torch.float32, "z"); _chk(tokens, torch.int32, "tokens"); _chk(table, torch.bfloat16, "table")
+    call("cuteafd_side_gate", ptr(z), z.stride(0), ptr(tokens), ptr(table), table.stride(0), col, n, table.shape[0], ptr(out), out.stride(0), rows, _f32(out), ptr(status), stream())
 
 
 def silu_rows(g, u, out, rows: int):

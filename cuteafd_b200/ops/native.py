@@ -100,29 +100,33 @@ _PROTOS = {
     "cuteafd_flag_pingpong": [P, P, C.c_uint, I, I, C.c_ulonglong, P, P, P],
     "cuteafd_dispatch_tok_push": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, C.c_uint, P, P],
     "cuteafd_combine_push_lanes": [P, P, P, P, P, P, P, I, I, I, I, I, I, C.c_uint, P, P],
-    "cuteafd_latent_attention": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
+    "cuteafd_latent_attention": [P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P],
     "cuteafd_tmap_encode_latent_rows": [P, P, U64, U64, U64],
-    "cuteafd_latent_prefill_attention": [P, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
+    "cuteafd_latent_prefill_attention": [P, P, P, P, I, I, P, L, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P],
     "cuteafd_latent_gather_ctx": [P, P, P, P, P, I, I, I, L, L, I, I, P, P],
-    "cuteafd_latent_attention_simt": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
+    "cuteafd_latent_attention_simt": [P, P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
     "cuteafd_latent_prepare": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P],
     "cuteafd_stack_embed": [P, P, P, P, P, P, I, I, I, I, I, I, P, P, P],
     "cuteafd_stack_stream": [P, P, P, I, I, I, P, P],
     "cuteafd_stack_combine": [P, P, P, P, P, P, P, I, I, I, I, P, P],
-    "cuteafd_f32_linear": [P, I, P, P, I, P, P, I, I, I, I, I, F, I, I, P],
+    "cuteafd_f32_linear": [P, I, P, P, I, P, P, I, I, I, I, I, F, I, I, P, P],
     "cuteafd_norm_rows": [P, I, I, I, P],
     "cuteafd_rope_table": [P, P, F, I, P, I, P],
     "cuteafd_conv_qkv": [P, I, P],
     "cuteafd_rglru_conv": [P, I, P],
     "cuteafd_lru_scan": [P, I, P],
     "cuteafd_glu_rows": [P, P, P, P, P, I, I, I, I, F, I, P],
-    "cuteafd_window_attention_simt": [P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P],
+    "cuteafd_window_attention_simt": [P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P, P],
     "cuteafd_window_attention": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P, P],
     "cuteafd_window_prefill_attention": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, P, P, P],
     "cuteafd_hyper_rows": [P, I, I, I, P],
     "cuteafd_decay_scan": [P, I, P],
     "cuteafd_silu_rows": [P, P, P, I, I, I, I, I, P],
-    "cuteafd_tmap_encode_heads": [P, P, I, I, U64, U64],
+    "cuteafd_tmap_encode_heads": [P, P, I, I, U64, U64, I],
+    "cuteafd_pool_kv": [P, I, I, P, I, I, I, I, I, P, I, P, P, I, I, I, P, P],
+    "cuteafd_latent_down": [P, I, P],
+    "cuteafd_latent_split": [P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
+    "cuteafd_side_gate": [P, I, P, P, I, I, I, I, P, I, I, I, P, P],
     "cuteafd_tc_linear": [I, I, I, P, P, P, P, P, P, I, P, P, P, P, I, P, P, I, I, I, I, I, I, P, P, P, I, P, P],
 }
 
@@ -156,18 +160,23 @@ def _fields(pointers: str, ints: str, floats: str = "") -> list:
 
 class NormRows(C.Structure):
     """`cuteafd_norm_rows` (`CaNormRows` of the C ABI)."""
-    _fields_ = _fields("x tokens table add bias post src_rows gain xn status", "W Wp vocab ldn", "mult eps")
+    _fields_ = _fields("x tokens table add bias post src_rows gain xn status", "W Wp vocab ldn raw", "mult eps scale")
 
 
 class ConvQkv(C.Structure):
     """`cuteafd_conv_qkv` (`CaConvQkv` of the C ABI)."""
-    _fields_ = _fields("proj w bias q_norm k_norm rope ring state_slot q_start q_len kv_len slot_map q cache status",
-                       "ldp q_stride row_stride n_slots H G dim dp vdim dvp pairs taps R C n_state n_seq max_q_len norm half v_from_k", "eps")
+    _fields_ = _fields("proj w bias q_norm k_norm rope ring state_slot q_start q_len kv_len slot_map q cache status pooled page_table",
+                       "ldp q_stride row_stride n_slots H G dim dp vdim dvp pairs taps R C n_state n_seq max_q_len norm half v_from_k pool pool_rows pool_stride n_pooled max_pages", "eps")
 
 
 class AttnExtras(C.Structure):
-    """Sink, output gate, kept first keys and output factor of a windowed attention call (`CaAttnExtras` of the C ABI)."""
-    _fields_ = _fields("sink gate", "ldg gate_values keep_first", "out_scale")
+    """Sink, output gate, kept first keys or pooled blocks, and output factor of a windowed attention call (`CaAttnExtras` of the C ABI)."""
+    _fields_ = _fields("sink gate pooled pool_maps", "ldg gate_values keep_first pool pool_rows", "out_scale")
+
+
+class LatentDown(C.Structure):
+    """`cuteafd_latent_down` (`CaLatentDown` of the C ABI)."""
+    _fields_ = _fields("proj q_norm kv_norm rope slot_map cq cache status", "ldp q_col kv_col q_rank ldq r rp rot rotp row_stride n_slots T", "eps")
 
 
 class HyperRows(C.Structure):
@@ -178,7 +187,7 @@ class HyperRows(C.Structure):
 
 class DecayScan(C.Structure):
     """`cuteafd_decay_scan` (`CaDecayScan` of the C ABI)."""
-    _fields_ = _fields("q k v g rope decay a1 a2 a2_b norm state tags ring state_slot q_start q_len kv_len out chunk_state chunk_decay chunk_tiles status",
+    _fields_ = _fields("q k v g rope decay a1 a2 a2_b norm state tags ring state_slot q_start q_len kv_len out chunk_state chunk_decay chunk_tiles status forget_b lower",
                        "ldp pairs rank ldo H dim vdim vp depth n_state n_seq max_q_len T chunks", "q_scale k_scale inv_tau eps out_scale")
 
 

@@ -222,7 +222,7 @@ def test_expanding_prefill_attention(H, d, dv, r, gate):
         assert torch.equal(lat[ctx[s]:ctx[s] + n, :r].float().cpu(), pg.rows[s])
     ops.tc_linear(w, ops.ActBuffer.wrap_bf16(lat, 256), kvb, rows=tot, status=status)
     qd, gd = q.reshape(H * ldt, dp).to(DEV), g.to(DEV) if gate else None
-    call("cuteafd_latent_prefill_attention", ptr(qd), ptr(kvb), cap, ptr(cs), ptr(kl), ptr(qs), ptr(ql), ptr(gd), ptr(out), T, ldt, 3, max(q_lens), H, dp, dvp, dv,
+    call("cuteafd_latent_prefill_attention", ptr(qd), None, ptr(kvb), None, 0, 0, None, cap, ptr(cs), ptr(kl), ptr(qs), ptr(ql), ptr(gd), ptr(out), T, ldt, 3, max(q_lens), H, dp, dvp, dv,
          ldo, 0.8, ptr(status), stream())
     assert int(status[0]) == 0
     got = out.float().cpu()

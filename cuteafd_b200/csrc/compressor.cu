@@ -32,33 +32,38 @@ __global__ void __launch_bounds__(1024) compress_pool_kernel(const CompressArgs 
   const int qlen = a.q_len[s], p0 = a.pos0[s], m = a.ratio;
   if (qlen <= 0) return;
   const int first_block = p0 / m, last_block = (p0 + qlen - 1) / m;
-  const int b = first_block + blockIdx.x;
-  if (b > last_block) return;
-  const int lo = max(b * m, p0), hi = min((b + 1) * m, p0 + qlen);       // positions of this block present in the step
-  const bool live = d < a.D;
-  float mx = -INFINITY, l = 0.f, acc = 0.f;
-  float* st = a.state + (size_t)a.state_slot[s] * 3 * a.D;
-  if (live && lo > b * m) { mx = st[d]; l = st[a.D + d]; acc = st[2 * a.D + d]; }           // the block was opened by an earlier step
-  if (live) {
-    for (int p = lo; p < hi; ++p) {
-      const size_t row = (size_t)(a.q_start[s] + p - p0) * a.D + d;
-      const float sc = a.scores[row], v = a.kv[row];
-      const float nm = fmaxf(mx, sc);
-      const float r = (mx == -INFINITY) ? 0.f : __expf(mx - nm), e = __expf(sc - nm);
-      l = l * r + e;
-      acc = acc * r + e * v;
-      mx = nm;
+  const int end = p0 + qlen, mine = first_block + blockIdx.x;
+  if (mine > last_block) return;
+  const bool live = d < a.D, open = end < (last_block + 1) * m;           // open: the step leaves its last block unfinished
+  // The last block's state takes the place of the first one's: where both have one, the same thread block reads the old before it leaves the new.
+  if (open && mine == last_block && mine != first_block) return;
+  for (int b = mine; b <= last_block; b += last_block - first_block) {
+    const int lo = max(b * m, p0), hi = min((b + 1) * m, end);            // positions of this block present in the step
+    float mx = -INFINITY, l = 0.f, acc = 0.f;
+    float* st = a.state + (size_t)a.state_slot[s] * 3 * a.D;
+    if (live && lo > b * m) { mx = st[d]; l = st[a.D + d]; acc = st[2 * a.D + d]; }         // the block was opened by an earlier step
+    if (live) {
+      for (int p = lo; p < hi; ++p) {
+        const size_t row = (size_t)(a.q_start[s] + p - p0) * a.D + d;
+        const float sc = a.scores[row], v = a.kv[row];
+        const float nm = fmaxf(mx, sc);
+        const float r = (mx == -INFINITY) ? 0.f : __expf(mx - nm), e = __expf(sc - nm);
+        l = l * r + e;
+        acc = acc * r + e * v;
+        mx = nm;
+      }
     }
-  }
-  if (hi < (b + 1) * m) {            // still open: only the last block of a sequence's step can be
-    if (live) { st[d] = mx; st[a.D + d] = l; st[2 * a.D + d] = acc; }
-    return;
-  }
-  const float pooled = live ? __bfloat162float(__float2bfloat16(acc / l)) : 0.f;
-  const float ss = block_sum(pooled * pooled, red);
-  if (live) {
-    const int orow = a.out_start[s] + (b - first_block);
-    a.out[(size_t)orow * a.D + d] = __float2bfloat16(pooled * rsqrtf(ss / a.D + a.eps) * a.norm_w[d]);
+    if (hi < (b + 1) * m) {          // still open: only the last block of a sequence's step can be
+      if (live) { st[d] = mx; st[a.D + d] = l; st[2 * a.D + d] = acc; }
+      return;
+    }
+    const float pooled = live ? __bfloat162float(__float2bfloat16(acc / l)) : 0.f;
+    const float ss = block_sum(pooled * pooled, red);
+    if (live) {
+      const int orow = a.out_start[s] + (b - first_block);
+      a.out[(size_t)orow * a.D + d] = __float2bfloat16(pooled * rsqrtf(ss / a.D + a.eps) * a.norm_w[d]);
+    }
+    if (!open || b != first_block || last_block == first_block) return;
   }
 }
 

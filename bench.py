@@ -153,7 +153,7 @@ def main():
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--config", default="qwen3-235b-decode", choices=["qwen3-235b-decode", "deepseek-v3-decode", "deepseek-v3-plain", "deepseek-v3-ttft", "hybrid-gdn-decode", "hybrid-kda-decode", "bedovik", "tudilix", "vozetar"],
+    ap.add_argument("--config", default="qwen3-235b-decode", choices=["qwen3-235b-decode", "deepseek-v3-decode", "deepseek-v3-plain", "deepseek-v3-ttft", "hybrid-gdn-decode", "hybrid-kda-decode", "bedovik", "tudilix", "vozetar", "sikazen"],
                     help="deepseek-v3-plain: one-token-per-step decode of the DeepSeek-V3 shape through the generic path (any --layout; no drafter)")
     ap.add_argument("--ttft-prompt", type=int, default=32768); ap.add_argument("--ttft-shared", type=int, default=28672)
     ap.add_argument("--ttft-sessions", type=int, default=8); ap.add_argument("--ttft-decode", type=int, default=256)
@@ -164,6 +164,8 @@ def main():
                     help="--config tudilix: layer sizes to measure, each beside the hybrid gated delta-rule stack of equal size (1 GPU)")
     ap.add_argument("--vozetar-size", default="all", choices=["all", "small", "medium", "moe", "large"],
                     help="--config vozetar: layer sizes to measure, each beside the hybrid per-channel delta-rule stack of equal size (1 GPU)")
+    ap.add_argument("--sikazen-size", default="all", choices=["all", "small", "medium", "large"],
+                    help="--config sikazen: layer sizes to measure, each beside the hyper-connected and the latent attention stack of equal size (1 GPU)")
     ap.add_argument("--batch-per-gpu", type=int, default=16)
     ap.add_argument("--batch-total", type=int, default=0, help="fixed global batch instead of a per-GPU batch (DeepSeek-V3 decode: 1 or 64)")
     ap.add_argument("--context", type=int, default=4096)
@@ -199,13 +201,15 @@ def main():
     if world != args.gpus:
         raise SystemExit(f"--gpus {args.gpus} but WORLD_SIZE={world}")
 
-    if args.config in ("bedovik", "tudilix", "vozetar"):
+    if args.config in ("bedovik", "tudilix", "vozetar", "sikazen"):
         if world > 1:
             raise SystemExit(f"--config {args.config} runs on one GPU")
         if args.config == "bedovik":
             from cuteafd_b200.bench.latent_stack import bench_line
         elif args.config == "tudilix":
             from cuteafd_b200.bench.hybrid_stack import bench_line
+        elif args.config == "sikazen":
+            from cuteafd_b200.bench.mixed_stack import bench_line
         else:
             from cuteafd_b200.bench.hyper_stack import bench_line
         print(json.dumps(bench_line(args, ClockSampler(local))))

@@ -52,7 +52,8 @@ def make_engine(spec: ModelSpec, pages: int, seqs: int, per_seq: int):
     else:
         w = load_weights(spec.name, spec, dev)
     eng = build_engine(spec, w, n_pages=pages, max_seqs=seqs, max_pages_per_seq=per_seq)
-    eng.kv.normal_(0, 1)
+    for t in eng.cache_buffers() if hasattr(eng, "cache_buffers") else [eng.kv]:
+        t.normal_(0, 1)
     return eng
 
 

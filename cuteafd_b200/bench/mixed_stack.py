@@ -62,7 +62,7 @@ def roofline(spec: ModelSpec, T: int, pairs: int, kv_rows: int, site: tuple, pre
             return ("context -> keys, values", lo(2.0 * rows * N * K, 2.0 * (N * K + rows * (N + K))))
         mats = 2 if sw else 1
         label = ("ffn gate + up" if sw else "side gate" if ours and N == spec.side_dim else "side projection" if ours and K == spec.side_dim else "queries from their latent" if K == q_rank else
-                 "output projection (+ ffn down)" if N == W else "input projection")
+                 "latent: down projection" if N in (q_rank, rank + 64, q_rank + rank + 64) else "output projection (+ ffn down)" if N == W else "input projection")
         return (label, lo(2.0 * T * N * K * mats, 2.0 * (mats * N * K + T * (N + K))))
     n = site[0]
     if n in ("latent_attention", "mla_attention"):

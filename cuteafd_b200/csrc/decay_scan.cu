@@ -9,8 +9,8 @@
 //   chunk_scan     state in front of every chunk (operand tiles), state behind the run     elementwise over the chunks
 //   chunk_out      o = (q k^T, decayed, causal) v + decay(start -> i) q S  three tcgen05 products per (head, chunk), output norm, gate
 // Everything that is not a projection enters the products as two bf16 terms (value and rounding error, 16 bits of mantissa together), with fp32
-// accumulators in tensor memory; the states stay fp32.  Per-channel decays are folded into q and k relative to the middle of the chunk; a chunk
-// whose decays span more than 2^80 on the way takes its scores from the ordinary cores instead, pair by pair.
+// accumulators in tensor memory; the states stay fp32.  Per-channel decays are folded into q and k relative to the middle of the chunk, or of
+// smaller blocks where they span too much for one reference (see `Channels`).
 // (Sibling of linear_attn.cu, whose delta rule has no such form yet; the reference's linear-attention programs are AOT exports without sources.)
 #define CA_PDL_CLASS 2
 #include "stack_rows.cuh"
@@ -39,8 +39,8 @@ struct DecayScan {
   int H, dim, vdim, vp, depth, n_state;
   int long_from;                                            // runs of more tokens take the chunk kernels (bf16): only their replay is done here
   // scratch of the long form, a run's chunks consecutive from q_start / DC_TOK + sequence: contributions [chunks, H, dim, vp], factors
-  // [chunks, H, 2 dim + 1] (decays of the chunk; what puts the state in front of it on the scale of the chunk's queries; whether the decays span too
-  // much for a common reference), states as operand tiles [chunks, H, tile set]
+  // [chunks, H, 2 dim + 1] (decays of the chunk; what puts the state in front of it on the scale of the chunk's queries; how often the chunk is halved
+  // for its scores), states as operand tiles [chunks, H, tile set]
   float* chunk_state; float* chunk_decay; uint8_t* chunk_tiles;
   int* status;
 };
@@ -50,8 +50,6 @@ __device__ __forceinline__ float2 forget_gate(float z, float l) {
   const float e = expf(-fabsf(z)), s = 1.f / (1.f + e), big = s, small = e * s;      // sigmoids of |z| and -|z|
   return make_float2(fmaf(1.f - l, z >= 0.f ? big : small, l), (1.f - l) * (z >= 0.f ? small : big));
 }
-// and the binary logarithm of that decay
-__device__ __forceinline__ float forget_log2(float2 f) { return f.y < 0.5f ? log1pf(-f.y) * 1.4426950408889634f : log2f(fmaxf(f.x, 1e-38f)); }
 __device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.f + __expf(-fmaxf(z, -80.f))); }
 
 // log alpha of a channel from its logit
@@ -233,16 +231,17 @@ __global__ void __launch_bounds__(DS_THREADS, NT == 1 ? 3 : 1) decay_scan_kernel
 #define DC_TOK 128
 #define DC_THREADS 512
 #define DC_PARTS (DC_THREADS / 128)      // threads that share a row of an accumulator
-#define DC_SPAN 80.f        // most binary digits a chunk's decays may span on either side of its middle
+#define DC_SPAN 80.f        // most binary digits that decays may span on either side of a common reference
 
 // Operand tiles: 64 columns x 128 rows in 128-byte rows, 128-byte swizzle.  DB 64-wide blocks of key dimensions; value tiles have up to 4 blocks.
 template <int DB>
 struct ChunkSmem {
   static constexpr int TILE = 16384, HL = 2 * DB * TILE;               // an operand of key dimensions: values, then rounding errors
   static constexpr int SMALL = 4096;                                   // vectors, barrier, flags
+  static constexpr int UNITS = 16 * DB * 64 * 4;                       // per-channel decays: sums over units of eight tokens
   static constexpr int X = 4 * TILE;                                   // decays [128, 64 DB] fp32, then the value tiles, then state tiles
   static constexpr int P = 4 * TILE;                                   // keys, then probabilities (two terms of two blocks), then state tiles
-  static constexpr int STATES = HL + X + SMALL, OUT = HL + P + X + SMALL;
+  static constexpr int STATES = HL + X + SMALL + UNITS, OUT = HL + P + X + SMALL + UNITS;
 };
 
 struct ChunkRun { int n, p0, row, len, ci, chunks; };                  // run, first row and length of the block's chunk, its place in the scratch
@@ -285,6 +284,8 @@ __device__ __forceinline__ void ldg8(const bf16* p, float* v) {
 #pragma unroll
   for (int j = 0; j < 4; ++j) { const float2 f = __bfloat1622float2(h[j]); v[2 * j] = f.x; v[2 * j + 1] = f.y; }
 }
+// Staged rows of float4: column groups of eight are turned by the row, so that a warp writes one column of 32 rows, or reads whole rows, without conflicts.
+__device__ __forceinline__ int stage_col(int row, int c) { return c ^ (row & 7); }
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
@@ -332,40 +333,160 @@ __device__ __forceinline__ void head8(const bf16* row, int d0, int dim, const fl
 // How the chunk kernels get their decays: a constant per head, from a low-rank projection, from HGRN2's forget gate.
 enum { DECAY_HEAD = 0, DECAY_LOW_RANK = 1, DECAY_FORGET = 2 };
 
-template <int MODE>
-__device__ __forceinline__ void query8(const DecayScan<bf16>& a, int h, size_t row, int d0, bool vec, float* v) {
-  head8(a.q + row * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + row * a.pairs : nullptr, a.pairs, a.q_scale, vec, v);
-  if (MODE == DECAY_FORGET)
-#pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] = silu_f(v[j]);
+// Per-channel decays: a thread owns two neighbouring channels of DC_SEG tokens - their decays, queries and keys stay in its registers, and every
+// operand tile is written from there relative to whatever reference its product needs.  Sums of the decays' logarithms travel between the threads
+// as sums over units of eight tokens.
+//
+// q_i k_j decays by 2^(P(i) - P(j)), P the running sum.  Referred to the middle of a block of D tokens, rows of its second half and keys of its first
+// half have factors of at most one; rows and keys of the same half have, on either side of the middle, up to 2^(sum over D / 2 tokens).  So the
+// chunk is cut into the largest blocks whose half-sums stay below DC_SPAN: their own scores are one product, and those between the halves of every
+// larger block one more per halving (`depth` of them).  A chunk whose blocks of 16 exceed it (a channel that forgets at once) takes its scores
+// from the ordinary cores, pair by pair.
+#define DC_UNITS (DC_TOK / 8)
+#define DC_PAIRWISE 4       // depth of such a chunk
+
+// Decays below 2^-126 are zero.
+__device__ __forceinline__ float exp2_f(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+// log2(1 - m) of a decay 1 - m, m up to 1/16: seven terms of the series, relative error below 2e-8.
+__device__ __forceinline__ float log2_near_one(float m) {
+  float p = fmaf(m, 1.f / 7.f, 1.f / 6.f);
+  p = fmaf(m, p, 0.2f); p = fmaf(m, p, 0.25f); p = fmaf(m, p, 1.f / 3.f); p = fmaf(m, p, 0.5f); p = fmaf(m, p, 1.f);
+  return m * p * -1.4426950408889634f;
 }
-template <int MODE>
-__device__ __forceinline__ void key8(const DecayScan<bf16>& a, int h, size_t row, int d0, bool vec, float* v) {
-  head8(a.k + row * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + row * a.pairs : nullptr, a.pairs, a.k_scale, vec, v);
-  if (MODE == DECAY_FORGET)
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int c = h * a.dim + d0 + j;
-      v[j] = d0 + j < a.dim ? (1.f - __ldg(a.lower + c)) * __fdividef(1.f, 1.f + __expf(fminf(v[j] + __ldg(a.forget_b + c), 80.f))) : 0.f;
-    }
+// log2 of the sigmoid of z
+__device__ __forceinline__ float log2_sigmoid(float z) {
+  const float e = __expf(-fabsf(z)), far = -fmaf(fmaxf(-z, 0.f), 1.4426950408889634f, __log2f(1.f + e));
+  return z > 2.75f ? log2_near_one(__fdividef(e, 1.f + e)) : far;
 }
 
-// log2 of the forget gate's decays -> X [128, DP] (zero past the run's end and past `dim`).
-template <int DP>
-__device__ __forceinline__ void chunk_forget(const DecayScan<bf16>& a, int h, const ChunkRun& r, bool vec, float* X) {
-  for (int i = threadIdx.x; i < DC_TOK * DP / 8; i += DC_THREADS) {
-    const int t = i / (DP / 8), d0 = (i % (DP / 8)) * 8;
-    float z[8];
-    head8(a.k + (size_t)(r.row + min(t, r.len - 1)) * a.ldp + h * a.dim, d0, a.dim, nullptr, 0, 1.f, vec, z);
+template <int DB, int MODE>
+struct Channels {
+  static constexpr int DP = DB * 64, PAIRS = DP / 2, SEGS = DC_THREADS / PAIRS, N = DC_TOK / SEGS;      // N: tokens of a thread
+  float2 b[N];                                              // running sums of log2 decays
+  uint32_t q[N], k[N];                                      // projected rows (bf16 pairs); FORGET: k are the gate's logits
+  float2 bias, keep;                                        // FORGET: bias and 1 - lower bound
+  int c, t0;                                                // first channel and token
+
+  static __device__ __forceinline__ float2 wide(uint32_t v) { return __bfloat1622float2(*(const bf162*)&v); }
+
+  // Two rows' worth of pairs.  No load stands behind a condition, so that all of them are in flight together.
+  static __device__ __forceinline__ void pairs(const bf16* p, int ldp, int t0, int last, bool one, bool two, bool aligned, uint32_t (&v)[N]) {
+    if (aligned) {
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int c = h * a.dim + d0 + j;
-      z[j] = t < r.len && d0 + j < a.dim ? forget_log2(forget_gate(z[j] + __ldg(a.forget_b + c), __ldg(a.lower + c))) : 0.f;
+      for (int i = 0; i < N; ++i) v[i] = __ldg((const unsigned int*)(p + (size_t)min(t0 + i, last) * ldp));
+    } else {
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const bf16* e = p + (size_t)min(t0 + i, last) * ldp;
+        v[i] = __bfloat16_as_ushort(e[0]) | (uint32_t)__bfloat16_as_ushort(e[two ? 1 : 0]) << 16;
+      }
     }
-    *(float4*)(X + t * DP + d0) = make_float4(z[0], z[1], z[2], z[3]);
-    *(float4*)(X + t * DP + d0 + 4) = make_float4(z[4], z[5], z[6], z[7]);
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = !one || t0 + i > last ? 0u : (two ? v[i] : v[i] & 0xFFFFu);
   }
-  __syncthreads();
+  __device__ __forceinline__ void load(const DecayScan<bf16>& a, int h, const ChunkRun& r, bool queries) {
+    c = (threadIdx.x % PAIRS) * 2; t0 = (threadIdx.x / PAIRS) * N; len = r.len;
+    const bool one = c < a.dim, two = c + 1 < a.dim, even = ((a.ldp | a.dim) & 1) == 0;
+    const size_t at = (size_t)r.row * a.ldp + h * a.dim + (one ? c : 0);
+    pairs(a.k + at, a.ldp, t0, len - 1, one, two, even && ((uintptr_t)a.k & 3) == 0, k);
+    if (queries) pairs(a.q + at, a.ldp, t0, len - 1, one, two, even && ((uintptr_t)a.q & 3) == 0, q);
+    if (MODE == DECAY_FORGET) {
+      const float* fb = a.forget_b + h * a.dim + c;
+      const float* lb = a.lower + h * a.dim + c;
+      bias = make_float2(one ? fb[0] : 0.f, two ? fb[1] : 0.f);
+      keep = make_float2(one ? 1.f - lb[0] : 0.f, two ? 1.f - lb[1] : 0.f);
+    }
+  }
+  // Sigmoids of -x and -y at the price of one reciprocal.
+  static __device__ __forceinline__ float2 sigmoid_neg2(float x, float y) {
+    const float ex = 1.f + __expf(fminf(x, 40.f)), ey = 1.f + __expf(fminf(y, 40.f)), inv = __fdividef(1.f, ex * ey);
+    return make_float2(inv * ey, inv * ex);
+  }
+  // log2(1 - m) of a decay 1 - m (what decays to less than 2^-26 in one step is gone)
+  static __device__ __forceinline__ float gate_log(float m) {
+    const float far = __log2f(fmaxf(1.f - m, 1.5e-8f));
+    return m < 0.0625f ? log2_near_one(m) : far;
+  }
+  // FORGET: the key, (1 - l) sigmoid(-z).
+  __device__ __forceinline__ float2 key(const DecayScan<bf16>& a, int i) const {
+    const float2 v = wide(k[i]);
+    if (MODE != DECAY_FORGET) return make_float2(v.x * a.k_scale, v.y * a.k_scale);
+    const float2 s = sigmoid_neg2(v.x + bias.x, v.y + bias.y);
+    return in_run(i) ? make_float2(keep.x * s.x, keep.y * s.y) : make_float2(0.f, 0.f);
+  }
+  __device__ __forceinline__ float2 query(const DecayScan<bf16>& a, int i) const {
+    const float2 v = wide(q[i]);
+    if (MODE != DECAY_FORGET) return make_float2(v.x * a.q_scale, v.y * a.q_scale);
+    const float2 s = sigmoid_neg2(-v.x, -v.y);
+    return make_float2(v.x * s.x, v.y * s.y);
+  }
+  int len;
+  __device__ __forceinline__ bool in_run(int i) const { return t0 + i < len; }
+
+  // Running sums; `X`: log2 decays [128, DP] (LOW_RANK); `units`: room for the units' sums [DC_UNITS, DP].  Ends with a barrier; all of `units` may be read.
+  __device__ __forceinline__ void sums(const DecayScan<bf16>& a, const float* X, float* units) {
+    float2 s = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      float2 l;
+      if (MODE == DECAY_FORGET) {
+        const float2 m = key(a, i);
+        l = make_float2(gate_log(m.x), gate_log(m.y));
+      } else {
+        l = *(const float2*)(X + (t0 + i) * DP + c);
+      }
+      if (i % 8 == 0) s = make_float2(0.f, 0.f);
+      s.x += l.x; s.y += l.y;
+      b[i] = s;
+      if (i % 8 == 7) *(float2*)(units + ((t0 + i) >> 3) * DP + c) = s;
+    }
+    __syncthreads();
+    float2 p = make_float2(0.f, 0.f);
+    for (int u = 0; u < t0 / 8; ++u) { const float2 v = *(const float2*)(units + u * DP + c); p.x += v.x; p.y += v.y; }
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      if (i && i % 8 == 0) { const float2 v = *(const float2*)(units + ((t0 + i) / 8 - 1) * DP + c); p.x += v.x; p.y += v.y; }
+      b[i].x += p.x; b[i].y += p.y;
+    }
+  }
+  // Running sum in front of token `t` (a multiple of 8).
+  __device__ __forceinline__ float2 front(const float* units, int t) const {
+    float2 p = make_float2(0.f, 0.f);
+    for (int u = 0; u < t / 8; ++u) { const float2 v = *(const float2*)(units + u * DP + c); p.x += v.x; p.y += v.y; }
+    return p;
+  }
+  // Token i of this thread into a tile set, value and rounding error.
+  __device__ __forceinline__ void put(uint8_t* tiles, int i, float2 v) const {
+    const int t = t0 + i;
+    const uint32_t at = tile_at(t, c & ~7, 16384) + (c & 7) * 2;
+    const bf162 hi = __floats2bfloat162_rn(v.x, v.y);
+    const float2 w = __bfloat1622float2(hi);
+    const bf162 lo = __floats2bfloat162_rn(v.x - w.x, v.y - w.y);
+    *(uint32_t*)(tiles + at) = *(const uint32_t*)&hi;
+    *(uint32_t*)(tiles + at + DB * 16384) = *(const uint32_t*)&lo;
+  }
+};
+// Smallest depth whose blocks' half-sums stay within DC_SPAN for this channel.
+template <int DP>
+__device__ __forceinline__ int span_depth(const float* units, int c) {
+  float u[DC_UNITS];
+#pragma unroll
+  for (int j = 0; j < DC_UNITS; ++j) u[j] = units[j * DP + c];
+  int depth = DC_PAIRWISE;
+#pragma unroll
+  for (int level = 3; level >= 0; --level) {                // halves of 8, 16, 32, 64 tokens: blocks of 16, 32, 64, 128
+    const int n = 8 >> level;                               // units of a half
+    float worst = 0.f;
+#pragma unroll
+    for (int j = 0; j < DC_UNITS; j += n) {
+      float s = 0.f;
+#pragma unroll
+      for (int q = 0; q < n; ++q) s += u[j + q];
+      worst = fminf(worst, s);
+    }
+    if (worst >= -DC_SPAN && depth == level + 1) depth = level;
+  }
+  return depth;
 }
 
 // log2 of the chunk's per-channel decays -> X [128, DP] (zero past the run's end and past `dim`); `stage`: 8 KB.
@@ -377,11 +498,14 @@ __device__ __forceinline__ void chunk_logs(const DecayScan<bf16>& a, int h, cons
     __syncthreads();
     for (int i = tid; i < DC_TOK * 16; i += DC_THREADS) {
       const int t = i >> 4, q = r0 + (i & 15);
-      stage[i] = t < r.len && q < a.rank ? to_f(a.a1[(size_t)(r.row + t) * a.ldp + q]) : 0.f;
+      const float v = to_f(a.a1[(size_t)(r.row + min(t, r.len - 1)) * a.ldp + min(q, a.rank - 1)]);
+      stage[i] = t < r.len && q < a.rank ? v : 0.f;
     }
     float w[16];
 #pragma unroll
-    for (int q = 0; q < 16; ++q) w[q] = c < a.dim && r0 + q < a.rank ? a.a2[(size_t)(h * a.dim + c) * a.rank + r0 + q] : 0.f;
+    for (int q = 0; q < 16; ++q) w[q] = __ldg(a.a2 + (size_t)(h * a.dim + min(c, a.dim - 1)) * a.rank + min(r0 + q, a.rank - 1));
+#pragma unroll
+    for (int q = 0; q < 16; ++q) w[q] = c < a.dim && r0 + q < a.rank ? w[q] : 0.f;
     __syncthreads();
     for (int t = tid / DP; t < DC_TOK; t += DC_THREADS / DP) {
       float z = r0 ? X[t * DP + c] : b;
@@ -390,7 +514,7 @@ __device__ __forceinline__ void chunk_logs(const DecayScan<bf16>& a, int h, cons
         const float4 s = *(const float4*)(stage + t * 16 + q);
         z = fmaf(w[q], s.x, z); z = fmaf(w[q + 1], s.y, z); z = fmaf(w[q + 2], s.z, z); z = fmaf(w[q + 3], s.w, z);
       }
-      X[t * DP + c] = r0 + 16 < a.rank ? z : (t < r.len && c < a.dim ? log_decay(z, a.inv_tau) * 1.4426950408889634f : 0.f);
+      X[t * DP + c] = r0 + 16 < a.rank ? z : (t < r.len && c < a.dim ? log2_sigmoid(z) * a.inv_tau : 0.f);
     }
   }
   __syncthreads();
@@ -447,7 +571,6 @@ template <int DB, int MODE>
 __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __grid_constant__ DecayScan<bf16> a) {
   pdl_launch(); pdl_wait();
   using Sm = ChunkSmem<DB>;
-  constexpr bool GLA = MODE != DECAY_HEAD;                            // a decay per key channel
   constexpr int DP = DB * 64;
   extern __shared__ __align__(1024) uint8_t dc_smem[];
   const int h = blockIdx.x, tid = threadIdx.x;
@@ -455,49 +578,56 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __gri
   if (!chunk_of(a, blockIdx.y, blockIdx.z, r)) return;                // block-uniform
   if (smem_u32(dc_smem) & 1023) { if (tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F4); return; }
   uint8_t* sK = dc_smem; uint8_t* sX = sK + Sm::HL; uint8_t* small = sX + Sm::X;
-  float* X = (float*)sX; float* rest = (float*)(small + 64); float* first = rest + DP;      // [DP] log2 decays of the second and the first half
   ChunkSync y = chunk_begin(small, 256, a.status);
   const int VB = (a.vp + 63) / 64;
-  const bool vec = ((a.dim | a.ldp | (a.rope ? a.pairs : 0)) & 7) == 0 && ((uintptr_t)a.k & 15) == 0;
-  const float l2 = GLA ? 0.f : decay_log2(a.decay[h]);
   float* factors = a.chunk_decay + ((size_t)r.ci * a.H + h) * (2 * a.dim + 1);
-  if (GLA) {
-    if (MODE == DECAY_FORGET) chunk_forget<DP>(a, h, r, vec, X);
-    else chunk_logs<DP>(a, h, r, X, (float*)sK);
-    bool far = false;
-    if (tid < 2 * DP) {                                               // decays behind every token, within its half
-      const int c = tid % DP, half = tid / DP;
-      float s = 0.f;
-      for (int t = half * 64 + 63; t >= half * 64; --t) { const float l = X[t * DP + c]; X[t * DP + c] = s; s += l; }
-      (half ? rest : first)[c] = s;
-      far = s < -DC_SPAN;
+  if constexpr (MODE != DECAY_HEAD) {
+    float* units = (float*)(small + Sm::SMALL);
+    Channels<DB, MODE> ch;
+    ch.load(a, h, r, false);
+    if (MODE == DECAY_FORGET) load_values(a, h, r, sX, VB);
+    else chunk_logs<DP>(a, h, r, (float*)sX, (float*)sK);
+    ch.sums(a, (const float*)sX, units);
+    if (MODE != DECAY_FORGET) load_values(a, h, r, sX, VB);           // (every thread has read its decays)
+    int* depth = (int*)(small + 24);
+    if (tid == 0) *depth = 0;
+    const float2 total = ch.front(units, DC_TOK);
+    __syncthreads();
+    float first = 0.f, all = 0.f;
+    if (tid < DP) {
+      const int d = span_depth<DP>(units, tid);
+      if (d) atomicMax(depth, d);
+      for (int u = 0; u < DC_UNITS; ++u) { all += units[u * DP + tid]; if (u == DC_UNITS / 2 - 1) first = all; }
     }
-    const bool wide = __syncthreads_or(far);
-    if (tid == 0) factors[2 * a.dim] = wide ? 1.f : 0.f;
-    if (tid < a.dim) { factors[tid] = exp2f(first[tid] + rest[tid]); factors[a.dim + tid] = wide ? 1.f : exp2f(first[tid]); }
+    __syncthreads();
+    if (tid == 0) factors[2 * a.dim] = (float)*depth;
+    if (tid < a.dim) { factors[tid] = exp2f(all); factors[a.dim + tid] = *depth ? 1.f : exp2f(first); }
+#pragma unroll
+    for (int i = 0; i < Channels<DB, MODE>::N; ++i) {
+      const float2 k = ch.key(a, i);
+      ch.put(sK, i, make_float2(k.x * exp2_f(total.x - ch.b[i].x), k.y * exp2_f(total.y - ch.b[i].y)));
+    }
   } else {
+    const bool vec = ((a.dim | a.ldp | (a.rope ? a.pairs : 0)) & 7) == 0 && ((uintptr_t)a.k & 15) == 0;
+    const float l2 = decay_log2(a.decay[h]);
     load_values(a, h, r, sX, VB);
     if (tid < a.dim) { factors[tid] = exp2f(l2 * (float)r.len); factors[a.dim + tid] = 1.f; }
-  }
 #pragma unroll 4
-  for (int i = tid; i < DC_TOK * DB * 8; i += DC_THREADS) {
-    const int t = i / (DB * 8), d0 = (i % (DB * 8)) * 8;
-    float v[8];
-    if (t < r.len) {
-      const size_t row = r.row + t;
-      key8<MODE>(a, h, row, d0, vec, v);
-      const float f = GLA ? 0.f : exp2f(l2 * (float)(r.len - 1 - t));
+    for (int i = tid; i < DC_TOK * DB * 8; i += DC_THREADS) {
+      const int t = i / (DB * 8), d0 = (i % (DB * 8)) * 8;
+      float v[8];
+      if (t < r.len) {
+        const size_t row = r.row + t;
+        head8(a.k + row * a.ldp + h * a.dim, d0, a.dim, a.rope ? a.rope + row * a.pairs : nullptr, a.pairs, a.k_scale, vec, v);
+        const float f = exp2f(l2 * (float)(r.len - 1 - t));
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] *= GLA ? exp2f(X[t * DP + d0 + j] + (t < 64 ? rest[d0 + j] : 0.f)) : f;
-    } else {
+        for (int j = 0; j < 8; ++j) v[j] *= f;
+      } else {
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] = 0.f;
+        for (int j = 0; j < 8; ++j) v[j] = 0.f;
+      }
+      put8_two(sK, tile_at(t, d0, Sm::TILE), DB * Sm::TILE, v);
     }
-    put8_two(sK, tile_at(t, d0, Sm::TILE), DB * Sm::TILE, v);
-  }
-  if (GLA) {
-    __syncthreads();                                                  // the decays have been read: values take their place
-    load_values(a, h, r, sX, VB);
   }
   cp_async_wait();
   y.publish();
@@ -510,17 +640,22 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_states_kernel(const __gri
   }
   __syncwarp();
   y.wait(0x6F5);
-  const int warp = tid >> 5, row = (warp & 3) * 32 + (tid & 31);
-  float* dst = a.chunk_state + (((size_t)r.ci * a.H + h) * a.dim + (row < a.dim ? row : 0)) * a.vp;
+  const int warp = tid >> 5, row = (warp & 3) * 32 + (tid & 31), pitch = VB * 16;
   constexpr int PW = 64 / DC_PARTS;                                   // columns of a 64-wide block that a thread takes
+  float4* stage = (float4*)sK;                                        // (keys and values have been read: rows of key dimensions, whole lines to memory)
   for (int c = (warp >> 2) * VB * PW; c < ((warp >> 2) + 1) * VB * PW; c += 16) {
     uint32_t o[16];
     tmem_ld_x16(y.tmem + ((uint32_t)((warp & 3) * 32) << 16) + c, o);
     tc_wait_ld();
-    if (row < a.dim)
+    if (row < DP)
 #pragma unroll
-      for (int j = 0; j < 16; j += 4)
-        if (c + j < a.vp) *(uint4*)(dst + c + j) = make_uint4(o[j], o[j + 1], o[j + 2], o[j + 3]);
+      for (int j = 0; j < 4; ++j) stage[row * pitch + stage_col(row, c / 4 + j)] = *(const float4*)(o + 4 * j);
+  }
+  __syncthreads();
+  float4* dst = (float4*)(a.chunk_state + ((size_t)r.ci * a.H + h) * a.dim * a.vp);
+  for (int i = tid; i < a.dim * (a.vp / 4); i += DC_THREADS) {
+    const int d = i / (a.vp / 4), c = i % (a.vp / 4);
+    dst[i] = stage[d * pitch + stage_col(d, c)];
   }
   chunk_end(y, 256);
 }
@@ -570,7 +705,6 @@ template <int DB, int MODE>
 __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_constant__ DecayScan<bf16> a) {
   pdl_launch(); pdl_wait();
   using Sm = ChunkSmem<DB>;
-  constexpr bool GLA = MODE != DECAY_HEAD;                            // a decay per key channel
   constexpr int DP = DB * 64, T = Sm::TILE;
   extern __shared__ __align__(1024) uint8_t dc_smem[];
   const int h = blockIdx.x, seq = blockIdx.z, tid = threadIdx.x;
@@ -579,71 +713,133 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
   const int slot = a.state_slot[seq];
   if (slot < 0 || slot >= a.n_state || (smem_u32(dc_smem) & 1023)) { if (tid == 0) ca_dev_fail(a.status, CA_DEV_BAD_INDEX, 0x6F6); return; }
   uint8_t* sQ = dc_smem; uint8_t* sP = sQ + Sm::HL; uint8_t* sX = sP + Sm::P; uint8_t* small = sX + Sm::X;
-  float* X = (float*)sX; float* mid = (float*)(small + 64); float* ssum = mid + DP;      // [DP] log2 decay up to the reference, [DC_PARTS, 128]
-  uint64_t* tiles_bar = (uint64_t*)(small + 32);
-  if (tid == 0) mbar_init(tiles_bar, 1);
+  float* ssum = (float*)(small + 64);                                 // [DC_PARTS, 128]
+  float* gain = ssum + DC_PARTS * 128;                                // [256]
+  uint64_t* tiles_bar = (uint64_t*)(small + 32);                      // [2]
+  if (tid == 0) { mbar_init(tiles_bar, 1); mbar_init(tiles_bar + 1, 1); }
+  if (a.norm && tid < a.vdim) gain[tid] = a.norm[tid];
   ChunkSync y = chunk_begin(small, 512, a.status);
   const uint32_t O1 = 0, O2 = 256, SC = 256;                          // scores stand where the state's share is accumulated later
   constexpr int KW = DC_TOK / DC_PARTS, PW = 64 / DC_PARTS;             // keys, and columns of a 64-wide block of values, that a thread takes of its row
   const int VB = (a.vp + 63) / 64, warp = tid >> 5, part = warp >> 2, row = (warp & 3) * 32 + (tid & 31);
   const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
-  const bool vec = ((a.dim | a.ldp | (a.rope ? a.pairs : 0)) & 7) == 0 && (((uintptr_t)a.q | (uintptr_t)a.k) & 15) == 0;
-  const float l2 = GLA ? 0.f : decay_log2(a.decay[h]);
-  bool wide = false;                                                  // decays that span too much for a common reference
-  if (!GLA) load_values(a, h, r, sX, VB);
-  if (GLA) {
-    if (MODE == DECAY_FORGET) chunk_forget<DP>(a, h, r, vec, X);
-    else chunk_logs<DP>(a, h, r, X, (float*)sQ);
-    wide = a.chunk_decay[((size_t)r.ci * a.H + h) * (2 * a.dim + 1) + 2 * a.dim] != 0.f;
-    if (tid < 2 * DP) {                                               // relative to the chunk's middle: in front of it up to 63 (positive), behind it (negative)
-      const int c = tid % DP;
-      float s = 0.f;
-      if (tid < DP) {
-        for (int t = 63; t >= 0; --t) { const float l = X[t * DP + c]; X[t * DP + c] = -s; s += l; }
-        mid[c] = s;
-      } else {
-        for (int t = 64; t < DC_TOK; ++t) { s += X[t * DP + c]; X[t * DP + c] = s; }
-      }
+  const uint32_t q0 = smem_u32(sQ), k0 = smem_u32(sP);
+  auto score = [&](uint32_t col) {                                    // one thread: queries x keys, value x value, value x error, error x value
+    const uint32_t id = dc_idesc(DC_TOK, 0, 0);
+    for (int part = 0; part < 3; ++part) {
+      const uint32_t qa = q0 + (part == 2 ? DB * T : 0), kb = k0 + (part == 1 ? DB * T : 0);
+      for (int b = 0; b < DB; ++b)
+        for (int k = 0; k < 4; ++k) tc_mma_f16(y.tmem + col, umma_desc_sw128(qa + b * T) + 2 * k, umma_desc_sw128(kb + b * T) + 2 * k, id, (part | b | k) ? 1u : 0u);
     }
-    __syncthreads();
-  }
-#pragma unroll 2
-  for (int i = tid; i < DC_TOK * DB * 8; i += DC_THREADS) {
-    const int t = i / (DB * 8), d0 = (i % (DB * 8)) * 8;
-    float q[8], k[8];
-    if (t < r.len) {
-      const size_t gr = r.row + t;
-      query8<MODE>(a, h, gr, d0, vec, q);
-      key8<MODE>(a, h, gr, d0, vec, k);
-      if (GLA) {
+    tc_commit(y.bar);
+  };
+  float sc[KW];                                                       // this thread's scores: its row, keys [part * KW, + KW)
+  float l2 = 0.f;
+  if constexpr (MODE != DECAY_HEAD) {
+    using Ch = Channels<DB, MODE>;
+    float* X = (float*)sX;
+    float* units = (float*)(small + Sm::SMALL);
+    const int depth = (int)a.chunk_decay[((size_t)r.ci * a.H + h) * (2 * a.dim + 1) + 2 * a.dim];
+    Ch ch;
+    ch.load(a, h, r, true);
+    if (MODE == DECAY_FORGET) { if (depth < DC_PAIRWISE) load_values(a, h, r, sX, VB); }
+    else chunk_logs<DP>(a, h, r, X, (float*)sQ);
+    ch.sums(a, X, units);
+    if (depth < DC_PAIRWISE) {
+      if (MODE != DECAY_FORGET) load_values(a, h, r, sX, VB);         // (every thread has read its decays)
+#pragma unroll 1
+      for (int l = 0; l <= depth; ++l) {                              // blocks of 128 >> l tokens, referred to the running sums in front of their middles
+        const int half = DC_TOK >> (l + 1);
+        const float2 ref = ch.front(units, (ch.t0 & -(2 * half)) + half);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          const float x = X[t * DP + d0 + j];
-          if (wide) q[j] *= exp2f(x + mid[d0 + j]);                   // from the chunk's start: for the state alone
-          else { q[j] *= exp2f(x); k[j] *= exp2f(-x); }
+        for (int i = 0; i < Ch::N; ++i) {
+          // rows that have no part in this product hold zeros
+          const bool second = (ch.t0 + i) & half, as_q = l == depth || second, as_k = l == depth || !second;
+          const float2 x = make_float2(ch.b[i].x - ref.x, ch.b[i].y - ref.y), q = ch.query(a, i), k = ch.key(a, i);
+          ch.put(sQ, i, as_q ? make_float2(q.x * exp2_f(x.x), q.y * exp2_f(x.y)) : make_float2(0.f, 0.f));
+          ch.put(sP, i, as_k ? make_float2(k.x * exp2_f(-x.x), k.y * exp2_f(-x.y)) : make_float2(0.f, 0.f));
+        }
+        y.publish();
+        if (tid == 0) score((SC + l * 128) & 511);
+        __syncwarp();
+        y.wait(0x6F7);
+      }
+#pragma unroll
+      for (int c = 0; c < KW; c += 16) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) sc[c + j] = 0.f;
+#pragma unroll 1
+        for (int l = 0; l <= depth; ++l) {
+          uint32_t o[16];
+          tmem_ld_x16(y.tmem + lanes + ((SC + l * 128) & 511) + part * KW + c, o);
+          tc_wait_ld();
+          const int half = DC_TOK >> (l + 1);
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            const int key = part * KW + c + j;
+            const bool same = ((row ^ key) & -(2 * half)) == 0;
+            if (same && key <= row && (l == depth || ((row & half) && !(key & half)))) sc[c + j] = __uint_as_float(o[j]);
+          }
         }
       }
     } else {
+      // pair by pair: the decays between two tokens as the difference of their sums
+      __syncthreads();                                                // the units' sums (LOW_RANK: the logarithms) have been read
 #pragma unroll
-      for (int j = 0; j < 8; ++j) q[j] = k[j] = 0.f;
+      for (int i = 0; i < Ch::N; ++i) { *(float2*)(X + (ch.t0 + i) * DP + ch.c) = ch.b[i]; ch.put(sP, i, ch.key(a, i)); ch.put(sQ, i, ch.query(a, i)); }
+      __syncthreads();
+#pragma unroll
+      for (int j = 0; j < KW; ++j) sc[j] = 0.f;
+      if (part * KW <= (warp & 3) * 32 + 31)                          // warp-uniform: some key is not behind every row of the warp
+        for (int d0 = 0; d0 < a.dim; d0 += 8) {
+          float q[8], e[8], x[8];
+          const uint8_t* qt = sQ + tile_at(row, d0, T);
+          load8<bf16>((const bf16*)qt, q);
+          load8<bf16>((const bf16*)(qt + DB * T), e);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) { q[j] += e[j]; x[j] = X[row * DP + d0 + j]; }
+#pragma unroll
+          for (int j = 0; j < KW; ++j) {
+            const int key = part * KW + j;
+            const uint8_t* at = sP + tile_at(key, d0, T);
+            float k[8], lo[8];
+            load8<bf16>((const bf16*)at, k);
+            load8<bf16>((const bf16*)(at + DB * T), lo);
+#pragma unroll
+            for (int e2 = 0; e2 < 8; ++e2) sc[j] = fmaf(q[e2] * (k[e2] + lo[e2]), exp2f(x[e2] - X[key * DP + d0 + e2]), sc[j]);
+          }
+        }
+#pragma unroll
+      for (int j = 0; j < KW; ++j) if (part * KW + j > row || row >= r.len) sc[j] = 0.f;       // (may not be a number)
+      __syncthreads();                                                // the decays have been read
+      load_values(a, h, r, sX, VB);
     }
-    put8_two(sQ, tile_at(t, d0, T), DB * T, q);
-    put8_two(sP, tile_at(t, d0, T), DB * T, k);                       // (wide: as they are)
-  }
-  float sc[KW];                                                       // this thread's scores: its row, keys [part * KW, + KW)
-  if (!wide) {
-    y.publish();
-    if (tid == 0) {
-      const uint32_t id = dc_idesc(DC_TOK, 0, 0), q0 = smem_u32(sQ), k0 = smem_u32(sP);
-      for (int part = 0; part < 3; ++part) {                          // value x value, value x error, error x value
-        const uint32_t qa = q0 + (part == 2 ? DB * T : 0), kb = k0 + (part == 1 ? DB * T : 0);
-        for (int b = 0; b < DB; ++b)
-          for (int k = 0; k < 4; ++k) tc_mma_f16(y.tmem + SC, umma_desc_sw128(qa + b * T) + 2 * k, umma_desc_sw128(kb + b * T) + 2 * k, id, (part | b | k) ? 1u : 0u);
+    if (depth)                                                        // the state is decayed from the chunk's start
+#pragma unroll
+      for (int i = 0; i < Ch::N; ++i) { const float2 q = ch.query(a, i); ch.put(sQ, i, make_float2(q.x * exp2_f(ch.b[i].x), q.y * exp2_f(ch.b[i].y))); }
+  } else {
+    const bool vec = ((a.dim | a.ldp | (a.rope ? a.pairs : 0)) & 7) == 0 && (((uintptr_t)a.q | (uintptr_t)a.k) & 15) == 0;
+    l2 = decay_log2(a.decay[h]);
+    load_values(a, h, r, sX, VB);
+#pragma unroll 2
+    for (int i = tid; i < DC_TOK * DB * 8; i += DC_THREADS) {
+      const int t = i / (DB * 8), d0 = (i % (DB * 8)) * 8;
+      float q[8], k[8];
+      if (t < r.len) {
+        const size_t gr = r.row + t;
+        const float2* cs = a.rope ? a.rope + gr * a.pairs : nullptr;
+        head8(a.q + gr * a.ldp + h * a.dim, d0, a.dim, cs, a.pairs, a.q_scale, vec, q);
+        head8(a.k + gr * a.ldp + h * a.dim, d0, a.dim, cs, a.pairs, a.k_scale, vec, k);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) q[j] = k[j] = 0.f;
       }
-      tc_commit(y.bar);
+      put8_two(sQ, tile_at(t, d0, T), DB * T, q);
+      put8_two(sP, tile_at(t, d0, T), DB * T, k);
     }
+    y.publish();
+    if (tid == 0) score(SC);
     __syncwarp();
-    if (GLA) load_values(a, h, r, sX, VB);                            // (every thread is past its decays)
     y.wait(0x6F7);
 #pragma unroll
     for (int c = 0; c < KW; c += 16) {
@@ -653,35 +849,9 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
 #pragma unroll
       for (int j = 0; j < 16; ++j) {
         const int back = row - (part * KW + c + j);
-        sc[c + j] = back < 0 ? 0.f : __uint_as_float(o[j]) * (GLA ? 1.f : exp2f(l2 * (float)back));
+        sc[c + j] = back < 0 ? 0.f : __uint_as_float(o[j]) * exp2f(l2 * (float)back);
       }
     }
-  } else {
-    // pairwise: the decays between two tokens as the difference of their sums
-    __syncthreads();                                                  // the keys are there
-#pragma unroll
-    for (int j = 0; j < KW; ++j) sc[j] = 0.f;
-    if (part * KW <= (warp & 3) * 32 + 31)                            // warp-uniform: some key is not behind every row of the warp
-      for (int d0 = 0; d0 < a.dim; d0 += 8) {
-        float q[8], x[8];
-        query8<MODE>(a, h, r.row + min(row, r.len - 1), d0, vec, q);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = X[row * DP + d0 + e];
-#pragma unroll
-        for (int j = 0; j < KW; ++j) {
-          const int key = part * KW + j;
-          const uint8_t* at = sP + tile_at(key, d0, T);
-          float k[8], lo[8];
-          load8<bf16>((const bf16*)at, k);
-          load8<bf16>((const bf16*)(at + DB * T), lo);
-#pragma unroll
-          for (int e = 0; e < 8; ++e) sc[j] = fmaf(q[e] * (k[e] + lo[e]), exp2f(x[e] - X[key * DP + d0 + e]), sc[j]);
-        }
-      }
-#pragma unroll
-    for (int j = 0; j < KW; ++j) if (part * KW + j > row || row >= r.len) sc[j] = 0.f;         // (may not be a number)
-    __syncthreads();                                                  // the decays have been read
-    load_values(a, h, r, sX, VB);
   }
   tc_fence_before();
   __syncthreads();                                                    // keys and scores have been read
@@ -699,48 +869,40 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
   }
   __syncwarp();
   y.wait(0x6F8);
-  // the state in front of the chunk takes the place of probabilities and values
+  // the state in front of the chunk takes the place of probabilities and values; its rounding errors arrive under the first two products
   if (tid == 0) {
     const uint32_t bytes = VB * DP * 128;
     const uint8_t* S = a.chunk_tiles + ((size_t)r.ci * a.H + h) * 2 * bytes;
-    mbar_expect_tx(tiles_bar, 2 * bytes);
-    bulk_load_1d(sP, S, bytes, tiles_bar);
-    bulk_load_1d(sX, S + bytes, bytes, tiles_bar);
-    if (!mbar_wait_bounded(tiles_bar, 0, (volatile int*)y.abortp)) ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, 0x6FA);
-    const uint32_t id = dc_idesc(VB * 64, 0, 1), q0 = smem_u32(sQ);
-    for (int part = 0; part < 3; ++part) {
-      const uint32_t qa = q0 + (part == 2 ? DB * T : 0), sb = smem_u32(part == 1 ? sX : sP);
+    for (int part = 0; part < 2; ++part) {
+      mbar_expect_tx(tiles_bar + part, bytes);
+      bulk_load_1d(part ? sX : sP, S + part * bytes, bytes, tiles_bar + part);
+    }
+    const uint32_t id = dc_idesc(VB * 64, 0, 1);
+    for (int part = 0; part < 3; ++part) {                            // value x value, error x value, value x error
+      if (part != 1 && !mbar_wait_bounded(tiles_bar + part / 2, 0, (volatile int*)y.abortp)) ca_dev_fail(a.status, CA_DEV_TIMEOUT_PRODUCER, 0x6FA);
+      const uint32_t qa = q0 + (part == 1 ? DB * T : 0), sb = smem_u32(part == 2 ? sX : sP);
       for (int k = 0; k < DP / 16; ++k) tc_mma_f16(y.tmem + O2, umma_desc_sw128(qa + (k >> 2) * T) + 2 * (k & 3), dc_desc_mn(sb + k * 2048, DP * 128), id, (part | k) ? 1u : 0u);
     }
     tc_commit(y.bar);
   }
   __syncwarp();
-  // the gates arrive under these products: a thread has its token's columns [c_lo, c_hi)
+  // the gates arrive under these products, in the order of the stores: piece i of a thread is eight columns of a row
   const int c_lo = part * VB * PW, c_hi = c_lo + VB * PW;
   const bool vout = ((a.vdim | a.ldp | a.ldo) & 7) == 0 && (((uintptr_t)a.g | (uintptr_t)a.out) & 15) == 0;
-  const size_t gr = r.row + min(row, r.len - 1);
-  const bf16* g = a.g ? a.g + gr * a.ldp + h * a.vdim : nullptr;
-  bf16* dst = a.out + gr * a.ldo + h * a.vdim;
-  constexpr int NG = 4 * PW / 8;
+  constexpr int NG = DC_TOK * 32 / DC_THREADS;
   uint4 gates[NG];
+  if (a.g && vout) {
 #pragma unroll
-  for (int p = 0; p < NG; ++p) {
-    const int c = c_lo + p * 8;
-    if (!g || c >= c_hi || c >= a.vdim) gates[p] = make_uint4(0, 0, 0, 0);
-    else if (vout) gates[p] = __ldg((const uint4*)(g + c));
-    else {
-      bf16 e[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) e[j] = c + j < a.vdim ? g[c + j] : __float2bfloat16(0.f);
-      uint32_t w[4];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) { const bf162 b2 = __halves2bfloat162(e[2 * j], e[2 * j + 1]); w[j] = *(const uint32_t*)&b2; }
-      gates[p] = make_uint4(w[0], w[1], w[2], w[3]);
+    for (int p = 0; p < NG; ++p) {
+      const int t = min((tid + p * DC_THREADS) >> 5, r.len - 1), c = min((tid & 31) * 8, a.vdim - 8);
+      gates[p] = __ldg((const uint4*)(a.g + (size_t)(r.row + t) * a.ldp + h * a.vdim + c));
     }
   }
   y.wait(0x6F9);
-  // output norm and gate
-  const float f2 = GLA ? 1.f : exp2f(l2 * (float)(row + 1));
+  // sum of both shares; its norm; rows through shared memory (nothing else is read there any more), gated and stored in whole lines
+  const float f2 = MODE != DECAY_HEAD ? 1.f : exp2f(l2 * (float)(row + 1));
+  float4* stage = (float4*)sP;
+  const int pitch = VB * 16;
   float ss = 0.f;
   for (int c = c_lo; c < c_hi; c += 16) {
     uint32_t o[16], s[16];
@@ -748,39 +910,44 @@ __global__ void __launch_bounds__(DC_THREADS, 1) chunk_out_kernel(const __grid_c
     tmem_ld_x16(y.tmem + lanes + O2 + c, s);
     tc_wait_ld();
 #pragma unroll
-    for (int j = 0; j < 16; ++j) { const float v = fmaf(f2, __uint_as_float(s[j]), __uint_as_float(o[j])); ss = fmaf(v, v, ss); }       // columns past vdim are zero
+    for (int j = 0; j < 16; j += 4) {
+      float4 v;
+      v.x = fmaf(f2, __uint_as_float(s[j]), __uint_as_float(o[j])); v.y = fmaf(f2, __uint_as_float(s[j + 1]), __uint_as_float(o[j + 1]));
+      v.z = fmaf(f2, __uint_as_float(s[j + 2]), __uint_as_float(o[j + 2])); v.w = fmaf(f2, __uint_as_float(s[j + 3]), __uint_as_float(o[j + 3]));
+      ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);        // columns past vdim are zero
+      stage[row * pitch + stage_col(row, (c + j) / 4)] = v;
+    }
   }
   ssum[part * 128 + row] = ss;
   __syncthreads();
-  ss = 0.f;
+  // a thread has the same columns of NG rows
+  const int c = (tid & 31) * 8;
+  float gains[8];
 #pragma unroll
-  for (int p = 0; p < DC_PARTS; ++p) ss += ssum[p * 128 + row];
-  const float inv = rsqrtf(ss / (float)a.vdim + a.eps) * a.out_scale;
+  for (int j = 0; j < 8; ++j) gains[j] = a.out_scale * (a.norm ? gain[min(c + j, a.vdim - 1)] : 1.f);
 #pragma unroll
-  for (int b = 0; b < NG / 2; ++b) {
-    const int c = c_lo + b * 16;
-    if (c >= c_hi) break;                                             // block-uniform
-    uint32_t o[16], s[16];
-    tmem_ld_x16(y.tmem + lanes + O1 + c, o);
-    tmem_ld_x16(y.tmem + lanes + O2 + c, s);
-    tc_wait_ld();
-    if (row >= r.len) continue;
+  for (int p = 0; p < NG; ++p) {
+    const int t = (tid + p * DC_THREADS) >> 5;
+    if (t >= r.len || c >= a.vdim) break;
+    const float4 u = stage[t * pitch + stage_col(t, c / 4)], w = stage[t * pitch + stage_col(t, c / 4 + 1)];
+    float v[8] = {u.x, u.y, u.z, u.w, w.x, w.y, w.z, w.w}, s = 0.f;
 #pragma unroll
-    for (int p = 0; p < 16; p += 8) {
-      if (c + p >= a.vdim) continue;
-      const bf162* gp = (const bf162*)&gates[b * 2 + p / 8];
-      float v[8];
+    for (int q = 0; q < DC_PARTS; ++q) s += ssum[q * 128 + t];
+    const float inv = rsqrtf(s / (float)a.vdim + a.eps);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const float2 g2 = __bfloat1622float2(gp[j / 2]);
-        const float gv = j & 1 ? g2.y : g2.x;
-        const float x = fmaf(f2, __uint_as_float(s[p + j]), __uint_as_float(o[p + j])) * inv;
-        v[j] = x * (a.norm && c + p + j < a.vdim ? __ldg(a.norm + c + p + j) : 1.f) * (g ? silu_f(gv) : 1.f);
+    for (int j = 0; j < 8; ++j) v[j] *= inv * gains[j];
+    bf16* dst = a.out + (size_t)(r.row + t) * a.ldo + h * a.vdim + c;
+    if (vout) {
+      if (a.g) {
+        const bf162* gp = (const bf162*)&gates[p];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { const float2 g = __bfloat1622float2(gp[j]); v[2 * j] *= silu_f(g.x); v[2 * j + 1] *= silu_f(g.y); }
       }
-      if (vout) store8<bf16>(dst + c + p, v);
-      else
+      store8<bf16>(dst, v);
+    } else {
+      const bf16* g = a.g ? a.g + (size_t)(r.row + t) * a.ldp + h * a.vdim + c : nullptr;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) if (c + p + j < a.vdim) dst[c + p + j] = __float2bfloat16(v[j]);
+      for (int j = 0; j < 8; ++j) if (c + j < a.vdim) dst[j] = __float2bfloat16(g ? v[j] * silu_f(to_f(g[j])) : v[j]);
     }
   }
   if (tid == 0 && (int)blockIdx.y == r.chunks - 1) {                  // no other block of this launch reads the tags
@@ -849,7 +1016,7 @@ static int chunk_launch(const CaDecayScan* c, cudaStream_t s) {
 }
 
 // Whether the chunk kernels take a step's long runs.
-static bool chunkable(const CaDecayScan* c, int f32) { return !f32 && c->chunk_state && c->chunk_decay && c->chunk_tiles && c->dim <= 128 && c->vdim <= 256 && c->max_q_len > DS_GROUP; }
+static bool chunkable(const CaDecayScan* c, int f32) { return !f32 && c->chunk_state && c->chunk_decay && c->chunk_tiles && c->dim <= 128 && c->vdim <= 256 && c->max_q_len > DS_GROUP && (c->decay || !c->pairs); }
 
 extern "C" int cuteafd_decay_scan(const CaDecayScan* c, int f32, cudaStream_t s) {
   CA_REQUIRE(c && c->q && c->k && c->v && (c->g || c->lower) && c->state && c->tags && c->ring && c->state_slot && c->q_start && c->q_len && c->kv_len && c->out, "decay_scan: null argument");

@@ -14,6 +14,7 @@ from ..ops.native import call, ptr, stream
 from .engine import Lane
 
 LANE_CAPS = (16, 32, 64, 256, 1024, 4096, 16384)
+NARROW_WEIGHTS = 36 << 20       # most weights of a product that 33 to 64 rows take in tiles of 32 (a cluster splits K; wider ones read their weights once)
 
 
 class StackLane(Lane):
@@ -49,6 +50,12 @@ class StackLane(Lane):
             self.logits = torch.zeros(rows, self.eng.spec.vocab, dtype=torch.float32, device=self.dev)
             self._head_acts.clear()
             self.eng.drop_graphs()                   # captured steps hold the old addresses
+
+    def retiled(self, act: ActBuffer, tn: int) -> ActBuffer:
+        """The same operand rows in token tiles of `tn` (made in the eager run of a new shape)."""
+        if tn == act.tn or act.kind != KIND_BF16:
+            return act
+        return self.get(("tiles", act.data.data_ptr(), act.K, tn), lambda: ActBuffer(act.kind, act.rows, act.K, tn, act.data, ops.encode_tmap(act.data, tn)))
 
     def head_operand(self, n: int) -> ActBuffer:
         """The head's operand in token tiles that fit the `n` rows it multiplies (a prompt's step has few)."""
@@ -134,6 +141,19 @@ class StackBase:
     def set_input_embeds(self, rows, vals):
         if vals is not None and len(rows):
             raise NotImplementedError("image / audio rows are not wired for layer stacks")
+
+    def _dense(self, w, x_act, y, T, residual=None, w_up=None):
+        """Products that leave most of the machine idle take smaller token tiles than their lane's: of 32 rows, whose clusters split K, in small steps;
+        in prompts as small as it takes for every SM to have one."""
+        if w_up is None and w.kind == KIND_BF16:
+            tn, nt = x_act.tn, -(-w.N // 128)
+            if 32 < T <= 64 and w.N * w.K <= NARROW_WEIGHTS:
+                tn = 32
+            elif T >= 1024:
+                while tn > 32 and nt * -(-T // tn) < self.sm_count:
+                    tn //= 2
+            x_act = self.lane(T).retiled(x_act, tn)
+        super()._dense(w, x_act, y, T, residual=residual, w_up=w_up)
 
     def _splits(self, N, K, T, tn, kind):
         return 1 if kind == KIND_F32 else super()._splits(N, K, T, tn, kind)

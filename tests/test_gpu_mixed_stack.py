@@ -404,15 +404,16 @@ LONG_STEPS = [[(0, 400), (0, 2), (0, 17)], [(400, 3), (2, 300), (17, 128)], [(40
 
 @pytest.mark.parametrize("form", [FP32, SHORT, CHUNKS])
 @pytest.mark.parametrize("H,d,dv,gates", [(3, 24, 40, "mild"), (1, 13, 7, "long"), (2, 128, 256, "mild"), (4, 64, 64, "harsh"), (2, 128, 128, "long"), (3, 9, 17, "harsh"), (2, 256, 64, "mild"),
-                                          (2, 96, 200, "harsh"), (2, 128, 64, "harsh")])
+                                          (2, 96, 200, "harsh"), (2, 128, 64, "harsh"), (2, 128, 64, 0.0), (2, 64, 128, -2.0), (3, 40, 40, -3.0), (2, 128, 256, -5.0), (2, 100, 72, -7.0)])
 def test_hgrn2_across_portions(H, d, dv, gates, form):
     """Gates, recurrence and output norm of every portion equal those of the whole sequence, wherever it is cut and after steps back.  "long": every
-    channel remembers for thousands of tokens; "harsh": channels that forget at once, beside ones that forget nothing, without lower bounds."""
+    channel remembers for thousands of tokens; "harsh": channels that forget at once, beside ones that forget nothing, without lower bounds; a number:
+    gates around it without lower bounds, which take more and more references in a chunk."""
     torch.manual_seed(11)
     f32 = form == FP32
     dt, tol, eps = torch.float32 if f32 else torch.bfloat16, 1e-5 if f32 else 8e-3, 1e-3
     slots, L = [1, 3, 0], 704
-    bias, lower = {"mild": (torch.randn(H * d) * 1.5 + 1.0, torch.rand(H * d) * 0.9), "long": (torch.randn(H * d) * 0.5 + 9.0, torch.zeros(H * d)),
+    bias, lower = (torch.randn(H * d) * 0.3 + gates, torch.zeros(H * d)) if isinstance(gates, float) else {"mild": (torch.randn(H * d) * 1.5 + 1.0, torch.rand(H * d) * 0.9), "long": (torch.randn(H * d) * 0.5 + 9.0, torch.zeros(H * d)),
                    "harsh": (torch.randn(H * d) * 4, torch.zeros(H * d))}[gates]
     if gates == "harsh":
         bias[0], bias[H * d - 1], lower[1] = 40.0, -60.0, 1.0        # forgets nothing and takes nothing; forgets at once; bound at one

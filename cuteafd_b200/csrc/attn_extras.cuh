@@ -4,7 +4,7 @@
 // constant factor.
 //
 // Pooled blocks: block b holds the positions [b P, b P + P).  Its row (laid out like the token rows) is kept in strips of eight blocks, and a strip
-// belongs to the page of its first token: strip s to page s P / 64, as the (s - ceil(64 j / 8 P))-th strip of logical page j.  So pooled rows
+// belongs to the page of its first token: strip s to page s P / 8, as the (s - ceil(8 j / P))-th strip of logical page j.  So pooled rows
 // need no pages of their own, are freed and used again with the tokens' pages, and eight of them are one 1 KB box of a 64-wide chunk whatever P is.
 #pragma once
 #include "stack_rows.cuh"
